@@ -41,6 +41,9 @@ void bind_runtime(py::module_& m) {
         std::vector<int32_t> out; if (!p.allocate(n, out)) return py::none(); return py::cast(out); })
       .def("release", &PagePool::release).def("is_used", &PagePool::is_used);
 
+  py::class_<SlotPool>(m, "SlotPool").def(py::init<int>(), py::arg("num_slots"))
+      .def_property_readonly("total_slots", &SlotPool::total_slots).def_property_readonly("free_slots", &SlotPool::free_slots)
+      .def("allocate", &SlotPool::allocate).def("release", &SlotPool::release);
   py::class_<SeqSpec>(m, "SeqSpec").def(py::init<>())
       .def(py::init([](uint64_t id, std::vector<int32_t> prompt, int max_new, bool ignore_eos, int eos) {
              SeqSpec s; s.id = id; s.prompt = std::move(prompt); s.max_new_tokens = max_new; s.ignore_eos = ignore_eos;
@@ -53,21 +56,24 @@ void bind_runtime(py::module_& m) {
       .def_readwrite("temperature", &SeqSpec::temperature).def_readwrite("top_p", &SeqSpec::top_p)
       .def_readwrite("top_k", &SeqSpec::top_k).def_readwrite("seed", &SeqSpec::seed);
   py::class_<SeqState>(m, "SeqState").def_readonly("spec", &SeqState::spec).def_readonly("generated", &SeqState::generated)
-      .def_readonly("pages", &SeqState::pages).def_readonly("cached_tokens", &SeqState::cached_tokens)
+      .def_readonly("pages", &SeqState::pages).def_readonly("slot", &SeqState::slot)
+      .def_readonly("cached_tokens", &SeqState::cached_tokens)
       .def_property_readonly("finish", [](const SeqState& s) { return static_cast<int>(s.finish); })
       .def("total_len", &SeqState::total_len);
   py::class_<MetaLayout>(m, "MetaLayout").def_static("make", &MetaLayout::make)
       .def_readonly("ids", &MetaLayout::ids).def_readonly("pos", &MetaLayout::pos).def_readonly("slot", &MetaLayout::slot)
       .def_readonly("tok_indptr", &MetaLayout::tok_indptr).def_readonly("page_indptr", &MetaLayout::page_indptr)
-      .def_readonly("last_page_len", &MetaLayout::last_page_len).def_readonly("page_indices", &MetaLayout::page_indices)
+      .def_readonly("last_page_len", &MetaLayout::last_page_len).def_readonly("page_indices", &MetaLayout::page_indices).def_readonly("seq_slot", &MetaLayout::seq_slot)
       .def_readonly("total", &MetaLayout::total);
-  py::class_<Batch>(m, "Batch").def(py::init<uint64_t, PagePool*>(), py::keep_alive<1, 3>())
+  py::class_<Batch>(m, "Batch").def(py::init<uint64_t, PagePool*, SlotPool*>(), py::arg("id"), py::arg("pool"),
+                                      py::arg("slots") = nullptr, py::keep_alive<1, 3>(), py::keep_alive<1, 4>())
       .def_property_readonly("id", &Batch::id).def_property_readonly("size", &Batch::size)
       .def_property_readonly("seqs", &Batch::seqs, py::return_value_policy::reference_internal)
       .def_property("decode", &Batch::is_decode, &Batch::set_decode)
       .def("max_tokens", &Batch::max_tokens).def("num_pages", &Batch::num_pages)
       .def("num_prompt_tokens", &Batch::num_prompt_tokens).def("max_seq_len", &Batch::max_seq_len)
-      .def("add_prompts", &Batch::add_prompts).def("mark_prefilled", &Batch::mark_prefilled)
+      .def("add_prompts", &Batch::add_prompts, py::arg("specs"), py::arg("reserve_next") = true)
+      .def("extend_prompt", &Batch::extend_prompt).def("advance", &Batch::advance).def("mark_prefilled", &Batch::mark_prefilled)
       .def("append_tokens", &Batch::append_tokens, py::arg("tokens"), py::arg("count_cached") = true)
       .def("filter", &Batch::filter).def("unfinished_ids", &Batch::unfinished_ids)
       .def("generated_tail", &Batch::generated_tail).def("finish_request", &Batch::finish_request)
@@ -87,6 +93,13 @@ void bind_runtime(py::module_& m) {
         if (h.size() < L.total) throw std::invalid_argument("staging array too small");
         auto c = b.fill_prefill_chunk(h.mutable_data(), L, tok0, max_tokens);
         return py::make_tuple(c.tokens, c.pages, c.rows, c.first_seq, c.q_lens, c.kv_lens, c.ended); })
+      .def("fill_step", [](const Batch& b, py::array_t<int32_t, py::array::c_style> h, const MetaLayout& L,
+                           const std::vector<int>& counts, int pad_to) {
+        if (h.size() < L.total) throw std::invalid_argument("staging array too small");
+        auto c = b.fill_step(h.mutable_data(), L, counts, pad_to);
+        return py::make_tuple(c.tokens, c.pages, c.rows, c.singles, c.order, c.q_lens, c.kv_lens); })
+      .def("cached_lens", [](const Batch& b) {
+        std::vector<int> v; for (auto& s : b.seqs()) v.push_back(s.cached_tokens); return v; })
       .def("fill_decode", [](const Batch& b, py::array_t<int32_t, py::array::c_style> h, const MetaLayout& L, int pad_to) {
         if (h.size() < L.total) throw std::invalid_argument("staging array too small");
         return b.fill_decode(h.mutable_data(), L, pad_to); });

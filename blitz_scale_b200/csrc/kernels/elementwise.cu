@@ -10,6 +10,7 @@
 #include "common.cuh"
 #include "launch.cuh"
 #include "ptx.cuh"
+#include "scalar.cuh"
 
 namespace blitz {
 
@@ -142,10 +143,9 @@ __global__ void argmax_kernel(const T* __restrict__ logits, int vocab, int64_t s
   float best = -INFINITY;
   int besti = 0x7fffffff;
   const int nvec = vocab >> 3;
-  const uint4* rv = reinterpret_cast<const uint4*>(row);
   for (int i = threadIdx.x; i < nvec; i += blockDim.x) {
     float f[8];
-    unpack8<T>(rv[i], f);
+    ldf8<T>(row + static_cast<int64_t>(i) * 8, f);
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       if (f[j] > best) {
@@ -155,7 +155,7 @@ __global__ void argmax_kernel(const T* __restrict__ logits, int vocab, int64_t s
     }
   }
   for (int i = (nvec << 3) + threadIdx.x; i < vocab; i += blockDim.x) {
-    float v = to_f<T>(row[i]);
+    float v = ldf<T>(row + i);
     if (v > best) {
       best = v;
       besti = i;
@@ -225,10 +225,10 @@ __global__ void sample_kernel(const T* __restrict__ logits, int vocab, int64_t s
   const float pcut = top_p[b] > 0.f ? fminf(top_p[b], 1.f) : 1.f;
 
   float mx = -INFINITY;
-  for (int i = threadIdx.x; i < vocab; i += blockDim.x) mx = fmaxf(mx, to_f<T>(row[i]) * inv_t);
+  for (int i = threadIdx.x; i < vocab; i += blockDim.x) mx = fmaxf(mx, ldf<T>(row + i) * inv_t);
   mx = block_max(mx, red);
   float z = 0.f;
-  for (int i = threadIdx.x; i < vocab; i += blockDim.x) z += __expf(to_f<T>(row[i]) * inv_t - mx);
+  for (int i = threadIdx.x; i < vocab; i += blockDim.x) z += __expf(ldf<T>(row + i) * inv_t - mx);
   z = block_sum(z, red);
 
   // threshold in "weight" space w = exp(l/T - mx) in (0, 1]
@@ -237,7 +237,7 @@ __global__ void sample_kernel(const T* __restrict__ logits, int vocab, int64_t s
     for (int it = 0; it < 30; ++it) {
       const float mid = 0.5f * (lo + hi);
       float cnt = 0.f;
-      for (int i = threadIdx.x; i < vocab; i += blockDim.x) cnt += (__expf(to_f<T>(row[i]) * inv_t - mx) >= mid) ? 1.f : 0.f;
+      for (int i = threadIdx.x; i < vocab; i += blockDim.x) cnt += (__expf(ldf<T>(row + i) * inv_t - mx) >= mid) ? 1.f : 0.f;
       cnt = block_sum(cnt, red);
       if (cnt >= static_cast<float>(k)) lo = mid; else hi = mid;
     }
@@ -249,7 +249,7 @@ __global__ void sample_kernel(const T* __restrict__ logits, int vocab, int64_t s
       const float mid = 0.5f * (lo2 + hi2);
       float mass = 0.f;
       for (int i = threadIdx.x; i < vocab; i += blockDim.x) {
-        float w = __expf(to_f<T>(row[i]) * inv_t - mx);
+        float w = __expf(ldf<T>(row + i) * inv_t - mx);
         mass += w >= mid ? w : 0.f;
       }
       mass = block_sum(mass, red);
@@ -262,7 +262,7 @@ __global__ void sample_kernel(const T* __restrict__ logits, int vocab, int64_t s
   const int beg = threadIdx.x * chunk, end = min(vocab, beg + chunk);
   float local = 0.f;
   for (int i = beg; i < end; ++i) {
-    float w = __expf(to_f<T>(row[i]) * inv_t - mx);
+    float w = __expf(ldf<T>(row + i) * inv_t - mx);
     local += w >= thr_k ? w : 0.f;
   }
   scan[threadIdx.x + 1] = local;
@@ -281,7 +281,7 @@ __global__ void sample_kernel(const T* __restrict__ logits, int vocab, int64_t s
     float acc = scan[threadIdx.x];
     int pick = -1;
     for (int i = beg; i < end; ++i) {
-      float w = __expf(to_f<T>(row[i]) * inv_t - mx);
+      float w = __expf(ldf<T>(row + i) * inv_t - mx);
       if (w >= thr_k) {
         acc += w;
         pick = i;
@@ -296,7 +296,7 @@ __global__ void sample_kernel(const T* __restrict__ logits, int vocab, int64_t s
     if (c < 0) {  // numerical corner: fall back to the arg-max token
       float best = -INFINITY;
       for (int i = 0; i < vocab; ++i) {
-        float v = to_f<T>(row[i]);
+        float v = ldf<T>(row + i);
         if (v > best) { best = v; c = i; }
       }
     }
@@ -454,7 +454,7 @@ int blitz_argmax(const void* logits, int batch, int vocab, int64_t stride, int32
   if (batch <= 0) return 0;
   if (stride & 7) return -1;
   cudaError_t blitz_last = cudaSuccess;
-  BLITZ_DISPATCH_DTYPE(dtype, (blitz_last = launch_pdl(argmax_kernel<T>, dim3(batch), dim3(1024), 0, stream, (const T*)logits, vocab, stride, out_idx,
+  BLITZ_DISPATCH_DTYPE3(dtype, (blitz_last = launch_pdl(argmax_kernel<T>, dim3(batch), dim3(1024), 0, stream, (const T*)logits, vocab, stride, out_idx,
                                                                             out_val, idx_offset)));
   return (int)blitz_last;
 }
@@ -464,7 +464,7 @@ int blitz_sample(const void* logits, int batch, int vocab, int64_t stride, const
                  int dtype, cudaStream_t stream) {
   if (batch <= 0) return 0;
   cudaError_t blitz_last = cudaSuccess;
-  BLITZ_DISPATCH_DTYPE(dtype, (blitz_last = launch_pdl(sample_kernel<T>, dim3(batch), dim3(1024), 0, stream, (const T*)logits, vocab, stride,
+  BLITZ_DISPATCH_DTYPE3(dtype, (blitz_last = launch_pdl(sample_kernel<T>, dim3(batch), dim3(1024), 0, stream, (const T*)logits, vocab, stride,
                                                                             temperature, top_k, top_p, seeds, step,
                                                                             out_idx)));
   return (int)blitz_last;

@@ -53,7 +53,9 @@ constexpr int kPairStagingBytes = 2 * 4 * 4096;  // two buffers of four 32-row x
 constexpr int kPairFinalStagingBytes = kPairSlabsMax * 4 * 4096;  // a pair's last tile: one box per slab and quarter, in the idle stages
 
 struct PairParams {
+  void* C;         // fp32 outputs (the 16-bit ones are stored through tmap_c)
   const void* R;
+  float alpha;     // axpy
   int64_t ldc;
   int M, N, K;
   int bnf;         // UMMA N = accumulator columns of a tile (128 or 256)
@@ -595,6 +597,25 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                     }
                   }
                 }
+                if (EPI == 4 || EPI == 5) {
+                  // fp32 output: a thread's 32 columns are a whole 128-byte line, stored directly
+                  if (row_ok) {
+                    float* dst = reinterpret_cast<float*>(p.C) + static_cast<int64_t>(row) * p.ldc + n0 + c;
+#pragma unroll
+                    for (int jj = 0; jj < 8; ++jj) {
+                      if (n0 + c + 4 * jj < p.N) {
+                        float4 o = make_float4(gt[4 * jj], gt[4 * jj + 1], gt[4 * jj + 2], gt[4 * jj + 3]);
+                        if (EPI == 5) {
+                          const float4 x = *reinterpret_cast<const float4*>(dst + 4 * jj);
+                          o = make_float4(x.x + p.alpha * o.x, x.y + p.alpha * o.y, x.z + p.alpha * o.z, x.w + p.alpha * o.w);
+                        }
+                        *reinterpret_cast<float4*>(dst + 4 * jj) = o;
+                      }
+                    }
+                  }
+                  ++own_idx;
+                  continue;
+                }
                 uint4 o4[4];
                 pair_convert32<T, EPI>(gt, up, rpre[i], o4);
                 // 128-byte rows, 16-byte chunks XOR-swizzled by row: the layout the TMA store expects
@@ -750,11 +771,12 @@ void blitz_gemm_pair_set_trace(unsigned long long* buf) { blitz::g_pair_trace = 
 
 // Whether blitz_gemm_pair takes this problem.
 int blitz_gemm_pair_supported(int M, int N, int K, int b_layout, int epilogue) {
-  return M >= 1 && b_layout == 0 && epilogue >= 0 && epilogue <= 2 && (N & 7) == 0 && (K & 7) == 0 && N >= 64;
+  return M >= 1 && b_layout == 0 && ((epilogue >= 0 && epilogue <= 2) || epilogue == 4 || epilogue == 5) && (N & 7) == 0 && (K & 7) == 0 && N >= 64;
 }
 
 // C = A W (+R | silu-mul).  A [M, lda>=K], W [K, ldb>=columns] row-major, C/R [M, ldc>=N].  dtype 0 fp16, 1 bf16.
-// epilogue 0 store, 1 add R (C may be R), 2 silu(gate)*up with the up columns starting at up_col_off.
+// epilogue 0 store, 1 add R (C may be R), 2 silu(gate)*up with the up columns starting at up_col_off, 4 store with C in
+// fp32, 5 C += alpha * acc with C in fp32.
 // bnf_hint: accumulator columns per tile (0 = choose, 128 or 256); nacc_hint: tiles per pair that share the
 // activation tiles (0 = choose, 1 or 2); upp_hint: units per CTA pair (0 = choose; -n = cut every tile into n
 // equal K parts, one pair each).
@@ -764,7 +786,7 @@ int blitz_gemm_pair_supported(int M, int N, int K, int b_layout, int epilogue) {
 int blitz_gemm_pair(const void* A, int64_t lda, const void* W, int64_t ldb, void* C, int64_t ldc, const void* R, int M,
                     int N, int K, int epilogue, int up_col_off, int dtype, int static_b, int bnf_hint, int nacc_hint,
                     int upp_hint, void* ws, int64_t ws_bytes, unsigned* flags, int num_flags, int* status,
-                    cudaStream_t stream) {
+                    float alpha, cudaStream_t stream) {
   using namespace blitz;
   if (!blitz_gemm_pair_supported(M, N, K, 0, epilogue) || !ws || !flags) return -1;
   if ((lda & 7) || (ldb & 7) || (ldc & 7) || (epilogue == 2 && (up_col_off & 7))) return -1;
@@ -773,6 +795,8 @@ int blitz_gemm_pair(const void* A, int64_t lda, const void* W, int64_t ldb, void
   const int sms = device_sm_count();
   PairParams p;
   p.R = R;
+  p.C = C;
+  p.alpha = alpha;
   p.ldc = ldc;
   p.M = M;
   p.N = N;
@@ -806,14 +830,22 @@ int blitz_gemm_pair(const void* A, int64_t lda, const void* W, int64_t ldb, void
   if (!get_tmap_2d(&ta, A, (uint64_t)K, (uint64_t)M, (uint64_t)lda * 2, kPairBK, kPairRows)) return -2;
   const int w_cols = epilogue == 2 ? up_col_off + N : N;
   if (!get_tmap_2d(&tb, W, (uint64_t)w_cols, (uint64_t)K, (uint64_t)ldb * 2, 64, kPairBK)) return -2;
-  if (!get_tmap_2d(&tc, C, (uint64_t)N, (uint64_t)M, (uint64_t)ldc * 2, 64, 32)) return -2;
+  if (epilogue >= 4) {
+    tc = ta;  // fp32 outputs are stored without TMA; the map is not used
+  } else if (!get_tmap_2d(&tc, C, (uint64_t)N, (uint64_t)M, (uint64_t)ldc * 2, 64, 32)) {
+    return -2;
+  }
 
   if (dtype == 1) {
     return epilogue == 2   ? pair_launch<__nv_bfloat16, 2>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
+           : epilogue == 4 ? pair_launch<__nv_bfloat16, 4>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
+           : epilogue == 5 ? pair_launch<__nv_bfloat16, 5>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
            : epilogue == 1 ? pair_launch<__nv_bfloat16, 1>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
                            : pair_launch<__nv_bfloat16, 0>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream);
   }
   return epilogue == 2   ? pair_launch<__half, 2>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
+           : epilogue == 4 ? pair_launch<__half, 4>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
+           : epilogue == 5 ? pair_launch<__half, 5>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
          : epilogue == 1 ? pair_launch<__half, 1>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
                          : pair_launch<__half, 0>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream);
 }

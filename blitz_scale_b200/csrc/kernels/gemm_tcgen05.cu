@@ -10,6 +10,12 @@
 //   store      C = acc
 //   add        C = acc + R                  (residual add of o_proj / down_proj)
 //   silu_mul   C = silu(acc_gate) * acc_up  (gate||up projection; B holds N gate columns, then N up columns)
+//   store f32  C = acc, C in fp32           (what a recurrence takes in 32 bits)
+//   axpy f32   C += alpha * acc, C in fp32  (output projections of models whose residual stream is fp32)
+//
+// Block-diagonal products (groups > 1): B is `groups` blocks [K,N] stacked along K; group g takes the K columns of A
+// from g * K on and the N columns of C from g * N on.  An N tile belongs to one group and simply starts its K walk there
+// (K is then a multiple of the 64-wide K block, so that no block reaches into a neighbour).
 //
 // Measured on B200: a 128-row tcgen05.mma of K = 16 occupies the tensor pipe for ~95 / 105 / 150 cycles at
 // N = 64 / 128 / 256, so (1) wide tiles are the most efficient per FLOP and (2) the time of a skinny GEMM
@@ -37,7 +43,7 @@ constexpr int kBK = 64;
 constexpr int kGemmThreads = 192;
 constexpr int kMaxSplitK = 16;
 
-enum GemmEpilogue : int { kEpiStore = 0, kEpiAdd = 1, kEpiSiluMul = 2, kEpiPushRS = 3 };
+enum GemmEpilogue : int { kEpiStore = 0, kEpiAdd = 1, kEpiSiluMul = 2, kEpiPushRS = 3, kEpiStoreF32 = 4, kEpiAxpyF32 = 5 };
 
 struct GemmParams {
   void* C;
@@ -65,6 +71,9 @@ struct GemmParams {
   uint32_t wait_value;
   int n_fast;  // tensor-parallel fusion: N runs fastest over the tiles, M blocks start at m_rot (see gemm_tile_blocks)
   int m_rot;
+  float alpha;      // axpy
+  int groups;       // diagonal blocks (1: an ordinary product); N and K are those of one block
+  int group_tiles;  // N tiles per block
 };
 
 // Tile number -> (M block, N block).  Normally M runs fastest.  When the rows of A arrive from other ranks
@@ -85,6 +94,14 @@ __device__ __forceinline__ void gemm_tile_blocks(const GemmParams& p, int tile, 
     mb = tile % p.tiles_m;
     nb = tile / p.tiles_m;
   }
+}
+
+// N block -> (diagonal block, N block within it).
+__device__ __forceinline__ int gemm_group(const GemmParams& p, int& nb) {
+  if (p.groups <= 1) return 0;
+  const int g = nb / p.group_tiles;
+  nb -= g * p.group_tiles;
+  return g;
 }
 
 template <int BN>
@@ -135,7 +152,23 @@ __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)
 // Epilogue of 32 consecutive output columns of one row: acc (and up for silu_mul) -> C.
 template <typename T, int EPI>
 __device__ __forceinline__ void store_chunk(const GemmParams& p, const float (&acc)[32], const float (&up)[32], int row,
-                                            int col0, bool row_ok) {
+                                            int col0, bool row_ok, int group = 0) {
+  if (EPI == kEpiStoreF32 || EPI == kEpiAxpyF32) {
+    if (!row_ok) return;
+    float* dst = reinterpret_cast<float*>(p.C) + static_cast<int64_t>(row) * p.ldc + static_cast<int64_t>(group) * p.N + col0;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      if (col0 + j * 4 < p.N) {
+        float4 v = make_float4(acc[4 * j], acc[4 * j + 1], acc[4 * j + 2], acc[4 * j + 3]);
+        if (EPI == kEpiAxpyF32) {
+          const float4 r = *reinterpret_cast<const float4*>(dst + 4 * j);
+          v = make_float4(r.x + p.alpha * v.x, r.y + p.alpha * v.y, r.z + p.alpha * v.z, r.w + p.alpha * v.w);
+        }
+        *reinterpret_cast<float4*>(dst + 4 * j) = v;
+      }
+    }
+    return;
+  }
   uint32_t out[16];
   if (EPI == kEpiSiluMul) {
 #pragma unroll
@@ -174,7 +207,7 @@ __device__ __forceinline__ void store_chunk(const GemmParams& p, const float (&a
                         make_uint4(out[4 * j], out[4 * j + 1], out[4 * j + 2], out[4 * j + 3]));
       }
     } else {
-      T* dst = reinterpret_cast<T*>(p.C) + static_cast<int64_t>(row) * p.ldc + col0;
+      T* dst = reinterpret_cast<T*>(p.C) + static_cast<int64_t>(row) * p.ldc + static_cast<int64_t>(group) * p.N + col0;
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         if (col0 + j * 8 < p.N)
@@ -271,6 +304,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
         const int tile = w / p.split_k, split = w % p.split_k;
         int mb, nb;
         gemm_tile_blocks(p, tile, mb, nb);
+        const int kb_group = gemm_group(p, nb) * num_kb;  // first K block of the tile's diagonal block
         const int m0 = mb * kBM;
         const int n0 = nb * kOutCols;
         if (p.n_wait > 0) {
@@ -292,8 +326,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
           }
           if (fresh) ptx::fence_proxy_async_all();
         }
-        const int kb_beg = split * p.kb_per_split;
-        const int kb_end = min(num_kb, kb_beg + p.kb_per_split);
+        const int kb_beg = kb_group + split * p.kb_per_split;
+        const int kb_end = min(kb_group + num_kb, kb_beg + p.kb_per_split);
         for (int kb = kb_beg; kb < kb_end; ++kb) {
           if (!ptx::bounded_mbar_wait(&empty_bar[stage], phase ^ 1u, abort_flag)) {
             if (p.status) atomicCAS(p.status, 0, kStatusTimeoutProducer);
@@ -397,6 +431,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
       const int tile = w / p.split_k;
       int mb, nb;
       gemm_tile_blocks(p, tile, mb, nb);
+      const int group = gemm_group(p, nb);
       const int m0 = mb * kBM;
       const int n0 = nb * kOutCols;
       if (!ptx::bounded_mbar_wait(&tfull_bar[acc], acc_phase, abort_flag)) {
@@ -424,7 +459,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
           }
 #pragma unroll
           for (int i = 0; i < 32; ++i) a[i] = __uint_as_float(v[i]);
-          store_chunk<T, EPI>(p, a, u, row, n0 + c, row_ok);
+          store_chunk<T, EPI>(p, a, u, row, n0 + c, row_ok, group);
         }
         ptx::tc_fence_before_sync();
         ptx::mbar_arrive(&tempty_bar[acc]);
@@ -486,7 +521,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
                 }
               }
             }
-            store_chunk<T, EPI>(p, a, u, row, n0 + c, row_ok);
+            store_chunk<T, EPI>(p, a, u, row, n0 + c, row_ok, group);
           }
           if (EPI == kEpiPushRS) push_signal(p, m0, epi_tid);
         }
@@ -535,6 +570,8 @@ static cudaError_t dispatch_epi(int epi, int bn, const CUtensorMap& ta, const CU
   switch (epi) {
     case kEpiAdd: return dispatch_bn<T, B_KMAJOR, kEpiAdd>(bn, ta, tb, p, grid, stream);
     case kEpiSiluMul: return dispatch_bn<T, B_KMAJOR, kEpiSiluMul>(bn, ta, tb, p, grid, stream);
+    case kEpiStoreF32: return dispatch_bn<T, B_KMAJOR, kEpiStoreF32>(bn, ta, tb, p, grid, stream);
+    case kEpiAxpyF32: return dispatch_bn<T, B_KMAJOR, kEpiAxpyF32>(bn, ta, tb, p, grid, stream);
     case kEpiPushRS: return dispatch_bn<T, B_KMAJOR, kEpiPushRS>(bn, ta, tb, p, grid, stream);
     default: return dispatch_bn<T, B_KMAJOR, kEpiStore>(bn, ta, tb, p, grid, stream);
   }
@@ -550,7 +587,8 @@ int64_t blitz_gemm_workspace_bytes(int sms) { return (int64_t)(sms + 16) * blitz
 
 // dtype: 0 = fp16, 1 = bf16.  b_layout: 0 = B is [K, ldb>=Ncols] row-major (weights stored in,out),
 // 1 = B is [Ncols, ldb>=K] row-major.  epilogue: 0 store, 1 add residual R (same pitch as C),
-// 2 silu(gate)*up where B carries N gate columns followed (at column `up_col_off`) by N up columns.
+// 2 silu(gate)*up where B carries N gate columns followed (at column `up_col_off`) by N up columns, 4 store with C in
+// fp32, 5 C += alpha * acc with C in fp32.  groups: number of diagonal blocks (see the top of the file), 1 = none.
 // bn_hint: 0 = 256-wide tiles, else 64/128/256.  split_hint: 0 = choose, 1 = never split, else the
 // number of K splits.  ws / ws_bytes: fp32 scratch for split-K partials, tickets / num_tickets:
 // zeroed uint32 array (both may be null: the GEMM then never splits).
@@ -583,15 +621,18 @@ struct BlitzGemmTp {
 static int gemm_impl(const void* A, int64_t lda, const void* B, int64_t ldb, void* C, int64_t ldc, const void* R, int M,
                      int N, int K, int b_layout, int epilogue, int up_col_off, int dtype, int bn_hint, int split_hint,
                      void* ws, int64_t ws_bytes, unsigned* tickets, int num_tickets, int* status,
-                     const BlitzGemmTp* tpa, cudaStream_t stream) {
+                     const BlitzGemmTp* tpa, float alpha, int groups, cudaStream_t stream) {
   using namespace blitz;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if (groups < 1 || (groups > 1 && ((K % kBK) != 0 || b_layout != 0 || tpa != nullptr ||
+                                    (epilogue != kEpiStore && epilogue != kEpiStoreF32))))
+    return -1;
   if ((N & 7) || (K & 7) || (lda & 7) || (ldb & 7) || (ldc & 7)) return -1;
   if (epilogue == kEpiSiluMul && (up_col_off & 7)) return -1;
   const int sms = device_sm_count();
   // 256-wide tiles are the most efficient per FLOP (a 128xNx16 instruction costs ~95 cycles at N = 64,
   // ~105 at N = 128, ~150 at N = 256); when they would leave SMs idle, 128-wide tiles plus split-K win.
-  const int bn = blitz_gemm_tile_n(M, N, epilogue, bn_hint);
+  const int bn = blitz_gemm_tile_n(M, N * groups, epilogue, bn_hint);
   const int out_cols = epilogue == kEpiSiluMul ? bn / 2 : bn;
   const int b_cols_total = epilogue == kEpiSiluMul ? up_col_off + N : N;
 
@@ -605,7 +646,10 @@ static int gemm_impl(const void* A, int64_t lda, const void* B, int64_t ldb, voi
   p.a_box_rows = M >= kBM ? kBM : ((M + 7) & ~7);
   p.up_col_off = up_col_off;
   p.tiles_m = (M + kBM - 1) / kBM;
-  p.tiles_n = (N + out_cols - 1) / out_cols;
+  p.group_tiles = (N + out_cols - 1) / out_cols;
+  p.tiles_n = p.group_tiles * groups;
+  p.groups = groups;
+  p.alpha = alpha;
   p.status = status;
   p.tp = 1; p.tp_rank = 0; p.rows_per_rank = M; p.wait_flags = nullptr; p.n_wait = 0; p.wait_value = 0; p.m_rot = 0; p.n_fast = 0;
   for (int i = 0; i < 8; ++i) { p.push_base[i] = nullptr; p.push_flags[i] = nullptr; }
@@ -644,10 +688,10 @@ static int gemm_impl(const void* A, int64_t lda, const void* B, int64_t ldb, voi
   p.tickets = tickets;
 
   CUtensorMap ta, tb;
-  if (!get_tmap_2d(&ta, A, (uint64_t)K, (uint64_t)M, (uint64_t)lda * 2, kBK, (uint32_t)p.a_box_rows)) return -2;
+  if (!get_tmap_2d(&ta, A, (uint64_t)K * groups, (uint64_t)M, (uint64_t)lda * 2, kBK, (uint32_t)p.a_box_rows)) return -2;
   bool okb;
   if (b_layout == 0) {
-    okb = get_tmap_2d(&tb, B, (uint64_t)b_cols_total, (uint64_t)K, (uint64_t)ldb * 2, 64, kBK);
+    okb = get_tmap_2d(&tb, B, (uint64_t)b_cols_total, (uint64_t)K * groups, (uint64_t)ldb * 2, 64, kBK);
   } else {
     const uint32_t box_rows = epilogue == kEpiSiluMul ? bn / 2 : bn;
     okb = get_tmap_2d(&tb, B, (uint64_t)K, (uint64_t)b_cols_total, (uint64_t)ldb * 2, kBK, box_rows);
@@ -669,9 +713,11 @@ static int gemm_impl(const void* A, int64_t lda, const void* B, int64_t ldb, voi
 
 int blitz_gemm(const void* A, int64_t lda, const void* B, int64_t ldb, void* C, int64_t ldc, const void* R, int M,
                int N, int K, int b_layout, int epilogue, int up_col_off, int dtype, int bn_hint, int split_hint,
-               void* ws, int64_t ws_bytes, unsigned* tickets, int num_tickets, int* status, cudaStream_t stream) {
+               void* ws, int64_t ws_bytes, unsigned* tickets, int num_tickets, int* status, float alpha, int groups,
+               cudaStream_t stream) {
+  if (epilogue == blitz::kEpiPushRS) return -1;
   return gemm_impl(A, lda, B, ldb, C, ldc, R, M, N, K, b_layout, epilogue, up_col_off, dtype, bn_hint, split_hint, ws,
-                   ws_bytes, tickets, num_tickets, status, nullptr, stream);
+                   ws_bytes, tickets, num_tickets, status, nullptr, alpha, groups, stream);
 }
 
 // Tensor-parallel variant: epilogue 3 pushes the partial result to the owner ranks' staging areas
@@ -682,7 +728,7 @@ int blitz_gemm_tp(const void* A, int64_t lda, const void* B, int64_t ldb, void* 
                   void* ws, int64_t ws_bytes, unsigned* tickets, int num_tickets, int* status, const BlitzGemmTp* tp,
                   cudaStream_t stream) {
   return gemm_impl(A, lda, B, ldb, C, ldc, R, M, N, K, b_layout, epilogue, up_col_off, dtype, bn_hint, split_hint, ws,
-                   ws_bytes, tickets, num_tickets, status, tp, stream);
+                   ws_bytes, tickets, num_tickets, status, tp, 1.f, 1, stream);
 }
 
 }  // extern "C"

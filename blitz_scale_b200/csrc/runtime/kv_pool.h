@@ -58,6 +58,34 @@ class PagePool {
   std::vector<uint8_t> in_use_;
 };
 
+// Slots of the per-sequence state that recurrent layers carry from token to token (one slot id addresses the same slot
+// in every layer's state array).  A sequence holds one slot from admission until it leaves.
+class SlotPool {
+ public:
+  explicit SlotPool(int num_slots) : in_use_(num_slots, 0) {
+    for (int i = num_slots - 1; i >= 0; --i) free_.push_back(i);
+  }
+  int total_slots() const { return static_cast<int>(in_use_.size()); }
+  int free_slots() const { return static_cast<int>(free_.size()); }
+  // -1 when none is free
+  int allocate() {
+    if (free_.empty()) return -1;
+    const int s = free_.back();
+    free_.pop_back();
+    in_use_[s] = 1;
+    return s;
+  }
+  void release(int s) {
+    if (s < 0 || s >= total_slots() || !in_use_[s]) throw std::logic_error("SlotPool: double free or bad slot id");
+    in_use_[s] = 0;
+    free_.push_back(s);
+  }
+
+ private:
+  std::vector<int32_t> free_;
+  std::vector<uint8_t> in_use_;
+};
+
 enum FinishReason : int { kFinishNone = -1, kFinishLength = 0, kFinishEos = 1, kFinishStop = 2 };
 
 struct SeqSpec {
@@ -77,14 +105,15 @@ struct SeqState {
   SeqSpec spec;
   std::vector<int32_t> generated;
   std::vector<int32_t> pages;
-  int cached_tokens = 0;  // tokens whose K/V are in the cache
+  int slot = -1;          // state slot (models with recurrent layers)
+  int cached_tokens = 0;  // tokens whose K/V (and state) are in the cache
   FinishReason finish = kFinishNone;
   int total_len() const { return static_cast<int>(spec.prompt.size() + generated.size()); }
 };
 
 // Offsets (in int32 elements) of the fields of the pinned staging array one step copies to the device.
 struct MetaLayout {
-  int ids = 0, pos = 0, slot = 0, tok_indptr = 0, page_indptr = 0, last_page_len = 0, page_indices = 0, total = 0;
+  int ids = 0, pos = 0, slot = 0, tok_indptr = 0, page_indptr = 0, last_page_len = 0, seq_slot = 0, page_indices = 0, total = 0;
   static MetaLayout make(int max_tokens, int max_batch, int max_pages) {
     MetaLayout m;
     m.ids = 0;
@@ -93,7 +122,8 @@ struct MetaLayout {
     m.tok_indptr = m.slot + max_tokens;
     m.page_indptr = m.tok_indptr + max_batch + 1;
     m.last_page_len = m.page_indptr + max_batch + 1;
-    m.page_indices = m.last_page_len + max_batch;
+    m.seq_slot = m.last_page_len + max_batch;
+    m.page_indices = m.seq_slot + max_batch;
     m.total = m.page_indices + max_pages;
     return m;
   }
@@ -101,7 +131,7 @@ struct MetaLayout {
 
 class Batch {
  public:
-  Batch(uint64_t id, PagePool* pool) : id_(id), pool_(pool) {}
+  Batch(uint64_t id, PagePool* pool, SlotPool* slots = nullptr) : id_(id), pool_(pool), slots_(slots) {}
   ~Batch() { clear(); }
   Batch(const Batch&) = delete;
   Batch& operator=(const Batch&) = delete;
@@ -130,19 +160,38 @@ class Batch {
     return n;
   }
 
-  // Admit prompts: each reserves ceil((len + 1) / page) pages.  All-or-nothing.
-  bool add_prompts(const std::vector<SeqSpec>& specs) {
-    const int ps = pool_->page_size();
+  // Admit prompts: each reserves ceil((len + 1) / page) pages (reserve_next = false: only the prompt's own, for callers
+  // that add further tokens themselves) and, where the model has recurrent layers, a state slot.  All-or-nothing.
+  bool add_prompts(const std::vector<SeqSpec>& specs, bool reserve_next = true) {
+    const int ps = pool_->page_size(), extra = reserve_next ? 1 : 0;
     int need = 0;
-    for (auto& sp : specs) need += (static_cast<int>(sp.prompt.size()) + 1 + ps - 1) / ps;
+    for (auto& sp : specs) need += (static_cast<int>(sp.prompt.size()) + extra + ps - 1) / ps;
     if (need > pool_->free_pages()) return false;
+    if (slots_ && static_cast<int>(specs.size()) > slots_->free_slots()) return false;
     for (auto& sp : specs) {
       SeqState st;
       st.spec = sp;
-      pool_->allocate((static_cast<int>(sp.prompt.size()) + 1 + ps - 1) / ps, st.pages);
+      pool_->allocate((static_cast<int>(sp.prompt.size()) + extra + ps - 1) / ps, st.pages);
+      if (slots_) st.slot = slots_->allocate();
       seqs_.push_back(std::move(st));
     }
     return true;
+  }
+
+  // Append given tokens (not sampled ones) to request `id`, with the pages they need.  False, with nothing changed, if
+  // the pool has too few pages.
+  bool extend_prompt(uint64_t id, const std::vector<int32_t>& tokens) {
+    const int ps = pool_->page_size();
+    for (auto& s : seqs_) {
+      if (s.spec.id != id) continue;
+      if (!s.generated.empty()) throw std::logic_error("extend_prompt: the request has generated tokens");
+      const int need = (static_cast<int>(s.spec.prompt.size() + tokens.size()) + ps - 1) / ps;
+      if (need > static_cast<int>(s.pages.size()) && !pool_->allocate(need - static_cast<int>(s.pages.size()), s.pages))
+        return false;
+      s.spec.prompt.insert(s.spec.prompt.end(), tokens.begin(), tokens.end());
+      return true;
+    }
+    throw std::invalid_argument("extend_prompt: unknown request");
   }
 
   // After a prefill forward: all prompt tokens are cached.
@@ -196,7 +245,7 @@ class Batch {
       if (std::find(keep.begin(), keep.end(), s.spec.id) != keep.end()) {
         kept.push_back(std::move(s));
       } else {
-        pool_->release(s.pages);
+        release(s);
       }
     }
     seqs_ = std::move(kept);
@@ -340,12 +389,12 @@ class Batch {
   }
   // Move the requests of `other` to the end of this batch (page ownership moves too).
   void extend(Batch& other) {
-    if (other.pool_ != pool_) throw std::invalid_argument("extend: different pools");
+    if (other.pool_ != pool_ || other.slots_ != slots_) throw std::invalid_argument("extend: different pools");
     for (auto& s : other.seqs_) seqs_.push_back(std::move(s));
     other.seqs_.clear();
   }
   void clear() {
-    for (auto& s : seqs_) pool_->release(s.pages);
+    for (auto& s : seqs_) release(s);
     seqs_.clear();
   }
 
@@ -371,6 +420,7 @@ class Batch {
       h[L.tok_indptr + b + 1] = t;
       h[L.page_indptr + b + 1] = np;
       h[L.last_page_len + b] = n ? n - (used - 1) * ps : 0;
+      h[L.seq_slot + b] = s.slot;
     }
     return {t, np};
   }
@@ -409,6 +459,7 @@ class Batch {
       h[L.tok_indptr + c.rows + 1] = c.tokens;
       h[L.page_indptr + c.rows + 1] = c.pages;
       h[L.last_page_len + c.rows] = static_cast<int32_t>(hi - static_cast<int64_t>(used - 1) * ps);
+      h[L.seq_slot + c.rows] = s.slot;
       c.q_lens.push_back(static_cast<int>(hi - lo));
       c.kv_lens.push_back(static_cast<int>(hi));
       c.ended.push_back(hi == n ? 1 : 0);
@@ -434,6 +485,7 @@ class Batch {
         h[L.slot + b] = -1;
         h[L.page_indptr + b + 1] = np;
         h[L.last_page_len + b] = 0;
+        h[L.seq_slot + b] = -1;
         continue;
       }
       h[L.ids + b] = s.generated.empty() ? s.spec.prompt.back() : s.generated.back();
@@ -444,15 +496,62 @@ class Batch {
       np += used;
       h[L.page_indptr + b + 1] = np;
       h[L.last_page_len + b] = n + 1 - (used - 1) * ps;
+      h[L.seq_slot + b] = s.slot;
     }
-    for (int b = B; b < pad_to; ++b) {
-      h[L.ids + b] = 0;
-      h[L.pos + b] = 0;
-      h[L.slot + b] = -1;
-      h[L.page_indptr + b + 1] = np;
-      h[L.last_page_len + b] = 0;
-    }
+    pad_rows(h, L, B, pad_to, np);
     return np;
+  }
+  // One step over any mixture of the batch's requests: counts[i] tokens of request i, from the first one that is not
+  // cached yet (0: the request sits this step out).  Rows with one token come first, so that the decode kernels can
+  // take rows [0, singles) and the prefill kernels the rest; `order` gives the request of every row.  Positions,
+  // page lists and lengths are those after the step.  pad_to: rows of padding behind a step of single tokens only.
+  struct StepRows {
+    int tokens = 0, pages = 0, rows = 0, singles = 0;
+    std::vector<int> order, q_lens, kv_lens;
+  };
+  StepRows fill_step(int32_t* h, const MetaLayout& L, const std::vector<int>& counts, int pad_to) const {
+    if (counts.size() != seqs_.size()) throw std::invalid_argument("fill_step: one count per request");
+    const int ps = pool_->page_size();
+    StepRows c;
+    h[L.tok_indptr] = 0;
+    h[L.page_indptr] = 0;
+    for (int pass = 0; pass < 2; ++pass) {
+      for (size_t b = 0; b < seqs_.size(); ++b) {
+        const int n = counts[b];
+        if (n <= 0 || (n == 1) != (pass == 0)) continue;
+        const auto& s = seqs_[b];
+        const int lo = s.cached_tokens, hi = lo + n;
+        const int used = (hi + ps - 1) / ps;
+        if (hi > s.total_len() || used > static_cast<int>(s.pages.size()))
+          throw std::invalid_argument("fill_step: more tokens than the request has");
+        const int np = static_cast<int>(s.spec.prompt.size());
+        for (int i = lo; i < hi; ++i) {
+          const int t = c.tokens + (i - lo);
+          h[L.ids + t] = i < np ? s.spec.prompt[i] : s.generated[i - np];
+          h[L.pos + t] = i;
+          h[L.slot + t] = s.pages[i / ps] * ps + i % ps;
+        }
+        c.tokens += n;
+        for (int i = 0; i < used; ++i) h[L.page_indices + c.pages + i] = s.pages[i];
+        c.pages += used;
+        h[L.tok_indptr + c.rows + 1] = c.tokens;
+        h[L.page_indptr + c.rows + 1] = c.pages;
+        h[L.last_page_len + c.rows] = hi - (used - 1) * ps;
+        h[L.seq_slot + c.rows] = s.slot;
+        c.order.push_back(static_cast<int>(b));
+        c.q_lens.push_back(n);
+        c.kv_lens.push_back(hi);
+        c.rows += 1;
+        c.singles += pass == 0;
+      }
+    }
+    if (c.singles == c.rows) pad_rows(h, L, c.rows, pad_to, c.pages);
+    return c;
+  }
+  // After such a step: its tokens are cached.
+  void advance(const std::vector<int>& counts) {
+    if (counts.size() != seqs_.size()) throw std::invalid_argument("advance: one count per request");
+    for (size_t b = 0; b < seqs_.size(); ++b) seqs_[b].cached_tokens += counts[b];
   }
   int max_seq_len() const {
     int m = 0;
@@ -463,8 +562,23 @@ class Batch {
   std::vector<SeqState>& mutable_seqs() { return seqs_; }
 
  private:
+  static void pad_rows(int32_t* h, const MetaLayout& L, int from, int pad_to, int np) {
+    for (int b = from; b < pad_to; ++b) {
+      h[L.ids + b] = 0;
+      h[L.pos + b] = 0;
+      h[L.slot + b] = -1;
+      h[L.page_indptr + b + 1] = np;
+      h[L.last_page_len + b] = 0;
+      h[L.seq_slot + b] = -1;
+    }
+  }
+  void release(SeqState& s) {
+    pool_->release(s.pages);
+    if (slots_ && s.slot >= 0) slots_->release(s.slot);
+  }
   uint64_t id_;
   PagePool* pool_;
+  SlotPool* slots_;
   std::vector<SeqState> seqs_;
   bool decode_ = false;
 };

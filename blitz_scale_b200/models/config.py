@@ -3,8 +3,9 @@
 The registry mirrors the shapes the reference serves (src/model/common_hyper.h:11-177:
 OPT, Llama-2 7B/13B/70B, Llama-3 8B, Mistral 13B/24B, Qwen 72B) plus the tiny shapes used by
 the CPU plumbing configuration and the GPU unit tests.  Only the Llama architecture (pre-RMSNorm,
-RoPE, GQA, SwiGLU, no biases) is executed, as in the reference, where every served model goes
-through the Llama hyper-parameter constructor.
+RoPE, GQA, SwiGLU, no biases) is executed from these records, as in the reference, where every served
+model goes through the Llama hyper-parameter constructor.  Models whose layers differ have records of
+their own (hybrid_config.py); `get_config` finds both, and reads checkpoint folders.
 
 Weight segment (one contiguous allocation per GPU = per TP rank, every matrix stored ``[in, out]``
 row-major, cf. src/model/llama.h:139-218 and scripts/util/make_dangertensors.py:9-30)::
@@ -43,6 +44,8 @@ class ModelConfig:
     param_gb: float = 0.0  # size used for flow accounting by the router
     eos_token: int = -1    # end-of-sequence id of the family's tokenizer (-1: none known); workers stop a request there
                            # unless it sets ignore_eos_token
+    family = "llama"       # which runner executes it (hybrid_config.HybridConfig has "hybrid")
+    recurrent = False      # no per-sequence state beside the KV cache
 
     def kv_bytes_per_token(self, tp: int = 1, elem: int = 2) -> int:
         return 2 * (self.kv_heads // tp) * self.head_dim * elem * self.layers
@@ -80,11 +83,49 @@ REGISTRY: Dict[str, ModelConfig] = {c.name: c for c in [
 ]}
 
 
-def get_config(name: str) -> ModelConfig:
-    try:
+def hybrid_registry():
+    """Shapes of the models whose layers differ (a separate table: the native twin of the registry holds the uniform ones)."""
+    from .fafudra import shape_config
+    mixed = ("gla", "attention", "rglru", "gla")
+    return {c.name: c for c in [
+        # small shapes for tests: one with the sizes the tensor-core kernels take, one with sizes that none of them take
+        shape_config("fafudra_tiny", 2048, 256, mixed, 512, heads=4, kv_heads=2, dim=64, window=96, gla_heads=4, gla_dim=32,
+                     gla_vdim=64, width=256, blocks=4, loop=(1, 3, 2)),
+        shape_config("fafudra_odd", 1003, 120, mixed, 100, heads=6, kv_heads=2, dim=20, window=50, gla_heads=3, gla_dim=12,
+                     gla_vdim=20, rank=5, width=90, blocks=3, loop=(0, 2, 2)),
+        # layer sizes of the 8 B Llama shape
+        shape_config("fafudra_8b", 128256, 4096, mixed * 8, 14336, heads=32, kv_heads=8, dim=128, window=2048,
+                     gla_heads=16, gla_dim=128, gla_vdim=256, width=4096, blocks=16, gb=16),
+    ]}
+
+
+def config_from_dir(path):
+    """Configuration of a checkpoint folder whose config.json names an architecture this package describes by data."""
+    import json
+    from pathlib import Path
+    from . import fafudra
+    from .convert import list_checkpoint
+    d = Path(path)
+    c = json.loads((d / "config.json").read_text())
+    parsers = {fafudra.ARCHITECTURE: fafudra.parse_config}
+    arch = c.get("architecture")
+    if arch not in parsers:
+        raise KeyError(f"{d / 'config.json'}: unknown architecture {arch!r}; known: {sorted(parsers)}")
+    shapes = {n: shape for n, _, shape in list_checkpoint(d)}
+    return parsers[arch](c, shapes, name=d.resolve().name)
+
+
+def get_config(name: str):
+    """A model by registry name, or by the path of a checkpoint folder with a config.json."""
+    import os
+    if name in REGISTRY:
         return REGISTRY[name]
-    except KeyError:
-        raise KeyError(f"unknown model {name!r}; known: {sorted(REGISTRY)}") from None
+    hybrid = hybrid_registry()
+    if name in hybrid:
+        return hybrid[name]
+    if os.path.isfile(os.path.join(str(name), "config.json")):
+        return config_from_dir(name)
+    raise KeyError(f"unknown model {name!r}; known: {sorted(REGISTRY) + sorted(hybrid)}, or a folder with config.json")
 
 
 @dataclass
@@ -129,6 +170,9 @@ def layer_tensor_shapes(cfg: ModelConfig, tp: int) -> List[Tuple[str, Tuple[int,
 
 
 def build_layout(cfg: ModelConfig, tp: int = 1, elem_bytes: int = 2) -> SegmentLayout:
+    if cfg.family == "hybrid":
+        from .hybrid_config import build_hybrid_layout
+        return build_hybrid_layout(cfg, tp, elem_bytes)
     if cfg.q_heads % tp or cfg.kv_heads % tp or cfg.inter % tp or cfg.vocab % tp:
         raise ValueError(f"{cfg.name}: heads/inter/vocab not divisible by tp={tp}")
     lay = SegmentLayout(cfg, tp, elem_bytes)

@@ -131,9 +131,17 @@ def segment_to_hf(seg: WeightSegment) -> Dict[str, torch.Tensor]:
     return out
 
 
+def checkpoint_to_segment(reader: CheckpointReader, cfg, dtype=torch.bfloat16) -> WeightSegment:
+    """Full (tp=1) segment on the host, by the naming scheme of the configuration's design."""
+    if cfg.family == "hybrid":
+        from .fafudra import to_segment
+        return to_segment(reader, cfg, dtype)
+    return hf_to_segment(reader, cfg, dtype)
+
+
 def convert(src, model: str, out_dir, tp: int = 1, dtype=torch.bfloat16) -> List[Path]:
     cfg = get_config(model)
-    full = hf_to_segment(CheckpointReader(src), cfg, dtype)
+    full = checkpoint_to_segment(CheckpointReader(src), cfg, dtype)
     paths = []
     for r in range(tp):
         shard = full if tp == 1 else shard_from_full(full, tp, r, device="cpu")
@@ -155,7 +163,7 @@ def verify(src, model: str, out_dir, tp: int = 1, dtype=torch.bfloat16) -> List[
     """Re-read the segment files under `out_dir` and compare every tensor of every TP rank with what the source
     checkpoint says it should be (the reference's check_dangertensors helper).  Returns the list of problems."""
     cfg = get_config(model)
-    full = hf_to_segment(CheckpointReader(src), cfg, dtype)
+    full = checkpoint_to_segment(CheckpointReader(src), cfg, dtype)
     problems = []
     d = Path(out_dir) / (f"tp{tp}" if tp > 1 else "")
     for r in range(tp):
@@ -181,10 +189,11 @@ def verify(src, model: str, out_dir, tp: int = 1, dtype=torch.bfloat16) -> List[
 def main(argv: Optional[Iterable[str]] = None) -> int:
     ap = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
     ap.add_argument("--src", required=True, help="directory of .safetensors shards, or one file")
-    ap.add_argument("--model", default="", help="registry name (llama3_8b, llama2_7b, mistral_24b, ...)")
+    ap.add_argument("--model", default="", help="registry name (llama3_8b, llama2_7b, mistral_24b, ...) or, for a "
+                    "checkpoint with a config.json of a design this package describes by data, its folder")
     ap.add_argument("--out", default="")
     ap.add_argument("--tp", type=int, default=1)
-    ap.add_argument("--dtype", default="bf16", choices=["bf16", "fp16"])
+    ap.add_argument("--dtype", default="bf16", choices=["bf16", "fp16", "fp32"])
     ap.add_argument("--list", action="store_true", help="only list the tensors of the source checkpoint")
     ap.add_argument("--verify", action="store_true", help="do not write: compare the segment files under --out with the source")
     a = ap.parse_args(argv)
@@ -194,7 +203,7 @@ def main(argv: Optional[Iterable[str]] = None) -> int:
         return 0
     if not a.model or not a.out:
         ap.error("--model and --out are required")
-    dt = torch.bfloat16 if a.dtype == "bf16" else torch.float16
+    dt = {"bf16": torch.bfloat16, "fp16": torch.float16, "fp32": torch.float32}[a.dtype]
     if a.verify:
         problems = verify(a.src, a.model, a.out, a.tp, dt)
         for p in problems:

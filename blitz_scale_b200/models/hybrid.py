@@ -1,0 +1,164 @@
+"""Forward pass of hybrid models (hybrid_config.py) over the weight segment, the paged KV pools and the state slots.
+
+Every layer run is: one norm (with whatever is added to the stream before it), one product for all projections of the
+mixer, the mixer's own kernels, one product for gate and up with SiLU * mul in its epilogue, and one product that adds
+``m * (mixer + feed-forward)`` to the fp32 stream in its epilogue::
+
+    stream_norm -> GEMM (in) -> mixer -> GEMM (gate||up, SiLU*mul) -> GEMM (out, fp32 axpy)
+
+    attention: rope_store (rotation, paged write) -> attention over the pages
+    gla:       one kernel (decay projection, recurrence, output norm, gate), or the chunked kernels for prompts
+    rglru:     conv_causal -> block-diagonal GEMM (gates, fp32 out) -> rglru_scan
+
+A step may hold rows of any length (StepMeta.singles of one token first): single tokens go to the decode kernels, the
+others to the prefill kernels, everything else runs over all tokens at once.
+"""
+from __future__ import annotations
+
+from typing import Dict, List, Optional
+
+import torch
+
+from .. import ops
+from ..runtime.hybrid_cache import HybridCache
+from .hybrid_config import AttentionMixer, GLAMixer, HybridConfig, LayerSpec, RGLRUMixer
+from .llama import StepMeta
+from .weights import WeightSegment
+
+
+class HybridRunner:
+    def __init__(self, seg: WeightSegment, cache: HybridCache, max_tokens: int, max_batch: int):
+        cfg: HybridConfig = seg.cfg
+        self.cfg, self.seg, self.cache = cfg, seg, cache
+        self.runs = cfg.runs()
+        self.page_size = cache.page_size
+        self.max_tokens, self.max_batch = max_tokens, max_batch
+        dev, dt = seg.buffer.device, seg.dtype
+        H = cfg.hidden
+        self.res = torch.empty(max_tokens, H, dtype=torch.float32, device=dev)      # residual stream
+        self.normed = torch.empty(max_tokens, H, dtype=dt, device=dev)
+        self._proj = torch.empty(max_tokens * max(s.in_columns()[1] for s in cfg.layer_specs), dtype=dt, device=dev)
+        # mixer output and feed-forward activation side by side, one buffer per column layout: its padding columns stay
+        # zero because nothing ever writes them
+        self._mid: Dict[tuple, torch.Tensor] = {}
+        for s in cfg.layer_specs:
+            key = self._mid_key(s)
+            if key not in self._mid:
+                self._mid[key] = torch.zeros(max_tokens, s.out_rows, dtype=dt, device=dev)
+        rw = max((m.width for m in cfg.run_mixers() if m.kind == "rglru"), default=0)
+        self._conv = torch.empty(max_tokens * rw, dtype=dt, device=dev) if rw else None
+        self._gates = torch.empty(max_tokens * 2 * rw, dtype=torch.float32, device=dev) if rw else None
+        self.last = torch.empty(max_batch, H, dtype=torch.float32, device=dev)
+        self._logits_pad = torch.zeros(max_batch, cfg.vocab_pad, dtype=torch.float32, device=dev)
+        self.logits = self._logits_pad[:, :cfg.vocab]
+        self.tokens = torch.empty(max_batch, dtype=torch.int32, device=dev)
+        self._freqs = {}
+        for m in cfg.run_mixers():
+            if m.kind == "attention" and (m.rot_dims, m.rot_base) not in self._freqs:
+                self._freqs[(m.rot_dims, m.rot_base)] = ops.rope_freqs(m.rot_dims, m.rot_base, dev)
+        self._ws: Optional[torch.Tensor] = None
+
+    @staticmethod
+    def _mid_key(s: LayerSpec) -> tuple:
+        return (s.mixer.out_width, s.ff)
+
+    def _w(self, l: int, name: str) -> torch.Tensor:
+        return self.seg[f"layers.{l}.{name}"]
+
+    # ------------------------------------------------------------------ pieces
+    def embed(self, m: StepMeta) -> None:
+        """Nothing: the first layer run's norm kernel starts the stream from the embedding table."""
+
+    def run_layer(self, r: int, m: StepMeta) -> None:
+        """Layer run `r` (an index into the executions of a pass, not a layer number)."""
+        run, T, c = self.runs[r], m.num_tokens, self.cfg
+        l = run.layer
+        spec = c.layer_specs[l]
+        step = self.seg["loop_step"][run.step] if run.step >= 0 else None
+        h = self.normed[:T]
+        needs_ids = r == 0 or run.add_embed
+        ops.stream_norm(self.res[:T], self._w(l, "norm1"), c.rms_eps, h, w_offset=1.0, ids=m.ids if needs_ids else None,
+                        embed=self.seg["embed"] if needs_ids else None, init=r == 0, add_embed=run.add_embed, step=step)
+        cols, width = spec.in_columns()
+        proj = self._proj[:T * width].view(T, width)
+        ops.gemm(h, self._w(l, "in"), out=proj, static_b=True)
+        mid = self._mid[self._mid_key(spec)][:T]
+        parts = {n: proj[:, at:at + w] for n, (at, w) in cols.items()}
+        getattr(self, "_" + spec.mixer.kind)(r, l, spec.mixer, parts, mid, m)
+        if spec.ff:
+            ops.gemm(h, self._w(l, "gate_up"), out=mid[:, spec.mix_rows:], epilogue="silu_mul", static_b=True)
+        ops.gemm(mid, self._w(l, "out"), out=self.res[:T], epilogue="axpy", alpha=c.residual_mult, static_b=True)
+
+    def _attention(self, r: int, l: int, mx: AttentionMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta) -> None:
+        T, kv = m.num_tokens, self.cache.runs[r].kv
+        ops.rope_store(p["q"], p["k"], p.get("v"), m.pos, m.slot, kv, self._freqs[(mx.rot_dims, mx.rot_base)],
+                       q_heads=mx.heads, kv_heads=mx.kv_heads, dim=mx.dim, rot_dims=mx.rot_dims, page_size=self.page_size,
+                       interleaved=mx.interleaved)
+        ops.attn_ragged(p["q"], kv, m.pos, m.tok_indptr if m.is_prefill else None, m.page_indptr, m.page_indices, mid,
+                        q_heads=mx.heads, kv_heads=mx.kv_heads, dim=mx.dim, page_size=self.page_size, scale=mx.scale,
+                        window=mx.window, keep_first=mx.keep_first, softcap=mx.softcap,
+                        sink=self._w(l, "sink") if mx.sink else None)
+
+    def _gla(self, r: int, l: int, mx: GLAMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta) -> None:
+        ns = m.batch if not m.is_prefill else m.singles
+        args = dict(rank=mx.rank, tau=mx.tau, eps=self.cfg.rms_eps)
+        w = [self._w(l, n) for n in ("a2", "a2_b", "o_norm")]
+        parts = [p[n] for n in ("q", "k", "v", "g", "low")]
+        state = self.cache.runs[r].state
+        if ns:
+            ops.gla_recurrent(*parts, *w, state, mid, m.pos, None, m.seq_slot[:ns], **args)
+        if m.batch > ns:
+            ops.gla_recurrent(*parts, *w, state, mid, m.pos, m.tok_indptr[ns:], m.seq_slot[ns:], **args)
+
+    def _rglru(self, r: int, l: int, mx: RGLRUMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta) -> None:
+        T, rc = m.num_tokens, self.cache.runs[r]
+        u = self._conv[:T * mx.width].view(T, mx.width)
+        gates = self._gates[:T * 2 * mx.width].view(T, 2 * mx.width)
+        indptr = m.tok_indptr if m.is_prefill else None
+        ops.conv_causal(p["x"], self._w(l, "x_b"), self._w(l, "conv"), self._w(l, "conv_b"), rc.hist, u, m.pos, indptr, m.seq_slot)
+        ops.gemm(u, self._w(l, "gates"), out=gates, groups=mx.blocks, static_b=True)
+        ops.rglru_scan(u, gates, self._w(l, "gate_b"), self._w(l, "lam"), p["y"], p["x"], self._w(l, "y_b"), rc.state, rc.hist,
+                       mid, m.pos, indptr, m.seq_slot, block=mx.block)
+
+    # ------------------------------------------------------------------ head
+    def logits_of(self, n: int, rows: Optional[torch.Tensor] = None, row_offset: int = 0) -> torch.Tensor:
+        """fp32 logits of `n` rows of the stream: rows 0 .. n - 1, or `rows` (+ row_offset)."""
+        ops.stream_norm(self.res, self.seg["final_norm"], self.cfg.rms_eps, self.normed[:n], w_offset=1.0, rows=rows,
+                        row_offset=row_offset, num_tokens=n)
+        ops.gemm(self.normed[:n], self.seg["lm_head"], out=self._logits_pad[:n], static_b=True)
+        return self.logits[:n]
+
+    def head(self, m: StepMeta) -> torch.Tensor:
+        B = m.batch
+        if m.is_prefill:
+            self.logits_of(B, m.tok_indptr[1:], -1)
+        else:
+            self.logits_of(B)
+        ops.argmax(self.logits[:B], out=self.tokens[:B])
+        return self.tokens[:B]
+
+    def last_rows(self, m: StepMeta) -> torch.Tensor:
+        """[batch, hidden]: the stream at the last row of every sequence of a prefill pass."""
+        return torch.index_select(self.res, 0, m.tok_indptr[1:] - 1, out=self.last[:m.batch])
+
+    def head_from_rows(self, rows: torch.Tensor) -> torch.Tensor:
+        """First tokens from rows collected with `last_rows` over several passes."""
+        B = rows.shape[0]
+        self.res[:B].copy_(rows)
+        return self.head(StepMeta(ids=None, pos=None, slot=None, page_indices=None, page_indptr=None, last_page_len=None,
+                                  is_prefill=False, batch=B, num_tokens=B))
+
+    def forward(self, m: StepMeta, lo: int = 0, hi: Optional[int] = None, with_embed: bool = True, with_head: bool = True,
+                after_layer=None) -> Optional[torch.Tensor]:
+        """Layer runs lo .. hi - 1; `after_layer(r)` is called once run r's kernels are in the stream."""
+        for r in range(lo, len(self.runs) if hi is None else hi):
+            self.run_layer(r, m)
+            if after_layer is not None:
+                after_layer(r)
+        return self.head(m) if with_head else None
+
+    def decode_launches(self) -> int:
+        """Kernels of this library in one decode step."""
+        per = {"attention": 2, "gla": 1, "rglru": 3}
+        n = sum(3 + per[self.cfg.layer_specs[r.layer].mixer.kind] + bool(self.cfg.layer_specs[r.layer].ff) for r in self.runs)
+        return n + 3      # final norm, head product, arg-max

@@ -46,6 +46,8 @@ class StepMeta:
     batch: int = 0
     num_tokens: int = 0
     num_splits: int = 1
+    seq_slot: Optional[torch.Tensor] = None                 # [B] state slot of every row (-1: padding row)
+    singles: int = 0                                        # of a ragged step: leading rows with one token
 
 
 class TPComm:
@@ -195,6 +197,13 @@ class LlamaRunner:
             best = vals.argmax(0, keepdim=True)
             self.tokens[:B].copy_(idxs.gather(0, best)[0])
         return self.tokens[:B]
+
+    def logits_of(self, n: int, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Logits of `n` rows of the residual stream (the first n, or `rows`); one GPU."""
+        src = self.res[:n] if rows is None else self.res.index_select(0, rows)
+        ops.rms_norm(src, self.seg["final_norm"], self.cfg.rms_eps, out=self.normed[:n])
+        ops.gemm(self.normed[:n], self.seg["lm_head"], static_b=True, out=self.logits[:n])
+        return self.logits[:n]
 
     def forward(self, m: StepMeta, lo: int = 0, hi: Optional[int] = None, with_embed: bool = True,
                 with_head: bool = True, after_layer=None) -> Optional[torch.Tensor]:

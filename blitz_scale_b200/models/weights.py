@@ -52,6 +52,8 @@ class WeightSegment:
         """Deterministic random weights with activations of order one (norm gains near 1, matrices ~ N(0, 1/in))."""
         gen = torch.Generator(device="cpu").manual_seed(seed * 1000003 + self.tp_rank)
         shared = torch.Generator(device="cpu").manual_seed(seed * 1000003 + 7919)   # replicated tensors: same on every rank
+        if self.cfg.family == "hybrid":
+            return self._hybrid_init(lambda shape: torch.randn(shape, generator=gen))
         for name, v in self._views.items():
             if v.dim() == 1:
                 val = 1.0 + 0.05 * torch.randn(v.shape, generator=shared)
@@ -67,6 +69,8 @@ class WeightSegment:
         gen = torch.Generator(device=self.buffer.device).manual_seed(seed * 1000003 + self.tp_rank)
         # norm gains are replicated across the TP ranks of a replica: they must not depend on the rank
         shared = torch.Generator(device=self.buffer.device).manual_seed(seed * 1000003 + 7919)
+        if self.cfg.family == "hybrid":
+            return self._hybrid_init(lambda shape: torch.randn(shape, generator=gen, device=self.buffer.device))
         for name, v in self._views.items():
             if v.dim() == 1:
                 v.copy_((1.0 + 0.05 * torch.randn(v.shape, generator=shared, device=v.device)).to(self.dtype))
@@ -76,6 +80,14 @@ class WeightSegment:
                 for r0 in range(0, v.shape[0], rows):
                     blk = v[r0:r0 + rows]
                     blk.copy_((torch.randn(blk.shape, generator=gen, device=v.device) * scale).to(self.dtype))
+        return self
+
+    def _hybrid_init(self, rand) -> "WeightSegment":
+        for name, v in self._views.items():
+            if name != "lm_head":
+                self.cfg.init_(name, v, rand)
+        self._views["lm_head"][:, :self.cfg.vocab].copy_(self._views["embed"].t())      # tied
+        self.cfg.zero_padding_(self._views)
         return self
 
     def save(self, directory) -> Path:

@@ -16,6 +16,7 @@ import torch
 from ._lib import lib, available, KernelLibraryMissing  # noqa: F401
 
 _DT = {torch.float16: 0, torch.bfloat16: 1}
+_DT3 = {torch.float16: 0, torch.bfloat16: 1, torch.float32: 2}
 _status = {}
 
 
@@ -24,6 +25,14 @@ def _dt(t: torch.Tensor) -> int:
         return _DT[t.dtype]
     except KeyError:
         raise TypeError(f"kernels take fp16/bf16 tensors, got {t.dtype}") from None
+
+
+def _dt3(t: torch.Tensor) -> int:
+    """Element type of kernels that also run in fp32."""
+    try:
+        return _DT3[t.dtype]
+    except KeyError:
+        raise TypeError(f"kernel takes fp16/bf16/fp32 tensors, got {t.dtype}") from None
 
 
 def _stream() -> ctypes.c_void_p:
@@ -68,7 +77,8 @@ def check_status(device=None, reset: bool = True) -> int:
 
 
 # ---------------------------------------------------------------------------------------------- GEMM
-_EPI = {"store": 0, "add": 1, "silu_mul": 2}
+_EPI = {"store": 0, "add": 1, "silu_mul": 2, "axpy": 5}
+_EPI_STORE_F32 = 4
 
 
 _gemm_ws = {}
@@ -102,8 +112,14 @@ def pair_gemm_workspace(device=None):
     return _pair_ws[key]
 
 
+def _tensor_core_operands(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, N: int, K: int) -> bool:
+    """Sizes, pitches and base addresses the TMA-fed kernels need (16-byte rows and bases)."""
+    return (N % 8 == 0 and K % 8 == 0 and a.stride(0) % 8 == 0 and b.stride(0) % 8 == 0 and out.stride(0) % 8 == 0
+            and a.data_ptr() % 16 == 0 and b.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0)
+
+
 def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *, residual=None,
-         epilogue: str = "store", b_layout: str = "kn", bn: int = 0, split_k: int = 0, static_b: bool = False,
+         epilogue: str = "store", alpha: float = 1.0, groups: int = 1, b_layout: str = "kn", bn: int = 0, split_k: int = 0, static_b: bool = False,
          decode_path: Optional[bool] = None, decode_split: int = 0, pair_path: Optional[bool] = None,
          pair_bnf: int = 0, pair_upp: int = 0, pair_nacc: int = 0) -> torch.Tensor:
     """``out = a @ b`` on tcgen05 with a fused epilogue.
@@ -122,11 +138,19 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *
     129..256 rows with 'kn' weights go to the paired-SM kernel (two CTAs issue one 256-row
     ``tcgen05.mma.cta_group::2``, stream-K over CTA pairs); ``pair_path`` forces (True) or forbids (False) it for
     any M, ``pair_bnf`` / ``pair_nacc`` / ``pair_upp`` override its tile width, tiles per pair and units per pair.
+
+    ``out`` may be fp32 with 16-bit operands (the accumulator is stored unrounded); epilogue 'axpy' adds
+    ``alpha * (a @ b)`` to an fp32 ``out`` (residual streams kept in 32 bits).  ``groups`` > 1: block-diagonal product,
+    a [M, groups * K], b [groups * K, N] (the blocks stacked), out [M, groups * N].  fp32 operands, and 16-bit ones
+    whose sizes the tensor-core kernels do not take, run on the CUDA cores in fp32 arithmetic.
     """
     assert a.is_cuda and a.dim() == 2 and b.dim() == 2 and a.stride(1) == 1 and b.stride(1) == 1
     M, K = a.shape
+    if groups > 1:
+        assert K % groups == 0 and epilogue == "store" and b_layout == "kn" and b.shape[0] == K
+        K //= groups
     if b_layout == "kn":
-        assert b.shape[0] == K
+        assert b.shape[0] == K * groups
         bcols = b.shape[1]
     else:
         assert b.shape[1] == K
@@ -134,20 +158,34 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *
     epi = _EPI[epilogue]
     N = bcols // 2 if epi == 2 else bcols
     if out is None:
-        out = torch.empty((M, N), dtype=a.dtype, device=a.device)
-    assert out.shape == (M, N) and out.stride(1) == 1
+        out = torch.empty((M, groups * N), dtype=a.dtype, device=a.device)
+    assert out.shape == (M, groups * N) and out.stride(1) == 1
+    if epi == 5:
+        assert out.dtype == torch.float32
+    elif out.dtype != a.dtype:
+        assert epi == 0 and out.dtype == torch.float32
+        epi = _EPI_STORE_F32
+    if M == 0:
+        return out
+    if a.dtype == torch.float32 or (groups > 1 and K % 64) or not _tensor_core_operands(a, b, out, N, K):
+        if epi == 1 or b_layout != "kn":
+            raise TypeError("gemm: epilogue 'add' and 'nk' weights need the tensor-core kernels")
+        assert b.dtype == a.dtype
+        _check(lib().blitz_gemm_simt(_p(a), a.stride(0), _p(b), b.stride(0), _p(out), out.stride(0), M, N, K, epi,
+                                     N if epi == 2 else 0, alpha, groups, _dt3(a), _stream()), "blitz_gemm_simt")
+        return out
     if epi == 1:
         assert residual is not None and residual.shape == (M, N) and residual.stride(0) == out.stride(0)
     ws, tickets = gemm_workspace(a.device)
     # the decode kernel re-reads the activation tile with every weight tile, which the SM's load path cannot keep up
     # with beyond ~128 rows; from there on the tiled kernel is faster
-    use_dec = M <= DECODE_GEMM_MAX_M and bn == 0 and split_k == 0 and \
+    use_dec = groups == 1 and M <= DECODE_GEMM_MAX_M and bn == 0 and split_k == 0 and \
         bool(lib().blitz_gemm_decode_supported(M, N, K, 0 if b_layout == "kn" else 1, epi))
     if decode_path is not None:
         assert not decode_path or lib().blitz_gemm_decode_supported(M, N, K, 0 if b_layout == "kn" else 1, epi)
         use_dec = decode_path
     pair_ok = bool(lib().blitz_gemm_pair_supported(M, N, K, 0 if b_layout == "kn" else 1, epi))
-    use_pair = (not use_dec and DECODE_GEMM_MAX_M < M <= PAIR_GEMM_MAX_M and bn == 0 and split_k == 0 and pair_ok)
+    use_pair = (groups == 1 and not use_dec and DECODE_GEMM_MAX_M < M <= PAIR_GEMM_MAX_M and bn == 0 and split_k == 0 and pair_ok)
     if pair_path is not None:
         assert not pair_path or pair_ok
         use_pair = pair_path
@@ -156,18 +194,19 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *
         rc = lib().blitz_gemm_pair(_p(a), a.stride(0), _p(b), b.stride(0), _p(out), out.stride(0), _p(residual), M, N,
                                    K, epi, N if epi == 2 else 0, _dt(a), int(static_b), pair_bnf, pair_nacc, pair_upp,
                                    _p(pws), pws.numel(), _p(pflags), pflags.numel(), _p(status_word(a.device)),
-                                   _stream())
+                                   alpha, _stream())
         _check(rc, "blitz_gemm_pair")
         return out
     if use_dec:
         rc = lib().blitz_gemm_decode(_p(a), a.stride(0), _p(b), b.stride(0), _p(out), out.stride(0), _p(residual), M, N,
                                      K, epi, N if epi == 2 else 0, _dt(a), int(static_b), decode_split,
-                                     _p(status_word(a.device)), _stream())
+                                     _p(status_word(a.device)), alpha, _stream())
         _check(rc, "blitz_gemm_decode")
         return out
     rc = lib().blitz_gemm(_p(a), a.stride(0), _p(b), b.stride(0), _p(out), out.stride(0), _p(residual), M, N, K,
                           0 if b_layout == "kn" else 1, epi, N if epi == 2 else 0, _dt(a), bn, split_k,
-                          _p(ws), ws.numel(), _p(tickets), tickets.numel(), _p(status_word(a.device)), _stream())
+                          _p(ws), ws.numel(), _p(tickets), tickets.numel(), _p(status_word(a.device)), alpha,
+                          groups, _stream())
     _check(rc, "blitz_gemm")
     return out
 
@@ -231,7 +270,7 @@ def argmax(logits: torch.Tensor, out: Optional[torch.Tensor] = None, out_val: Op
     B, V = logits.shape
     if out is None:
         out = torch.empty(B, dtype=torch.int32, device=logits.device)
-    _check(lib().blitz_argmax(_p(logits), B, V, logits.stride(0), _p(out), _p(out_val), idx_offset, _dt(logits),
+    _check(lib().blitz_argmax(_p(logits), B, V, logits.stride(0), _p(out), _p(out_val), idx_offset, _dt3(logits),
                               _stream()), "blitz_argmax")
     return out
 
@@ -244,7 +283,7 @@ def sample(logits: torch.Tensor, temperature: torch.Tensor, top_k: torch.Tensor,
     assert temperature.dtype == torch.float32 and top_k.dtype == torch.int32 and top_p.dtype == torch.float32
     assert seeds.dtype in (torch.int64, torch.uint64)
     _check(lib().blitz_sample(_p(logits), B, V, logits.stride(0), _p(temperature), _p(top_k), _p(top_p), _p(seeds),
-                              step, _p(out), _dt(logits), _stream()), "blitz_sample")
+                              step, _p(out), _dt3(logits), _stream()), "blitz_sample")
     return out
 
 
@@ -285,17 +324,17 @@ def attn_decode(q: torch.Tensor, kv_layer: torch.Tensor, indices: torch.Tensor, 
     return out
 
 
-def prefill_work_list(q_lens, kv_lens, page_size: int, device) -> torch.Tensor:
+def prefill_work_list(q_lens, kv_lens, page_size: int, device, skip: int = 0) -> torch.Tensor:
     """Work records of `attn_prefill_paged`, one per (sequence, 256 rows of it): first row of the sequence in the
     activation, its rows in this pass, index of its first page id, number of its pages, tokens cached for it (this
     pass included), which 256-row pair.  Ordered by the number of key blocks the pair walks, heaviest first; the kernel
-    deals the list back and forth over its CTAs."""
+    deals the list back and forth over its CTAs.  The first `skip` sequences get no record."""
     items = []
     row0 = pg0 = 0
-    for n, kv in zip(q_lens, kv_lens):
+    for s, (n, kv) in enumerate(zip(q_lens, kv_lens)):
         n, kv = int(n), int(kv)
         npages = (kv + page_size - 1) // page_size
-        for pair in range((n + 255) // 256):
+        for pair in range((n + 255) // 256 if s >= skip else 0):
             items.append((min(kv, kv - n + 256 * (pair + 1)), row0, n, pg0, npages, kv, pair))
         row0 += n
         pg0 += npages
@@ -321,4 +360,98 @@ def attn_prefill_paged(qkv: torch.Tensor, kv_layer: torch.Tensor, page_indices: 
                                           work.shape[0], T, q_heads, kv_heads, head_dim, page_size, max_pages, sm_scale,
                                           1 if poly_exp else 0, _p(status_word(qkv.device)), _dt(qkv), _stream()),
            "blitz_attn_prefill_paged")
+    return out
+
+
+# ---------------------------------------------------------------------------------------------- fp32-stream models
+def stream_norm(x: torch.Tensor, w: Optional[torch.Tensor], eps: float, out: Optional[torch.Tensor], *,
+                w_offset: float = 0.0, ids: Optional[torch.Tensor] = None, embed: Optional[torch.Tensor] = None,
+                init: bool = False, add_embed: bool = False, step: Optional[torch.Tensor] = None,
+                rows: Optional[torch.Tensor] = None, row_offset: int = 0,
+                num_tokens: Optional[int] = None) -> Optional[torch.Tensor]:
+    """Additions to the fp32 residual stream ``x`` ([T, hidden], in place) and the RMSNorm that follows, in one kernel.
+
+    ``init``: x starts as ``embed[ids]``; ``add_embed``: the embeddings are added to it; ``step``: a vector added to
+    every row.  ``out`` (None: no norm) = x / rms(x) * (w_offset + w).  ``rows``: output row t takes row
+    ``rows[t] + row_offset`` of x."""
+    n = num_tokens if num_tokens is not None else (rows.numel() if rows is not None else x.shape[0])
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    ref = out if out is not None else embed
+    assert out is None or out.is_contiguous()
+    _check(lib().blitz_stream_norm(_p(ids), _p(embed), _p(step), _p(rows), row_offset, _p(x), _p(w), _p(out), n,
+                                   x.shape[1], embed.shape[0] if embed is not None else 0, int(init), int(add_embed),
+                                   eps, w_offset, _p(status_word(x.device)), _dt3(ref), _stream()), "blitz_stream_norm")
+    return out
+
+
+def rope_freqs(dims: int, base: float, device) -> torch.Tensor:
+    """[dims / 2, 2]: base^(-2 i / dims) as an unevaluated sum of two fp32 numbers."""
+    i = torch.arange(0, dims // 2, dtype=torch.float64)
+    f = torch.pow(torch.tensor(base, dtype=torch.float64), -2.0 * i / max(1, dims))
+    hi = f.to(torch.float32)
+    lo = (f - hi.to(torch.float64)).to(torch.float32)
+    return torch.stack([hi, lo], 1).contiguous().to(device)
+
+
+def rope_store(q: torch.Tensor, k: torch.Tensor, v: Optional[torch.Tensor], pos: torch.Tensor, slot: torch.Tensor,
+               kv_layer: torch.Tensor, freqs: torch.Tensor, *, q_heads: int, kv_heads: int, dim: int, rot_dims: int,
+               page_size: int, interleaved: bool) -> None:
+    """Rotate q in place and write rotated keys and the values to the paged cache.  q, k, v: column ranges of one
+    projection ([T, ...] views with a common row pitch); ``v`` None: the values are the keys before rotation."""
+    T = q.shape[0]
+    assert q.stride(0) == k.stride(0) and q.stride(1) == 1 and k.stride(1) == 1
+    assert v is None or v.stride(0) == q.stride(0)
+    _check(lib().blitz_rope_store(_p(q), _p(k), _p(v), q.stride(0), _p(pos), _p(slot), _p(kv_layer), _p(freqs), T, q_heads,
+                                  kv_heads, dim, rot_dims, int(interleaved), page_size, kv_layer.shape[0],
+                                  _p(status_word(q.device)), _dt3(q), _stream()), "blitz_rope_store")
+
+
+def attn_ragged(q: torch.Tensor, kv_layer: torch.Tensor, pos: torch.Tensor, tok_indptr: Optional[torch.Tensor],
+                page_indptr: torch.Tensor, page_indices: torch.Tensor, out: torch.Tensor, *, q_heads: int, kv_heads: int,
+                dim: int, page_size: int, scale: float, window: int = 0, keep_first: int = 0, softcap: float = 0.0,
+                sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """General paged attention (CUDA cores, any head size, any element type); see csrc/kernels/attn_ragged.cu."""
+    T = q.shape[0]
+    rows = page_indptr.numel() - 1
+    assert q.stride(1) == 1 and out.stride(1) == 1
+    _check(lib().blitz_attn_ragged(_p(q), q.stride(0), _p(kv_layer), _p(out), out.stride(0), _p(pos), _p(tok_indptr),
+                                   _p(page_indptr), _p(page_indices), _p(sink), T, rows, q_heads, kv_heads, dim, page_size,
+                                   kv_layer.shape[0], window, keep_first, scale, softcap, _p(status_word(q.device)),
+                                   _dt3(q), _stream()), "blitz_attn_ragged")
+    return out
+
+
+def gla_recurrent(q, k, v, g, low, a2, a2_b, norm, state: torch.Tensor, out: torch.Tensor, pos, tok_indptr, seq_slot, *,
+                  rank: int, tau: float, eps: float) -> torch.Tensor:
+    """Gated linear attention token by token over the rows of a step; ``state`` [slots, heads, dim, vdim] fp32.
+    ``tok_indptr`` None: one token per row (decode)."""
+    slots, heads, dim, vdim = state.shape
+    assert state.dtype == torch.float32 and state.is_contiguous() and out.stride(1) == 1
+    _check(lib().blitz_gla_recurrent(_p(q), _p(k), _p(v), _p(g), _p(low), q.stride(0), _p(a2), _p(a2_b), _p(norm),
+                                     _p(state), _p(out), out.stride(0), _p(pos), _p(tok_indptr), _p(seq_slot),
+                                     seq_slot.numel(), heads, dim, vdim, rank, slots, dim ** -0.5, tau, eps,
+                                     int(tok_indptr is not None), _p(status_word(q.device)), _dt3(q), _stream()),
+           "blitz_gla_recurrent")
+    return out
+
+
+def conv_causal(x, x_b, conv, conv_b, hist: torch.Tensor, u: torch.Tensor, pos, tok_indptr, seq_slot) -> torch.Tensor:
+    """Causal short convolution per channel over the rows of a step; ``hist`` [slots, taps - 1, width], only read."""
+    slots, keep, width = hist.shape
+    _check(lib().blitz_conv_causal(_p(x), x.stride(0), _p(x_b), _p(conv), _p(conv_b), _p(hist), _p(u), u.stride(0), _p(pos),
+                                   _p(tok_indptr), _p(seq_slot), x.shape[0], seq_slot.numel(), width, keep + 1, slots,
+                                   _p(status_word(x.device)), _dt3(x), _stream()), "blitz_conv_causal")
+    return u
+
+
+def rglru_scan(u, gates: torch.Tensor, gate_b, lam, y, x, y_b, state: torch.Tensor, hist: torch.Tensor, out, pos,
+               tok_indptr, seq_slot, *, block: int) -> torch.Tensor:
+    """Real-gated linear recurrent unit over the rows of a step, times gelu(y); updates ``state`` [slots, width] and the
+    convolution's history."""
+    slots, width = state.shape
+    assert gates.dtype == torch.float32 and gates.is_contiguous() and y.stride(0) == x.stride(0)
+    _check(lib().blitz_rglru_scan(_p(u), u.stride(0), _p(gates), _p(gate_b), _p(lam), _p(y), _p(x), y.stride(0), _p(y_b),
+                                  _p(state), _p(hist), _p(out), out.stride(0), _p(pos), _p(tok_indptr), _p(seq_slot),
+                                  seq_slot.numel(), width, block, hist.shape[1] + 1, slots, int(tok_indptr is None),
+                                  _p(status_word(u.device)), _dt3(u), _stream()), "blitz_rglru_scan")
     return out

@@ -39,7 +39,7 @@ class Engine:
                  device: Optional[torch.device] = None, comm: Optional[TPComm] = None, use_graphs: bool = True,
                  seg_buffer: Optional[torch.Tensor] = None, kv_buffer: Optional[torch.Tensor] = None,
                  ready: bool = True, seed: int = 0, fused_tp: bool = True, oneshot_max_rows: int = 1024,
-                 tp_contexts: int = 1, use_switch: bool = True):
+                 tp_contexts: int = 1, use_switch: bool = True, state_slots: Optional[int] = None):
         self.cfg = get_config(model) if isinstance(model, str) else model
         self.device = device or torch.device("cuda", torch.cuda.current_device())
         self.dtype, self.tp, self.tp_rank = dtype, tp, tp_rank
@@ -47,15 +47,29 @@ class Engine:
         self.max_batch, self.max_batch_tokens = max_batch, max_batch_tokens
         c = self.cfg
         self.seg = WeightSegment(c, tp, tp_rank, dtype, device=self.device, buffer=seg_buffer)
-        kvh = c.kv_heads // tp
-        kv_shape = (c.layers, num_pages, 2, page_size, kvh, c.head_dim)
-        if kv_buffer is None:
-            # zero-filled: the attention kernels require finite values in every slot of an allocated page
-            self.kv = torch.zeros(kv_shape, dtype=dtype, device=self.device)
-        else:
-            self.kv = kv_buffer.view(dtype)[:int(np.prod(kv_shape))].view(kv_shape)
         self.fused = None
-        if tp > 1 and comm is not None and fused_tp:
+        self.slots = None           # state slots of models with recurrent layers
+        if c.family == "hybrid":
+            if tp > 1 or kv_buffer is not None:
+                raise ValueError(f"{c.name}: a hybrid model runs on one GPU, with its own cache memory")
+            from ..models.hybrid import HybridRunner
+            from .hybrid_cache import HybridCache
+            self.cache = HybridCache(c, num_pages, page_size, state_slots or max_batch, dtype, self.device)
+            if c.recurrent:
+                self.slots = core.SlotPool(self.cache.num_slots)
+        else:
+            if dtype == torch.float32:
+                raise ValueError(f"{c.name}: the kernels of this model take 16-bit types")
+            kvh = c.kv_heads // tp
+            kv_shape = (c.layers, num_pages, 2, page_size, kvh, c.head_dim)
+            if kv_buffer is None:
+                # zero-filled: the attention kernels require finite values in every slot of an allocated page
+                self.kv = torch.zeros(kv_shape, dtype=dtype, device=self.device)
+            else:
+                self.kv = kv_buffer.view(dtype)[:int(np.prod(kv_shape))].view(kv_shape)
+        if c.family == "hybrid":
+            self.runner = HybridRunner(self.seg, self.cache, max(max_batch_tokens, max_batch), max_batch)
+        elif tp > 1 and comm is not None and fused_tp:
             # tensor-parallel layers through the fused peer-memory kernels (GEMM -> reduce-scatter push, reduce + norm +
             # all-gather push, flag-gated GEMM); the NCCL all-reduce runner is the baseline (`fused_tp=False`)
             from ..parallel.tp import FusedTP, LlamaRunnerTP
@@ -87,17 +101,20 @@ class Engine:
 
     # ------------------------------------------------------------------ meta views
     def _views(self, T: int, B: int, P: int, prefill: bool, seq_lens: Sequence[int] = (), splits: int = 1,
-               kv_lens: Sequence[int] = (), work: Optional[torch.Tensor] = None) -> StepMeta:
+               kv_lens: Sequence[int] = (), work: Optional[torch.Tensor] = None, singles: int = 0) -> StepMeta:
         L, d = self.layout, self.dev
         kv_lens = list(kv_lens) if kv_lens else list(seq_lens)
         if prefill and work is None:
-            work = ops.prefill_work_list(seq_lens, kv_lens, self.page_size, self.device)
+            # the hybrid runner takes the leading single tokens of a ragged step through its decode kernels
+            work = ops.prefill_work_list(seq_lens, kv_lens, self.page_size, self.device,
+                                         skip=singles if self.cfg.family == "hybrid" else 0)
         return StepMeta(kv_lens_host=kv_lens, prefill_work=work,
                         ids=d[L.ids:L.ids + T], pos=d[L.pos:L.pos + T], slot=d[L.slot:L.slot + T],
                         page_indices=d[L.page_indices:L.page_indices + max(P, 1)],
                         page_indptr=d[L.page_indptr:L.page_indptr + B + 1],
                         last_page_len=d[L.last_page_len:L.last_page_len + B],
                         tok_indptr=d[L.tok_indptr:L.tok_indptr + B + 1] if prefill else None,
+                        seq_slot=d[L.seq_slot:L.seq_slot + B], singles=singles,
                         seq_lens_host=list(seq_lens), is_prefill=prefill, batch=B, num_tokens=T, num_splits=splits)
 
     def _h2d(self, hi: int) -> None:
@@ -112,13 +129,19 @@ class Engine:
 
     # ------------------------------------------------------------------ batches
     def new_batch(self, batch_id: int, specs) -> Optional["core.Batch"]:
-        b = core.Batch(batch_id, self.pool)
+        b = core.Batch(batch_id, self.pool, self.slots)
         if not b.add_prompts(specs):
             return None
         return b
 
     def choose_splits(self, B: int, max_len: int) -> int:
-        ctas = B * (self.cfg.kv_heads // self.tp)
+        if self.cfg.family == "hybrid":
+            kv_heads, max_len = self.cfg.attention_work(max_len)
+            if kv_heads == 0:
+                return 1
+        else:
+            kv_heads = self.cfg.kv_heads // self.tp
+        ctas = B * kv_heads
         if ctas >= 2 * 148 or max_len <= 256:
             return 1
         want = (2 * 148 + ctas - 1) // ctas
@@ -172,7 +195,7 @@ class Engine:
         if forced is not None:
             runner.force_switch = True          # tensor parallel: keep the residual stream replicated in every pass
         try:
-            states = torch.empty(B, self.cfg.hidden, dtype=self.dtype, device=self.device)
+            states = torch.empty(B, self.cfg.hidden, dtype=runner.res.dtype, device=self.device)
             tok0 = 0
             while tok0 < total:
                 T, P, rows, s0, q_lens, kv_lens, ended = batch.fill_prefill_chunk(self.host_np, self.layout, tok0,
@@ -223,6 +246,73 @@ class Engine:
         batch.append_tokens(out, True)
         return out
 
+    @torch.no_grad()
+    def step(self, batch: "core.Batch", counts: Sequence[int], want: Sequence[Sequence[int]] = ()) -> Optional[torch.Tensor]:
+        """One step over any mixture of the batch's requests: `counts[i]` tokens of request i, from the first one that is
+        not cached yet (0: it sits this step out); portions of prompts and single tokens run together.  `want[i]`: places
+        among these tokens whose logits are returned, [total, vocab] fp32, in the order of the requests (None if there
+        are none).  Nothing is sampled.  Steps beyond `max_batch_tokens` are cut into several passes."""
+        if not self.status.fully_loaded():
+            raise RuntimeError("model parameters are not loaded")
+        if self.tp > 1:
+            raise RuntimeError("steps of given tokens run on one GPU")
+        if batch.size > self.max_batch:
+            raise ValueError(f"step over {batch.size} sequences exceeds max_batch={self.max_batch}")
+        counts = list(counts)
+        want = [list(w) for w in want] if len(want) else [[] for _ in counts]
+        first = [sum(len(w) for w in want[:i]) for i in range(len(want))]
+        total = sum(len(w) for w in want)
+        out = torch.empty(total, self.cfg.vocab, dtype=torch.float32, device=self.device) if total else None
+        done = [0] * len(counts)
+        while any(d < c for d, c in zip(done, counts)):
+            room, take = self.max_batch_tokens, []
+            for d, c in zip(done, counts):
+                take.append(min(room, c - d))
+                room -= take[-1]
+            dest, src = [], []           # rows of `out` this pass fills, and where they come from
+            for i, w in enumerate(want):
+                for j, p in enumerate(w):
+                    if done[i] <= p < done[i] + take[i]:
+                        dest.append(first[i] + j)
+                        src.append((i, p - done[i]))
+            rows = self._step_pass(batch, take, src)
+            if dest:
+                out[torch.tensor(dest, device=self.device)] = rows
+            done = [d + t for d, t in zip(done, take)]
+        return out
+
+    def _step_pass(self, batch: "core.Batch", counts: List[int], src: List[tuple]) -> Optional[torch.Tensor]:
+        """One forward pass of `step`: logits of the (request, place) pairs in `src`."""
+        single = all(c <= 1 for c in counts)
+        rows_max = sum(1 for c in counts if c)
+        pad = min(_bucket(rows_max), self.max_batch) if self.use_graphs else rows_max
+        T, P, rows, singles, order, q_lens, kv_lens = batch.fill_step(self.host_np, self.layout, counts, pad)
+        self._h2d(self.layout.page_indices + P)
+        row_of = {b: r for r, b in enumerate(order)}
+        if single:
+            splits = self.choose_splits(pad, max(kv_lens))
+            if self.use_graphs:
+                (self._graphs.get((pad, splits)) or self._capture(pad, splits)).replay()
+            else:
+                self.runner.forward(self._views(pad, pad, self.num_pages, False, splits=splits))
+            got = None
+            if src:
+                got = self.runner.logits[torch.tensor([row_of[b] for b, _ in src], device=self.device)].float()
+        else:
+            m = self._views(T, rows, P, True, q_lens, kv_lens=kv_lens, singles=singles)
+            with nvtx_range("step"):
+                self.runner.forward(m, with_head=False)
+                starts = [sum(q_lens[:r]) for r in range(rows)]
+                flat = [starts[row_of[b]] + p for b, p in src]
+                parts = []
+                for i in range(0, len(flat), self.max_batch):
+                    idx = torch.tensor(flat[i:i + self.max_batch], dtype=torch.int32, device=self.device)
+                    parts.append(self.runner.logits_of(idx.numel(), idx).float().clone())
+                got = torch.cat(parts) if parts else None
+        torch.cuda.current_stream().synchronize()       # the staging arrays are reused by the next pass
+        batch.advance(counts)
+        return got
+
     def _sample_rows(self, batch: "core.Batch", B: int, toks: torch.Tensor) -> torch.Tensor:
         """Rows whose request asked for sampling (`do_sample` with temperature / top-k / top-p / seed) draw their token
         from this step's logits with the sampling kernel; all other rows keep the arg-max.  One extra small launch,
@@ -263,7 +353,11 @@ class Engine:
     def _capture(self, Bp: int, splits: int) -> torch.cuda.CUDAGraph:
         m = self._views(Bp, Bp, self.num_pages, False, splits=splits)
         # warm up outside capture: first-use work (attribute setup, descriptor cache, workspace allocation)
+        # (its rows carry no state slot: a K/V write repeats itself, a recurrence would advance the state twice)
+        slots = m.seq_slot.clone()
+        m.seq_slot.fill_(-1)
         self.runner.forward(m)
+        m.seq_slot.copy_(slots)
         torch.cuda.current_stream().synchronize()
         g = torch.cuda.CUDAGraph()
         # thread-local capture: transfer and RPC threads of a worker keep making CUDA calls (small copies, flag reads)
@@ -311,10 +405,23 @@ class Engine:
 
     def decode_launch_count(self) -> int:
         """Kernels of this library launched by one decode step at tp = 1 (for the bench's launch accounting)."""
+        if self.cfg.family == "hybrid":
+            return self.runner.decode_launches()
         per_layer = 8  # rms_norm, qkv gemm, rope_kv_store, attention, o gemm, rms_norm, gate_up gemm, down gemm
         return 1 + per_layer * self.cfg.layers + 3  # embedding + layers + final norm, lm_head gemm, argmax
 
     # ------------------------------------------------------------------ parameters
+    def load_checkpoint(self, directory) -> None:
+        """Weights straight from a checkpoint folder (.safetensors), without a segment file in between (one GPU)."""
+        from ..models.convert import CheckpointReader, checkpoint_to_segment
+        if self.tp > 1:
+            raise ValueError("sharded replicas load segment files (see models/convert.py)")
+        seg = checkpoint_to_segment(CheckpointReader(directory), self.cfg, self.dtype)
+        n = self.seg.layout.total_bytes
+        self.seg.buffer[:n].copy_(seg.buffer[:n])
+        torch.cuda.synchronize()
+        self.status.set_ready()
+
     def set_status_ready(self) -> None:
         self.status.set_ready()
 
