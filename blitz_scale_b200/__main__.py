@@ -5,6 +5,7 @@
     router        router / autoscaler with the HTTP API                                 -> router.server
     client        trace-replay client (writes client.jsonl)                             -> sim.request_sim
     convert       Hugging Face safetensors -> weight-segment files                      -> models.convert
+    trace-run     replay a trace of given tokens, step by step, and write the logits      -> runtime.trace_run
     repl          interactive gRPC client / load-latency / broadcast benchmark          -> utils.worker_client
     logs          log debuggers (merge, grep, zigzag, usage, migrations)                -> utils.logtools
     trace         trace-file tools (slice, scale, concat, stats, compare)               -> sim.trace_tools
@@ -19,7 +20,7 @@ import sys
 COMMANDS = {
     "worker": "blitz_scale_b200.worker.launcher", "stub-worker": "blitz_scale_b200.sim.stub_worker",
     "router": "blitz_scale_b200.router.server", "client": "blitz_scale_b200.sim.request_sim",
-    "convert": "blitz_scale_b200.models.convert", "repl": "blitz_scale_b200.utils.worker_client",
+    "convert": "blitz_scale_b200.models.convert", "trace-run": "blitz_scale_b200.runtime.trace_run", "repl": "blitz_scale_b200.utils.worker_client",
     "logs": "blitz_scale_b200.utils.logtools", "trace": "blitz_scale_b200.sim.trace_tools",
     "report": "blitz_scale_b200.utils.plots", "chrome-trace": "blitz_scale_b200.utils.tracing",
     "build": "blitz_scale_b200.build", "proto": "blitz_scale_b200.pb.schema",

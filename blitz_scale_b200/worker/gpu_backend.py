@@ -18,6 +18,7 @@ memory (`parallel/symm.py`) instead of RDMA / NCCL calls:
 from __future__ import annotations
 
 import logging
+import os
 import threading
 import time
 from concurrent.futures import Future
@@ -57,10 +58,16 @@ class GpuBackend(Backend):
         self.use_multimem, self.copy_ctas = use_multimem, copy_ctas
         dt = torch.bfloat16
         probe = WeightSegment(self.cfg, tp, rank % tp, dt, device="meta")
-        kvh = self.cfg.kv_heads // tp
-        self.page_bytes = 2 * page_size * kvh * self.cfg.head_dim * 2
-        self.kv_layer_stride = num_pages * self.page_bytes
-        kv_bytes = self.cfg.layers * self.kv_layer_stride
+        self.hybrid = self.cfg.family == "hybrid"
+        if self.hybrid:
+            # pools of several shapes plus state slots, in the engine's own memory: nothing of it is a peer region
+            self.page_bytes = self.cfg.kv_bytes_per_token(tp, 2) * page_size
+            self.kv_layer_stride, kv_bytes = 0, 256
+        else:
+            kvh = self.cfg.kv_heads // tp
+            self.page_bytes = 2 * page_size * kvh * self.cfg.head_dim * 2
+            self.kv_layer_stride = num_pages * self.page_bytes
+            kv_bytes = self.cfg.layers * self.kv_layer_stride
         self.slot_bytes = max_batch_tokens * self.cfg.hidden * 2
         self.fabric: Optional[symm.PeerFabric] = None
         seg_buf = kv_buf = None
@@ -78,14 +85,19 @@ class GpuBackend(Backend):
             self.fabric = symm.PeerFabric(symm.FabricSizes(weight_bytes=probe.layout.total_bytes, kv_bytes=kv_bytes,
                                                            mailbox_slots=4, mailbox_slot_bytes=self.slot_bytes),
                                           weight_group=column)
-            seg_buf, kv_buf = self.fabric.weights.local, self.fabric.kv.local
+            seg_buf, kv_buf = self.fabric.weights.local, None if self.hybrid else self.fabric.kv.local
             self.ctl = symm.SymmRegion(symm.KV_SLOTS * CTL_SLOT_WORDS * 4 + symm.KV_SLOTS * 4)  # id lists, then tags
             self.ctl.local.zero_()
         comm = TPComm(tp_group) if tp > 1 else None
+        # a checkpoint folder as the model: its weights are what a ready replica serves
+        from_checkpoint = ready and os.path.isfile(os.path.join(model, "config.json"))
         self.engine = Engine(self.cfg, num_pages=num_pages, page_size=page_size, max_batch=max_batch,
                              max_batch_tokens=max_batch_tokens, tp=tp, tp_rank=rank % tp, dtype=dt, comm=comm,
-                             seg_buffer=seg_buf, kv_buffer=kv_buf, ready=ready, seed=seed, fused_tp=fused_tp,
-                             tp_contexts=5 if tp > 1 else 1)     # context 0 + one per live-execution slot
+                             seg_buffer=seg_buf, kv_buffer=kv_buf, ready=ready and not from_checkpoint, seed=seed,
+                             fused_tp=fused_tp, tp_contexts=5 if tp > 1 else 1,     # context 0 + one per live-execution slot
+                             state_slots=2 * max_batch)                             # a full decode batch and a prefill batch
+        if from_checkpoint:
+            self.engine.load_checkpoint(model)
         self.units = [(n, o, b) for n, o, b in self.engine.seg.layout.units]
         if precapture:
             # every decode graph is captured now, whether or not the parameters are here yet, so that neither a
@@ -101,7 +113,7 @@ class GpuBackend(Backend):
         self.zag = core.ZigzagScheduler(L, 4)
         self._zag_layers_seen = 0
         self.zag_tasks: Dict[int, dict] = {}
-        self.zag_slots = torch.empty(4, max_batch_tokens, self.cfg.hidden, dtype=dt, device=self.device)
+        self.zag_slots = None if self.hybrid else torch.empty(4, max_batch_tokens, self.cfg.hidden, dtype=dt, device=self.device)
         self.zag_cv = threading.Condition(self.lock)
         self._stop = False
         # transfers (parameter copies, KV push / arrival waits, relays) run on their own high-priority stream so that
@@ -161,6 +173,11 @@ class GpuBackend(Backend):
             self.batches.pop(b.id, None)
         return gens, (self._cached(b) if b.size else None)
 
+    def _refuse_hybrid(self, what: str) -> None:
+        if self.hybrid:
+            raise RuntimeError(f"{what} is not available for {self.cfg.name}: its sequences carry recurrent state and "
+                               "its layers may run several times")
+
     # ------------------------------------------------------------------ inference
     def prefill(self, batch, forward_case, pp_info, pipe_peer):
         with self.lock:
@@ -168,7 +185,10 @@ class GpuBackend(Backend):
                 raise RuntimeError("model parameters are not loaded")
             b = self.engine.new_batch(batch.id, self._specs(batch))
             if b is None:
-                raise RuntimeError("out of KV pages")
+                raise RuntimeError("out of KV pages" if self.engine.slots is None else "out of KV pages or state slots")
+            if forward_case & (pb.PREFILL_CASE_NAIVE_PP | pb.PREFILL_CASE_MIGRATE_PROGRESSIVE) and self.hybrid:
+                b.clear()
+                self._refuse_hybrid("a relayed or migrating prefill")
             if forward_case & pb.PREFILL_CASE_NAIVE_PP:
                 start = 0
                 if pp_info is not None and pp_info.WhichOneof("start_layer") == "tfm_layer":
@@ -311,6 +331,7 @@ class GpuBackend(Backend):
 
     # ------------------------------------------------------------------ live execution (ZigZag)
     def zag_prefill(self, batch, forward_case, pp_info, zag_layers, zag_seq):
+        self._refuse_hybrid("live execution")
         if self.engine.fused is not None and not self.engine.fused.has_mc:
             # tensor-parallel live execution keeps one residual stream per task in symmetric memory and updates it
             # through the switch-reduced kernel, which needs the fabric's multicast address
@@ -470,6 +491,7 @@ class GpuBackend(Backend):
             self.zag_tasks.pop(d.batch_id)["future"].set_result((gens, cb, None))
 
     def relay(self, rank, relax_not_head):
+        self._refuse_hybrid("live execution")
         if self.steplog is not None and not self.steplog.leader:
             # the leading shard chooses the task and the layer; this shard's live-execution thread acts when it reads
             # that choice in the log
@@ -560,6 +582,7 @@ class GpuBackend(Backend):
         return ids
 
     def immigrate(self, batch, src, dst, partial=0, num_layer=0):
+        self._refuse_hybrid("KV migration")
         lo, hi = self._layer_range(partial, num_layer)
         half = {pb.PARTIAL_CASE_FIRST: " first half", pb.PARTIAL_CASE_SECOND: " second half"}.get(partial, "")
         slot = batch.id % symm.KV_SLOTS
@@ -627,6 +650,7 @@ class GpuBackend(Backend):
         symm._check(symm._L.lib().blitz_flag_set(ctypes.c_void_p(ptr), value, 0, symm._stream()), "blitz_flag_set")
 
     def migrate(self, batch, src, dst, partial=0, num_layer=0):
+        self._refuse_hybrid("KV migration")
         with self.lock:
             b = self.batches.get(batch.id)
             if b is None:
@@ -737,6 +761,8 @@ class GpuBackend(Backend):
         with self.lock:
             if load_case == pb.LOAD_FROM_HOST_MEM and self.host_mirror is not None:
                 self.engine.load_params_from_host(self.host_mirror)
+            elif os.path.isfile(os.path.join(path, "config.json")) and not os.path.isfile(os.path.join(path, "segment.0.json")):
+                self.engine.load_checkpoint(path)
             else:
                 res = self.engine.load_params_from_disk(path, self.host_mirror)
                 self.host_mirror = res["host_mirror"]

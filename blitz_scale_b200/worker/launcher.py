@@ -27,7 +27,8 @@ import torch.distributed as dist
 def parse_args(argv=None):
     ap = argparse.ArgumentParser("blitz-worker")
     ap.add_argument("--model-path", default="")
-    ap.add_argument("--model-name", default="llama3_8b")
+    ap.add_argument("--model-name", default="llama3_8b", help="registry name, or a checkpoint folder whose config.json names "
+                    "an architecture this package describes by data (ready ranks then serve its weights)")
     ap.add_argument("-T", "--tokenizer", default="", help="tokenizer.json: text of generated tokens, which the worker "
                     "needs to apply the stop sequences of a request (without it they match the <id> text of its generations)")
     ap.add_argument("-V", "--vocab-json", default="")
