@@ -25,6 +25,10 @@
 // memory is cleared and the barriers are set up while the previous kernel is
 // still running; the first load waits for it.
 //
+// Models that ask for it get a sliding window with kept first tokens (only the 64-token chunks that hold a visible key
+// are fetched: a sequence costs at most window + kept tokens whatever its length), soft-capped scores
+// (cap * tanh(s / cap)) and a per-head sink, a term e^sink in the softmax denominator, which the merge adds once.
+//
 // The cache must hold finite values in every slot of an allocated page (the
 // pool is zero-filled at creation): masked positions get probability 0, and
 // 0 x NaN would still poison the accumulator.
@@ -56,6 +60,9 @@ struct DecodeTcParams {
   int batch, q_heads, kv_heads, group, page_size, max_pages, num_splits, box_tokens;
   int tail_box_tokens;  // box height of the second tensor map, used for the last (partly filled) chunk of a sequence
   float scale_log2;
+  int window, keep_first;       // 0: every key; else a token sees the last `window` positions and the first `keep_first`
+  float cap_scale, cap_log2;    // soft cap (cap_log2 > 0): score in log2 units = cap_log2 * tanh(q.k * cap_scale)
+  const void* sink;             // [q_heads] in the activation type, or null
   int* status;
   long long* trace;  // profiling aid (null in production): clock stamps of CTA 0's first items, see blitz_attn_decode_set_trace
 };
@@ -106,7 +113,11 @@ struct TcCfg {
 // blockIdx.x, blockIdx.x + gridDim.x, ... and the producer keeps streaming the next item's pages while
 // the consumers finish the current one, so the 4-stage pipeline never drains between items.
 struct DecItem {
-  int b, h, split, pg_beg, seq_len, c_beg, c_end;
+  int b, h, split, pg_beg, seq_len, c_beg, c_end;  // c_beg .. c_end: this split's share of the visible chunks
+  int lo, first;         // visible keys: [0, first) and [lo, seq_len)
+  int n_first, c_window; // chunks of the kept tokens; first chunk of the window behind them
+  // the n-th visible chunk
+  __device__ __forceinline__ int chunk(int n) const { return n < n_first ? n : c_window + n - n_first; }
 };
 __device__ __forceinline__ DecItem dec_item(const DecodeTcParams& p, int item) {
   DecItem it;
@@ -116,7 +127,11 @@ __device__ __forceinline__ DecItem dec_item(const DecodeTcParams& p, int item) {
   it.pg_beg = p.indptr[it.b];
   const int npages = p.indptr[it.b + 1] - it.pg_beg;
   it.seq_len = npages > 0 ? (npages - 1) * p.page_size + p.last_page_len[it.b] : 0;
-  const int nchunks = (it.seq_len + kTcChunk - 1) / kTcChunk;
+  it.lo = p.window > 0 ? max(0, it.seq_len - p.window) : 0;
+  it.first = min(p.keep_first, it.lo);
+  it.n_first = (it.first + kTcChunk - 1) / kTcChunk;
+  it.c_window = max(it.lo / kTcChunk, it.n_first);
+  const int nchunks = it.n_first + max(0, (it.seq_len + kTcChunk - 1) / kTcChunk - it.c_window);
   const int cps = (nchunks + p.num_splits - 1) / p.num_splits;
   it.c_beg = min(nchunks, it.split * cps);
   it.c_end = min(nchunks, (it.split + 1) * cps);
@@ -179,7 +194,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
     bool ok = true;
     int item = blockIdx.x;
     DecItem it = item < num_items ? dec_item(p, item) : DecItem{};
-    int win_base = item < num_items ? (it.c_beg * kTcChunk) / ps : 0;
+    int win_base = item < num_items ? (it.chunk(it.c_beg) * kTcChunk) / ps : 0;
     int win = item < num_items ? load_window(it, win_base) : 0;
     int n_done = 0;
     while (item < num_items && ok) {
@@ -187,10 +202,10 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
       // next item's metadata and first window: in flight while this item streams
       const int next = item + gridDim.x;
       DecItem nit = next < num_items ? dec_item(p, next) : DecItem{};
-      const int nwin_base = next < num_items ? (nit.c_beg * kTcChunk) / ps : 0;
+      const int nwin_base = next < num_items ? (nit.chunk(nit.c_beg) * kTcChunk) / ps : 0;
       const int nwin = next < num_items ? load_window(nit, nwin_base) : 0;
       for (int c = it.c_beg; c < it.c_end && ok; ++c) {
-        const int tok0 = c * kTcChunk;
+        const int tok0 = it.chunk(c) * kTcChunk;
         const int ntok = min(kTcChunk, it.seq_len - tok0);
         // a full chunk comes in boxes of box_tokens rows; the last chunk of a sequence only as far as it is
         // filled, in the smaller boxes of the second map (a 64-token page with 18 live tokens costs 32 rows)
@@ -292,8 +307,11 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
           ok = false;
         }
         if (tracer && c == it.c_beg) tc_trace(p, n_done, 1);
-        const int nvalid = min(kTcChunk, it.seq_len - c * kTcChunk);
-        if (ok && tokw < nvalid) {
+        const int tok0 = it.chunk(c) * kTcChunk;
+        const int nvalid = min(kTcChunk, it.seq_len - tok0);
+        // visible keys of this warp's 16: below `kept` or from `from` on (both relative to the chunk)
+        const int kept = it.first - tok0, from = it.lo - tok0;
+        if (ok && tokw < nvalid && (tokw < kept || (tokw + 16 > from && nvalid > from))) {
           const uint32_t kbase = ptx::smem_u32(smem + stage * Cfg::kStageBytes);
           const uint32_t vbase = kbase + SL * kTcSlabBytes;
           float s_lo[4] = {0.f, 0.f, 0.f, 0.f}, s_hi[4] = {0.f, 0.f, 0.f, 0.f};
@@ -310,7 +328,16 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
             }
           }
           const int col = tokw + 2 * t4;
-          const bool v0 = col < nvalid, v1 = col + 1 < nvalid, v2 = col + 8 < nvalid, v3 = col + 9 < nvalid;
+          auto visible = [&](int k) { return k < nvalid && (k >= from || k < kept); };
+          const bool v0 = visible(col), v1 = visible(col + 1), v2 = visible(col + 8), v3 = visible(col + 9);
+          auto score = [&](float x) {  // log2 units
+            return p.cap_log2 > 0.f ? p.cap_log2 * ptx::tanh_ex2(x * p.cap_scale) : x * p.scale_log2;
+          };
+#pragma unroll
+          for (int k = 0; k < 2; ++k) {  // rows 8..15 of the fragments are padding
+            s_lo[k] = score(s_lo[k]);
+            s_hi[k] = score(s_hi[k]);
+          }
           float mx = -INFINITY;
           if (v0) mx = fmaxf(mx, s_lo[0]);
           if (v1) mx = fmaxf(mx, s_lo[1]);
@@ -318,12 +345,12 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
           if (v3) mx = fmaxf(mx, s_hi[1]);
           mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
           mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-          const float m_new = fmaxf(m, mx * p.scale_log2);
+          const float m_new = fmaxf(m, mx);
           const float alpha = exp2f(m - m_new);  // m = -inf -> 0
-          const float p0 = v0 ? exp2f(s_lo[0] * p.scale_log2 - m_new) : 0.f;
-          const float p1 = v1 ? exp2f(s_lo[1] * p.scale_log2 - m_new) : 0.f;
-          const float p2 = v2 ? exp2f(s_hi[0] * p.scale_log2 - m_new) : 0.f;
-          const float p3 = v3 ? exp2f(s_hi[1] * p.scale_log2 - m_new) : 0.f;
+          const float p0 = v0 ? exp2f(s_lo[0] - m_new) : 0.f;
+          const float p1 = v1 ? exp2f(s_lo[1] - m_new) : 0.f;
+          const float p2 = v2 ? exp2f(s_hi[0] - m_new) : 0.f;
+          const float p3 = v3 ? exp2f(s_hi[1] - m_new) : 0.f;
           l = l * alpha + (p0 + p1 + p2 + p3);
           m = m_new;
           const uint32_t pa0 = pk2<T>(p0, p1), pa2 = pk2<T>(p2, p3);
@@ -371,6 +398,10 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
         float M = -INFINITY;
 #pragma unroll
         for (int w = 0; w < 4; ++w) M = fmaxf(M, mrg_m[w * 8 + gg]);
+        const int head = it.h * G + gg;
+        const bool with_sink = p.sink != nullptr && p.num_splits == 1;  // several splits: the merge kernel adds it
+        const float sink = with_sink ? to_f<T>(reinterpret_cast<const T*>(p.sink)[head]) * 1.4426950408889634f : -INFINITY;
+        M = fmaxf(M, sink);
         float L = 0.f, O = 0.f;
         if (M > -INFINITY) {
 #pragma unroll
@@ -380,8 +411,8 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
             O += mrg_o[(w * 8 + gg) * HD + d] * sc;
           }
         }
+        if (with_sink) L += exp2f(sink - M);
         const float val = L > 0.f ? O / L : 0.f;
-        const int head = it.h * G + gg;
         if (p.num_splits == 1) {
           T* op = reinterpret_cast<T*>(p.out) + static_cast<int64_t>(it.b) * p.out_stride +
                   static_cast<int64_t>(head) * HD;
@@ -407,14 +438,17 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
   }
 }
 
-// Combine split partials: out = sum_s w_s o_s / sum_s w_s, w_s = 2^(lse_s - max lse).
+// Combine split partials: out = sum_s w_s o_s / (sum_s w_s + e^sink), w_s = 2^(lse_s - max lse).
 template <typename T>
 __global__ void attn_merge_tc_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
-                                     T* __restrict__ out, int64_t out_stride, int q_heads, int hd, int num_splits) {
+                                     T* __restrict__ out, int64_t out_stride, int q_heads, int hd, int num_splits,
+                                     const T* __restrict__ sink) {
   const int b = blockIdx.x, head = blockIdx.y;
   const int64_t base = (static_cast<int64_t>(b) * q_heads + head) * num_splits;
   float M = -INFINITY;
   for (int s = 0; s < num_splits; ++s) M = fmaxf(M, part_lse[base + s]);
+  const float snk = sink ? to_f<T>(sink[head]) * 1.4426950408889634f : -INFINITY;
+  M = fmaxf(M, snk);
   for (int d = threadIdx.x; d < hd; d += blockDim.x) {
     float acc = 0.f, wsum = 0.f;
     if (M > -INFINITY) {
@@ -423,6 +457,7 @@ __global__ void attn_merge_tc_kernel(const float* __restrict__ part_o, const flo
         wsum += w;
         acc += w * part_o[(base + s) * hd + d];
       }
+      if (sink) wsum += exp2f(snk - M);
     }
     const float val = wsum > 0.f ? acc / wsum : 0.f;
     T* op = out + static_cast<int64_t>(b) * out_stride + static_cast<int64_t>(head) * hd;
@@ -469,12 +504,15 @@ int64_t blitz_attn_decode_workspace_bytes(int batch, int q_heads, int head_dim, 
 // kv_layer: [max_pages][2][page_size][kv_heads][head_dim].  workspace: scratch of
 // blitz_attn_decode_workspace_bytes() bytes (may be null when num_splits == 1).
 // page_size must be a power of two >= 8 (pages smaller than 64 tokens are fetched as
-// several boxes per stage).  q_heads / kv_heads <= 8; head_dim 64 or 128.
+// several boxes per stage).  q_heads / kv_heads <= 8; head_dim 64 or 128.  window (0 = none) / keep_first, softcap (0 =
+// none) and sink (null = none) as described at the top of the file.
 int blitz_attn_decode(const void* q, int64_t q_stride, const void* kv_layer, const int32_t* indices,
                       const int32_t* indptr, const int32_t* last_page_len, void* out, int64_t out_stride,
                       void* workspace, int batch, int q_heads, int kv_heads, int head_dim, int page_size,
-                      int max_pages, int num_splits, float sm_scale, int* status, int dtype, cudaStream_t stream) {
+                      int max_pages, int num_splits, float sm_scale, int window, int keep_first, float softcap,
+                      const void* sink, int* status, int dtype, cudaStream_t stream) {
   if (batch <= 0) return 0;
+  if (window < 0 || keep_first < 0 || softcap < 0.f) return -1;
   if (num_splits < 1 || (q_heads % kv_heads) != 0 || (q_stride & 1) || (out_stride & 1)) return -1;
   const int G = q_heads / kv_heads;
   if (G > 8 || (head_dim != 64 && head_dim != 128)) return -1;
@@ -497,6 +535,8 @@ int blitz_attn_decode(const void* q, int64_t q_stride, const void* kv_layer, con
   p.batch = batch; p.q_heads = q_heads; p.kv_heads = kv_heads; p.group = G; p.page_size = page_size; p.max_pages = max_pages;
   p.num_splits = num_splits; p.box_tokens = bt; p.tail_box_tokens = bt_tail;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = g_tc_trace;
+  p.window = window; p.keep_first = keep_first; p.sink = sink;
+  p.cap_scale = softcap > 0.f ? sm_scale / softcap : 0.f; p.cap_log2 = softcap * 1.4426950408889634f;
   int rc;
   if (dtype == 1)
     rc = head_dim == 128 ? launch_tc<__nv_bfloat16, 128>(tm, tm_tail, p, batch, stream)
@@ -509,10 +549,10 @@ int blitz_attn_decode(const void* q, int64_t q_stride, const void* kv_layer, con
     dim3 grid(batch, q_heads);
     if (dtype == 1)
       attn_merge_tc_kernel<__nv_bfloat16><<<grid, head_dim, 0, stream>>>(p.part_o, p.part_lse, (__nv_bfloat16*)out,
-                                                                         out_stride, q_heads, head_dim, num_splits);
+                                                                         out_stride, q_heads, head_dim, num_splits, (const __nv_bfloat16*)sink);
     else
       attn_merge_tc_kernel<__half><<<grid, head_dim, 0, stream>>>(p.part_o, p.part_lse, (__half*)out, out_stride,
-                                                                  q_heads, head_dim, num_splits);
+                                                                  q_heads, head_dim, num_splits, (const __half*)sink);
     rc = (int)cudaGetLastError();
   }
   return rc;
@@ -614,6 +654,7 @@ extern "C" int blitz_attn_decode_noalloc(const void* q, int64_t q_stride, const 
   p.batch = batch; p.q_heads = q_heads; p.kv_heads = kv_heads; p.group = G; p.page_size = page_size;
   p.max_pages = max_pages; p.num_splits = num_splits; p.box_tokens = bt; p.tail_box_tokens = bt_tail;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = nullptr;
+  p.window = 0; p.keep_first = 0; p.sink = nullptr; p.cap_scale = p.cap_log2 = 0.f;
   int sms = 0;
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
   if (sms <= 0) sms = 148;
@@ -628,9 +669,9 @@ extern "C" int blitz_attn_decode_noalloc(const void* q, int64_t q_stride, const 
   dim3 grid(batch, q_heads);
   if (dtype == 1)
     attn_merge_tc_kernel<__nv_bfloat16><<<grid, head_dim, 0, stream>>>(p.part_o, p.part_lse, (__nv_bfloat16*)out, out_stride,
-                                                                       q_heads, head_dim, num_splits);
+                                                                       q_heads, head_dim, num_splits, nullptr);
   else
     attn_merge_tc_kernel<__half><<<grid, head_dim, 0, stream>>>(p.part_o, p.part_lse, (__half*)out, out_stride, q_heads,
-                                                                head_dim, num_splits);
+                                                                head_dim, num_splits, nullptr);
   return (int)cudaGetLastError();
 }

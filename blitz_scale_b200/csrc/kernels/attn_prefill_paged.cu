@@ -27,6 +27,13 @@
 // loaded and its first S products issued while the warpgroups still write the previous item's output, so the
 // latency of starting an item (its page ids, its first loads, the first MMA) is paid once per CTA, not per item.
 //
+// Models that ask for it (template parameter EXT) get a sliding window with kept first tokens, soft-capped scores and a
+// per-head sink.  The two tiles of an item then walk the key blocks of the kept tokens and those from the first row's
+// window edge on; blocks in between are never loaded.  A block that is wholly visible to a tile needs no mask.  The cap,
+// cap * tanh(s / cap), is applied to the scores as they turn into probabilities: a polynomial on the FMA pipe where all
+// of a warp's scores of the block stay below 0.9 cap (one vote per block), the special-function unit otherwise; tanh being monotonic, the
+// row maximum is capped alone.  The sink is one more term of the row sum at the end.
+//
 // Replaces FlashInfer's BatchPrefillWithRaggedKVCacheWrapper / paged wrapper calls and their host Plan()
 // (src/kernel/attention_prefill.cu:11-45, src/kernel/flashinfer_types.cu:24-49).
 #include "launch.cuh"
@@ -48,6 +55,9 @@ struct PagedPrefillParams {
   const int32_t* work;          // [entries][kPpWorkInts], heaviest first
   int entries, q_heads, kv_heads, page_size, box_tokens, oob_row;
   float scale_log2;
+  int window, keep_first;     // EXT: a row sees the last `window` positions (0: all) and the first `keep_first`
+  float cap_scale, cap_log2;  // EXT: soft cap (cap_log2 > 0): score in log2 units = cap_log2 * tanh(q.k * cap_scale)
+  const void* sink;           // EXT: [q_heads] in the activation type, or null
   int* status;
   long long* trace;  // profiling aid (null in production): clock stamps of CTA 0's first item, see the set_trace call
 };
@@ -68,9 +78,12 @@ struct PpCfg {
 struct PpItem {
   int seq_start, q_len, pg0, npages, kv_len, prefix, q0, nt, nblk, head, kv_head;
   int nblk_t[2];
+  int n_first, b_window;  // key blocks walked: [0, n_first), then from b_window on
+  __device__ __forceinline__ int block(int j) const { return j < n_first ? j : b_window + j - n_first; }
 };
 // Work item `idx` of the flattened list (entry x q head; the heads of one entry are neighbours, so CTAs that run
 // at the same time share its K and V in L2).
+template <bool EXT>
 __device__ __forceinline__ PpItem pp_item(const PagedPrefillParams& p, int idx) {
   PpItem it;
   const int entry = idx / p.q_heads;
@@ -87,6 +100,15 @@ __device__ __forceinline__ PpItem pp_item(const PagedPrefillParams& p, int idx) 
     const int last = min(it.kv_len, it.prefix + min(it.q_len, it.q0 + kPpTile * (t + 1)));
     it.nblk_t[t] = t < it.nt ? (last + kPpTile - 1) / kPpTile : 0;
   }
+  it.n_first = it.b_window = 0;
+  if (EXT && p.window > 0) {
+    const int lo = max(0, it.prefix + it.q0 - p.window + 1);  // first key in the window of the item's first row
+    it.n_first = (min(p.keep_first, lo) + kPpTile - 1) / kPpTile;
+    it.b_window = max(lo / kPpTile, it.n_first);
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+      if (it.nblk_t[t] > 0) it.nblk_t[t] = it.n_first + max(0, it.nblk_t[t] - it.b_window);
+  }
   it.nblk = max(it.nblk_t[0], it.nblk_t[1]);
   return it;
 }
@@ -97,7 +119,19 @@ __device__ __forceinline__ int pp_index(int r, int total) {
   return idx < total ? idx : -1;
 }
 
-template <typename T, int HD, bool POLY>
+// Odd polynomial for tanh on |x| <= 0.9 (Chebyshev interpolation of tanh(x) / x in x^2): absolute error 1.4e-7.
+constexpr float kTanhPolyMax = 0.9f;
+__device__ __forceinline__ float tanh_poly(float x) {
+  const float y = x * x;
+  float r = fmaf(-0.00366952f, y, 0.01797143f);
+  r = fmaf(r, y, -0.0524757f);
+  r = fmaf(r, y, 0.13306333f);
+  r = fmaf(r, y, -0.33331502f);
+  r = fmaf(r, y, 0.99999979f);
+  return x * r;
+}
+
+template <typename T, int HD, bool POLY, bool EXT>
 __global__ void __launch_bounds__(kPpThreads, 1)
 attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_kv,
                           const PagedPrefillParams p) {
@@ -165,7 +199,7 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
     const int bt = p.box_tokens;
     const bool mine = lane < kPpTile / bt;
     auto box_row = [&](const PpItem& it, int j) {  // this lane's first K row of block j (V: + page_size)
-      const int tok = j * kPpTile + lane * bt;
+      const int tok = it.block(j) * kPpTile + lane * bt;
       const int slot = tok / p.page_size;
       if (!mine || slot >= it.npages) return p.oob_row;  // past the pool: the box arrives as zeros
       return p.page_indices[it.pg0 + slot] * 2 * p.page_size + (tok & (p.page_size - 1));
@@ -189,7 +223,7 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
     for (int r = 0; r * static_cast<int>(gridDim.x) < total && ok; ++r) {
       const int idx = pp_index(r, total);
       if (idx < 0) continue;
-      const PpItem it = pp_item(p, idx);
+      const PpItem it = pp_item<EXT>(p, idx);
       if (n_items > 0) ok = wait(q_empty, (n_items - 1) & 1);  // the previous item's S products have read Q
       if (!ok) break;
       if (lane == 0) {
@@ -250,7 +284,7 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       for (int r = 0; r * static_cast<int>(gridDim.x) < total && ok; ++r) {
         const int idx = pp_index(r, total);
         if (idx < 0) continue;
-        const PpItem it = pp_item(p, idx);
+        const PpItem it = pp_item<EXT>(p, idx);
         const int nb0 = it.nblk_t[0], nb1 = it.nblk_t[1], nblk = it.nblk;
         const bool tr = n_items == 0 && blockIdx.x == 0;
         ok = wait(q_full, n_items & 1) && wait(&k_full[g & 1], (g >> 1) & 1);
@@ -315,7 +349,7 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
     for (int r = 0; r * static_cast<int>(gridDim.x) < total && ok; ++r) {
       const int idx = pp_index(r, total);
       if (idx < 0) continue;
-      const PpItem it = pp_item(p, idx);
+      const PpItem it = pp_item<EXT>(p, idx);
       const int my_blocks = it.nblk_t[t];
       if (my_blocks == 0) continue;  // a short last pair has no second tile
       const bool tracer = first && blockIdx.x == 0 && (warp & 3) == 0 && lane == 0;
@@ -339,11 +373,23 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         ptx::tmem_ld_wait();
         pp_trace(p, tracer, t, j, 2);
         auto score = [&](int i) -> uint32_t& { return i < 32 ? v0[i] : i < 64 ? v1[i - 32] : i < 96 ? v2[i - 64] : v3[i - 96]; };
-        const int kv0 = j * kPpTile;
-        if (kv0 + kPpTile - 1 > it.prefix + it.q0 + t * kPpTile) {  // the block reaches past the tile's first row: mask
+        const int kv0 = it.block(j) * kPpTile;
+        bool masked = false;
+        if (EXT && p.window > 0) {
+          const int row0 = it.prefix + it.q0 + t * kPpTile;  // position of the tile's first row
+          const bool in_window = kv0 + kPpTile - 1 <= row0 && kv0 > row0 + kPpTile - 1 - p.window;
+          masked = !in_window && !(kv0 + kPpTile <= p.keep_first && kv0 + kPpTile - 1 <= row0);
+          if (masked) {
+            const int from = limit - p.window + 1;
+#pragma unroll
+            for (int i = 0; i < kPpTile; ++i)
+              if (kv0 + i > limit || (kv0 + i < from && kv0 + i >= p.keep_first)) score(i) = 0xff800000u;
+          }
+        } else if (kv0 + kPpTile - 1 > it.prefix + it.q0 + t * kPpTile) {  // the block reaches past the tile's first row: mask
 #pragma unroll
           for (int i = 0; i < kPpTile; ++i)
             if (kv0 + i > limit) score(i) = 0xff800000u;  // -inf
+          masked = true;
         }
         // eight independent chains of three-input maxima: with two softmax warps per scheduler nothing else hides a
         // serial one
@@ -359,11 +405,26 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         for (int i = kPpTile - 8; i < kPpTile; ++i) mxs[i & 7] = fmaxf(mxs[i & 7], __uint_as_float(score(i)));
         float mx = fmaxf(ptx::fmax3(mxs[0], mxs[1], mxs[2]), ptx::fmax3(mxs[3], mxs[4], mxs[5]));
         mx = ptx::fmax3(mx, mxs[6], mxs[7]);
-        mx *= p.scale_log2;
+        bool small = false;  // every score of the warp within the range of tanh_poly
+        if (EXT && p.cap_log2 > 0.f) {
+          if (!masked) {
+            float mns[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) mns[i] = __uint_as_float(score(i));
+#pragma unroll
+            for (int i = 8; i < kPpTile; ++i) mns[i & 7] = fminf(mns[i & 7], __uint_as_float(score(i)));
+            const float mn = fminf(fminf(fminf(mns[0], mns[1]), fminf(mns[2], mns[3])),
+                                   fminf(fminf(mns[4], mns[5]), fminf(mns[6], mns[7])));
+            small = __all_sync(0xffffffffu, fmaxf(mx, -mn) * fabsf(p.cap_scale) <= kTanhPolyMax);
+          }
+          mx = mx == -INFINITY ? mx : p.cap_log2 * ptx::tanh_ex2(mx * p.cap_scale);
+        } else {
+          mx *= p.scale_log2;
+        }
         // (S of this block was issued after P V of the previous one, so that product is complete: O_t is stable and
         // the columns P is about to overwrite have been read)
         if (j == 0) {
-          m_ref = (mx == -INFINITY) ? 0.f : mx;
+          m_ref = (!EXT && mx == -INFINITY) ? 0.f : mx;  // EXT: a row may see nothing of its first blocks
         } else {
           const bool grow = mx > m_ref + kPpRescaleAt;
           if (__any_sync(0xffffffffu, grow)) {
@@ -385,21 +446,34 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         pp_trace(p, tracer, t, j, 3);
         // probabilities (16 bit) -> tensor memory over the scores; row sum
         float rs[4] = {0.f, 0.f, 0.f, 0.f};
-        const float neg_m = -m_ref;
+        const float neg_m = (EXT && m_ref == -INFINITY) ? 0.f : -m_ref;
+        auto probabilities = [&](auto&& exponent) {
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {  // 64 scores -> 32 columns of pairs
-          uint32_t pk[32];
+          for (int h = 0; h < 2; ++h) {  // 64 scores -> 32 columns of pairs
+            uint32_t pk[32];
 #pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            const int c = h * 64 + 2 * i;
-            const float x0 = fmaf(__uint_as_float(score(c)), p.scale_log2, neg_m);
-            const float x1 = fmaf(__uint_as_float(score(c + 1)), p.scale_log2, neg_m);
-            const float e0 = ptx::ex2_approx(x0);
-            const float e1 = (POLY && (i & 1)) ? ptx::ex2_poly(x1) : ptx::ex2_approx(x1);
-            rs[i & 3] += e0 + e1;
-            pk[i] = pk2<T>(e0, e1);
+            for (int i = 0; i < 32; ++i) {
+              const int c = h * 64 + 2 * i;
+              const float x0 = exponent(__uint_as_float(score(c)));
+              const float x1 = exponent(__uint_as_float(score(c + 1)));
+              const float e0 = ptx::ex2_approx(x0);
+              const float e1 = (POLY && (i & 1)) ? ptx::ex2_poly(x1) : ptx::ex2_approx(x1);
+              rs[i & 3] += e0 + e1;
+              pk[i] = pk2<T>(e0, e1);
+            }
+            ptx::tmem_st_32x32(tS + h * 32, pk);
           }
-          ptx::tmem_st_32x32(tS + h * 32, pk);
+        };
+        if (EXT && p.cap_log2 > 0.f) {
+          if (small) {
+            probabilities([&](float x) { return fmaf(tanh_poly(x * p.cap_scale), p.cap_log2, neg_m); });
+          } else {
+            probabilities([&](float x) {
+              return x == -INFINITY ? x : fmaf(ptx::tanh_ex2(x * p.cap_scale), p.cap_log2, neg_m);
+            });
+          }
+        } else {
+          probabilities([&](float x) { return fmaf(x, p.scale_log2, neg_m); });
         }
         pp_trace(p, tracer, t, j, 4);
         ptx::tmem_st_wait();
@@ -412,6 +486,8 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       if (!ok) break;
       cnt += my_blocks;
       ptx::tc_fence_after_sync();
+      if (EXT && p.sink != nullptr && l > 0.f)
+        l += ptx::ex2_approx(to_f<T>(reinterpret_cast<const T*>(p.sink)[it.head]) * 1.4426950408889634f - m_ref);
       const float inv = l > 0.f ? 1.f / l : 0.f;
       T* dst = reinterpret_cast<T*>(p.out) + static_cast<int64_t>(it.seq_start + q_idx) * p.out_stride + it.head * HD;
 #pragma unroll 1
@@ -446,16 +522,16 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   }
 }
 
-template <typename T, int HD, bool POLY>
+template <typename T, int HD, bool POLY, bool EXT>
 static int launch_paged_prefill(const CUtensorMap& tq, const CUtensorMap& tkv, const PagedPrefillParams& p, int grid,
                                 cudaStream_t stream) {
   static PerDeviceOnce once;
   cudaError_t e = once.run([] {
-    return cudaFuncSetAttribute(attn_prefill_paged_kernel<T, HD, POLY>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    return cudaFuncSetAttribute(attn_prefill_paged_kernel<T, HD, POLY, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                 PpCfg<HD>::kSmemBytes);
   });
   if (e != cudaSuccess) return (int)e;
-  attn_prefill_paged_kernel<T, HD, POLY><<<grid, kPpThreads, PpCfg<HD>::kSmemBytes, stream>>>(tq, tkv, p);
+  attn_prefill_paged_kernel<T, HD, POLY, EXT><<<grid, kPpThreads, PpCfg<HD>::kSmemBytes, stream>>>(tq, tkv, p);
   return (int)cudaGetLastError();
 }
 
@@ -470,25 +546,27 @@ using namespace blitz;
 // following launch records when its warpgroups and its MMA thread pass each phase of its first work item.
 void blitz_attn_prefill_paged_set_trace(long long* buf) { blitz::g_pp_trace = buf; }
 
-// qkv: [num_tokens, (q_heads + 2 kv_heads) * head_dim] of the current chunk, rotated in place; kv_layer: the
+// q: [num_tokens, q_stride >= q_heads * head_dim] of the current chunk, rotated; kv_layer: the
 // layer's pool [max_pages][2][page_size][kv_heads][head_dim], which already holds the chunk's keys and values;
 // out: [num_tokens, q_heads * head_dim].  page_indices: device array of the sequences' page ids, back to back (the
 // lists cover prefix + chunk).  work: device array (16-byte aligned) of `entries` records of 8 int32, one per
 // (sequence, 256 rows of it), heaviest first: first row of the sequence in qkv, rows of the sequence in this chunk,
 // index of its first page id, number of its pages, tokens cached for it (chunk included), which 256-row pair, 0, 0.
-// page_size: a power of two >= 8.  flags bit 0: compute a quarter of the exponentials on the FMA pipe.
-int blitz_attn_prefill_paged(const void* qkv, const void* kv_layer, void* out, int64_t out_stride,
+// page_size: a power of two >= 8.  flags bit 0: compute a quarter of the exponentials on the FMA pipe (not with a window,
+// cap or sink).  window (0 = none) / keep_first, softcap (0 = none), sink (null = none): see the top of the file.
+int blitz_attn_prefill_paged(const void* q, int64_t q_stride, const void* kv_layer, void* out, int64_t out_stride,
                              const int32_t* page_indices, const int32_t* work, int entries, int num_tokens,
                              int q_heads, int kv_heads, int head_dim, int page_size, int max_pages, float sm_scale,
-                             int flags, int* status, int dtype, cudaStream_t stream) {
+                             int flags, int window, int keep_first, float softcap, const void* sink, int* status,
+                             int dtype, cudaStream_t stream) {
   if (num_tokens <= 0 || entries <= 0) return 0;
-  if ((head_dim != 64 && head_dim != 128) || (q_heads % kv_heads) != 0 || (out_stride & 7)) return -1;
+  if ((head_dim != 64 && head_dim != 128) || (q_heads % kv_heads) != 0 || (out_stride & 7) || (q_stride & 7)) return -1;
+  if (window < 0 || keep_first < 0 || softcap < 0.f) return -1;
   if (page_size < 8 || (page_size & (page_size - 1)) != 0 || work == nullptr) return -1;
   if ((reinterpret_cast<uintptr_t>(work) & 15) != 0) return -1;
-  const uint64_t row = (uint64_t)(q_heads + 2 * kv_heads) * head_dim;
   const int bt = page_size < 64 ? page_size : 64;
   CUtensorMap tq, tkv;
-  if (!get_tmap_2d(&tq, qkv, row, (uint64_t)num_tokens, row * 2, 64, kPpTile)) return -2;
+  if (!get_tmap_2d(&tq, q, (uint64_t)q_heads * head_dim, (uint64_t)num_tokens, (uint64_t)q_stride * 2, 64, kPpTile)) return -2;
   if (!get_tmap_3d(&tkv, kv_layer, (uint64_t)head_dim, (uint64_t)kv_heads, (uint64_t)max_pages * 2 * page_size,
                    (uint64_t)head_dim * 2, (uint64_t)kv_heads * head_dim * 2, 64, 1, (uint32_t)bt))
     return -2;
@@ -497,22 +575,24 @@ int blitz_attn_prefill_paged(const void* qkv, const void* kv_layer, void* out, i
   p.q_heads = q_heads; p.kv_heads = kv_heads; p.page_size = page_size; p.box_tokens = bt;
   p.oob_row = max_pages * 2 * page_size;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = g_pp_trace;
+  p.window = window; p.keep_first = keep_first; p.sink = sink;
+  p.cap_scale = softcap > 0.f ? sm_scale / softcap : 0.f; p.cap_log2 = softcap * 1.4426950408889634f;
   const long long total = (long long)entries * q_heads;
   const int sms = device_sm_count();
   const int grid = (int)(total < sms ? total : sms);
-  const bool poly = (flags & 1) != 0;
-  if (dtype == 1) {
-    if (head_dim == 128)
-      return poly ? launch_paged_prefill<__nv_bfloat16, 128, true>(tq, tkv, p, grid, stream)
-                  : launch_paged_prefill<__nv_bfloat16, 128, false>(tq, tkv, p, grid, stream);
-    return poly ? launch_paged_prefill<__nv_bfloat16, 64, true>(tq, tkv, p, grid, stream)
-                : launch_paged_prefill<__nv_bfloat16, 64, false>(tq, tkv, p, grid, stream);
-  }
-  if (head_dim == 128)
-    return poly ? launch_paged_prefill<__half, 128, true>(tq, tkv, p, grid, stream)
-                : launch_paged_prefill<__half, 128, false>(tq, tkv, p, grid, stream);
-  return poly ? launch_paged_prefill<__half, 64, true>(tq, tkv, p, grid, stream)
-              : launch_paged_prefill<__half, 64, false>(tq, tkv, p, grid, stream);
+  const bool poly = (flags & 1) != 0, ext = window > 0 || softcap > 0.f || sink != nullptr;
+  auto launch = [&](auto type) {
+    using T = decltype(type);
+    if (ext)
+      return head_dim == 128 ? launch_paged_prefill<T, 128, false, true>(tq, tkv, p, grid, stream)
+                             : launch_paged_prefill<T, 64, false, true>(tq, tkv, p, grid, stream);
+    if (poly)
+      return head_dim == 128 ? launch_paged_prefill<T, 128, true, false>(tq, tkv, p, grid, stream)
+                             : launch_paged_prefill<T, 64, true, false>(tq, tkv, p, grid, stream);
+    return head_dim == 128 ? launch_paged_prefill<T, 128, false, false>(tq, tkv, p, grid, stream)
+                           : launch_paged_prefill<T, 64, false, false>(tq, tkv, p, grid, stream);
+  };
+  return dtype == 1 ? launch(__nv_bfloat16{}) : launch(__half{});
 }
 
 }  // extern "C"

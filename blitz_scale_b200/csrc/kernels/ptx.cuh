@@ -357,6 +357,11 @@ __device__ __forceinline__ float ex2_poly(float x) {
   return __int_as_float(__float_as_int(p) + (__float_as_int(t) << 23));
 }
 
+// tanh x = 1 - 2 / (e^(2x) + 1) on the special-function unit: absolute error of a few 1e-7, exact limits at +-inf.
+__device__ __forceinline__ float tanh_ex2(float x) {
+  return 1.f - __fdividef(2.f, ex2_approx(x * 2.8853900817779268f) + 1.f);
+}
+
 // Shared-memory operand descriptor for UMMA (sm_100 format, version field = 1).
 //   start address, leading-dimension byte offset and stride byte offset are
 //   stored without their 4 LSBs; layout 2 = 128-byte swizzle.

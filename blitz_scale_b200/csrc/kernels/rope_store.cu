@@ -41,8 +41,9 @@ __global__ void rope_store_kernel(const RopeStoreParams p) {
     const float err = fmaf(pos, f.x, -a) + pos * f.y;
     float sn, cs;
     sincosf(a, &sn, &cs);
-    s_ang[i] = cs - err * sn;
-    s_ang[half + i] = sn + err * cs;
+    const float c_err = 1.f - 0.5f * err * err;  // cos and sin of the small angle `err`, to second order
+    s_ang[i] = cs * c_err - err * sn;
+    s_ang[half + i] = sn * c_err + err * cs;
   }
   __syncthreads();
   int s = p.slot[t];

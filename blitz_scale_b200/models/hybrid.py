@@ -57,6 +57,7 @@ class HybridRunner:
             if m.kind == "attention" and (m.rot_dims, m.rot_base) not in self._freqs:
                 self._freqs[(m.rot_dims, m.rot_base)] = ops.rope_freqs(m.rot_dims, m.rot_base, dev)
         self._ws: Optional[torch.Tensor] = None
+        self._ws_old: List[Optional[torch.Tensor]] = []
 
     @staticmethod
     def _mid_key(s: LayerSpec) -> tuple:
@@ -94,10 +95,29 @@ class HybridRunner:
         ops.rope_store(p["q"], p["k"], p.get("v"), m.pos, m.slot, kv, self._freqs[(mx.rot_dims, mx.rot_base)],
                        q_heads=mx.heads, kv_heads=mx.kv_heads, dim=mx.dim, rot_dims=mx.rot_dims, page_size=self.page_size,
                        interleaved=mx.interleaved)
-        ops.attn_ragged(p["q"], kv, m.pos, m.tok_indptr if m.is_prefill else None, m.page_indptr, m.page_indices, mid,
-                        q_heads=mx.heads, kv_heads=mx.kv_heads, dim=mx.dim, page_size=self.page_size, scale=mx.scale,
-                        window=mx.window, keep_first=mx.keep_first, softcap=mx.softcap,
-                        sink=self._w(l, "sink") if mx.sink else None)
+        extra = dict(window=mx.window, keep_first=mx.keep_first, softcap=mx.softcap,
+                     sink=self._w(l, "sink") if mx.sink else None)
+        if not ops.attn_tensor_core(p["q"], mx.heads, mx.kv_heads, mx.dim, self.page_size):
+            ops.attn_ragged(p["q"], kv, m.pos, m.tok_indptr if m.is_prefill else None, m.page_indptr, m.page_indices, mid,
+                            q_heads=mx.heads, kv_heads=mx.kv_heads, dim=mx.dim, page_size=self.page_size, scale=mx.scale, **extra)
+            return
+        args = dict(q_heads=mx.heads, kv_heads=mx.kv_heads, head_dim=mx.dim, page_size=self.page_size, sm_scale=mx.scale, **extra)
+        ns = m.singles if m.is_prefill else m.batch
+        if ns:
+            ops.attn_decode(p["q"][:ns], kv, m.page_indices, m.page_indptr[:ns + 1], m.last_page_len[:ns],
+                            num_splits=m.num_splits, workspace=self._workspace(ns, mx, m.num_splits), out=mid[:ns], **args)
+        if m.batch > ns:
+            ops.attn_prefill_paged(p["q"], kv, m.page_indices, m.prefill_work, out=mid, **args)
+
+    def _workspace(self, B: int, mx: AttentionMixer, splits: int) -> Optional[torch.Tensor]:
+        if splits <= 1:
+            return None
+        n = ops.attn_decode_workspace_bytes(B, mx.heads, mx.dim, splits)
+        if self._ws is None or self._ws.numel() < n:
+            # an earlier buffer may be named by captured graphs: keep it
+            self._ws_old.append(self._ws)
+            self._ws = torch.empty(n, dtype=torch.uint8, device=self.res.device)
+        return self._ws
 
     def _gla(self, r: int, l: int, mx: GLAMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta) -> None:
         ns = m.batch if not m.is_prefill else m.singles

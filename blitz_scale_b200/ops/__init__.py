@@ -307,8 +307,11 @@ def attn_decode_workspace_bytes(batch: int, q_heads: int, head_dim: int, num_spl
 def attn_decode(q: torch.Tensor, kv_layer: torch.Tensor, indices: torch.Tensor, indptr: torch.Tensor,
                 last_page_len: torch.Tensor, *, q_heads: int, kv_heads: int, head_dim: int, page_size: int,
                 num_splits: int = 1, workspace: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
-                sm_scale: Optional[float] = None) -> torch.Tensor:
-    """q: [batch, >= q_heads*head_dim] (row pitch free, e.g. a view of the fused qkv buffer)."""
+                sm_scale: Optional[float] = None, window: int = 0, keep_first: int = 0, softcap: float = 0.0,
+                sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """q: [batch, >= q_heads*head_dim] (row pitch free, e.g. a view of the fused qkv buffer).  ``window`` > 0: only the
+    last that many positions and the first ``keep_first`` are visible (and read); ``softcap`` > 0:
+    scores are cap * tanh(score / cap); ``sink`` [q_heads]: a term e^sink in the softmax denominator."""
     B = indptr.numel() - 1
     if out is None:
         out = torch.empty((B, q_heads * head_dim), dtype=q.dtype, device=q.device)
@@ -319,9 +322,15 @@ def attn_decode(q: torch.Tensor, kv_layer: torch.Tensor, indices: torch.Tensor, 
         sm_scale = head_dim ** -0.5
     _check(lib().blitz_attn_decode(_p(q), q.stride(0), _p(kv_layer), _p(indices), _p(indptr), _p(last_page_len),
                                    _p(out), out.stride(0), _p(workspace), B, q_heads, kv_heads, head_dim, page_size,
-                                   kv_layer.shape[0], num_splits, sm_scale, _p(status_word(q.device)), _dt(q),
-                                   _stream()), "blitz_attn_decode")
+                                   kv_layer.shape[0], num_splits, sm_scale, window, keep_first, softcap, _p(sink),
+                                   _p(status_word(q.device)), _dt(q), _stream()), "blitz_attn_decode")
     return out
+
+
+def attn_tensor_core(q: torch.Tensor, q_heads: int, kv_heads: int, head_dim: int, page_size: int) -> bool:
+    """Whether attn_decode and attn_prefill_paged take this head shape (attn_ragged takes every one)."""
+    return (q.dtype in _DT and head_dim in (64, 128) and q_heads // kv_heads <= 8 and page_size >= 8
+            and page_size & (page_size - 1) == 0 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0)
 
 
 def prefill_work_list(q_lens, kv_lens, page_size: int, device, skip: int = 0) -> torch.Tensor:
@@ -343,23 +352,25 @@ def prefill_work_list(q_lens, kv_lens, page_size: int, device, skip: int = 0) ->
     return torch.tensor(rec, dtype=torch.int32).reshape(-1, 8).to(device, non_blocking=True)
 
 
-def attn_prefill_paged(qkv: torch.Tensor, kv_layer: torch.Tensor, page_indices: torch.Tensor, work: torch.Tensor, *,
+def attn_prefill_paged(q: torch.Tensor, kv_layer: torch.Tensor, page_indices: torch.Tensor, work: torch.Tensor, *,
                        q_heads: int, kv_heads: int, head_dim: int, page_size: int, out: Optional[torch.Tensor] = None,
-                       sm_scale: Optional[float] = None, poly_exp: bool = False) -> torch.Tensor:
+                       sm_scale: Optional[float] = None, poly_exp: bool = False, window: int = 0, keep_first: int = 0,
+                       softcap: float = 0.0, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of the pass's rows over the paged cache (which already holds the rows' own keys and values,
-    after whatever earlier passes stored).  ``qkv`` rotated (rope_kv_store); ``page_indices``: the sequences' page
-    ids back to back, covering prefix + rows; ``work`` from `prefill_work_list` for the same sequences."""
-    T = qkv.shape[0]
+    after whatever earlier passes stored).  ``q``: rotated query columns, e.g. the fused qkv buffer (rope_kv_store);
+    ``page_indices``: the sequences' page ids back to back, covering prefix + rows; ``work`` from `prefill_work_list`
+    for the same sequences.  ``window`` / ``keep_first`` / ``softcap`` / ``sink`` as for `attn_decode`."""
+    T = q.shape[0]
     if out is None:
-        out = torch.empty((T, q_heads * head_dim), dtype=qkv.dtype, device=qkv.device)
+        out = torch.empty((T, q_heads * head_dim), dtype=q.dtype, device=q.device)
     if sm_scale is None:
         sm_scale = head_dim ** -0.5
     assert work.dtype == torch.int32 and work.dim() == 2 and work.shape[1] == 8 and work.is_contiguous()
     max_pages = kv_layer.shape[0]
-    _check(lib().blitz_attn_prefill_paged(_p(qkv), _p(kv_layer), _p(out), out.stride(0), _p(page_indices), _p(work),
-                                          work.shape[0], T, q_heads, kv_heads, head_dim, page_size, max_pages, sm_scale,
-                                          1 if poly_exp else 0, _p(status_word(qkv.device)), _dt(qkv), _stream()),
-           "blitz_attn_prefill_paged")
+    _check(lib().blitz_attn_prefill_paged(_p(q), q.stride(0), _p(kv_layer), _p(out), out.stride(0), _p(page_indices),
+                                          _p(work), work.shape[0], T, q_heads, kv_heads, head_dim, page_size, max_pages,
+                                          sm_scale, 1 if poly_exp else 0, window, keep_first, softcap, _p(sink),
+                                          _p(status_word(q.device)), _dt(q), _stream()), "blitz_attn_prefill_paged")
     return out
 
 
@@ -455,3 +466,10 @@ def rglru_scan(u, gates: torch.Tensor, gate_b, lam, y, x, y_b, state: torch.Tens
                                   seq_slot.numel(), width, block, hist.shape[1] + 1, slots, int(tok_indptr is None),
                                   _p(status_word(u.device)), _dt3(u), _stream()), "blitz_rglru_scan")
     return out
+
+
+def gla(q, k, v, g, low, a2, a2_b, norm, state: torch.Tensor, out: torch.Tensor, pos, tok_indptr, seq_slot, *, rank: int,
+        tau: float, eps: float, row_lens=None) -> torch.Tensor:
+    """Gated linear attention over the rows of a step; ``row_lens``: tokens per row (host), needed where rows are longer
+    than one token."""
+    return gla_recurrent(q, k, v, g, low, a2, a2_b, norm, state, out, pos, tok_indptr, seq_slot, rank=rank, tau=tau, eps=eps)

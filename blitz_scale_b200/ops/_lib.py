@@ -87,9 +87,9 @@ def _declare(L: ctypes.CDLL) -> None:
     sig("blitz_rope_kv_store", [c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_p, c_i, c_p])
     sig("blitz_attn_decode_workspace_bytes", [c_i, c_i, c_i, c_i], c_i64)
     sig("blitz_attn_decode", [c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f,
-                              c_p, c_i, c_p])
-    sig("blitz_attn_prefill_paged", [c_p, c_p, c_p, c_i64, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p,
-                                     c_i, c_p])
+                              c_i, c_i, c_f, c_p, c_p, c_i, c_p])
+    sig("blitz_attn_prefill_paged", [c_p, c_i64, c_p, c_p, c_i64, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i,
+                                     c_i, c_i, c_f, c_p, c_p, c_i, c_p])
     # models with an fp32 residual stream and recurrent layers
     sig("blitz_gemm_simt", [c_p, c_i64, c_p, c_i64, c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_p])
     sig("blitz_stream_norm", [c_p, c_p, c_p, c_p, c_i, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_p, c_i, c_p])

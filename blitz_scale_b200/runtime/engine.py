@@ -299,7 +299,8 @@ class Engine:
             if src:
                 got = self.runner.logits[torch.tensor([row_of[b] for b, _ in src], device=self.device)].float()
         else:
-            m = self._views(T, rows, P, True, q_lens, kv_lens=kv_lens, singles=singles)
+            splits = self.choose_splits(singles, max(kv_lens[:singles])) if singles else 1
+            m = self._views(T, rows, P, True, q_lens, splits=splits, kv_lens=kv_lens, singles=singles)
             with nvtx_range("step"):
                 self.runner.forward(m, with_head=False)
                 starts = [sum(q_lens[:r]) for r in range(rows)]

@@ -335,7 +335,8 @@ def test_attn_decode_simt_matches_tc(ops):
     a = ops.attn_decode(q, kv, idx, indptr, last, q_heads=8, kv_heads=2, head_dim=128, page_size=16)
     b = torch.empty_like(a)
     L = ops.lib()
-    L.blitz_attn_decode_simt.argtypes = L.blitz_attn_decode.argtypes
+    p_, i_ = ctypes.c_void_p, ctypes.c_int
+    L.blitz_attn_decode_simt.argtypes = [p_, ctypes.c_int64, p_, p_, p_, p_, p_, ctypes.c_int64, p_] + [i_] * 7 + [ctypes.c_float, p_, i_, p_]
     rc = L.blitz_attn_decode_simt(q.data_ptr(), q.stride(0), kv.data_ptr(), idx.data_ptr(), indptr.data_ptr(),
                                   last.data_ptr(), b.data_ptr(), b.stride(0), None, 3, 8, 2, 128, 16, kv.shape[0], 1,
                                   128 ** -0.5, None, 1, ctypes.c_void_p(torch.cuda.current_stream().cuda_stream))
