@@ -1,0 +1,509 @@
+// Gated linear attention of prompts, in chunks on the tensor cores (bf16 activations, fp32 state; gla.cu has the
+// recurrence itself and serves single tokens and everything this kernel does not take).
+//
+// With b_t the running sum of the log decays within a chunk of 64 tokens (per key channel, b <= 0 and falling):
+//
+//   o_t   = (q_t e^(b_t))^T S_0 + sum_{s <= t} (sum_c q_tc k_sc e^(b_tc - b_sc)) v_s
+//   S_end = diag(e^(b_end)) S_0 + sum_s (k_s e^(b_end - b_s)) v_s^T
+//
+// (the chunkwise form of Yang, Wang, Shen, Panda and Kim, "Gated Linear Attention Transformers with Hardware-Efficient
+// Training").  e^(b_t - b_s) must be split between q and k to become a matrix product, and e^(-b_s) alone overflows for
+// fast decays, so the chunk is cut into four blocks of 16 tokens with r_i = b at the end of block i - 1 (r_0 = 0):
+//
+//   q'_t = q_t e^(b_t - r_i),  t in block i          <= |q|
+//   k~_s = k_s e^(r_(j+1) - b_s),  s in block j      <= |k|
+//
+// and every product takes the factor between two block borders from a table: block (i, j < i) scales k~ by
+// e^(r_i - r_(j+1)) <= 1, the state term scales q' by e^(r_i), the state update scales k~ by e^(b_end - r_(j+1)).  Only
+// within one block is the factor e^(r_i - r_(i+1)) >= 1; when a channel decays by more than e^-80 within 16 tokens, which
+// that form cannot hold, the block's 136 scores are computed one by one from the unscaled inputs.
+//
+// 32-bit arithmetic where the design asks for it: decays, their sums and exponentials and the state are fp32, and the
+// products that involve them split their fp32 operands into two bf16 numbers (x = hi + lo, relative error 2^-17) and
+// drop only the lo * lo term.
+//
+// A block of 8 warps owns (row, head, 64 value columns) and walks the row's chunks with the state in registers; the
+// blocks of one head form a thread-block cluster, which exchanges the 64 partial sums of squares per chunk through
+// distributed shared memory, so that the output norm and the gate are applied here and nothing but the result is
+// written.  (gla_decay_kernel computes b beforehand: every value block of a head needs it.)
+#include "launch.cuh"
+#include "mma.cuh"
+#include "ptx.cuh"
+#include "scalar.cuh"
+
+namespace blitz {
+
+constexpr int kGcC = 64;        // tokens per chunk
+constexpr int kGcB = 16;        // tokens per block
+constexpr int kGcV = 64;        // value columns per CTA
+constexpr int kGcThreads = 256;
+constexpr int kGcMaxCluster = 8;
+constexpr float kGcMaxDecay = 80.f;
+
+struct GlaChunkParams {
+  const __nv_bfloat16 *q, *k, *v, *g, *low;
+  int64_t row;
+  const __nv_bfloat16 *a2, *a2_b, *norm;
+  float* cum;      // [tokens][heads * dim]: running sums of the log decays within each chunk
+  float* state;    // [slots][heads][dim][vdim]
+  __nv_bfloat16* out;
+  int64_t out_stride;
+  const int32_t *pos, *tok_indptr, *seq_slot;
+  int heads, dim, vdim, rank, num_slots;
+  float q_scale, inv_tau, eps;
+  int* status;
+};
+
+// Running sum of log(sigmoid(low a2 + b)) / tau over a chunk; a thread per channel.
+constexpr int kGdThreads = 128;
+__global__ void __launch_bounds__(kGdThreads) gla_decay_kernel(const GlaChunkParams p) {
+  ptx::griddep_launch_dependents();
+  ptx::griddep_wait();
+  extern __shared__ float s_low[];  // [64][rank]
+  const int r = blockIdx.z, hk = p.heads * p.dim;
+  const int t0 = p.tok_indptr[r] + blockIdx.y * kGcC, n = min(kGcC, p.tok_indptr[r + 1] - t0);
+  if (n <= 0) return;
+  for (int i = threadIdx.x; i < n * p.rank; i += kGdThreads)
+    s_low[i] = ldf(p.low + static_cast<int64_t>(t0 + i / p.rank) * p.row + i % p.rank);
+  __syncthreads();
+  const int c = blockIdx.x * kGdThreads + threadIdx.x;
+  if (c >= hk) return;
+  constexpr int kKeep = 16;  // coefficients kept in registers
+  float w[kKeep];
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) w[i] = i < p.rank ? ldf(p.a2 + static_cast<int64_t>(i) * hk + c) : 0.f;
+  const float bias = ldf(p.a2_b + c);
+  float sum = 0.f;
+  for (int t = 0; t < n; ++t) {
+    const float* low = s_low + t * p.rank;
+    float z = bias;
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i)
+      if (i < p.rank) z += low[i] * w[i];
+    for (int i = kKeep; i < p.rank; ++i) z += low[i] * ldf(p.a2 + static_cast<int64_t>(i) * hk + c);
+    sum += log_sigmoid(z) * p.inv_tau;
+    p.cum[static_cast<int64_t>(t0 + t) * hk + c] = sum;
+  }
+}
+
+// x = hi + lo in bf16, two neighbours at a time
+__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
+  hi = pk2<__nv_bfloat16>(x, y);
+  const float2 h = cvt2<__nv_bfloat16>(hi);
+  lo = pk2<__nv_bfloat16>(x - h.x, y - h.y);
+}
+
+template <int DK>
+struct GcSmem {
+  static constexpr int kQ = DK + 8;       // row pitch of q' (bf16)
+  static constexpr int kK = DK + 8;       // row pitch of k~ (fp32)
+  static constexpr int kV = kGcV + 8;     // row pitch of v, S, A (bf16)
+  static constexpr int kParts = kGcMaxCluster;
+  float k[kGcC * kK];
+  float ref[5 * DK];                      // r_0 .. r_4 (r_4 = b_end)
+  float ss[2][kParts][kGcC];              // partial sums of squares of every cluster rank, by parity of the chunk
+  float part[2][kGcC];
+  int wide[4];                            // block whose decay the factored form cannot hold
+  __nv_bfloat16 qh[kGcC * kQ], ql[kGcC * kQ];
+  __nv_bfloat16 v[kGcC * kV];
+  __nv_bfloat16 ah[kGcC * kV], al[kGcC * kV];
+  __nv_bfloat16 sh[DK * kV], sl[DK * kV];
+};
+
+template <int DK>
+__global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunkParams p) {
+  using bf = __nv_bfloat16;
+  using SM = GcSmem<DK>;
+  constexpr int RB = DK / 16;             // 16-row blocks of the state
+  constexpr int CP = 8 / RB;              // warps that share a row block of it
+  constexpr int NT = kGcV / CP / 8;       // 8-column tiles of the state per warp
+  constexpr int NV = kGcC * DK / 8 / kGcThreads;  // vectors of 8 q (k, b) elements per thread
+  static_assert(RB * CP == 8 && NV >= 1, "DK is 32, 64 or 128");
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  SM& sm = *reinterpret_cast<SM*>(smem_raw);
+  ptx::griddep_launch_dependents();
+  ptx::griddep_wait();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int mi = lane >> 3, mr = lane & 7;
+  const int h = blockIdx.y, r = blockIdx.z, nrank = gridDim.x, rank = blockIdx.x;
+  const int v0 = blockIdx.x * kGcV, nv = min(kGcV, p.vdim - v0);
+  const int slot = p.seq_slot[r];
+  const int t_beg = p.tok_indptr[r], len = p.tok_indptr[r + 1] - t_beg;
+  const int hk = p.heads * p.dim;
+  // the CTAs of a cluster have the same row: they take the same way out
+  if (slot < 0 || slot >= p.num_slots || len <= 0) {
+    if (slot >= p.num_slots && tid == 0 && p.status) atomicCAS(p.status, 0, kStatusBadIndex);
+    return;
+  }
+  ptx::cluster_arrive_release();  // every CTA of the cluster runs: its shared memory may be written
+  ptx::cluster_wait_acquire();
+  const int rbS = warp % RB, cS = (warp / RB) * (kGcV / CP);  // this warp's part of the state
+  const int rowS = rbS * 16 + g;
+  float* gstate = p.state + (static_cast<int64_t>(slot) * p.heads + h) * p.dim * p.vdim + v0;
+  float S[NT][4];
+  const bool fresh = p.pos[t_beg] == 0;
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int c = rowS + (e >> 1) * 8, col = cS + n * 8 + 2 * t4 + (e & 1);
+      S[n][e] = (fresh || c >= p.dim || col >= nv) ? 0.f : gstate[static_cast<int64_t>(c) * p.vdim + col];
+    }
+  auto publish_state = [&] {
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+      const int at = rowS * SM::kV + cS + n * 8 + 2 * t4;
+      uint32_t hi, lo;
+      split2(S[n][0], S[n][1], hi, lo);
+      *reinterpret_cast<uint32_t*>(sm.sh + at) = hi;
+      *reinterpret_cast<uint32_t*>(sm.sl + at) = lo;
+      split2(S[n][2], S[n][3], hi, lo);
+      *reinterpret_cast<uint32_t*>(sm.sh + at + 8 * SM::kV) = hi;
+      *reinterpret_cast<uint32_t*>(sm.sl + at + 8 * SM::kV) = lo;
+    }
+  };
+  publish_state();
+  const int rb = warp >> 1, cO = (warp & 1) * 32;  // this warp's 16 x 32 part of the chunk's output
+  const int nchunks = (len + kGcC - 1) / kGcC;
+
+  // q, k and v of a chunk, requested one chunk ahead
+  uint4 rq[NV], rk[NV], rv[2];
+  auto request = [&](int chunk) {
+    const int base = chunk * kGcC;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int e = tid + i * kGcThreads, t = base + e / (DK / 8), c = (e % (DK / 8)) * 8;
+      rq[i] = rk[i] = make_uint4(0, 0, 0, 0);
+      if (t < len && c < p.dim) {
+        const int64_t at = static_cast<int64_t>(t_beg + t) * p.row + h * p.dim + c;
+        rq[i] = *reinterpret_cast<const uint4*>(p.q + at);
+        rk[i] = *reinterpret_cast<const uint4*>(p.k + at);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int e = tid + i * kGcThreads, t = base + e / 8, c = (e % 8) * 8;
+      rv[i] = make_uint4(0, 0, 0, 0);
+      if (t < len && c < nv)
+        rv[i] = *reinterpret_cast<const uint4*>(p.v + static_cast<int64_t>(t_beg + t) * p.row + h * p.vdim + v0 + c);
+    }
+  };
+  request(0);
+
+  for (int ch = 0; ch < nchunks; ++ch) {
+    const int base = ch * kGcC, n_tok = min(kGcC, len - base);
+    // b at token t of the chunk (tokens past the end do not decay)
+    const float* cum = p.cum + static_cast<int64_t>(t_beg + base) * hk + h * p.dim;
+    auto b_at = [&](int t) { return cum + static_cast<int64_t>(min(t, n_tok - 1)) * hk; };
+    // ---- 1. q', k~, v and the block borders' table into shared memory
+    if (tid < 4) sm.wide[tid] = 0;
+    for (int e = tid; e < 5 * DK; e += kGcThreads) {
+      const int i = e / DK, c = e % DK;
+      sm.ref[e] = (i == 0 || c >= p.dim) ? 0.f : b_at(i * kGcB - 1)[c];
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int e = tid + i * kGcThreads, t = e / (DK / 8), c = (e % (DK / 8)) * 8, blk = t / kGcB;
+      float q8[8], k8[8];
+      unpack8<bf>(rq[i], q8);
+      unpack8<bf>(rk[i], k8);
+      if (c < p.dim) {
+        float b8[8], lo8[8], hi8[8];
+        ldf8(b_at(t) + c, b8);
+        ldf8(b_at(blk * kGcB + kGcB - 1) + c, hi8);
+        if (blk > 0) ldf8(b_at(blk * kGcB - 1) + c, lo8);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          q8[j] *= p.q_scale * __expf(b8[j] - (blk > 0 ? lo8[j] : 0.f));
+          k8[j] *= __expf(hi8[j] - b8[j]);
+        }
+      }
+      uint4 hi, lo;
+      split2(q8[0], q8[1], hi.x, lo.x);
+      split2(q8[2], q8[3], hi.y, lo.y);
+      split2(q8[4], q8[5], hi.z, lo.z);
+      split2(q8[6], q8[7], hi.w, lo.w);
+      *reinterpret_cast<uint4*>(sm.qh + t * SM::kQ + c) = hi;
+      *reinterpret_cast<uint4*>(sm.ql + t * SM::kQ + c) = lo;
+      *reinterpret_cast<float4*>(sm.k + t * SM::kK + c) = make_float4(k8[0], k8[1], k8[2], k8[3]);
+      *reinterpret_cast<float4*>(sm.k + t * SM::kK + c + 4) = make_float4(k8[4], k8[5], k8[6], k8[7]);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int e = tid + i * kGcThreads;
+      *reinterpret_cast<uint4*>(sm.v + (e / 8) * SM::kV + (e % 8) * 8) = rv[i];
+    }
+    __syncthreads();
+    for (int e = tid; e < 4 * DK; e += kGcThreads)
+      if (sm.ref[e] - sm.ref[e + DK] > kGcMaxDecay) sm.wide[e / DK] = 1;
+    if (ch + 1 < nchunks) request(ch + 1);
+    __syncthreads();
+
+    // ---- 2. scores within the chunk: ten 16 x 16 tiles on and below the diagonal
+    for (int tile = warp; tile < 10; tile += 8) {
+      // 0..5: (1,0) (2,0) (2,1) (3,0) (3,1) (3,2); 6..9: the diagonal
+      const int i = tile >= 6 ? tile - 6 : (tile >= 3 ? 3 : tile >= 1 ? 2 : 1);
+      const int j = tile >= 6 ? i : (tile >= 3 ? tile - 3 : tile >= 1 ? tile - 1 : 0);
+      float acc[2][4];
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
+      if (i == j && sm.wide[i]) {
+        // one score at a time: entry e of the fragment
+#pragma unroll 1
+        for (int e = 0; e < 8; ++e) {
+          const int t = i * kGcB + g + ((e >> 1) & 1) * 8, s = i * kGcB + (e >> 2) * 8 + 2 * t4 + (e & 1);
+          float x = 0.f;
+          if (s <= t && t < n_tok) {
+            const bf* qr = p.q + static_cast<int64_t>(t_beg + base + t) * p.row + h * p.dim;
+            const bf* kr = p.k + static_cast<int64_t>(t_beg + base + s) * p.row + h * p.dim;
+            const float *bt = b_at(t), *bs = b_at(s);
+            for (int c = 0; c < p.dim; ++c) x += ldf(qr + c) * ldf(kr + c) * __expf(bt[c] - bs[c]);
+            x *= p.q_scale;
+          }
+#pragma unroll
+          for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int f = 0; f < 4; ++f)
+              if (n * 4 + f == e) acc[n][f] = x;
+        }
+      } else {
+        const float *ri = sm.ref + i * DK, *rj = sm.ref + (j + 1) * DK;
+#pragma unroll
+        for (int kk = 0; kk < DK / 16; ++kk) {
+          const uint32_t off = static_cast<uint32_t>((i * kGcB + (mi & 1) * 8 + mr) * SM::kQ + kk * 16 + (mi >> 1) * 8);
+          uint32_t ah[4], al[4];
+          ldmatrix_x4(ptx::smem_u32(sm.qh + off), ah[0], ah[1], ah[2], ah[3]);
+          ldmatrix_x4(ptx::smem_u32(sm.ql + off), al[0], al[1], al[2], al[3]);
+          float f[4];  // factors of channels 2 t4, + 1, + 8, + 9
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int c = kk * 16 + 2 * t4 + (e >> 1) * 8 + (e & 1);
+            f[e] = __expf(ri[c] - rj[c]);
+          }
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            const float* kr = sm.k + (j * kGcB + n * 8 + g) * SM::kK + kk * 16 + 2 * t4;
+            const float2 x = *reinterpret_cast<const float2*>(kr), y = *reinterpret_cast<const float2*>(kr + 8);
+            uint32_t bh0, bl0, bh1, bl1;
+            split2(x.x * f[0], x.y * f[1], bh0, bl0);
+            split2(y.x * f[2], y.y * f[3], bh1, bl1);
+            mma16816<bf>(acc[n], ah[0], ah[1], ah[2], ah[3], bh0, bh1);
+            mma16816<bf>(acc[n], ah[0], ah[1], ah[2], ah[3], bl0, bl1);
+            mma16816<bf>(acc[n], al[0], al[1], al[2], al[3], bh0, bh1);
+          }
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int t = g + half * 8, s = n * 8 + 2 * t4;
+          float x = acc[n][2 * half], y = acc[n][2 * half + 1];
+          if (i == j) {  // above the diagonal (a factored score may be anything there)
+            if (s > t) x = 0.f;
+            if (s + 1 > t) y = 0.f;
+          }
+          uint32_t hi, lo;
+          split2(x, y, hi, lo);
+          const int at = (i * kGcB + t) * SM::kV + j * kGcB + s;
+          *reinterpret_cast<uint32_t*>(sm.ah + at) = hi;
+          *reinterpret_cast<uint32_t*>(sm.al + at) = lo;
+        }
+    }
+    __syncthreads();
+
+    // ---- 3. output: state term, then the chunk's own values
+    float O[4][4];
+#pragma unroll
+    for (int n = 0; n < 4; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) O[n][e] = 0.f;
+    {
+      const float* ri = sm.ref + rb * DK;
+#pragma unroll
+      for (int kk = 0; kk < DK / 16; ++kk) {
+        const uint32_t off = static_cast<uint32_t>((rb * kGcB + (mi & 1) * 8 + mr) * SM::kQ + kk * 16 + (mi >> 1) * 8);
+        uint32_t ah[4], al[4];
+        ldmatrix_x4(ptx::smem_u32(sm.qh + off), ah[0], ah[1], ah[2], ah[3]);
+        ldmatrix_x4(ptx::smem_u32(sm.ql + off), al[0], al[1], al[2], al[3]);
+        float f[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) f[e] = __expf(ri[kk * 16 + 2 * t4 + (e >> 1) * 8 + (e & 1)]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {  // fragments 0, 1: channels 2 t4, + 1; 2, 3: + 8, + 9
+          const float2 a = cvt2<bf>(ah[e]), b = cvt2<bf>(al[e]);
+          split2((a.x + b.x) * f[(e >> 1) * 2], (a.y + b.y) * f[(e >> 1) * 2 + 1], ah[e], al[e]);
+        }
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+          const uint32_t at = static_cast<uint32_t>((kk * 16 + (mi & 1) * 8 + mr) * SM::kV + cO + m * 16 + (mi >> 1) * 8);
+          uint32_t b0, b1, b2, b3, d0, d1, d2, d3;
+          ldmatrix_x4_trans(ptx::smem_u32(sm.sh + at), b0, b1, b2, b3);
+          ldmatrix_x4_trans(ptx::smem_u32(sm.sl + at), d0, d1, d2, d3);
+          mma16816<bf>(O[2 * m], ah[0], ah[1], ah[2], ah[3], b0, b1);
+          mma16816<bf>(O[2 * m + 1], ah[0], ah[1], ah[2], ah[3], b2, b3);
+          mma16816<bf>(O[2 * m], ah[0], ah[1], ah[2], ah[3], d0, d1);
+          mma16816<bf>(O[2 * m + 1], ah[0], ah[1], ah[2], ah[3], d2, d3);
+          mma16816<bf>(O[2 * m], al[0], al[1], al[2], al[3], b0, b1);
+          mma16816<bf>(O[2 * m + 1], al[0], al[1], al[2], al[3], b2, b3);
+        }
+      }
+      for (int j = 0; j <= rb; ++j) {
+        const uint32_t off = static_cast<uint32_t>((rb * kGcB + (mi & 1) * 8 + mr) * SM::kV + j * kGcB + (mi >> 1) * 8);
+        uint32_t ah[4], al[4];
+        ldmatrix_x4(ptx::smem_u32(sm.ah + off), ah[0], ah[1], ah[2], ah[3]);
+        ldmatrix_x4(ptx::smem_u32(sm.al + off), al[0], al[1], al[2], al[3]);
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+          const uint32_t at = static_cast<uint32_t>((j * kGcB + (mi & 1) * 8 + mr) * SM::kV + cO + m * 16 + (mi >> 1) * 8);
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4_trans(ptx::smem_u32(sm.v + at), b0, b1, b2, b3);
+          mma16816<bf>(O[2 * m], ah[0], ah[1], ah[2], ah[3], b0, b1);
+          mma16816<bf>(O[2 * m + 1], ah[0], ah[1], ah[2], ah[3], b2, b3);
+          mma16816<bf>(O[2 * m], al[0], al[1], al[2], al[3], b0, b1);
+          mma16816<bf>(O[2 * m + 1], al[0], al[1], al[2], al[3], b2, b3);
+        }
+      }
+    }
+    {
+      float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+      for (int n = 0; n < 4; ++n) {
+        s0 += O[n][0] * O[n][0] + O[n][1] * O[n][1];
+        s1 += O[n][2] * O[n][2] + O[n][3] * O[n][3];
+      }
+#pragma unroll
+      for (int o = 1; o <= 2; o <<= 1) {
+        s0 += __shfl_xor_sync(0xffffffffu, s0, o);
+        s1 += __shfl_xor_sync(0xffffffffu, s1, o);
+      }
+      if (t4 == 0) {
+        sm.part[warp & 1][rb * 16 + g] = s0;
+        sm.part[warp & 1][rb * 16 + g + 8] = s1;
+      }
+    }
+    __syncthreads();
+    // sums of squares of this CTA's columns to every CTA of the head (two sets by parity: a CTA is at most one chunk ahead)
+    if (tid < kGcC) {
+      const float s = sm.part[0][tid] + sm.part[1][tid];
+      const uint32_t mine = ptx::smem_u32(&sm.ss[ch & 1][rank][tid]);
+      for (int d = 0; d < nrank; ++d) ptx::st_shared_cluster_f32(ptx::mapa_shared(mine, d), s);
+    }
+    ptx::cluster_arrive_release();
+
+    // ---- 4. state update (meanwhile the sums travel)
+    {
+      const float* be = sm.ref + 4 * DK;
+      const float d0 = __expf(be[rowS]), d1 = __expf(be[rowS + 8]);
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        S[n][0] *= d0; S[n][1] *= d0;
+        S[n][2] *= d1; S[n][3] *= d1;
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float f0 = __expf(be[rowS] - sm.ref[(j + 1) * DK + rowS]), f1 = __expf(be[rowS + 8] - sm.ref[(j + 1) * DK + rowS + 8]);
+        const float* kc = sm.k + (j * kGcB + 2 * t4) * SM::kK + rowS;
+        uint32_t ah[4], al[4];
+        split2(kc[0] * f0, kc[SM::kK] * f0, ah[0], al[0]);
+        split2(kc[8] * f1, kc[SM::kK + 8] * f1, ah[1], al[1]);
+        split2(kc[8 * SM::kK] * f0, kc[9 * SM::kK] * f0, ah[2], al[2]);
+        split2(kc[8 * SM::kK + 8] * f1, kc[9 * SM::kK + 8] * f1, ah[3], al[3]);
+#pragma unroll
+        for (int m = 0; m < NT / 2; ++m) {
+          const uint32_t at = static_cast<uint32_t>((j * kGcB + (mi & 1) * 8 + mr) * SM::kV + cS + m * 16 + (mi >> 1) * 8);
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4_trans(ptx::smem_u32(sm.v + at), b0, b1, b2, b3);
+          mma16816<bf>(S[2 * m], ah[0], ah[1], ah[2], ah[3], b0, b1);
+          mma16816<bf>(S[2 * m + 1], ah[0], ah[1], ah[2], ah[3], b2, b3);
+          mma16816<bf>(S[2 * m], al[0], al[1], al[2], al[3], b0, b1);
+          mma16816<bf>(S[2 * m + 1], al[0], al[1], al[2], al[3], b2, b3);
+        }
+      }
+      publish_state();
+    }
+    ptx::cluster_wait_acquire();
+
+    // ---- 5. output norm and gate
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int t = rb * 16 + g + half * 8;
+      if (t < n_tok) {
+        float ss = 0.f;
+        for (int d = 0; d < nrank; ++d) ss += sm.ss[ch & 1][d][t];
+        const float scale = rsqrtf(ss / static_cast<float>(p.vdim) + p.eps);
+        const int64_t tok = t_beg + base + t;
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+          const int col = cO + n * 8 + 2 * t4;
+          if (col < nv) {
+            const float2 w = ldf2(p.norm + v0 + col), gate = ldf2(p.g + tok * p.row + h * p.vdim + v0 + col);
+            stf2(p.out + tok * p.out_stride + h * p.vdim + v0 + col, O[n][2 * half] * scale * w.x * silu_acc(gate.x),
+                 O[n][2 * half + 1] * scale * w.y * silu_acc(gate.y));
+          }
+        }
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int c = rowS + (e >> 1) * 8, col = cS + n * 8 + 2 * t4 + (e & 1);
+      if (c < p.dim && col < nv) gstate[static_cast<int64_t>(c) * p.vdim + col] = S[n][e];
+    }
+}
+
+template <int DK>
+static cudaError_t launch_gla_chunk(const GlaChunkParams& p, int rows, cudaStream_t stream) {
+  static PerDeviceOnce once;
+  cudaError_t e = once.run([] {
+    return cudaFuncSetAttribute(gla_chunk_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(GcSmem<DK>));
+  });
+  if (e != cudaSuccess) return e;
+  const unsigned vb = (p.vdim + kGcV - 1) / kGcV;
+  return launch_pdl_cluster(gla_chunk_kernel<DK>, dim3(vb, p.heads, rows), dim3(kGcThreads), sizeof(GcSmem<DK>), vb, stream, p);
+}
+
+}  // namespace blitz
+
+extern "C" {
+using namespace blitz;
+
+// Whether the chunked kernel takes these sizes (bf16 only; vectors of 8 elements).
+int blitz_gla_chunk_supported(int dim, int vdim, int rank) {
+  return dim > 0 && dim <= 128 && (dim & 7) == 0 && vdim > 0 && (vdim & 7) == 0 && vdim <= kGcV * kGcMaxCluster && rank > 0 &&
+         rank <= 128;
+}
+
+// Rows of at least one token each: tokens tok_indptr[r] .. tok_indptr[r + 1]; max_len: the longest row.  cum: fp32 scratch
+// [tokens][heads * dim], indexed by token number.  The pitch `row` and the five column pointers are multiples of 8 elements.
+int blitz_gla_chunk(const void* q, const void* k, const void* v, const void* g, const void* low, int64_t row, const void* a2,
+                    const void* a2_b, const void* norm, float* cum, float* state, void* out, int64_t out_stride,
+                    const int32_t* pos, const int32_t* tok_indptr, const int32_t* seq_slot, int rows, int max_len, int heads,
+                    int dim, int vdim, int rank, int num_slots, float q_scale, float tau, float eps, int* status,
+                    cudaStream_t stream) {
+  using bf = __nv_bfloat16;
+  if (rows <= 0 || max_len <= 0) return 0;
+  if (!blitz_gla_chunk_supported(dim, vdim, rank) || (row & 7) || (out_stride & 1) || !(tau > 0.f) || heads > 65535 || rows > 65535)
+    return -1;
+  for (const void* x : {q, k, v})
+    if (reinterpret_cast<uintptr_t>(x) & 15) return -1;
+  if ((reinterpret_cast<uintptr_t>(g) | reinterpret_cast<uintptr_t>(norm) | reinterpret_cast<uintptr_t>(out)) & 3) return -1;
+  if (reinterpret_cast<uintptr_t>(cum) & 15) return -1;
+  GlaChunkParams p{(const bf*)q, (const bf*)k, (const bf*)v, (const bf*)g, (const bf*)low, row, (const bf*)a2, (const bf*)a2_b,
+                   (const bf*)norm, cum, state, (bf*)out, out_stride, pos, tok_indptr, seq_slot, heads, dim, vdim, rank,
+                   num_slots, q_scale, 1.f / tau, eps, status};
+  const int hk = heads * dim;
+  cudaError_t e = launch_pdl(gla_decay_kernel, dim3((hk + kGdThreads - 1) / kGdThreads, (max_len + kGcC - 1) / kGcC, rows),
+                             dim3(kGdThreads), (size_t)kGcC * rank * sizeof(float), stream, p);
+  if (e != cudaSuccess) return (int)e;
+  e = dim <= 32 ? launch_gla_chunk<32>(p, rows, stream) : dim <= 64 ? launch_gla_chunk<64>(p, rows, stream)
+                                                                   : launch_gla_chunk<128>(p, rows, stream);
+  return (int)e;
+}
+
+}  // extern "C"

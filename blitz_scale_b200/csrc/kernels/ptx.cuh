@@ -118,6 +118,10 @@ __device__ __forceinline__ void st_shared_cluster_v4(uint32_t cluster_addr, uint
                : "memory");
 }
 
+__device__ __forceinline__ void st_shared_cluster_f32(uint32_t cluster_addr, float v) {
+  asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(cluster_addr), "f"(v) : "memory");
+}
+
 // ---------------------------------------------------------------- programmatic dependent launch
 // wait: returns when every kernel this one depends on has completed and its writes are visible (a no-op for
 // a kernel launched without the attribute).  launch_dependents: lets the next kernel of the stream be

@@ -48,6 +48,8 @@ class HybridRunner:
         rw = max((m.width for m in cfg.run_mixers() if m.kind == "rglru"), default=0)
         self._conv = torch.empty(max_tokens * rw, dtype=dt, device=dev) if rw else None
         self._gates = torch.empty(max_tokens * 2 * rw, dtype=torch.float32, device=dev) if rw else None
+        ck = max((m.heads * m.dim for m in cfg.run_mixers() if m.kind == "gla"), default=0)
+        self._cum = torch.empty(max_tokens * ck, dtype=torch.float32, device=dev) if ck and dt == torch.bfloat16 else None
         self.last = torch.empty(max_batch, H, dtype=torch.float32, device=dev)
         self._logits_pad = torch.zeros(max_batch, cfg.vocab_pad, dtype=torch.float32, device=dev)
         self.logits = self._logits_pad[:, :cfg.vocab]
@@ -128,7 +130,8 @@ class HybridRunner:
         if ns:
             ops.gla_recurrent(*parts, *w, state, mid, m.pos, None, m.seq_slot[:ns], **args)
         if m.batch > ns:
-            ops.gla_recurrent(*parts, *w, state, mid, m.pos, m.tok_indptr[ns:], m.seq_slot[ns:], **args)
+            ops.gla(*parts, *w, state, mid, m.pos, m.tok_indptr[ns:], m.seq_slot[ns:], row_lens=m.seq_lens_host[ns:],
+                    cum=self._cum, **args)
 
     def _rglru(self, r: int, l: int, mx: RGLRUMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta) -> None:
         T, rc = m.num_tokens, self.cache.runs[r]

@@ -468,8 +468,26 @@ def rglru_scan(u, gates: torch.Tensor, gate_b, lam, y, x, y_b, state: torch.Tens
     return out
 
 
+GLA_CHUNK_MIN_LEN = 16      # rows shorter than this are faster token by token
+
+
 def gla(q, k, v, g, low, a2, a2_b, norm, state: torch.Tensor, out: torch.Tensor, pos, tok_indptr, seq_slot, *, rank: int,
-        tau: float, eps: float, row_lens=None) -> torch.Tensor:
+        tau: float, eps: float, row_lens=None, cum: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Gated linear attention over the rows of a step; ``row_lens``: tokens per row (host), needed where rows are longer
-    than one token."""
-    return gla_recurrent(q, k, v, g, low, a2, a2_b, norm, state, out, pos, tok_indptr, seq_slot, rank=rank, tau=tau, eps=eps)
+    than one token.  Prompts in bf16 go through the chunked tensor-core kernel, everything else token by token.
+    ``cum``: fp32 scratch of the chunked kernel, tokens x heads x dim elements (allocated when missing)."""
+    slots, heads, dim, vdim = state.shape
+    longest = 1 if tok_indptr is None else max(row_lens)
+    aligned = all(t.data_ptr() % 16 == 0 for t in (q, k, v)) and q.stride(0) % 8 == 0 and g.data_ptr() % 4 == 0
+    if (longest < GLA_CHUNK_MIN_LEN or q.dtype != torch.bfloat16 or not aligned or out.stride(0) % 2 or out.data_ptr() % 4
+            or not lib().blitz_gla_chunk_supported(dim, vdim, rank)):
+        return gla_recurrent(q, k, v, g, low, a2, a2_b, norm, state, out, pos, tok_indptr, seq_slot, rank=rank, tau=tau, eps=eps)
+    n = q.shape[0] * heads * dim
+    if cum is None:
+        cum = torch.empty(n, dtype=torch.float32, device=q.device)
+    assert cum.dtype == torch.float32 and cum.numel() >= n and state.dtype == torch.float32 and state.is_contiguous()
+    _check(lib().blitz_gla_chunk(_p(q), _p(k), _p(v), _p(g), _p(low), q.stride(0), _p(a2), _p(a2_b), _p(norm), _p(cum),
+                                 _p(state), _p(out), out.stride(0), _p(pos), _p(tok_indptr), _p(seq_slot), seq_slot.numel(),
+                                 longest, heads, dim, vdim, rank, slots, dim ** -0.5, tau, eps, _p(status_word(q.device)),
+                                 _stream()), "blitz_gla_chunk")
+    return out

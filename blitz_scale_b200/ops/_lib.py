@@ -98,6 +98,9 @@ def _declare(L: ctypes.CDLL) -> None:
                               c_i, c_f, c_f, c_p, c_i, c_p])
     sig("blitz_gla_recurrent", [c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_i, c_i,
                                 c_i, c_i, c_i, c_i, c_f, c_f, c_f, c_i, c_p, c_i, c_p])
+    sig("blitz_gla_chunk", [c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i,
+                            c_i, c_i, c_i, c_i, c_f, c_f, c_f, c_p, c_p])
+    sig("blitz_gla_chunk_supported", [c_i, c_i, c_i], c_i)
     sig("blitz_conv_causal", [c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_p, c_i,
                               c_p])
     sig("blitz_rglru_scan", [c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_i, c_i,
