@@ -159,9 +159,21 @@ def main():
     ap.add_argument("--no-baseline", action="store_true", help="do not run the stand-in baseline arm first")
     ap.add_argument("--no-extra-tp", action="store_true", help="N > 1: do not add the tensor-parallel record "
                     "(one replica over all N GPUs, fused peer-memory runner against the NCCL runner)")
+    ap.add_argument("--hybrid", action="store_true", help="instead: throughput of the hybrid models beside the uniform model of "
+                    "equal size, and their kernels against the roofline (bench/hybrid_bench.py; one GPU)")
+    ap.add_argument("--hybrid-part", default="all", choices=["all", "models", "kernels"])
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm()
+    if args.hybrid:
+        sys.path.insert(0, os.path.join(ROOT, "bench"))
+        import hybrid_bench
+        sampler = ClockSampler(0)
+        sampler.start()
+        result = hybrid_bench.run(args.hybrid_part)
+        result["clocks"] = sampler.stop()
+        print(json.dumps(result))
+        return 0
     args.warmup = max(args.warmup, 3)
 
     import torch
