@@ -30,9 +30,11 @@
 // Models that ask for it (template parameter EXT) get a sliding window with kept first tokens, soft-capped scores and a
 // per-head sink.  The two tiles of an item then walk the key blocks of the kept tokens and those from the first row's
 // window edge on; blocks in between are never loaded.  A block that is wholly visible to a tile needs no mask.  The cap,
-// cap * tanh(s / cap), is applied to the scores as they turn into probabilities: a polynomial on the FMA pipe where all
-// of a warp's scores of the block stay below 0.9 cap (one vote per block), the special-function unit otherwise; tanh being monotonic, the
-// row maximum is capped alone.  The sink is one more term of the row sum at the end.
+// cap * tanh(s / cap), is applied to the scores as they turn into probabilities.  Where all of a warp's scores of the
+// block stay below half the cap (one vote per block, the usual case), that is an odd polynomial on the FMA pipe, two
+// scores per instruction, and the largest magnitude serves as the row's reference instead of its maximum, so that one
+// pass over the scores decides both; else the special-function unit does it (tanh being monotonic, the row maximum is
+// capped alone).  The sink is one more term of the row sum at the end.
 //
 // Replaces FlashInfer's BatchPrefillWithRaggedKVCacheWrapper / paged wrapper calls and their host Plan()
 // (src/kernel/attention_prefill.cu:11-45, src/kernel/flashinfer_types.cu:24-49).
@@ -40,6 +42,7 @@
 #include "ptx.cuh"
 #include "tmap.cuh"
 #include "common.cuh"
+#include <cmath>
 
 namespace blitz {
 
@@ -57,6 +60,8 @@ struct PagedPrefillParams {
   float scale_log2;
   int window, keep_first;     // EXT: a row sees the last `window` positions (0: all) and the first `keep_first`
   float cap_scale, cap_log2;  // EXT: soft cap (cap_log2 > 0): score in log2 units = cap_log2 * tanh(q.k * cap_scale)
+  float small_max;            // EXT: largest |q.k| the polynomial takes (0: never)
+  float poly[4];              // EXT: score in log2 units = x (poly[0] + poly[1] x^2 + poly[2] x^4 + poly[3] x^6), x = q.k
   const void* sink;           // EXT: [q_heads] in the activation type, or null
   int* status;
   long long* trace;  // profiling aid (null in production): clock stamps of CTA 0's first item, see the set_trace call
@@ -117,18 +122,6 @@ __device__ __forceinline__ int pp_index(int r, int total) {
   const int G = gridDim.x;
   const int idx = r * G + ((r & 1) ? G - 1 - static_cast<int>(blockIdx.x) : static_cast<int>(blockIdx.x));
   return idx < total ? idx : -1;
-}
-
-// Odd polynomial for tanh on |x| <= 0.9 (Chebyshev interpolation of tanh(x) / x in x^2): absolute error 1.4e-7.
-constexpr float kTanhPolyMax = 0.9f;
-__device__ __forceinline__ float tanh_poly(float x) {
-  const float y = x * x;
-  float r = fmaf(-0.00366952f, y, 0.01797143f);
-  r = fmaf(r, y, -0.0524757f);
-  r = fmaf(r, y, 0.13306333f);
-  r = fmaf(r, y, -0.33331502f);
-  r = fmaf(r, y, 0.99999979f);
-  return x * r;
 }
 
 template <typename T, int HD, bool POLY, bool EXT>
@@ -374,52 +367,49 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         pp_trace(p, tracer, t, j, 2);
         auto score = [&](int i) -> uint32_t& { return i < 32 ? v0[i] : i < 64 ? v1[i - 32] : i < 96 ? v2[i - 64] : v3[i - 96]; };
         const int kv0 = it.block(j) * kPpTile;
-        bool masked = false;
-        if (EXT && p.window > 0) {
-          const int row0 = it.prefix + it.q0 + t * kPpTile;  // position of the tile's first row
-          const bool in_window = kv0 + kPpTile - 1 <= row0 && kv0 > row0 + kPpTile - 1 - p.window;
-          masked = !in_window && !(kv0 + kPpTile <= p.keep_first && kv0 + kPpTile - 1 <= row0);
+        const int row0 = it.prefix + it.q0 + t * kPpTile;  // position of the tile's first row
+        // does the block hold a key that some row of the tile may not see?
+        bool masked = kv0 + kPpTile - 1 > row0;
+        if (EXT && p.window > 0)
+          masked = masked || (kv0 <= row0 + kPpTile - 1 - p.window && kv0 + kPpTile > p.keep_first);
+        const int from = (EXT && p.window > 0) ? limit - p.window + 1 : 0;
+        auto visible = [&](int i) {  // key i of the block to this row
+          return kv0 + i <= limit && (!EXT || kv0 + i >= from || kv0 + i < p.keep_first);
+        };
+        const bool capped = EXT && p.cap_log2 > 0.f;
+        // largest of the row's 128 scores, or of their magnitudes: eight independent chains of three-input maxima (with two
+        // softmax warps per scheduler nothing else hides a serial one)
+        auto largest = [&](auto&& max3) {
+          float mxs[8];
+#pragma unroll
+          for (int i = 0; i < 8; ++i) mxs[i] = __uint_as_float(score(i));
+#pragma unroll
+          for (int i = 8; i < kPpTile - 8; i += 16)
+#pragma unroll
+            for (int k = 0; k < 8; ++k)
+              mxs[k] = max3(mxs[k], __uint_as_float(score(i + 2 * k)), __uint_as_float(score(i + 2 * k + 1)));
+#pragma unroll
+          for (int i = kPpTile - 8; i < kPpTile; ++i) mxs[i & 7] = max3(mxs[i & 7], __uint_as_float(score(i)), __uint_as_float(score(i)));
+          const float mx = fmaxf(max3(mxs[0], mxs[1], mxs[2]), max3(mxs[3], mxs[4], mxs[5]));
+          return max3(mx, mxs[6], mxs[7]);
+        };
+        float mx = 0.f;
+        bool small = false;
+        if (capped && std::is_same<T, __nv_bfloat16>::value) {  // (fp16 probabilities need the maximum itself)
+          mx = largest([](float a, float b, float c) { return ptx::fmax3_abs(a, b, c); });
+          small = __all_sync(0xffffffffu, mx <= p.small_max);
+        }
+        if (small) {
+          mx *= p.scale_log2;  // |cap tanh(x / cap)| <= |x|
+        } else {
           if (masked) {
-            const int from = limit - p.window + 1;
 #pragma unroll
             for (int i = 0; i < kPpTile; ++i)
-              if (kv0 + i > limit || (kv0 + i < from && kv0 + i >= p.keep_first)) score(i) = 0xff800000u;
+              if (!visible(i)) score(i) = 0xff800000u;  // -inf
           }
-        } else if (kv0 + kPpTile - 1 > it.prefix + it.q0 + t * kPpTile) {  // the block reaches past the tile's first row: mask
-#pragma unroll
-          for (int i = 0; i < kPpTile; ++i)
-            if (kv0 + i > limit) score(i) = 0xff800000u;  // -inf
-          masked = true;
-        }
-        // eight independent chains of three-input maxima: with two softmax warps per scheduler nothing else hides a
-        // serial one
-        float mxs[8];
-#pragma unroll
-        for (int i = 0; i < 8; ++i) mxs[i] = __uint_as_float(score(i));
-#pragma unroll
-        for (int i = 8; i < kPpTile - 8; i += 16)
-#pragma unroll
-          for (int k = 0; k < 8; ++k)
-            mxs[k] = ptx::fmax3(mxs[k], __uint_as_float(score(i + 2 * k)), __uint_as_float(score(i + 2 * k + 1)));
-#pragma unroll
-        for (int i = kPpTile - 8; i < kPpTile; ++i) mxs[i & 7] = fmaxf(mxs[i & 7], __uint_as_float(score(i)));
-        float mx = fmaxf(ptx::fmax3(mxs[0], mxs[1], mxs[2]), ptx::fmax3(mxs[3], mxs[4], mxs[5]));
-        mx = ptx::fmax3(mx, mxs[6], mxs[7]);
-        bool small = false;  // every score of the warp within the range of tanh_poly
-        if (EXT && p.cap_log2 > 0.f) {
-          if (!masked) {
-            float mns[8];
-#pragma unroll
-            for (int i = 0; i < 8; ++i) mns[i] = __uint_as_float(score(i));
-#pragma unroll
-            for (int i = 8; i < kPpTile; ++i) mns[i & 7] = fminf(mns[i & 7], __uint_as_float(score(i)));
-            const float mn = fminf(fminf(fminf(mns[0], mns[1]), fminf(mns[2], mns[3])),
-                                   fminf(fminf(mns[4], mns[5]), fminf(mns[6], mns[7])));
-            small = __all_sync(0xffffffffu, fmaxf(mx, -mn) * fabsf(p.cap_scale) <= kTanhPolyMax);
-          }
-          mx = mx == -INFINITY ? mx : p.cap_log2 * ptx::tanh_ex2(mx * p.cap_scale);
-        } else {
-          mx *= p.scale_log2;
+          mx = largest([](float a, float b, float c) { return ptx::fmax3(a, b, c); });
+          if (capped) mx = mx == -INFINITY ? mx : p.cap_log2 * ptx::tanh_ex2(mx * p.cap_scale);
+          else mx *= p.scale_log2;
         }
         // (S of this block was issued after P V of the previous one, so that product is complete: O_t is stable and
         // the columns P is about to overwrite have been read)
@@ -447,33 +437,50 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         // probabilities (16 bit) -> tensor memory over the scores; row sum
         float rs[4] = {0.f, 0.f, 0.f, 0.f};
         const float neg_m = (EXT && m_ref == -INFINITY) ? 0.f : -m_ref;
-        auto probabilities = [&](auto&& exponent) {
+        auto probabilities = [&](auto&& exponents) {  // exponents(c): those of scores c and c + 1
 #pragma unroll
           for (int h = 0; h < 2; ++h) {  // 64 scores -> 32 columns of pairs
             uint32_t pk[32];
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
-              const int c = h * 64 + 2 * i;
-              const float x0 = exponent(__uint_as_float(score(c)));
-              const float x1 = exponent(__uint_as_float(score(c + 1)));
-              const float e0 = ptx::ex2_approx(x0);
-              const float e1 = (POLY && (i & 1)) ? ptx::ex2_poly(x1) : ptx::ex2_approx(x1);
+              const float2 x = exponents(h * 64 + 2 * i);
+              const float e0 = ptx::ex2_approx(x.x);
+              const float e1 = (POLY && (i & 1)) ? ptx::ex2_poly(x.y) : ptx::ex2_approx(x.y);
               rs[i & 3] += e0 + e1;
               pk[i] = pk2<T>(e0, e1);
             }
             ptx::tmem_st_32x32(tS + h * 32, pk);
           }
         };
-        if (EXT && p.cap_log2 > 0.f) {
-          if (small) {
-            probabilities([&](float x) { return fmaf(tanh_poly(x * p.cap_scale), p.cap_log2, neg_m); });
-          } else {
-            probabilities([&](float x) {
-              return x == -INFINITY ? x : fmaf(ptx::tanh_ex2(x * p.cap_scale), p.cap_log2, neg_m);
+        if (EXT && small) {
+          const uint64_t c0 = ptx::f32x2(p.poly[0], p.poly[0]), c1 = ptx::f32x2(p.poly[1], p.poly[1]),
+                         c2 = ptx::f32x2(p.poly[2], p.poly[2]), c3 = ptx::f32x2(p.poly[3], p.poly[3]), nm = ptx::f32x2(neg_m, neg_m);
+          auto poly = [&](int c) {
+            const uint64_t x = ptx::f32x2(__uint_as_float(score(c)), __uint_as_float(score(c + 1)));
+            const uint64_t y = ptx::mul_f32x2(x, x);
+            uint64_t r = ptx::fma_f32x2(c3, y, c2);
+            r = ptx::fma_f32x2(r, y, c1);
+            r = ptx::fma_f32x2(r, y, c0);
+            return ptx::f32x2_get(ptx::fma_f32x2(x, r, nm));
+          };
+          if (masked) {
+            probabilities([&](int c) {
+              float2 e = poly(c);
+              if (!visible(c)) e.x = -INFINITY;
+              if (!visible(c + 1)) e.y = -INFINITY;
+              return e;
             });
+          } else {
+            probabilities(poly);
           }
+        } else if (capped) {
+          auto cap = [&](float x) { return x == -INFINITY ? x : fmaf(ptx::tanh_ex2(x * p.cap_scale), p.cap_log2, neg_m); };
+          probabilities([&](int c) { return make_float2(cap(__uint_as_float(score(c))), cap(__uint_as_float(score(c + 1)))); });
         } else {
-          probabilities([&](float x) { return fmaf(x, p.scale_log2, neg_m); });
+          probabilities([&](int c) {
+            return make_float2(fmaf(__uint_as_float(score(c)), p.scale_log2, neg_m),
+                               fmaf(__uint_as_float(score(c + 1)), p.scale_log2, neg_m));
+          });
         }
         pp_trace(p, tracer, t, j, 4);
         ptx::tmem_st_wait();
@@ -577,6 +584,13 @@ int blitz_attn_prefill_paged(const void* q, int64_t q_stride, const void* kv_lay
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = g_pp_trace;
   p.window = window; p.keep_first = keep_first; p.sink = sink;
   p.cap_scale = softcap > 0.f ? sm_scale / softcap : 0.f; p.cap_log2 = softcap * 1.4426950408889634f;
+  // tanh(z) = z (k0 + k1 z^2 + k2 z^4 + k3 z^6) for |z| <= 0.5 (Chebyshev interpolation of tanh(z) / z in z^2, absolute
+  // error 2.5e-7), with z = q.k * cap_scale folded in.  Scores below 40 log2 units keep every probability that refers to
+  // the largest magnitude above 2^-80.  A tiny scale / cap would underflow in the coefficients: no polynomial then.
+  const double z = p.cap_scale, k[4] = {0.99999945, -0.33326284, 0.13189939, -0.04439274};
+  double zn = z * p.cap_log2;
+  for (int i = 0; i < 4; ++i, zn *= z * z) p.poly[i] = (float)(k[i] * zn);
+  p.small_max = z > 1e-5 ? (float)fmin(0.5 / z, 40.0 / p.scale_log2) : 0.f;
   const long long total = (long long)entries * q_heads;
   const int sms = device_sm_count();
   const int grid = (int)(total < sms ? total : sms);

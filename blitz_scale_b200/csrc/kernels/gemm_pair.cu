@@ -601,15 +601,19 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                   // fp32 output: a thread's 32 columns are a whole 128-byte line, stored directly
                   if (row_ok) {
                     float* dst = reinterpret_cast<float*>(p.C) + static_cast<int64_t>(row) * p.ldc + n0 + c;
+                    float old[4][8];
+                    if (EPI == 5) {
 #pragma unroll
-                    for (int jj = 0; jj < 8; ++jj) {
-                      if (n0 + c + 4 * jj < p.N) {
-                        float4 o = make_float4(gt[4 * jj], gt[4 * jj + 1], gt[4 * jj + 2], gt[4 * jj + 3]);
-                        if (EPI == 5) {
-                          const float4 x = *reinterpret_cast<const float4*>(dst + 4 * jj);
-                          o = make_float4(x.x + p.alpha * o.x, x.y + p.alpha * o.y, x.z + p.alpha * o.z, x.w + p.alpha * o.w);
-                        }
-                        *reinterpret_cast<float4*>(dst + 4 * jj) = o;
+                      for (int jj = 0; jj < 4; ++jj)
+                        if (n0 + c + 8 * jj < p.N) ptx::ld_global_v8(dst + 8 * jj, old[jj]);
+                    }
+#pragma unroll
+                    for (int jj = 0; jj < 4; ++jj) {
+                      if (n0 + c + 8 * jj < p.N) {
+                        float o[8];
+#pragma unroll
+                        for (int k = 0; k < 8; ++k) o[k] = EPI == 5 ? old[jj][k] + p.alpha * gt[8 * jj + k] : gt[8 * jj + k];
+                        ptx::st_global_v8(dst + 8 * jj, o);
                       }
                     }
                   }

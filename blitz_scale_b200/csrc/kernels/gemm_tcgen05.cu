@@ -156,15 +156,19 @@ __device__ __forceinline__ void store_chunk(const GemmParams& p, const float (&a
   if (EPI == kEpiStoreF32 || EPI == kEpiAxpyF32) {
     if (!row_ok) return;
     float* dst = reinterpret_cast<float*>(p.C) + static_cast<int64_t>(row) * p.ldc + static_cast<int64_t>(group) * p.N + col0;
+    float old[4][8];
+    if (EPI == kEpiAxpyF32) {
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      if (col0 + j * 4 < p.N) {
-        float4 v = make_float4(acc[4 * j], acc[4 * j + 1], acc[4 * j + 2], acc[4 * j + 3]);
-        if (EPI == kEpiAxpyF32) {
-          const float4 r = *reinterpret_cast<const float4*>(dst + 4 * j);
-          v = make_float4(r.x + p.alpha * v.x, r.y + p.alpha * v.y, r.z + p.alpha * v.z, r.w + p.alpha * v.w);
-        }
-        *reinterpret_cast<float4*>(dst + 4 * j) = v;
+      for (int j = 0; j < 4; ++j)
+        if (col0 + j * 8 < p.N) ptx::ld_global_v8(dst + 8 * j, old[j]);
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      if (col0 + j * 8 < p.N) {
+        float v[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) v[i] = EPI == kEpiAxpyF32 ? old[j][i] + p.alpha * acc[8 * j + i] : acc[8 * j + i];
+        ptx::st_global_v8(dst + 8 * j, v);
       }
     }
     return;

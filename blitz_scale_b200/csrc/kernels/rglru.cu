@@ -37,47 +37,84 @@ struct ConvParams {
   int* status;
 };
 
-constexpr int kConvTok = 8;  // tokens per thread
+constexpr int kConvTok = 16;  // tokens per thread
+constexpr int kConvThreads = 128;
 
-template <typename T>
-__global__ void __launch_bounds__(128) conv_causal_kernel(const ConvParams p) {
+// A thread computes VEC channels of kConvTok consecutive tokens (one token per row in decode).  The last TAPS - 1 inputs
+// stay in registers; they are filled where a row's portion begins, from the history or from the sequence's start.
+template <typename T, int VEC, int TAPS>
+__global__ void __launch_bounds__(kConvThreads) conv_causal_kernel(const ConvParams p) {
   ptx::griddep_launch_dependents();
   ptx::griddep_wait();
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  const int c = (blockIdx.x * kConvThreads + threadIdx.x) * VEC;
   if (c >= p.width) return;
-  const int t0 = blockIdx.y * kConvTok, t1 = min(p.num_tokens, t0 + kConvTok);
+  auto load = [](const T* q) { return VEC == 2 ? ldf2<T>(q) : make_float2(ldf<T>(q), 0.f); };
   const T* x = reinterpret_cast<const T*>(p.x) + c;
   const T* hist = reinterpret_cast<const T*>(p.hist) + c;
-  float w[kMaxTaps];
+  T* u = reinterpret_cast<T*>(p.u) + c;
+  float2 w[TAPS];
 #pragma unroll
-  for (int j = 0; j < kMaxTaps; ++j) w[j] = j < p.taps ? ldf<T>(reinterpret_cast<const T*>(p.conv) + j * p.width + c) : 0.f;
-  const float xb = ldf<T>(reinterpret_cast<const T*>(p.x_b) + c), ub = ldf<T>(reinterpret_cast<const T*>(p.conv_b) + c);
-  int b = p.tok_indptr ? row_of_token(p.tok_indptr, p.rows, t0) : t0;
-  for (int t = t0; t < t1; ++t) {
-    if (p.tok_indptr) {
-      while (b + 1 < p.rows && p.tok_indptr[b + 1] <= t) ++b;
-    } else {
-      b = t;
-    }
-    const int i = p.tok_indptr ? t - p.tok_indptr[b] : 0;  // place in the row's portion
-    const int slot = p.seq_slot[b], at = p.pos[t];
-    float acc = ub;
-    if (slot >= 0) {
-      if (slot >= p.num_slots) {
-        if (p.status) atomicCAS(p.status, 0, kStatusBadIndex);
-        continue;
-      }
+  for (int j = 0; j < TAPS; ++j)  // fewer taps than TAPS: the missing ones come first and are zero
+    w[j] = j >= TAPS - p.taps ? load(reinterpret_cast<const T*>(p.conv) + (j - (TAPS - p.taps)) * p.width + c) : make_float2(0.f, 0.f);
+  const float2 xb = load(reinterpret_cast<const T*>(p.x_b) + c), ub = load(reinterpret_cast<const T*>(p.conv_b) + c);
+  const bool single = p.tok_indptr == nullptr;
+  const int t0 = single ? blockIdx.y : blockIdx.y * kConvTok, t1 = single ? t0 + 1 : min(p.num_tokens, t0 + kConvTok);
+  float2 in[TAPS];  // inputs with bias, oldest first; in[TAPS - 1] is the current token's
+  auto fill = [&](int b, int t, int first) {  // the inputs before token t of row b, whose portion begins at token `first`
+    const int slot = p.seq_slot[b], at = p.pos[t], i = t - first;
+    const bool ok = slot < p.num_slots;
+    if (!ok && p.status) atomicCAS(p.status, 0, kStatusBadIndex);
 #pragma unroll
-      for (int j = 0; j < kMaxTaps; ++j) {
-        if (j >= p.taps) break;
-        const int back = p.taps - 1 - j;
-        if (at < back) continue;  // before the start of the sequence
-        const float v = back <= i ? ldf<T>(x + (t - back) * p.row)
-                                  : ldf<T>(hist + (static_cast<int64_t>(slot) * (p.taps - 1) + (p.taps - 1 - (back - i))) * p.width);
-        acc += w[j] * (v + xb);
+    for (int j = 1; j < TAPS; ++j) {
+      const int back = TAPS - j;
+      float2 v = make_float2(0.f, 0.f);
+      if (back < p.taps && at >= back && slot >= 0 && ok) {
+        const float2 raw = back <= i ? load(x + static_cast<int64_t>(t - back) * p.row)
+                                     : load(hist + (static_cast<int64_t>(slot) * (p.taps - 1) + (p.taps - 1 - (back - i))) * p.width);
+        v = make_float2(raw.x + xb.x, raw.y + xb.y);
       }
+      in[j] = v;  // shifted down by one when the token itself comes in
     }
-    stf<T>(reinterpret_cast<T*>(p.u) + t * p.u_stride + c, acc);
+  };
+  auto emit = [&](int t, const float2& raw) {
+#pragma unroll
+    for (int j = 0; j + 1 < TAPS; ++j) in[j] = in[j + 1];
+    in[TAPS - 1] = make_float2(raw.x + xb.x, raw.y + xb.y);
+    float2 acc = ub;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      acc.x += w[j].x * in[j].x;
+      acc.y += w[j].y * in[j].y;
+    }
+    if (VEC == 2) stf2<T>(u + static_cast<int64_t>(t) * p.u_stride, acc.x, acc.y);
+    else stf<T>(u + static_cast<int64_t>(t) * p.u_stride, acc.x);
+  };
+  if (single) {
+    fill(t0, t0, t0);
+    emit(t0, load(x + static_cast<int64_t>(t0) * p.row));
+    return;
+  }
+  float2 raw[kConvTok];
+#pragma unroll
+  for (int k = 0; k < kConvTok; ++k)
+    raw[k] = t0 + k < t1 ? load(x + static_cast<int64_t>(t0 + k) * p.row) : make_float2(0.f, 0.f);
+  int b = row_of_token(p.tok_indptr, p.rows, t0);
+  int first = p.tok_indptr[b], end = p.tok_indptr[b + 1];
+  fill(b, t0, first);
+#pragma unroll
+  for (int k = 0; k < kConvTok; ++k) {
+    const int t = t0 + k;
+    if (t < t1) {
+      if (t >= end) {
+        do {
+          ++b;
+          first = end;
+          end = p.tok_indptr[b + 1];
+        } while (t >= end);
+        fill(b, t, first);
+      }
+      emit(t, raw[k]);
+    }
   }
 }
 
@@ -102,8 +139,51 @@ struct ScanParams {
   int* status;
 };
 
+// decay and input of one token: S <- a S + b
+__device__ __forceinline__ void rglru_gates(float rate, float r, float i, float u, float& a, float& b) {
+  const float la = rate * __fdividef(1.f, 1.f + __expf(-r));
+  a = __expf(la);
+  const float x = 2.f * la;  // 1 - a^2 = 1 - e^x, by its series where the difference would lose digits
+  const float rest = x > -0.03f ? -x * (1.f + x * (0.5f + x * (0.16666667f + x * 0.041666667f))) : 1.f - a * a;
+  b = sqrtf(rest) * __fdividef(1.f, 1.f + __expf(-i)) * u;
+}
+__device__ __forceinline__ float gelu_tanh_ex2(float z) {
+  return 0.5f * z * (1.f + ptx::tanh_ex2(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
+// Decode: one token per row, a thread per channel.
+constexpr int kStepThreads = 256;
+template <typename T>
+__global__ void __launch_bounds__(kStepThreads) rglru_step_kernel(const ScanParams p) {
+  ptx::griddep_launch_dependents();
+  ptx::griddep_wait();
+  const int r = blockIdx.y, c = blockIdx.x * kStepThreads + threadIdx.x;
+  const int slot = p.seq_slot[r];
+  if (slot < 0 || c >= p.width) return;
+  if (slot >= p.num_slots) {
+    if (p.status) atomicCAS(p.status, 0, kStatusBadIndex);
+    return;
+  }
+  const int keep = p.taps - 1;
+  const int rcol = (c / p.block) * 2 * p.block + c % p.block, icol = rcol + p.block;
+  float* state = p.state + static_cast<int64_t>(slot) * p.width + c;
+  const float* gt = p.gates + static_cast<int64_t>(r) * 2 * p.width;
+  T* hist = reinterpret_cast<T*>(p.hist) + static_cast<int64_t>(slot) * keep * p.width + c;
+  const T x = reinterpret_cast<const T*>(p.x)[static_cast<int64_t>(r) * p.row + c];
+  const float y = ldf<T>(reinterpret_cast<const T*>(p.y) + static_cast<int64_t>(r) * p.row + c) + ldf<T>(reinterpret_cast<const T*>(p.y_b) + c);
+  float a, b;
+  rglru_gates(-8.f * softplus_f(ldf<T>(reinterpret_cast<const T*>(p.lam) + c)),
+              gt[rcol] + ldf<T>(reinterpret_cast<const T*>(p.gate_b) + rcol), gt[icol] + ldf<T>(reinterpret_cast<const T*>(p.gate_b) + icol),
+              ldf<T>(reinterpret_cast<const T*>(p.u) + static_cast<int64_t>(r) * p.u_stride + c), a, b);
+  const float S = (p.pos[r] == 0 ? 0.f : a * *state) + b;
+  *state = S;
+  stf<T>(reinterpret_cast<T*>(p.out) + static_cast<int64_t>(r) * p.out_stride + c, S * gelu_tanh_ex2(y));
+  for (int j = 0; j + 1 < keep; ++j) hist[static_cast<int64_t>(j) * p.width] = hist[static_cast<int64_t>(j + 1) * p.width];
+  if (keep > 0) hist[static_cast<int64_t>(keep - 1) * p.width] = x;
+}
+
 template <typename T, int NW, int TS>
-__global__ void __launch_bounds__(NW * 32) rglru_scan_kernel(const ScanParams p) {
+__global__ void __launch_bounds__(NW * 32, 2) rglru_scan_kernel(const ScanParams p) {
   ptx::griddep_launch_dependents();
   ptx::griddep_wait();
   __shared__ float sA[NW][32], sB[NW][32], s_carry[2][32];
@@ -111,7 +191,7 @@ __global__ void __launch_bounds__(NW * 32) rglru_scan_kernel(const ScanParams p)
   const int c = blockIdx.x * 32 + lane;
   const bool live = c < p.width;
   const int slot = p.seq_slot[r];
-  const int t_beg = p.tok_indptr ? p.tok_indptr[r] : r, t_end = p.tok_indptr ? p.tok_indptr[r + 1] : r + 1;
+  const int t_beg = p.tok_indptr[r], t_end = p.tok_indptr[r + 1];
   if (slot < 0 || t_end <= t_beg) return;
   if (slot >= p.num_slots) {
     if (threadIdx.x == 0 && p.status) atomicCAS(p.status, 0, kStatusBadIndex);
@@ -130,21 +210,26 @@ __global__ void __launch_bounds__(NW * 32) rglru_scan_kernel(const ScanParams p)
   T* out = reinterpret_cast<T*>(p.out) + cc;
   int cur = 0;
   for (int base = t_beg; base < t_end; base += NW * TS, cur ^= 1) {
-    float a[TS], b[TS];
+    const int t0 = base + warp * TS;
+    float gr[TS], gi[TS], uu[TS], yy[TS];
+#pragma unroll
+    for (int s = 0; s < TS; ++s) {  // every load of the tile before the first use of one
+      const int t = min(t0 + s, t_end - 1);
+      const float* gt = p.gates + static_cast<int64_t>(t) * 2 * p.width;
+      gr[s] = gt[rcol];
+      gi[s] = gt[icol];
+      uu[s] = ldf<T>(u + static_cast<int64_t>(t) * p.u_stride);
+      yy[s] = ldf<T>(y + static_cast<int64_t>(t) * p.row);
+    }
     float A = 1.f, B = 0.f;
 #pragma unroll
     for (int s = 0; s < TS; ++s) {
-      const int t = base + warp * TS + s;
-      a[s] = 1.f;
-      b[s] = 0.f;
-      if (t < t_end && live) {
-        const float* gt = p.gates + static_cast<int64_t>(t) * 2 * p.width;
-        const float la = rate * sigmoid_f(gt[rcol] + rb);
-        a[s] = expf(la);
-        b[s] = sqrtf(-expm1f(2.f * la)) * sigmoid_f(gt[icol] + ib) * ldf<T>(u + t * p.u_stride);
-      }
-      B = a[s] * B + b[s];
-      A *= a[s];
+      float a = 1.f, b = 0.f;
+      if (t0 + s < t_end) rglru_gates(rate, gr[s] + rb, gi[s] + ib, uu[s], a, b);
+      gr[s] = a;
+      gi[s] = b;
+      B = a * B + b;
+      A *= a;
     }
     sA[warp][lane] = A;
     sB[warp][lane] = B;
@@ -154,9 +239,8 @@ __global__ void __launch_bounds__(NW * 32) rglru_scan_kernel(const ScanParams p)
     if (warp == NW - 1) s_carry[cur ^ 1][lane] = A * S + B;
 #pragma unroll
     for (int s = 0; s < TS; ++s) {
-      const int t = base + warp * TS + s;
-      S = a[s] * S + b[s];
-      if (t < t_end && live) stf<T>(out + t * p.out_stride, S * gelu_tanh_f(ldf<T>(y + t * p.row) + yb));
+      S = gr[s] * S + gi[s];
+      if (t0 + s < t_end && live) stf<T>(out + static_cast<int64_t>(t0 + s) * p.out_stride, S * gelu_tanh_ex2(yy[s] + yb));
     }
     __syncthreads();
   }
@@ -169,9 +253,18 @@ __global__ void __launch_bounds__(NW * 32) rglru_scan_kernel(const ScanParams p)
     const T* x = reinterpret_cast<const T*>(p.x) + c;
     for (int j = 0; j < keep; ++j) {
       const int i = n - keep + j;
-      hist[static_cast<int64_t>(j) * p.width] = i >= 0 ? x[(t_beg + i) * p.row] : hist[static_cast<int64_t>(j + n) * p.width];
+      hist[static_cast<int64_t>(j) * p.width] = i >= 0 ? x[static_cast<int64_t>(t_beg + i) * p.row] : hist[static_cast<int64_t>(j + n) * p.width];
     }
   }
+}
+
+template <typename T, int VEC>
+static cudaError_t launch_conv(const ConvParams& p, cudaStream_t stream) {
+  const int units = (p.width + VEC - 1) / VEC;
+  const int spans = p.tok_indptr ? (p.num_tokens + kConvTok - 1) / kConvTok : p.num_tokens;
+  const dim3 grid((units + kConvThreads - 1) / kConvThreads, spans), block(kConvThreads);
+  return p.taps <= 4 ? launch_pdl(conv_causal_kernel<T, VEC, 4>, grid, block, 0, stream, p)
+                     : launch_pdl(conv_causal_kernel<T, VEC, kMaxTaps>, grid, block, 0, stream, p);
 }
 
 }  // namespace blitz
@@ -187,9 +280,17 @@ int blitz_conv_causal(const void* x, int64_t row, const void* x_b, const void* c
   if (taps < 1 || taps > kMaxTaps) return -1;
   ConvParams p{x, row, x_b, conv, conv_b, hist, u, u_stride, pos, tok_indptr, seq_slot, num_tokens, rows, width, taps,
                num_slots, status};
-  const dim3 grid((width + 127) / 128, (num_tokens + kConvTok - 1) / kConvTok);
+  if (num_tokens > 65535 * (tok_indptr ? kConvTok : 1)) return -1;
   cudaError_t e = cudaSuccess;
-  BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(conv_causal_kernel<T>, grid, dim3(128), 0, stream, p)));
+  // two channels at a time where every row starts on an even element
+  const uintptr_t pair = 2 * (dtype == 2 ? 4 : 2);
+  bool vec = ((width | row | u_stride) & 1) == 0;
+  for (const void* q : {x, x_b, conv, conv_b, hist, (const void*)u}) vec = vec && (reinterpret_cast<uintptr_t>(q) % pair) == 0;
+  if (vec) {
+    BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_conv<T, 2>(p, stream)));
+  } else {
+    BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_conv<T, 1>(p, stream)));
+  }
   return (int)e;
 }
 
@@ -203,12 +304,13 @@ int blitz_rglru_scan(const void* u, int64_t u_stride, const float* gates, const 
   if (block <= 0 || width % block != 0 || rows > 65535 || taps < 1 || taps > kMaxTaps) return -1;
   ScanParams p{u, u_stride, gates, gate_b, lam, y, x, row, y_b, state, hist, out, out_stride, pos, tok_indptr, seq_slot,
                rows, width, block, taps, num_slots, status};
-  const dim3 grid((width + 31) / 32, rows);
   cudaError_t e = cudaSuccess;
   if (single) {
-    BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(rglru_scan_kernel<T, 1, 1>, grid, dim3(32), 0, stream, p)));
+    const dim3 grid((width + kStepThreads - 1) / kStepThreads, rows);
+    BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(rglru_step_kernel<T>, grid, dim3(kStepThreads), 0, stream, p)));
   } else {
-    BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(rglru_scan_kernel<T, 16, 4>, grid, dim3(512), 0, stream, p)));
+    const dim3 grid((width + 31) / 32, rows);
+    BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(rglru_scan_kernel<T, 16, 8>, grid, dim3(512), 0, stream, p)));
   }
   return (int)e;
 }

@@ -23,7 +23,7 @@ struct RopeStoreParams {
   const int32_t* slot;
   void* kv;
   const float2* freq;  // [rot_dims / 2] (high, low)
-  int q_heads, kv_heads, dim, rot_dims, interleaved, page_size, max_pages;
+  int q_heads, kv_heads, dim, rot_dims, interleaved, page_size, max_pages, wide;
   int* status;
 };
 
@@ -58,6 +58,37 @@ __global__ void rope_store_kernel(const RopeStoreParams p) {
   T* vdst = kdst + plane;
   T* q = reinterpret_cast<T*>(p.q) + t * p.row;
   const T* k = reinterpret_cast<const T*>(p.k) + t * p.row;
+  if (p.wide) {
+    // interleaved heads: eight elements (four pairs) per access; dimensions that pass unchanged ride along
+    const int vec = p.dim >> 3;
+    for (int it = threadIdx.x; it < (p.q_heads + p.kv_heads) * vec; it += blockDim.x) {
+      const int head = it / vec, d0 = (it - head * vec) * 8;
+      const bool is_q = head < p.q_heads;
+      if ((!is_q && s < 0) || (is_q && d0 >= p.rot_dims)) continue;
+      const int64_t at = static_cast<int64_t>(is_q ? head : head - p.q_heads) * p.dim + d0;
+      float x[8], y[8];
+      ldf8<T>((is_q ? q : k) + at, x);
+#pragma unroll
+      for (int j = 0; j < 8; j += 2) {
+        const int i = (d0 + j) >> 1;
+        const bool rot = d0 + j < p.rot_dims;
+        const float cs = rot ? s_ang[i] : 1.f, sn = rot ? s_ang[half + i] : 0.f;
+        y[j] = x[j] * cs - x[j + 1] * sn;
+        y[j + 1] = x[j + 1] * cs + x[j] * sn;
+      }
+      stf8<T>((is_q ? q : kdst) + at, y);
+      if (!is_q && p.v == nullptr) stf8<T>(vdst + at, x);
+    }
+    if (p.v != nullptr && s >= 0) {
+      const T* v = reinterpret_cast<const T*>(p.v) + t * p.row;
+      for (int i = threadIdx.x * 8; i < kvrow; i += blockDim.x * 8) {
+        float x[8];
+        ldf8<T>(v + i, x);
+        stf8<T>(vdst + i, x);
+      }
+    }
+    return;
+  }
   // Rotated pairs of q and k.  With two-element accesses only where pairs are neighbours and rows even.
   const bool vec = p.interleaved && ((p.dim | p.row) & 1) == 0;
   const int items = (p.q_heads + p.kv_heads) * half;
@@ -118,9 +149,12 @@ int blitz_rope_store(void* q, const void* k, const void* v, int64_t row, const i
   if (num_tokens <= 0) return 0;
   if (rot_dims < 0 || (rot_dims & 1) || rot_dims > dim || rot_dims > 4096 || (rot_dims > 0 && freq == nullptr)) return -1;
   RopeStoreParams p{q, k, v, row, pos, slot, kv_layer, reinterpret_cast<const float2*>(freq), q_heads, kv_heads, dim,
-                    rot_dims, interleaved, page_size, max_pages, status};
+                    rot_dims, interleaved, page_size, max_pages, 0, status};
+  const uintptr_t al = dtype == 2 ? 32 : 16;
+  p.wide = interleaved && ((dim | row) & 7) == 0;
+  for (const void* x : {(const void*)q, k, v, (const void*)kv_layer}) p.wide = p.wide && (reinterpret_cast<uintptr_t>(x) % al) == 0;
   cudaError_t e = cudaSuccess;
-  BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(rope_store_kernel<T>, dim3(num_tokens), dim3(256),
+  BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(rope_store_kernel<T>, dim3(num_tokens), dim3(p.wide && (q_heads + kv_heads) * dim <= 2048 ? 128 : 256),
                                                (size_t)rot_dims * sizeof(float), stream, p)));
   return (int)e;
 }

@@ -113,9 +113,11 @@ def pair_gemm_workspace(device=None):
 
 
 def _tensor_core_operands(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, N: int, K: int) -> bool:
-    """Sizes, pitches and base addresses the TMA-fed kernels need (16-byte rows and bases)."""
+    """Sizes, pitches and base addresses the TMA-fed kernels need (16-byte rows and bases; fp32 outputs are accessed 32
+    bytes at a time)."""
     return (N % 8 == 0 and K % 8 == 0 and a.stride(0) % 8 == 0 and b.stride(0) % 8 == 0 and out.stride(0) % 8 == 0
-            and a.data_ptr() % 16 == 0 and b.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0)
+            and a.data_ptr() % 16 == 0 and b.data_ptr() % 16 == 0
+            and out.data_ptr() % (32 if out.dtype == torch.float32 else 16) == 0)
 
 
 def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *, residual=None,
