@@ -22,8 +22,8 @@
 // products that involve them split their fp32 operands into two bf16 numbers (x = hi + lo, relative error 2^-17) and
 // drop only the lo * lo term.
 //
-// A block of 8 warps owns (row, head, 64 value columns) and walks the row's chunks with the state in registers; the
-// blocks of one head form a thread-block cluster, which exchanges the 64 partial sums of squares per chunk through
+// A block of 16 warps owns (row, head, 64 value columns) and walks the row's chunks with the state in registers; everything
+// a chunk reads from global memory is requested one chunk (the gates: half a chunk) ahead.  The blocks of one head form a thread-block cluster, which exchanges the 64 partial sums of squares per chunk through
 // distributed shared memory, so that the output norm and the gate are applied here and nothing but the result is
 // written.  (gla_decay_kernel computes b beforehand: every value block of a head needs it.)
 #include "launch.cuh"
@@ -36,7 +36,7 @@ namespace blitz {
 constexpr int kGcC = 64;        // tokens per chunk
 constexpr int kGcB = 16;        // tokens per block
 constexpr int kGcV = 64;        // value columns per CTA
-constexpr int kGcThreads = 256;
+constexpr int kGcThreads = 512;
 constexpr int kGcMaxCluster = 8;
 constexpr float kGcMaxDecay = 80.f;
 
@@ -53,6 +53,13 @@ struct GlaChunkParams {
   float q_scale, inv_tau, eps;
   int* status;
 };
+
+// log(sigmoid(z)) = min(z, 0) - log(1 + e^-|z|) on the special-function unit; the series keeps the digits of a slow decay
+__device__ __forceinline__ float log_sigmoid_ex2(float z) {
+  const float e = __expf(-fabsf(z));
+  const float l = e < 0.03f ? e * (1.f - e * (0.5f - e * (0.33333333f - e * 0.25f))) : __logf(1.f + e);
+  return fminf(z, 0.f) - l;
+}
 
 // Running sum of log(sigmoid(low a2 + b)) / tau over a chunk; a thread per channel.
 constexpr int kGdThreads = 128;
@@ -81,10 +88,12 @@ __global__ void __launch_bounds__(kGdThreads) gla_decay_kernel(const GlaChunkPar
     for (int i = 0; i < kKeep; ++i)
       if (i < p.rank) z += low[i] * w[i];
     for (int i = kKeep; i < p.rank; ++i) z += low[i] * ldf(p.a2 + static_cast<int64_t>(i) * hk + c);
-    sum += log_sigmoid(z) * p.inv_tau;
+    sum += log_sigmoid_ex2(z) * p.inv_tau;
     p.cum[static_cast<int64_t>(t0 + t) * hk + c] = sum;
   }
 }
+
+__device__ __forceinline__ float silu_ex2(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 
 // x = hi + lo in bf16, two neighbours at a time
 __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
@@ -100,25 +109,35 @@ struct GcSmem {
   static constexpr int kV = kGcV + 8;     // row pitch of v, S, A (bf16)
   static constexpr int kParts = kGcMaxCluster;
   float k[kGcC * kK];
-  float ref[5 * DK];                      // r_0 .. r_4 (r_4 = b_end)
+  float ref[2][5 * DK];                   // r_0 .. r_4 (r_4 = b_end), by parity of the chunk
+  float fs[10 * DK];                      // e^(r_i - r_(j+1)) of the ten score tiles
+  float fe[5 * DK];                       // e^(b_end - r_(j+1)), j = 0 .. 3, and e^(b_end)
   float ss[2][kParts][kGcC];              // partial sums of squares of every cluster rank, by parity of the chunk
-  float part[2][kGcC];
+  float part[4][kGcC];
   int wide[4];                            // block whose decay the factored form cannot hold
-  __nv_bfloat16 qh[kGcC * kQ], ql[kGcC * kQ];
+  __nv_bfloat16 qh[kGcC * kQ], ql[kGcC * kQ];  // q'
+  __nv_bfloat16 ih[kGcC * kQ], il[kGcC * kQ];  // q e^b
   __nv_bfloat16 v[kGcC * kV];
   __nv_bfloat16 ah[kGcC * kV], al[kGcC * kV];
   __nv_bfloat16 sh[DK * kV], sl[DK * kV];
 };
+
+// Tiles 0 .. 5: (1,0) (2,0) (2,1) (3,0) (3,1) (3,2); 6 .. 9: the diagonal.
+__device__ __forceinline__ void gc_tile(int tile, int& i, int& j) {
+  i = tile >= 6 ? tile - 6 : (tile >= 3 ? 3 : tile >= 1 ? 2 : 1);
+  j = tile >= 6 ? i : (tile >= 3 ? tile - 3 : tile >= 1 ? tile - 1 : 0);
+}
 
 template <int DK>
 __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunkParams p) {
   using bf = __nv_bfloat16;
   using SM = GcSmem<DK>;
   constexpr int RB = DK / 16;             // 16-row blocks of the state
-  constexpr int CP = 8 / RB;              // warps that share a row block of it
+  constexpr int CP = RB >= 4 ? 16 / RB : 4;  // warps that share a row block of it (DK = 32: half the warps have no part)
   constexpr int NT = kGcV / CP / 8;       // 8-column tiles of the state per warp
-  constexpr int NV = kGcC * DK / 8 / kGcThreads;  // vectors of 8 q (k, b) elements per thread
-  static_assert(RB * CP == 8 && NV >= 1, "DK is 32, 64 or 128");
+  constexpr int kVecs = kGcC * DK / 8;    // vectors of 8 q (k, b) elements of a chunk
+  constexpr int NV = (kVecs + kGcThreads - 1) / kGcThreads;
+  static_assert(RB * CP <= 16 && (NT & 1) == 0, "DK is 32, 64 or 128");
   extern __shared__ __align__(16) uint8_t smem_raw[];
   SM& sm = *reinterpret_cast<SM*>(smem_raw);
   ptx::griddep_launch_dependents();
@@ -137,7 +156,8 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
   }
   ptx::cluster_arrive_release();  // every CTA of the cluster runs: its shared memory may be written
   ptx::cluster_wait_acquire();
-  const int rbS = warp % RB, cS = (warp / RB) * (kGcV / CP);  // this warp's part of the state
+  const bool has_state = warp < RB * CP;
+  const int rbS = warp % RB, cS = has_state ? (warp / RB) * (kGcV / CP) : 0;  // this warp's part of the state
   const int rowS = rbS * 16 + g;
   float* gstate = p.state + (static_cast<int64_t>(slot) * p.heads + h) * p.dim * p.vdim + v0;
   float S[NT][4];
@@ -147,9 +167,10 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int c = rowS + (e >> 1) * 8, col = cS + n * 8 + 2 * t4 + (e & 1);
-      S[n][e] = (fresh || c >= p.dim || col >= nv) ? 0.f : gstate[static_cast<int64_t>(c) * p.vdim + col];
+      S[n][e] = (fresh || !has_state || c >= p.dim || col >= nv) ? 0.f : gstate[static_cast<int64_t>(c) * p.vdim + col];
     }
   auto publish_state = [&] {
+    if (!has_state) return;
 #pragma unroll
     for (int n = 0; n < NT; ++n) {
       const int at = rowS * SM::kV + cS + n * 8 + 2 * t4;
@@ -163,93 +184,107 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
     }
   };
   publish_state();
-  const int rb = warp >> 1, cO = (warp & 1) * 32;  // this warp's 16 x 32 part of the chunk's output
+  const int rb = warp >> 2, cO = (warp & 3) * 16;  // this warp's 16 x 16 part of the chunk's output
   const int nchunks = (len + kGcC - 1) / kGcC;
 
-  // q, k and v of a chunk, requested one chunk ahead
-  uint4 rq[NV], rk[NV], rv[2];
+  // what a chunk reads, requested one chunk ahead: q, k and b by vectors, v, and the table of block borders
+  uint4 rq[NV], rk[NV], rv;
+  float rb8[NV][8], rref[2];
   auto request = [&](int chunk) {
-    const int base = chunk * kGcC;
+    const int base = chunk * kGcC, last = min(kGcC, len - base) - 1;
+    const float* cum = p.cum + static_cast<int64_t>(t_beg + base) * hk + h * p.dim;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int e = tid + i * kGcThreads, t = base + e / (DK / 8), c = (e % (DK / 8)) * 8;
+      const int e = tid + i * kGcThreads, t = e / (DK / 8), c = (e % (DK / 8)) * 8;
       rq[i] = rk[i] = make_uint4(0, 0, 0, 0);
-      if (t < len && c < p.dim) {
-        const int64_t at = static_cast<int64_t>(t_beg + t) * p.row + h * p.dim + c;
-        rq[i] = *reinterpret_cast<const uint4*>(p.q + at);
-        rk[i] = *reinterpret_cast<const uint4*>(p.k + at);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) rb8[i][j] = 0.f;
+      if (e < kVecs && c < p.dim) {
+        ldf8(cum + static_cast<int64_t>(min(t, last)) * hk + c, rb8[i]);  // tokens past the end do not decay
+        if (t <= last) {
+          const int64_t at = static_cast<int64_t>(t_beg + base + t) * p.row + h * p.dim + c;
+          rq[i] = *reinterpret_cast<const uint4*>(p.q + at);
+          rk[i] = *reinterpret_cast<const uint4*>(p.k + at);
+        }
       }
     }
+    rv = make_uint4(0, 0, 0, 0);
+    if (tid / 8 <= last && (tid % 8) * 8 < nv)
+      rv = *reinterpret_cast<const uint4*>(p.v + static_cast<int64_t>(t_beg + base + tid / 8) * p.row + h * p.vdim + v0 + (tid % 8) * 8);
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
-      const int e = tid + i * kGcThreads, t = base + e / 8, c = (e % 8) * 8;
-      rv[i] = make_uint4(0, 0, 0, 0);
-      if (t < len && c < nv)
-        rv[i] = *reinterpret_cast<const uint4*>(p.v + static_cast<int64_t>(t_beg + t) * p.row + h * p.vdim + v0 + c);
+      const int e = tid + i * kGcThreads, blk = e / DK, c = e % DK;
+      rref[i] = (e < 5 * DK && blk > 0 && c < p.dim) ? cum[static_cast<int64_t>(min(blk * kGcB - 1, last)) * hk + c] : 0.f;
     }
   };
+  auto keep_borders = [&](int chunk) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+      if (tid + i * kGcThreads < 5 * DK) sm.ref[chunk & 1][tid + i * kGcThreads] = rref[i];
+  };
   request(0);
+  keep_borders(0);
+  if (tid < 4) sm.wide[tid] = 0;
+  __syncthreads();
 
   for (int ch = 0; ch < nchunks; ++ch) {
     const int base = ch * kGcC, n_tok = min(kGcC, len - base);
-    // b at token t of the chunk (tokens past the end do not decay)
-    const float* cum = p.cum + static_cast<int64_t>(t_beg + base) * hk + h * p.dim;
-    auto b_at = [&](int t) { return cum + static_cast<int64_t>(min(t, n_tok - 1)) * hk; };
-    // ---- 1. q', k~, v and the block borders' table into shared memory
-    if (tid < 4) sm.wide[tid] = 0;
-    for (int e = tid; e < 5 * DK; e += kGcThreads) {
-      const int i = e / DK, c = e % DK;
-      sm.ref[e] = (i == 0 || c >= p.dim) ? 0.f : b_at(i * kGcB - 1)[c];
-    }
+    const float* ref = sm.ref[ch & 1];
+    // ---- 1. q', q e^b, k~, v and the factor tables into shared memory
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int e = tid + i * kGcThreads, t = e / (DK / 8), c = (e % (DK / 8)) * 8, blk = t / kGcB;
-      float q8[8], k8[8];
-      unpack8<bf>(rq[i], q8);
-      unpack8<bf>(rk[i], k8);
-      if (c < p.dim) {
-        float b8[8], lo8[8], hi8[8];
-        ldf8(b_at(t) + c, b8);
-        ldf8(b_at(blk * kGcB + kGcB - 1) + c, hi8);
-        if (blk > 0) ldf8(b_at(blk * kGcB - 1) + c, lo8);
+      if (e < kVecs) {
+        float q8[8], k8[8], i8[8], lo8[8], hi8[8];
+        unpack8<bf>(rq[i], q8);
+        unpack8<bf>(rk[i], k8);
+        ldf8(ref + blk * DK + c, lo8);
+        ldf8(ref + (blk + 1) * DK + c, hi8);
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-          q8[j] *= p.q_scale * __expf(b8[j] - (blk > 0 ? lo8[j] : 0.f));
-          k8[j] *= __expf(hi8[j] - b8[j]);
+          q8[j] *= p.q_scale;
+          i8[j] = q8[j] * __expf(rb8[i][j]);
+          q8[j] *= __expf(rb8[i][j] - lo8[j]);
+          k8[j] *= __expf(hi8[j] - rb8[i][j]);
         }
+        auto put = [&](const float (&x)[8], bf* dh, bf* dl) {
+          uint4 hi, lo;
+          split2(x[0], x[1], hi.x, lo.x);
+          split2(x[2], x[3], hi.y, lo.y);
+          split2(x[4], x[5], hi.z, lo.z);
+          split2(x[6], x[7], hi.w, lo.w);
+          *reinterpret_cast<uint4*>(dh + t * SM::kQ + c) = hi;
+          *reinterpret_cast<uint4*>(dl + t * SM::kQ + c) = lo;
+        };
+        put(q8, sm.qh, sm.ql);
+        put(i8, sm.ih, sm.il);
+        stf8(sm.k + t * SM::kK + c, k8);
       }
-      uint4 hi, lo;
-      split2(q8[0], q8[1], hi.x, lo.x);
-      split2(q8[2], q8[3], hi.y, lo.y);
-      split2(q8[4], q8[5], hi.z, lo.z);
-      split2(q8[6], q8[7], hi.w, lo.w);
-      *reinterpret_cast<uint4*>(sm.qh + t * SM::kQ + c) = hi;
-      *reinterpret_cast<uint4*>(sm.ql + t * SM::kQ + c) = lo;
-      *reinterpret_cast<float4*>(sm.k + t * SM::kK + c) = make_float4(k8[0], k8[1], k8[2], k8[3]);
-      *reinterpret_cast<float4*>(sm.k + t * SM::kK + c + 4) = make_float4(k8[4], k8[5], k8[6], k8[7]);
     }
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int e = tid + i * kGcThreads;
-      *reinterpret_cast<uint4*>(sm.v + (e / 8) * SM::kV + (e % 8) * 8) = rv[i];
+    *reinterpret_cast<uint4*>(sm.v + (tid / 8) * SM::kV + (tid % 8) * 8) = rv;
+    for (int e = tid; e < 10 * DK; e += kGcThreads) {
+      int i, j;
+      gc_tile(e / DK, i, j);
+      const float d = ref[i * DK + e % DK] - ref[(j + 1) * DK + e % DK];
+      if (i == j && d > kGcMaxDecay) sm.wide[i] = 1;
+      sm.fs[e] = __expf(d);
     }
+    for (int e = tid; e < 5 * DK; e += kGcThreads)
+      sm.fe[e] = __expf(ref[4 * DK + e % DK] - (e < 4 * DK ? ref[e + DK] : 0.f));
     __syncthreads();
-    for (int e = tid; e < 4 * DK; e += kGcThreads)
-      if (sm.ref[e] - sm.ref[e + DK] > kGcMaxDecay) sm.wide[e / DK] = 1;
     if (ch + 1 < nchunks) request(ch + 1);
-    __syncthreads();
 
     // ---- 2. scores within the chunk: ten 16 x 16 tiles on and below the diagonal
-    for (int tile = warp; tile < 10; tile += 8) {
-      // 0..5: (1,0) (2,0) (2,1) (3,0) (3,1) (3,2); 6..9: the diagonal
-      const int i = tile >= 6 ? tile - 6 : (tile >= 3 ? 3 : tile >= 1 ? 2 : 1);
-      const int j = tile >= 6 ? i : (tile >= 3 ? tile - 3 : tile >= 1 ? tile - 1 : 0);
+    if (warp < 10) {
+      int i, j;
+      gc_tile(warp, i, j);
       float acc[2][4];
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
       if (i == j && sm.wide[i]) {
+        const float* cum = p.cum + static_cast<int64_t>(t_beg + base) * hk + h * p.dim;
         // one score at a time: entry e of the fragment
 #pragma unroll 1
         for (int e = 0; e < 8; ++e) {
@@ -258,7 +293,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
           if (s <= t && t < n_tok) {
             const bf* qr = p.q + static_cast<int64_t>(t_beg + base + t) * p.row + h * p.dim;
             const bf* kr = p.k + static_cast<int64_t>(t_beg + base + s) * p.row + h * p.dim;
-            const float *bt = b_at(t), *bs = b_at(s);
+            const float *bt = cum + static_cast<int64_t>(t) * hk, *bs = cum + static_cast<int64_t>(s) * hk;
             for (int c = 0; c < p.dim; ++c) x += ldf(qr + c) * ldf(kr + c) * __expf(bt[c] - bs[c]);
             x *= p.q_scale;
           }
@@ -269,26 +304,22 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
               if (n * 4 + f == e) acc[n][f] = x;
         }
       } else {
-        const float *ri = sm.ref + i * DK, *rj = sm.ref + (j + 1) * DK;
+        const float* fs = sm.fs + warp * DK + 2 * t4;
 #pragma unroll
         for (int kk = 0; kk < DK / 16; ++kk) {
           const uint32_t off = static_cast<uint32_t>((i * kGcB + (mi & 1) * 8 + mr) * SM::kQ + kk * 16 + (mi >> 1) * 8);
           uint32_t ah[4], al[4];
           ldmatrix_x4(ptx::smem_u32(sm.qh + off), ah[0], ah[1], ah[2], ah[3]);
           ldmatrix_x4(ptx::smem_u32(sm.ql + off), al[0], al[1], al[2], al[3]);
-          float f[4];  // factors of channels 2 t4, + 1, + 8, + 9
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int c = kk * 16 + 2 * t4 + (e >> 1) * 8 + (e & 1);
-            f[e] = __expf(ri[c] - rj[c]);
-          }
+          // factors of channels 2 t4, + 1 and + 8, + 9
+          const float2 f0 = *reinterpret_cast<const float2*>(fs + kk * 16), f1 = *reinterpret_cast<const float2*>(fs + kk * 16 + 8);
 #pragma unroll
           for (int n = 0; n < 2; ++n) {
             const float* kr = sm.k + (j * kGcB + n * 8 + g) * SM::kK + kk * 16 + 2 * t4;
             const float2 x = *reinterpret_cast<const float2*>(kr), y = *reinterpret_cast<const float2*>(kr + 8);
             uint32_t bh0, bl0, bh1, bl1;
-            split2(x.x * f[0], x.y * f[1], bh0, bl0);
-            split2(y.x * f[2], y.y * f[3], bh1, bl1);
+            split2(x.x * f0.x, x.y * f0.y, bh0, bl0);
+            split2(y.x * f1.x, y.y * f1.y, bh1, bl1);
             mma16816<bf>(acc[n], ah[0], ah[1], ah[2], ah[3], bh0, bh1);
             mma16816<bf>(acc[n], ah[0], ah[1], ah[2], ah[3], bl0, bl1);
             mma16816<bf>(acc[n], al[0], al[1], al[2], al[3], bh0, bh1);
@@ -315,62 +346,54 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
     __syncthreads();
 
     // ---- 3. output: state term, then the chunk's own values
-    float O[4][4];
+    float O[2][4];
 #pragma unroll
-    for (int n = 0; n < 4; ++n)
+    for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) O[n][e] = 0.f;
-    {
-      const float* ri = sm.ref + rb * DK;
+    float2 gate[2][2];  // [half][n], on their way while the products run
 #pragma unroll
-      for (int kk = 0; kk < DK / 16; ++kk) {
-        const uint32_t off = static_cast<uint32_t>((rb * kGcB + (mi & 1) * 8 + mr) * SM::kQ + kk * 16 + (mi >> 1) * 8);
-        uint32_t ah[4], al[4];
-        ldmatrix_x4(ptx::smem_u32(sm.qh + off), ah[0], ah[1], ah[2], ah[3]);
-        ldmatrix_x4(ptx::smem_u32(sm.ql + off), al[0], al[1], al[2], al[3]);
-        float f[4];
+    for (int half = 0; half < 2; ++half)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) f[e] = __expf(ri[kk * 16 + 2 * t4 + (e >> 1) * 8 + (e & 1)]);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {  // fragments 0, 1: channels 2 t4, + 1; 2, 3: + 8, + 9
-          const float2 a = cvt2<bf>(ah[e]), b = cvt2<bf>(al[e]);
-          split2((a.x + b.x) * f[(e >> 1) * 2], (a.y + b.y) * f[(e >> 1) * 2 + 1], ah[e], al[e]);
-        }
-#pragma unroll
-        for (int m = 0; m < 2; ++m) {
-          const uint32_t at = static_cast<uint32_t>((kk * 16 + (mi & 1) * 8 + mr) * SM::kV + cO + m * 16 + (mi >> 1) * 8);
-          uint32_t b0, b1, b2, b3, d0, d1, d2, d3;
-          ldmatrix_x4_trans(ptx::smem_u32(sm.sh + at), b0, b1, b2, b3);
-          ldmatrix_x4_trans(ptx::smem_u32(sm.sl + at), d0, d1, d2, d3);
-          mma16816<bf>(O[2 * m], ah[0], ah[1], ah[2], ah[3], b0, b1);
-          mma16816<bf>(O[2 * m + 1], ah[0], ah[1], ah[2], ah[3], b2, b3);
-          mma16816<bf>(O[2 * m], ah[0], ah[1], ah[2], ah[3], d0, d1);
-          mma16816<bf>(O[2 * m + 1], ah[0], ah[1], ah[2], ah[3], d2, d3);
-          mma16816<bf>(O[2 * m], al[0], al[1], al[2], al[3], b0, b1);
-          mma16816<bf>(O[2 * m + 1], al[0], al[1], al[2], al[3], b2, b3);
-        }
+      for (int n = 0; n < 2; ++n) {
+        const int t = rb * 16 + g + half * 8, col = cO + n * 8 + 2 * t4;
+        gate[half][n] = make_float2(0.f, 0.f);
+        if (t < n_tok && col < nv) gate[half][n] = ldf2(p.g + static_cast<int64_t>(t_beg + base + t) * p.row + h * p.vdim + v0 + col);
       }
-      for (int j = 0; j <= rb; ++j) {
-        const uint32_t off = static_cast<uint32_t>((rb * kGcB + (mi & 1) * 8 + mr) * SM::kV + j * kGcB + (mi >> 1) * 8);
-        uint32_t ah[4], al[4];
-        ldmatrix_x4(ptx::smem_u32(sm.ah + off), ah[0], ah[1], ah[2], ah[3]);
-        ldmatrix_x4(ptx::smem_u32(sm.al + off), al[0], al[1], al[2], al[3]);
 #pragma unroll
-        for (int m = 0; m < 2; ++m) {
-          const uint32_t at = static_cast<uint32_t>((j * kGcB + (mi & 1) * 8 + mr) * SM::kV + cO + m * 16 + (mi >> 1) * 8);
-          uint32_t b0, b1, b2, b3;
-          ldmatrix_x4_trans(ptx::smem_u32(sm.v + at), b0, b1, b2, b3);
-          mma16816<bf>(O[2 * m], ah[0], ah[1], ah[2], ah[3], b0, b1);
-          mma16816<bf>(O[2 * m + 1], ah[0], ah[1], ah[2], ah[3], b2, b3);
-          mma16816<bf>(O[2 * m], al[0], al[1], al[2], al[3], b0, b1);
-          mma16816<bf>(O[2 * m + 1], al[0], al[1], al[2], al[3], b2, b3);
-        }
-      }
+    for (int kk = 0; kk < DK / 16; ++kk) {
+      const uint32_t off = static_cast<uint32_t>((rb * kGcB + (mi & 1) * 8 + mr) * SM::kQ + kk * 16 + (mi >> 1) * 8);
+      uint32_t ah[4], al[4];
+      ldmatrix_x4(ptx::smem_u32(sm.ih + off), ah[0], ah[1], ah[2], ah[3]);
+      ldmatrix_x4(ptx::smem_u32(sm.il + off), al[0], al[1], al[2], al[3]);
+      const uint32_t at = static_cast<uint32_t>((kk * 16 + (mi & 1) * 8 + mr) * SM::kV + cO + (mi >> 1) * 8);
+      uint32_t b0, b1, b2, b3, d0, d1, d2, d3;
+      ldmatrix_x4_trans(ptx::smem_u32(sm.sh + at), b0, b1, b2, b3);
+      ldmatrix_x4_trans(ptx::smem_u32(sm.sl + at), d0, d1, d2, d3);
+      mma16816<bf>(O[0], ah[0], ah[1], ah[2], ah[3], b0, b1);
+      mma16816<bf>(O[1], ah[0], ah[1], ah[2], ah[3], b2, b3);
+      mma16816<bf>(O[0], ah[0], ah[1], ah[2], ah[3], d0, d1);
+      mma16816<bf>(O[1], ah[0], ah[1], ah[2], ah[3], d2, d3);
+      mma16816<bf>(O[0], al[0], al[1], al[2], al[3], b0, b1);
+      mma16816<bf>(O[1], al[0], al[1], al[2], al[3], b2, b3);
+    }
+    for (int j = 0; j <= rb; ++j) {
+      const uint32_t off = static_cast<uint32_t>((rb * kGcB + (mi & 1) * 8 + mr) * SM::kV + j * kGcB + (mi >> 1) * 8);
+      uint32_t ah[4], al[4];
+      ldmatrix_x4(ptx::smem_u32(sm.ah + off), ah[0], ah[1], ah[2], ah[3]);
+      ldmatrix_x4(ptx::smem_u32(sm.al + off), al[0], al[1], al[2], al[3]);
+      const uint32_t at = static_cast<uint32_t>((j * kGcB + (mi & 1) * 8 + mr) * SM::kV + cO + (mi >> 1) * 8);
+      uint32_t b0, b1, b2, b3;
+      ldmatrix_x4_trans(ptx::smem_u32(sm.v + at), b0, b1, b2, b3);
+      mma16816<bf>(O[0], ah[0], ah[1], ah[2], ah[3], b0, b1);
+      mma16816<bf>(O[1], ah[0], ah[1], ah[2], ah[3], b2, b3);
+      mma16816<bf>(O[0], al[0], al[1], al[2], al[3], b0, b1);
+      mma16816<bf>(O[1], al[0], al[1], al[2], al[3], b2, b3);
     }
     {
       float s0 = 0.f, s1 = 0.f;
 #pragma unroll
-      for (int n = 0; n < 4; ++n) {
+      for (int n = 0; n < 2; ++n) {
         s0 += O[n][0] * O[n][0] + O[n][1] * O[n][1];
         s1 += O[n][2] * O[n][2] + O[n][3] * O[n][3];
       }
@@ -380,23 +403,25 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
         s1 += __shfl_xor_sync(0xffffffffu, s1, o);
       }
       if (t4 == 0) {
-        sm.part[warp & 1][rb * 16 + g] = s0;
-        sm.part[warp & 1][rb * 16 + g + 8] = s1;
+        sm.part[warp & 3][rb * 16 + g] = s0;
+        sm.part[warp & 3][rb * 16 + g + 8] = s1;
       }
     }
+    if (ch + 1 < nchunks) keep_borders(ch + 1);
     __syncthreads();
     // sums of squares of this CTA's columns to every CTA of the head (two sets by parity: a CTA is at most one chunk ahead)
     if (tid < kGcC) {
-      const float s = sm.part[0][tid] + sm.part[1][tid];
+      const float s = (sm.part[0][tid] + sm.part[1][tid]) + (sm.part[2][tid] + sm.part[3][tid]);
       const uint32_t mine = ptx::smem_u32(&sm.ss[ch & 1][rank][tid]);
       for (int d = 0; d < nrank; ++d) ptx::st_shared_cluster_f32(ptx::mapa_shared(mine, d), s);
     }
     ptx::cluster_arrive_release();
 
     // ---- 4. state update (meanwhile the sums travel)
-    {
-      const float* be = sm.ref + 4 * DK;
-      const float d0 = __expf(be[rowS]), d1 = __expf(be[rowS + 8]);
+    if (tid < 4) sm.wide[tid] = 0;
+    if (has_state) {
+      const float* fe = sm.fe + rowS;
+      const float d0 = fe[4 * DK], d1 = fe[4 * DK + 8];
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
         S[n][0] *= d0; S[n][1] *= d0;
@@ -404,7 +429,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
       }
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const float f0 = __expf(be[rowS] - sm.ref[(j + 1) * DK + rowS]), f1 = __expf(be[rowS + 8] - sm.ref[(j + 1) * DK + rowS + 8]);
+        const float f0 = fe[j * DK], f1 = fe[j * DK + 8];
         const float* kc = sm.k + (j * kGcB + 2 * t4) * SM::kK + rowS;
         uint32_t ah[4], al[4];
         split2(kc[0] * f0, kc[SM::kK] * f0, ah[0], al[0]);
@@ -436,12 +461,12 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
         const float scale = rsqrtf(ss / static_cast<float>(p.vdim) + p.eps);
         const int64_t tok = t_beg + base + t;
 #pragma unroll
-        for (int n = 0; n < 4; ++n) {
+        for (int n = 0; n < 2; ++n) {
           const int col = cO + n * 8 + 2 * t4;
           if (col < nv) {
-            const float2 w = ldf2(p.norm + v0 + col), gate = ldf2(p.g + tok * p.row + h * p.vdim + v0 + col);
-            stf2(p.out + tok * p.out_stride + h * p.vdim + v0 + col, O[n][2 * half] * scale * w.x * silu_acc(gate.x),
-                 O[n][2 * half + 1] * scale * w.y * silu_acc(gate.y));
+            const float2 w = ldf2(p.norm + v0 + col), z = gate[half][n];
+            stf2(p.out + tok * p.out_stride + h * p.vdim + v0 + col, O[n][2 * half] * scale * w.x * silu_ex2(z.x),
+                 O[n][2 * half + 1] * scale * w.y * silu_ex2(z.y));
           }
         }
       }
@@ -453,7 +478,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int c = rowS + (e >> 1) * 8, col = cS + n * 8 + 2 * t4 + (e & 1);
-      if (c < p.dim && col < nv) gstate[static_cast<int64_t>(c) * p.vdim + col] = S[n][e];
+      if (has_state && c < p.dim && col < nv) gstate[static_cast<int64_t>(c) * p.vdim + col] = S[n][e];
     }
 }
 
