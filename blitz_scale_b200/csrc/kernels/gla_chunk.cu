@@ -22,7 +22,7 @@
 // products that involve them split their fp32 operands into two bf16 numbers (x = hi + lo, relative error 2^-17) and
 // drop only the lo * lo term.
 //
-// A block of 16 warps owns (row, head, 64 value columns) and walks the row's chunks with the state in registers; everything
+// A block of 16 warps owns (row, head, 64 or 128 value columns) and walks the row's chunks with the state in registers; everything
 // a chunk reads from global memory is requested one chunk (the gates: half a chunk) ahead.  The blocks of one head form a thread-block cluster, which exchanges the 64 partial sums of squares per chunk through
 // distributed shared memory, so that the output norm and the gate are applied here and nothing but the result is
 // written.  (gla_decay_kernel computes b beforehand: every value block of a head needs it.)
@@ -30,12 +30,13 @@
 #include "mma.cuh"
 #include "ptx.cuh"
 #include "scalar.cuh"
+#include "tmap.cuh"
 
 namespace blitz {
 
 constexpr int kGcC = 64;        // tokens per chunk
 constexpr int kGcB = 16;        // tokens per block
-constexpr int kGcV = 64;        // value columns per CTA
+constexpr int kGcV = 64;        // value columns per CTA: this many, or twice as many when that still fills the GPU
 constexpr int kGcThreads = 512;
 constexpr int kGcMaxCluster = 8;
 constexpr float kGcMaxDecay = 80.f;
@@ -102,11 +103,12 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
   lo = pk2<__nv_bfloat16>(x - h.x, y - h.y);
 }
 
-template <int DK>
+template <int DK, int VB>
 struct GcSmem {
   static constexpr int kQ = DK + 8;       // row pitch of q' (bf16)
   static constexpr int kK = DK + 8;       // row pitch of k~ (fp32)
-  static constexpr int kV = kGcV + 8;     // row pitch of v, S, A (bf16)
+  static constexpr int kV = VB + 8;       // row pitch of v and S (bf16)
+  static constexpr int kA = kGcC + 8;     // row pitch of A (bf16)
   static constexpr int kParts = kGcMaxCluster;
   float k[kGcC * kK];
   float ref[2][5 * DK];                   // r_0 .. r_4 (r_4 = b_end), by parity of the chunk
@@ -118,7 +120,7 @@ struct GcSmem {
   __nv_bfloat16 qh[kGcC * kQ], ql[kGcC * kQ];  // q'
   __nv_bfloat16 ih[kGcC * kQ], il[kGcC * kQ];  // q e^b
   __nv_bfloat16 v[kGcC * kV];
-  __nv_bfloat16 ah[kGcC * kV], al[kGcC * kV];
+  __nv_bfloat16 ah[kGcC * kA], al[kGcC * kA];
   __nv_bfloat16 sh[DK * kV], sl[DK * kV];
 };
 
@@ -128,13 +130,14 @@ __device__ __forceinline__ void gc_tile(int tile, int& i, int& j) {
   j = tile >= 6 ? i : (tile >= 3 ? tile - 3 : tile >= 1 ? tile - 1 : 0);
 }
 
-template <int DK>
+template <int DK, int VB>
 __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunkParams p) {
   using bf = __nv_bfloat16;
-  using SM = GcSmem<DK>;
+  using SM = GcSmem<DK, VB>;
   constexpr int RB = DK / 16;             // 16-row blocks of the state
   constexpr int CP = RB >= 4 ? 16 / RB : 4;  // warps that share a row block of it (DK = 32: half the warps have no part)
-  constexpr int NT = kGcV / CP / 8;       // 8-column tiles of the state per warp
+  constexpr int NT = VB / CP / 8;       // 8-column tiles of the state per warp
+  constexpr int NO = VB / 32;             // 8-column tiles of a chunk's output per warp
   constexpr int kVecs = kGcC * DK / 8;    // vectors of 8 q (k, b) elements of a chunk
   constexpr int NV = (kVecs + kGcThreads - 1) / kGcThreads;
   static_assert(RB * CP <= 16 && (NT & 1) == 0, "DK is 32, 64 or 128");
@@ -145,7 +148,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const int mi = lane >> 3, mr = lane & 7;
   const int h = blockIdx.y, r = blockIdx.z, nrank = gridDim.x, rank = blockIdx.x;
-  const int v0 = blockIdx.x * kGcV, nv = min(kGcV, p.vdim - v0);
+  const int v0 = blockIdx.x * VB, nv = min(VB, p.vdim - v0);
   const int slot = p.seq_slot[r];
   const int t_beg = p.tok_indptr[r], len = p.tok_indptr[r + 1] - t_beg;
   const int hk = p.heads * p.dim;
@@ -157,7 +160,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
   ptx::cluster_arrive_release();  // every CTA of the cluster runs: its shared memory may be written
   ptx::cluster_wait_acquire();
   const bool has_state = warp < RB * CP;
-  const int rbS = warp % RB, cS = has_state ? (warp / RB) * (kGcV / CP) : 0;  // this warp's part of the state
+  const int rbS = warp % RB, cS = has_state ? (warp / RB) * (VB / CP) : 0;  // this warp's part of the state
   const int rowS = rbS * 16 + g;
   float* gstate = p.state + (static_cast<int64_t>(slot) * p.heads + h) * p.dim * p.vdim + v0;
   float S[NT][4];
@@ -184,11 +187,11 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
     }
   };
   publish_state();
-  const int rb = warp >> 2, cO = (warp & 3) * 16;  // this warp's 16 x 16 part of the chunk's output
+  const int rb = warp >> 2, cO = (warp & 3) * (VB / 4);  // this warp's part of the chunk's output
   const int nchunks = (len + kGcC - 1) / kGcC;
 
   // what a chunk reads, requested one chunk ahead: q, k and b by vectors, v, and the table of block borders
-  uint4 rq[NV], rk[NV], rv;
+  uint4 rq[NV], rk[NV], rv[VB / 64];
   float rb8[NV][8], rref[2];
   auto request = [&](int chunk) {
     const int base = chunk * kGcC, last = min(kGcC, len - base) - 1;
@@ -208,9 +211,13 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
         }
       }
     }
-    rv = make_uint4(0, 0, 0, 0);
-    if (tid / 8 <= last && (tid % 8) * 8 < nv)
-      rv = *reinterpret_cast<const uint4*>(p.v + static_cast<int64_t>(t_beg + base + tid / 8) * p.row + h * p.vdim + v0 + (tid % 8) * 8);
+#pragma unroll
+    for (int i = 0; i < VB / 64; ++i) {
+      const int t = tid / 8, c = (tid % 8) * 8 + i * 64;
+      rv[i] = make_uint4(0, 0, 0, 0);
+      if (t <= last && c < nv)
+        rv[i] = *reinterpret_cast<const uint4*>(p.v + static_cast<int64_t>(t_beg + base + t) * p.row + h * p.vdim + v0 + c);
+    }
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const int e = tid + i * kGcThreads, blk = e / DK, c = e % DK;
@@ -261,7 +268,8 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
         stf8(sm.k + t * SM::kK + c, k8);
       }
     }
-    *reinterpret_cast<uint4*>(sm.v + (tid / 8) * SM::kV + (tid % 8) * 8) = rv;
+#pragma unroll
+    for (int i = 0; i < VB / 64; ++i) *reinterpret_cast<uint4*>(sm.v + (tid / 8) * SM::kV + (tid % 8) * 8 + i * 64) = rv[i];
     for (int e = tid; e < 10 * DK; e += kGcThreads) {
       int i, j;
       gc_tile(e / DK, i, j);
@@ -338,7 +346,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
           }
           uint32_t hi, lo;
           split2(x, y, hi, lo);
-          const int at = (i * kGcB + t) * SM::kV + j * kGcB + s;
+          const int at = (i * kGcB + t) * SM::kA + j * kGcB + s;
           *reinterpret_cast<uint32_t*>(sm.ah + at) = hi;
           *reinterpret_cast<uint32_t*>(sm.al + at) = lo;
         }
@@ -346,16 +354,16 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
     __syncthreads();
 
     // ---- 3. output: state term, then the chunk's own values
-    float O[2][4];
+    float O[NO][4];
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+    for (int n = 0; n < NO; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) O[n][e] = 0.f;
-    float2 gate[2][2];  // [half][n], on their way while the products run
+    float2 gate[2][NO];  // [half][n], on their way while the products run
 #pragma unroll
     for (int half = 0; half < 2; ++half)
 #pragma unroll
-      for (int n = 0; n < 2; ++n) {
+      for (int n = 0; n < NO; ++n) {
         const int t = rb * 16 + g + half * 8, col = cO + n * 8 + 2 * t4;
         gate[half][n] = make_float2(0.f, 0.f);
         if (t < n_tok && col < nv) gate[half][n] = ldf2(p.g + static_cast<int64_t>(t_beg + base + t) * p.row + h * p.vdim + v0 + col);
@@ -366,34 +374,40 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
       uint32_t ah[4], al[4];
       ldmatrix_x4(ptx::smem_u32(sm.ih + off), ah[0], ah[1], ah[2], ah[3]);
       ldmatrix_x4(ptx::smem_u32(sm.il + off), al[0], al[1], al[2], al[3]);
-      const uint32_t at = static_cast<uint32_t>((kk * 16 + (mi & 1) * 8 + mr) * SM::kV + cO + (mi >> 1) * 8);
-      uint32_t b0, b1, b2, b3, d0, d1, d2, d3;
-      ldmatrix_x4_trans(ptx::smem_u32(sm.sh + at), b0, b1, b2, b3);
-      ldmatrix_x4_trans(ptx::smem_u32(sm.sl + at), d0, d1, d2, d3);
-      mma16816<bf>(O[0], ah[0], ah[1], ah[2], ah[3], b0, b1);
-      mma16816<bf>(O[1], ah[0], ah[1], ah[2], ah[3], b2, b3);
-      mma16816<bf>(O[0], ah[0], ah[1], ah[2], ah[3], d0, d1);
-      mma16816<bf>(O[1], ah[0], ah[1], ah[2], ah[3], d2, d3);
-      mma16816<bf>(O[0], al[0], al[1], al[2], al[3], b0, b1);
-      mma16816<bf>(O[1], al[0], al[1], al[2], al[3], b2, b3);
+#pragma unroll
+      for (int m = 0; m < NO / 2; ++m) {
+        const uint32_t at = static_cast<uint32_t>((kk * 16 + (mi & 1) * 8 + mr) * SM::kV + cO + m * 16 + (mi >> 1) * 8);
+        uint32_t b0, b1, b2, b3, d0, d1, d2, d3;
+        ldmatrix_x4_trans(ptx::smem_u32(sm.sh + at), b0, b1, b2, b3);
+        ldmatrix_x4_trans(ptx::smem_u32(sm.sl + at), d0, d1, d2, d3);
+        mma16816<bf>(O[2 * m], ah[0], ah[1], ah[2], ah[3], b0, b1);
+        mma16816<bf>(O[2 * m + 1], ah[0], ah[1], ah[2], ah[3], b2, b3);
+        mma16816<bf>(O[2 * m], ah[0], ah[1], ah[2], ah[3], d0, d1);
+        mma16816<bf>(O[2 * m + 1], ah[0], ah[1], ah[2], ah[3], d2, d3);
+        mma16816<bf>(O[2 * m], al[0], al[1], al[2], al[3], b0, b1);
+        mma16816<bf>(O[2 * m + 1], al[0], al[1], al[2], al[3], b2, b3);
+      }
     }
     for (int j = 0; j <= rb; ++j) {
-      const uint32_t off = static_cast<uint32_t>((rb * kGcB + (mi & 1) * 8 + mr) * SM::kV + j * kGcB + (mi >> 1) * 8);
+      const uint32_t off = static_cast<uint32_t>((rb * kGcB + (mi & 1) * 8 + mr) * SM::kA + j * kGcB + (mi >> 1) * 8);
       uint32_t ah[4], al[4];
       ldmatrix_x4(ptx::smem_u32(sm.ah + off), ah[0], ah[1], ah[2], ah[3]);
       ldmatrix_x4(ptx::smem_u32(sm.al + off), al[0], al[1], al[2], al[3]);
-      const uint32_t at = static_cast<uint32_t>((j * kGcB + (mi & 1) * 8 + mr) * SM::kV + cO + (mi >> 1) * 8);
-      uint32_t b0, b1, b2, b3;
-      ldmatrix_x4_trans(ptx::smem_u32(sm.v + at), b0, b1, b2, b3);
-      mma16816<bf>(O[0], ah[0], ah[1], ah[2], ah[3], b0, b1);
-      mma16816<bf>(O[1], ah[0], ah[1], ah[2], ah[3], b2, b3);
-      mma16816<bf>(O[0], al[0], al[1], al[2], al[3], b0, b1);
-      mma16816<bf>(O[1], al[0], al[1], al[2], al[3], b2, b3);
+#pragma unroll
+      for (int m = 0; m < NO / 2; ++m) {
+        const uint32_t at = static_cast<uint32_t>((j * kGcB + (mi & 1) * 8 + mr) * SM::kV + cO + m * 16 + (mi >> 1) * 8);
+        uint32_t b0, b1, b2, b3;
+        ldmatrix_x4_trans(ptx::smem_u32(sm.v + at), b0, b1, b2, b3);
+        mma16816<bf>(O[2 * m], ah[0], ah[1], ah[2], ah[3], b0, b1);
+        mma16816<bf>(O[2 * m + 1], ah[0], ah[1], ah[2], ah[3], b2, b3);
+        mma16816<bf>(O[2 * m], al[0], al[1], al[2], al[3], b0, b1);
+        mma16816<bf>(O[2 * m + 1], al[0], al[1], al[2], al[3], b2, b3);
+      }
     }
     {
       float s0 = 0.f, s1 = 0.f;
 #pragma unroll
-      for (int n = 0; n < 2; ++n) {
+      for (int n = 0; n < NO; ++n) {
         s0 += O[n][0] * O[n][0] + O[n][1] * O[n][1];
         s1 += O[n][2] * O[n][2] + O[n][3] * O[n][3];
       }
@@ -461,7 +475,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
         const float scale = rsqrtf(ss / static_cast<float>(p.vdim) + p.eps);
         const int64_t tok = t_beg + base + t;
 #pragma unroll
-        for (int n = 0; n < 2; ++n) {
+        for (int n = 0; n < NO; ++n) {
           const int col = cO + n * 8 + 2 * t4;
           if (col < nv) {
             const float2 w = ldf2(p.norm + v0 + col), z = gate[half][n];
@@ -482,15 +496,24 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
     }
 }
 
-template <int DK>
+template <int DK, int VB>
 static cudaError_t launch_gla_chunk(const GlaChunkParams& p, int rows, cudaStream_t stream) {
+  auto kern = gla_chunk_kernel<DK, VB>;
+  constexpr int smem = (int)sizeof(GcSmem<DK, VB>);
+  static_assert(smem <= 227 * 1024, "shared memory");
   static PerDeviceOnce once;
-  cudaError_t e = once.run([] {
-    return cudaFuncSetAttribute(gla_chunk_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(GcSmem<DK>));
-  });
+  cudaError_t e = once.run([&] { return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); });
   if (e != cudaSuccess) return e;
-  const unsigned vb = (p.vdim + kGcV - 1) / kGcV;
-  return launch_pdl_cluster(gla_chunk_kernel<DK>, dim3(vb, p.heads, rows), dim3(kGcThreads), sizeof(GcSmem<DK>), vb, stream, p);
+  const unsigned vb = (p.vdim + VB - 1) / VB;
+  return launch_pdl_cluster(kern, dim3(vb, p.heads, rows), dim3(kGcThreads), (size_t)smem, vb, stream, p);
+}
+
+// 128 value columns per block halve the work that every block of a head repeats (scaled operands, scores); 64 give twice
+// as many blocks, which is worth more while they do not fill the GPU.
+template <int DK>
+static cudaError_t launch_gla_width(const GlaChunkParams& p, int rows, int sms, cudaStream_t stream) {
+  const bool wide = p.vdim > kGcV && (int64_t)rows * p.heads * ((p.vdim + kGcV - 1) / kGcV) > sms;
+  return wide ? launch_gla_chunk<DK, 2 * kGcV>(p, rows, stream) : launch_gla_chunk<DK, kGcV>(p, rows, stream);
 }
 
 }  // namespace blitz
@@ -526,8 +549,9 @@ int blitz_gla_chunk(const void* q, const void* k, const void* v, const void* g, 
   cudaError_t e = launch_pdl(gla_decay_kernel, dim3((hk + kGdThreads - 1) / kGdThreads, (max_len + kGcC - 1) / kGcC, rows),
                              dim3(kGdThreads), (size_t)kGcC * rank * sizeof(float), stream, p);
   if (e != cudaSuccess) return (int)e;
-  e = dim <= 32 ? launch_gla_chunk<32>(p, rows, stream) : dim <= 64 ? launch_gla_chunk<64>(p, rows, stream)
-                                                                   : launch_gla_chunk<128>(p, rows, stream);
+  const int sms = device_sm_count();
+  e = dim <= 32 ? launch_gla_width<32>(p, rows, sms, stream) : dim <= 64 ? launch_gla_width<64>(p, rows, sms, stream)
+                                                                        : launch_gla_width<128>(p, rows, sms, stream);
   return (int)e;
 }
 

@@ -34,13 +34,14 @@ struct ConvParams {
   const int32_t* tok_indptr;
   const int32_t* seq_slot;
   int num_tokens, rows, width, taps, num_slots;
+  int span;  // tokens per thread
   int* status;
 };
 
-constexpr int kConvTok = 16;  // tokens per thread
+constexpr int kConvTok = 8;  // tokens a thread loads at once
 constexpr int kConvThreads = 128;
 
-// A thread computes VEC channels of kConvTok consecutive tokens (one token per row in decode).  The last TAPS - 1 inputs
+// A thread computes VEC channels of `span` consecutive tokens (one token per row in decode).  The last TAPS - 1 inputs
 // stay in registers; they are filled where a row's portion begins, from the history or from the sequence's start.
 template <typename T, int VEC, int TAPS>
 __global__ void __launch_bounds__(kConvThreads) conv_causal_kernel(const ConvParams p) {
@@ -58,7 +59,7 @@ __global__ void __launch_bounds__(kConvThreads) conv_causal_kernel(const ConvPar
     w[j] = j >= TAPS - p.taps ? load(reinterpret_cast<const T*>(p.conv) + (j - (TAPS - p.taps)) * p.width + c) : make_float2(0.f, 0.f);
   const float2 xb = load(reinterpret_cast<const T*>(p.x_b) + c), ub = load(reinterpret_cast<const T*>(p.conv_b) + c);
   const bool single = p.tok_indptr == nullptr;
-  const int t0 = single ? blockIdx.y : blockIdx.y * kConvTok, t1 = single ? t0 + 1 : min(p.num_tokens, t0 + kConvTok);
+  const int t0 = single ? blockIdx.y : blockIdx.y * p.span, t1 = single ? t0 + 1 : min(p.num_tokens, t0 + p.span);
   float2 in[TAPS];  // inputs with bias, oldest first; in[TAPS - 1] is the current token's
   auto fill = [&](int b, int t, int first) {  // the inputs before token t of row b, whose portion begins at token `first`
     const int slot = p.seq_slot[b], at = p.pos[t], i = t - first;
@@ -94,27 +95,35 @@ __global__ void __launch_bounds__(kConvThreads) conv_causal_kernel(const ConvPar
     emit(t0, load(x + static_cast<int64_t>(t0) * p.row));
     return;
   }
-  float2 raw[kConvTok];
+  float2 raw[kConvTok], next[kConvTok];
+  auto request = [&](int t, float2 (&dst)[kConvTok]) {
 #pragma unroll
-  for (int k = 0; k < kConvTok; ++k)
-    raw[k] = t0 + k < t1 ? load(x + static_cast<int64_t>(t0 + k) * p.row) : make_float2(0.f, 0.f);
+    for (int k = 0; k < kConvTok; ++k)
+      dst[k] = t + k < t1 ? load(x + static_cast<int64_t>(t + k) * p.row) : make_float2(0.f, 0.f);
+  };
+  request(t0, raw);
   int b = row_of_token(p.tok_indptr, p.rows, t0);
   int first = p.tok_indptr[b], end = p.tok_indptr[b + 1];
   fill(b, t0, first);
+  for (int base = t0; base < t1; base += kConvTok) {
+    request(base + kConvTok, next);
 #pragma unroll
-  for (int k = 0; k < kConvTok; ++k) {
-    const int t = t0 + k;
-    if (t < t1) {
-      if (t >= end) {
-        do {
-          ++b;
-          first = end;
-          end = p.tok_indptr[b + 1];
-        } while (t >= end);
-        fill(b, t, first);
+    for (int k = 0; k < kConvTok; ++k) {
+      const int t = base + k;
+      if (t < t1) {
+        if (t >= end) {
+          do {
+            ++b;
+            first = end;
+            end = p.tok_indptr[b + 1];
+          } while (t >= end);
+          fill(b, t, first);
+        }
+        emit(t, raw[k]);
       }
-      emit(t, raw[k]);
     }
+#pragma unroll
+    for (int k = 0; k < kConvTok; ++k) raw[k] = next[k];
   }
 }
 
@@ -183,7 +192,7 @@ __global__ void __launch_bounds__(kStepThreads) rglru_step_kernel(const ScanPara
 }
 
 template <typename T, int NW, int TS>
-__global__ void __launch_bounds__(NW * 32, 2) rglru_scan_kernel(const ScanParams p) {
+__global__ void __launch_bounds__(NW * 32, 1) rglru_scan_kernel(const ScanParams p) {
   ptx::griddep_launch_dependents();
   ptx::griddep_wait();
   __shared__ float sA[NW][32], sB[NW][32], s_carry[2][32];
@@ -209,23 +218,28 @@ __global__ void __launch_bounds__(NW * 32, 2) rglru_scan_kernel(const ScanParams
   const T* y = reinterpret_cast<const T*>(p.y) + cc;
   T* out = reinterpret_cast<T*>(p.out) + cc;
   int cur = 0;
-  for (int base = t_beg; base < t_end; base += NW * TS, cur ^= 1) {
-    const int t0 = base + warp * TS;
-    float gr[TS], gi[TS], uu[TS], yy[TS];
+  float gr[TS], gi[TS], nr[TS], ni[TS];
+  T uu[TS], yy[TS], nu[TS], ny[TS];
+  auto request = [&](int t0, float (&r_)[TS], float (&i_)[TS], T (&u_)[TS], T (&y_)[TS]) {
 #pragma unroll
-    for (int s = 0; s < TS; ++s) {  // every load of the tile before the first use of one
+    for (int s = 0; s < TS; ++s) {
       const int t = min(t0 + s, t_end - 1);
       const float* gt = p.gates + static_cast<int64_t>(t) * 2 * p.width;
-      gr[s] = gt[rcol];
-      gi[s] = gt[icol];
-      uu[s] = ldf<T>(u + static_cast<int64_t>(t) * p.u_stride);
-      yy[s] = ldf<T>(y + static_cast<int64_t>(t) * p.row);
+      r_[s] = gt[rcol];
+      i_[s] = gt[icol];
+      u_[s] = u[static_cast<int64_t>(t) * p.u_stride];
+      y_[s] = y[static_cast<int64_t>(t) * p.row];
     }
+  };
+  request(t_beg + warp * TS, gr, gi, uu, yy);
+  for (int base = t_beg; base < t_end; base += NW * TS, cur ^= 1) {
+    const int t0 = base + warp * TS;
+    if (base + NW * TS < t_end) request(t0 + NW * TS, nr, ni, nu, ny);  // the next tile's, while this one is computed
     float A = 1.f, B = 0.f;
 #pragma unroll
     for (int s = 0; s < TS; ++s) {
       float a = 1.f, b = 0.f;
-      if (t0 + s < t_end) rglru_gates(rate, gr[s] + rb, gi[s] + ib, uu[s], a, b);
+      if (t0 + s < t_end) rglru_gates(rate, gr[s] + rb, gi[s] + ib, ldf<T>(&uu[s]), a, b);
       gr[s] = a;
       gi[s] = b;
       B = a * B + b;
@@ -240,7 +254,14 @@ __global__ void __launch_bounds__(NW * 32, 2) rglru_scan_kernel(const ScanParams
 #pragma unroll
     for (int s = 0; s < TS; ++s) {
       S = gr[s] * S + gi[s];
-      if (t0 + s < t_end && live) stf<T>(out + static_cast<int64_t>(t0 + s) * p.out_stride, S * gelu_tanh_ex2(yy[s] + yb));
+      if (t0 + s < t_end && live) stf<T>(out + static_cast<int64_t>(t0 + s) * p.out_stride, S * gelu_tanh_ex2(ldf<T>(&yy[s]) + yb));
+    }
+#pragma unroll
+    for (int s = 0; s < TS; ++s) {
+      gr[s] = nr[s];
+      gi[s] = ni[s];
+      uu[s] = nu[s];
+      yy[s] = ny[s];
     }
     __syncthreads();
   }
@@ -261,7 +282,7 @@ __global__ void __launch_bounds__(NW * 32, 2) rglru_scan_kernel(const ScanParams
 template <typename T, int VEC>
 static cudaError_t launch_conv(const ConvParams& p, cudaStream_t stream) {
   const int units = (p.width + VEC - 1) / VEC;
-  const int spans = p.tok_indptr ? (p.num_tokens + kConvTok - 1) / kConvTok : p.num_tokens;
+  const int spans = p.tok_indptr ? (p.num_tokens + p.span - 1) / p.span : p.num_tokens;
   const dim3 grid((units + kConvThreads - 1) / kConvThreads, spans), block(kConvThreads);
   return p.taps <= 4 ? launch_pdl(conv_causal_kernel<T, VEC, 4>, grid, block, 0, stream, p)
                      : launch_pdl(conv_causal_kernel<T, VEC, kMaxTaps>, grid, block, 0, stream, p);
@@ -279,8 +300,8 @@ int blitz_conv_causal(const void* x, int64_t row, const void* x_b, const void* c
   if (num_tokens <= 0 || rows <= 0) return 0;
   if (taps < 1 || taps > kMaxTaps) return -1;
   ConvParams p{x, row, x_b, conv, conv_b, hist, u, u_stride, pos, tok_indptr, seq_slot, num_tokens, rows, width, taps,
-               num_slots, status};
-  if (num_tokens > 65535 * (tok_indptr ? kConvTok : 1)) return -1;
+               num_slots, num_tokens >= 2048 ? 64 : 16, status};
+  if ((tok_indptr ? num_tokens / p.span : num_tokens) >= 65535) return -1;
   cudaError_t e = cudaSuccess;
   // two channels at a time where every row starts on an even element
   const uintptr_t pair = 2 * (dtype == 2 ? 4 : 2);

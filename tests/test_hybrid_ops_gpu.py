@@ -271,7 +271,8 @@ def _cut(n, sizes):
 
 
 @pytest.mark.parametrize("sizes", [[1000], [1], [2, 5, 64, 63, 1, 17], [128, 1, 30]])
-@pytest.mark.parametrize("heads,dim,vdim,rank,tau", [(2, 64, 64, 16, 16.0), (3, 32, 128, 4, 1.0), (2, 12, 22, 5, 2.0), (1, 128, 256, 16, 8.0)])
+@pytest.mark.parametrize("heads,dim,vdim,rank,tau", [(2, 64, 64, 16, 16.0), (3, 32, 128, 4, 1.0), (2, 12, 22, 5, 2.0), (1, 128, 256, 16, 8.0),
+                                                      (16, 48, 200, 8, 1.0), (13, 128, 256, 16, 16.0)])
 @pytest.mark.parametrize("dt", [BF, F32])
 def test_gated_linear_attention(ops, heads, dim, vdim, rank, tau, sizes, dt):
     """Three sequences cut alike, on scattered state slots that hold garbage before; decays from nearly none to nearly
