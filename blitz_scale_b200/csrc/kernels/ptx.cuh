@@ -396,6 +396,11 @@ __device__ __forceinline__ float ex2_poly(float x) {
   return __int_as_float(__float_as_int(p) + (__float_as_int(t) << 23));
 }
 
+__device__ __forceinline__ float sqrt_approx(float x) {
+  float y;
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 // tanh x = 1 - 2 / (e^(2x) + 1) on the special-function unit: absolute error of a few 1e-7, exact limits at +-inf.
 __device__ __forceinline__ float tanh_ex2(float x) {
   return 1.f - __fdividef(2.f, ex2_approx(x * 2.8853900817779268f) + 1.f);

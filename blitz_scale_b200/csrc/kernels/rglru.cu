@@ -154,7 +154,7 @@ __device__ __forceinline__ void rglru_gates(float rate, float r, float i, float 
   a = __expf(la);
   const float x = 2.f * la;  // 1 - a^2 = 1 - e^x, by its series where the difference would lose digits
   const float rest = x > -0.03f ? -x * (1.f + x * (0.5f + x * (0.16666667f + x * 0.041666667f))) : 1.f - a * a;
-  b = sqrtf(rest) * __fdividef(1.f, 1.f + __expf(-i)) * u;
+  b = ptx::sqrt_approx(rest) * __fdividef(1.f, 1.f + __expf(-i)) * u;
 }
 __device__ __forceinline__ float gelu_tanh_ex2(float z) {
   return 0.5f * z * (1.f + ptx::tanh_ex2(0.7978845608028654f * (z + 0.044715f * z * z * z)));
@@ -331,7 +331,7 @@ int blitz_rglru_scan(const void* u, int64_t u_stride, const float* gates, const 
     BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(rglru_step_kernel<T>, grid, dim3(kStepThreads), 0, stream, p)));
   } else {
     const dim3 grid((width + 31) / 32, rows);
-    BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(rglru_scan_kernel<T, 16, 8>, grid, dim3(512), 0, stream, p)));
+    BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(rglru_scan_kernel<T, 32, 4>, grid, dim3(1024), 0, stream, p)));
   }
   return (int)e;
 }
