@@ -116,6 +116,7 @@ struct GcSmem {
   float fe[5 * DK];                       // e^(b_end - r_(j+1)), j = 0 .. 3, and e^(b_end)
   float ss[2][kParts][kGcC];              // partial sums of squares of every cluster rank, by parity of the chunk
   float part[4][kGcC];
+  float norm[VB];
   int wide[4];                            // block whose decay the factored form cannot hold
   __nv_bfloat16 qh[kGcC * kQ], ql[kGcC * kQ];  // q'
   __nv_bfloat16 ih[kGcC * kQ], il[kGcC * kQ];  // q e^b
@@ -232,6 +233,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
   request(0);
   keep_borders(0);
   if (tid < 4) sm.wide[tid] = 0;
+  if (tid < nv) sm.norm[tid] = ldf(p.norm + v0 + tid);
   __syncthreads();
 
   for (int ch = 0; ch < nchunks; ++ch) {
@@ -359,14 +361,15 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
     for (int n = 0; n < NO; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) O[n][e] = 0.f;
-    float2 gate[2][NO];  // [half][n], on their way while the products run
+    uint32_t gate[2][NO];  // [half][n], two values each, on their way while the products run
 #pragma unroll
     for (int half = 0; half < 2; ++half)
 #pragma unroll
       for (int n = 0; n < NO; ++n) {
         const int t = rb * 16 + g + half * 8, col = cO + n * 8 + 2 * t4;
-        gate[half][n] = make_float2(0.f, 0.f);
-        if (t < n_tok && col < nv) gate[half][n] = ldf2(p.g + static_cast<int64_t>(t_beg + base + t) * p.row + h * p.vdim + v0 + col);
+        gate[half][n] = 0u;
+        if (t < n_tok && col < nv)
+          gate[half][n] = *reinterpret_cast<const uint32_t*>(p.g + static_cast<int64_t>(t_beg + base + t) * p.row + h * p.vdim + v0 + col);
       }
 #pragma unroll
     for (int kk = 0; kk < DK / 16; ++kk) {
@@ -478,7 +481,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
         for (int n = 0; n < NO; ++n) {
           const int col = cO + n * 8 + 2 * t4;
           if (col < nv) {
-            const float2 w = ldf2(p.norm + v0 + col), z = gate[half][n];
+            const float2 w = *reinterpret_cast<const float2*>(sm.norm + col), z = cvt2<bf>(gate[half][n]);
             stf2(p.out + tok * p.out_stride + h * p.vdim + v0 + col, O[n][2 * half] * scale * w.x * silu_ex2(z.x),
                  O[n][2 * half + 1] * scale * w.y * silu_ex2(z.y));
           }
@@ -540,7 +543,7 @@ int blitz_gla_chunk(const void* q, const void* k, const void* v, const void* g, 
     return -1;
   for (const void* x : {q, k, v})
     if (reinterpret_cast<uintptr_t>(x) & 15) return -1;
-  if ((reinterpret_cast<uintptr_t>(g) | reinterpret_cast<uintptr_t>(norm) | reinterpret_cast<uintptr_t>(out)) & 3) return -1;
+  if ((reinterpret_cast<uintptr_t>(g) | reinterpret_cast<uintptr_t>(out)) & 3) return -1;
   if (reinterpret_cast<uintptr_t>(cum) & 15) return -1;
   GlaChunkParams p{(const bf*)q, (const bf*)k, (const bf*)v, (const bf*)g, (const bf*)low, row, (const bf*)a2, (const bf*)a2_b,
                    (const bf*)norm, cum, state, (bf*)out, out_stride, pos, tok_indptr, seq_slot, heads, dim, vdim, rank,
