@@ -191,9 +191,22 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
   const int rb = warp >> 2, cO = (warp & 3) * (VB / 4);  // this warp's part of the chunk's output
   const int nchunks = (len + kGcC - 1) / kGcC;
 
-  // what a chunk reads, requested one chunk ahead: q, k and b by vectors, v, and the table of block borders
+  // what a chunk reads, requested one chunk ahead: q, k and b by vectors, v, and the table of block borders (with wide
+  // blocks the registers do not hold b as well: it is read, from L2, when the chunk starts)
+  constexpr bool kAheadB = VB == kGcV;
   uint4 rq[NV], rk[NV], rv[VB / 64];
   float rb8[NV][8], rref[2];
+  auto request_b = [&](int chunk) {
+    const int base = chunk * kGcC, last = min(kGcC, len - base) - 1;
+    const float* cum = p.cum + static_cast<int64_t>(t_beg + base) * hk + h * p.dim;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int e = tid + i * kGcThreads, t = e / (DK / 8), c = (e % (DK / 8)) * 8;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) rb8[i][j] = 0.f;
+      if (e < kVecs && c < p.dim) ldf8(cum + static_cast<int64_t>(min(t, last)) * hk + c, rb8[i]);  // no decay past the end
+    }
+  };
   auto request = [&](int chunk) {
     const int base = chunk * kGcC, last = min(kGcC, len - base) - 1;
     const float* cum = p.cum + static_cast<int64_t>(t_beg + base) * hk + h * p.dim;
@@ -201,17 +214,13 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
     for (int i = 0; i < NV; ++i) {
       const int e = tid + i * kGcThreads, t = e / (DK / 8), c = (e % (DK / 8)) * 8;
       rq[i] = rk[i] = make_uint4(0, 0, 0, 0);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) rb8[i][j] = 0.f;
-      if (e < kVecs && c < p.dim) {
-        ldf8(cum + static_cast<int64_t>(min(t, last)) * hk + c, rb8[i]);  // tokens past the end do not decay
-        if (t <= last) {
-          const int64_t at = static_cast<int64_t>(t_beg + base + t) * p.row + h * p.dim + c;
-          rq[i] = *reinterpret_cast<const uint4*>(p.q + at);
-          rk[i] = *reinterpret_cast<const uint4*>(p.k + at);
-        }
+      if (e < kVecs && c < p.dim && t <= last) {
+        const int64_t at = static_cast<int64_t>(t_beg + base + t) * p.row + h * p.dim + c;
+        rq[i] = *reinterpret_cast<const uint4*>(p.q + at);
+        rk[i] = *reinterpret_cast<const uint4*>(p.k + at);
       }
     }
+    if (kAheadB) request_b(chunk);
 #pragma unroll
     for (int i = 0; i < VB / 64; ++i) {
       const int t = tid / 8, c = (tid % 8) * 8 + i * 64;
@@ -239,6 +248,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
   for (int ch = 0; ch < nchunks; ++ch) {
     const int base = ch * kGcC, n_tok = min(kGcC, len - base);
     const float* ref = sm.ref[ch & 1];
+    if (!kAheadB) request_b(ch);
     // ---- 1. q', q e^b, k~, v and the factor tables into shared memory
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
