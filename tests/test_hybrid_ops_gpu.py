@@ -189,7 +189,7 @@ def _dense(q, k, v, pos, window, first, cap, sink, scale):
 
 
 # (heads, kv heads, dim, page, window, kept, cap, sink)
-ATT = [(8, 1, 64, 64, 72, 6, 30.0, True), (8, 2, 128, 16, 100, 3, 0.0, True), (4, 4, 64, 16, 1, 1, 10.0, False),
+ATT = [(8, 1, 64, 64, 90, 7, 25.0, True), (8, 2, 128, 16, 100, 3, 0.0, True), (4, 4, 64, 16, 1, 1, 10.0, False),
        (4, 2, 128, 64, 130, 0, 5.0, True), (8, 4, 64, 32, 500, 200, 40.0, True), (4, 1, 128, 16, 0, 0, 20.0, True),
        (6, 2, 20, 16, 33, 5, 8.0, True), (4, 2, 64, 16, 70, 130, 25.0, True)]
 
