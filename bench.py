@@ -161,16 +161,19 @@ def main():
                     "(one replica over all N GPUs, fused peer-memory runner against the NCCL runner)")
     ap.add_argument("--hybrid", action="store_true", help="instead: throughput of the hybrid models beside the uniform model of "
                     "equal size, and their kernels against the roofline (bench/hybrid_bench.py; one GPU)")
+    ap.add_argument("--komulorn", action="store_true", help="instead: the same for the Komulorn design, attention with shared caches "
+                    "and a mixture of experts (bench/komulorn_bench.py; one GPU)")
     ap.add_argument("--hybrid-part", default="all", choices=["all", "models", "kernels"])
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm()
-    if args.hybrid:
+    if args.hybrid or args.komulorn:
         sys.path.insert(0, os.path.join(ROOT, "bench"))
         import hybrid_bench
+        import komulorn_bench
         sampler = ClockSampler(0)
         sampler.start()
-        result = hybrid_bench.run(args.hybrid_part)
+        result = (komulorn_bench if args.komulorn else hybrid_bench).run(args.hybrid_part)
         result["clocks"] = sampler.stop()
         print(json.dumps(result))
         return 0

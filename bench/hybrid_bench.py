@@ -49,13 +49,12 @@ def _median(fn, n=7, warmup=3):
     return sorted(times)[n // 2] * 1e-3
 
 
-def bench_models(out, sizes=("h4096", "h2048")):
+def bench_models(out, sizes=("h4096", "h2048"), configs=configs):
     from blitz_scale_b200.runtime import core
     from blitz_scale_b200.runtime.engine import Engine, _bucket
     for size in sizes:
         for name, cfg in configs(size).items():
             eng = Engine(cfg, num_pages=4224, page_size=64, max_batch=256, max_batch_tokens=8192, seed=0, state_slots=256)
-            weights = eng.seg.layout.total_bytes - 2 * VOCAB * cfg.hidden
             g = torch.Generator().manual_seed(1)
             for lens in ([8192], [2048] * 4, [256] * 32):
                 b = eng.new_batch(0, [core.SeqSpec(i, torch.randint(0, VOCAB, (n,), generator=g).tolist(), 4) for i, n in enumerate(lens)])
@@ -80,9 +79,14 @@ def bench_models(out, sizes=("h4096", "h2048")):
                 ops.check_status()
                 b.clear()
                 eng._graphs.clear()
+                weights = eng.seg.layout.total_bytes - 2 * VOCAB * cfg.hidden       # (of the embedding table only rows)
                 if cfg.family == "hybrid":
+                    for e in (s.moe for s in cfg.layer_specs if s.moe):
+                        # experts that no token of the step chooses are not read (expected number, choices being random)
+                        weights -= e.experts * (1 - e.top / e.experts) ** B * 4 * cfg.hidden * e.ff_pad
                     # window and kept tokens of the attention layers; states are read and written
-                    kv = sum(2 * x.kv_heads * x.dim * 2 * min(ctx, x.window + x.keep_first) for x in cfg.run_mixers() if x.kind == "attention")
+                    kv = sum(x.kv_heads * (x.dim + x.vdim) * 2 * (min(ctx, x.window + x.keep_first) if x.window else ctx)
+                             for x in cfg.run_mixers() if x.kind == "attention")
                     data = B * (kv + 2 * cfg.state_bytes_per_sequence())
                 else:
                     data = B * ctx * cfg.kv_bytes_per_token()

@@ -33,6 +33,11 @@
 // pool is zero-filled at creation): masked positions get probability 0, and
 // 0 x NaN would still poison the accumulator.
 //
+// Keys and values may differ in size, and either may be smaller than the tile it is computed in (64 or 128 columns, a
+// multiple of 8): TMA fills the columns behind a head's end with zeros.  A gate (one number per head and row, through a
+// sigmoid) multiplies a head's output as it is stored.  More than 8 query heads per KV head run as several groups that
+// read the same keys and values (the second one from L2).
+//
 // Replaces src/kernel/attention_decode.cu:13-40 and the host-side plan of
 // src/kernel/flashinfer_types.cu:52-80.
 #include "launch.cuh"
@@ -59,6 +64,10 @@ struct DecodeTcParams {
   float* part_o;
   float* part_lse;
   int batch, q_heads, kv_heads, group, page_size, max_pages, num_splits, box_tokens;
+  int kv_div;               // kv_heads counts groups of at most 8 query heads: kv_div of them share a KV head
+  int dim, vdim, page_rows; // page n's token `off` is row n * page_rows + off of both pools
+  const void* gate;         // [batch][gate_stride], a column per query head, or null
+  int64_t gate_stride;
   int tail_box_tokens;  // box height of the second tensor map, used for the last (partly filled) chunk of a sequence
   float scale_log2;
   int window, keep_first;       // 0: every key; else a token sees the last `window` positions and the first `keep_first`
@@ -73,13 +82,16 @@ __device__ __forceinline__ void tc_trace(const DecodeTcParams& p, int n, int slo
   if (p.trace != nullptr && blockIdx.x == 0 && n < kTcTraceItems) p.trace[n * kTcTraceSlots + slot] = clock64();
 }
 
-template <int HD>
+template <int HD, int VD = HD>
 struct TcCfg {
-  static constexpr int kSlabs = HD / 64;
-  static constexpr int kStageBytes = 2 * kSlabs * kTcSlabBytes;
-  static constexpr int kMergeFloats = 4 * 8 * HD + 2 * 4 * 8;
+  static constexpr int kSlabs = HD / 64, kValueSlabs = VD / 64;
+  static constexpr int kStageBytes = (kSlabs + kValueSlabs) * kTcSlabBytes;
+  static constexpr int kMergeFloats = 4 * 8 * VD + 2 * 4 * 8;
   static constexpr int kSmemBytes = kTcStages * kStageBytes + kMergeFloats * 4 + 1024 + 128;
 };
+
+template <typename T>
+__device__ __forceinline__ float head_gate(const T* z) { return 1.f / (1.f + expf(-to_f<T>(*z))); }
 
 // Work item = (sequence, kv head, split).  The kernel is persistent: each CTA walks items
 // blockIdx.x, blockIdx.x + gridDim.x, ... and the producer keeps streaming the next item's pages while
@@ -110,17 +122,18 @@ __device__ __forceinline__ DecItem dec_item(const DecodeTcParams& p, int item) {
   return it;
 }
 
-template <typename T, int HD>
-__global__ void __launch_bounds__(kTcThreads)
-attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_constant__ CUtensorMap tmap_tail,
+template <typename T, int HD, int VD = HD>
+__global__ void __launch_bounds__(kTcThreads, 1)
+attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_k_tail,
+                      const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_v_tail,
                       const DecodeTcParams p) {
-  using Cfg = TcCfg<HD>;
-  constexpr int SL = Cfg::kSlabs;
+  using Cfg = TcCfg<HD, VD>;
+  constexpr int SL = Cfg::kSlabs, SV = Cfg::kValueSlabs;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw_addr = ptx::smem_u32(smem_raw);
   uint8_t* smem = smem_raw + (((raw_addr + 1023u) & ~1023u) - raw_addr);
-  float* mrg_o = reinterpret_cast<float*>(smem + kTcStages * Cfg::kStageBytes);  // [4][8][HD]
-  float* mrg_m = mrg_o + 4 * 8 * HD;                                              // [4][8]
+  float* mrg_o = reinterpret_cast<float*>(smem + kTcStages * Cfg::kStageBytes);  // [4][8][VD]
+  float* mrg_m = mrg_o + 4 * 8 * VD;                                              // [4][8]
   float* mrg_l = mrg_m + 32;                                                      // [4][8]
   uint64_t* full_bar = reinterpret_cast<uint64_t*>(mrg_l + 32);
   uint64_t* empty_bar = full_bar + kTcStages;
@@ -140,8 +153,10 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
     }
     *abort_flag = 0;
     ptx::fence_mbar_init();
-    ptx::tma_prefetch_desc(&tmap);
-    ptx::tma_prefetch_desc(&tmap_tail);
+    ptx::tma_prefetch_desc(&tmap_k);
+    ptx::tma_prefetch_desc(&tmap_v);
+    ptx::tma_prefetch_desc(&tmap_k_tail);
+    ptx::tma_prefetch_desc(&tmap_v_tail);
   }
   ptx::fence_proxy_async_smem();
   __syncthreads();
@@ -183,7 +198,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
         // filled, in the smaller boxes of the second map (a 64-token page with 18 live tokens costs 32 rows)
         const bool tail = ntok < kTcChunk;
         const int bt = tail ? p.tail_box_tokens : p.box_tokens;
-        const CUtensorMap* tm = tail ? &tmap_tail : &tmap;
+        const CUtensorMap *tk = tail ? &tmap_k_tail : &tmap_k, *tv = tail ? &tmap_v_tail : &tmap_v;
         const uint32_t box_bytes = static_cast<uint32_t>(bt) * 128u;
         const int pieces = (ntok + bt - 1) / bt;
         const int last_page = (tok0 + ntok - 1) / ps;
@@ -197,7 +212,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
             if (p.status) atomicCAS(p.status, 0, kStatusTimeoutProducer);
             good = 0;
           } else {
-            ptx::mbar_expect_tx(&full_bar[stage], static_cast<uint32_t>(pieces) * 2u * SL * box_bytes);
+            ptx::mbar_expect_tx(&full_bar[stage], static_cast<uint32_t>(pieces) * (SL + SV) * box_bytes);
           }
         }
         good = __shfl_sync(0xffffffffu, good, 0);
@@ -214,11 +229,11 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
               if (p.status) atomicCAS(p.status, 0, kStatusBadIndex);
               page = 0;
             }
-            const int z = page * 2 * ps + (t % ps);
+            const int z = page * p.page_rows + (t % ps), h = it.h / p.kv_div;
 #pragma unroll
-            for (int s = 0; s < SL; ++s) {
-              ptx::tma_load_3d(sb + s * kTcSlabBytes + i * box_bytes, tm, &full_bar[stage], s * 64, it.h, z);
-              ptx::tma_load_3d(sb + (SL + s) * kTcSlabBytes + i * box_bytes, tm, &full_bar[stage], s * 64, it.h, z + ps);
+            for (int s = 0; s < (SL > SV ? SL : SV); ++s) {
+              if (s < SL) ptx::tma_load_3d(sb + s * kTcSlabBytes + i * box_bytes, tk, &full_bar[stage], s * 64, h, z);
+              if (s < SV) ptx::tma_load_3d(sb + (SL + s) * kTcSlabBytes + i * box_bytes, tv, &full_bar[stage], s * 64, h, z);
             }
           }
         }
@@ -246,13 +261,14 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
     // pause longer than the pipeline can absorb empties the memory pipe, which then costs a full latency to refill.
     // So the next item's descriptor and Q fragments are requested while the current item is being processed.
     auto load_q = [&](const DecItem& d, uint32_t (&a0)[HD / 16], uint32_t (&a2)[HD / 16]) {
-      // Q as A fragments (rows >= G are zero padding; rows 8..15 are never populated since G <= 8)
+      // Q as A fragments (rows >= G and columns >= dim are zero padding; rows 8..15 are never populated since G <= 8)
+      const int cols = g < G ? p.dim : 0;
       const T* qrow = reinterpret_cast<const T*>(p.q) + static_cast<int64_t>(d.b) * p.q_stride +
-                      static_cast<int64_t>(d.h * G + g) * HD;
+                      static_cast<int64_t>(d.h * G + g) * p.dim;
 #pragma unroll
       for (int ks = 0; ks < HD / 16; ++ks) {
-        a0[ks] = g < G ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + 2 * t4) : 0u;
-        a2[ks] = g < G ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + 2 * t4 + 8) : 0u;
+        a0[ks] = ks * 16 < cols ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + 2 * t4) : 0u;
+        a2[ks] = ks * 16 + 8 < cols ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + 2 * t4 + 8) : 0u;
       }
     };
     DecItem it = blockIdx.x < num_items ? dec_item(p, blockIdx.x) : DecItem{};
@@ -269,9 +285,9 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
         nit = dec_item(p, next);
         load_q(nit, nqa0, nqa2);
       }
-      float o[HD / 8][4];
+      float o[VD / 8][4];
 #pragma unroll
-      for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+      for (int i = 0; i < VD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
       float m = -INFINITY, l = 0.f;
       for (int c = it.c_beg; c < it.c_end; ++c) {
         if (ok && !ptx::bounded_mbar_wait(&full_bar[stage], phase, abort_flag)) {
@@ -327,14 +343,14 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
           m = m_new;
           const uint32_t pa0 = pk2<T>(p0, p1), pa2 = pk2<T>(p2, p3);
 #pragma unroll
-          for (int i = 0; i < HD / 8; ++i) {
+          for (int i = 0; i < VD / 8; ++i) {
             o[i][0] *= alpha;
             o[i][1] *= alpha;
           }
           {
             const int tok = tokw + (mi & 1) * 8 + mr;
 #pragma unroll
-            for (int np = 0; np < HD / 16; ++np) {
+            for (int np = 0; np < VD / 16; ++np) {
               const int ch = np * 2 + (mi >> 1);
               const uint32_t addr = vbase + (ch >> 3) * kTcSlabBytes + tok * 128 + (((ch & 7) ^ (tok & 7)) << 4);
               uint32_t b0, b1, b2, b3;
@@ -360,13 +376,14 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
         mrg_l[warp * 8 + g] = l;
       }
 #pragma unroll
-      for (int i = 0; i < HD / 8; ++i) {
+      for (int i = 0; i < VD / 8; ++i) {
         float2 v = make_float2(o[i][0], o[i][1]);
-        *reinterpret_cast<float2*>(&mrg_o[(warp * 8 + g) * HD + i * 8 + 2 * t4]) = v;
+        *reinterpret_cast<float2*>(&mrg_o[(warp * 8 + g) * VD + i * 8 + 2 * t4]) = v;
       }
       asm volatile("bar.sync 1, 128;" ::: "memory");
-      for (int e = threadIdx.x; e < G * HD; e += 128) {
-        const int gg = e / HD, d = e % HD;
+      for (int e = threadIdx.x; e < G * VD; e += 128) {
+        const int gg = e / VD, d = e % VD;
+        if (d >= p.vdim) continue;
         float M = -INFINITY;
 #pragma unroll
         for (int w = 0; w < 4; ++w) M = fmaxf(M, mrg_m[w * 8 + gg]);
@@ -380,21 +397,22 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
           for (int w = 0; w < 4; ++w) {
             const float sc = exp2f(mrg_m[w * 8 + gg] - M);
             L += mrg_l[w * 8 + gg] * sc;
-            O += mrg_o[(w * 8 + gg) * HD + d] * sc;
+            O += mrg_o[(w * 8 + gg) * VD + d] * sc;
           }
         }
         if (with_sink) L += exp2f(sink - M);
-        const float val = L > 0.f ? O / L : 0.f;
+        float val = L > 0.f ? O / L : 0.f;
         if (p.num_splits == 1) {
+          if (p.gate != nullptr) val *= head_gate(reinterpret_cast<const T*>(p.gate) + it.b * p.gate_stride + head);
           T* op = reinterpret_cast<T*>(p.out) + static_cast<int64_t>(it.b) * p.out_stride +
-                  static_cast<int64_t>(head) * HD;
+                  static_cast<int64_t>(head) * p.vdim;
           if (std::is_same<T, __nv_bfloat16>::value)
             reinterpret_cast<__nv_bfloat16*>(op)[d] = __float2bfloat16(val);
           else
             reinterpret_cast<__half*>(op)[d] = __float2half(val);
         } else {
           const int64_t base = (static_cast<int64_t>(it.b) * p.q_heads + head) * p.num_splits + it.split;
-          p.part_o[base * HD + d] = val;
+          p.part_o[base * p.vdim + d] = val;
           if (d == 0) p.part_lse[base] = L > 0.f ? M + log2f(L) : -INFINITY;
         }
       }
@@ -414,13 +432,14 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap, const __grid_con
 template <typename T>
 __global__ void attn_merge_tc_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
                                      T* __restrict__ out, int64_t out_stride, int q_heads, int hd, int num_splits,
-                                     const T* __restrict__ sink) {
+                                     const T* __restrict__ sink, const T* __restrict__ gate, int64_t gate_stride) {
   const int b = blockIdx.x, head = blockIdx.y;
   const int64_t base = (static_cast<int64_t>(b) * q_heads + head) * num_splits;
   float M = -INFINITY;
   for (int s = 0; s < num_splits; ++s) M = fmaxf(M, part_lse[base + s]);
   const float snk = sink ? to_f<T>(sink[head]) * 1.4426950408889634f : -INFINITY;
   M = fmaxf(M, snk);
+  const float g = gate ? head_gate(gate + b * gate_stride + head) : 1.f;
   for (int d = threadIdx.x; d < hd; d += blockDim.x) {
     float acc = 0.f, wsum = 0.f;
     if (M > -INFINITY) {
@@ -431,7 +450,7 @@ __global__ void attn_merge_tc_kernel(const float* __restrict__ part_o, const flo
       }
       if (sink) wsum += exp2f(snk - M);
     }
-    const float val = wsum > 0.f ? acc / wsum : 0.f;
+    const float val = wsum > 0.f ? acc / wsum * g : 0.f;
     T* op = out + static_cast<int64_t>(b) * out_stride + static_cast<int64_t>(head) * hd;
     if (std::is_same<T, __nv_bfloat16>::value)
       reinterpret_cast<__nv_bfloat16*>(op)[d] = __float2bfloat16(val);
@@ -440,17 +459,23 @@ __global__ void attn_merge_tc_kernel(const float* __restrict__ part_o, const flo
   }
 }
 
-template <typename T, int HD>
-static int launch_tc(const CUtensorMap& tm, const CUtensorMap& tm_tail, const DecodeTcParams& p, int batch,
-                     cudaStream_t stream) {
-  auto kern = attn_decode_tc_kernel<T, HD>;
+template <typename T, int HD, int VD>
+static int launch_tc(const CUtensorMap (&tm)[4], const DecodeTcParams& p, int batch, cudaStream_t stream) {
+  using Cfg = TcCfg<HD, VD>;
+  auto kern = attn_decode_tc_kernel<T, HD, VD>;
   static PerDeviceOnce once;
-  cudaError_t e = once.run([&] { return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, TcCfg<HD>::kSmemBytes); });
+  cudaError_t e = once.run([&] { return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes); });
   if (e != cudaSuccess) return (int)e;
   const int items = batch * p.kv_heads * p.num_splits;
   const int sms = device_sm_count();
-  return (int)launch_pdl(kern, dim3(items < sms ? items : sms), dim3(kTcThreads), TcCfg<HD>::kSmemBytes, stream, tm,
-                         tm_tail, p);
+  return (int)launch_pdl(kern, dim3(items < sms ? items : sms), dim3(kTcThreads), Cfg::kSmemBytes, stream, tm[0], tm[1], tm[2],
+                         tm[3], p);
+}
+
+template <typename T>
+static int launch_tc(const CUtensorMap (&tm)[4], const DecodeTcParams& p, int batch, cudaStream_t stream) {
+  if (p.dim > 64) return p.vdim > 64 ? launch_tc<T, 128, 128>(tm, p, batch, stream) : launch_tc<T, 128, 64>(tm, p, batch, stream);
+  return p.vdim > 64 ? launch_tc<T, 64, 128>(tm, p, batch, stream) : launch_tc<T, 64, 64>(tm, p, batch, stream);
 }
 
 }  // namespace blitz
@@ -473,58 +498,58 @@ int64_t blitz_attn_decode_workspace_bytes(int batch, int q_heads, int head_dim, 
   return (int64_t)batch * q_heads * num_splits * (head_dim + 1) * (int64_t)sizeof(float);
 }
 
-// kv_layer: [max_pages][2][page_size][kv_heads][head_dim].  workspace: scratch of
-// blitz_attn_decode_workspace_bytes() bytes (may be null when num_splits == 1).
-// page_size must be a power of two >= 8 (pages smaller than 64 tokens are fetched as
-// several boxes per stage).  q_heads / kv_heads <= 8; head_dim 64 or 128.  window (0 = none) / keep_first, softcap (0 =
-// none) and sink (null = none) as described at the top of the file.
-int blitz_attn_decode(const void* q, int64_t q_stride, const void* kv_layer, const int32_t* indices,
+// k_pool, v_pool: [max_pages][page_rows][kv_heads][dim or vdim], a page's tokens in its first page_size rows (one tensor for
+// keys and values: page_rows = 2 page_size, v_pool at the first value plane).  workspace: scratch of
+// blitz_attn_decode_workspace_bytes() bytes for value heads of vdim (may be null when num_splits == 1).
+// page_size must be a power of two >= 8 (pages smaller than 64 tokens are fetched as several boxes per stage).  dim and
+// vdim: multiples of 8 up to 128.  window (0 = none) / keep_first, softcap (0 = none), sink and gate (null = none) as
+// described at the top of the file.
+int blitz_attn_decode(const void* q, int64_t q_stride, const void* k_pool, const void* v_pool, const int32_t* indices,
                       const int32_t* indptr, const int32_t* last_page_len, void* out, int64_t out_stride,
-                      void* workspace, int batch, int q_heads, int kv_heads, int head_dim, int page_size,
+                      void* workspace, int batch, int q_heads, int kv_heads, int dim, int vdim, int page_size, int page_rows,
                       int max_pages, int num_splits, float sm_scale, int window, int keep_first, float softcap,
-                      const void* sink, int* status, int dtype, cudaStream_t stream) {
+                      const void* sink, const void* gate, int64_t gate_stride, int* status, int dtype, cudaStream_t stream) {
   if (batch <= 0) return 0;
   if (window < 0 || keep_first < 0 || softcap < 0.f) return -1;
-  if (num_splits < 1 || (q_heads % kv_heads) != 0 || (q_stride & 1) || (out_stride & 1)) return -1;
-  const int G = q_heads / kv_heads;
-  if (G > 8 || (head_dim != 64 && head_dim != 128)) return -1;
-  if (page_size < 8 || (page_size & (page_size - 1)) != 0) return -1;
+  if (num_splits < 1 || kv_heads < 1 || (q_heads % kv_heads) != 0 || (q_stride & 1)) return -1;
+  if (dim < 8 || dim > 128 || (dim & 7) || vdim < 8 || vdim > 128 || (vdim & 7)) return -1;
+  if (page_size < 8 || (page_size & (page_size - 1)) != 0 || page_rows < page_size) return -1;
   if (num_splits > 1 && workspace == nullptr) return -1;
+  const int group = q_heads / kv_heads;
+  int div = (group + 7) / 8;
+  while (group % div) ++div;
   const int bt = page_size < kTcChunk ? page_size : kTcChunk;
   const int bt_tail = bt < 16 ? bt : 16;
-  CUtensorMap tm, tm_tail;
-  if (!get_tmap_3d(&tm, kv_layer, (uint64_t)head_dim, (uint64_t)kv_heads, (uint64_t)max_pages * 2 * page_size,
-                   (uint64_t)head_dim * 2, (uint64_t)kv_heads * head_dim * 2, 64, 1, (uint32_t)bt))
-    return -2;
-  if (!get_tmap_3d(&tm_tail, kv_layer, (uint64_t)head_dim, (uint64_t)kv_heads, (uint64_t)max_pages * 2 * page_size,
-                   (uint64_t)head_dim * 2, (uint64_t)kv_heads * head_dim * 2, 64, 1, (uint32_t)bt_tail))
-    return -2;
+  // rows of a pool: those of the last page end with its tokens
+  const uint64_t rows = (uint64_t)(max_pages - 1) * page_rows + page_size;
+  CUtensorMap tm[4];
+  for (int i = 0; i < 4; ++i) {
+    const uint64_t d = i < 2 ? dim : vdim;
+    if (!get_tmap_3d(&tm[i], i < 2 ? k_pool : v_pool, d, (uint64_t)kv_heads, rows, d * 2, d * 2 * kv_heads, 64, 1,
+                     (uint32_t)(i & 1 ? bt_tail : bt)))
+      return -2;
+  }
   DecodeTcParams p;
   p.q = q; p.q_stride = q_stride; p.indices = indices; p.indptr = indptr; p.last_page_len = last_page_len;
   p.out = out; p.out_stride = out_stride;
   p.part_o = reinterpret_cast<float*>(workspace);
-  p.part_lse = p.part_o ? p.part_o + (int64_t)batch * q_heads * num_splits * head_dim : nullptr;
-  p.batch = batch; p.q_heads = q_heads; p.kv_heads = kv_heads; p.group = G; p.page_size = page_size; p.max_pages = max_pages;
+  p.part_lse = p.part_o ? p.part_o + (int64_t)batch * q_heads * num_splits * vdim : nullptr;
+  p.batch = batch; p.q_heads = q_heads; p.kv_heads = kv_heads * div; p.kv_div = div; p.group = group / div;
+  p.page_size = page_size; p.max_pages = max_pages; p.dim = dim; p.vdim = vdim; p.page_rows = page_rows;
   p.num_splits = num_splits; p.box_tokens = bt; p.tail_box_tokens = bt_tail;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = g_tc_trace;
-  p.window = window; p.keep_first = keep_first; p.sink = sink;
+  p.window = window; p.keep_first = keep_first; p.sink = sink; p.gate = gate; p.gate_stride = gate_stride;
   p.cap_scale = softcap > 0.f ? sm_scale / softcap : 0.f; p.cap_log2 = softcap * 1.4426950408889634f;
-  int rc;
-  if (dtype == 1)
-    rc = head_dim == 128 ? launch_tc<__nv_bfloat16, 128>(tm, tm_tail, p, batch, stream)
-                         : launch_tc<__nv_bfloat16, 64>(tm, tm_tail, p, batch, stream);
-  else
-    rc = head_dim == 128 ? launch_tc<__half, 128>(tm, tm_tail, p, batch, stream)
-                         : launch_tc<__half, 64>(tm, tm_tail, p, batch, stream);
+  int rc = dtype == 1 ? launch_tc<__nv_bfloat16>(tm, p, batch, stream) : launch_tc<__half>(tm, p, batch, stream);
   if (rc != 0) return rc;
   if (num_splits > 1) {
-    dim3 grid(batch, q_heads);
-    if (dtype == 1)
-      attn_merge_tc_kernel<__nv_bfloat16><<<grid, head_dim, 0, stream>>>(p.part_o, p.part_lse, (__nv_bfloat16*)out,
-                                                                         out_stride, q_heads, head_dim, num_splits, (const __nv_bfloat16*)sink);
-    else
-      attn_merge_tc_kernel<__half><<<grid, head_dim, 0, stream>>>(p.part_o, p.part_lse, (__half*)out, out_stride,
-                                                                  q_heads, head_dim, num_splits, (const __half*)sink);
+    auto merge = [&](auto type) {
+      using T = decltype(type);
+      attn_merge_tc_kernel<T><<<dim3(batch, q_heads), vdim > 64 ? 128 : 64, 0, stream>>>(
+          p.part_o, p.part_lse, (T*)out, out_stride, q_heads, vdim, num_splits, (const T*)sink, (const T*)gate, gate_stride);
+    };
+    if (dtype == 1) merge(__nv_bfloat16{});
+    else merge(__half{});
     rc = (int)cudaGetLastError();
   }
   return rc;
@@ -568,25 +593,24 @@ static cudaError_t noalloc_setup(int dev) {
   return cudaSuccess;
 }
 
-// Tensor map of one KV layer built on the stack (the cached builder keeps a host-side table; this path keeps nothing).
-static bool noalloc_tmap(CUtensorMap* out, const void* kv_layer, int head_dim, int kv_heads, int max_pages, int page_size,
+// Tensor map of the key or value planes of one KV layer built on the stack (the cached builder keeps a host-side table; this path keeps nothing).
+static bool noalloc_tmap(CUtensorMap* out, const void* pool, int head_dim, int kv_heads, int max_pages, int page_size,
                          int box_tokens) {
   PFN_encodeTiled enc = get_encode_fn();
-  if (!enc || (reinterpret_cast<uintptr_t>(kv_layer) & 15) != 0) return false;
-  cuuint64_t dims[3] = {(cuuint64_t)head_dim, (cuuint64_t)kv_heads, (cuuint64_t)max_pages * 2 * page_size};
+  if (!enc || (reinterpret_cast<uintptr_t>(pool) & 15) != 0) return false;
+  cuuint64_t dims[3] = {(cuuint64_t)head_dim, (cuuint64_t)kv_heads, (cuuint64_t)(2 * max_pages - 1) * page_size};
   cuuint64_t strides[2] = {(cuuint64_t)head_dim * 2, (cuuint64_t)kv_heads * head_dim * 2};
   cuuint32_t box[3] = {64, 1, (cuuint32_t)box_tokens};
   cuuint32_t estr[3] = {1, 1, 1};
-  return enc(out, CU_TENSOR_MAP_DATA_TYPE_UINT16, 3, const_cast<void*>(kv_layer), dims, strides, box, estr,
+  return enc(out, CU_TENSOR_MAP_DATA_TYPE_UINT16, 3, const_cast<void*>(pool), dims, strides, box, estr,
              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
 template <typename T, int HD>
-static int noalloc_launch(const CUtensorMap& tm, const CUtensorMap& tm_tail, const DecodeTcParams& p, int sms,
-                          cudaStream_t stream) {
+static int noalloc_launch(const CUtensorMap (&tm)[4], const DecodeTcParams& p, int sms, cudaStream_t stream) {
   const int items = p.batch * p.kv_heads * p.num_splits;
-  attn_decode_tc_kernel<T, HD><<<items < sms ? items : sms, kTcThreads, TcCfg<HD>::kSmemBytes, stream>>>(tm, tm_tail, p);
+  attn_decode_tc_kernel<T, HD><<<items < sms ? items : sms, kTcThreads, TcCfg<HD>::kSmemBytes, stream>>>(tm[0], tm[1], tm[2], tm[3], p);
   return (int)cudaGetLastError();
 }
 
@@ -615,9 +639,11 @@ extern "C" int blitz_attn_decode_noalloc(const void* q, int64_t q_stride, const 
   if (scratch == nullptr) return (int)cudaErrorInvalidSymbol;
   const int bt = page_size < kTcChunk ? page_size : kTcChunk;
   const int bt_tail = bt < 16 ? bt : 16;
-  CUtensorMap tm, tm_tail;
-  if (!noalloc_tmap(&tm, kv_layer, head_dim, kv_heads, max_pages, page_size, bt)) return -2;
-  if (!noalloc_tmap(&tm_tail, kv_layer, head_dim, kv_heads, max_pages, page_size, bt_tail)) return -2;
+  CUtensorMap tm[4];
+  for (int i = 0; i < 4; ++i) {
+    const char* pool = reinterpret_cast<const char*>(kv_layer) + (i < 2 ? 0 : (int64_t)page_size * kv_heads * head_dim * 2);
+    if (!noalloc_tmap(&tm[i], pool, head_dim, kv_heads, max_pages, page_size, i & 1 ? bt_tail : bt)) return -2;
+  }
   DecodeTcParams p;
   p.q = q; p.q_stride = q_stride; p.indices = indices; p.indptr = indptr; p.last_page_len = last_page_len;
   p.out = out; p.out_stride = out_stride;
@@ -626,24 +652,25 @@ extern "C" int blitz_attn_decode_noalloc(const void* q, int64_t q_stride, const 
   p.batch = batch; p.q_heads = q_heads; p.kv_heads = kv_heads; p.group = G; p.page_size = page_size;
   p.max_pages = max_pages; p.num_splits = num_splits; p.box_tokens = bt; p.tail_box_tokens = bt_tail;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = nullptr;
+  p.kv_div = 1; p.dim = p.vdim = head_dim; p.page_rows = 2 * page_size; p.gate = nullptr; p.gate_stride = 0;
   p.window = 0; p.keep_first = 0; p.sink = nullptr; p.cap_scale = p.cap_log2 = 0.f;
   int sms = 0;
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
   if (sms <= 0) sms = 148;
   int rc;
   if (dtype == 1)
-    rc = head_dim == 128 ? noalloc_launch<__nv_bfloat16, 128>(tm, tm_tail, p, sms, stream)
-                         : noalloc_launch<__nv_bfloat16, 64>(tm, tm_tail, p, sms, stream);
+    rc = head_dim == 128 ? noalloc_launch<__nv_bfloat16, 128>(tm, p, sms, stream)
+                         : noalloc_launch<__nv_bfloat16, 64>(tm, p, sms, stream);
   else
-    rc = head_dim == 128 ? noalloc_launch<__half, 128>(tm, tm_tail, p, sms, stream)
-                         : noalloc_launch<__half, 64>(tm, tm_tail, p, sms, stream);
+    rc = head_dim == 128 ? noalloc_launch<__half, 128>(tm, p, sms, stream)
+                         : noalloc_launch<__half, 64>(tm, p, sms, stream);
   if (rc != 0 || num_splits == 1) return rc;
   dim3 grid(batch, q_heads);
   if (dtype == 1)
     attn_merge_tc_kernel<__nv_bfloat16><<<grid, head_dim, 0, stream>>>(p.part_o, p.part_lse, (__nv_bfloat16*)out, out_stride,
-                                                                       q_heads, head_dim, num_splits, nullptr);
+                                                                       q_heads, head_dim, num_splits, nullptr, nullptr, 0);
   else
     attn_merge_tc_kernel<__half><<<grid, head_dim, 0, stream>>>(p.part_o, p.part_lse, (__half*)out, out_stride, q_heads,
-                                                                head_dim, num_splits, nullptr);
+                                                                head_dim, num_splits, nullptr, nullptr, 0);
   return (int)cudaGetLastError();
 }

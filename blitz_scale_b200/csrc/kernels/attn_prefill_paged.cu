@@ -1,4 +1,4 @@
-// Causal prefill attention over the paged KV cache on tcgen05 for sm_100a: GQA, head_dim 64 or 128, queries of
+// Causal prefill attention over the paged KV cache on tcgen05 for sm_100a: GQA, heads of up to 128, queries of
 // the current chunk against everything the cache holds for the sequence (earlier chunks and the chunk itself).
 //
 // Q comes from the fused QKV activation of the chunk (2-D TMA boxes); K and V come from the paged pool, where
@@ -36,6 +36,10 @@
 // pass over the scores decides both; else the special-function unit does it (tanh being monotonic, the row maximum is
 // capped alone).  The sink is one more term of the row sum at the end.
 //
+// Keys and values may differ in size, and either may be smaller than the tile it is computed in (64 or 128 columns, a
+// multiple of 8): TMA fills the columns behind a head's end with zeros.  A gate (one number per head and row, through a
+// sigmoid) multiplies a head's output rows as they leave tensor memory.
+//
 // Replaces FlashInfer's BatchPrefillWithRaggedKVCacheWrapper / paged wrapper calls and their host Plan()
 // (src/kernel/attention_prefill.cu:11-45, src/kernel/flashinfer_types.cu:24-49).
 #include "launch.cuh"
@@ -52,11 +56,12 @@ constexpr float kPpRescaleAt = 8.f;  // log2 units
 constexpr int kPpWorkInts = 8;   // per (sequence, pair of tiles): first row, rows, first page entry, pages, cached tokens, pair
 
 struct PagedPrefillParams {
-  void* out;  // [tokens, q_heads * HD]
-  int64_t out_stride;
+  void* out;  // [tokens, q_heads * vdim]
+  const void* gate;  // [tokens][gate_stride], a column per query head, or null
+  int64_t out_stride, gate_stride;
   const int32_t* page_indices;  // page ids of every sequence, back to back
   const int32_t* work;          // [entries][kPpWorkInts], heaviest first
-  int entries, q_heads, kv_heads, page_size, box_tokens, oob_row;
+  int entries, q_heads, kv_heads, vdim, page_size, page_rows, box_tokens, oob_row;  // page n's token `off`: pool row n * page_rows + off
   float scale_log2;
   int window, keep_first;     // EXT: a row sees the last `window` positions (0: all) and the first `keep_first`
   float cap_scale, cap_log2;  // EXT: soft cap (cap_log2 > 0): score in log2 units = cap_log2 * tanh(q.k * cap_scale)
@@ -73,11 +78,12 @@ __device__ __forceinline__ void pp_trace(const PagedPrefillParams& p, bool on, i
   if (on && p.trace != nullptr && j < kPpTraceIters) p.trace[(role * kPpTraceIters + j) * kPpTraceSlots + slot] = clock64();
 }
 
-template <int HD>
+template <int HD, int VD>
 struct PpCfg {
-  static constexpr int kTileBytes = kPpTile * HD * 2;  // one Q, K or V tile
-  static constexpr int kSlabs = HD / 64;               // 64-column slabs of 128 rows x 128 bytes
-  static constexpr int kSmemBytes = 6 * kTileBytes + 1024 + 256;  // Q x 2 tiles, K x 2 stages, V x 2 stages
+  static constexpr int kSlabBytes = kPpTile * 128;     // 64 columns of a tile: 128 rows x 128 bytes
+  static constexpr int kSlabs = HD / 64, kValueSlabs = VD / 64;
+  static constexpr int kTileBytes = kSlabs * kSlabBytes, kValueBytes = kValueSlabs * kSlabBytes;  // a Q or K tile, a V tile
+  static constexpr int kSmemBytes = 4 * kTileBytes + 2 * kValueBytes + 1024 + 256;  // Q x 2 tiles, K x 2 stages, V x 2 stages
 };
 
 struct PpItem {
@@ -124,15 +130,15 @@ __device__ __forceinline__ int pp_index(int r, int total) {
   return idx < total ? idx : -1;
 }
 
-template <typename T, int HD, bool POLY, bool EXT>
+template <typename T, int HD, int VD, bool POLY, bool EXT>
 __global__ void __launch_bounds__(kPpThreads, 1)
-attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_kv,
-                          const PagedPrefillParams p) {
-  using C = PpCfg<HD>;
-  constexpr int TB = C::kTileBytes;
+attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
+                          const __grid_constant__ CUtensorMap tmap_v, const PagedPrefillParams p) {
+  using C = PpCfg<HD, VD>;
+  constexpr int TB = C::kTileBytes, VB = C::kValueBytes, SB = C::kSlabBytes;
   constexpr uint32_t kFmt = std::is_same<T, __nv_bfloat16>::value ? 1u : 0u;
   constexpr uint32_t kIdescS = ptx::make_idesc_f16(kFmt, 0u, 0u, 128, 128);
-  constexpr uint32_t kIdescPV = ptx::make_idesc_f16(kFmt, 0u, 1u, 128, HD);
+  constexpr uint32_t kIdescPV = ptx::make_idesc_f16(kFmt, 0u, 1u, 128, VD);
 
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw_addr = ptx::smem_u32(smem_raw);
@@ -140,7 +146,7 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   uint8_t* sQ = smem;            // [2 tiles]
   uint8_t* sK = sQ + 2 * TB;     // [2 stages]
   uint8_t* sV = sK + 2 * TB;     // [2 stages]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + 2 * TB);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + 2 * VB);
   uint64_t* q_full = bars;        // once per item
   uint64_t* q_empty = bars + 1;   // once per item: its last S products are done
   uint64_t* k_full = bars + 2;    // [2] per block
@@ -173,7 +179,8 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
     *abort_flag = 0;
     ptx::fence_mbar_init();
     ptx::tma_prefetch_desc(&tmap_q);
-    ptx::tma_prefetch_desc(&tmap_kv);
+    ptx::tma_prefetch_desc(&tmap_k);
+    ptx::tma_prefetch_desc(&tmap_v);
   }
   if (warp == 8) {
     ptx::tmem_alloc(tmem_slot, 512);
@@ -184,26 +191,25 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   ptx::tc_fence_after_sync();
   const uint32_t tmem_base = *tmem_slot;
   const uint32_t tmem_S = tmem_base;        // S_t (and P_t over its first 64 columns) at + 128 t
-  const uint32_t tmem_O = tmem_base + 256;  // O_t at + HD t
+  const uint32_t tmem_O = tmem_base + 256;  // O_t at + VD t
 
   if (warp == 9) {
     // ------------------------------------------------------------ load warp: Q, then K and V block by block
     // K or V block j -> one tile of 128 token rows: every lane fetches one box (a page, or 64 tokens of one)
     const int bt = p.box_tokens;
     const bool mine = lane < kPpTile / bt;
-    auto box_row = [&](const PpItem& it, int j) {  // this lane's first K row of block j (V: + page_size)
+    auto box_row = [&](const PpItem& it, int j) {  // this lane's first row of block j in the pools
       const int tok = it.block(j) * kPpTile + lane * bt;
       const int slot = tok / p.page_size;
       if (!mine || slot >= it.npages) return p.oob_row;  // past the pool: the box arrives as zeros
-      return p.page_indices[it.pg0 + slot] * 2 * p.page_size + (tok & (p.page_size - 1));
+      return p.page_indices[it.pg0 + slot] * p.page_rows + (tok & (p.page_size - 1));
     };
-    auto load_kv = [&](uint8_t* dst, uint64_t* bar, int kv_head, int row) {
-      if (lane == 0) ptx::mbar_expect_tx(bar, TB);
+    auto load_kv = [&](uint8_t* dst, const CUtensorMap* map, int slabs, uint64_t* bar, int kv_head, int row) {
+      if (lane == 0) ptx::mbar_expect_tx(bar, slabs * SB);
       __syncwarp();
       if (mine) {
 #pragma unroll
-        for (int s = 0; s < C::kSlabs; ++s)
-          ptx::tma_load_3d(dst + s * (TB / C::kSlabs) + lane * bt * 128, &tmap_kv, bar, s * 64, kv_head, row);
+        for (int s = 0; s < slabs; ++s) ptx::tma_load_3d(dst + s * SB + lane * bt * 128, map, bar, s * 64, kv_head, row);
       }
     };
     auto wait = [&](uint64_t* bar, uint32_t parity) {
@@ -224,8 +230,7 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         for (int t = 0; t < it.nt; ++t)
 #pragma unroll
           for (int s = 0; s < C::kSlabs; ++s)
-            ptx::tma_load_2d(sQ + t * TB + s * (TB / C::kSlabs), &tmap_q, q_full, it.head * HD + s * 64,
-                             it.seq_start + it.q0 + t * kPpTile);
+            ptx::tma_load_3d(sQ + t * TB + s * SB, &tmap_q, q_full, s * 64, it.head, it.seq_start + it.q0 + t * kPpTile);
       }
       int row = box_row(it, 0);
       for (int j = 0; j < it.nblk && ok; ++j, ++g) {
@@ -233,10 +238,10 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         // a block's K goes where the K of two blocks ago was, once the S products of that block are done; V likewise
         if (g >= 2) ok = wait(&k_empty[g & 1], ((g - 2) >> 1) & 1);
         if (!ok) break;
-        load_kv(sK + (g & 1) * TB, &k_full[g & 1], it.kv_head, row);
+        load_kv(sK + (g & 1) * TB, &tmap_k, C::kSlabs, &k_full[g & 1], it.kv_head, row);
         if (g >= 2) ok = wait(&v_empty[g & 1], ((g - 2) >> 1) & 1);
         if (!ok) break;
-        load_kv(sV + (g & 1) * TB, &v_full[g & 1], it.kv_head, row == p.oob_row ? row : row + p.page_size);
+        load_kv(sV + (g & 1) * VB, &tmap_v, C::kValueSlabs, &v_full[g & 1], it.kv_head, row);
         row = row_next;
       }
       ++n_items;
@@ -249,20 +254,20 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         const uint32_t a = ptx::smem_u32(sQ + t * TB), bb = ptx::smem_u32(sK + stage * TB);
 #pragma unroll
         for (int k = 0; k < HD / 16; ++k) {
-          const uint32_t off = (k >> 2) * (TB / C::kSlabs) + (k & 3) * 32;
+          const uint32_t off = (k >> 2) * SB + (k & 3) * 32;
           ptx::umma_f16_ss(tmem_S + t * 128, ptx::make_smem_desc(a + off, 16, 1024, ptx::kLayoutSw128),
                            ptx::make_smem_desc(bb + off, 16, 1024, ptx::kLayoutSw128), kIdescS, k != 0 ? 1u : 0u);
         }
         ptx::umma_commit(&s_full[t]);
       };
       auto issue_PV = [&](int t, int stage, bool accumulate) {
-        const uint32_t bb = ptx::smem_u32(sV + stage * TB);
+        const uint32_t bb = ptx::smem_u32(sV + stage * VB);
 #pragma unroll
         for (int k = 0; k < kPpTile / 16; ++k) {
           // A = P in tensor memory: row = lane, 16 tokens = 8 columns.  B = V: N-major, slabs of 64 head-dim
           // columns; 16 tokens (K) advance 2 KB.
-          ptx::umma_f16_ts(tmem_O + t * HD, tmem_S + t * 128 + k * 8,
-                           ptx::make_smem_desc(bb + k * 2048, TB / C::kSlabs, 1024, ptx::kLayoutSw128), kIdescPV,
+          ptx::umma_f16_ts(tmem_O + t * VD, tmem_S + t * 128 + k * 8,
+                           ptx::make_smem_desc(bb + k * 2048, SB, 1024, ptx::kLayoutSw128), kIdescPV,
                            (accumulate || k != 0) ? 1u : 0u);
         }
         ptx::umma_commit(&o_full[t]);
@@ -335,7 +340,7 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
     const int r_ = (warp & 3) * 32 + lane;
     const uint32_t lane_addr = static_cast<uint32_t>((warp & 3) * 32) << 16;
     const uint32_t tS = tmem_S + t * 128 + lane_addr;
-    const uint32_t tO = tmem_O + t * HD + lane_addr;
+    const uint32_t tO = tmem_O + t * VD + lane_addr;
     bool ok = true;
     uint32_t cnt = 0;  // blocks this tile has been through
     bool first = true;
@@ -420,7 +425,7 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
           if (__any_sync(0xffffffffu, grow)) {
             const float alpha = grow ? ptx::ex2_approx(m_ref - mx) : 1.f;
 #pragma unroll 1
-            for (int c = 0; c < HD; c += 32) {
+            for (int c = 0; c < VD; c += 32) {
               uint32_t o[32];
               ptx::tmem_ld_32x32(tO + c, o);
               ptx::tmem_ld_wait();
@@ -495,21 +500,25 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       ptx::tc_fence_after_sync();
       if (EXT && p.sink != nullptr && l > 0.f)
         l += ptx::ex2_approx(to_f<T>(reinterpret_cast<const T*>(p.sink)[it.head]) * 1.4426950408889634f - m_ref);
-      const float inv = l > 0.f ? 1.f / l : 0.f;
-      T* dst = reinterpret_cast<T*>(p.out) + static_cast<int64_t>(it.seq_start + q_idx) * p.out_stride + it.head * HD;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (p.gate != nullptr && q_idx < it.q_len) {
+        const T z = reinterpret_cast<const T*>(p.gate)[static_cast<int64_t>(it.seq_start + q_idx) * p.gate_stride + it.head];
+        inv /= 1.f + expf(-to_f<T>(z));
+      }
+      T* dst = reinterpret_cast<T*>(p.out) + static_cast<int64_t>(it.seq_start + q_idx) * p.out_stride + it.head * p.vdim;
 #pragma unroll 1
-      for (int c = 0; c < HD; c += 32) {
+      for (int c = 0; c < VD; c += 32) {
         uint32_t o[32];
         ptx::tmem_ld_32x32(tO + c, o);
         ptx::tmem_ld_wait();
-        if (c + 32 >= HD) {  // all of this item's output rows are in registers: the next item may overwrite them
+        if (c + 32 >= VD) {  // all of this item's output rows are in registers: the next item may overwrite them
           ptx::tc_fence_before_sync();
           ptx::mbar_arrive(&o_free[t]);
         }
         if (q_idx < it.q_len) {
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
-            *reinterpret_cast<uint4*>(dst + c + i) = make_uint4(
+            if (c + i < p.vdim) *reinterpret_cast<uint4*>(dst + c + i) = make_uint4(
                 pk2<T>(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv),
                 pk2<T>(__uint_as_float(o[i + 2]) * inv, __uint_as_float(o[i + 3]) * inv),
                 pk2<T>(__uint_as_float(o[i + 4]) * inv, __uint_as_float(o[i + 5]) * inv),
@@ -529,16 +538,15 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   }
 }
 
-template <typename T, int HD, bool POLY, bool EXT>
-static int launch_paged_prefill(const CUtensorMap& tq, const CUtensorMap& tkv, const PagedPrefillParams& p, int grid,
-                                cudaStream_t stream) {
+template <typename T, int HD, int VD, bool POLY, bool EXT>
+static int launch_paged_prefill(const CUtensorMap (&tm)[3], const PagedPrefillParams& p, int grid, cudaStream_t stream) {
+  constexpr int kSmem = PpCfg<HD, VD>::kSmemBytes;
   static PerDeviceOnce once;
   cudaError_t e = once.run([] {
-    return cudaFuncSetAttribute(attn_prefill_paged_kernel<T, HD, POLY, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                PpCfg<HD>::kSmemBytes);
+    return cudaFuncSetAttribute(attn_prefill_paged_kernel<T, HD, VD, POLY, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
   });
   if (e != cudaSuccess) return (int)e;
-  attn_prefill_paged_kernel<T, HD, POLY, EXT><<<grid, kPpThreads, PpCfg<HD>::kSmemBytes, stream>>>(tq, tkv, p);
+  attn_prefill_paged_kernel<T, HD, VD, POLY, EXT><<<grid, kPpThreads, kSmem, stream>>>(tm[0], tm[1], tm[2], p);
   return (int)cudaGetLastError();
 }
 
@@ -553,34 +561,42 @@ using namespace blitz;
 // following launch records when its warpgroups and its MMA thread pass each phase of its first work item.
 void blitz_attn_prefill_paged_set_trace(long long* buf) { blitz::g_pp_trace = buf; }
 
-// q: [num_tokens, q_stride >= q_heads * head_dim] of the current chunk, rotated; kv_layer: the
-// layer's pool [max_pages][2][page_size][kv_heads][head_dim], which already holds the chunk's keys and values;
-// out: [num_tokens, q_heads * head_dim].  page_indices: device array of the sequences' page ids, back to back (the
+// q: [num_tokens, q_stride >= q_heads * dim] of the current chunk, rotated; k_pool, v_pool: the layer's pools
+// [max_pages][page_rows][kv_heads][dim or vdim], a page's tokens in its first page_size rows (one tensor for keys and values:
+// page_rows = 2 page_size, v_pool at the first value plane), which already hold the chunk's keys and values;
+// out: [num_tokens, q_heads * vdim].  page_indices: device array of the sequences' page ids, back to back (the
 // lists cover prefix + chunk).  work: device array (16-byte aligned) of `entries` records of 8 int32, one per
 // (sequence, 256 rows of it), heaviest first: first row of the sequence in qkv, rows of the sequence in this chunk,
 // index of its first page id, number of its pages, tokens cached for it (chunk included), which 256-row pair, 0, 0.
-// page_size: a power of two >= 8.  flags bit 0: compute a quarter of the exponentials on the FMA pipe (not with a window,
-// cap or sink).  window (0 = none) / keep_first, softcap (0 = none), sink (null = none): see the top of the file.
-int blitz_attn_prefill_paged(const void* q, int64_t q_stride, const void* kv_layer, void* out, int64_t out_stride,
+// page_size: a power of two >= 8.  dim and vdim: multiples of 8 up to 128.  flags bit 0: compute a quarter of the
+// exponentials on the FMA pipe (not with a window, cap or sink).  window (0 = none) / keep_first, softcap (0 = none), sink
+// and gate (null = none): see the top of the file.
+int blitz_attn_prefill_paged(const void* q, int64_t q_stride, const void* k_pool, const void* v_pool, void* out, int64_t out_stride,
                              const int32_t* page_indices, const int32_t* work, int entries, int num_tokens,
-                             int q_heads, int kv_heads, int head_dim, int page_size, int max_pages, float sm_scale,
-                             int flags, int window, int keep_first, float softcap, const void* sink, int* status,
-                             int dtype, cudaStream_t stream) {
+                             int q_heads, int kv_heads, int dim, int vdim, int page_size, int page_rows, int max_pages,
+                             float sm_scale, int flags, int window, int keep_first, float softcap, const void* sink,
+                             const void* gate, int64_t gate_stride, int* status, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0 || entries <= 0) return 0;
-  if ((head_dim != 64 && head_dim != 128) || (q_heads % kv_heads) != 0 || (out_stride & 7) || (q_stride & 7)) return -1;
+  if (dim < 8 || dim > 128 || (dim & 7) || vdim < 8 || vdim > 128 || (vdim & 7)) return -1;
+  if (kv_heads < 1 || (q_heads % kv_heads) != 0 || (out_stride & 7) || (q_stride & 7)) return -1;
   if (window < 0 || keep_first < 0 || softcap < 0.f) return -1;
-  if (page_size < 8 || (page_size & (page_size - 1)) != 0 || work == nullptr) return -1;
-  if ((reinterpret_cast<uintptr_t>(work) & 15) != 0) return -1;
+  if (page_size < 8 || (page_size & (page_size - 1)) != 0 || page_rows < page_size || work == nullptr) return -1;
+  if ((reinterpret_cast<uintptr_t>(work) & 15) != 0 || (reinterpret_cast<uintptr_t>(out) & 15) != 0) return -1;
   const int bt = page_size < 64 ? page_size : 64;
-  CUtensorMap tq, tkv;
-  if (!get_tmap_2d(&tq, q, (uint64_t)q_heads * head_dim, (uint64_t)num_tokens, (uint64_t)q_stride * 2, 64, kPpTile)) return -2;
-  if (!get_tmap_3d(&tkv, kv_layer, (uint64_t)head_dim, (uint64_t)kv_heads, (uint64_t)max_pages * 2 * page_size,
-                   (uint64_t)head_dim * 2, (uint64_t)kv_heads * head_dim * 2, 64, 1, (uint32_t)bt))
+  // rows of a pool: those of the last page end with its tokens
+  const uint64_t rows = (uint64_t)(max_pages - 1) * page_rows + page_size;
+  CUtensorMap tm[3];
+  if (!get_tmap_3d(&tm[0], q, (uint64_t)dim, (uint64_t)q_heads, (uint64_t)num_tokens, (uint64_t)dim * 2, (uint64_t)q_stride * 2, 64, 1, kPpTile))
     return -2;
+  for (int i = 1; i < 3; ++i) {
+    const uint64_t d = i == 1 ? dim : vdim;
+    if (!get_tmap_3d(&tm[i], i == 1 ? k_pool : v_pool, d, (uint64_t)kv_heads, rows, d * 2, d * 2 * kv_heads, 64, 1, (uint32_t)bt)) return -2;
+  }
   PagedPrefillParams p;
   p.out = out; p.out_stride = out_stride; p.page_indices = page_indices; p.work = work; p.entries = entries;
+  p.gate = gate; p.gate_stride = gate_stride; p.vdim = vdim; p.page_rows = page_rows;
   p.q_heads = q_heads; p.kv_heads = kv_heads; p.page_size = page_size; p.box_tokens = bt;
-  p.oob_row = max_pages * 2 * page_size;
+  p.oob_row = (int)rows;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = g_pp_trace;
   p.window = window; p.keep_first = keep_first; p.sink = sink;
   p.cap_scale = softcap > 0.f ? sm_scale / softcap : 0.f; p.cap_log2 = softcap * 1.4426950408889634f;
@@ -595,16 +611,19 @@ int blitz_attn_prefill_paged(const void* q, int64_t q_stride, const void* kv_lay
   const int sms = device_sm_count();
   const int grid = (int)(total < sms ? total : sms);
   const bool poly = (flags & 1) != 0, ext = window > 0 || softcap > 0.f || sink != nullptr;
-  auto launch = [&](auto type) {
+  auto sized = [&](auto type, auto poly_, auto ext_) {
     using T = decltype(type);
-    if (ext)
-      return head_dim == 128 ? launch_paged_prefill<T, 128, false, true>(tq, tkv, p, grid, stream)
-                             : launch_paged_prefill<T, 64, false, true>(tq, tkv, p, grid, stream);
-    if (poly)
-      return head_dim == 128 ? launch_paged_prefill<T, 128, true, false>(tq, tkv, p, grid, stream)
-                             : launch_paged_prefill<T, 64, true, false>(tq, tkv, p, grid, stream);
-    return head_dim == 128 ? launch_paged_prefill<T, 128, false, false>(tq, tkv, p, grid, stream)
-                           : launch_paged_prefill<T, 64, false, false>(tq, tkv, p, grid, stream);
+    constexpr bool P = decltype(poly_)::value, X = decltype(ext_)::value;
+    if (dim > 64)
+      return vdim > 64 ? launch_paged_prefill<T, 128, 128, P, X>(tm, p, grid, stream)
+                       : launch_paged_prefill<T, 128, 64, P, X>(tm, p, grid, stream);
+    return vdim > 64 ? launch_paged_prefill<T, 64, 128, P, X>(tm, p, grid, stream)
+                     : launch_paged_prefill<T, 64, 64, P, X>(tm, p, grid, stream);
+  };
+  auto launch = [&](auto type) {
+    if (ext) return sized(type, std::false_type{}, std::true_type{});
+    if (poly) return sized(type, std::true_type{}, std::false_type{});
+    return sized(type, std::false_type{}, std::false_type{});
   };
   return dtype == 1 ? launch(__nv_bfloat16{}) : launch(__half{});
 }

@@ -55,7 +55,7 @@ struct DecGemmParams {
   int kb_per_split;  // K blocks per CTA of a cluster
   int slice;         // tokens each cluster rank reduces and stores (multiple of 32: TMEM is read 32 columns at a time)
   int static_w;      // weights do not depend on earlier kernels of the stream
-  float alpha;       // axpy
+  float alpha;       // axpy; soft cap
   int smem_bytes;    // dynamic shared memory of this launch (227 KB, or about half of it for two CTAs per SM)
   int* status;
 };
@@ -100,13 +100,14 @@ __device__ __forceinline__ float dec_f32<__half>(__half v) { return __half2float
 
 __device__ __forceinline__ float dec_silu(float x) { return x / (1.0f + __expf(-x)); }
 
-// EPI: 0 store, 1 add residual, 2 silu(gate)*up, 4 store as fp32, 5 C += alpha * acc with C fp32.  Thread = output feature n; tokens b0 .. min(b0 + 32, b_end).
+// EPI: 0 store, 1 add residual, 2 silu(gate)*up, 4 store as fp32, 5 C += alpha * acc with C fp32, 6 alpha * tanh(acc / alpha)
+// as fp32.  Thread = output feature n; tokens b0 .. min(b0 + 32, b_end).
 // A warp writes 64 contiguous bytes per token.
 template <typename T, int EPI>
 __device__ __forceinline__ void dec_store32(const DecGemmParams& p, const float (&g)[32], const float (&u)[32], int n,
                                             int b0, int b_end) {
   if (n >= p.N) return;
-  if (EPI == 4 || EPI == 5) {
+  if (EPI >= 4) {
     float* cf = reinterpret_cast<float*>(p.C) + n;
     float old[32];
     if (EPI == 5) {
@@ -115,7 +116,7 @@ __device__ __forceinline__ void dec_store32(const DecGemmParams& p, const float 
     }
 #pragma unroll
     for (int i = 0; i < 32; ++i)
-      if (b0 + i < b_end) cf[static_cast<int64_t>(b0 + i) * p.ldc] = EPI == 5 ? old[i] + p.alpha * g[i] : g[i];
+      if (b0 + i < b_end) cf[static_cast<int64_t>(b0 + i) * p.ldc] = EPI == 5 ? old[i] + p.alpha * g[i] : EPI == 6 ? p.alpha * tanhf(g[i] / p.alpha) : g[i];
     return;
   }
   T* c = reinterpret_cast<T*>(p.C) + n;
@@ -533,12 +534,12 @@ int blitz_get_pdl() { return blitz::pdl_flag(); }
 // Whether blitz_gemm_decode takes this problem (the general GEMM handles everything else).
 int blitz_gemm_decode_supported(int M, int N, int K, int b_layout, int epilogue) {
   return M >= 1 && M <= 256 && b_layout == 0 &&
-         ((epilogue >= 0 && epilogue <= 2) || epilogue == 4 || epilogue == 5) && (N & 7) == 0 && (K & 7) == 0;
+         ((epilogue >= 0 && epilogue <= 2) || (epilogue >= 4 && epilogue <= 6)) && (N & 7) == 0 && (K & 7) == 0;
 }
 
 // C = X W (+R | silu-mul).  X [M, lda>=K], W [K, ldb>=columns] row-major, C/R [M, ldc>=N].  dtype 0 fp16, 1 bf16.
 // epilogue 0 store, 1 add R (C may be R), 2 silu(gate)*up with the up columns starting at up_col_off, 4 store with C in
-// fp32, 5 C += alpha * acc with C in fp32.
+// fp32, 5 C += alpha * acc with C in fp32, 6 alpha * tanh(acc / alpha) with C in fp32.
 // static_w != 0 promises that W was not written by kernels still running in this stream (weights), which lets
 // the kernel start streaming it before its predecessor has finished.  split_hint: 0 = choose, 1 = no K split,
 // n = at most n CTAs (a cluster) per 128-feature tile.
@@ -575,12 +576,14 @@ int blitz_gemm_decode(const void* X, int64_t lda, const void* W, int64_t ldb, vo
   if (dtype == 1) {
     e = epilogue == 2   ? launch_dec<__nv_bfloat16, 2>(tx, tw, p, split_hint, sms, stream)
         : epilogue == 4 ? launch_dec<__nv_bfloat16, 4>(tx, tw, p, split_hint, sms, stream)
+        : epilogue == 6 ? launch_dec<__nv_bfloat16, 6>(tx, tw, p, split_hint, sms, stream)
         : epilogue == 5 ? launch_dec<__nv_bfloat16, 5>(tx, tw, p, split_hint, sms, stream)
         : epilogue == 1 ? launch_dec<__nv_bfloat16, 1>(tx, tw, p, split_hint, sms, stream)
                         : launch_dec<__nv_bfloat16, 0>(tx, tw, p, split_hint, sms, stream);
   } else {
     e = epilogue == 2   ? launch_dec<__half, 2>(tx, tw, p, split_hint, sms, stream)
         : epilogue == 4 ? launch_dec<__half, 4>(tx, tw, p, split_hint, sms, stream)
+        : epilogue == 6 ? launch_dec<__half, 6>(tx, tw, p, split_hint, sms, stream)
         : epilogue == 5 ? launch_dec<__half, 5>(tx, tw, p, split_hint, sms, stream)
         : epilogue == 1 ? launch_dec<__half, 1>(tx, tw, p, split_hint, sms, stream)
                         : launch_dec<__half, 0>(tx, tw, p, split_hint, sms, stream);

@@ -55,7 +55,7 @@ constexpr int kPairFinalStagingBytes = kPairSlabsMax * 4 * 4096;  // a pair's la
 struct PairParams {
   void* C;         // fp32 outputs (the 16-bit ones are stored through tmap_c)
   const void* R;
-  float alpha;     // axpy
+  float alpha;     // axpy; soft cap
   int64_t ldc;
   int M, N, K;
   int bnf;         // UMMA N = accumulator columns of a tile (128 or 256)
@@ -597,7 +597,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                     }
                   }
                 }
-                if (EPI == 4 || EPI == 5) {
+                if (EPI >= 4) {
                   // fp32 output: a thread's 32 columns are a whole 128-byte line, stored directly
                   if (row_ok) {
                     float* dst = reinterpret_cast<float*>(p.C) + static_cast<int64_t>(row) * p.ldc + n0 + c;
@@ -612,7 +612,10 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                       if (n0 + c + 8 * jj < p.N) {
                         float o[8];
 #pragma unroll
-                        for (int k = 0; k < 8; ++k) o[k] = EPI == 5 ? old[jj][k] + p.alpha * gt[8 * jj + k] : gt[8 * jj + k];
+                        for (int k = 0; k < 8; ++k)
+                          o[k] = EPI == 5   ? old[jj][k] + p.alpha * gt[8 * jj + k]
+                                 : EPI == 6 ? p.alpha * tanhf(gt[8 * jj + k] / p.alpha)
+                                            : gt[8 * jj + k];
                         ptx::st_global_v8(dst + 8 * jj, o);
                       }
                     }
@@ -775,12 +778,12 @@ void blitz_gemm_pair_set_trace(unsigned long long* buf) { blitz::g_pair_trace = 
 
 // Whether blitz_gemm_pair takes this problem.
 int blitz_gemm_pair_supported(int M, int N, int K, int b_layout, int epilogue) {
-  return M >= 1 && b_layout == 0 && ((epilogue >= 0 && epilogue <= 2) || epilogue == 4 || epilogue == 5) && (N & 7) == 0 && (K & 7) == 0 && N >= 64;
+  return M >= 1 && b_layout == 0 && ((epilogue >= 0 && epilogue <= 2) || (epilogue >= 4 && epilogue <= 6)) && (N & 7) == 0 && (K & 7) == 0 && N >= 64;
 }
 
 // C = A W (+R | silu-mul).  A [M, lda>=K], W [K, ldb>=columns] row-major, C/R [M, ldc>=N].  dtype 0 fp16, 1 bf16.
 // epilogue 0 store, 1 add R (C may be R), 2 silu(gate)*up with the up columns starting at up_col_off, 4 store with C in
-// fp32, 5 C += alpha * acc with C in fp32.
+// fp32, 5 C += alpha * acc with C in fp32, 6 alpha * tanh(acc / alpha) with C in fp32.
 // bnf_hint: accumulator columns per tile (0 = choose, 128 or 256); nacc_hint: tiles per pair that share the
 // activation tiles (0 = choose, 1 or 2); upp_hint: units per CTA pair (0 = choose; -n = cut every tile into n
 // equal K parts, one pair each).
@@ -843,12 +846,14 @@ int blitz_gemm_pair(const void* A, int64_t lda, const void* W, int64_t ldb, void
   if (dtype == 1) {
     return epilogue == 2   ? pair_launch<__nv_bfloat16, 2>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
            : epilogue == 4 ? pair_launch<__nv_bfloat16, 4>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
+           : epilogue == 6 ? pair_launch<__nv_bfloat16, 6>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
            : epilogue == 5 ? pair_launch<__nv_bfloat16, 5>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
            : epilogue == 1 ? pair_launch<__nv_bfloat16, 1>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
                            : pair_launch<__nv_bfloat16, 0>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream);
   }
   return epilogue == 2   ? pair_launch<__half, 2>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
            : epilogue == 4 ? pair_launch<__half, 4>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
+           : epilogue == 6 ? pair_launch<__half, 6>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
            : epilogue == 5 ? pair_launch<__half, 5>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
          : epilogue == 1 ? pair_launch<__half, 1>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
                          : pair_launch<__half, 0>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream);

@@ -12,6 +12,7 @@
 //   silu_mul   C = silu(acc_gate) * acc_up  (gate||up projection; B holds N gate columns, then N up columns)
 //   store f32  C = acc, C in fp32           (what a recurrence takes in 32 bits)
 //   axpy f32   C += alpha * acc, C in fp32  (output projections of models whose residual stream is fp32)
+//   cap f32    C = alpha * tanh(acc / alpha), C in fp32  (soft-capped logits)
 //
 // Block-diagonal products (groups > 1): B is `groups` blocks [K,N] stacked along K; group g takes the K columns of A
 // from g * K on and the N columns of C from g * N on.  An N tile belongs to one group and simply starts its K walk there
@@ -43,7 +44,7 @@ constexpr int kBK = 64;
 constexpr int kGemmThreads = 192;
 constexpr int kMaxSplitK = 16;
 
-enum GemmEpilogue : int { kEpiStore = 0, kEpiAdd = 1, kEpiSiluMul = 2, kEpiPushRS = 3, kEpiStoreF32 = 4, kEpiAxpyF32 = 5 };
+enum GemmEpilogue : int { kEpiStore = 0, kEpiAdd = 1, kEpiSiluMul = 2, kEpiPushRS = 3, kEpiStoreF32 = 4, kEpiAxpyF32 = 5, kEpiCapF32 = 6 };
 
 struct GemmParams {
   void* C;
@@ -71,7 +72,7 @@ struct GemmParams {
   uint32_t wait_value;
   int n_fast;  // tensor-parallel fusion: N runs fastest over the tiles, M blocks start at m_rot (see gemm_tile_blocks)
   int m_rot;
-  float alpha;      // axpy
+  float alpha;      // axpy; soft cap
   int groups;       // diagonal blocks (1: an ordinary product); N and K are those of one block
   int group_tiles;  // N tiles per block
 };
@@ -153,7 +154,7 @@ __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)
 template <typename T, int EPI>
 __device__ __forceinline__ void store_chunk(const GemmParams& p, const float (&acc)[32], const float (&up)[32], int row,
                                             int col0, bool row_ok, int group = 0) {
-  if (EPI == kEpiStoreF32 || EPI == kEpiAxpyF32) {
+  if (EPI == kEpiStoreF32 || EPI == kEpiAxpyF32 || EPI == kEpiCapF32) {
     if (!row_ok) return;
     float* dst = reinterpret_cast<float*>(p.C) + static_cast<int64_t>(row) * p.ldc + static_cast<int64_t>(group) * p.N + col0;
     float old[4][8];
@@ -167,7 +168,10 @@ __device__ __forceinline__ void store_chunk(const GemmParams& p, const float (&a
       if (col0 + j * 8 < p.N) {
         float v[8];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) v[i] = EPI == kEpiAxpyF32 ? old[j][i] + p.alpha * acc[8 * j + i] : acc[8 * j + i];
+        for (int i = 0; i < 8; ++i)
+          v[i] = EPI == kEpiAxpyF32  ? old[j][i] + p.alpha * acc[8 * j + i]
+                 : EPI == kEpiCapF32 ? p.alpha * tanhf(acc[8 * j + i] / p.alpha)
+                                     : acc[8 * j + i];
         ptx::st_global_v8(dst + 8 * j, v);
       }
     }
@@ -575,6 +579,7 @@ static cudaError_t dispatch_epi(int epi, int bn, const CUtensorMap& ta, const CU
     case kEpiAdd: return dispatch_bn<T, B_KMAJOR, kEpiAdd>(bn, ta, tb, p, grid, stream);
     case kEpiSiluMul: return dispatch_bn<T, B_KMAJOR, kEpiSiluMul>(bn, ta, tb, p, grid, stream);
     case kEpiStoreF32: return dispatch_bn<T, B_KMAJOR, kEpiStoreF32>(bn, ta, tb, p, grid, stream);
+    case kEpiCapF32: return dispatch_bn<T, B_KMAJOR, kEpiCapF32>(bn, ta, tb, p, grid, stream);
     case kEpiAxpyF32: return dispatch_bn<T, B_KMAJOR, kEpiAxpyF32>(bn, ta, tb, p, grid, stream);
     case kEpiPushRS: return dispatch_bn<T, B_KMAJOR, kEpiPushRS>(bn, ta, tb, p, grid, stream);
     default: return dispatch_bn<T, B_KMAJOR, kEpiStore>(bn, ta, tb, p, grid, stream);
@@ -592,7 +597,7 @@ int64_t blitz_gemm_workspace_bytes(int sms) { return (int64_t)(sms + 16) * blitz
 // dtype: 0 = fp16, 1 = bf16.  b_layout: 0 = B is [K, ldb>=Ncols] row-major (weights stored in,out),
 // 1 = B is [Ncols, ldb>=K] row-major.  epilogue: 0 store, 1 add residual R (same pitch as C),
 // 2 silu(gate)*up where B carries N gate columns followed (at column `up_col_off`) by N up columns, 4 store with C in
-// fp32, 5 C += alpha * acc with C in fp32.  groups: number of diagonal blocks (see the top of the file), 1 = none.
+// fp32, 5 C += alpha * acc with C in fp32, 6 alpha * tanh(acc / alpha) with C in fp32.  groups: number of diagonal blocks (see the top of the file), 1 = none.
 // bn_hint: 0 = 256-wide tiles, else 64/128/256.  split_hint: 0 = choose, 1 = never split, else the
 // number of K splits.  ws / ws_bytes: fp32 scratch for split-K partials, tickets / num_tickets:
 // zeroed uint32 array (both may be null: the GEMM then never splits).

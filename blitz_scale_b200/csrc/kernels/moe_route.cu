@@ -1,0 +1,214 @@
+// Router of a mixture of experts: from logits to the work list of the grouped products (gemm_grouped.cu), in one kernel.
+//
+//   score(t, e) = sigmoid(z[t][e])                     the `top` largest per token are its experts
+//   weight      = score, or score / sum of the chosen  multiplies the expert's input or its output
+//   shared      = sigmoid(z[t][experts])               multiplies the shared expert's output
+//
+// Every (token, expert) pair gets a row of the sorted activations: pairs of one expert are neighbours, experts follow one
+// another without gaps, the rows of the shared expert (token t is row pairs + t) come last.  Per row: the token it reads and
+// the factors before and after the expert.  `place[t][k]` names the rows of token t.  The work list has one entry (expert,
+// first row, rows) per `tile_rows` rows of an expert.
+//
+// A warp picks a token's experts; the block that finishes last sorts the pairs by expert (counting sort; the order of an
+// expert's rows is not fixed, and nothing that is computed depends on it) and clears the counters for the next launch.
+#include "launch.cuh"
+#include "ptx.cuh"
+#include "scalar.cuh"
+
+namespace blitz {
+
+constexpr int kMoeMaxExperts = 1024;
+
+struct MoeRouteParams {
+  const float* z;        // [tokens][ld]
+  int64_t ld;
+  int tokens, experts, top, shared, weight_on_input, renormalize, tile_rows, max_tiles;
+  int2* pairs;           // [tokens * top] (expert, weight bits), scratch
+  int* counters;         // [experts + 1], zero between launches: rows per expert, finished blocks
+  int* src;              // [rows] token of a sorted row
+  float2* factors;       // [rows] (before, after) the expert
+  int* place;            // [tokens][top + shared]
+  int4* tiles;           // [max_tiles]
+  int* num_tiles;
+  int* status;
+};
+
+// order-preserving map of a float to an unsigned integer
+__device__ __forceinline__ uint32_t order_key(float x) {
+  const uint32_t u = __float_as_uint(x);
+  return (u & 0x80000000u) ? ~u : (u | 0x80000000u);
+}
+
+__global__ void __launch_bounds__(1024) moe_route_kernel(const MoeRouteParams p) {
+  ptx::griddep_launch_dependents();
+  ptx::griddep_wait();
+  extern __shared__ int s_dyn[];
+  int* s_count = s_dyn;                 // [experts]
+  int* s_cursor = s_count + p.experts;  // [experts]
+  int* s_tile = s_cursor + p.experts;   // [experts]
+  uint32_t* s_keys = reinterpret_cast<uint32_t*>(s_tile + p.experts);  // [warps][experts]
+  __shared__ int s_scan[2][33];
+  __shared__ int s_last;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const int E = p.experts, per = p.top + p.shared, pairs = p.tokens * p.top;
+  for (int e = threadIdx.x; e < E; e += blockDim.x) s_count[e] = 0;
+  __syncthreads();
+
+  const int t = blockIdx.x * warps + warp;
+  if (t < p.tokens) {
+    const float* z = p.z + t * p.ld;
+    uint32_t* keys = s_keys + warp * E;
+    uint32_t best = 0;  // this lane's largest key (0: none left) and its expert
+    int best_e = 0x7fffffff;
+    for (int e = lane; e < E; e += 32) {
+      const uint32_t k = max(order_key(z[e]), 1u);
+      keys[e] = k;
+      if (k > best) {
+        best = k;
+        best_e = e;
+      }
+    }
+    float weight = 0.f, sum = 0.f;  // lane k < top keeps the k-th pair's weight (top <= 32), the sum is everyone's
+    int expert = 0;
+    for (int k = 0; k < p.top; ++k) {
+      const uint32_t mx = __reduce_max_sync(0xffffffffu, best);
+      const int e = __reduce_min_sync(0xffffffffu, best == mx ? best_e : 0x7fffffff);
+      const float s = sigmoid_f(z[e]);
+      sum += s;
+      if (lane == k) {
+        weight = s;
+        expert = e;
+      }
+      if ((e & 31) == lane) {  // the expert's owner looks for its next best
+        keys[e] = 0;
+        best = 0;
+        best_e = 0x7fffffff;
+        for (int j = lane; j < E; j += 32)
+          if (keys[j] > best) {
+            best = keys[j];
+            best_e = j;
+          }
+      }
+    }
+    if (lane < p.top) {
+      if (p.renormalize) weight /= sum;
+      p.pairs[t * p.top + lane] = make_int2(expert, __float_as_int(weight));
+      atomicAdd(&s_count[expert], 1);
+    }
+    if (p.shared && lane == 0) {
+      p.src[pairs + t] = t;
+      p.factors[pairs + t] = make_float2(1.f, sigmoid_f(z[E]));
+      p.place[t * per + p.top] = pairs + t;
+    }
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += blockDim.x)
+    if (s_count[e]) atomicAdd(&p.counters[e], s_count[e]);
+  __threadfence();
+  __syncthreads();
+  if (threadIdx.x == 0) s_last = atomicAdd(&p.counters[E], 1) == static_cast<int>(gridDim.x) - 1;
+  __syncthreads();
+  if (!s_last) return;
+  __threadfence();
+
+  // rows and tiles of every expert: exclusive sums over the experts
+  int rows_before = 0, tiles_before = 0;
+  for (int e0 = 0; e0 < E; e0 += blockDim.x) {
+    const int e = e0 + threadIdx.x;
+    const int n = e < E ? __ldcg(&p.counters[e]) : 0;
+    const int nt = (n + p.tile_rows - 1) / p.tile_rows;
+    int a = n, b = nt;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int x = __shfl_up_sync(0xffffffffu, a, o), y = __shfl_up_sync(0xffffffffu, b, o);
+      if (lane >= o) {
+        a += x;
+        b += y;
+      }
+    }
+    if (lane == 31) {
+      s_scan[0][warp] = a;
+      s_scan[1][warp] = b;
+    }
+    __syncthreads();
+    if (threadIdx.x == 0) {
+      int x = 0, y = 0;
+      for (int w = 0; w < warps; ++w) {
+        const int u = s_scan[0][w], v = s_scan[1][w];
+        s_scan[0][w] = x;
+        s_scan[1][w] = y;
+        x += u;
+        y += v;
+      }
+      s_scan[0][32] = x;
+      s_scan[1][32] = y;
+    }
+    __syncthreads();
+    if (e < E) {
+      s_count[e] = n;
+      s_cursor[e] = rows_before + s_scan[0][warp] + a - n;
+      s_tile[e] = tiles_before + s_scan[1][warp] + b - nt;
+    }
+    rows_before += s_scan[0][32];
+    tiles_before += s_scan[1][32];
+    __syncthreads();
+  }
+  if (threadIdx.x == 0) {
+    if (tiles_before > p.max_tiles) {
+      if (p.status) atomicCAS(p.status, 0, kStatusTooLarge);
+      tiles_before = p.max_tiles;
+    }
+    *p.num_tiles = tiles_before;
+  }
+  for (int e = warp; e < E; e += warps) {
+    const int n = s_count[e], r0 = s_cursor[e], t0 = s_tile[e];
+    for (int i = lane; i * p.tile_rows < n; i += 32)
+      if (t0 + i < p.max_tiles) p.tiles[t0 + i] = make_int4(e, r0 + i * p.tile_rows, min(p.tile_rows, n - i * p.tile_rows), 0);
+  }
+  for (int e = threadIdx.x; e <= E; e += blockDim.x) p.counters[e] = 0;
+  __syncthreads();
+  constexpr int kAhead = 4;  // pairs a thread reads at once
+  for (int i0 = threadIdx.x; i0 < pairs; i0 += kAhead * blockDim.x) {
+    int2 pr[kAhead];
+#pragma unroll
+    for (int j = 0; j < kAhead; ++j) {
+      const int i = i0 + j * blockDim.x;
+      if (i < pairs) pr[j] = __ldcg(&p.pairs[i]);
+    }
+#pragma unroll
+    for (int j = 0; j < kAhead; ++j) {
+      const int i = i0 + j * blockDim.x;
+      if (i >= pairs) break;
+      const int r = atomicAdd(&s_cursor[pr[j].x], 1);
+      const int tok = i / p.top;
+      const float w = __int_as_float(pr[j].y);
+      p.src[r] = tok;
+      p.factors[r] = p.weight_on_input ? make_float2(w, 1.f) : make_float2(1.f, w);
+      p.place[tok * per + (i - tok * p.top)] = r;
+    }
+  }
+}
+
+}  // namespace blitz
+
+extern "C" {
+using namespace blitz;
+
+// z [tokens][ld] fp32: router logits, the shared expert's in column `experts` (shared = 1).  Scratch: pairs (tokens * top
+// int2), counters (experts + 1 int32, zeroed once).  Results as described at the top of the file; rows = tokens * (top + shared).
+int blitz_moe_route(const float* z, int64_t ld, int tokens, int experts, int top, int shared, int weight_on_input, int renormalize,
+                    int tile_rows, int max_tiles, void* pairs, int* counters, int* src, void* factors, int* place, void* tiles,
+                    int* num_tiles, int* status, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (experts < 1 || experts > kMoeMaxExperts || top < 1 || top > experts || top > 32 || tile_rows < 1) return -1;
+  int warps = 32;
+  while (warps > 1 && warps * experts * 4 > 32768) warps >>= 1;
+  while (warps > 4 && (tokens + warps - 1) / warps < 16) warps >>= 1;  // small steps: tokens side by side on several SMs
+  MoeRouteParams p{z, ld, tokens, experts, top, shared, weight_on_input, renormalize, tile_rows, max_tiles,
+                   reinterpret_cast<int2*>(pairs), counters, src, reinterpret_cast<float2*>(factors), place,
+                   reinterpret_cast<int4*>(tiles), num_tiles, status};
+  return (int)launch_pdl(moe_route_kernel, dim3((tokens + warps - 1) / warps), dim3(warps * 32),
+                         (size_t)(3 + warps) * experts * sizeof(int), stream, p);
+}
+
+}  // extern "C"

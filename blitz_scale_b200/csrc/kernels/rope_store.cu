@@ -1,7 +1,9 @@
 // Rotary embedding of q and k with the paged KV write, general form: rotation of the first `rot_dims` dimensions of a
-// head (0 = none), interleaved (dimensions 2i, 2i + 1 are a pair) or half-split pairs, any head size, fp32 or 16-bit
-// activations, and a choice of what the value plane of the cache receives: the value columns of the projection, or
-// the keys as projected, before rotation (models without a value projection).
+// head (0 = none), interleaved (dimensions 2i, 2i + 1 are a pair) or half-split pairs (i, i + rot_dims / 2), any head size,
+// values of another size than the keys, fp32 or 16-bit activations, and a choice of what the value plane of the cache
+// receives: the value columns of the projection, or the keys as projected, before rotation (models without a value
+// projection).  Biases of the projections are added here, in fp32, before the rotation; `gain` multiplies the rotated
+// dimensions (scaled rotations).  Layers that read another layer's cache pass no keys: only q is rotated.
 //
 // (elementwise.cu's rope_kv_store is the special case of a fully rotated half-split head with a value projection.)
 //
@@ -16,14 +18,16 @@ namespace blitz {
 
 struct RopeStoreParams {
   void* q;           // [tokens][q_heads * dim], rotated in place
-  const void* k;     // [tokens][kv_heads * dim]
-  const void* v;     // [tokens][kv_heads * dim] or null: the value plane receives the keys before rotation
+  const void* k;     // [tokens][kv_heads * dim] or null: no keys and values to store
+  const void* v;     // [tokens][kv_heads * vdim] or null: the value plane receives the keys before rotation
+  const void *q_b, *k_b, *v_b;  // biases, or null
   int64_t row;       // row pitch of q, k and v
   const int32_t* pos;
   const int32_t* slot;
-  void* kv;
+  void *k_pool, *v_pool;  // row of token `off` of page n: n * page_rows + off
   const float2* freq;  // [rot_dims / 2] (high, low)
-  int q_heads, kv_heads, dim, rot_dims, interleaved, page_size, max_pages, wide;
+  float gain;
+  int q_heads, kv_heads, dim, vdim, rot_dims, interleaved, page_size, page_rows, max_pages, wide;
   int* status;
 };
 
@@ -42,48 +46,96 @@ __global__ void rope_store_kernel(const RopeStoreParams p) {
     float sn, cs;
     sincosf(a, &sn, &cs);
     const float c_err = 1.f - 0.5f * err * err;  // cos and sin of the small angle `err`, to second order
-    s_ang[i] = cs * c_err - err * sn;
-    s_ang[half + i] = sn * c_err + err * cs;
+    s_ang[i] = (cs * c_err - err * sn) * p.gain;
+    s_ang[half + i] = (sn * c_err + err * cs) * p.gain;
   }
   __syncthreads();
-  int s = p.slot[t];
+  int s = p.k ? p.slot[t] : -1;
   if (s >= p.max_pages * p.page_size) {
     if (threadIdx.x == 0 && p.status) atomicCAS(p.status, 0, kStatusBadIndex);
     s = -1;
   }
   const int page = s >= 0 ? s / p.page_size : 0, off = s >= 0 ? s % p.page_size : 0;
-  const int64_t kvrow = static_cast<int64_t>(p.kv_heads) * p.dim;
-  const int64_t plane = p.page_size * kvrow;
-  T* kdst = reinterpret_cast<T*>(p.kv) + static_cast<int64_t>(page) * 2 * plane + off * kvrow;
-  T* vdst = kdst + plane;
+  const int64_t krow = static_cast<int64_t>(p.kv_heads) * p.dim, vrow = static_cast<int64_t>(p.kv_heads) * p.vdim;
+  const int64_t at_row = static_cast<int64_t>(page) * p.page_rows + off;
+  T* kdst = reinterpret_cast<T*>(p.k_pool) + at_row * krow;
+  T* vdst = reinterpret_cast<T*>(p.v_pool) + at_row * vrow;
   T* q = reinterpret_cast<T*>(p.q) + t * p.row;
   const T* k = reinterpret_cast<const T*>(p.k) + t * p.row;
+  const T *q_b = reinterpret_cast<const T*>(p.q_b), *k_b = reinterpret_cast<const T*>(p.k_b), *v_b = reinterpret_cast<const T*>(p.v_b);
+  const int heads = p.q_heads + (s >= 0 ? p.kv_heads : 0);
   if (p.wide) {
-    // interleaved heads: eight elements (four pairs) per access; dimensions that pass unchanged ride along
-    const int vec = p.dim >> 3;
-    for (int it = threadIdx.x; it < (p.q_heads + p.kv_heads) * vec; it += blockDim.x) {
-      const int head = it / vec, d0 = (it - head * vec) * 8;
-      const bool is_q = head < p.q_heads;
-      if ((!is_q && s < 0) || (is_q && d0 >= p.rot_dims)) continue;
-      const int64_t at = static_cast<int64_t>(is_q ? head : head - p.q_heads) * p.dim + d0;
-      float x[8], y[8];
-      ldf8<T>((is_q ? q : k) + at, x);
+    auto load8 = [&](const T* src, const T* bias, int64_t at, float (&x)[8]) {
+      ldf8<T>(src + at, x);
+      if (bias) {
+        float b[8];
+        ldf8<T>(bias + at, b);
 #pragma unroll
-      for (int j = 0; j < 8; j += 2) {
-        const int i = (d0 + j) >> 1;
-        const bool rot = d0 + j < p.rot_dims;
-        const float cs = rot ? s_ang[i] : 1.f, sn = rot ? s_ang[half + i] : 0.f;
-        y[j] = x[j] * cs - x[j + 1] * sn;
-        y[j + 1] = x[j + 1] * cs + x[j] * sn;
+        for (int j = 0; j < 8; ++j) x[j] += b[j];
       }
-      stf8<T>((is_q ? q : kdst) + at, y);
-      if (!is_q && p.v == nullptr) stf8<T>(vdst + at, x);
+    };
+    if (p.interleaved) {
+      // eight elements (four pairs) per access; dimensions that pass unchanged ride along
+      const int vec = p.dim >> 3;
+      for (int it = threadIdx.x; it < heads * vec; it += blockDim.x) {
+        const int head = it / vec, d0 = (it - head * vec) * 8;
+        const bool is_q = head < p.q_heads;
+        if (is_q && d0 >= p.rot_dims && !q_b) continue;
+        const int64_t at = static_cast<int64_t>(is_q ? head : head - p.q_heads) * p.dim + d0;
+        float x[8], y[8];
+        load8(is_q ? q : k, is_q ? q_b : k_b, at, x);
+#pragma unroll
+        for (int j = 0; j < 8; j += 2) {
+          const int i = (d0 + j) >> 1;
+          const bool rot = d0 + j < p.rot_dims;
+          const float cs = rot ? s_ang[i] : 1.f, sn = rot ? s_ang[half + i] : 0.f;
+          y[j] = x[j] * cs - x[j + 1] * sn;
+          y[j + 1] = x[j + 1] * cs + x[j] * sn;
+        }
+        stf8<T>((is_q ? q : kdst) + at, y);
+        if (!is_q && p.v == nullptr) stf8<T>(vdst + at, x);
+      }
+    } else {
+      // half-split heads: eight pairs per item, or eight dimensions that pass unchanged
+      const int turns = half >> 3, vec = turns + ((p.dim - p.rot_dims) >> 3);
+      for (int it = threadIdx.x; it < heads * vec; it += blockDim.x) {
+        const int head = it / vec, c = it - head * vec;
+        const bool is_q = head < p.q_heads;
+        if (is_q && c >= turns && !q_b) continue;
+        const int64_t base = static_cast<int64_t>(is_q ? head : head - p.q_heads) * p.dim;
+        const T *src = is_q ? q : k, *bias = is_q ? q_b : k_b;
+        T* dst = is_q ? q : kdst;
+        float u[8];
+        if (c >= turns) {
+          const int64_t at = base + p.rot_dims + (c - turns) * 8;
+          load8(src, bias, at, u);
+          stf8<T>(dst + at, u);
+          if (!is_q && p.v == nullptr) stf8<T>(vdst + at, u);
+          continue;
+        }
+        const int i0 = c * 8;
+        float v[8], ru[8], rv[8];
+        load8(src, bias, base + i0, u);
+        load8(src, bias, base + half + i0, v);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          const float cs = s_ang[i0 + j], sn = s_ang[half + i0 + j];
+          ru[j] = u[j] * cs - v[j] * sn;
+          rv[j] = v[j] * cs + u[j] * sn;
+        }
+        stf8<T>(dst + base + i0, ru);
+        stf8<T>(dst + base + half + i0, rv);
+        if (!is_q && p.v == nullptr) {
+          stf8<T>(vdst + base + i0, u);
+          stf8<T>(vdst + base + half + i0, v);
+        }
+      }
     }
     if (p.v != nullptr && s >= 0) {
       const T* v = reinterpret_cast<const T*>(p.v) + t * p.row;
-      for (int i = threadIdx.x * 8; i < kvrow; i += blockDim.x * 8) {
+      for (int i = threadIdx.x * 8; i < vrow; i += blockDim.x * 8) {
         float x[8];
-        ldf8<T>(v + i, x);
+        load8(v, v_b, i, x);
         stf8<T>(vdst + i, x);
       }
     }
@@ -91,15 +143,14 @@ __global__ void rope_store_kernel(const RopeStoreParams p) {
   }
   // Rotated pairs of q and k.  With two-element accesses only where pairs are neighbours and rows even.
   const bool vec = p.interleaved && ((p.dim | p.row) & 1) == 0;
-  const int items = (p.q_heads + p.kv_heads) * half;
-  for (int it = threadIdx.x; it < items; it += blockDim.x) {
+  for (int it = threadIdx.x; it < heads * half; it += blockDim.x) {
     const int head = it / half, i = it - head * half;
     const float cs = s_ang[i], sn = s_ang[half + i];
     const int iu = p.interleaved ? 2 * i : i, iv = p.interleaved ? 2 * i + 1 : i + half;
     const bool is_q = head < p.q_heads;
     const int64_t base = static_cast<int64_t>(is_q ? head : head - p.q_heads) * p.dim;
-    if (!is_q && s < 0) continue;
     const T* src = (is_q ? q : k) + base;
+    const T* bias = is_q ? q_b : k_b;
     T* dst = (is_q ? q : kdst) + base;
     float u, v;
     if (vec) {
@@ -107,6 +158,10 @@ __global__ void rope_store_kernel(const RopeStoreParams p) {
       u = f.x; v = f.y;
     } else {
       u = ldf<T>(src + iu); v = ldf<T>(src + iv);
+    }
+    if (bias) {
+      u += ldf<T>(bias + base + iu);
+      v += ldf<T>(bias + base + iv);
     }
     const float ru = u * cs - v * sn, rv = v * cs + u * sn;
     if (vec) {
@@ -124,17 +179,20 @@ __global__ void rope_store_kernel(const RopeStoreParams p) {
       }
     }
   }
-  if (s < 0) return;
-  const int rest = p.dim - p.rot_dims;  // dimensions that pass unchanged: keys, and values taken from them
-  for (int it = threadIdx.x; it < p.kv_heads * rest; it += blockDim.x) {
-    const int64_t at = static_cast<int64_t>(it / rest) * p.dim + p.rot_dims + it % rest;
-    const T x = k[at];
-    kdst[at] = x;
-    if (p.v == nullptr) vdst[at] = x;
+  const int rest = p.dim - p.rot_dims;  // dimensions that pass unchanged: keys, values taken from them, queries with a bias
+  for (int it = threadIdx.x; it < heads * rest; it += blockDim.x) {
+    const int head = it / rest;
+    const bool is_q = head < p.q_heads;
+    if (is_q && !q_b) continue;
+    const int64_t at = static_cast<int64_t>(is_q ? head : head - p.q_heads) * p.dim + p.rot_dims + it % rest;
+    const T* bias = is_q ? q_b : k_b;
+    const float x = ldf<T>((is_q ? q : k) + at) + (bias ? ldf<T>(bias + at) : 0.f);
+    stf<T>((is_q ? q : kdst) + at, x);
+    if (!is_q && p.v == nullptr) stf<T>(vdst + at, x);
   }
-  if (p.v != nullptr) {
+  if (p.v != nullptr && s >= 0) {
     const T* v = reinterpret_cast<const T*>(p.v) + t * p.row;
-    for (int i = threadIdx.x; i < kvrow; i += blockDim.x) vdst[i] = v[i];
+    for (int i = threadIdx.x; i < vrow; i += blockDim.x) stf<T>(vdst + i, ldf<T>(v + i) + (v_b ? ldf<T>(v_b + i) : 0.f));
   }
 }
 
@@ -143,16 +201,21 @@ __global__ void rope_store_kernel(const RopeStoreParams p) {
 extern "C" {
 using namespace blitz;
 
-int blitz_rope_store(void* q, const void* k, const void* v, int64_t row, const int32_t* pos, const int32_t* slot,
-                     void* kv_layer, const void* freq, int num_tokens, int q_heads, int kv_heads, int dim, int rot_dims,
-                     int interleaved, int page_size, int max_pages, int* status, int dtype, cudaStream_t stream) {
+// Pools: [max_pages][page_rows][heads][size]; a page's `page_size` token rows are its first ones (with one tensor for keys
+// and values page_rows is 2 page_size and v_pool points at the first value plane).
+int blitz_rope_store(void* q, const void* k, const void* v, const void* q_b, const void* k_b, const void* v_b, int64_t row,
+                     const int32_t* pos, const int32_t* slot, void* k_pool, void* v_pool, const void* freq, float gain,
+                     int num_tokens, int q_heads, int kv_heads, int dim, int vdim, int rot_dims, int interleaved, int page_size,
+                     int page_rows, int max_pages, int* status, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (rot_dims < 0 || (rot_dims & 1) || rot_dims > dim || rot_dims > 4096 || (rot_dims > 0 && freq == nullptr)) return -1;
-  RopeStoreParams p{q, k, v, row, pos, slot, kv_layer, reinterpret_cast<const float2*>(freq), q_heads, kv_heads, dim,
-                    rot_dims, interleaved, page_size, max_pages, 0, status};
+  if (k != nullptr && v == nullptr && vdim != dim) return -1;
+  RopeStoreParams p{q, k, v, q_b, k_b, v_b, row, pos, slot, k_pool, v_pool, reinterpret_cast<const float2*>(freq), gain, q_heads,
+                    kv_heads, dim, vdim, rot_dims, interleaved, page_size, page_rows, max_pages, 0, status};
   const uintptr_t al = dtype == 2 ? 32 : 16;
-  p.wide = interleaved && ((dim | row) & 7) == 0;
-  for (const void* x : {(const void*)q, k, v, (const void*)kv_layer}) p.wide = p.wide && (reinterpret_cast<uintptr_t>(x) % al) == 0;
+  p.wide = ((dim | vdim | row) & 7) == 0 && (interleaved || (rot_dims & 15) == 0);
+  for (const void* x : {(const void*)q, k, v, q_b, k_b, v_b, (const void*)k_pool, (const void*)v_pool})
+    p.wide = p.wide && (reinterpret_cast<uintptr_t>(x) % al) == 0;
   cudaError_t e = cudaSuccess;
   BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(rope_store_kernel<T>, dim3(num_tokens), dim3(p.wide && (q_heads + kv_heads) * dim <= 2048 ? 128 : 256),
                                                (size_t)rot_dims * sizeof(float), stream, p)));

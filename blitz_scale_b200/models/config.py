@@ -85,6 +85,7 @@ REGISTRY: Dict[str, ModelConfig] = {c.name: c for c in [
 
 def hybrid_registry():
     """Shapes of the models whose layers differ (a separate table: the native twin of the registry holds the uniform ones)."""
+    from . import komulorn
     from .fafudra import shape_config
     mixed = ("gla", "attention", "rglru", "gla")
     return {c.name: c for c in [
@@ -96,23 +97,38 @@ def hybrid_registry():
         # layer sizes of the 8 B Llama shape
         shape_config("fafudra_8b", 128256, 4096, mixed * 8, 14336, heads=32, kv_heads=8, dim=128, window=2048,
                      gla_heads=16, gla_dim=128, gla_vdim=256, width=4096, blocks=16, gb=16),
+        # attention with shared key/value caches and experts: a test shape for the tensor-core kernels, one whose sizes none
+        # of them takes, and one of 13 B parameters, a mixture of experts
+        komulorn.shape_config("komulorn_tiny", 2048, 320, 4, heads=4, kv_heads=2, dim=64, vdim=32, rot_dims=32, experts=8, top=2,
+                              ff=128, shared_ff=192),
+        komulorn.shape_config("komulorn_odd", 1003, 122, 3, heads=9, kv_heads=3, dim=22, vdim=13, rot_dims=10, experts=5, top=3,
+                              ff=51, shared_ff=30, share=3),
+        komulorn.shape_config("komulorn_13b", 128256, 2048, 32, heads=32, kv_heads=4, dim=128, vdim=128, rot_dims=64, experts=64,
+                              top=6, ff=1408, shared_ff=2816, gb=27),
     ]}
+
+
+# designs described by data: "architecture" of config.json -> module of this package with parse_config and to_segment
+DESIGNS = {"Fafudra": "fafudra", "Komulorn": "komulorn"}
+
+
+def design_module(name: str):
+    import importlib
+    return importlib.import_module("." + name, __package__)
 
 
 def config_from_dir(path):
     """Configuration of a checkpoint folder whose config.json names an architecture this package describes by data."""
     import json
     from pathlib import Path
-    from . import fafudra
     from .convert import list_checkpoint
     d = Path(path)
     c = json.loads((d / "config.json").read_text())
-    parsers = {fafudra.ARCHITECTURE: fafudra.parse_config}
     arch = c.get("architecture")
-    if arch not in parsers:
-        raise KeyError(f"{d / 'config.json'}: unknown architecture {arch!r}; known: {sorted(parsers)}")
+    if arch not in DESIGNS:
+        raise KeyError(f"{d / 'config.json'}: unknown architecture {arch!r}; known: {sorted(DESIGNS)}")
     shapes = {n: shape for n, _, shape in list_checkpoint(d)}
-    return parsers[arch](c, shapes, name=d.resolve().name)
+    return design_module(DESIGNS[arch]).parse_config(c, shapes, name=d.resolve().name)
 
 
 def get_config(name: str):

@@ -25,7 +25,7 @@ from typing import Dict, Iterable, List, Optional, Tuple
 import torch
 
 from ..runtime import core
-from .config import ModelConfig, get_config
+from .config import ModelConfig, design_module, get_config
 from .weights import WeightSegment, shard_from_full
 
 _DT = {"BF16": torch.bfloat16, "F16": torch.float16, "F32": torch.float32, "F64": torch.float64, "I64": torch.int64,
@@ -134,8 +134,7 @@ def segment_to_hf(seg: WeightSegment) -> Dict[str, torch.Tensor]:
 def checkpoint_to_segment(reader: CheckpointReader, cfg, dtype=torch.bfloat16) -> WeightSegment:
     """Full (tp=1) segment on the host, by the naming scheme of the configuration's design."""
     if cfg.family == "hybrid":
-        from .fafudra import to_segment
-        return to_segment(reader, cfg, dtype)
+        return design_module(cfg.design).to_segment(reader, cfg, dtype)
     return hf_to_segment(reader, cfg, dtype)
 
 

@@ -1,12 +1,20 @@
 """Forward pass of hybrid models (hybrid_config.py) over the weight segment, the paged KV pools and the state slots.
 
-Every layer run is: one norm (with whatever is added to the stream before it), one product for all projections of the
+A layer run with its feed-forward beside the mixer is: one norm (with whatever is added to the stream before it), one product for all projections of the
 mixer, the mixer's own kernels, one product for gate and up with SiLU * mul in its epilogue, and one product that adds
 ``m * (mixer + feed-forward)`` to the fp32 stream in its epilogue::
 
     stream_norm -> GEMM (in) -> mixer -> GEMM (gate||up, SiLU*mul) -> GEMM (out, fp32 axpy)
 
-    attention: rope_store (rotation, paged write) -> attention over the pages
+A layer run with experts behind the mixer::
+
+    stream_norm -> GEMM (in) -> mixer -> GEMM (out, fp32 axpy)
+    -> stream_norm -> GEMM (router, fp32) -> moe_route -> grouped GEMM (up, act) -> grouped GEMM (down)
+
+The experts' output rows stay where the last product leaves them: the next layer's norm kernel adds them to the stream
+(`flush` does where a pass ends).
+
+    attention: rope_store (biases, rotation, paged write) -> attention over the pages (window, cap, sink, gate per head)
     gla:       one kernel (decay projection, recurrence, output norm, gate), or the chunked kernels for prompts
     rglru:     conv_causal -> block-diagonal GEMM (gates, fp32 out) -> rglru_scan
 
@@ -21,7 +29,7 @@ import torch
 
 from .. import ops
 from ..runtime.hybrid_cache import HybridCache
-from .hybrid_config import AttentionMixer, GLAMixer, HybridConfig, LayerSpec, RGLRUMixer
+from .hybrid_config import AttentionMixer, ExpertsSpec, GLAMixer, HybridConfig, LayerSpec, RGLRUMixer
 from .llama import StepMeta
 from .weights import WeightSegment
 
@@ -50,14 +58,16 @@ class HybridRunner:
         self._gates = torch.empty(max_tokens * 2 * rw, dtype=torch.float32, device=dev) if rw else None
         ck = max((m.heads * m.dim for m in cfg.run_mixers() if m.kind == "gla"), default=0)
         self._cum = torch.empty(max_tokens * ck, dtype=torch.float32, device=dev) if ck and dt == torch.bfloat16 else None
+        self._init_experts(max_tokens, dev, dt)
         self.last = torch.empty(max_batch, H, dtype=torch.float32, device=dev)
         self._logits_pad = torch.zeros(max_batch, cfg.vocab_pad, dtype=torch.float32, device=dev)
         self.logits = self._logits_pad[:, :cfg.vocab]
         self.tokens = torch.empty(max_batch, dtype=torch.int32, device=dev)
         self._freqs = {}
         for m in cfg.run_mixers():
-            if m.kind == "attention" and (m.rot_dims, m.rot_base) not in self._freqs:
-                self._freqs[(m.rot_dims, m.rot_base)] = ops.rope_freqs(m.rot_dims, m.rot_base, dev)
+            if m.kind == "attention" and self._rot_key(m) not in self._freqs:
+                stretch = m.yarn.stretch(m.rot_dims, m.rot_base) if m.yarn else None
+                self._freqs[self._rot_key(m)] = ops.rope_freqs(m.rot_dims, m.rot_base, dev, stretch)
         self._ws: Optional[torch.Tensor] = None
         self._ws_old: List[Optional[torch.Tensor]] = []
 
@@ -65,8 +75,33 @@ class HybridRunner:
     def _mid_key(s: LayerSpec) -> tuple:
         return (s.mixer.out_width, s.ff)
 
+    @staticmethod
+    def _rot_key(m: AttentionMixer) -> tuple:
+        return (m.rot_dims, m.rot_base, m.yarn)
+
     def _w(self, l: int, name: str) -> torch.Tensor:
         return self.seg[f"layers.{l}.{name}"]
+
+    def _init_experts(self, max_tokens: int, dev, dt) -> None:
+        """Buffers of the layers with experts: router logits, work lists (one per shape of router), activations of the sorted
+        rows, and output rows."""
+        moes = [s.moe for s in self.cfg.layer_specs if s.moe]
+        self._pending: Optional[tuple] = None        # output rows of experts that are not in the stream yet, and where they go
+        self._plans: Dict[tuple, ops.ExpertPlan] = {}
+        if not moes:
+            return
+        for e in moes:
+            key = self._plan_key(e)
+            if key not in self._plans:
+                self._plans[key] = ops.ExpertPlan(max_tokens, e.experts, e.top, bool(e.shared_ff), dev)
+        rows = max_tokens * max(e.per_token for e in moes)
+        self._router = torch.empty(max_tokens * max(e.router_cols for e in moes), dtype=torch.float32, device=dev)
+        self._act = torch.empty(rows * max(max(e.ff_pad, e.shared_pad) for e in moes), dtype=dt, device=dev)
+        self._expert_out = torch.empty(rows, self.cfg.hidden, dtype=dt, device=dev)
+
+    @staticmethod
+    def _plan_key(e: ExpertsSpec) -> tuple:
+        return (e.experts, e.top, bool(e.shared_ff))
 
     # ------------------------------------------------------------------ pieces
     def embed(self, m: StepMeta) -> None:
@@ -80,8 +115,11 @@ class HybridRunner:
         step = self.seg["loop_step"][run.step] if run.step >= 0 else None
         h = self.normed[:T]
         needs_ids = r == 0 or run.add_embed
-        ops.stream_norm(self.res[:T], self._w(l, "norm1"), c.rms_eps, h, w_offset=1.0, ids=m.ids if needs_ids else None,
-                        embed=self.seg["embed"] if needs_ids else None, init=r == 0, add_embed=run.add_embed, step=step)
+        if r == 0:
+            self._pending = None
+        ops.stream_norm(self.res[:T], self._w(l, "norm1"), c.rms_eps, h, w_offset=c.norm_offset, ids=m.ids if needs_ids else None,
+                        embed=self.seg["embed"] if needs_ids else None, init=r == 0, add_embed=run.add_embed, step=step,
+                        **self._take_pending())
         cols, width = spec.in_columns()
         proj = self._proj[:T * width].view(T, width)
         ops.gemm(h, self._w(l, "in"), out=proj, static_b=True)
@@ -91,30 +129,59 @@ class HybridRunner:
         if spec.ff:
             ops.gemm(h, self._w(l, "gate_up"), out=mid[:, spec.mix_rows:], epilogue="silu_mul", static_b=True)
         ops.gemm(mid, self._w(l, "out"), out=self.res[:T], epilogue="axpy", alpha=c.residual_mult, static_b=True)
+        if spec.moe:
+            ops.stream_norm(self.res[:T], self._w(l, "norm2"), c.rms_eps, h, w_offset=c.norm_offset)
+            self._experts(l, spec.moe, h)
+
+    def _take_pending(self) -> dict:
+        p, self._pending = self._pending, None
+        return dict(add=p[0], add_rows=p[1]) if p else {}
+
+    def flush(self, T: int) -> None:
+        """Everything the layers so far have produced is in the stream."""
+        if self._pending:
+            ops.stream_norm(self.res[:T], None, 0.0, None, **self._take_pending())
+
+    def _experts(self, l: int, e: ExpertsSpec, h: torch.Tensor) -> None:
+        T, H = h.shape
+        plan = self._plans[self._plan_key(e)]
+        z = self._router[:T * e.router_cols].view(T, e.router_cols)
+        ops.gemm(h, self._w(l, "router"), out=z, static_b=True)
+        up, down = self._w(l, "up").view(e.experts, H, e.ff_pad), self._w(l, "down").view(e.experts, e.ff_pad, H)
+        s_up, s_down = (self._w(l, "shared_up"), self._w(l, "shared_down")) if e.shared_ff else (None, None)
+        tc = ops.grouped_tensor_core(h, up, down, s_up, s_down)
+        ops.moe_route(z, plan, weight_on_input=e.weight_on_input, renormalize=e.renormalize, tile_rows=128 if tc else 64)
+        width = max(e.ff_pad, e.shared_pad)
+        act, out = self._act[:plan.rows * width].view(plan.rows, width), self._expert_out[:plan.rows]
+        ops.gemm_grouped(h, up, plan, act, shared=s_up, gather=True, act="relu2", factors=True)
+        ops.gemm_grouped(act, down, plan, out, shared=s_down)
+        self._pending = (out, plan.place)
 
     def _attention(self, r: int, l: int, mx: AttentionMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta) -> None:
         T, kv = m.num_tokens, self.cache.runs[r].kv
-        ops.rope_store(p["q"], p["k"], p.get("v"), m.pos, m.slot, kv, self._freqs[(mx.rot_dims, mx.rot_base)],
-                       q_heads=mx.heads, kv_heads=mx.kv_heads, dim=mx.dim, rot_dims=mx.rot_dims, page_size=self.page_size,
-                       interleaved=mx.interleaved)
-        extra = dict(window=mx.window, keep_first=mx.keep_first, softcap=mx.softcap,
-                     sink=self._w(l, "sink") if mx.sink else None)
-        if not ops.attn_tensor_core(p["q"], mx.heads, mx.kv_heads, mx.dim, self.page_size):
+        biases = {n: self._w(l, n) for n, _ in mx.tensors() if n != "sink"}
+        ops.rope_store(p["q"], p.get("k"), p.get("v"), m.pos, m.slot, kv, self._freqs[self._rot_key(mx)], q_heads=mx.heads,
+                       kv_heads=mx.kv_heads, dim=mx.dim, rot_dims=mx.rot_dims, page_size=self.page_size,
+                       interleaved=mx.interleaved, gain=mx.yarn.gain if mx.yarn else 1.0, **biases)
+        extra = dict(window=mx.window, keep_first=mx.keep_first, softcap=mx.softcap, sink=self._w(l, "sink") if mx.sink else None)
+        gate = p.get("g")
+        if not ops.attn_tensor_core(p["q"], mx.heads, mx.kv_heads, mx.dim, self.page_size, mx.vdim):
             ops.attn_ragged(p["q"], kv, m.pos, m.tok_indptr if m.is_prefill else None, m.page_indptr, m.page_indices, mid,
-                            q_heads=mx.heads, kv_heads=mx.kv_heads, dim=mx.dim, page_size=self.page_size, scale=mx.scale, **extra)
+                            q_heads=mx.heads, kv_heads=mx.kv_heads, dim=mx.dim, page_size=self.page_size, scale=mx.scale, gate=gate, **extra)
             return
         args = dict(q_heads=mx.heads, kv_heads=mx.kv_heads, head_dim=mx.dim, page_size=self.page_size, sm_scale=mx.scale, **extra)
         ns = m.singles if m.is_prefill else m.batch
         if ns:
             ops.attn_decode(p["q"][:ns], kv, m.page_indices, m.page_indptr[:ns + 1], m.last_page_len[:ns],
-                            num_splits=m.num_splits, workspace=self._workspace(ns, mx, m.num_splits), out=mid[:ns], **args)
+                            num_splits=m.num_splits, workspace=self._workspace(ns, mx, m.num_splits), out=mid[:ns],
+                            gate=gate[:ns] if gate is not None else None, **args)
         if m.batch > ns:
-            ops.attn_prefill_paged(p["q"], kv, m.page_indices, m.prefill_work, out=mid, **args)
+            ops.attn_prefill_paged(p["q"], kv, m.page_indices, m.prefill_work, out=mid, gate=gate, **args)
 
     def _workspace(self, B: int, mx: AttentionMixer, splits: int) -> Optional[torch.Tensor]:
         if splits <= 1:
             return None
-        n = ops.attn_decode_workspace_bytes(B, mx.heads, mx.dim, splits)
+        n = ops.attn_decode_workspace_bytes(B, mx.heads, mx.vdim, splits)
         if self._ws is None or self._ws.numel() < n:
             # an earlier buffer may be named by captured graphs: keep it
             self._ws_old.append(self._ws)
@@ -146,9 +213,12 @@ class HybridRunner:
     # ------------------------------------------------------------------ head
     def logits_of(self, n: int, rows: Optional[torch.Tensor] = None, row_offset: int = 0) -> torch.Tensor:
         """fp32 logits of `n` rows of the stream: rows 0 .. n - 1, or `rows` (+ row_offset)."""
-        ops.stream_norm(self.res, self.seg["final_norm"], self.cfg.rms_eps, self.normed[:n], w_offset=1.0, rows=rows,
-                        row_offset=row_offset, num_tokens=n)
-        ops.gemm(self.normed[:n], self.seg["lm_head"], out=self._logits_pad[:n], static_b=True)
+        c = self.cfg
+        add = {} if rows is not None else self._take_pending()
+        ops.stream_norm(self.res, self.seg["final_norm"], c.rms_eps, self.normed[:n], w_offset=c.norm_offset, rows=rows,
+                        row_offset=row_offset, num_tokens=n, **add)
+        cap = dict(epilogue="softcap", alpha=c.logit_softcap) if c.logit_softcap else {}
+        ops.gemm(self.normed[:n], self.seg["lm_head"], out=self._logits_pad[:n], static_b=True, **cap)
         return self.logits[:n]
 
     def head(self, m: StepMeta) -> torch.Tensor:
@@ -178,10 +248,13 @@ class HybridRunner:
             self.run_layer(r, m)
             if after_layer is not None:
                 after_layer(r)
+        if m.is_prefill or not with_head:
+            self.flush(m.num_tokens)             # (in a decode step the final norm adds them)
         return self.head(m) if with_head else None
 
     def decode_launches(self) -> int:
         """Kernels of this library in one decode step."""
         per = {"attention": 2, "gla": 1, "rglru": 3}
-        n = sum(3 + per[self.cfg.layer_specs[r.layer].mixer.kind] + bool(self.cfg.layer_specs[r.layer].ff) for r in self.runs)
+        specs = [self.cfg.layer_specs[r.layer] for r in self.runs]
+        n = sum(3 + per[s.mixer.kind] + bool(s.ff) + 5 * bool(s.moe) for s in specs)
         return n + 3      # final norm, head product, arg-max

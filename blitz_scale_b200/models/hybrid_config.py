@@ -1,25 +1,30 @@
-"""Shapes and constants of models whose layers differ: a list of layers, each with a mixer (attention, gated linear
-attention, gated linear recurrence) and an optional gated feed-forward that read the same normalised input, over an
-fp32 residual stream, with an optional block of layers that runs several times.
+"""Shapes and constants of models whose layers differ: a list of layers over an fp32 residual stream, each with a mixer
+(attention, gated linear attention, gated linear recurrence) and an optional feed-forward, with an optional block of
+layers that runs several times.  The feed-forward is either a gated one beside the mixer (both read one norm) or a
+mixture of experts behind it (with a norm of its own).
 
-Everything a kernel needs is a field here, so a design is described by data: `models/fafudra.py` fills these records
-from a checkpoint's config.json, the registry at the end from shapes.  `ModelConfig` (config.py) stays the record of
+Everything a kernel needs is a field here, so a design is described by data: `models/fafudra.py` and
+`models/komulorn.py` fill these records from a checkpoint's config.json, the registry from shapes.  `ModelConfig` (config.py) stays the record of
 the uniform Llama-type models; both offer what the engine, the worker and the router read (name, vocab, hidden,
 layers, eos_token, param_gb, kv_bytes_per_token).
 
 Weight segment of such a model (one allocation, matrices ``[in, out]``, every tensor on a 256-byte boundary)::
 
     embed [vocab, hidden] | loop_step [times, hidden]
-    L x { norm1 | in [hidden, projections] | mixer tensors | out [mixer out + ff, hidden] | gate_up [hidden, 2 ff] }
+    L x { norm1 | in [hidden, projections] | mixer tensors | out [mixer out + ff, hidden] | gate_up [hidden, 2 ff]
+          | norm2 | router [hidden, experts + 1] | up [experts x hidden, ff] | down [experts x ff, hidden]
+          | shared_up [hidden, shared ff] | shared_down [shared ff, hidden] }
     final_norm [hidden] | lm_head [hidden, vocab]
 
 A layer has two wide projections per side: ``in`` holds every projection of the mixer next to each other and ``out``
 the mixer's and the feed-forward's output projections on top of each other, so that the sum of both sublayers is one
-matrix product.  The column ranges of ``in`` and the row ranges of ``out`` start on multiples of 8 elements (16 bytes
+matrix product.  Experts are stacked along their input dimension, as the blocks of a block-diagonal product are; the
+column behind the router's is the gate of the shared expert.  The column ranges of ``in`` and the row ranges of ``out`` start on multiples of 8 elements (16 bytes
 in 16-bit types, what TMA and vector loads need); the padding is zero.
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 from typing import Dict, List, Optional, Tuple, Union
 
@@ -42,6 +47,28 @@ def _columns(widths: List[Tuple[str, int]]) -> Tuple[Dict[str, Tuple[int, int]],
 
 
 @dataclass(frozen=True)
+class YarnScaling:
+    """Rotary frequencies stretched for long contexts: pair i's frequency goes from f_i (pairs that turn more than `fast`
+    times over the `original` context) to f_i / factor (fewer than `slow` times) along a linear ramp, and the rotated
+    vectors grow by a constant."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+    @property
+    def gain(self) -> float:
+        return 0.1 * math.log(self.factor) + 1.0
+
+    def stretch(self, dims: int, base: float) -> List[float]:
+        """What every pair's frequency is multiplied with."""
+        pair_of = lambda turns: dims * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+        lo, hi = max(math.floor(pair_of(self.fast)), 0), min(math.ceil(pair_of(self.slow)), dims - 1)
+        ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(dims // 2)]
+        return [r / self.factor + (1.0 - r) for r in ramp]
+
+
+@dataclass(frozen=True)
 class AttentionMixer:
     heads: int
     kv_heads: int
@@ -55,22 +82,40 @@ class AttentionMixer:
     softcap: float = 0.0          # 0: none
     sink: bool = False            # learned number per head in the softmax denominator
     value_is_key: bool = False    # no value projection: values are the keys before rotation
+    value_dim: int = 0            # size of a value head; 0: as `dim`
+    bias: bool = False            # biases on the q, k and v projections
+    gate: bool = False            # a head's output is multiplied by the sigmoid of a projection, one number per head
+    yarn: Optional[YarnScaling] = None
+    kv_from: Optional[int] = None  # layer whose cached keys and values are used; no k and v projections then
     kind = "attention"
 
     def __post_init__(self):
         if self.heads % self.kv_heads or self.rot_dims % 2 or self.rot_dims > self.dim:
             raise ValueError("attention mixer: heads must be a multiple of kv_heads, rotated dimensions even and within a head")
+        if self.value_is_key and self.vdim != self.dim:
+            raise ValueError("attention mixer: values that are keys have the keys' size")
+
+    @property
+    def vdim(self) -> int:
+        return self.value_dim or self.dim
 
     @property
     def out_width(self) -> int:
-        return self.heads * self.dim
+        return self.heads * self.vdim
+
+    def _qkv(self) -> List[Tuple[str, int]]:
+        out = [("q", self.heads * self.dim)]
+        if self.kv_from is None:
+            out.append(("k", self.kv_heads * self.dim))
+            if not self.value_is_key:
+                out.append(("v", self.kv_heads * self.vdim))
+        return out
 
     def projections(self) -> List[Tuple[str, int]]:
-        kv = [("k", self.kv_heads * self.dim)] + ([] if self.value_is_key else [("v", self.kv_heads * self.dim)])
-        return [("q", self.heads * self.dim)] + kv
+        return self._qkv() + ([("g", self.heads)] if self.gate else [])
 
     def tensors(self) -> List[Tuple[str, Tuple[int, ...]]]:
-        return [("sink", (self.heads,))] if self.sink else []
+        return ([("sink", (self.heads,))] if self.sink else []) + ([(n + "_b", (w,)) for n, w in self._qkv()] if self.bias else [])
 
 
 @dataclass(frozen=True)
@@ -131,9 +176,49 @@ Mixer = Union[AttentionMixer, GLAMixer, RGLRUMixer]
 
 
 @dataclass(frozen=True)
+class ExpertsSpec:
+    """Mixture of experts without biases: W_down act(W_up h), act = the square of relu.  A token goes to the `top` experts
+    with the largest router scores (sigmoid of the logits, optionally divided by the sum of the chosen ones); the score
+    multiplies the expert's input or its output.  A shared expert runs for every token and is added, multiplied by the
+    sigmoid of a projection."""
+    experts: int
+    top: int
+    ff: int
+    shared_ff: int = 0            # 0: no shared expert
+    weight_on_input: bool = True
+    renormalize: bool = False
+
+    def __post_init__(self):
+        if not 1 <= self.top <= self.experts or self.ff < 1:
+            raise ValueError(f"{self.top} of {self.experts} experts of width {self.ff}")
+
+    @property
+    def ff_pad(self) -> int:
+        return pad8(self.ff)
+
+    @property
+    def shared_pad(self) -> int:
+        return pad8(self.shared_ff)
+
+    @property
+    def per_token(self) -> int:
+        """Expert rows of a token, the shared expert's included."""
+        return self.top + bool(self.shared_ff)
+
+    @property
+    def router_cols(self) -> int:
+        return pad8(self.experts + bool(self.shared_ff))
+
+
+@dataclass(frozen=True)
 class LayerSpec:
     mixer: Mixer
     ff: int = 0                   # width of the gated feed-forward beside the mixer; 0: none
+    moe: Optional[ExpertsSpec] = None   # experts behind the mixer, with a norm of their own
+
+    def __post_init__(self):
+        if self.ff and self.moe:
+            raise ValueError("a layer has a feed-forward beside its mixer or experts behind it, not both")
 
     def in_columns(self) -> Tuple[Dict[str, Tuple[int, int]], int]:
         return _columns(self.mixer.projections())
@@ -179,9 +264,23 @@ class HybridConfig:
     param_gb: float = 0.0
     eos_token: int = -1
     max_positions: int = 1 << 20
+    norm_offset: float = 1.0      # added to the stored norm weights (1: they are stored around zero)
+    logit_softcap: float = 0.0    # logits become cap * tanh(logits / cap); 0: none
+    tied: bool = True             # the head is the embedding table
+    design: str = "fafudra"       # module of this package that maps checkpoint names (weights of a folder)
     family = "hybrid"
 
     def __post_init__(self):
+        for i, s in enumerate(self.layer_specs):
+            j = getattr(s.mixer, "kv_from", None)
+            if j is None:
+                continue
+            src = self.layer_specs[j].mixer if 0 <= j < i else None
+            if src is None or src.kind != "attention" or src.kv_from is not None:
+                raise ValueError(f"{self.name}: layer {i} takes keys and values from layer {j}, which has none of its own before it")
+            same = ("kv_heads", "dim", "vdim")
+            if any(getattr(src, n) != getattr(s.mixer, n) for n in same):
+                raise ValueError(f"{self.name}: layers {j} and {i} share keys and values but differ in {', '.join(same)}")
         lp = self.loop
         if lp is not None and not (0 <= lp.start < lp.stop <= len(self.layer_specs) and lp.times >= 1):
             raise ValueError(f"{self.name}: loop of layers {lp.start}..{lp.stop} x {lp.times} does not fit "
@@ -205,8 +304,18 @@ class HybridConfig:
     def run_mixers(self) -> List[Mixer]:
         return [self.layer_specs[r.layer].mixer for r in self.runs()]
 
+    def kv_runs(self) -> List[int]:
+        """For every layer run the run whose keys and values it reads (its own, but for layers that share another's)."""
+        latest: Dict[int, int] = {}
+        out = []
+        for r, run in enumerate(self.runs()):
+            latest[run.layer] = r
+            j = getattr(self.layer_specs[run.layer].mixer, "kv_from", None)
+            out.append(r if j is None else latest[j])
+        return out
+
     def kv_bytes_per_token(self, tp: int = 1, elem: int = 2) -> int:
-        return sum(2 * m.kv_heads * m.dim * elem for m in self.run_mixers() if m.kind == "attention")
+        return sum(m.kv_heads * (m.dim + m.vdim) * elem for m in self.run_mixers() if m.kind == "attention" and m.kv_from is None)
 
     def state_bytes_per_sequence(self, elem: int = 2) -> int:
         n = 0
@@ -237,16 +346,22 @@ class HybridConfig:
     def init_(self, name: str, v: torch.Tensor, rand) -> None:
         """Random weights with activations of order one; `rand(shape)` gives normal numbers on v's device."""
         leaf = name.rsplit(".", 1)[-1]
-        if leaf in ("norm1", "final_norm"):
-            x = 0.1 * rand(v.shape)                          # stored around zero
+        if leaf in ("norm1", "norm2", "final_norm"):
+            x = 1.0 - self.norm_offset + 0.1 * rand(v.shape)
         elif leaf == "o_norm":
             x = 1.0 + 0.1 * rand(v.shape)
         elif leaf == "a2_b":
             x = 2.0 + rand(v.shape)                          # slow decays with some fast channels
         elif leaf == "lam":
             x = -4.0 + rand(v.shape)                         # a between about 0.8 and 0.99
-        elif leaf in ("x_b", "y_b", "conv_b", "gate_b", "sink", "loop_step"):
+        elif leaf in ("x_b", "y_b", "conv_b", "gate_b", "sink", "loop_step", "q_b", "k_b", "v_b"):
             x = 0.2 * rand(v.shape)
+        elif leaf in ("up", "down"):                         # experts stacked along their inputs
+            moe = self.layer_specs[int(name.split(".")[1])].moe
+            n = v.shape[0] // moe.experts
+            for e in range(moe.experts):
+                v[e * n:(e + 1) * n].copy_((rand((n, v.shape[1])) * n ** -0.5).to(v.dtype))
+            return
         elif leaf == "conv":
             x = rand(v.shape) * v.shape[0] ** -0.5
         elif leaf == "embed":
@@ -273,6 +388,14 @@ class HybridConfig:
                 g = tensors[p + "gate_up"]
                 g[:, s.ff:s.ff_pad] = 0
                 g[:, s.ff_pad + s.ff:] = 0
+            if s.moe:
+                e = s.moe
+                tensors[p + "router"][:, e.experts + bool(e.shared_ff):] = 0
+                tensors[p + "up"][:, e.ff:] = 0
+                tensors[p + "down"].view(e.experts, e.ff_pad, self.hidden)[:, e.ff:] = 0
+                if e.shared_ff:
+                    tensors[p + "shared_up"][:, e.shared_ff:] = 0
+                    tensors[p + "shared_down"][e.shared_ff:] = 0
 
 
 def build_hybrid_layout(cfg: HybridConfig, tp: int = 1, elem_bytes: int = 2) -> SegmentLayout:
@@ -303,6 +426,15 @@ def build_hybrid_layout(cfg: HybridConfig, tp: int = 1, elem_bytes: int = 2) -> 
         add(p + "out", (s.out_rows, cfg.hidden))
         if s.ff:
             add(p + "gate_up", (cfg.hidden, 2 * s.ff_pad))
+        if s.moe:
+            e = s.moe
+            add(p + "norm2", (cfg.hidden,))
+            add(p + "router", (cfg.hidden, e.router_cols))
+            add(p + "up", (e.experts * cfg.hidden, e.ff_pad))
+            add(p + "down", (e.experts * e.ff_pad, cfg.hidden))
+            if e.shared_ff:
+                add(p + "shared_up", (cfg.hidden, e.shared_pad))
+                add(p + "shared_down", (e.shared_pad, cfg.hidden))
         lay.units.append((f"layer.{l}", start, cur - start))
     start = cur
     add("final_norm", (cfg.hidden,))

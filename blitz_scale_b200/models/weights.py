@@ -84,9 +84,10 @@ class WeightSegment:
 
     def _hybrid_init(self, rand) -> "WeightSegment":
         for name, v in self._views.items():
-            if name != "lm_head":
+            if name != "lm_head" or not self.cfg.tied:
                 self.cfg.init_(name, v, rand)
-        self._views["lm_head"][:, :self.cfg.vocab].copy_(self._views["embed"].t())      # tied
+        if self.cfg.tied:
+            self._views["lm_head"][:, :self.cfg.vocab].copy_(self._views["embed"].t())
         self.cfg.zero_padding_(self._views)
         return self
 

@@ -9,7 +9,7 @@ cache ``[page][K|V][token][kv_head][head_dim]`` per layer.
 from __future__ import annotations
 
 import ctypes
-from typing import Optional
+from typing import NamedTuple, Optional, Sequence, Union
 
 import torch
 
@@ -50,6 +50,30 @@ def _check(rc: int, what: str) -> None:
             " (TMA descriptor encoder unavailable)" if rc == -2 else ""))
 
 
+class KVPair(NamedTuple):
+    """Paged cache of a layer whose keys and values differ in size: [pages, page, kv_heads, dim] and [.., vdim].  (Where they
+    are equal, the cache is one tensor [pages, 2, page, kv_heads, dim].)"""
+    k: torch.Tensor
+    v: torch.Tensor
+
+
+KVLayer = Union[torch.Tensor, KVPair]
+
+
+def _kv(kv: KVLayer):
+    """(key pool, value pool, rows per page in the pools, pages, value size)"""
+    if isinstance(kv, KVPair):
+        assert kv.k.is_contiguous() and kv.v.is_contiguous() and kv.k.shape[:3] == kv.v.shape[:3]
+        return _p(kv.k), _p(kv.v), kv.k.shape[1], kv.k.shape[0], kv.v.shape[3]
+    assert kv.is_contiguous()
+    return _p(kv), ctypes.c_void_p(kv.data_ptr() + kv.stride(1) * kv.element_size()), 2 * kv.shape[2], kv.shape[0], kv.shape[4]
+
+
+def _gate(gate: Optional[torch.Tensor]):
+    assert gate is None or gate.stride(1) == 1
+    return _p(gate), 0 if gate is None else gate.stride(0)
+
+
 def status_word(device=None) -> torch.Tensor:
     """Per-device int32 word the kernels write a non-zero code into when a bounded wait or an index check fails."""
     dev = torch.device("cuda", torch.cuda.current_device()) if device is None else torch.device(device)
@@ -77,7 +101,7 @@ def check_status(device=None, reset: bool = True) -> int:
 
 
 # ---------------------------------------------------------------------------------------------- GEMM
-_EPI = {"store": 0, "add": 1, "silu_mul": 2, "axpy": 5}
+_EPI = {"store": 0, "add": 1, "silu_mul": 2, "axpy": 5, "softcap": 6}
 _EPI_STORE_F32 = 4
 
 
@@ -142,7 +166,8 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *
     any M, ``pair_bnf`` / ``pair_nacc`` / ``pair_upp`` override its tile width, tiles per pair and units per pair.
 
     ``out`` may be fp32 with 16-bit operands (the accumulator is stored unrounded); epilogue 'axpy' adds
-    ``alpha * (a @ b)`` to an fp32 ``out`` (residual streams kept in 32 bits).  ``groups`` > 1: block-diagonal product,
+    ``alpha * (a @ b)`` to an fp32 ``out`` (residual streams kept in 32 bits); 'softcap' stores
+    ``alpha * tanh((a @ b) / alpha)`` in fp32 (logits).  ``groups`` > 1: block-diagonal product,
     a [M, groups * K], b [groups * K, N] (the blocks stacked), out [M, groups * N].  fp32 operands, and 16-bit ones
     whose sizes the tensor-core kernels do not take, run on the CUDA cores in fp32 arithmetic.
     """
@@ -162,7 +187,7 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *
     if out is None:
         out = torch.empty((M, groups * N), dtype=a.dtype, device=a.device)
     assert out.shape == (M, groups * N) and out.stride(1) == 1
-    if epi == 5:
+    if epi in (5, 6):
         assert out.dtype == torch.float32
     elif out.dtype != a.dtype:
         assert epi == 0 and out.dtype == torch.float32
@@ -302,36 +327,38 @@ def rope_kv_store(qkv: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor, kv_l
 
 
 # ---------------------------------------------------------------------------------------------- attention
-def attn_decode_workspace_bytes(batch: int, q_heads: int, head_dim: int, num_splits: int) -> int:
-    return int(lib().blitz_attn_decode_workspace_bytes(batch, q_heads, head_dim, num_splits))
+def attn_decode_workspace_bytes(batch: int, q_heads: int, value_dim: int, num_splits: int) -> int:
+    return int(lib().blitz_attn_decode_workspace_bytes(batch, q_heads, value_dim, num_splits))
 
 
-def attn_decode(q: torch.Tensor, kv_layer: torch.Tensor, indices: torch.Tensor, indptr: torch.Tensor,
+def attn_decode(q: torch.Tensor, kv_layer: KVLayer, indices: torch.Tensor, indptr: torch.Tensor,
                 last_page_len: torch.Tensor, *, q_heads: int, kv_heads: int, head_dim: int, page_size: int,
                 num_splits: int = 1, workspace: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
                 sm_scale: Optional[float] = None, window: int = 0, keep_first: int = 0, softcap: float = 0.0,
-                sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """q: [batch, >= q_heads*head_dim] (row pitch free, e.g. a view of the fused qkv buffer).  ``window`` > 0: only the
     last that many positions and the first ``keep_first`` are visible (and read); ``softcap`` > 0:
-    scores are cap * tanh(score / cap); ``sink`` [q_heads]: a term e^sink in the softmax denominator."""
+    scores are cap * tanh(score / cap); ``sink`` [q_heads]: a term e^sink in the softmax denominator; ``gate``
+    [batch, q_heads]: a head's output is multiplied by its sigmoid.  Values may have a size of their own (KVPair)."""
     B = indptr.numel() - 1
+    kp, vp, page_rows, pages, vdim = _kv(kv_layer)
     if out is None:
-        out = torch.empty((B, q_heads * head_dim), dtype=q.dtype, device=q.device)
+        out = torch.empty((B, q_heads * vdim), dtype=q.dtype, device=q.device)
     if num_splits > 1 and workspace is None:
-        workspace = torch.empty(attn_decode_workspace_bytes(B, q_heads, head_dim, num_splits), dtype=torch.uint8,
+        workspace = torch.empty(attn_decode_workspace_bytes(B, q_heads, vdim, num_splits), dtype=torch.uint8,
                                 device=q.device)
     if sm_scale is None:
         sm_scale = head_dim ** -0.5
-    _check(lib().blitz_attn_decode(_p(q), q.stride(0), _p(kv_layer), _p(indices), _p(indptr), _p(last_page_len),
-                                   _p(out), out.stride(0), _p(workspace), B, q_heads, kv_heads, head_dim, page_size,
-                                   kv_layer.shape[0], num_splits, sm_scale, window, keep_first, softcap, _p(sink),
+    _check(lib().blitz_attn_decode(_p(q), q.stride(0), kp, vp, _p(indices), _p(indptr), _p(last_page_len),
+                                   _p(out), out.stride(0), _p(workspace), B, q_heads, kv_heads, head_dim, vdim, page_size,
+                                   page_rows, pages, num_splits, sm_scale, window, keep_first, softcap, _p(sink), *_gate(gate),
                                    _p(status_word(q.device)), _dt(q), _stream()), "blitz_attn_decode")
     return out
 
 
-def attn_tensor_core(q: torch.Tensor, q_heads: int, kv_heads: int, head_dim: int, page_size: int) -> bool:
-    """Whether attn_decode and attn_prefill_paged take this head shape (attn_ragged takes every one)."""
-    return (q.dtype in _DT and head_dim in (64, 128) and q_heads // kv_heads <= 8 and page_size >= 8
+def attn_tensor_core(q: torch.Tensor, q_heads: int, kv_heads: int, head_dim: int, page_size: int, value_dim: int = 0) -> bool:
+    """Whether attn_decode and attn_prefill_paged take these head sizes (attn_ragged takes every one)."""
+    return (q.dtype in _DT and all(8 <= d <= 128 and d % 8 == 0 for d in (head_dim, value_dim or head_dim)) and page_size >= 8
             and page_size & (page_size - 1) == 0 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0)
 
 
@@ -354,25 +381,26 @@ def prefill_work_list(q_lens, kv_lens, page_size: int, device, skip: int = 0) ->
     return torch.tensor(rec, dtype=torch.int32).reshape(-1, 8).to(device, non_blocking=True)
 
 
-def attn_prefill_paged(q: torch.Tensor, kv_layer: torch.Tensor, page_indices: torch.Tensor, work: torch.Tensor, *,
+def attn_prefill_paged(q: torch.Tensor, kv_layer: KVLayer, page_indices: torch.Tensor, work: torch.Tensor, *,
                        q_heads: int, kv_heads: int, head_dim: int, page_size: int, out: Optional[torch.Tensor] = None,
                        sm_scale: Optional[float] = None, poly_exp: bool = False, window: int = 0, keep_first: int = 0,
-                       softcap: float = 0.0, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                       softcap: float = 0.0, sink: Optional[torch.Tensor] = None,
+                       gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of the pass's rows over the paged cache (which already holds the rows' own keys and values,
     after whatever earlier passes stored).  ``q``: rotated query columns, e.g. the fused qkv buffer (rope_kv_store);
     ``page_indices``: the sequences' page ids back to back, covering prefix + rows; ``work`` from `prefill_work_list`
-    for the same sequences.  ``window`` / ``keep_first`` / ``softcap`` / ``sink`` as for `attn_decode`."""
+    for the same sequences.  ``window`` / ``keep_first`` / ``softcap`` / ``sink`` / ``gate`` as for `attn_decode`."""
     T = q.shape[0]
+    kp, vp, page_rows, pages, vdim = _kv(kv_layer)
     if out is None:
-        out = torch.empty((T, q_heads * head_dim), dtype=q.dtype, device=q.device)
+        out = torch.empty((T, q_heads * vdim), dtype=q.dtype, device=q.device)
     if sm_scale is None:
         sm_scale = head_dim ** -0.5
     assert work.dtype == torch.int32 and work.dim() == 2 and work.shape[1] == 8 and work.is_contiguous()
-    max_pages = kv_layer.shape[0]
-    _check(lib().blitz_attn_prefill_paged(_p(q), q.stride(0), _p(kv_layer), _p(out), out.stride(0), _p(page_indices),
-                                          _p(work), work.shape[0], T, q_heads, kv_heads, head_dim, page_size, max_pages,
-                                          sm_scale, 1 if poly_exp else 0, window, keep_first, softcap, _p(sink),
-                                          _p(status_word(q.device)), _dt(q), _stream()), "blitz_attn_prefill_paged")
+    _check(lib().blitz_attn_prefill_paged(_p(q), q.stride(0), kp, vp, _p(out), out.stride(0), _p(page_indices),
+                                          _p(work), work.shape[0], T, q_heads, kv_heads, head_dim, vdim, page_size, page_rows,
+                                          pages, sm_scale, 1 if poly_exp else 0, window, keep_first, softcap, _p(sink),
+                                          *_gate(gate), _p(status_word(q.device)), _dt(q), _stream()), "blitz_attn_prefill_paged")
     return out
 
 
@@ -380,57 +408,149 @@ def attn_prefill_paged(q: torch.Tensor, kv_layer: torch.Tensor, page_indices: to
 def stream_norm(x: torch.Tensor, w: Optional[torch.Tensor], eps: float, out: Optional[torch.Tensor], *,
                 w_offset: float = 0.0, ids: Optional[torch.Tensor] = None, embed: Optional[torch.Tensor] = None,
                 init: bool = False, add_embed: bool = False, step: Optional[torch.Tensor] = None,
-                rows: Optional[torch.Tensor] = None, row_offset: int = 0,
-                num_tokens: Optional[int] = None) -> Optional[torch.Tensor]:
+                rows: Optional[torch.Tensor] = None, row_offset: int = 0, num_tokens: Optional[int] = None,
+                add: Optional[torch.Tensor] = None, add_rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """Additions to the fp32 residual stream ``x`` ([T, hidden], in place) and the RMSNorm that follows, in one kernel.
 
     ``init``: x starts as ``embed[ids]``; ``add_embed``: the embeddings are added to it; ``step``: a vector added to
-    every row.  ``out`` (None: no norm) = x / rms(x) * (w_offset + w).  ``rows``: output row t takes row
+    every row; ``add``: row t receives the rows ``add_rows[t]`` ([T, n] int32) of it.  ``out`` (None: no norm) = x / rms(x) * (w_offset + w).  ``rows``: output row t takes row
     ``rows[t] + row_offset`` of x."""
     n = num_tokens if num_tokens is not None else (rows.numel() if rows is not None else x.shape[0])
     assert x.dtype == torch.float32 and x.is_contiguous()
-    ref = out if out is not None else embed
+    ref = out if out is not None else embed if embed is not None else add
     assert out is None or out.is_contiguous()
-    _check(lib().blitz_stream_norm(_p(ids), _p(embed), _p(step), _p(rows), row_offset, _p(x), _p(w), _p(out), n,
+    n_add = 0
+    if add is not None:
+        n_add = add_rows.shape[1]
+        assert add.is_contiguous() and add.shape[1] == x.shape[1] and add_rows.is_contiguous() and add_rows.dtype == torch.int32
+        assert add_rows.shape[0] >= n and add.dtype == ref.dtype
+    _check(lib().blitz_stream_norm(_p(ids), _p(embed), _p(step), _p(rows), row_offset, _p(x), _p(w), _p(out), _p(add), _p(add_rows),
+                                   n_add, n,
                                    x.shape[1], embed.shape[0] if embed is not None else 0, int(init), int(add_embed),
                                    eps, w_offset, _p(status_word(x.device)), _dt3(ref), _stream()), "blitz_stream_norm")
     return out
 
 
-def rope_freqs(dims: int, base: float, device) -> torch.Tensor:
-    """[dims / 2, 2]: base^(-2 i / dims) as an unevaluated sum of two fp32 numbers."""
+def rope_freqs(dims: int, base: float, device, stretch: Optional[Sequence[float]] = None) -> torch.Tensor:
+    """[dims / 2, 2]: base^(-2 i / dims) (times ``stretch[i]``) as an unevaluated sum of two fp32 numbers."""
     i = torch.arange(0, dims // 2, dtype=torch.float64)
     f = torch.pow(torch.tensor(base, dtype=torch.float64), -2.0 * i / max(1, dims))
+    if stretch is not None:
+        f = f * torch.tensor(stretch, dtype=torch.float64)
     hi = f.to(torch.float32)
     lo = (f - hi.to(torch.float64)).to(torch.float32)
     return torch.stack([hi, lo], 1).contiguous().to(device)
 
 
-def rope_store(q: torch.Tensor, k: torch.Tensor, v: Optional[torch.Tensor], pos: torch.Tensor, slot: torch.Tensor,
-               kv_layer: torch.Tensor, freqs: torch.Tensor, *, q_heads: int, kv_heads: int, dim: int, rot_dims: int,
-               page_size: int, interleaved: bool) -> None:
+def rope_store(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tensor], pos: torch.Tensor, slot: torch.Tensor,
+               kv_layer: KVLayer, freqs: torch.Tensor, *, q_heads: int, kv_heads: int, dim: int, rot_dims: int,
+               page_size: int, interleaved: bool, gain: float = 1.0, q_b: Optional[torch.Tensor] = None,
+               k_b: Optional[torch.Tensor] = None, v_b: Optional[torch.Tensor] = None) -> None:
     """Rotate q in place and write rotated keys and the values to the paged cache.  q, k, v: column ranges of one
-    projection ([T, ...] views with a common row pitch); ``v`` None: the values are the keys before rotation."""
+    projection ([T, ...] views with a common row pitch); ``v`` None: the values are the keys before rotation; ``k`` None:
+    nothing is written.  ``q_b``, ``k_b``, ``v_b``: biases, added first.  ``gain`` multiplies the rotated dimensions."""
     T = q.shape[0]
-    assert q.stride(0) == k.stride(0) and q.stride(1) == 1 and k.stride(1) == 1
-    assert v is None or v.stride(0) == q.stride(0)
-    _check(lib().blitz_rope_store(_p(q), _p(k), _p(v), q.stride(0), _p(pos), _p(slot), _p(kv_layer), _p(freqs), T, q_heads,
-                                  kv_heads, dim, rot_dims, int(interleaved), page_size, kv_layer.shape[0],
+    assert q.stride(1) == 1 and all(x is None or (x.stride(0) == q.stride(0) and x.stride(1) == 1) for x in (k, v))
+    kp, vp, page_rows, pages, vdim = _kv(kv_layer)
+    _check(lib().blitz_rope_store(_p(q), _p(k), _p(v), _p(q_b), _p(k_b), _p(v_b), q.stride(0), _p(pos), _p(slot), kp, vp, _p(freqs),
+                                  gain, T, q_heads, kv_heads, dim, vdim, rot_dims, int(interleaved), page_size, page_rows, pages,
                                   _p(status_word(q.device)), _dt3(q), _stream()), "blitz_rope_store")
 
 
-def attn_ragged(q: torch.Tensor, kv_layer: torch.Tensor, pos: torch.Tensor, tok_indptr: Optional[torch.Tensor],
+def attn_ragged(q: torch.Tensor, kv_layer: KVLayer, pos: torch.Tensor, tok_indptr: Optional[torch.Tensor],
                 page_indptr: torch.Tensor, page_indices: torch.Tensor, out: torch.Tensor, *, q_heads: int, kv_heads: int,
                 dim: int, page_size: int, scale: float, window: int = 0, keep_first: int = 0, softcap: float = 0.0,
-                sink: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """General paged attention (CUDA cores, any head size, any element type); see csrc/kernels/attn_ragged.cu."""
+                sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """General paged attention (CUDA cores, any head sizes, any element type); see csrc/kernels/attn_ragged.cu.  ``gate``
+    [T, q_heads]: a head's output is multiplied by its sigmoid."""
     T = q.shape[0]
     rows = page_indptr.numel() - 1
     assert q.stride(1) == 1 and out.stride(1) == 1
-    _check(lib().blitz_attn_ragged(_p(q), q.stride(0), _p(kv_layer), _p(out), out.stride(0), _p(pos), _p(tok_indptr),
-                                   _p(page_indptr), _p(page_indices), _p(sink), T, rows, q_heads, kv_heads, dim, page_size,
-                                   kv_layer.shape[0], window, keep_first, scale, softcap, _p(status_word(q.device)),
+    kp, vp, page_rows, pages, vdim = _kv(kv_layer)
+    _check(lib().blitz_attn_ragged(_p(q), q.stride(0), kp, vp, _p(out), out.stride(0), _p(pos), _p(tok_indptr),
+                                   _p(page_indptr), _p(page_indices), _p(sink), *_gate(gate), T, rows, q_heads, kv_heads, dim, vdim,
+                                   page_size, page_rows, pages, window, keep_first, scale, softcap, _p(status_word(q.device)),
                                    _dt3(q), _stream()), "blitz_attn_ragged")
+    return out
+
+
+# ---------------------------------------------------------------------------------------------- mixture of experts
+class ExpertPlan:
+    """Work list of the grouped products of a step, in buffers for up to ``max_tokens`` tokens (see csrc/kernels/moe_route.cu):
+    filled by `moe_route` on the device, read by `gemm_grouped` and by `stream_norm` (``place``)."""
+
+    def __init__(self, max_tokens: int, experts: int, top: int, shared: bool, device):
+        i32 = lambda *shape: torch.zeros(*shape, dtype=torch.int32, device=device)
+        self.experts, self.top, self.shared, self.max_tokens = experts, top, int(shared), max_tokens
+        rows = max_tokens * (top + self.shared)
+        self.pairs, self.counters, self.num_tiles = i32(max_tokens * top, 2), i32(experts + 1), i32(1)
+        self.src, self.factors = i32(rows), torch.zeros(rows, 2, dtype=torch.float32, device=device)
+        self._place, self._tiles = i32(rows), i32(self.tiles_at_most(max_tokens, 64), 4)
+        self.tokens, self.tile_rows = 0, 128
+
+    def tiles_at_most(self, tokens: int, tile_rows: int) -> int:
+        pairs = tokens * self.top
+        return min(pairs, self.experts) + pairs // tile_rows
+
+    @property
+    def rows(self) -> int:
+        return self.tokens * (self.top + self.shared)
+
+    @property
+    def place(self) -> torch.Tensor:
+        return self._place[:self.rows].view(self.tokens, self.top + self.shared)
+
+    def tiles_usually(self) -> int:
+        pairs = self.tokens * self.top
+        return max(1, round(self.experts * (1.0 - (1.0 - 1.0 / self.experts) ** pairs)) + pairs // self.tile_rows)
+
+
+def moe_route(logits: torch.Tensor, plan: ExpertPlan, *, weight_on_input: bool = True, renormalize: bool = False,
+              tile_rows: int = 128) -> ExpertPlan:
+    """Choose experts from fp32 router logits [T, experts (+ 1: gate of the shared expert)] and sort the rows by expert."""
+    T = logits.shape[0]
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1 and logits.shape[1] >= plan.experts + plan.shared
+    assert T <= plan.max_tokens and tile_rows >= 64
+    plan.tokens, plan.tile_rows = T, tile_rows
+    _check(lib().blitz_moe_route(_p(logits), logits.stride(0), T, plan.experts, plan.top, plan.shared, int(weight_on_input),
+                                 int(renormalize), tile_rows, plan.tiles_at_most(T, tile_rows), _p(plan.pairs), _p(plan.counters),
+                                 _p(plan.src), _p(plan.factors), _p(plan._place), _p(plan._tiles), _p(plan.num_tiles),
+                                 _p(status_word(logits.device)), _stream()), "blitz_moe_route")
+    return plan
+
+
+_ACT = {"none": 0, "relu2": 1}
+
+
+def grouped_tensor_core(a: torch.Tensor, *matrices: Optional[torch.Tensor]) -> bool:
+    """Whether `gemm_grouped` runs these operands on the tensor cores (else on the CUDA cores, with tile_rows 64)."""
+    return (a.dtype in _DT and a.stride(0) % 8 == 0 and a.data_ptr() % 16 == 0
+            and all(m is None or (m.shape[-1] % 8 == 0 and m.shape[-2] % 8 == 0 and m.data_ptr() % 16 == 0) for m in matrices))
+
+
+def gemm_grouped(a: torch.Tensor, b: torch.Tensor, plan: ExpertPlan, out: torch.Tensor, *, shared: Optional[torch.Tensor] = None,
+                 gather: bool = False, act: str = "none", factors: bool = False, bn: int = 0) -> torch.Tensor:
+    """out[r] = after_r * act(before_r * (a[row] @ b[expert of r])) for the plan's sorted rows r; ``b`` [experts, K, N];
+    ``shared`` [K', N']: the shared expert's matrix for the rows behind (K' and N' columns of a and out).  ``gather``: row r
+    reads the activation of its token, else sorted row r.  ``factors``: apply the plan's factors (else both are 1)."""
+    E, K, N = b.shape
+    assert E == plan.experts and b.is_contiguous() and a.stride(1) == 1 and out.stride(1) == 1 and a.dtype == b.dtype == out.dtype
+    assert (shared is not None) == bool(plan.shared) and out.shape[0] >= plan.rows
+    Ks, Ns = (K, N) if shared is None else shared.shape
+    assert a.shape[1] >= max(K, Ks) and out.shape[1] >= max(N, Ns) and (shared is None or shared.is_contiguous())
+    src, fac = plan.src if gather else None, plan.factors if factors else None
+    row0, shared_rows = plan.tokens * plan.top, plan.tokens * plan.shared
+    most = plan.tiles_at_most(plan.tokens, plan.tile_rows)
+    if plan.tile_rows == 64:
+        _check(lib().blitz_gemm_grouped_simt(_p(a), a.stride(0), _p(src), _p(b), N, K, _p(shared), Ns, Ks, _p(out), out.stride(0),
+                                             _p(fac), _p(plan._tiles), _p(plan.num_tiles), most, row0, shared_rows, _ACT[act],
+                                             _dt3(a), _stream()), "blitz_gemm_grouped_simt")
+        return out
+    assert plan.tile_rows == 128 and grouped_tensor_core(a, b, shared) and out.stride(0) % 8 == 0
+    _check(lib().blitz_gemm_grouped(_p(a), a.stride(0), plan.tokens if gather else plan.rows, _p(src), _p(b), E, N, K, _p(shared), Ns,
+                                    Ks, _p(out), out.stride(0), _p(fac), _p(plan._tiles), _p(plan.num_tiles), most,
+                                    plan.tiles_usually(), row0, shared_rows, plan.tokens, _ACT[act], bn,
+                                    _p(status_word(a.device)), _dt(a), _stream()), "blitz_gemm_grouped")
     return out
 
 

@@ -86,16 +86,23 @@ def _declare(L: ctypes.CDLL) -> None:
     sig("blitz_sample", [c_p, c_i, c_i, c_i64, c_p, c_p, c_p, c_p, c_u64, c_p, c_i, c_p])
     sig("blitz_rope_kv_store", [c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_p, c_i, c_p])
     sig("blitz_attn_decode_workspace_bytes", [c_i, c_i, c_i, c_i], c_i64)
-    sig("blitz_attn_decode", [c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f,
-                              c_i, c_i, c_f, c_p, c_p, c_i, c_p])
-    sig("blitz_attn_prefill_paged", [c_p, c_i64, c_p, c_p, c_i64, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i,
-                                     c_i, c_i, c_f, c_p, c_p, c_i, c_p])
+    sig("blitz_attn_decode", [c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f,
+                              c_i, c_i, c_f, c_p, c_p, c_i64, c_p, c_i, c_p])
+    sig("blitz_attn_prefill_paged", [c_p, c_i64, c_p, c_p, c_p, c_i64, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f,
+                                     c_i, c_i, c_i, c_f, c_p, c_p, c_i64, c_p, c_i, c_p])
     # models with an fp32 residual stream and recurrent layers
     sig("blitz_gemm_simt", [c_p, c_i64, c_p, c_i64, c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_p])
-    sig("blitz_stream_norm", [c_p, c_p, c_p, c_p, c_i, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_p, c_i, c_p])
-    sig("blitz_rope_store", [c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_i, c_p])
-    sig("blitz_attn_ragged", [c_p, c_i64, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i,
-                              c_i, c_f, c_f, c_p, c_i, c_p])
+    sig("blitz_stream_norm", [c_p, c_p, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_p, c_i,
+                              c_p])
+    sig("blitz_rope_store", [c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_f, c_i, c_i, c_i, c_i, c_i, c_i, c_i,
+                             c_i, c_i, c_i, c_p, c_i, c_p])
+    sig("blitz_attn_ragged", [c_p, c_i64, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_i,
+                              c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_p, c_i, c_p])
+    sig("blitz_moe_route", [c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p])
+    sig("blitz_gemm_grouped", [c_p, c_i64, c_i, c_p, c_p, c_i, c_i, c_i, c_p, c_i, c_i, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i, c_i,
+                               c_i, c_i, c_i, c_p, c_i, c_p])
+    sig("blitz_gemm_grouped_simt", [c_p, c_i64, c_p, c_p, c_i, c_i, c_p, c_i, c_i, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i,
+                                    c_p])
     sig("blitz_gla_recurrent", [c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_i, c_i,
                                 c_i, c_i, c_i, c_i, c_f, c_f, c_f, c_i, c_p, c_i, c_p])
     sig("blitz_gla_chunk", [c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i,

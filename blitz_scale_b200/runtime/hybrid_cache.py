@@ -2,23 +2,27 @@
 
 A page id addresses the same page in the pool of every attention run, and a slot id the same slot in the state arrays
 of every recurrent run, so the host bookkeeping (native PagePool, SlotPool and Batch) does not know how many runs there
-are or what shape each has.  A layer that runs several times in one forward pass has one entry per run.
+are or what shape each has.  A layer that runs several times in one forward pass has one entry per run; a layer that
+reads another layer's keys and values has that layer's pool as its entry.
+
+A pool is one tensor with a key and a value plane per page, or a pair of tensors where keys and values differ in size.
 
 Slots are not cleared when they change hands: the kernels start from zero at position 0.  KV pools are zero-filled once
 (the attention kernels require finite values in every slot of an allocated page)."""
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import List, Optional
+from typing import List, Optional, Union
 
 import torch
 
 from ..models.hybrid_config import HybridConfig
+from ..ops import KVPair
 
 
 @dataclass
 class RunCache:
-    kv: Optional[torch.Tensor] = None      # [pages, 2, page, kv_heads, dim]
+    kv: Optional[Union[torch.Tensor, KVPair]] = None   # [pages, 2, page, kv_heads, dim], or two [pages, page, kv_heads, size]
     state: Optional[torch.Tensor] = None   # fp32: [slots, heads, dim, vdim] or [slots, width]
     hist: Optional[torch.Tensor] = None    # last inputs of a short convolution: [slots, taps - 1, width]
 
@@ -27,9 +31,14 @@ class HybridCache:
     def __init__(self, cfg: HybridConfig, num_pages: int, page_size: int, num_slots: int, dtype, device):
         self.cfg, self.num_pages, self.page_size, self.num_slots = cfg, num_pages, page_size, num_slots
         self.runs: List[RunCache] = []
-        for m in cfg.run_mixers():
-            if m.kind == "attention":
-                self.runs.append(RunCache(kv=torch.zeros(num_pages, 2, page_size, m.kv_heads, m.dim, dtype=dtype, device=device)))
+        zeros = lambda *shape: torch.zeros(*shape, dtype=dtype, device=device)
+        for r, (m, source) in enumerate(zip(cfg.run_mixers(), cfg.kv_runs())):
+            if m.kind == "attention" and source != r:
+                self.runs.append(RunCache(kv=self.runs[source].kv))
+            elif m.kind == "attention" and m.vdim != m.dim:
+                self.runs.append(RunCache(kv=KVPair(*(zeros(num_pages, page_size, m.kv_heads, n) for n in (m.dim, m.vdim)))))
+            elif m.kind == "attention":
+                self.runs.append(RunCache(kv=zeros(num_pages, 2, page_size, m.kv_heads, m.dim)))
             elif m.kind == "gla":
                 self.runs.append(RunCache(state=torch.zeros(num_slots, m.heads, m.dim, m.vdim, device=device)))
             else:
@@ -37,4 +46,9 @@ class HybridCache:
                                           hist=torch.zeros(num_slots, m.taps - 1, m.width, dtype=dtype, device=device)))
 
     def bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for r in self.runs for t in (r.kv, r.state, r.hist) if t is not None)
+        held = {}
+        for r in self.runs:
+            for t in (*(r.kv if isinstance(r.kv, KVPair) else (r.kv,)), r.state, r.hist):
+                if t is not None:
+                    held[t.data_ptr()] = t.numel() * t.element_size()
+        return sum(held.values())
