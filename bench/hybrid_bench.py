@@ -71,7 +71,7 @@ def bench_models(out, sizes=("h4096", "h2048"), configs=configs):
                 b = eng.new_batch(1, [core.SeqSpec(i, [1] * ctx, 4) for i in range(B)])
                 assert b is not None
                 b.mark_prefilled()                      # contents do not matter for the time
-                b.append_tokens([1] * B, False)
+                b.append_tokens(torch.randint(0, VOCAB, (B,), generator=g).tolist(), False)   # (they choose experts)
                 P = b.fill_decode(eng.host_np, eng.layout, _bucket(B))
                 eng._h2d(eng.layout.page_indices + P)
                 graph = eng._capture(_bucket(B), eng.choose_splits(_bucket(B), b.max_seq_len()))

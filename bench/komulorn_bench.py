@@ -129,7 +129,8 @@ def bench_kernels(out, size):
         rw = rnd(H, (E + 8) // 8 * 8)
         zs = torch.empty(T, rw.shape[1], device=dev)
         hs = [rnd(T, H) for _ in range(n_copies(T * H * 2))][:40]
-        t = timeit(lambda i: ops.gemm(hs[i], rw, out=zs, static_b=True), copies=len(hs))
+        narrow = dict(bn=64, split_k=4 if T <= 2048 else 1) if T > ops.DECODE_GEMM_MAX_M else {}         # as the runner does
+        t = timeit(lambda i: ops.gemm(hs[i], rw, out=zs, static_b=True, **narrow), copies=len(hs))
         rep("gemm router", t, by=2.0 * (T * H + H * rw.shape[1]) + 4.0 * T * rw.shape[1], fl=2.0 * T * H * rw.shape[1], M=T)
         # the head with capped logits beside the plain one
         if T <= 256:

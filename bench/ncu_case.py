@@ -2,6 +2,7 @@
 
     python bench/ncu_case.py gemm M N K [epilogue]       # 3 launches of the tcgen05 GEMM
     python bench/ncu_case.py attn_decode B CTX            # 3 launches of the paged decode attention
+    python bench/ncu_case.py experts T                    # 3 rounds of router, grouped up and grouped down product
     python bench/ncu_case.py attn_prefill_paged B N       # 3 launches of the paged prefill attention (64-token pages)
 """
 import os
@@ -45,6 +46,17 @@ def main():
         work = ops.prefill_work_list([n] * B, [n] * B, ps, "cuda")
         for _ in range(3):
             ops.attn_prefill_paged(qkv, pool, ids, work, q_heads=qh, kv_heads=kvh, head_dim=hd, page_size=ps)
+    elif kind == "experts":
+        T = int(sys.argv[2])
+        H, E, top, ff, sff = 2048, 64, 6, 1408, 2816
+        rnd = lambda *s: torch.randn(*s, device="cuda", dtype=torch.bfloat16)
+        up, down, s_up, s_down = rnd(E, H, ff), rnd(E, ff, H), rnd(H, sff), rnd(sff, H)
+        h, z, plan = rnd(T, H), torch.randn(T, E + 8, device="cuda"), ops.ExpertPlan(T, E, top, True, "cuda")
+        act, y = torch.empty(T * (top + 1), sff, device="cuda", dtype=torch.bfloat16), rnd(T * (top + 1), H)
+        for _ in range(3):
+            ops.moe_route(z, plan)
+            ops.gemm_grouped(h, up, plan, act, shared=s_up, gather=True, act="relu2", factors=True)
+            ops.gemm_grouped(act, down, plan, y, shared=s_down)
     elif kind == "decode_step":
         # two eager decode steps of the full model (no CUDA graph), for a per-kernel launch list of one step:
         #   ncu --metrics gpu__time_duration.sum -k regex:"blitz|gemm|attn|rms|rope|argmax|embedding|sample" ...

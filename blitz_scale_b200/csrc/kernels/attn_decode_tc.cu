@@ -66,6 +66,7 @@ struct DecodeTcParams {
   int batch, q_heads, kv_heads, group, page_size, max_pages, num_splits, box_tokens;
   int kv_div;               // kv_heads counts groups of at most 8 query heads: kv_div of them share a KV head
   int dim, vdim, page_rows; // page n's token `off` is row n * page_rows + off of both pools
+  int v_rows;               // > 0: one tensor (and one map) for keys and values, which lie this many rows behind their keys
   const void* gate;         // [batch][gate_stride], a column per query head, or null
   int64_t gate_stride;
   int tail_box_tokens;  // box height of the second tensor map, used for the last (partly filled) chunk of a sequence
@@ -97,7 +98,7 @@ __device__ __forceinline__ float head_gate(const T* z) { return 1.f / (1.f + exp
 // blockIdx.x, blockIdx.x + gridDim.x, ... and the producer keeps streaming the next item's pages while
 // the consumers finish the current one, so the 4-stage pipeline never drains between items.
 struct DecItem {
-  int b, h, split, pg_beg, seq_len, c_beg, c_end;  // c_beg .. c_end: this split's share of the visible chunks
+  int b, h, kv_head, split, pg_beg, seq_len, c_beg, c_end;  // c_beg .. c_end: this split's share of the visible chunks
   int lo, first;         // visible keys: [0, first) and [lo, seq_len)
   int n_first, c_window; // chunks of the kept tokens; first chunk of the window behind them
   // the n-th visible chunk
@@ -107,6 +108,7 @@ __device__ __forceinline__ DecItem dec_item(const DecodeTcParams& p, int item) {
   DecItem it;
   it.split = item % p.num_splits;
   it.h = (item / p.num_splits) % p.kv_heads;
+  it.kv_head = p.kv_div == 1 ? it.h : it.h / p.kv_div;
   it.b = item / (p.num_splits * p.kv_heads);
   it.pg_beg = p.indptr[it.b];
   const int npages = p.indptr[it.b + 1] - it.pg_beg;
@@ -122,13 +124,15 @@ __device__ __forceinline__ DecItem dec_item(const DecodeTcParams& p, int item) {
   return it;
 }
 
-template <typename T, int HD, int VD = HD>
+// PLAIN: heads as large as the tiles, one tensor for keys and values, no gate, at most 8 query heads per KV head.
+template <typename T, int HD, int VD = HD, bool PLAIN = true>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_k_tail,
                       const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_v_tail,
                       const DecodeTcParams p) {
   using Cfg = TcCfg<HD, VD>;
   constexpr int SL = Cfg::kSlabs, SV = Cfg::kValueSlabs;
+  const int dim = PLAIN ? HD : p.dim, vdim = PLAIN ? VD : p.vdim;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw_addr = ptx::smem_u32(smem_raw);
   uint8_t* smem = smem_raw + (((raw_addr + 1023u) & ~1023u) - raw_addr);
@@ -198,7 +202,8 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
         // filled, in the smaller boxes of the second map (a 64-token page with 18 live tokens costs 32 rows)
         const bool tail = ntok < kTcChunk;
         const int bt = tail ? p.tail_box_tokens : p.box_tokens;
-        const CUtensorMap *tk = tail ? &tmap_k_tail : &tmap_k, *tv = tail ? &tmap_v_tail : &tmap_v;
+        const CUtensorMap* tk = tail ? &tmap_k_tail : &tmap_k;
+        const CUtensorMap* tv = PLAIN || p.v_rows > 0 ? tk : tail ? &tmap_v_tail : &tmap_v;
         const uint32_t box_bytes = static_cast<uint32_t>(bt) * 128u;
         const int pieces = (ntok + bt - 1) / bt;
         const int last_page = (tok0 + ntok - 1) / ps;
@@ -229,11 +234,11 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
               if (p.status) atomicCAS(p.status, 0, kStatusBadIndex);
               page = 0;
             }
-            const int z = page * p.page_rows + (t % ps), h = it.h / p.kv_div;
+            const int z = page * (PLAIN ? 2 * ps : p.page_rows) + (t % ps), h = PLAIN ? it.h : it.kv_head;
 #pragma unroll
             for (int s = 0; s < (SL > SV ? SL : SV); ++s) {
               if (s < SL) ptx::tma_load_3d(sb + s * kTcSlabBytes + i * box_bytes, tk, &full_bar[stage], s * 64, h, z);
-              if (s < SV) ptx::tma_load_3d(sb + (SL + s) * kTcSlabBytes + i * box_bytes, tv, &full_bar[stage], s * 64, h, z);
+              if (s < SV) ptx::tma_load_3d(sb + (SL + s) * kTcSlabBytes + i * box_bytes, tv, &full_bar[stage], s * 64, h, z + (PLAIN ? ps : p.v_rows));
             }
           }
         }
@@ -262,9 +267,9 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
     // So the next item's descriptor and Q fragments are requested while the current item is being processed.
     auto load_q = [&](const DecItem& d, uint32_t (&a0)[HD / 16], uint32_t (&a2)[HD / 16]) {
       // Q as A fragments (rows >= G and columns >= dim are zero padding; rows 8..15 are never populated since G <= 8)
-      const int cols = g < G ? p.dim : 0;
+      const int cols = g < G ? dim : 0;
       const T* qrow = reinterpret_cast<const T*>(p.q) + static_cast<int64_t>(d.b) * p.q_stride +
-                      static_cast<int64_t>(d.h * G + g) * p.dim;
+                      static_cast<int64_t>(d.h * G + g) * dim;
 #pragma unroll
       for (int ks = 0; ks < HD / 16; ++ks) {
         a0[ks] = ks * 16 < cols ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + 2 * t4) : 0u;
@@ -383,7 +388,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
       asm volatile("bar.sync 1, 128;" ::: "memory");
       for (int e = threadIdx.x; e < G * VD; e += 128) {
         const int gg = e / VD, d = e % VD;
-        if (d >= p.vdim) continue;
+        if (!PLAIN && d >= vdim) continue;
         float M = -INFINITY;
 #pragma unroll
         for (int w = 0; w < 4; ++w) M = fmaxf(M, mrg_m[w * 8 + gg]);
@@ -403,16 +408,16 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
         if (with_sink) L += exp2f(sink - M);
         float val = L > 0.f ? O / L : 0.f;
         if (p.num_splits == 1) {
-          if (p.gate != nullptr) val *= head_gate(reinterpret_cast<const T*>(p.gate) + it.b * p.gate_stride + head);
+          if (!PLAIN && p.gate != nullptr) val *= head_gate(reinterpret_cast<const T*>(p.gate) + it.b * p.gate_stride + head);
           T* op = reinterpret_cast<T*>(p.out) + static_cast<int64_t>(it.b) * p.out_stride +
-                  static_cast<int64_t>(head) * p.vdim;
+                  static_cast<int64_t>(head) * vdim;
           if (std::is_same<T, __nv_bfloat16>::value)
             reinterpret_cast<__nv_bfloat16*>(op)[d] = __float2bfloat16(val);
           else
             reinterpret_cast<__half*>(op)[d] = __float2half(val);
         } else {
           const int64_t base = (static_cast<int64_t>(it.b) * p.q_heads + head) * p.num_splits + it.split;
-          p.part_o[base * p.vdim + d] = val;
+          p.part_o[base * vdim + d] = val;
           if (d == 0) p.part_lse[base] = L > 0.f ? M + log2f(L) : -INFINITY;
         }
       }
@@ -459,10 +464,10 @@ __global__ void attn_merge_tc_kernel(const float* __restrict__ part_o, const flo
   }
 }
 
-template <typename T, int HD, int VD>
+template <typename T, int HD, int VD, bool PLAIN>
 static int launch_tc(const CUtensorMap (&tm)[4], const DecodeTcParams& p, int batch, cudaStream_t stream) {
   using Cfg = TcCfg<HD, VD>;
-  auto kern = attn_decode_tc_kernel<T, HD, VD>;
+  auto kern = attn_decode_tc_kernel<T, HD, VD, PLAIN>;
   static PerDeviceOnce once;
   cudaError_t e = once.run([&] { return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes); });
   if (e != cudaSuccess) return (int)e;
@@ -474,8 +479,11 @@ static int launch_tc(const CUtensorMap (&tm)[4], const DecodeTcParams& p, int ba
 
 template <typename T>
 static int launch_tc(const CUtensorMap (&tm)[4], const DecodeTcParams& p, int batch, cudaStream_t stream) {
-  if (p.dim > 64) return p.vdim > 64 ? launch_tc<T, 128, 128>(tm, p, batch, stream) : launch_tc<T, 128, 64>(tm, p, batch, stream);
-  return p.vdim > 64 ? launch_tc<T, 64, 128>(tm, p, batch, stream) : launch_tc<T, 64, 64>(tm, p, batch, stream);
+  const bool plain = p.dim == p.vdim && (p.dim == 64 || p.dim == 128) && p.v_rows > 0 && p.gate == nullptr && p.kv_div == 1;
+  if (plain) return p.dim == 64 ? launch_tc<T, 64, 64, true>(tm, p, batch, stream) : launch_tc<T, 128, 128, true>(tm, p, batch, stream);
+  if (p.dim > 64)
+    return p.vdim > 64 ? launch_tc<T, 128, 128, false>(tm, p, batch, stream) : launch_tc<T, 128, 64, false>(tm, p, batch, stream);
+  return p.vdim > 64 ? launch_tc<T, 64, 128, false>(tm, p, batch, stream) : launch_tc<T, 64, 64, false>(tm, p, batch, stream);
 }
 
 }  // namespace blitz
@@ -520,8 +528,11 @@ int blitz_attn_decode(const void* q, int64_t q_stride, const void* k_pool, const
   while (group % div) ++div;
   const int bt = page_size < kTcChunk ? page_size : kTcChunk;
   const int bt_tail = bt < 16 ? bt : 16;
+  const bool one = dim == vdim && page_rows == 2 * page_size &&
+                   v_pool == reinterpret_cast<const char*>(k_pool) + (int64_t)page_size * kv_heads * dim * 2;
+  if (one) v_pool = k_pool;
   // rows of a pool: those of the last page end with its tokens
-  const uint64_t rows = (uint64_t)(max_pages - 1) * page_rows + page_size;
+  const uint64_t rows = one ? (uint64_t)max_pages * page_rows : (uint64_t)(max_pages - 1) * page_rows + page_size;
   CUtensorMap tm[4];
   for (int i = 0; i < 4; ++i) {
     const uint64_t d = i < 2 ? dim : vdim;
@@ -535,7 +546,7 @@ int blitz_attn_decode(const void* q, int64_t q_stride, const void* k_pool, const
   p.part_o = reinterpret_cast<float*>(workspace);
   p.part_lse = p.part_o ? p.part_o + (int64_t)batch * q_heads * num_splits * vdim : nullptr;
   p.batch = batch; p.q_heads = q_heads; p.kv_heads = kv_heads * div; p.kv_div = div; p.group = group / div;
-  p.page_size = page_size; p.max_pages = max_pages; p.dim = dim; p.vdim = vdim; p.page_rows = page_rows;
+  p.page_size = page_size; p.max_pages = max_pages; p.dim = dim; p.vdim = vdim; p.page_rows = page_rows; p.v_rows = one ? page_size : 0;
   p.num_splits = num_splits; p.box_tokens = bt; p.tail_box_tokens = bt_tail;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = g_tc_trace;
   p.window = window; p.keep_first = keep_first; p.sink = sink; p.gate = gate; p.gate_stride = gate_stride;
@@ -593,16 +604,16 @@ static cudaError_t noalloc_setup(int dev) {
   return cudaSuccess;
 }
 
-// Tensor map of the key or value planes of one KV layer built on the stack (the cached builder keeps a host-side table; this path keeps nothing).
-static bool noalloc_tmap(CUtensorMap* out, const void* pool, int head_dim, int kv_heads, int max_pages, int page_size,
+// Tensor map of one KV layer built on the stack (the cached builder keeps a host-side table; this path keeps nothing).
+static bool noalloc_tmap(CUtensorMap* out, const void* kv_layer, int head_dim, int kv_heads, int max_pages, int page_size,
                          int box_tokens) {
   PFN_encodeTiled enc = get_encode_fn();
-  if (!enc || (reinterpret_cast<uintptr_t>(pool) & 15) != 0) return false;
-  cuuint64_t dims[3] = {(cuuint64_t)head_dim, (cuuint64_t)kv_heads, (cuuint64_t)(2 * max_pages - 1) * page_size};
+  if (!enc || (reinterpret_cast<uintptr_t>(kv_layer) & 15) != 0) return false;
+  cuuint64_t dims[3] = {(cuuint64_t)head_dim, (cuuint64_t)kv_heads, (cuuint64_t)max_pages * 2 * page_size};
   cuuint64_t strides[2] = {(cuuint64_t)head_dim * 2, (cuuint64_t)kv_heads * head_dim * 2};
   cuuint32_t box[3] = {64, 1, (cuuint32_t)box_tokens};
   cuuint32_t estr[3] = {1, 1, 1};
-  return enc(out, CU_TENSOR_MAP_DATA_TYPE_UINT16, 3, const_cast<void*>(pool), dims, strides, box, estr,
+  return enc(out, CU_TENSOR_MAP_DATA_TYPE_UINT16, 3, const_cast<void*>(kv_layer), dims, strides, box, estr,
              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
@@ -640,10 +651,8 @@ extern "C" int blitz_attn_decode_noalloc(const void* q, int64_t q_stride, const 
   const int bt = page_size < kTcChunk ? page_size : kTcChunk;
   const int bt_tail = bt < 16 ? bt : 16;
   CUtensorMap tm[4];
-  for (int i = 0; i < 4; ++i) {
-    const char* pool = reinterpret_cast<const char*>(kv_layer) + (i < 2 ? 0 : (int64_t)page_size * kv_heads * head_dim * 2);
-    if (!noalloc_tmap(&tm[i], pool, head_dim, kv_heads, max_pages, page_size, i & 1 ? bt_tail : bt)) return -2;
-  }
+  for (int i = 0; i < 4; ++i)
+    if (!noalloc_tmap(&tm[i], kv_layer, head_dim, kv_heads, max_pages, page_size, i & 1 ? bt_tail : bt)) return -2;
   DecodeTcParams p;
   p.q = q; p.q_stride = q_stride; p.indices = indices; p.indptr = indptr; p.last_page_len = last_page_len;
   p.out = out; p.out_stride = out_stride;
@@ -652,7 +661,7 @@ extern "C" int blitz_attn_decode_noalloc(const void* q, int64_t q_stride, const 
   p.batch = batch; p.q_heads = q_heads; p.kv_heads = kv_heads; p.group = G; p.page_size = page_size;
   p.max_pages = max_pages; p.num_splits = num_splits; p.box_tokens = bt; p.tail_box_tokens = bt_tail;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = nullptr;
-  p.kv_div = 1; p.dim = p.vdim = head_dim; p.page_rows = 2 * page_size; p.gate = nullptr; p.gate_stride = 0;
+  p.kv_div = 1; p.dim = p.vdim = head_dim; p.page_rows = 2 * page_size; p.v_rows = page_size; p.gate = nullptr; p.gate_stride = 0;
   p.window = 0; p.keep_first = 0; p.sink = nullptr; p.cap_scale = p.cap_log2 = 0.f;
   int sms = 0;
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);

@@ -110,13 +110,14 @@ __device__ __forceinline__ void dec_store32(const DecGemmParams& p, const float 
   if (EPI >= 4) {
     float* cf = reinterpret_cast<float*>(p.C) + n;
     float old[32];
+    const float inv = EPI == 6 ? 1.f / p.alpha : 0.f;
     if (EPI == 5) {
 #pragma unroll
       for (int i = 0; i < 32; ++i) old[i] = (b0 + i < b_end) ? cf[static_cast<int64_t>(b0 + i) * p.ldc] : 0.f;
     }
 #pragma unroll
     for (int i = 0; i < 32; ++i)
-      if (b0 + i < b_end) cf[static_cast<int64_t>(b0 + i) * p.ldc] = EPI == 5 ? old[i] + p.alpha * g[i] : EPI == 6 ? p.alpha * tanhf(g[i] / p.alpha) : g[i];
+      if (b0 + i < b_end) cf[static_cast<int64_t>(b0 + i) * p.ldc] = EPI == 5 ? old[i] + p.alpha * g[i] : EPI == 6 ? p.alpha * ptx::tanh_ex2(g[i] * inv) : g[i];
     return;
   }
   T* c = reinterpret_cast<T*>(p.C) + n;

@@ -4,8 +4,10 @@
 //
 // Sorted rows r and their work list come from moe_route.cu on the device, so the launch does not depend on how tokens are
 // spread over the experts and can be captured in a graph.  The shared expert, whose matrix may have another size, is one
-// more group over all tokens.  The first product of an expert gathers its rows through `src` while loading (TMA gather,
-// four rows per request), so tokens are never copied into expert order; the second one reads the first one's sorted rows.
+// more group over all tokens.  The first product of an expert gathers its rows through `src` while loading, so tokens are
+// never copied into expert order; the second one reads the first one's sorted rows.  Two ways to gather: TMA gather (four
+// rows per request, about 90 cycles each: right for the few rows per expert of a decode step), and four more warps that copy
+// 16-byte pieces with cp.async into the swizzled tile (which keeps up with full tiles).
 //
 // A work item is one tile of at most 128 rows of one expert and BN columns.  Persistent grid, warp-specialised as in
 // gemm_tcgen05.cu: load warp (every lane requests four gathered rows, or one box; some lanes a 64-column slab of B), one
@@ -21,11 +23,17 @@
 
 namespace blitz {
 
-constexpr int kGgRows = 128, kGgK = 64, kGgThreads = 192, kGgMaxStages = 16, kGgBox = 32;
+constexpr int kGgRows = 128, kGgK = 64, kGgThreads = 192, kGgMaxStages = 16;
+constexpr int kGgGather4Rows = 64;   // tiles of more rows than this are gathered by the copying warps
+constexpr int kGgCopyThreads = 128;
+
+// how a tile of A is fetched: sorted rows by boxes, or gathered by TMA or by copying warps
+enum GgFetch : int { kGgBoxes = 0, kGgGather4 = 1, kGgCopy = 2 };
 
 struct GroupedTcParams {
   GroupedParams g;
   int a_rows;      // rows a stage of A holds: min(128, rows any tile can have), a multiple of 32
+  int box;         // rows per box of A: 32, or 128 where tiles are mostly full
   int src_rows;    // rows of A (bound of src)
   int sh_tiles, tn, tn_shared;
   int* status;
@@ -38,9 +46,21 @@ struct GgCfg {
   static constexpr int kSmemBytes = 227 * 1024;
   static constexpr int kUsable = kSmemBytes - 1024 - kBarBytes;
   // (the 128-row view of the last short stage of A ends in the B stages that follow, which are larger than a tile of A)
-  __host__ __device__ static int stages(int a_rows) {
+  __host__ __device__ static constexpr int stages(int a_rows) {
     const int s = kUsable / (a_rows * 128 + kBBytes);
     return s > kGgMaxStages ? kGgMaxStages : s;
+  }
+};
+
+struct Ring {  // position in the ring of pipeline stages
+  int stage;
+  uint32_t phase;
+  int size;
+  __device__ __forceinline__ void next() {
+    if (++stage == size) {
+      stage = 0;
+      phase ^= 1u;
+    }
   }
 };
 
@@ -67,8 +87,8 @@ __device__ __forceinline__ GgItem gg_item(const GroupedTcParams& p, int w, int n
   return it;
 }
 
-template <typename T, int BN, int ACT, bool GATHER>
-__global__ void __launch_bounds__(kGgThreads, 1)
+template <typename T, int BN, int FETCH>
+__global__ void __launch_bounds__(FETCH == kGgCopy ? kGgThreads + kGgCopyThreads : kGgThreads, 1)
 gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_a_shared,
                     const __grid_constant__ CUtensorMap tmap_b, const __grid_constant__ CUtensorMap tmap_b_shared,
                     const GroupedTcParams p) {
@@ -93,7 +113,7 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < S; ++i) {
-      ptx::mbar_init(&full_bar[i], 1);
+      ptx::mbar_init(&full_bar[i], FETCH == kGgCopy ? 1 + kGgCopyThreads : 1);
       ptx::mbar_init(&empty_bar[i], 1);
     }
     for (int i = 0; i < 2; ++i) {
@@ -120,17 +140,18 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
 
   if (warp == 0) {
     // ------------------------------------------------------------ load warp
-    int stage = 0;
-    uint32_t phase = 0;
+    Ring g{0, 0u, S};
     bool ok = true;
     for (int w = blockIdx.x; w < items && ok; w += gridDim.x) {
       const GgItem it = gg_item(p, w, num_tiles);
       const int n0 = it.n0 * BN, num_kb = (it.t.K + kGgK - 1) / kGgK;
       const CUtensorMap* ta = it.t.shared ? &tmap_a_shared : &tmap_a;
       const CUtensorMap* tb = it.t.shared ? &tmap_b_shared : &tmap_b;
-      int pieces;
+      int pieces = 0;
       int idx[4] = {0, 0, 0, 0};
-      if (GATHER) {
+      // the shared expert's rows are the tokens in order: no need to gather them row by row
+      const bool gather = FETCH == kGgGather4 && !it.t.shared;
+      if (gather) {
         pieces = (it.t.rows + 3) >> 2;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
@@ -141,42 +162,36 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
             idx[j] = 0;
           }
         }
-      } else {
-        pieces = (it.t.rows + kGgBox - 1) / kGgBox;
+      } else if (FETCH != kGgCopy) {
+        pieces = (it.t.rows + p.box - 1) / p.box;
       }
-      const uint32_t tx = static_cast<uint32_t>(pieces) * (GATHER ? 512u : kGgBox * 128u) + Cfg::kBBytes;
+      const uint32_t tx = static_cast<uint32_t>(pieces) * (gather ? 512u : p.box * 128u) + Cfg::kBBytes;
+      const int row0 = FETCH == kGgGather4 ? it.t.row0 - p.g.shared_row0 : it.t.row0;  // of the boxes
       for (int kb = 0; kb < num_kb; ++kb) {
         int good = 1;
         if (lane == 0) {
-          good = ptx::bounded_mbar_wait(&empty_bar[stage], phase ^ 1u, abort_flag) ? 1 : 0;
-          if (good) ptx::mbar_expect_tx(&full_bar[stage], tx);
+          good = ptx::bounded_mbar_wait(&empty_bar[g.stage], g.phase ^ 1u, abort_flag) ? 1 : 0;
+          if (good) ptx::mbar_expect_tx(&full_bar[g.stage], tx);
           else if (p.status) atomicCAS(p.status, 0, kStatusTimeoutProducer);
         }
-        good = __shfl_sync(0xffffffffu, good, 0);
-        if (!good) {
-          ok = false;
-          break;
-        }
-        uint8_t* sa = smem_a + stage * a_stage;
+        ok = __shfl_sync(0xffffffffu, good, 0) != 0;
+        if (!ok) break;
         if (lane < BN / 64)  // slabs of 64 columns x 64 K rows
-          ptx::tma_load_2d(smem_b + stage * Cfg::kBBytes + lane * 8192, tb, &full_bar[stage], n0 + lane * 64, it.t.b_row + kb * kGgK);
+          ptx::tma_load_2d(smem_b + g.stage * Cfg::kBBytes + lane * 8192, tb, &full_bar[g.stage], n0 + lane * 64, it.t.b_row + kb * kGgK);
         if (lane < pieces) {
-          if (GATHER)
-            ptx::tma_gather4(sa + lane * 512, ta, &full_bar[stage], kb * kGgK, idx[0], idx[1], idx[2], idx[3]);
+          uint8_t* sa = smem_a + g.stage * a_stage;
+          if (gather)
+            ptx::tma_gather4(sa + lane * 512, ta, &full_bar[g.stage], kb * kGgK, idx[0], idx[1], idx[2], idx[3]);
           else
-            ptx::tma_load_2d(sa + lane * (kGgBox * 128), ta, &full_bar[stage], kb * kGgK, it.t.row0 + lane * kGgBox);
+            ptx::tma_load_2d(sa + lane * (p.box * 128), ta, &full_bar[g.stage], kb * kGgK, row0 + lane * p.box);
         }
-        if (++stage == S) {
-          stage = 0;
-          phase ^= 1u;
-        }
+        g.next();
       }
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------ UMMA issuer
     if (lane == 0) {
-      int stage = 0;
-      uint32_t phase = 0;
+      Ring g{0, 0u, S};
       int acc = 0;
       uint32_t acc_phase = 0;
       bool ok = true;
@@ -190,25 +205,22 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
         ptx::tc_fence_after_sync();
         const uint32_t d_tmem = tmem_base + static_cast<uint32_t>(acc * BN);
         for (int kb = 0; kb < num_kb; ++kb) {
-          if (!ptx::bounded_mbar_wait(&full_bar[stage], phase, abort_flag)) {
+          if (!ptx::bounded_mbar_wait(&full_bar[g.stage], g.phase, abort_flag)) {
             if (p.status) atomicCAS(p.status, 0, kStatusTimeoutMma);
             ok = false;
             break;
           }
           ptx::tc_fence_after_sync();
-          const uint32_t a_base = ptx::smem_u32(smem_a + stage * a_stage);
-          const uint32_t b_base = ptx::smem_u32(smem_b + stage * Cfg::kBBytes);
+          const uint32_t a_base = ptx::smem_u32(smem_a + g.stage * a_stage);
+          const uint32_t b_base = ptx::smem_u32(smem_b + g.stage * Cfg::kBBytes);
 #pragma unroll
           for (int k = 0; k < kGgK / 16; ++k) {
             const uint64_t adesc = ptx::make_smem_desc(a_base + k * 32, 16, 1024, ptx::kLayoutSw128);
             const uint64_t bdesc = ptx::make_smem_desc(b_base + k * 2048, 8192, 1024, ptx::kLayoutSw128);
             ptx::umma_f16_ss(d_tmem, adesc, bdesc, kIdesc, (kb | k) != 0 ? 1u : 0u);
           }
-          ptx::umma_commit(&empty_bar[stage]);
-          if (++stage == S) {
-            stage = 0;
-            phase ^= 1u;
-          }
+          ptx::umma_commit(&empty_bar[g.stage]);
+          g.next();
         }
         if (!ok) break;
         ptx::umma_commit(&tfull_bar[acc]);
@@ -216,6 +228,58 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
         if (acc == 0) acc_phase ^= 1u;
       }
     }
+  } else if (FETCH == kGgCopy && warp >= 6) {
+    // ------------------------------------------------------------ copying warps: eight lanes per row of 128 bytes
+    const int tid = threadIdx.x - kGgThreads, chunk = tid & 7, r0 = tid >> 3;
+    constexpr int kPasses = kGgRows * 8 / kGgCopyThreads, kStep = kGgCopyThreads / 8;
+    constexpr int kAhead = Cfg::stages(kGgRows) - 2;  // stages in flight behind the one being requested
+    Ring g{0, 0u, S};
+    int behind = 0, signal = 0;  // stages requested but not signalled yet, the next of them
+    bool ok = true;
+    auto done = [&]() {  // the oldest stage's pieces have landed: hand them to the tensor core's proxy
+      ptx::fence_proxy_async_smem();
+      ptx::mbar_arrive(&full_bar[signal]);
+      if (++signal == S) signal = 0;
+      --behind;
+    };
+    for (int w = blockIdx.x; w < items && ok; w += gridDim.x) {
+      const GgItem it = gg_item(p, w, num_tiles);
+      const int num_kb = (it.t.K + kGgK - 1) / kGgK;
+      const T* row[kPasses];
+#pragma unroll
+      for (int j = 0; j < kPasses; ++j) {
+        const int r = r0 + j * kStep;
+        int i = r < it.t.rows ? p.g.src[it.t.row0 + r] : -1;
+        if (i >= p.src_rows || (i < 0 && r < it.t.rows)) {
+          if (p.status) atomicCAS(p.status, 0, kStatusBadIndex);
+          i = -1;
+        }
+        row[j] = i < 0 ? nullptr : reinterpret_cast<const T*>(p.g.A) + static_cast<int64_t>(i) * p.g.lda + chunk * 8;
+      }
+      for (int kb = 0; kb < num_kb; ++kb) {
+        if (!ptx::bounded_mbar_wait(&empty_bar[g.stage], g.phase ^ 1u, abort_flag)) {
+          if (p.status && tid == 0) atomicCAS(p.status, 0, kStatusTimeoutProducer);
+          ok = false;
+          break;
+        }
+        const uint32_t sa = ptx::smem_u32(smem_a + g.stage * a_stage);
+        const bool inside = kb * kGgK + chunk * 8 < it.t.K;  // beyond K: zeros
+#pragma unroll
+        for (int j = 0; j < kPasses; ++j) {
+          const int r = r0 + j * kStep;
+          if (row[j] != nullptr)
+            ptx::cp_async_16(sa + r * 128 + ((chunk ^ (r & 7)) << 4), inside ? row[j] + kb * kGgK : row[j], inside ? 16u : 0u);
+        }
+        ptx::cp_async_commit();
+        g.next();
+        if (++behind > kAhead) {
+          ptx::cp_async_wait<kAhead>();
+          done();
+        }
+      }
+    }
+    ptx::cp_async_wait<0>();
+    while (behind > 0) done();
   } else {
     // ------------------------------------------------------------ epilogue warps
     const int q = warp & 3;  // TMEM lane quarter this warp may read
@@ -248,7 +312,7 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
               if (c + 8 * j < cols) {
                 float x[8];
 #pragma unroll
-                for (int i = 0; i < 8; ++i) x[i] = grouped_act(ACT, __uint_as_float(v[8 * j + i]), f);
+                for (int i = 0; i < 8; ++i) x[i] = grouped_act(p.g.act, __uint_as_float(v[8 * j + i]), f);
                 *reinterpret_cast<uint4*>(dst + c + 8 * j) = pack8<T>(x);
               }
             }
@@ -270,14 +334,14 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
   }
 }
 
-template <typename T, int BN, int ACT, bool GATHER>
+template <typename T, int BN, int FETCH>
 static int launch_grouped(const CUtensorMap& ta, const CUtensorMap& tas, const CUtensorMap& tb, const CUtensorMap& tbs,
                           const GroupedTcParams& p, int grid, cudaStream_t stream) {
-  auto kern = gemm_grouped_kernel<T, BN, ACT, GATHER>;
+  auto kern = gemm_grouped_kernel<T, BN, FETCH>;
   static PerDeviceOnce once;
   cudaError_t e = once.run([&] { return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, GgCfg<BN>::kSmemBytes); });
   if (e != cudaSuccess) return (int)e;
-  return (int)launch_pdl(kern, dim3(grid), dim3(kGgThreads), GgCfg<BN>::kSmemBytes, stream, ta, tas, tb, tbs, p);
+  return (int)launch_pdl(kern, dim3(grid), dim3(FETCH == kGgCopy ? kGgThreads + kGgCopyThreads : kGgThreads), GgCfg<BN>::kSmemBytes, stream, ta, tas, tb, tbs, p);
 }
 
 }  // namespace blitz
@@ -285,15 +349,16 @@ static int launch_grouped(const CUtensorMap& ta, const CUtensorMap& tas, const C
 extern "C" {
 using namespace blitz;
 
-// A [a_rows][lda]; src: row of A behind each sorted row (null: the sorted row itself).  B: the experts' matrices [K][N]
+// A [a_rows][lda]; src: row of A behind each sorted row (null: the sorted row itself); those of the shared expert are rows
+// 0 .. shared_rows - 1.  B: the experts' matrices [K][N]
 // stacked along K; B_shared [K_shared][N_shared] or null.  C [sorted rows][ldc].  factors: per sorted row (before, after), or
-// null.  tiles / num_tiles / max_tiles: work list with tile_rows 128; max_rows: most rows any tile can have (for the height of
-// a stage).  act: 0 none, 1 square of relu.  dtype 0 fp16, 1 bf16.  bn_hint: 0 = choose, else 64 / 128 / 256.  N, K, pitches:
-// multiples of 8.  Expert's K rows are read up to the next multiple of 64: what lies behind them meets zero columns of A.
+// null.  tiles / num_tiles / max_tiles: work list with tile_rows 128; typical_*: expected tiles and rows of a tile,
+// max_rows: most rows any tile can have (all three for the launch's shape only).  act: 0 none, 1 square of relu.  dtype 0 fp16, 1 bf16.  bn_hint: 0 = choose, else 64 / 128 / 256.  fetch_hint: 0 = choose
+// how rows are gathered, 1 TMA, 2 copying warps.  N, K, pitches: multiples of 8.  Expert's K rows are read up to the next multiple of 64: what lies behind them meets zero columns of A.
 int blitz_gemm_grouped(const void* A, int64_t lda, int a_rows, const int* src, const void* B, int experts, int N, int K,
                        const void* B_shared, int N_shared, int K_shared, void* C, int64_t ldc, const void* factors,
-                       const void* tiles, const int* num_tiles, int max_tiles, int typical_tiles, int shared_row0, int shared_rows,
-                       int max_rows, int act, int bn_hint, int* status, int dtype, cudaStream_t stream) {
+                       const void* tiles, const int* num_tiles, int max_tiles, int typical_tiles, int typical_rows, int shared_row0, int shared_rows,
+                       int max_rows, int act, int bn_hint, int fetch_hint, int* status, int dtype, cudaStream_t stream) {
   if (a_rows <= 0 || N <= 0 || K <= 0) return 0;
   if (((N | K | N_shared | K_shared) & 7) || (lda & 7) || (ldc & 7) || act < 0 || act > 1) return -1;
   if ((reinterpret_cast<uintptr_t>(C) & 15) != 0 || (reinterpret_cast<uintptr_t>(tiles) & 15) != 0) return -1;
@@ -302,27 +367,40 @@ int blitz_gemm_grouped(const void* A, int64_t lda, int a_rows, const int* src, c
   GroupedTcParams p;
   p.g = GroupedParams{A, B, B_shared, C, lda, ldc, N, K, N_shared, K_shared, src, reinterpret_cast<const float2*>(factors),
                       reinterpret_cast<const int4*>(tiles), num_tiles, shared_row0, B_shared ? shared_rows : 0, kGgRows, act};
-  p.a_rows = max_rows >= kGgRows ? kGgRows : (max_rows + kGgBox - 1) / kGgBox * kGgBox;
+  p.a_rows = max_rows >= kGgRows ? kGgRows : (max_rows + 31) / 32 * 32;
+  p.box = p.a_rows == kGgRows && typical_rows > 64 ? kGgRows : 32;
   p.src_rows = a_rows;
   p.status = status;
   p.sh_tiles = (p.g.shared_rows + kGgRows - 1) / kGgRows;
   int bn = bn_hint;
   if (bn != 64 && bn != 128 && bn != 256) {
-    // the widest tile that still gives every SM something to do
-    auto items = [&](int b) { return p.sh_tiles * ((N_shared + b - 1) / b) + typical_tiles * ((N + b - 1) / b); };
-    bn = items(256) >= 2 * sms ? 256 : items(128) >= sms ? 128 : 64;
+    // Rounds of items per SM times the cycles of a 64-deep step.  Full tiles are bound by the tensor pipe (a 128-row MMA of
+    // K = 16 takes 95 / 105 / 150 cycles at N = 64 / 128 / 256), tiles of few rows by what one SM can stream (50 GB/s).
+    const bool stream_bound = max_rows <= kGgRows;
+    int64_t best = INT64_MAX;
+    for (int b = 256; b >= 64; b /= 2) {
+      const int64_t items = (int64_t)p.sh_tiles * ((N_shared + b - 1) / b) + (int64_t)typical_tiles * ((N + b - 1) / b);
+      const int step = b == 64 ? 430 : b == 128 ? (stream_bound ? 630 : 480) : (stream_bound ? 1260 : 650);
+      const int64_t cost = (items + sms - 1) / sms * step;
+      if (cost < best) {
+        best = cost;
+        bn = b;
+      }
+    }
   }
   p.tn = (N + bn - 1) / bn;
   p.tn_shared = B_shared ? (N_shared + bn - 1) / bn : 0;
+  const bool copy = src && (fetch_hint ? fetch_hint == kGgCopy : max_rows > kGgGather4Rows);
+  if (copy) p.a_rows = kGgRows;
   CUtensorMap ta, tas, tb, tbs;
   if (src) {
     if (!get_tmap_2d(&ta, A, (uint64_t)K, (uint64_t)a_rows, (uint64_t)lda * 2, kGgK, 1)) return -2;
     tas = ta;
-    if (B_shared && K_shared != K && !get_tmap_2d(&tas, A, (uint64_t)K_shared, (uint64_t)a_rows, (uint64_t)lda * 2, kGgK, 1)) return -2;
+    if (B_shared && !get_tmap_2d(&tas, A, (uint64_t)K_shared, (uint64_t)a_rows, (uint64_t)lda * 2, kGgK, (uint32_t)p.box)) return -2;
   } else {
-    if (!get_tmap_2d(&ta, A, (uint64_t)K, (uint64_t)a_rows, (uint64_t)lda * 2, kGgK, kGgBox)) return -2;
+    if (!get_tmap_2d(&ta, A, (uint64_t)K, (uint64_t)a_rows, (uint64_t)lda * 2, kGgK, (uint32_t)p.box)) return -2;
     tas = ta;
-    if (B_shared && !get_tmap_2d(&tas, A, (uint64_t)K_shared, (uint64_t)a_rows, (uint64_t)lda * 2, kGgK, kGgBox)) return -2;
+    if (B_shared && !get_tmap_2d(&tas, A, (uint64_t)K_shared, (uint64_t)a_rows, (uint64_t)lda * 2, kGgK, (uint32_t)p.box)) return -2;
   }
   if (!get_tmap_2d(&tb, B, (uint64_t)N, (uint64_t)experts * K, (uint64_t)N * 2, 64, kGgK)) return -2;
   tbs = tb;
@@ -333,11 +411,9 @@ int blitz_gemm_grouped(const void* A, int64_t lda, int a_rows, const int* src, c
   auto go = [&](auto type, auto width) -> int {
     using T = decltype(type);
     constexpr int BN = decltype(width)::value;
-    if (act == kActReluSquared)
-      return src ? launch_grouped<T, BN, kActReluSquared, true>(ta, tas, tb, tbs, p, grid, stream)
-                 : launch_grouped<T, BN, kActReluSquared, false>(ta, tas, tb, tbs, p, grid, stream);
-    return src ? launch_grouped<T, BN, kActNone, true>(ta, tas, tb, tbs, p, grid, stream)
-               : launch_grouped<T, BN, kActNone, false>(ta, tas, tb, tbs, p, grid, stream);
+    if (src == nullptr) return launch_grouped<T, BN, kGgBoxes>(ta, tas, tb, tbs, p, grid, stream);
+    return copy ? launch_grouped<T, BN, kGgCopy>(ta, tas, tb, tbs, p, grid, stream)
+                : launch_grouped<T, BN, kGgGather4>(ta, tas, tb, tbs, p, grid, stream);
   };
   auto width = [&](auto type) -> int {
     if (bn == 256) return go(type, std::integral_constant<int, 256>{});

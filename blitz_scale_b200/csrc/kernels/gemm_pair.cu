@@ -602,6 +602,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                   if (row_ok) {
                     float* dst = reinterpret_cast<float*>(p.C) + static_cast<int64_t>(row) * p.ldc + n0 + c;
                     float old[4][8];
+                    const float inv = EPI == 6 ? 1.f / p.alpha : 0.f;
                     if (EPI == 5) {
 #pragma unroll
                       for (int jj = 0; jj < 4; ++jj)
@@ -614,7 +615,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
 #pragma unroll
                         for (int k = 0; k < 8; ++k)
                           o[k] = EPI == 5   ? old[jj][k] + p.alpha * gt[8 * jj + k]
-                                 : EPI == 6 ? p.alpha * tanhf(gt[8 * jj + k] / p.alpha)
+                                 : EPI == 6 ? p.alpha * ptx::tanh_ex2(gt[8 * jj + k] * inv)
                                             : gt[8 * jj + k];
                         ptx::st_global_v8(dst + 8 * jj, o);
                       }

@@ -158,6 +158,7 @@ __device__ __forceinline__ void store_chunk(const GemmParams& p, const float (&a
     if (!row_ok) return;
     float* dst = reinterpret_cast<float*>(p.C) + static_cast<int64_t>(row) * p.ldc + static_cast<int64_t>(group) * p.N + col0;
     float old[4][8];
+    const float inv = EPI == kEpiCapF32 ? 1.f / p.alpha : 0.f;
     if (EPI == kEpiAxpyF32) {
 #pragma unroll
       for (int j = 0; j < 4; ++j)
@@ -170,7 +171,7 @@ __device__ __forceinline__ void store_chunk(const GemmParams& p, const float (&a
 #pragma unroll
         for (int i = 0; i < 8; ++i)
           v[i] = EPI == kEpiAxpyF32  ? old[j][i] + p.alpha * acc[8 * j + i]
-                 : EPI == kEpiCapF32 ? p.alpha * tanhf(acc[8 * j + i] / p.alpha)
+                 : EPI == kEpiCapF32 ? p.alpha * ptx::tanh_ex2(acc[8 * j + i] * inv)
                                      : acc[8 * j + i];
         ptx::st_global_v8(dst + 8 * j, v);
       }

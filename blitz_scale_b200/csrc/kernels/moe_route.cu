@@ -9,8 +9,9 @@
 // the factors before and after the expert.  `place[t][k]` names the rows of token t.  The work list has one entry (expert,
 // first row, rows) per `tile_rows` rows of an expert.
 //
-// A warp picks a token's experts; the block that finishes last sorts the pairs by expert (counting sort; the order of an
-// expert's rows is not fixed, and nothing that is computed depends on it) and clears the counters for the next launch.
+// A warp picks a token's experts; the block that finishes last finds where every expert's rows begin and clears the counters
+// for the next launch.  The pairs are put into their rows (counting sort) by that block too, or, where they are many, by a
+// second kernel.  The order of an expert's rows is not fixed, and nothing that is computed depends on it.
 #include "launch.cuh"
 #include "ptx.cuh"
 #include "scalar.cuh"
@@ -18,13 +19,16 @@
 namespace blitz {
 
 constexpr int kMoeMaxExperts = 1024;
+constexpr int kMoeKeep = 4;           // keys a lane keeps in registers: up to 32 * kMoeKeep experts
+constexpr int kMoeSortPairs = 2048;   // more pairs than this go to the second kernel
+constexpr int kMoePlacePairs = 4;     // pairs per thread there
 
 struct MoeRouteParams {
   const float* z;        // [tokens][ld]
   int64_t ld;
-  int tokens, experts, top, shared, weight_on_input, renormalize, tile_rows, max_tiles;
+  int tokens, experts, top, shared, weight_on_input, renormalize, tile_rows, max_tiles, second;
   int2* pairs;           // [tokens * top] (expert, weight bits), scratch
-  int* counters;         // [experts + 1], zero between launches: rows per expert, finished blocks
+  int* counters;         // [2 experts + 1]: rows per expert and finished blocks (zero between launches), next free rows
   int* src;              // [rows] token of a sorted row
   float2* factors;       // [rows] (before, after) the expert
   int* place;            // [tokens][top + shared]
@@ -37,6 +41,19 @@ struct MoeRouteParams {
 __device__ __forceinline__ uint32_t order_key(float x) {
   const uint32_t u = __float_as_uint(x);
   return (u & 0x80000000u) ? ~u : (u | 0x80000000u);
+}
+
+__device__ __forceinline__ float key_value(uint32_t k) {
+  return __uint_as_float((k & 0x80000000u) ? k & 0x7fffffffu : ~k);
+}
+
+// Row r belongs to pair i (expert and weight in pr).
+__device__ __forceinline__ void place_pair(const MoeRouteParams& p, int i, int2 pr, int r) {
+  const int tok = i / p.top;
+  const float w = __int_as_float(pr.y);
+  p.src[r] = tok;
+  p.factors[r] = p.weight_on_input ? make_float2(w, 1.f) : make_float2(1.f, w);
+  p.place[tok * (p.top + p.shared) + (i - tok * p.top)] = r;
 }
 
 __global__ void __launch_bounds__(1024) moe_route_kernel(const MoeRouteParams p) {
@@ -57,15 +74,29 @@ __global__ void __launch_bounds__(1024) moe_route_kernel(const MoeRouteParams p)
   const int t = blockIdx.x * warps + warp;
   if (t < p.tokens) {
     const float* z = p.z + t * p.ld;
-    uint32_t* keys = s_keys + warp * E;
+    uint32_t* keys = s_keys + warp * E;  // only beyond what the registers hold
+    uint32_t kept[kMoeKeep];
+    const bool in_regs = E <= 32 * kMoeKeep;
     uint32_t best = 0;  // this lane's largest key (0: none left) and its expert
     int best_e = 0x7fffffff;
-    for (int e = lane; e < E; e += 32) {
-      const uint32_t k = max(order_key(z[e]), 1u);
-      keys[e] = k;
+    auto consider = [&](uint32_t k, int e) {
       if (k > best) {
         best = k;
         best_e = e;
+      }
+    };
+    if (in_regs) {
+#pragma unroll
+      for (int j = 0; j < kMoeKeep; ++j) {
+        const int e = lane + 32 * j;
+        kept[j] = e < E ? max(order_key(z[e]), 1u) : 0u;
+      }
+#pragma unroll
+      for (int j = 0; j < kMoeKeep; ++j) consider(kept[j], lane + 32 * j);
+    } else {
+      for (int e = lane; e < E; e += 32) {
+        keys[e] = max(order_key(z[e]), 1u);
+        consider(keys[e], e);
       }
     }
     float weight = 0.f, sum = 0.f;  // lane k < top keeps the k-th pair's weight (top <= 32), the sum is everyone's
@@ -73,23 +104,27 @@ __global__ void __launch_bounds__(1024) moe_route_kernel(const MoeRouteParams p)
     for (int k = 0; k < p.top; ++k) {
       const uint32_t mx = __reduce_max_sync(0xffffffffu, best);
       const int e = __reduce_min_sync(0xffffffffu, best == mx ? best_e : 0x7fffffff);
-      const float s = sigmoid_f(z[e]);
-      sum += s;
       if (lane == k) {
-        weight = s;
+        weight = key_value(mx);
         expert = e;
       }
       if ((e & 31) == lane) {  // the expert's owner looks for its next best
-        keys[e] = 0;
         best = 0;
         best_e = 0x7fffffff;
-        for (int j = lane; j < E; j += 32)
-          if (keys[j] > best) {
-            best = keys[j];
-            best_e = j;
+        if (in_regs) {
+#pragma unroll
+          for (int j = 0; j < kMoeKeep; ++j) {
+            if (lane + 32 * j == e) kept[j] = 0;
+            consider(kept[j], lane + 32 * j);
           }
+        } else {
+          keys[e] = 0;
+          for (int j = lane; j < E; j += 32) consider(keys[j], j);
+        }
       }
     }
+    weight = lane < p.top ? sigmoid_f(weight) : 0.f;
+    if (p.renormalize) sum = warp_sum(weight);
     if (lane < p.top) {
       if (p.renormalize) weight /= sum;
       p.pairs[t * p.top + lane] = make_int2(expert, __float_as_int(weight));
@@ -102,20 +137,23 @@ __global__ void __launch_bounds__(1024) moe_route_kernel(const MoeRouteParams p)
     }
   }
   __syncthreads();
-  for (int e = threadIdx.x; e < E; e += blockDim.x)
-    if (s_count[e]) atomicAdd(&p.counters[e], s_count[e]);
-  __threadfence();
-  __syncthreads();
-  if (threadIdx.x == 0) s_last = atomicAdd(&p.counters[E], 1) == static_cast<int>(gridDim.x) - 1;
-  __syncthreads();
-  if (!s_last) return;
-  __threadfence();
+  const bool alone = gridDim.x == 1;
+  if (!alone) {
+    for (int e = threadIdx.x; e < E; e += blockDim.x)
+      if (s_count[e]) atomicAdd(&p.counters[e], s_count[e]);
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) s_last = atomicAdd(&p.counters[E], 1) == static_cast<int>(gridDim.x) - 1;
+    __syncthreads();
+    if (!s_last) return;
+    __threadfence();
+  }
 
   // rows and tiles of every expert: exclusive sums over the experts
   int rows_before = 0, tiles_before = 0;
   for (int e0 = 0; e0 < E; e0 += blockDim.x) {
     const int e = e0 + threadIdx.x;
-    const int n = e < E ? __ldcg(&p.counters[e]) : 0;
+    const int n = e < E ? (alone ? s_count[e] : __ldcg(&p.counters[e])) : 0;
     const int nt = (n + p.tile_rows - 1) / p.tile_rows;
     int a = n, b = nt;
 #pragma unroll
@@ -165,7 +203,12 @@ __global__ void __launch_bounds__(1024) moe_route_kernel(const MoeRouteParams p)
     for (int i = lane; i * p.tile_rows < n; i += 32)
       if (t0 + i < p.max_tiles) p.tiles[t0 + i] = make_int4(e, r0 + i * p.tile_rows, min(p.tile_rows, n - i * p.tile_rows), 0);
   }
-  for (int e = threadIdx.x; e <= E; e += blockDim.x) p.counters[e] = 0;
+  if (!alone)
+    for (int e = threadIdx.x; e <= E; e += blockDim.x) p.counters[e] = 0;
+  if (p.second) {
+    for (int e = threadIdx.x; e < E; e += blockDim.x) p.counters[E + 1 + e] = s_cursor[e];
+    return;
+  }
   __syncthreads();
   constexpr int kAhead = 4;  // pairs a thread reads at once
   for (int i0 = threadIdx.x; i0 < pairs; i0 += kAhead * blockDim.x) {
@@ -178,14 +221,37 @@ __global__ void __launch_bounds__(1024) moe_route_kernel(const MoeRouteParams p)
 #pragma unroll
     for (int j = 0; j < kAhead; ++j) {
       const int i = i0 + j * blockDim.x;
-      if (i >= pairs) break;
-      const int r = atomicAdd(&s_cursor[pr[j].x], 1);
-      const int tok = i / p.top;
-      const float w = __int_as_float(pr[j].y);
-      p.src[r] = tok;
-      p.factors[r] = p.weight_on_input ? make_float2(w, 1.f) : make_float2(1.f, w);
-      p.place[tok * per + (i - tok * p.top)] = r;
+      if (i < pairs) place_pair(p, i, pr[j], atomicAdd(&s_cursor[pr[j].x], 1));
     }
+  }
+}
+
+// Many pairs: a block counts its share per expert, takes that many rows of each, and fills them.
+__global__ void __launch_bounds__(256) moe_place_kernel(const MoeRouteParams p) {
+  ptx::griddep_launch_dependents();
+  ptx::griddep_wait();
+  extern __shared__ int s_row[];  // [experts]: this block's pairs, then the next free row
+  const int E = p.experts, pairs = p.tokens * p.top, i0 = blockIdx.x * blockDim.x * kMoePlacePairs + threadIdx.x;
+  for (int e = threadIdx.x; e < E; e += blockDim.x) s_row[e] = 0;
+  __syncthreads();
+  int2 pr[kMoePlacePairs];
+  int nth[kMoePlacePairs];
+#pragma unroll
+  for (int j = 0; j < kMoePlacePairs; ++j) {
+    const int i = i0 + j * blockDim.x;
+    if (i < pairs) pr[j] = p.pairs[i];
+  }
+#pragma unroll
+  for (int j = 0; j < kMoePlacePairs; ++j)
+    if (i0 + j * static_cast<int>(blockDim.x) < pairs) nth[j] = atomicAdd(&s_row[pr[j].x], 1);
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += blockDim.x)
+    if (s_row[e]) s_row[e] = atomicAdd(&p.counters[E + 1 + e], s_row[e]);
+  __syncthreads();
+#pragma unroll
+  for (int j = 0; j < kMoePlacePairs; ++j) {
+    const int i = i0 + j * blockDim.x;
+    if (i < pairs) place_pair(p, i, pr[j], s_row[pr[j].x] + nth[j]);
   }
 }
 
@@ -195,7 +261,7 @@ extern "C" {
 using namespace blitz;
 
 // z [tokens][ld] fp32: router logits, the shared expert's in column `experts` (shared = 1).  Scratch: pairs (tokens * top
-// int2), counters (experts + 1 int32, zeroed once).  Results as described at the top of the file; rows = tokens * (top + shared).
+// int2), counters (2 experts + 1 int32, zeroed once).  Results as described at the top of the file; rows = tokens * (top + shared).
 int blitz_moe_route(const float* z, int64_t ld, int tokens, int experts, int top, int shared, int weight_on_input, int renormalize,
                     int tile_rows, int max_tiles, void* pairs, int* counters, int* src, void* factors, int* place, void* tiles,
                     int* num_tiles, int* status, cudaStream_t stream) {
@@ -203,12 +269,18 @@ int blitz_moe_route(const float* z, int64_t ld, int tokens, int experts, int top
   if (experts < 1 || experts > kMoeMaxExperts || top < 1 || top > experts || top > 32 || tile_rows < 1) return -1;
   int warps = 32;
   while (warps > 1 && warps * experts * 4 > 32768) warps >>= 1;
-  while (warps > 4 && (tokens + warps - 1) / warps < 16) warps >>= 1;  // small steps: tokens side by side on several SMs
+  // small steps: all of it in one block, or tokens side by side on several SMs
+  while (tokens > warps && warps > 4 && (tokens + warps - 1) / warps < 16) warps >>= 1;
   MoeRouteParams p{z, ld, tokens, experts, top, shared, weight_on_input, renormalize, tile_rows, max_tiles,
-                   reinterpret_cast<int2*>(pairs), counters, src, reinterpret_cast<float2*>(factors), place,
-                   reinterpret_cast<int4*>(tiles), num_tiles, status};
-  return (int)launch_pdl(moe_route_kernel, dim3((tokens + warps - 1) / warps), dim3(warps * 32),
-                         (size_t)(3 + warps) * experts * sizeof(int), stream, p);
+                   tokens * top > kMoeSortPairs, reinterpret_cast<int2*>(pairs), counters, src, reinterpret_cast<float2*>(factors),
+                   place, reinterpret_cast<int4*>(tiles), num_tiles, status};
+  cudaError_t e = launch_pdl(moe_route_kernel, dim3((tokens + warps - 1) / warps), dim3(warps * 32),
+                             (size_t)(3 + (experts > 32 * kMoeKeep ? warps : 0)) * experts * sizeof(int), stream, p);
+  if (e == cudaSuccess && p.second) {
+    const int per = 256 * kMoePlacePairs;
+    e = launch_pdl(moe_place_kernel, dim3((tokens * top + per - 1) / per), dim3(256), (size_t)experts * sizeof(int), stream, p);
+  }
+  return (int)e;
 }
 
 }  // extern "C"

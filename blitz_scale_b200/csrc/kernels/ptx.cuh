@@ -194,6 +194,16 @@ __device__ __forceinline__ void tma_store_wait() {
   asm volatile("cp.async.bulk.wait_group %0;" ::"n"(N) : "memory");
 }
 
+// 16-byte copy global -> shared by this thread (`bytes` 0: zeros are written instead).
+__device__ __forceinline__ void cp_async_16(uint32_t smem_dst, const void* src, uint32_t bytes) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_dst), "l"(src), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() {
+  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
+}
+
 // L2 eviction policies for the cache_hint operand.
 __device__ __forceinline__ uint64_t policy_evict_first() {
   uint64_t p;

@@ -27,29 +27,19 @@ struct RopeStoreParams {
   void *k_pool, *v_pool;  // row of token `off` of page n: n * page_rows + off
   const float2* freq;  // [rot_dims / 2] (high, low)
   float gain;
-  int q_heads, kv_heads, dim, vdim, rot_dims, interleaved, page_size, page_rows, max_pages, wide;
+  int q_heads, kv_heads, dim, vdim, rot_dims, interleaved, page_size, page_rows, max_pages;
   int* status;
 };
 
-template <typename T>
-__global__ void rope_store_kernel(const RopeStoreParams p) {
+enum RopeMode : int { kRopeAny = 0, kRopeWidePairs = 1, kRopeWideHalves = 2 };  // wide: eight elements per access
+
+template <typename T, int MODE>
+__global__ void __launch_bounds__(256, MODE == kRopeAny ? 5 : 4) rope_store_kernel(const RopeStoreParams p) {
   ptx::griddep_launch_dependents();
   ptx::griddep_wait();
   extern __shared__ float s_ang[];  // [rot_dims / 2] cos, [rot_dims / 2] sin
   const int t = blockIdx.x;
   const int half = p.rot_dims >> 1;
-  const float pos = static_cast<float>(p.pos[t]);
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    const float2 f = p.freq[i];
-    const float a = pos * f.x;
-    const float err = fmaf(pos, f.x, -a) + pos * f.y;
-    float sn, cs;
-    sincosf(a, &sn, &cs);
-    const float c_err = 1.f - 0.5f * err * err;  // cos and sin of the small angle `err`, to second order
-    s_ang[i] = (cs * c_err - err * sn) * p.gain;
-    s_ang[half + i] = (sn * c_err + err * cs) * p.gain;
-  }
-  __syncthreads();
   int s = p.k ? p.slot[t] : -1;
   if (s >= p.max_pages * p.page_size) {
     if (threadIdx.x == 0 && p.status) atomicCAS(p.status, 0, kStatusBadIndex);
@@ -64,7 +54,22 @@ __global__ void rope_store_kernel(const RopeStoreParams p) {
   const T* k = reinterpret_cast<const T*>(p.k) + t * p.row;
   const T *q_b = reinterpret_cast<const T*>(p.q_b), *k_b = reinterpret_cast<const T*>(p.k_b), *v_b = reinterpret_cast<const T*>(p.v_b);
   const int heads = p.q_heads + (s >= 0 ? p.kv_heads : 0);
-  if (p.wide) {
+  auto angles = [&]() {
+    const float pos = static_cast<float>(p.pos[t]);
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+      const float2 f = p.freq[i];
+      const float a = pos * f.x;
+      const float err = fmaf(pos, f.x, -a) + pos * f.y;
+      float sn, cs;
+      sincosf(a, &sn, &cs);
+      const float c_err = 1.f - 0.5f * err * err;  // cos and sin of the small angle `err`, to second order
+      s_ang[i] = (cs * c_err - err * sn) * p.gain;
+      s_ang[half + i] = (sn * c_err + err * cs) * p.gain;
+    }
+    __syncthreads();
+  };
+  if (MODE != kRopeWideHalves) angles();
+  if (MODE != kRopeAny) {
     auto load8 = [&](const T* src, const T* bias, int64_t at, float (&x)[8]) {
       ldf8<T>(src + at, x);
       if (bias) {
@@ -74,7 +79,7 @@ __global__ void rope_store_kernel(const RopeStoreParams p) {
         for (int j = 0; j < 8; ++j) x[j] += b[j];
       }
     };
-    if (p.interleaved) {
+    if (MODE == kRopeWidePairs) {
       // eight elements (four pairs) per access; dimensions that pass unchanged ride along
       const int vec = p.dim >> 3;
       for (int it = threadIdx.x; it < heads * vec; it += blockDim.x) {
@@ -96,39 +101,55 @@ __global__ void rope_store_kernel(const RopeStoreParams p) {
         if (!is_q && p.v == nullptr) stf8<T>(vdst + at, x);
       }
     } else {
-      // half-split heads: eight pairs per item, or eight dimensions that pass unchanged
+      // half-split heads: eight pairs per item, or eight dimensions that pass unchanged.  A thread's first item is requested
+      // before the angles are computed.
       const int turns = half >> 3, vec = turns + ((p.dim - p.rot_dims) >> 3);
-      for (int it = threadIdx.x; it < heads * vec; it += blockDim.x) {
-        const int head = it / vec, c = it - head * vec;
-        const bool is_q = head < p.q_heads;
-        if (is_q && c >= turns && !q_b) continue;
-        const int64_t base = static_cast<int64_t>(is_q ? head : head - p.q_heads) * p.dim;
-        const T *src = is_q ? q : k, *bias = is_q ? q_b : k_b;
-        T* dst = is_q ? q : kdst;
-        float u[8];
-        if (c >= turns) {
-          const int64_t at = base + p.rot_dims + (c - turns) * 8;
-          load8(src, bias, at, u);
-          stf8<T>(dst + at, u);
-          if (!is_q && p.v == nullptr) stf8<T>(vdst + at, u);
-          continue;
+      const int items = (p.q_heads + (p.k ? p.kv_heads : 0)) * vec;  // (known before the slot is)
+      struct Item {
+        int64_t base;
+        int c;
+        bool is_q, on;
+      };
+      auto item = [&](int it) {
+        Item m;
+        const int head = it / vec;
+        m.c = it - head * vec;
+        m.is_q = head < p.q_heads;
+        m.base = static_cast<int64_t>(m.is_q ? head : head - p.q_heads) * p.dim;
+        m.on = it < items && !(m.is_q && m.c >= turns && !q_b);
+        return m;
+      };
+      auto first = [&](const Item& m) { return m.base + (m.c < turns ? m.c * 8 : p.rot_dims + (m.c - turns) * 8); };
+      Item m = item(threadIdx.x);
+      float u[8], v[8];
+      auto request = [&]() {
+        if (!m.on) return;
+        load8(m.is_q ? q : k, m.is_q ? q_b : k_b, first(m), u);
+        if (m.c < turns) load8(m.is_q ? q : k, m.is_q ? q_b : k_b, first(m) + half, v);
+      };
+      request();
+      angles();
+      for (int it = threadIdx.x; it < items; it += blockDim.x) {
+        if (it != static_cast<int>(threadIdx.x)) {
+          m = item(it);
+          request();
         }
-        const int i0 = c * 8;
-        float v[8], ru[8], rv[8];
-        load8(src, bias, base + i0, u);
-        load8(src, bias, base + half + i0, v);
+        if (!m.on || (!m.is_q && s < 0)) continue;
+        T* dst = m.is_q ? q : kdst;
+        const int64_t at = first(m);
+        const bool both = !m.is_q && p.v == nullptr;  // values are the keys before rotation
+        if (both) stf8<T>(vdst + at, u);
+        if (m.c < turns) {
+          if (both) stf8<T>(vdst + at + half, v);
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          const float cs = s_ang[i0 + j], sn = s_ang[half + i0 + j];
-          ru[j] = u[j] * cs - v[j] * sn;
-          rv[j] = v[j] * cs + u[j] * sn;
+          for (int j = 0; j < 8; ++j) {
+            const float cs = s_ang[m.c * 8 + j], sn = s_ang[half + m.c * 8 + j], x = u[j];
+            u[j] = x * cs - v[j] * sn;
+            v[j] = v[j] * cs + x * sn;
+          }
+          stf8<T>(dst + at + half, v);
         }
-        stf8<T>(dst + base + i0, ru);
-        stf8<T>(dst + base + half + i0, rv);
-        if (!is_q && p.v == nullptr) {
-          stf8<T>(vdst + base + i0, u);
-          stf8<T>(vdst + base + half + i0, v);
-        }
+        stf8<T>(dst + at, u);
       }
     }
     if (p.v != nullptr && s >= 0) {
@@ -211,14 +232,21 @@ int blitz_rope_store(void* q, const void* k, const void* v, const void* q_b, con
   if (rot_dims < 0 || (rot_dims & 1) || rot_dims > dim || rot_dims > 4096 || (rot_dims > 0 && freq == nullptr)) return -1;
   if (k != nullptr && v == nullptr && vdim != dim) return -1;
   RopeStoreParams p{q, k, v, q_b, k_b, v_b, row, pos, slot, k_pool, v_pool, reinterpret_cast<const float2*>(freq), gain, q_heads,
-                    kv_heads, dim, vdim, rot_dims, interleaved, page_size, page_rows, max_pages, 0, status};
+                    kv_heads, dim, vdim, rot_dims, interleaved, page_size, page_rows, max_pages, status};
   const uintptr_t al = dtype == 2 ? 32 : 16;
-  p.wide = ((dim | vdim | row) & 7) == 0 && (interleaved || (rot_dims & 15) == 0);
+  bool wide = ((dim | vdim | row) & 7) == 0 && (interleaved || (rot_dims & 15) == 0);
   for (const void* x : {(const void*)q, k, v, q_b, k_b, v_b, (const void*)k_pool, (const void*)v_pool})
-    p.wide = p.wide && (reinterpret_cast<uintptr_t>(x) % al) == 0;
+    wide = wide && (reinterpret_cast<uintptr_t>(x) % al) == 0;
+  const dim3 grid(num_tokens), block(wide && (q_heads + kv_heads) * dim <= 2048 ? 128 : 256);
+  const size_t smem = (size_t)rot_dims * sizeof(float);
+  auto go = [&](auto type) {
+    using T = decltype(type);
+    if (!wide) return launch_pdl(rope_store_kernel<T, kRopeAny>, grid, block, smem, stream, p);
+    return interleaved ? launch_pdl(rope_store_kernel<T, kRopeWidePairs>, grid, block, smem, stream, p)
+                       : launch_pdl(rope_store_kernel<T, kRopeWideHalves>, grid, block, smem, stream, p);
+  };
   cudaError_t e = cudaSuccess;
-  BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(rope_store_kernel<T>, dim3(num_tokens), dim3(p.wide && (q_heads + kv_heads) * dim <= 2048 ? 128 : 256),
-                                               (size_t)rot_dims * sizeof(float), stream, p)));
+  BLITZ_DISPATCH_DTYPE3(dtype, (e = go(T{})));
   return (int)e;
 }
 

@@ -31,7 +31,7 @@ struct StreamNormParams {
 
 constexpr int kSnKeep = 8;  // float4 groups a thread keeps
 
-template <typename T, int VEC>
+template <typename T, int VEC, bool ADD>
 __global__ void stream_norm_kernel(const StreamNormParams p) {
   ptx::griddep_launch_dependents();
   ptx::griddep_wait();
@@ -40,7 +40,7 @@ __global__ void stream_norm_kernel(const StreamNormParams p) {
   const int src = p.rows ? p.rows[t] + p.row_offset : t;
   float* xr = p.x + static_cast<int64_t>(src) * p.hidden;
   const T* step = reinterpret_cast<const T*>(p.step);
-  const bool change = p.init || p.add_embed || step != nullptr || p.n_add > 0;
+  const bool change = p.init || p.add_embed || step != nullptr || ADD;
   const T* er = nullptr;
   if (p.init || p.add_embed) {
     const int id = p.ids[t];
@@ -64,7 +64,8 @@ __global__ void stream_norm_kernel(const StreamNormParams p) {
     float4 a = p.init ? make_float4(0.f, 0.f, 0.f, 0.f) : load(xr + i * VEC);
     if (er) add(a, er + i * VEC);
     if (step) add(a, step + i * VEC);
-    for (int k = 0; k < p.n_add; ++k) add(a, reinterpret_cast<const T*>(p.add) + static_cast<int64_t>(add_row[k]) * p.hidden + i * VEC);
+    if (ADD)
+      for (int k = 0; k < p.n_add; ++k) add(a, reinterpret_cast<const T*>(p.add) + static_cast<int64_t>(add_row[k]) * p.hidden + i * VEC);
     if (change) {
       if (VEC == 4) *reinterpret_cast<float4*>(xr + i * VEC) = a;
       else xr[i] = a.x;
@@ -122,12 +123,14 @@ int blitz_stream_norm(const int32_t* ids, const void* embed, const void* step, c
   const int n = (hidden & 3) ? hidden : hidden / 4;
   int threads = 32;
   while (threads < n && threads < (n > 1024 ? 512 : 256)) threads <<= 1;
+  auto go = [&](auto type, auto vec) {
+    using T = decltype(type);
+    constexpr int V = decltype(vec)::value;
+    return n_add > 0 ? launch_pdl(stream_norm_kernel<T, V, true>, dim3(num_tokens), dim3(threads), 0, stream, p)
+                     : launch_pdl(stream_norm_kernel<T, V, false>, dim3(num_tokens), dim3(threads), 0, stream, p);
+  };
   cudaError_t e = cudaSuccess;
-  if (hidden & 3) {
-    BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(stream_norm_kernel<T, 1>, dim3(num_tokens), dim3(threads), 0, stream, p)));
-  } else {
-    BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(stream_norm_kernel<T, 4>, dim3(num_tokens), dim3(threads), 0, stream, p)));
-  }
+  BLITZ_DISPATCH_DTYPE3(dtype, (e = (hidden & 3) ? go(T{}, std::integral_constant<int, 1>{}) : go(T{}, std::integral_constant<int, 4>{})));
   return (int)e;
 }
 

@@ -146,7 +146,9 @@ class HybridRunner:
         T, H = h.shape
         plan = self._plans[self._plan_key(e)]
         z = self._router[:T * e.router_cols].view(T, e.router_cols)
-        ops.gemm(h, self._w(l, "router"), out=z, static_b=True)
+        # few columns: beyond a decode batch, narrow tiles with K split keep more SMs loading
+        narrow = dict(bn=64, split_k=4 if T <= 2048 else 1) if T > ops.DECODE_GEMM_MAX_M else {}
+        ops.gemm(h, self._w(l, "router"), out=z, static_b=True, **narrow)
         up, down = self._w(l, "up").view(e.experts, H, e.ff_pad), self._w(l, "down").view(e.experts, e.ff_pad, H)
         s_up, s_down = (self._w(l, "shared_up"), self._w(l, "shared_down")) if e.shared_ff else (None, None)
         tc = ops.grouped_tensor_core(h, up, down, s_up, s_down)

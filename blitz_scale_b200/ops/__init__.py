@@ -483,7 +483,7 @@ class ExpertPlan:
         i32 = lambda *shape: torch.zeros(*shape, dtype=torch.int32, device=device)
         self.experts, self.top, self.shared, self.max_tokens = experts, top, int(shared), max_tokens
         rows = max_tokens * (top + self.shared)
-        self.pairs, self.counters, self.num_tiles = i32(max_tokens * top, 2), i32(experts + 1), i32(1)
+        self.pairs, self.counters, self.num_tiles = i32(max_tokens * top, 2), i32(2 * experts + 1), i32(1)
         self.src, self.factors = i32(rows), torch.zeros(rows, 2, dtype=torch.float32, device=device)
         self._place, self._tiles = i32(rows), i32(self.tiles_at_most(max_tokens, 64), 4)
         self.tokens, self.tile_rows = 0, 128
@@ -500,9 +500,11 @@ class ExpertPlan:
     def place(self) -> torch.Tensor:
         return self._place[:self.rows].view(self.tokens, self.top + self.shared)
 
-    def tiles_usually(self) -> int:
+    def tiles_usually(self):
+        """(tiles, rows of one) of an even spread over the experts."""
         pairs = self.tokens * self.top
-        return max(1, round(self.experts * (1.0 - (1.0 - 1.0 / self.experts) ** pairs)) + pairs // self.tile_rows)
+        used = max(1, round(self.experts * (1.0 - (1.0 - 1.0 / self.experts) ** pairs)))
+        return used + max(0, pairs - used * self.tile_rows // 2) // self.tile_rows, min(self.tile_rows, -(-pairs // used))
 
 
 def moe_route(logits: torch.Tensor, plan: ExpertPlan, *, weight_on_input: bool = True, renormalize: bool = False,
@@ -529,10 +531,11 @@ def grouped_tensor_core(a: torch.Tensor, *matrices: Optional[torch.Tensor]) -> b
 
 
 def gemm_grouped(a: torch.Tensor, b: torch.Tensor, plan: ExpertPlan, out: torch.Tensor, *, shared: Optional[torch.Tensor] = None,
-                 gather: bool = False, act: str = "none", factors: bool = False, bn: int = 0) -> torch.Tensor:
+                 gather: bool = False, act: str = "none", factors: bool = False, bn: int = 0, fetch: int = 0) -> torch.Tensor:
     """out[r] = after_r * act(before_r * (a[row] @ b[expert of r])) for the plan's sorted rows r; ``b`` [experts, K, N];
     ``shared`` [K', N']: the shared expert's matrix for the rows behind (K' and N' columns of a and out).  ``gather``: row r
-    reads the activation of its token, else sorted row r.  ``factors``: apply the plan's factors (else both are 1)."""
+    reads the activation of its token, else sorted row r.  ``factors``: apply the plan's factors (else both are 1).  ``bn``
+    forces the tile width, ``fetch`` how rows are gathered (1 TMA, 2 copying warps)."""
     E, K, N = b.shape
     assert E == plan.experts and b.is_contiguous() and a.stride(1) == 1 and out.stride(1) == 1 and a.dtype == b.dtype == out.dtype
     assert (shared is not None) == bool(plan.shared) and out.shape[0] >= plan.rows
@@ -549,7 +552,7 @@ def gemm_grouped(a: torch.Tensor, b: torch.Tensor, plan: ExpertPlan, out: torch.
     assert plan.tile_rows == 128 and grouped_tensor_core(a, b, shared) and out.stride(0) % 8 == 0
     _check(lib().blitz_gemm_grouped(_p(a), a.stride(0), plan.tokens if gather else plan.rows, _p(src), _p(b), E, N, K, _p(shared), Ns,
                                     Ks, _p(out), out.stride(0), _p(fac), _p(plan._tiles), _p(plan.num_tiles), most,
-                                    plan.tiles_usually(), row0, shared_rows, plan.tokens, _ACT[act], bn,
+                                    *plan.tiles_usually(), row0, shared_rows, plan.tokens, _ACT[act], bn, fetch,
                                     _p(status_word(a.device)), _dt(a), _stream()), "blitz_gemm_grouped")
     return out
 

@@ -100,7 +100,7 @@ def _declare(L: ctypes.CDLL) -> None:
                               c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_p, c_i, c_p])
     sig("blitz_moe_route", [c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p])
     sig("blitz_gemm_grouped", [c_p, c_i64, c_i, c_p, c_p, c_i, c_i, c_i, c_p, c_i, c_i, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i, c_i,
-                               c_i, c_i, c_i, c_p, c_i, c_p])
+                               c_i, c_i, c_i, c_i, c_i, c_p, c_i, c_p])
     sig("blitz_gemm_grouped_simt", [c_p, c_i64, c_p, c_p, c_i, c_i, c_p, c_i, c_i, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i,
                                     c_p])
     sig("blitz_gla_recurrent", [c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_i, c_i,

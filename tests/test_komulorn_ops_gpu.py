@@ -204,7 +204,7 @@ def _experts(T, E, top, H, ff, sff, dt, seed, skew=0.0):
     return h, w, z
 
 
-def _run_experts(ops, h, w, z, E, top, sff, plan, bn=0, tile_rows=128, **how):
+def _run_experts(ops, h, w, z, E, top, sff, plan, bn=0, tile_rows=128, fetch=0, **how):
     dev = lambda n: torch.stack([w[f"e{e}.{n}"].T.contiguous() for e in range(E)]).to(DEV)
     up, down = dev("up"), dev("down")
     s_up, s_down = (w[f"shared.{n}"].T.contiguous().to(DEV) if sff else None for n in ("up", "down"))
@@ -212,7 +212,7 @@ def _run_experts(ops, h, w, z, E, top, sff, plan, bn=0, tile_rows=128, **how):
     ops.moe_route(z.to(DEV), plan, tile_rows=tile_rows, **how)
     act = torch.full((plan.rows, max(up.shape[2], sff)), math.nan, dtype=h.dtype, device=DEV)      # nothing unwritten may be read
     y = torch.full((plan.rows, H), math.nan, dtype=h.dtype, device=DEV)
-    ops.gemm_grouped(h.to(DEV), up, plan, act, shared=s_up, gather=True, act="relu2", factors=True, bn=bn)
+    ops.gemm_grouped(h.to(DEV), up, plan, act, shared=s_up, gather=True, act="relu2", factors=True, bn=bn, fetch=fetch)
     ops.gemm_grouped(act, down, plan, y, shared=s_down, bn=bn)
     x = torch.ones(T, H, device=DEV)
     out = torch.empty(T, H, dtype=h.dtype, device=DEV)
@@ -246,8 +246,9 @@ def test_experts_on_the_tensor_cores(ops, T, E, top, H, ff, sff, skew, dt):
     h, w, z = _experts(T, E, top, H, ff, sff, dt, T + E, skew)
     want = _want_experts(h, w, z, E, top, sff)
     plan = ops.ExpertPlan(300, E, top, bool(sff), DEV)
-    for bn in (0, 64, 128, 256):
-        assert _rel(_run_experts(ops, h, w, z, E, top, sff, plan, bn), want) < (8e-3 if dt == BF else 1e-3), bn
+    for bn, fetch in ((0, 0), (64, 1), (128, 1), (256, 1), (64, 2), (128, 2), (256, 2)):
+        got = _run_experts(ops, h, w, z, E, top, sff, plan, bn, fetch=fetch)
+        assert _rel(got, want) < (8e-3 if dt == BF else 1e-3), (bn, fetch)
 
 
 @pytest.mark.parametrize("T,E,top,H,ff,sff", [(1, 5, 2, 33, 21, 7), (130, 5, 3, 121, 51, 30), (90, 9, 1, 64, 72, 136), (200, 2, 2, 40, 10, 0)])
@@ -291,7 +292,7 @@ def test_router(ops, T, E, top, shared):
             assert torch.allclose(fac[T * top:T * per, 1], torch.sigmoid(z[:, E].double()), rtol=1e-6) and bool((fac[T * top:T * per, 0] == 1).all())
         want = [[e, int(begin[e]) + 128 * i, min(128, int(counts[e]) - 128 * i), 0] for e in range(E) for i in range(-(-int(counts[e]) // 128))]
         assert tiles == want
-        assert not plan.counters.any()
+        assert not plan.counters[:E + 1].any()
 
 
 @pytest.mark.parametrize("H", [7, 64, 250, 4096, 9000])
