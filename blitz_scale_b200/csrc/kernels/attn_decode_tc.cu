@@ -38,6 +38,9 @@
 // sigmoid) multiplies a head's output as it is stored.  More than 8 query heads per KV head run as several groups that
 // read the same keys and values (the second one from L2).
 //
+// A bias by distance per head, bias[h][min(i - j, bias_len - 1)], is added to the scaled scores; only chunks with a distance
+// inside the table look it up (four entries a lane, requested before the wait for the chunk).
+//
 // Replaces src/kernel/attention_decode.cu:13-40 and the host-side plan of
 // src/kernel/flashinfer_types.cu:52-80.
 #include "launch.cuh"
@@ -74,6 +77,8 @@ struct DecodeTcParams {
   int window, keep_first;       // 0: every key; else a token sees the last `window` positions and the first `keep_first`
   float cap_scale, cap_log2;    // soft cap (cap_log2 > 0): score in log2 units = cap_log2 * tanh(q.k * cap_scale)
   const void* sink;             // [q_heads] in the activation type, or null
+  const void* bias;             // [q_heads][bias_len] in the activation type, or null
+  int bias_len;
   int* status;
   long long* trace;  // profiling aid (null in production): clock stamps of CTA 0's first items, see blitz_attn_decode_set_trace
 };
@@ -294,7 +299,22 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
 #pragma unroll
       for (int i = 0; i < VD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
       float m = -INFINITY, l = 0.f;
+      const T* bias_row = nullptr;
+      float far_bias = 0.f;
+      if (!PLAIN && p.bias != nullptr && g < G) {
+        bias_row = reinterpret_cast<const T*>(p.bias) + static_cast<int64_t>(it.h * G + g) * p.bias_len;
+        far_bias = to_f<T>(bias_row[p.bias_len - 1]) * 1.4426950408889634f;
+      }
       for (int c = it.c_beg; c < it.c_end; ++c) {
+        float bias[4] = {far_bias, far_bias, far_bias, far_bias};  // of the lane's four keys, in log2 units
+        if (!PLAIN && bias_row != nullptr) {
+          const int d0 = it.seq_len - 1 - (it.chunk(c) * kTcChunk + tokw + 2 * t4);  // distance of the first of them
+          if (it.seq_len - 1 - (it.chunk(c) * kTcChunk + tokw + 15) < p.bias_len - 1) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+              bias[k] = to_f<T>(bias_row[min(max(d0 - (k & 1) - (k >> 1) * 8, 0), p.bias_len - 1)]) * 1.4426950408889634f;
+          }
+        }
         if (ok && !ptx::bounded_mbar_wait(&full_bar[stage], phase, abort_flag)) {
           if (p.status && lane == 0) atomicCAS(p.status, 0, kStatusTimeoutEpilogue);
           ok = false;
@@ -328,8 +348,8 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
           };
 #pragma unroll
           for (int k = 0; k < 2; ++k) {  // rows 8..15 of the fragments are padding
-            s_lo[k] = score(s_lo[k]);
-            s_hi[k] = score(s_hi[k]);
+            s_lo[k] = score(s_lo[k]) + (PLAIN ? 0.f : bias[k]);
+            s_hi[k] = score(s_hi[k]) + (PLAIN ? 0.f : bias[2 + k]);
           }
           float mx = -INFINITY;
           if (v0) mx = fmaxf(mx, s_lo[0]);
@@ -479,7 +499,7 @@ static int launch_tc(const CUtensorMap (&tm)[4], const DecodeTcParams& p, int ba
 
 template <typename T>
 static int launch_tc(const CUtensorMap (&tm)[4], const DecodeTcParams& p, int batch, cudaStream_t stream) {
-  const bool plain = p.dim == p.vdim && (p.dim == 64 || p.dim == 128) && p.v_rows > 0 && p.gate == nullptr && p.kv_div == 1;
+  const bool plain = p.dim == p.vdim && (p.dim == 64 || p.dim == 128) && p.v_rows > 0 && p.gate == nullptr && p.bias == nullptr && p.kv_div == 1;
   if (plain) return p.dim == 64 ? launch_tc<T, 64, 64, true>(tm, p, batch, stream) : launch_tc<T, 128, 128, true>(tm, p, batch, stream);
   if (p.dim > 64)
     return p.vdim > 64 ? launch_tc<T, 128, 128, false>(tm, p, batch, stream) : launch_tc<T, 128, 64, false>(tm, p, batch, stream);
@@ -511,14 +531,14 @@ int64_t blitz_attn_decode_workspace_bytes(int batch, int q_heads, int head_dim, 
 // blitz_attn_decode_workspace_bytes() bytes for value heads of vdim (may be null when num_splits == 1).
 // page_size must be a power of two >= 8 (pages smaller than 64 tokens are fetched as several boxes per stage).  dim and
 // vdim: multiples of 8 up to 128.  window (0 = none) / keep_first, softcap (0 = none), sink and gate (null = none) as
-// described at the top of the file.
+// described at the top of the file.  bias: [q_heads][bias_len] in the activation type, or null.
 int blitz_attn_decode(const void* q, int64_t q_stride, const void* k_pool, const void* v_pool, const int32_t* indices,
                       const int32_t* indptr, const int32_t* last_page_len, void* out, int64_t out_stride,
                       void* workspace, int batch, int q_heads, int kv_heads, int dim, int vdim, int page_size, int page_rows,
                       int max_pages, int num_splits, float sm_scale, int window, int keep_first, float softcap,
-                      const void* sink, const void* gate, int64_t gate_stride, int* status, int dtype, cudaStream_t stream) {
+                      const void* sink, const void* bias, int bias_len, const void* gate, int64_t gate_stride, int* status, int dtype, cudaStream_t stream) {
   if (batch <= 0) return 0;
-  if (window < 0 || keep_first < 0 || softcap < 0.f) return -1;
+  if (window < 0 || keep_first < 0 || softcap < 0.f || (bias != nullptr && bias_len < 1)) return -1;
   if (num_splits < 1 || kv_heads < 1 || (q_heads % kv_heads) != 0 || (q_stride & 1)) return -1;
   if (dim < 8 || dim > 128 || (dim & 7) || vdim < 8 || vdim > 128 || (vdim & 7)) return -1;
   if (page_size < 8 || (page_size & (page_size - 1)) != 0 || page_rows < page_size) return -1;
@@ -549,7 +569,7 @@ int blitz_attn_decode(const void* q, int64_t q_stride, const void* k_pool, const
   p.page_size = page_size; p.max_pages = max_pages; p.dim = dim; p.vdim = vdim; p.page_rows = page_rows; p.v_rows = one ? page_size : 0;
   p.num_splits = num_splits; p.box_tokens = bt; p.tail_box_tokens = bt_tail;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = g_tc_trace;
-  p.window = window; p.keep_first = keep_first; p.sink = sink; p.gate = gate; p.gate_stride = gate_stride;
+  p.window = window; p.keep_first = keep_first; p.sink = sink; p.bias = bias; p.bias_len = bias_len; p.gate = gate; p.gate_stride = gate_stride;
   p.cap_scale = softcap > 0.f ? sm_scale / softcap : 0.f; p.cap_log2 = softcap * 1.4426950408889634f;
   int rc = dtype == 1 ? launch_tc<__nv_bfloat16>(tm, p, batch, stream) : launch_tc<__half>(tm, p, batch, stream);
   if (rc != 0) return rc;
@@ -662,7 +682,7 @@ extern "C" int blitz_attn_decode_noalloc(const void* q, int64_t q_stride, const 
   p.max_pages = max_pages; p.num_splits = num_splits; p.box_tokens = bt; p.tail_box_tokens = bt_tail;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = nullptr;
   p.kv_div = 1; p.dim = p.vdim = head_dim; p.page_rows = 2 * page_size; p.v_rows = page_size; p.gate = nullptr; p.gate_stride = 0;
-  p.window = 0; p.keep_first = 0; p.sink = nullptr; p.cap_scale = p.cap_log2 = 0.f;
+  p.window = 0; p.keep_first = 0; p.sink = nullptr; p.bias = nullptr; p.bias_len = 0; p.cap_scale = p.cap_log2 = 0.f;
   int sms = 0;
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
   if (sms <= 0) sms = 148;

@@ -40,6 +40,11 @@
 // multiple of 8): TMA fills the columns behind a head's end with zeros.  A gate (one number per head and row, through a
 // sigmoid) multiplies a head's output rows as they leave tensor memory.
 //
+// A bias by distance per head (template parameter BIAS): bias[h][min(i - j, bias_len - 1)] is added to the scaled scores.  A
+// block of 128 keys against a tile of 128 rows has 255 distances; the tile's warpgroup fetches their biases (two a thread,
+// requested before it waits for the scores) into shared memory, where the lanes of a warp, rows that follow one another, read
+// neighbouring words.  Blocks whose every distance is beyond the table share its last entry, which moves the reference.
+//
 // Replaces FlashInfer's BatchPrefillWithRaggedKVCacheWrapper / paged wrapper calls and their host Plan()
 // (src/kernel/attention_prefill.cu:11-45, src/kernel/flashinfer_types.cu:24-49).
 #include "launch.cuh"
@@ -68,6 +73,8 @@ struct PagedPrefillParams {
   float small_max;            // EXT: largest |q.k| the polynomial takes (0: never)
   float poly[4];              // EXT: score in log2 units = x (poly[0] + poly[1] x^2 + poly[2] x^4 + poly[3] x^6), x = q.k
   const void* sink;           // EXT: [q_heads] in the activation type, or null
+  const void* bias;           // BIAS: [q_heads][bias_len] in the activation type
+  int bias_len;
   int* status;
   long long* trace;  // profiling aid (null in production): clock stamps of CTA 0's first item, see the set_trace call
 };
@@ -83,7 +90,9 @@ struct PpCfg {
   static constexpr int kSlabBytes = kPpTile * 128;     // 64 columns of a tile: 128 rows x 128 bytes
   static constexpr int kSlabs = HD / 64, kValueSlabs = VD / 64;
   static constexpr int kTileBytes = kSlabs * kSlabBytes, kValueBytes = kValueSlabs * kSlabBytes;  // a Q or K tile, a V tile
-  static constexpr int kSmemBytes = 4 * kTileBytes + 2 * kValueBytes + 1024 + 256;  // Q x 2 tiles, K x 2 stages, V x 2 stages
+  static constexpr int kBarBytes = 256;
+  static constexpr int kBiasFloats = 2 * 2 * 256;  // per tile: two blocks' distances
+  static constexpr int kSmemBytes = 4 * kTileBytes + 2 * kValueBytes + 1024 + kBarBytes;  // Q x 2 tiles, K x 2 stages, V x 2 stages
 };
 
 struct PpItem {
@@ -130,7 +139,7 @@ __device__ __forceinline__ int pp_index(int r, int total) {
   return idx < total ? idx : -1;
 }
 
-template <typename T, int HD, int VD, bool POLY, bool EXT>
+template <typename T, int HD, int VD, bool POLY, bool EXT, bool BIAS>
 __global__ void __launch_bounds__(kPpThreads, 1)
 attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                           const __grid_constant__ CUtensorMap tmap_v, const PagedPrefillParams p) {
@@ -159,6 +168,7 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   uint64_t* o_free = bars + 16;   // [2] per tile and item: the warpgroup has read its output rows
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 18);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  float* s_bias = reinterpret_cast<float*>(sV + 2 * VB + C::kBarBytes);  // BIAS only
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int total = p.entries * p.q_heads;
@@ -355,8 +365,19 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       const int q_idx = it.q0 + t * kPpTile + r_;  // row within the chunk
       const int limit = it.prefix + q_idx;         // last key position this row may see
       float m_ref = 0.f, l = 0.f;
+      const T* bias_row = BIAS ? reinterpret_cast<const T*>(p.bias) + static_cast<int64_t>(it.head) * p.bias_len : nullptr;
+      const float far_bias = BIAS ? to_f<T>(bias_row[p.bias_len - 1]) * 1.4426950408889634f : 0.f;
       for (int j = 0; j < my_blocks; ++j) {
         pp_trace(p, tracer, t, j, 0);
+        // the block's smallest distance; is any of them inside the table?
+        const int nearest = it.prefix + it.q0 + t * kPpTile - (it.block(j) * kPpTile + kPpTile - 1);
+        const bool near = BIAS && nearest < p.bias_len - 1;
+        float bias_pair[2];
+        if (near) {
+#pragma unroll
+          for (int k = 0; k < 2; ++k)
+            bias_pair[k] = to_f<T>(bias_row[min(max(nearest + r_ + k * kPpTile, 0), p.bias_len - 1)]) * 1.4426950408889634f;
+        }
         if (!ptx::bounded_mbar_wait(&s_full[t], (cnt + j) & 1, abort_flag)) {
           ok = false;
           break;
@@ -382,6 +403,21 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
           return kv0 + i <= limit && (!EXT || kv0 + i >= from || kv0 + i < p.keep_first);
         };
         const bool capped = EXT && p.cap_log2 > 0.f;
+        float bias = 0.f;  // of every score of the block, in log2 units
+        if (near) {
+          float* sb = s_bias + (t * 2 + (j & 1)) * 256;  // (the buffer of two blocks ago: every warp has passed the last barrier)
+          sb[r_] = bias_pair[0];
+          sb[r_ + kPpTile] = bias_pair[1];
+          if (t == 0) asm volatile("bar.sync 1, 128;" ::: "memory");
+          else asm volatile("bar.sync 2, 128;" ::: "memory");
+          // distance of key i to this row: nearest + r_ + 127 - i
+#pragma unroll
+          for (int i = 0; i < kPpTile; ++i)
+            score(i) = __float_as_uint(fmaf(__uint_as_float(score(i)), p.scale_log2, sb[r_ + kPpTile - 1 - i]));
+        } else if (BIAS) {
+          bias = far_bias;
+        }
+        const float score_scale = near ? 1.f : p.scale_log2;
         // largest of the row's 128 scores, or of their magnitudes: eight independent chains of three-input maxima (with two
         // softmax warps per scheduler nothing else hides a serial one)
         auto largest = [&](auto&& max3) {
@@ -414,7 +450,7 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
           }
           mx = largest([](float a, float b, float c) { return ptx::fmax3(a, b, c); });
           if (capped) mx = mx == -INFINITY ? mx : p.cap_log2 * ptx::tanh_ex2(mx * p.cap_scale);
-          else mx *= p.scale_log2;
+          else mx = BIAS ? fmaf(mx, score_scale, bias) : mx * p.scale_log2;
         }
         // (S of this block was issued after P V of the previous one, so that product is complete: O_t is stable and
         // the columns P is about to overwrite have been read)
@@ -441,7 +477,7 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         pp_trace(p, tracer, t, j, 3);
         // probabilities (16 bit) -> tensor memory over the scores; row sum
         float rs[4] = {0.f, 0.f, 0.f, 0.f};
-        const float neg_m = (EXT && m_ref == -INFINITY) ? 0.f : -m_ref;
+        const float neg_m = ((EXT && m_ref == -INFINITY) ? 0.f : -m_ref) + (BIAS ? bias : 0.f);
         auto probabilities = [&](auto&& exponents) {  // exponents(c): those of scores c and c + 1
 #pragma unroll
           for (int h = 0; h < 2; ++h) {  // 64 scores -> 32 columns of pairs
@@ -483,8 +519,8 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
           probabilities([&](int c) { return make_float2(cap(__uint_as_float(score(c))), cap(__uint_as_float(score(c + 1)))); });
         } else {
           probabilities([&](int c) {
-            return make_float2(fmaf(__uint_as_float(score(c)), p.scale_log2, neg_m),
-                               fmaf(__uint_as_float(score(c + 1)), p.scale_log2, neg_m));
+            return make_float2(fmaf(__uint_as_float(score(c)), BIAS ? score_scale : p.scale_log2, neg_m),
+                               fmaf(__uint_as_float(score(c + 1)), BIAS ? score_scale : p.scale_log2, neg_m));
           });
         }
         pp_trace(p, tracer, t, j, 4);
@@ -538,15 +574,15 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   }
 }
 
-template <typename T, int HD, int VD, bool POLY, bool EXT>
+template <typename T, int HD, int VD, bool POLY, bool EXT, bool BIAS>
 static int launch_paged_prefill(const CUtensorMap (&tm)[3], const PagedPrefillParams& p, int grid, cudaStream_t stream) {
-  constexpr int kSmem = PpCfg<HD, VD>::kSmemBytes;
+  constexpr int kSmem = PpCfg<HD, VD>::kSmemBytes + (BIAS ? PpCfg<HD, VD>::kBiasFloats * 4 : 0);
   static PerDeviceOnce once;
   cudaError_t e = once.run([] {
-    return cudaFuncSetAttribute(attn_prefill_paged_kernel<T, HD, VD, POLY, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
+    return cudaFuncSetAttribute(attn_prefill_paged_kernel<T, HD, VD, POLY, EXT, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
   });
   if (e != cudaSuccess) return (int)e;
-  attn_prefill_paged_kernel<T, HD, VD, POLY, EXT><<<grid, kPpThreads, kSmem, stream>>>(tm[0], tm[1], tm[2], p);
+  attn_prefill_paged_kernel<T, HD, VD, POLY, EXT, BIAS><<<grid, kPpThreads, kSmem, stream>>>(tm[0], tm[1], tm[2], p);
   return (int)cudaGetLastError();
 }
 
@@ -570,12 +606,13 @@ void blitz_attn_prefill_paged_set_trace(long long* buf) { blitz::g_pp_trace = bu
 // index of its first page id, number of its pages, tokens cached for it (chunk included), which 256-row pair, 0, 0.
 // page_size: a power of two >= 8.  dim and vdim: multiples of 8 up to 128.  flags bit 0: compute a quarter of the
 // exponentials on the FMA pipe (not with a window, cap or sink).  window (0 = none) / keep_first, softcap (0 = none), sink
-// and gate (null = none): see the top of the file.
+// and gate (null = none): see the top of the file.  bias: [q_heads][bias_len] in the activation type, or null (not with a
+// window, cap or sink).
 int blitz_attn_prefill_paged(const void* q, int64_t q_stride, const void* k_pool, const void* v_pool, void* out, int64_t out_stride,
                              const int32_t* page_indices, const int32_t* work, int entries, int num_tokens,
                              int q_heads, int kv_heads, int dim, int vdim, int page_size, int page_rows, int max_pages,
                              float sm_scale, int flags, int window, int keep_first, float softcap, const void* sink,
-                             const void* gate, int64_t gate_stride, int* status, int dtype, cudaStream_t stream) {
+                             const void* bias, int bias_len, const void* gate, int64_t gate_stride, int* status, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0 || entries <= 0) return 0;
   if (dim < 8 || dim > 128 || (dim & 7) || vdim < 8 || vdim > 128 || (vdim & 7)) return -1;
   if (kv_heads < 1 || (q_heads % kv_heads) != 0 || (out_stride & 7) || (q_stride & 7)) return -1;
@@ -598,7 +635,7 @@ int blitz_attn_prefill_paged(const void* q, int64_t q_stride, const void* k_pool
   p.q_heads = q_heads; p.kv_heads = kv_heads; p.page_size = page_size; p.box_tokens = bt;
   p.oob_row = (int)rows;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = g_pp_trace;
-  p.window = window; p.keep_first = keep_first; p.sink = sink;
+  p.window = window; p.keep_first = keep_first; p.sink = sink; p.bias = bias; p.bias_len = bias_len;
   p.cap_scale = softcap > 0.f ? sm_scale / softcap : 0.f; p.cap_log2 = softcap * 1.4426950408889634f;
   // tanh(z) = z (k0 + k1 z^2 + k2 z^4 + k3 z^6) for |z| <= 0.5 (Chebyshev interpolation of tanh(z) / z in z^2, absolute
   // error 2.5e-7), with z = q.k * cap_scale folded in.  Scores below 40 log2 units keep every probability that refers to
@@ -611,19 +648,21 @@ int blitz_attn_prefill_paged(const void* q, int64_t q_stride, const void* k_pool
   const int sms = device_sm_count();
   const int grid = (int)(total < sms ? total : sms);
   const bool poly = (flags & 1) != 0, ext = window > 0 || softcap > 0.f || sink != nullptr;
-  auto sized = [&](auto type, auto poly_, auto ext_) {
+  if (bias != nullptr && (ext || bias_len < 1)) return -1;
+  auto sized = [&](auto type, auto poly_, auto ext_, auto bias_) {
     using T = decltype(type);
-    constexpr bool P = decltype(poly_)::value, X = decltype(ext_)::value;
+    constexpr bool P = decltype(poly_)::value, X = decltype(ext_)::value, B = decltype(bias_)::value;
     if (dim > 64)
-      return vdim > 64 ? launch_paged_prefill<T, 128, 128, P, X>(tm, p, grid, stream)
-                       : launch_paged_prefill<T, 128, 64, P, X>(tm, p, grid, stream);
-    return vdim > 64 ? launch_paged_prefill<T, 64, 128, P, X>(tm, p, grid, stream)
-                     : launch_paged_prefill<T, 64, 64, P, X>(tm, p, grid, stream);
+      return vdim > 64 ? launch_paged_prefill<T, 128, 128, P, X, B>(tm, p, grid, stream)
+                       : launch_paged_prefill<T, 128, 64, P, X, B>(tm, p, grid, stream);
+    return vdim > 64 ? launch_paged_prefill<T, 64, 128, P, X, B>(tm, p, grid, stream)
+                     : launch_paged_prefill<T, 64, 64, P, X, B>(tm, p, grid, stream);
   };
   auto launch = [&](auto type) {
-    if (ext) return sized(type, std::false_type{}, std::true_type{});
-    if (poly) return sized(type, std::true_type{}, std::false_type{});
-    return sized(type, std::false_type{}, std::false_type{});
+    if (bias != nullptr) return sized(type, std::false_type{}, std::false_type{}, std::true_type{});
+    if (ext) return sized(type, std::false_type{}, std::true_type{}, std::false_type{});
+    if (poly) return sized(type, std::true_type{}, std::false_type{}, std::false_type{});
+    return sized(type, std::false_type{}, std::false_type{}, std::false_type{});
   };
   return dtype == 1 ? launch(__nv_bfloat16{}) : launch(__half{});
 }

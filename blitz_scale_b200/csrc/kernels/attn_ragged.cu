@@ -3,10 +3,11 @@
 //
 //   visible(i, j) = j <= i and (i - j < window or j < keep_first)          window 0: everything
 //   score         = cap * tanh(scale * q.k / cap)                           cap 0: scale * q.k
+//   score        += bias[h][min(i - j, bias_len - 1)]                       no bias: nothing
 //   out           = sum_j e^score_j v_j / (e^sink + sum_j e^score_j)        no sink: the plain softmax
 //   out           = sigmoid(gate) * out                                     no gate: as it is
 //
-// Keys and values may differ in size.
+// Keys and values may differ in size, and values may be the first columns of the keys' rows (v_row: their pitch).
 // It serves the 32-bit mode and head sizes that the tensor-core kernels do not take.  A warp owns one (token, query
 // head): keys go over the lanes 32 at a time for the scores, head dimensions go over the lanes for the weighted sum.
 // Only the blocks of 32 keys with a visible key are read.  Everything is fp32.
@@ -31,6 +32,8 @@ struct RaggedAttnParams {
   const int32_t* page_indptr;  // [rows + 1]
   const int32_t* page_indices;
   const void* sink;
+  const void* bias;   // [q_heads][bias_len] by distance, the last entry for all longer ones; or null
+  int bias_len, v_row;
   int num_tokens, rows, q_heads, kv_heads, dim, vdim, page_size, page_rows, max_pages, window, keep_first;
   float scale, softcap;
   int* status;
@@ -58,9 +61,10 @@ __global__ void __launch_bounds__(kRgWarps * 32) attn_ragged_kernel(const Ragged
   for (int d = lane; d < D; d += 32) sq[d] = ldf<T>(q + d) * p.scale;
   __syncwarp();
   const int kvh = h / (p.q_heads / p.kv_heads);
-  const int64_t krow = static_cast<int64_t>(p.kv_heads) * D, vrow = static_cast<int64_t>(p.kv_heads) * DV;
+  const int64_t krow = static_cast<int64_t>(p.kv_heads) * D, vrow = static_cast<int64_t>(p.kv_heads) * p.v_row;
+  const T* bias = p.bias ? reinterpret_cast<const T*>(p.bias) + static_cast<int64_t>(h) * p.bias_len : nullptr;
   const T* k_pool = reinterpret_cast<const T*>(p.k_pool) + static_cast<int64_t>(kvh) * D;
-  const T* v_pool = reinterpret_cast<const T*>(p.v_pool) + static_cast<int64_t>(kvh) * DV;
+  const T* v_pool = reinterpret_cast<const T*>(p.v_pool) + static_cast<int64_t>(kvh) * p.v_row;
   // key j's row in the pools; -1 where the page table does not reach (reported)
   auto key_row = [&](int j) -> int {
     const int slot = j / p.page_size;
@@ -91,6 +95,7 @@ __global__ void __launch_bounds__(kRgWarps * 32) attn_ragged_kernel(const Ragged
       s = 0.f;
       for (int d = 0; d < D; ++d) s += sq[d] * ldf<T>(kr + d);
       if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+      if (bias) s += ldf<T>(bias + min(i - (n < first ? n : lo + n - first), p.bias_len - 1));
     }
     const float mx = fmaxf(m, warp_max(s));
     if (mx == -INFINITY) continue;
@@ -130,18 +135,20 @@ using namespace blitz;
 // q: [tokens, q_stride], rotated; k_pool, v_pool: [max_pages][page_rows][kv_heads][dim or vdim] (see rope_store.cu) with
 // every key up to a token's own position already stored; out: [tokens, out_stride].  Rows are the sequences of the step: tokens
 // tok_indptr[r] .. tok_indptr[r + 1] (null: one token per row), pages page_indices[page_indptr[r] ..].  A row without
-// pages gives zeros.  window 0 = unlimited; softcap 0 = none; sink may be null ([q_heads], activation type).
+// pages gives zeros.  window 0 = unlimited; softcap 0 = none; sink may be null ([q_heads], activation type).  v_row: elements
+// from a value head to the next one in a pool row (vdim, or dim where values are the first columns of the keys).  bias:
+// [q_heads][bias_len] in the activation type, by distance, or null.
 int blitz_attn_ragged(const void* q, int64_t q_stride, const void* k_pool, const void* v_pool, void* out, int64_t out_stride,
                       const int32_t* pos, const int32_t* tok_indptr, const int32_t* page_indptr,
-                      const int32_t* page_indices, const void* sink, const void* gate, int64_t gate_stride, int num_tokens,
+                      const int32_t* page_indices, const void* sink, const void* bias, int bias_len, int v_row, const void* gate, int64_t gate_stride, int num_tokens,
                       int rows, int q_heads, int kv_heads, int dim, int vdim, int page_size, int page_rows, int max_pages,
                       int window, int keep_first, float scale, float softcap, int* status, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0 || rows <= 0) return 0;
   if (dim <= 0 || vdim <= 0 || vdim > kRgMaxDim || dim > kRgMaxQueryDim || kv_heads <= 0 || q_heads % kv_heads != 0 || window < 0 ||
-      keep_first < 0)
+      keep_first < 0 || v_row < vdim || (bias && bias_len < 1))
     return -1;
   RaggedAttnParams p{q, k_pool, v_pool, gate, out, q_stride, out_stride, gate_stride, pos, tok_indptr, page_indptr, page_indices,
-                     sink, num_tokens, rows, q_heads, kv_heads, dim, vdim, page_size, page_rows, max_pages, window, keep_first,
+                     sink, bias, bias_len, v_row, num_tokens, rows, q_heads, kv_heads, dim, vdim, page_size, page_rows, max_pages, window, keep_first,
                      scale, softcap, status};
   const int64_t items = static_cast<int64_t>(num_tokens) * q_heads;
   const dim3 grid((unsigned)((items + kRgWarps - 1) / kRgWarps));

@@ -299,8 +299,27 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
       ptx::tc_fence_after_sync();
       if (q * 32 < it.t.rows) {
         const uint32_t taddr = tmem_base + (static_cast<uint32_t>(q * 32) << 16) + static_cast<uint32_t>(acc * BN);
-        T* dst = reinterpret_cast<T*>(p.g.C) + static_cast<int64_t>(row) * p.g.ldc + n0;
+        const bool gated = p.g.act == kActSiluGate;
+        T* dst = reinterpret_cast<T*>(p.g.C) + static_cast<int64_t>(row) * p.g.ldc + (gated ? n0 / 2 : n0);
         const int cols = min(BN, it.t.N - n0);
+        if (gated) {
+#pragma unroll 1
+          for (int c = 0; c < cols; c += 64) {
+            uint32_t v[32], u[32];
+            ptx::tmem_ld_32x32(taddr + c, v);
+            ptx::tmem_ld_32x32(taddr + c + 32, u);
+            ptx::tmem_ld_wait();
+            if (row_ok) {
+#pragma unroll
+              for (int j = 0; j < 4; ++j) {
+                float x[8];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) x[i] = grouped_silu_gate(__uint_as_float(v[8 * j + i]), __uint_as_float(u[8 * j + i]), f);
+                *reinterpret_cast<uint4*>(dst + c / 2 + 8 * j) = pack8<T>(x);
+              }
+            }
+          }
+        } else
 #pragma unroll 1
         for (int c = 0; c < cols; c += 32) {
           uint32_t v[32];
@@ -353,14 +372,16 @@ using namespace blitz;
 // 0 .. shared_rows - 1.  B: the experts' matrices [K][N]
 // stacked along K; B_shared [K_shared][N_shared] or null.  C [sorted rows][ldc].  factors: per sorted row (before, after), or
 // null.  tiles / num_tiles / max_tiles: work list with tile_rows 128; typical_*: expected tiles and rows of a tile,
-// max_rows: most rows any tile can have (all three for the launch's shape only).  act: 0 none, 1 square of relu.  dtype 0 fp16, 1 bf16.  bn_hint: 0 = choose, else 64 / 128 / 256.  fetch_hint: 0 = choose
+// max_rows: most rows any tile can have (all three for the launch's shape only).  act: 0 none, 1 square of relu, 2 silu(gate) * up
+// (grouped.cuh; N a multiple of 64, C has N / 2 columns; without a shared expert).  dtype 0 fp16, 1 bf16.  bn_hint: 0 = choose, else 64 / 128 / 256.  fetch_hint: 0 = choose
 // how rows are gathered, 1 TMA, 2 copying warps.  N, K, pitches: multiples of 8.  Expert's K rows are read up to the next multiple of 64: what lies behind them meets zero columns of A.
 int blitz_gemm_grouped(const void* A, int64_t lda, int a_rows, const int* src, const void* B, int experts, int N, int K,
                        const void* B_shared, int N_shared, int K_shared, void* C, int64_t ldc, const void* factors,
                        const void* tiles, const int* num_tiles, int max_tiles, int typical_tiles, int typical_rows, int shared_row0, int shared_rows,
                        int max_rows, int act, int bn_hint, int fetch_hint, int* status, int dtype, cudaStream_t stream) {
   if (a_rows <= 0 || N <= 0 || K <= 0) return 0;
-  if (((N | K | N_shared | K_shared) & 7) || (lda & 7) || (ldc & 7) || act < 0 || act > 1) return -1;
+  if (((N | K | N_shared | K_shared) & 7) || (lda & 7) || (ldc & 7) || act < 0 || act > 2) return -1;
+  if (act == kActSiluGate && ((N & 63) || B_shared)) return -1;
   if ((reinterpret_cast<uintptr_t>(C) & 15) != 0 || (reinterpret_cast<uintptr_t>(tiles) & 15) != 0) return -1;
   if (lda < K || (B_shared && lda < K_shared)) return -1;
   const int sms = device_sm_count();

@@ -5,7 +5,7 @@
 // Epilogues: store (as T or as fp32), C += alpha * acc on an fp32 C (residual stream), silu(gate) * up, soft-capped fp32
 // store (alpha * tanh(acc / alpha)).
 // groups > 1: block-diagonal product.  B holds `groups` blocks [K, N] stacked along K; group g multiplies the K
-// columns of A from g * K on and writes the N columns of C from g * N on.
+// columns of A from g * a_step on and writes the N columns of C from g * c_step on.
 //
 // The second kernel is the grouped product of a mixture of experts (see gemm_grouped.cu) in the same arithmetic.
 #include "launch.cuh"
@@ -22,7 +22,7 @@ struct SimtGemmParams {
   const void* B;
   void* C;
   int64_t lda, ldb, ldc;
-  int M, N, K, up_off;
+  int M, N, K, up_off, a_step, c_step;
   float alpha;
 };
 
@@ -37,7 +37,7 @@ __global__ void __launch_bounds__(kSgThreads) gemm_simt_kernel(const SimtGemmPar
   __shared__ float sB[H][kSgK][kSgT];
   const int m0 = blockIdx.y * kSgT, n0 = blockIdx.x * kSgT, g = blockIdx.z;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-  const T* A = reinterpret_cast<const T*>(p.A) + static_cast<int64_t>(g) * p.K;
+  const T* A = reinterpret_cast<const T*>(p.A) + static_cast<int64_t>(g) * p.a_step;
   const T* B = reinterpret_cast<const T*>(p.B) + static_cast<int64_t>(g) * p.K * p.ldb;
   float acc[H][4][4];
 #pragma unroll
@@ -82,7 +82,7 @@ __global__ void __launch_bounds__(kSgThreads) gemm_simt_kernel(const SimtGemmPar
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx + 16 * j;
       if (n >= p.N) continue;
-      const int64_t at = static_cast<int64_t>(m) * p.ldc + static_cast<int64_t>(g) * p.N + n;
+      const int64_t at = static_cast<int64_t>(m) * p.ldc + static_cast<int64_t>(g) * p.c_step + n;
       if (EPI == kSimtAxpyF32) {
         float* c = reinterpret_cast<float*>(p.C) + at;
         *c += p.alpha * acc[0][i][j];
@@ -161,8 +161,15 @@ __global__ void __launch_bounds__(kSgThreads) gemm_grouped_simt_kernel(const Gro
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx + 16 * j;
-      if (n < g.N)
-        stf<T>(reinterpret_cast<T*>(p.C) + static_cast<int64_t>(g.row0 + m) * p.ldc + n, grouped_act(p.act, acc[i][j], f));
+      T* dst = reinterpret_cast<T*>(p.C) + static_cast<int64_t>(g.row0 + m) * p.ldc;
+      if (p.act == kActSiluGate) {  // columns 0 .. 31 of the tile gate columns 32 .. 63
+        if (j < 2 && n < g.N) {
+          const float z = acc[i][j] * f.x;
+          stf<T>(dst + n0 / 2 + tx + 16 * j, silu_acc(z) * (acc[i][(j + 2) & 3] * f.x) * f.y);
+        }
+      } else if (n < g.N) {
+        stf<T>(dst + n, grouped_act(p.act, acc[i][j], f));
+      }
     }
   }
 }
@@ -174,14 +181,14 @@ using namespace blitz;
 
 // C[M, N] = A[M, K] B[K, N] per group; dtype 0 fp16, 1 bf16, 2 fp32 (of A and B, and of C unless the epilogue says
 // fp32).  epilogue 0 store, 2 silu(gate) * up with the up columns of B from up_off on, 4 store as fp32,
-// 5 C += alpha * acc with C fp32, 6 alpha * tanh(acc / alpha) as fp32.
+// 5 C += alpha * acc with C fp32, 6 alpha * tanh(acc / alpha) as fp32.  a_step, c_step: columns of A and C between two groups.
 int blitz_gemm_simt(const void* A, int64_t lda, const void* B, int64_t ldb, void* C, int64_t ldc, int M, int N, int K,
-                    int epilogue, int up_off, float alpha, int groups, int dtype, cudaStream_t stream) {
+                    int epilogue, int up_off, float alpha, int groups, int a_step, int c_step, int dtype, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0 || groups <= 0) return 0;
   if (epilogue != 0 && epilogue != 2 && epilogue != 4 && epilogue != 5 && epilogue != 6) return -1;
   if (epilogue == 6 && !(alpha > 0.f)) return -1;
   if ((M + kSgT - 1) / kSgT > 65535 || groups > 65535) return -1;
-  SimtGemmParams p{A, B, C, lda, ldb, ldc, M, N, K, up_off, alpha};
+  SimtGemmParams p{A, B, C, lda, ldb, ldc, M, N, K, up_off, a_step, c_step, alpha};
   cudaError_t e = cudaSuccess;
   BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_simt<T>(p, epilogue, groups, stream)));
   return (int)e;

@@ -15,7 +15,7 @@
 //   cap f32    C = alpha * tanh(acc / alpha), C in fp32  (soft-capped logits)
 //
 // Block-diagonal products (groups > 1): B is `groups` blocks [K,N] stacked along K; group g takes the K columns of A
-// from g * K on and the N columns of C from g * N on.  An N tile belongs to one group and simply starts its K walk there
+// from g * a_step on and the N columns of C from g * c_step on (heads of a wider activation).  An N tile belongs to one group and simply starts its K walk there
 // (K is then a multiple of the 64-wide K block, so that no block reaches into a neighbour).
 //
 // Measured on B200: a 128-row tcgen05.mma of K = 16 occupies the tensor pipe for ~95 / 105 / 150 cycles at
@@ -75,6 +75,7 @@ struct GemmParams {
   float alpha;      // axpy; soft cap
   int groups;       // diagonal blocks (1: an ordinary product); N and K are those of one block
   int group_tiles;  // N tiles per block
+  int a_step, c_step;  // columns of A and C between two blocks
 };
 
 // Tile number -> (M block, N block).  Normally M runs fastest.  When the rows of A arrive from other ranks
@@ -156,7 +157,7 @@ __device__ __forceinline__ void store_chunk(const GemmParams& p, const float (&a
                                             int col0, bool row_ok, int group = 0) {
   if (EPI == kEpiStoreF32 || EPI == kEpiAxpyF32 || EPI == kEpiCapF32) {
     if (!row_ok) return;
-    float* dst = reinterpret_cast<float*>(p.C) + static_cast<int64_t>(row) * p.ldc + static_cast<int64_t>(group) * p.N + col0;
+    float* dst = reinterpret_cast<float*>(p.C) + static_cast<int64_t>(row) * p.ldc + static_cast<int64_t>(group) * p.c_step + col0;
     float old[4][8];
     const float inv = EPI == kEpiCapF32 ? 1.f / p.alpha : 0.f;
     if (EPI == kEpiAxpyF32) {
@@ -216,7 +217,7 @@ __device__ __forceinline__ void store_chunk(const GemmParams& p, const float (&a
                         make_uint4(out[4 * j], out[4 * j + 1], out[4 * j + 2], out[4 * j + 3]));
       }
     } else {
-      T* dst = reinterpret_cast<T*>(p.C) + static_cast<int64_t>(row) * p.ldc + static_cast<int64_t>(group) * p.N + col0;
+      T* dst = reinterpret_cast<T*>(p.C) + static_cast<int64_t>(row) * p.ldc + static_cast<int64_t>(group) * p.c_step + col0;
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         if (col0 + j * 8 < p.N)
@@ -313,7 +314,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
         const int tile = w / p.split_k, split = w % p.split_k;
         int mb, nb;
         gemm_tile_blocks(p, tile, mb, nb);
-        const int kb_group = gemm_group(p, nb) * num_kb;  // first K block of the tile's diagonal block
+        const int group = gemm_group(p, nb);  // the tile's diagonal block
+        const int a_col = group * p.a_step;
         const int m0 = mb * kBM;
         const int n0 = nb * kOutCols;
         if (p.n_wait > 0) {
@@ -335,8 +337,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
           }
           if (fresh) ptx::fence_proxy_async_all();
         }
-        const int kb_beg = kb_group + split * p.kb_per_split;
-        const int kb_end = min(kb_group + num_kb, kb_beg + p.kb_per_split);
+        const int kb_beg = split * p.kb_per_split;
+        const int kb_end = min(num_kb, kb_beg + p.kb_per_split);
         for (int kb = kb_beg; kb < kb_end; ++kb) {
           if (!ptx::bounded_mbar_wait(&empty_bar[stage], phase ^ 1u, abort_flag)) {
             if (p.status) atomicCAS(p.status, 0, kStatusTimeoutProducer);
@@ -344,7 +346,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
             break;
           }
           ptx::mbar_expect_tx(&full_bar[stage], tx_bytes);
-          ptx::tma_load_2d(smem_a + stage * a_stage, &tmap_a, &full_bar[stage], kb * kBK, m0);
+          ptx::tma_load_2d(smem_a + stage * a_stage, &tmap_a, &full_bar[stage], a_col + kb * kBK, m0);
           uint8_t* sb = smem_b + stage * Cfg::kBBytes;
           if (B_KMAJOR) {
             // B is [N,K]: one box of BN rows x 64 K-elements per half (silu: gate rows then up rows).
@@ -366,7 +368,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
               } else {
                 col = n0 + s * 64;
               }
-              ptx::tma_load_2d(sb + s * 8192, &tmap_b, &full_bar[stage], col, kb * kBK);
+              if (p.groups > 1)  // rows behind a block's end arrive as zeros
+                ptx::tma_load_3d(sb + s * 8192, &tmap_b, &full_bar[stage], col, kb * kBK, group);
+              else
+                ptx::tma_load_2d(sb + s * 8192, &tmap_b, &full_bar[stage], col, kb * kBK);
             }
           }
           if (++stage == S) {
@@ -598,7 +603,8 @@ int64_t blitz_gemm_workspace_bytes(int sms) { return (int64_t)(sms + 16) * blitz
 // dtype: 0 = fp16, 1 = bf16.  b_layout: 0 = B is [K, ldb>=Ncols] row-major (weights stored in,out),
 // 1 = B is [Ncols, ldb>=K] row-major.  epilogue: 0 store, 1 add residual R (same pitch as C),
 // 2 silu(gate)*up where B carries N gate columns followed (at column `up_col_off`) by N up columns, 4 store with C in
-// fp32, 5 C += alpha * acc with C in fp32, 6 alpha * tanh(acc / alpha) with C in fp32.  groups: number of diagonal blocks (see the top of the file), 1 = none.
+// fp32, 5 C += alpha * acc with C in fp32, 6 alpha * tanh(acc / alpha) with C in fp32.  groups: number of diagonal blocks (see the top of the file), 1 = none;
+// a_step, c_step: columns of A and C between two blocks, multiples of 8.
 // bn_hint: 0 = 256-wide tiles, else 64/128/256.  split_hint: 0 = choose, 1 = never split, else the
 // number of K splits.  ws / ws_bytes: fp32 scratch for split-K partials, tickets / num_tickets:
 // zeroed uint32 array (both may be null: the GEMM then never splits).
@@ -631,10 +637,10 @@ struct BlitzGemmTp {
 static int gemm_impl(const void* A, int64_t lda, const void* B, int64_t ldb, void* C, int64_t ldc, const void* R, int M,
                      int N, int K, int b_layout, int epilogue, int up_col_off, int dtype, int bn_hint, int split_hint,
                      void* ws, int64_t ws_bytes, unsigned* tickets, int num_tickets, int* status,
-                     const BlitzGemmTp* tpa, float alpha, int groups, cudaStream_t stream) {
+                     const BlitzGemmTp* tpa, float alpha, int groups, int a_step, int c_step, cudaStream_t stream) {
   using namespace blitz;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
-  if (groups < 1 || (groups > 1 && ((K % kBK) != 0 || b_layout != 0 || tpa != nullptr ||
+  if (groups < 1 || (groups > 1 && (((a_step | c_step) & 7) != 0 || a_step < 0 || c_step < N || b_layout != 0 || tpa != nullptr ||
                                     (epilogue != kEpiStore && epilogue != kEpiStoreF32))))
     return -1;
   if ((N & 7) || (K & 7) || (lda & 7) || (ldb & 7) || (ldc & 7)) return -1;
@@ -659,6 +665,8 @@ static int gemm_impl(const void* A, int64_t lda, const void* B, int64_t ldb, voi
   p.group_tiles = (N + out_cols - 1) / out_cols;
   p.tiles_n = p.group_tiles * groups;
   p.groups = groups;
+  p.a_step = a_step;
+  p.c_step = c_step;
   p.alpha = alpha;
   p.status = status;
   p.tp = 1; p.tp_rank = 0; p.rows_per_rank = M; p.wait_flags = nullptr; p.n_wait = 0; p.wait_value = 0; p.m_rot = 0; p.n_fast = 0;
@@ -698,10 +706,12 @@ static int gemm_impl(const void* A, int64_t lda, const void* B, int64_t ldb, voi
   p.tickets = tickets;
 
   CUtensorMap ta, tb;
-  if (!get_tmap_2d(&ta, A, (uint64_t)K * groups, (uint64_t)M, (uint64_t)lda * 2, kBK, (uint32_t)p.a_box_rows)) return -2;
+  if (!get_tmap_2d(&ta, A, (uint64_t)a_step * (groups - 1) + K, (uint64_t)M, (uint64_t)lda * 2, kBK, (uint32_t)p.a_box_rows)) return -2;
   bool okb;
-  if (b_layout == 0) {
-    okb = get_tmap_2d(&tb, B, (uint64_t)b_cols_total, (uint64_t)K * groups, (uint64_t)ldb * 2, 64, kBK);
+  if (groups > 1) {
+    okb = get_tmap_3d(&tb, B, (uint64_t)N, (uint64_t)K, (uint64_t)groups, (uint64_t)ldb * 2, (uint64_t)K * ldb * 2, 64, kBK, 1);
+  } else if (b_layout == 0) {
+    okb = get_tmap_2d(&tb, B, (uint64_t)b_cols_total, (uint64_t)K, (uint64_t)ldb * 2, 64, kBK);
   } else {
     const uint32_t box_rows = epilogue == kEpiSiluMul ? bn / 2 : bn;
     okb = get_tmap_2d(&tb, B, (uint64_t)K, (uint64_t)b_cols_total, (uint64_t)ldb * 2, kBK, box_rows);
@@ -724,10 +734,10 @@ static int gemm_impl(const void* A, int64_t lda, const void* B, int64_t ldb, voi
 int blitz_gemm(const void* A, int64_t lda, const void* B, int64_t ldb, void* C, int64_t ldc, const void* R, int M,
                int N, int K, int b_layout, int epilogue, int up_col_off, int dtype, int bn_hint, int split_hint,
                void* ws, int64_t ws_bytes, unsigned* tickets, int num_tickets, int* status, float alpha, int groups,
-               cudaStream_t stream) {
+               int a_step, int c_step, cudaStream_t stream) {
   if (epilogue == blitz::kEpiPushRS) return -1;
   return gemm_impl(A, lda, B, ldb, C, ldc, R, M, N, K, b_layout, epilogue, up_col_off, dtype, bn_hint, split_hint, ws,
-                   ws_bytes, tickets, num_tickets, status, nullptr, alpha, groups, stream);
+                   ws_bytes, tickets, num_tickets, status, nullptr, alpha, groups, a_step, c_step, stream);
 }
 
 // Tensor-parallel variant: epilogue 3 pushes the partial result to the owner ranks' staging areas
@@ -738,7 +748,7 @@ int blitz_gemm_tp(const void* A, int64_t lda, const void* B, int64_t ldb, void* 
                   void* ws, int64_t ws_bytes, unsigned* tickets, int num_tickets, int* status, const BlitzGemmTp* tp,
                   cudaStream_t stream) {
   return gemm_impl(A, lda, B, ldb, C, ldc, R, M, N, K, b_layout, epilogue, up_col_off, dtype, bn_hint, split_hint, ws,
-                   ws_bytes, tickets, num_tickets, status, tp, 1.f, 1, stream);
+                   ws_bytes, tickets, num_tickets, status, tp, 1.f, 1, 0, 0, stream);
 }
 
 }  // extern "C"

@@ -6,7 +6,9 @@
 
 namespace blitz {
 
-enum GroupedAct : int { kActNone = 0, kActReluSquared = 1 };
+// kActSiluGate: a matrix holds 32 gate columns, the 32 up columns they gate, the next 32 gate columns, and so on; the output
+// has half as many columns, silu(gate) * up.
+enum GroupedAct : int { kActNone = 0, kActReluSquared = 1, kActSiluGate = 2 };
 
 struct GroupedParams {
   const void* A;
@@ -57,6 +59,12 @@ __device__ __forceinline__ float grouped_act(int act, float acc, float2 f) {
     z *= z;
   }
   return z * f.y;
+}
+
+// silu(gate) * up with the factors before (of both accumulators) and after
+__device__ __forceinline__ float grouped_silu_gate(float gate, float up, float2 f) {
+  const float z = gate * f.x;
+  return z / (1.f + __expf(-z)) * (up * f.x) * f.y;
 }
 
 }  // namespace blitz

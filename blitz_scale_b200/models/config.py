@@ -85,7 +85,7 @@ REGISTRY: Dict[str, ModelConfig] = {c.name: c for c in [
 
 def hybrid_registry():
     """Shapes of the models whose layers differ (a separate table: the native twin of the registry holds the uniform ones)."""
-    from . import komulorn
+    from . import komulorn, vofidra
     from .fafudra import shape_config
     mixed = ("gla", "attention", "rglru", "gla")
     return {c.name: c for c in [
@@ -105,11 +105,20 @@ def hybrid_registry():
                               ff=51, shared_ff=30, share=3),
         komulorn.shape_config("komulorn_13b", 128256, 2048, 32, heads=32, kv_heads=4, dim=128, vdim=128, rot_dims=64, experts=64,
                               top=6, ff=1408, shared_ff=2816, gb=27),
+        # several residual streams, attention with a bias by distance, latent attention, a mixture of experts with identity
+        # experts: likewise, the last one of 13 B parameters
+        vofidra.shape_config("vofidra_tiny", 2048, 320, 4, heads=8, kv_heads=2, dim=64, latent=dict(heads=4, dim=64, rot_dim=32, vdim=64,
+                             q_rank=192, kv_rank=128), experts=10, identity=6, top=4, groups=4, keep=2, ff=96, dense_ff=512, streams=2),
+        vofidra.shape_config("vofidra_odd", 1003, 122, 3, heads=6, kv_heads=3, dim=22, latent=dict(heads=3, dim=13, rot_dim=6, vdim=11,
+                             q_rank=35, kv_rank=21), experts=5, identity=1, top=3, groups=3, keep=2, ff=51, dense_ff=77, streams=3),
+        vofidra.shape_config("vofidra_13b", 128256, 2048, 28, heads=16, kv_heads=4, dim=128, latent=dict(heads=32, dim=64, rot_dim=32,
+                             vdim=64, q_rank=768, kv_rank=256), experts=48, identity=16, top=6, groups=8, keep=4, ff=1536,
+                             dense_ff=8192, streams=4, gb=26),
     ]}
 
 
 # designs described by data: "architecture" of config.json -> module of this package with parse_config and to_segment
-DESIGNS = {"Fafudra": "fafudra", "Komulorn": "komulorn"}
+DESIGNS = {"Fafudra": "fafudra", "Komulorn": "komulorn", "Vofidra": "vofidra"}
 
 
 def design_module(name: str):

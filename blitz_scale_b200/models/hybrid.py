@@ -14,7 +14,18 @@ A layer run with experts behind the mixer::
 The experts' output rows stay where the last product leaves them: the next layer's norm kernel adds them to the stream
 (`flush` does where a pass ends).
 
-    attention: rope_store (biases, rotation, paged write) -> attention over the pages (window, cap, sink, gate per head)
+A model with several residual streams: every sublayer starts with one kernel that lets the streams take up the output of the
+sublayer before it, joins them and norms the result::
+
+    stream_mix -> GEMM (in) -> mixer -> GEMM (out)
+    -> stream_mix -> GEMM (gate||up, SiLU*mul) -> GEMM (down)     or router, moe_route and the grouped products as above
+
+    attention: rope_store (biases, rotation, paged write) or norm_store (norm of every head, paged write)
+               -> attention over the pages (window, cap, sink, gate per head, bias by distance)
+    latent:    latent_store (norms, shared rotated key, paged write) -> GEMM (queries), then
+               single tokens: block-diagonal GEMM (queries into the latent space) -> rotation -> attention over the cached
+               rows, one key and value for all heads -> block-diagonal GEMM (values out of the latent space);
+               prompts: rotation -> gather of the cached rows -> GEMMs (keys, values of all heads) -> attention
     gla:       one kernel (decay projection, recurrence, output norm, gate), or the chunked kernels for prompts
     rglru:     conv_causal -> block-diagonal GEMM (gates, fp32 out) -> rglru_scan
 
@@ -29,7 +40,7 @@ import torch
 
 from .. import ops
 from ..runtime.hybrid_cache import HybridCache
-from .hybrid_config import AttentionMixer, ExpertsSpec, GLAMixer, HybridConfig, LayerSpec, RGLRUMixer
+from .hybrid_config import AttentionMixer, ExpertsSpec, GLAMixer, HybridConfig, LatentAttentionMixer, LayerSpec, RGLRUMixer
 from .llama import StepMeta
 from .weights import WeightSegment
 
@@ -43,7 +54,8 @@ class HybridRunner:
         self.max_tokens, self.max_batch = max_tokens, max_batch
         dev, dt = seg.buffer.device, seg.dtype
         H = cfg.hidden
-        self.res = torch.empty(max_tokens, H, dtype=torch.float32, device=dev)      # residual stream
+        # residual stream, or streams
+        self.res = torch.empty(*(max_tokens, cfg.streams, H) if cfg.streams else (max_tokens, H), dtype=torch.float32, device=dev)
         self.normed = torch.empty(max_tokens, H, dtype=dt, device=dev)
         self._proj = torch.empty(max_tokens * max(s.in_columns()[1] for s in cfg.layer_specs), dtype=dt, device=dev)
         # mixer output and feed-forward activation side by side, one buffer per column layout: its padding columns stay
@@ -59,6 +71,8 @@ class HybridRunner:
         ck = max((m.heads * m.dim for m in cfg.run_mixers() if m.kind == "gla"), default=0)
         self._cum = torch.empty(max_tokens * ck, dtype=torch.float32, device=dev) if ck and dt == torch.bfloat16 else None
         self._init_experts(max_tokens, dev, dt)
+        self._init_streams(max_tokens, max_batch, dev, dt)
+        self._init_latent(max_tokens, max_batch, dev, dt)
         self.last = torch.empty(max_batch, H, dtype=torch.float32, device=dev)
         self._logits_pad = torch.zeros(max_batch, cfg.vocab_pad, dtype=torch.float32, device=dev)
         self.logits = self._logits_pad[:, :cfg.vocab]
@@ -68,6 +82,8 @@ class HybridRunner:
             if m.kind == "attention" and self._rot_key(m) not in self._freqs:
                 stretch = m.yarn.stretch(m.rot_dims, m.rot_base) if m.yarn else None
                 self._freqs[self._rot_key(m)] = ops.rope_freqs(m.rot_dims, m.rot_base, dev, stretch)
+            elif m.kind == "latent":
+                self._freqs[(m.rot_dim, m.rot_base, None)] = ops.rope_freqs(m.rot_dim, m.rot_base, dev)
         self._ws: Optional[torch.Tensor] = None
         self._ws_old: List[Optional[torch.Tensor]] = []
 
@@ -93,7 +109,7 @@ class HybridRunner:
         for e in moes:
             key = self._plan_key(e)
             if key not in self._plans:
-                self._plans[key] = ops.ExpertPlan(max_tokens, e.experts, e.top, bool(e.shared_ff), dev)
+                self._plans[key] = ops.ExpertPlan(max_tokens, e.experts, e.top, bool(e.shared_ff), dev, e.identity)
         rows = max_tokens * max(e.per_token for e in moes)
         self._router = torch.empty(max_tokens * max(e.router_cols for e in moes), dtype=torch.float32, device=dev)
         self._act = torch.empty(rows * max(max(e.ff_pad, e.shared_pad) for e in moes), dtype=dt, device=dev)
@@ -101,7 +117,35 @@ class HybridRunner:
 
     @staticmethod
     def _plan_key(e: ExpertsSpec) -> tuple:
-        return (e.experts, e.top, bool(e.shared_ff))
+        return (e.experts, e.top, bool(e.shared_ff), e.identity)
+
+    def _init_streams(self, max_tokens: int, max_batch: int, dev, dt) -> None:
+        """Buffers of a model with several streams: the last sublayer's output, a feed-forward's activations, the head's input."""
+        c = self.cfg
+        self._fresh = False          # the streams are still the embeddings (of self._ids) and not in memory
+        self._ids: Optional[torch.Tensor] = None
+        if not c.streams:
+            return
+        self._y = torch.empty(max_tokens, c.hidden, dtype=dt, device=dev)
+        self._head_in = torch.empty(max_batch, c.hidden, dtype=dt, device=dev)
+        ff = max(s.ff_after_pad for s in c.layer_specs)
+        self._ff = torch.empty(max_tokens * ff, dtype=dt, device=dev) if ff else None
+
+    def _init_latent(self, max_tokens: int, max_batch: int, dev, dt) -> None:
+        """Buffers of latent attention: queries, and queries and outputs in the latent space (of single tokens where the prompts'
+        keys and values are expanded, else of all tokens)."""
+        ms = [m for m in self.cfg.run_mixers() if m.kind == "latent"]
+        self._scratch: Dict[str, torch.Tensor] = {}
+        if not ms:
+            return
+        rows = lambda m: max_batch if self._expands(m, dt) else max_tokens
+        self._q = torch.empty(max_tokens * max(m.heads * m.qdim for m in ms), dtype=dt, device=dev)
+        self._q_latent = torch.empty(max(rows(m) * m.heads * m.width for m in ms), dtype=dt, device=dev)
+        self._o_latent = torch.empty(max(rows(m) * m.heads * m.kv_rank for m in ms), dtype=dt, device=dev)
+
+    def _expands(self, m: LatentAttentionMixer, dt) -> bool:
+        """Whether prompts run over expanded keys and values on the tensor cores (else over the latent rows)."""
+        return dt != torch.float32 and ops.attn_head_sizes(m.qdim, m.vdim, self.page_size) and m.width % 8 == 0
 
     # ------------------------------------------------------------------ pieces
     def embed(self, m: StepMeta) -> None:
@@ -112,6 +156,8 @@ class HybridRunner:
         run, T, c = self.runs[r], m.num_tokens, self.cfg
         l = run.layer
         spec = c.layer_specs[l]
+        if c.streams:
+            return self._run_layer_streams(r, l, spec, m)
         step = self.seg["loop_step"][run.step] if run.step >= 0 else None
         h = self.normed[:T]
         needs_ids = r == 0 or run.add_embed
@@ -131,41 +177,91 @@ class HybridRunner:
         ops.gemm(mid, self._w(l, "out"), out=self.res[:T], epilogue="axpy", alpha=c.residual_mult, static_b=True)
         if spec.moe:
             ops.stream_norm(self.res[:T], self._w(l, "norm2"), c.rms_eps, h, w_offset=c.norm_offset)
-            self._experts(l, spec.moe, h)
+            out, plan = self._experts(l, spec.moe, h)
+            self._pending = (out, plan.place)
+
+    def _norm(self, name: str) -> tuple:
+        return self.seg[name], self.seg[name + "_alpha"], self.seg[name + "_b"]
+
+    def _join(self, l: int, q: int, T: int) -> torch.Tensor:
+        """Input of sublayer q of layer l; the streams take up what is pending."""
+        take, h = self._pending is not None, self.normed[:T]
+        ops.stream_mix(self.res[:T], **self._embeddings(), pending=self._pending, read=self._w(l, f"hc{q}_in"),
+                       norm=self._norm(f"layers.{l}.norm{q}"), out=h, write=take)
+        self._fresh = self._fresh and not take
+        return h
+
+    def _embeddings(self) -> dict:
+        return dict(ids=self._ids, embed=self.seg["embed"]) if self._fresh else {}
+
+    def _leave(self, l: int, q: int, y: torch.Tensor, **rows) -> None:
+        self._pending = ops.Pending(y, self._w(l, f"hc{q}_mix"), self._w(l, f"hc{q}_out"), **rows)
+
+    def _run_layer_streams(self, r: int, l: int, spec: LayerSpec, m: StepMeta) -> None:
+        T = m.num_tokens
+        if r == 0:
+            self._pending, self._fresh, self._ids = None, True, m.ids
+        h, y = self._join(l, 1, T), self._y[:T]
+        cols, width = spec.in_columns()
+        proj = self._proj[:T * width].view(T, width)
+        ops.gemm(h, self._w(l, "in"), out=proj, static_b=True)
+        mid = self._mid[self._mid_key(spec)][:T]
+        getattr(self, "_" + spec.mixer.kind)(r, l, spec.mixer, {n: proj[:, at:at + w] for n, (at, w) in cols.items()}, mid, m)
+        ops.gemm(mid, self._w(l, "out"), out=y, static_b=True)
+        self._leave(l, 1, y)
+        if spec.ff_after:
+            h = self._join(l, 2, T)
+            act = self._ff[:T * spec.ff_after_pad].view(T, spec.ff_after_pad)
+            ops.gemm(h, self._w(l, "gate_up"), out=act, epilogue="silu_mul", static_b=True)
+            ops.gemm(act, self._w(l, "down"), out=y, static_b=True)
+            self._leave(l, 2, y)
+        elif spec.moe:
+            h = self._join(l, 2, T)
+            out, plan = self._experts(l, spec.moe, h)
+            self._leave(l, 2, out, place=plan.place, ident=plan.ident, prev=h if spec.moe.identity else None)
 
     def _take_pending(self) -> dict:
         p, self._pending = self._pending, None
         return dict(add=p[0], add_rows=p[1]) if p else {}
 
     def flush(self, T: int) -> None:
-        """Everything the layers so far have produced is in the stream."""
-        if self._pending:
+        """Everything the layers so far have produced is in the stream (several streams: what reads them takes it up)."""
+        if self._pending and not self.cfg.streams:
             ops.stream_norm(self.res[:T], None, 0.0, None, **self._take_pending())
 
-    def _experts(self, l: int, e: ExpertsSpec, h: torch.Tensor) -> None:
+    def _experts(self, l: int, e: ExpertsSpec, h: torch.Tensor) -> tuple:
+        """Output rows of the chosen experts, and the plan that says whose they are."""
         T, H = h.shape
         plan = self._plans[self._plan_key(e)]
         z = self._router[:T * e.router_cols].view(T, e.router_cols)
         # few columns: beyond a decode batch, narrow tiles with K split keep more SMs loading
         narrow = dict(bn=64, split_k=4 if T <= 2048 else 1) if T > ops.DECODE_GEMM_MAX_M else {}
         ops.gemm(h, self._w(l, "router"), out=z, static_b=True, **narrow)
-        up, down = self._w(l, "up").view(e.experts, H, e.ff_pad), self._w(l, "down").view(e.experts, e.ff_pad, H)
+        up, down = self._w(l, "up").view(e.experts, H, e.up_cols), self._w(l, "down").view(e.experts, e.ff_pad, H)
         s_up, s_down = (self._w(l, "shared_up"), self._w(l, "shared_down")) if e.shared_ff else (None, None)
         tc = ops.grouped_tensor_core(h, up, down, s_up, s_down)
-        ops.moe_route(z, plan, weight_on_input=e.weight_on_input, renormalize=e.renormalize, tile_rows=128 if tc else 64)
+        ops.moe_route(z, plan, weight_on_input=e.weight_on_input, renormalize=e.renormalize, softmax=e.softmax,
+                      correction=self._w(l, "correction") if e.correction else None, groups=e.groups, keep=e.keep,
+                      tile_rows=128 if tc else 64)
         width = max(e.ff_pad, e.shared_pad)
         act, out = self._act[:plan.rows * width].view(plan.rows, width), self._expert_out[:plan.rows]
-        ops.gemm_grouped(h, up, plan, act, shared=s_up, gather=True, act="relu2", factors=True)
+        ops.gemm_grouped(h, up, plan, act, shared=s_up, gather=True, act="silu_gate" if e.gated else "relu2", factors=True)
         ops.gemm_grouped(act, down, plan, out, shared=s_down)
-        self._pending = (out, plan.place)
+        return out, plan
 
     def _attention(self, r: int, l: int, mx: AttentionMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta) -> None:
         T, kv = m.num_tokens, self.cache.runs[r].kv
-        biases = {n: self._w(l, n) for n, _ in mx.tensors() if n != "sink"}
-        ops.rope_store(p["q"], p.get("k"), p.get("v"), m.pos, m.slot, kv, self._freqs[self._rot_key(mx)], q_heads=mx.heads,
-                       kv_heads=mx.kv_heads, dim=mx.dim, rot_dims=mx.rot_dims, page_size=self.page_size,
-                       interleaved=mx.interleaved, gain=mx.yarn.gain if mx.yarn else 1.0, **biases)
-        extra = dict(window=mx.window, keep_first=mx.keep_first, softcap=mx.softcap, sink=self._w(l, "sink") if mx.sink else None)
+        if mx.qk_norm:
+            temp = dict(temp_coef=mx.q_temp.coef, temp_every=mx.q_temp.every) if mx.q_temp else {}
+            ops.norm_store(p["q"], p["k"], p["v"], m.pos, m.slot, kv, self._w(l, "q_norm"), self._w(l, "k_norm"), q_heads=mx.heads,
+                           kv_heads=mx.kv_heads, dim=mx.dim, page_size=self.page_size, eps=self.cfg.rms_eps, **temp)
+        else:
+            biases = {n + "_b": self._w(l, n + "_b") for n in ("q", "k", "v") if mx.bias and n in p}
+            ops.rope_store(p["q"], p.get("k"), p.get("v"), m.pos, m.slot, kv, self._freqs[self._rot_key(mx)], q_heads=mx.heads,
+                           kv_heads=mx.kv_heads, dim=mx.dim, rot_dims=mx.rot_dims, page_size=self.page_size,
+                           interleaved=mx.interleaved, gain=mx.yarn.gain if mx.yarn else 1.0, **biases)
+        extra = dict(window=mx.window, keep_first=mx.keep_first, softcap=mx.softcap, sink=self._w(l, "sink") if mx.sink else None,
+                     bias=self._w(l, "rel_by_distance") if mx.rel else None)
         gate = p.get("g")
         if not ops.attn_tensor_core(p["q"], mx.heads, mx.kv_heads, mx.dim, self.page_size, mx.vdim):
             ops.attn_ragged(p["q"], kv, m.pos, m.tok_indptr if m.is_prefill else None, m.page_indptr, m.page_indices, mid,
@@ -189,6 +285,61 @@ class HybridRunner:
             self._ws_old.append(self._ws)
             self._ws = torch.empty(n, dtype=torch.uint8, device=self.res.device)
         return self._ws
+
+    def _latent(self, r: int, l: int, mx: LatentAttentionMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta) -> None:
+        T, H, R, W, kv = m.num_tokens, mx.heads, mx.kv_rank, mx.width, self.cache.runs[r].kv
+        freqs, gate = self._freqs[(mx.rot_dim, mx.rot_base, None)], p.get("g")
+        ops.latent_store(p["dq"], p["dkv"], m.pos, m.slot, kv, self._w(l, "dq_norm"), self._w(l, "dkv_norm"), freqs, eps=self.cfg.rms_eps)
+        q = self._q[:T * H * mx.qdim].view(T, H * mx.qdim)
+        ops.gemm(p["dq"], self._w(l, "uq"), out=q, static_b=True)
+        rotate = dict(heads=H, dim=mx.dim, rot=mx.rot_dim)
+        n = m.batch if not m.is_prefill else m.singles if self._expands(mx, q.dtype) else T    # rows that go through the latent space
+        if n:
+            ql, ol = self._q_latent[:n * H * W].view(n, H * W), self._o_latent[:n * H * R].view(n, H * R)
+            ops.gemm(q[:n], self._w(l, "uk"), out=ql, groups=H, a_step=mx.qdim, out_step=W, static_b=True)
+            ops.latent_rotate(q[:n], ql[:, R:], m.pos[:n], freqs, out_step=W, **rotate)
+            single = not m.is_prefill or n == m.singles
+            ops.attn_ragged(ql, kv, m.pos, None if single else m.tok_indptr, m.page_indptr[:n + 1] if single else m.page_indptr,
+                            m.page_indices, ol, q_heads=H, kv_heads=1, dim=W, page_size=self.page_size, scale=mx.scale,
+                            gate=gate[:n] if gate is not None else None)
+            ops.gemm(ol, self._w(l, "uv"), out=mid[:n, :H * mx.vdim], groups=H, a_step=R, out_step=mx.vdim, static_b=True)
+        if n < T:
+            self._latent_prompts(l, mx, q, gate, kv, mid, m, n, freqs, rotate)
+
+    def _latent_prompts(self, l: int, mx: LatentAttentionMixer, q, gate, kv: ops.LatentKV, mid, m: StepMeta, n: int, freqs, rotate) -> None:
+        """Rows from n on: keys and values of all their sequences' cached rows are expanded into a pool of their own, some heads
+        at a time where that would be large."""
+        ops.latent_rotate(q[n:], q[n:, mx.dim:], m.pos[n:], freqs, out_step=mx.qdim, **rotate)
+        ps = self.page_size
+        pages = [-(-kv_len // ps) for kv_len in m.kv_lens_host]
+        first, total = sum(pages[:n]), sum(pages)
+        np_ = total - first
+        # page i of the expanded pool is the i-th page of these sequences
+        index = torch.arange(-first, np_, dtype=torch.int32, device=q.device)
+        rows = ops.latent_gather(kv, m.page_indices[first:total], self._room("rows", (np_ * ps, mx.width), q.dtype))
+        H = mx.heads
+        heads = max(1, min(H, self.EXPANDED_BYTES // (np_ * ps * (mx.qdim + mx.vdim) * 2)))
+        for h0 in range(0, H, heads):
+            hn = min(heads, H - h0)
+            k = self._room("keys", (np_, ps, hn, mx.qdim), q.dtype)
+            v = self._room("values", (np_, ps, hn, mx.vdim), q.dtype)
+            ops.gemm(rows, self._w(l, "k_up")[:, h0 * mx.qdim:(h0 + hn) * mx.qdim], out=k.view(np_ * ps, -1), static_b=True)
+            ops.gemm(rows[:, :mx.kv_rank], self._w(l, "v_up")[:, h0 * mx.vdim:(h0 + hn) * mx.vdim], out=v.view(np_ * ps, -1), static_b=True)
+            ops.attn_prefill_paged(q[:, h0 * mx.qdim:(h0 + hn) * mx.qdim], ops.KVPair(k, v), index, m.prefill_work, q_heads=hn, kv_heads=hn,
+                                   head_dim=mx.qdim, page_size=ps, sm_scale=mx.scale, out=mid[:, h0 * mx.vdim:(h0 + hn) * mx.vdim],
+                                   gate=gate[:, h0:h0 + hn] if gate is not None else None)
+
+    EXPANDED_BYTES = 1 << 30      # of expanded keys and values at a time
+
+    def _room(self, name: str, shape: tuple, dt) -> torch.Tensor:
+        """Scratch of a prefill pass (grows with the longest one)."""
+        n = 1
+        for s in shape:
+            n *= s
+        have = self._scratch.get(name)
+        if have is None or have.numel() < n:
+            have = self._scratch[name] = torch.empty(n, dtype=dt, device=self.res.device)
+        return have[:n].view(shape)
 
     def _gla(self, r: int, l: int, mx: GLAMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta) -> None:
         ns = m.batch if not m.is_prefill else m.singles
@@ -216,10 +367,16 @@ class HybridRunner:
     def logits_of(self, n: int, rows: Optional[torch.Tensor] = None, row_offset: int = 0) -> torch.Tensor:
         """fp32 logits of `n` rows of the stream: rows 0 .. n - 1, or `rows` (+ row_offset)."""
         c = self.cfg
+        cap = dict(epilogue="softcap", alpha=c.logit_softcap) if c.logit_softcap else {}
+        if c.streams:
+            h = self._head_in[:n]
+            ops.stream_mix(self.res, n=n, **self._embeddings(), pending=self._pending, norm=self._norm("final_norm"), out=h, rows=rows,
+                           row_offset=row_offset)
+            ops.gemm(h, self.seg["lm_head"], out=self._logits_pad[:n], static_b=True, **cap)
+            return self.logits[:n]
         add = {} if rows is not None else self._take_pending()
         ops.stream_norm(self.res, self.seg["final_norm"], c.rms_eps, self.normed[:n], w_offset=c.norm_offset, rows=rows,
                         row_offset=row_offset, num_tokens=n, **add)
-        cap = dict(epilogue="softcap", alpha=c.logit_softcap) if c.logit_softcap else {}
         ops.gemm(self.normed[:n], self.seg["lm_head"], out=self._logits_pad[:n], static_b=True, **cap)
         return self.logits[:n]
 
@@ -233,13 +390,22 @@ class HybridRunner:
         return self.tokens[:B]
 
     def last_rows(self, m: StepMeta) -> torch.Tensor:
-        """[batch, hidden]: the stream at the last row of every sequence of a prefill pass."""
+        """[batch, hidden]: the stream (or the sum of the streams) at the last row of every sequence of a prefill pass."""
+        if self.cfg.streams:
+            last = self.last[:m.batch]
+            ops.stream_mix(self.res, n=m.batch, **self._embeddings(), pending=self._pending, total=last, rows=m.tok_indptr[1:], row_offset=-1)
+            return last
         return torch.index_select(self.res, 0, m.tok_indptr[1:] - 1, out=self.last[:m.batch])
 
     def head_from_rows(self, rows: torch.Tensor) -> torch.Tensor:
         """First tokens from rows collected with `last_rows` over several passes."""
         B = rows.shape[0]
-        self.res[:B].copy_(rows)
+        if self.cfg.streams:
+            self.res[:B].zero_()
+            self.res[:B, 0].copy_(rows)
+            self._pending, self._fresh = None, False
+        else:
+            self.res[:B].copy_(rows)
         return self.head(StepMeta(ids=None, pos=None, slot=None, page_indices=None, page_indptr=None, last_page_len=None,
                                   is_prefill=False, batch=B, num_tokens=B))
 
@@ -256,7 +422,7 @@ class HybridRunner:
 
     def decode_launches(self) -> int:
         """Kernels of this library in one decode step."""
-        per = {"attention": 2, "gla": 1, "rglru": 3}
+        per = {"attention": 2, "latent": 6, "gla": 1, "rglru": 3}
         specs = [self.cfg.layer_specs[r.layer] for r in self.runs]
-        n = sum(3 + per[s.mixer.kind] + bool(s.ff) + 5 * bool(s.moe) for s in specs)
+        n = sum(3 + per[s.mixer.kind] + bool(s.ff) + 3 * bool(s.ff_after) + 5 * bool(s.moe) for s in specs)
         return n + 3      # final norm, head product, arg-max

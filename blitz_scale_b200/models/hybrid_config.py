@@ -1,10 +1,10 @@
-"""Shapes and constants of models whose layers differ: a list of layers over an fp32 residual stream, each with a mixer
-(attention, gated linear attention, gated linear recurrence) and an optional feed-forward, with an optional block of
-layers that runs several times.  The feed-forward is either a gated one beside the mixer (both read one norm) or a
-mixture of experts behind it (with a norm of its own).
+"""Shapes and constants of models whose layers differ: a list of layers over an fp32 residual stream, or several of them,
+each with a mixer (attention, latent attention, gated linear attention, gated linear recurrence) and an optional
+feed-forward, with an optional block of layers that runs several times.  The feed-forward is a gated one beside the mixer
+(both read one norm), or a gated one or a mixture of experts behind it (with a norm of its own).
 
-Everything a kernel needs is a field here, so a design is described by data: `models/fafudra.py` and
-`models/komulorn.py` fill these records from a checkpoint's config.json, the registry from shapes.  `ModelConfig` (config.py) stays the record of
+Everything a kernel needs is a field here, so a design is described by data: `models/fafudra.py`, `models/komulorn.py` and
+`models/vofidra.py` fill these records from a checkpoint's config.json, the registry from shapes.  `ModelConfig` (config.py) stays the record of
 the uniform Llama-type models; both offer what the engine, the worker and the router read (name, vocab, hidden,
 layers, eos_token, param_gb, kv_bytes_per_token).
 
@@ -15,6 +15,11 @@ Weight segment of such a model (one allocation, matrices ``[in, out]``, every te
           | norm2 | router [hidden, experts + 1] | up [experts x hidden, ff] | down [experts x ff, hidden]
           | shared_up [hidden, shared ff] | shared_down [shared ff, hidden] }
     final_norm [hidden] | lm_head [hidden, vocab]
+
+Every norm of a model with the dynamic-tanh norm has two more tensors (``norm1_b`` and ``norm1_alpha``), a sublayer of a
+model with several streams its coefficients (``hc1_in``, ``hc1_out``, ``hc1_mix``), a gated feed-forward behind the mixer
+``gate_up`` and ``down``.  Some tensors are derived from others when a segment is filled (`derive_`): forms of one matrix that
+different kernels read.
 
 A layer has two wide projections per side: ``in`` holds every projection of the mixer next to each other and ``out``
 the mixer's and the feed-forward's output projections on top of each other, so that the sum of both sublayers is one
@@ -69,6 +74,42 @@ class YarnScaling:
 
 
 @dataclass(frozen=True)
+class QueryTemperature:
+    """Queries at position p are multiplied by 1 + coef * ln(floor((p + 1) / every) + 1)."""
+    coef: float
+    every: int
+
+    def __post_init__(self):
+        if self.every < 1:
+            raise ValueError("query temperature: the step must be a positive whole number")
+
+
+@dataclass(frozen=True)
+class DistanceBias:
+    """A table of `rows` numbers per head.  Distances below rows / 2 have a row each; longer ones share the others on a
+    logarithmic scale that reaches the last row at distance `far`."""
+    rows: int
+    far: int
+
+    def __post_init__(self):
+        if self.rows < 2 or self.far <= self.rows // 2:
+            raise ValueError(f"bias by distance: {self.rows} rows up to distance {self.far}")
+
+    def row(self, n: int) -> int:
+        half = self.rows // 2
+        if n < half:
+            return n
+        return min(self.rows - 1, half + math.floor(math.log(n / half) / math.log(self.far / half) * (self.rows - half)))
+
+    def rows_by_distance(self) -> List[int]:
+        """The rows of distances 0, 1, ..; the last entry holds for all longer ones."""
+        out = []
+        while not out or out[-1] != self.rows - 1:
+            out.append(self.row(len(out)))
+        return out
+
+
+@dataclass(frozen=True)
 class AttentionMixer:
     heads: int
     kv_heads: int
@@ -87,6 +128,9 @@ class AttentionMixer:
     gate: bool = False            # a head's output is multiplied by the sigmoid of a projection, one number per head
     yarn: Optional[YarnScaling] = None
     kv_from: Optional[int] = None  # layer whose cached keys and values are used; no k and v projections then
+    qk_norm: bool = False         # RMSNorm of every query and key head (no rotation, no biases)
+    q_temp: Optional["QueryTemperature"] = None   # with qk_norm: queries grow with the position
+    rel: Optional["DistanceBias"] = None          # learned bias by distance and head, added to the scaled scores
     kind = "attention"
 
     def __post_init__(self):
@@ -94,6 +138,12 @@ class AttentionMixer:
             raise ValueError("attention mixer: heads must be a multiple of kv_heads, rotated dimensions even and within a head")
         if self.value_is_key and self.vdim != self.dim:
             raise ValueError("attention mixer: values that are keys have the keys' size")
+        if self.qk_norm and (self.rot_dims or self.bias or self.value_is_key or self.kv_from is not None):
+            raise ValueError("attention mixer: normed queries and keys come without rotation, biases or shared caches")
+        if self.q_temp and not self.qk_norm:
+            raise ValueError("attention mixer: a query temperature goes with normed queries")
+        if self.rel and (self.window or self.softcap or self.sink):
+            raise ValueError("attention mixer: a bias by distance does not go with a window, a cap or a sink")
 
     @property
     def vdim(self) -> int:
@@ -115,7 +165,69 @@ class AttentionMixer:
         return self._qkv() + ([("g", self.heads)] if self.gate else [])
 
     def tensors(self) -> List[Tuple[str, Tuple[int, ...]]]:
-        return ([("sink", (self.heads,))] if self.sink else []) + ([(n + "_b", (w,)) for n, w in self._qkv()] if self.bias else [])
+        out = ([("sink", (self.heads,))] if self.sink else []) + ([(n + "_b", (w,)) for n, w in self._qkv()] if self.bias else [])
+        if self.qk_norm:
+            out += [("q_norm", (self.dim,)), ("k_norm", (self.dim,))]
+        if self.rel:
+            out += [("rel", (self.rel.rows, self.heads)), ("rel_by_distance", (self.heads, len(self.rel.rows_by_distance())))]
+        return out
+
+    def derive_(self, t) -> None:
+        if self.rel:      # the table spread out by distance: what the attention kernels read
+            t("rel_by_distance").copy_(t("rel")[torch.tensor(self.rel.rows_by_distance(), device=t("rel").device)].t())
+
+
+@dataclass(frozen=True)
+class LatentAttentionMixer:
+    """Attention whose keys and values come from one latent vector per token, which is cached together with a rotated key part
+    that all heads share; queries come from a latent of their own.  Per head: `dim` unrotated and `rot_dim` rotated query and
+    key dimensions (half-split pairs), values of `vdim`."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    rot_base: float
+    gate: bool = True             # as in AttentionMixer
+    kind = "latent"
+    kv_heads = 1                  # as the cache sees it: one key, its first kv_rank columns the value
+
+    def __post_init__(self):
+        if self.rot_dim % 2 or min(self.heads, self.dim, self.vdim, self.q_rank, self.kv_rank) < 1:
+            raise ValueError("latent attention mixer: sizes must be positive and rotated dimensions even")
+
+    @property
+    def qdim(self) -> int:
+        return self.dim + self.rot_dim
+
+    @property
+    def width(self) -> int:
+        """Of a cached row."""
+        return self.kv_rank + self.rot_dim
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    def projections(self) -> List[Tuple[str, int]]:
+        return [("dq", self.q_rank), ("dkv", self.width)] + ([("g", self.heads)] if self.gate else [])
+
+    def tensors(self) -> List[Tuple[str, Tuple[int, ...]]]:
+        # uk and uv: blocks of a head stacked along their inputs (absorbed into queries and outputs); k_up and v_up: the
+        # same matrices as one product from cached rows to the keys and the values of all heads
+        H = self.heads
+        return [("dq_norm", (self.q_rank,)), ("dkv_norm", (self.kv_rank,)), ("uq", (self.q_rank, H * self.qdim)),
+                ("uk", (H * self.dim, self.kv_rank)), ("uv", (H * self.kv_rank, self.vdim)),
+                ("k_up", (self.width, H * self.qdim)), ("v_up", (self.kv_rank, H * self.vdim))]
+
+    def derive_(self, t) -> None:
+        H, R = self.heads, self.kv_rank
+        k = t("k_up").zero_().view(self.width, H, self.qdim)
+        k[:R, :, :self.dim].copy_(t("uk").view(H, self.dim, R).permute(2, 0, 1))
+        k[R:, :, self.dim:].copy_(torch.eye(self.rot_dim, dtype=k.dtype, device=k.device)[:, None, :].expand(-1, H, -1))
+        t("v_up").view(R, H, self.vdim).copy_(t("uv").view(H, R, self.vdim).permute(1, 0, 2))
 
 
 @dataclass(frozen=True)
@@ -172,33 +284,65 @@ class RGLRUMixer:
                 ("gate_b", (2 * w,)), ("lam", (w,))]
 
 
-Mixer = Union[AttentionMixer, GLAMixer, RGLRUMixer]
+Mixer = Union[AttentionMixer, LatentAttentionMixer, GLAMixer, RGLRUMixer]
+PAGED = ("attention", "latent")   # mixers with a paged cache; the others keep a state per sequence
 
 
 @dataclass(frozen=True)
 class ExpertsSpec:
-    """Mixture of experts without biases: W_down act(W_up h), act = the square of relu.  A token goes to the `top` experts
-    with the largest router scores (sigmoid of the logits, optionally divided by the sum of the chosen ones); the score
-    multiplies the expert's input or its output.  A shared expert runs for every token and is added, multiplied by the
-    sigmoid of a projection."""
+    """Mixture of experts without biases: W_down act(W_up h), act = the square of relu, or W_down (silu(W_gate h) * W_up h).  A
+    token goes to the `top` experts with the largest router scores (sigmoid of the logits, or their softmax; optionally
+    divided by the sum of the chosen ones); the score multiplies the expert's input or its output.  A shared expert runs for
+    every token and is added, multiplied by the sigmoid of a projection.
+
+    Choices may be made by scores with a learned correction (the weights use them without it), and among the experts of the
+    best groups only: `groups` equal ones of neighbours, of which the `keep` with the largest choice scores stay.  The last
+    `identity` of the router's outputs are experts that return their input."""
     experts: int
     top: int
     ff: int
     shared_ff: int = 0            # 0: no shared expert
     weight_on_input: bool = True
     renormalize: bool = False
+    gated: bool = False           # silu(gate) * up instead of the square of relu
+    softmax: bool = False
+    correction: bool = False
+    identity: int = 0
+    groups: int = 0               # 0: any expert can be chosen
+    keep: int = 0
 
     def __post_init__(self):
-        if not 1 <= self.top <= self.experts or self.ff < 1:
-            raise ValueError(f"{self.top} of {self.experts} experts of width {self.ff}")
+        if not 1 <= self.top <= self.outputs or self.ff < 1 or self.experts < 1 or self.identity < 0:
+            raise ValueError(f"{self.top} of {self.experts} experts (and {self.identity} identity ones) of width {self.ff}")
+        if (self.gated or self.identity) and self.shared_ff:
+            raise ValueError("a shared expert comes with plain experts only")
+        if self.identity and self.weight_on_input:
+            raise ValueError("identity experts go with weights on the output")
+        if self.groups and (self.outputs % self.groups or not 1 <= self.keep <= self.groups
+                            or self.keep * (self.outputs // self.groups) < self.top):
+            raise ValueError(f"{self.keep} of {self.groups} groups over {self.outputs} experts, {self.top} chosen")
+
+    @property
+    def outputs(self) -> int:
+        """Of the router, the shared expert's gate not counted."""
+        return self.experts + self.identity
 
     @property
     def ff_pad(self) -> int:
-        return pad8(self.ff)
+        return (self.ff + 31) // 32 * 32 if self.gated else pad8(self.ff)
+
+    @property
+    def up_cols(self) -> int:
+        """Columns of an expert's first matrix (gated: 32 of the gate and 32 of up in turn)."""
+        return 2 * self.ff_pad if self.gated else self.ff_pad
 
     @property
     def shared_pad(self) -> int:
         return pad8(self.shared_ff)
+
+    def gate_and_up(self, up: torch.Tensor) -> torch.Tensor:
+        """View [.., ff_pad / 32, (gate, up), 32] of a gated first matrix."""
+        return up.view(*up.shape[:-1], self.ff_pad // 32, 2, 32)
 
     @property
     def per_token(self) -> int:
@@ -207,7 +351,7 @@ class ExpertsSpec:
 
     @property
     def router_cols(self) -> int:
-        return pad8(self.experts + bool(self.shared_ff))
+        return pad8(self.outputs + bool(self.shared_ff))
 
 
 @dataclass(frozen=True)
@@ -215,10 +359,20 @@ class LayerSpec:
     mixer: Mixer
     ff: int = 0                   # width of the gated feed-forward beside the mixer; 0: none
     moe: Optional[ExpertsSpec] = None   # experts behind the mixer, with a norm of their own
+    ff_after: int = 0             # width of a gated feed-forward behind the mixer, with a norm of its own; 0: none
 
     def __post_init__(self):
-        if self.ff and self.moe:
-            raise ValueError("a layer has a feed-forward beside its mixer or experts behind it, not both")
+        if bool(self.ff) + bool(self.moe) + bool(self.ff_after) > 1:
+            raise ValueError("a layer has a feed-forward beside its mixer, one behind it, or experts behind it")
+
+    @property
+    def sublayers(self) -> Tuple[int, ...]:
+        """Numbers of the parts with a norm of their own."""
+        return (1, 2) if self.moe or self.ff_after else (1,)
+
+    @property
+    def ff_after_pad(self) -> int:
+        return pad8(self.ff_after)
 
     def in_columns(self) -> Tuple[Dict[str, Tuple[int, int]], int]:
         return _columns(self.mixer.projections())
@@ -267,6 +421,8 @@ class HybridConfig:
     norm_offset: float = 1.0      # added to the stored norm weights (1: they are stored around zero)
     logit_softcap: float = 0.0    # logits become cap * tanh(logits / cap); 0: none
     tied: bool = True             # the head is the embedding table
+    norm: str = "rms"             # "tanh": the dynamic-tanh norm, tanh(alpha x) w + b
+    streams: int = 0              # residual streams joined by learned coefficients; 0: one, with plain sums
     design: str = "fafudra"       # module of this package that maps checkpoint names (weights of a folder)
     family = "hybrid"
 
@@ -282,6 +438,14 @@ class HybridConfig:
             if any(getattr(src, n) != getattr(s.mixer, n) for n in same):
                 raise ValueError(f"{self.name}: layers {j} and {i} share keys and values but differ in {', '.join(same)}")
         lp = self.loop
+        if self.norm not in ("rms", "tanh") or (self.norm == "tanh") != (self.streams > 0):
+            raise ValueError(f"{self.name}: the dynamic-tanh norm and several streams come together")
+        if not 0 <= self.streams <= 8:
+            raise ValueError(f"{self.name}: at most 8 streams")
+        if self.streams and (lp is not None or any(s.ff or (s.moe and s.moe.shared_ff) for s in self.layer_specs)):
+            raise ValueError(f"{self.name}: streams go with layers that run once, feed-forwards behind the mixer and no shared expert")
+        if not self.streams and (any(s.ff_after for s in self.layer_specs) or any(s.moe and s.moe.identity for s in self.layer_specs)):
+            raise ValueError(f"{self.name}: feed-forwards behind the mixer and identity experts go with streams")
         if lp is not None and not (0 <= lp.start < lp.stop <= len(self.layer_specs) and lp.times >= 1):
             raise ValueError(f"{self.name}: loop of layers {lp.start}..{lp.stop} x {lp.times} does not fit "
                              f"{len(self.layer_specs)} layers")
@@ -315,7 +479,8 @@ class HybridConfig:
         return out
 
     def kv_bytes_per_token(self, tp: int = 1, elem: int = 2) -> int:
-        return sum(m.kv_heads * (m.dim + m.vdim) * elem for m in self.run_mixers() if m.kind == "attention" and m.kv_from is None)
+        per = lambda m: m.width if m.kind == "latent" else m.kv_heads * (m.dim + m.vdim) if m.kv_from is None else 0
+        return sum(per(m) * elem for m in self.run_mixers() if m.kind in PAGED)
 
     def state_bytes_per_sequence(self, elem: int = 2) -> int:
         n = 0
@@ -329,15 +494,15 @@ class HybridConfig:
     def attention_work(self, length: int) -> Tuple[int, int]:
         """(KV heads, positions) of the attention run with the fewest heads and of the one that looks furthest back, for a
         sequence of `length` tokens: what the number of key splits is chosen from.  (0, 0) without attention."""
-        a = [m for m in self.run_mixers() if m.kind == "attention"]
+        a = [m for m in self.run_mixers() if m.kind in PAGED]
         if not a:
             return 0, 0
-        span = max(min(length, m.window + m.keep_first) if m.window else length for m in a)
+        span = max(min(length, m.window + m.keep_first) if getattr(m, "window", 0) else length for m in a)
         return min(m.kv_heads for m in a), span
 
     @property
     def recurrent(self) -> bool:
-        return any(m.kind != "attention" for m in self.run_mixers())
+        return any(m.kind not in PAGED for m in self.run_mixers())
 
     @property
     def vocab_pad(self) -> int:
@@ -346,7 +511,23 @@ class HybridConfig:
     def init_(self, name: str, v: torch.Tensor, rand) -> None:
         """Random weights with activations of order one; `rand(shape)` gives normal numbers on v's device."""
         leaf = name.rsplit(".", 1)[-1]
-        if leaf in ("norm1", "norm2", "final_norm"):
+        if leaf.endswith("norm_alpha") or leaf in ("norm1_alpha", "norm2_alpha"):
+            x = 0.7 + 0.1 * rand(v.shape)
+        elif leaf in ("norm1_b", "norm2_b", "final_norm_b", "rel", "correction"):
+            x = 0.1 * rand(v.shape)
+        elif leaf in ("hc1_in", "hc2_in"):
+            x = 1.0 / v.numel() + 0.2 * rand(v.shape)
+        elif leaf in ("hc1_out", "hc2_out"):
+            x = 1.0 + 0.2 * rand(v.shape)
+        elif leaf in ("hc1_mix", "hc2_mix"):
+            x = torch.eye(v.shape[0], device=v.device) + 0.1 * rand(v.shape)
+        elif leaf in ("q_norm", "k_norm", "dq_norm", "dkv_norm"):
+            x = 1.0 + 0.1 * rand(v.shape)
+        elif leaf == "uk":                                   # stacked by head: [heads * dim, rank], the rank is the input
+            x = rand(v.shape) * v.shape[1] ** -0.5
+        elif leaf == "uv":
+            x = rand(v.shape) * (v.shape[0] // self.layer_specs[int(name.split(".")[1])].mixer.heads) ** -0.5
+        elif leaf in ("norm1", "norm2", "final_norm"):
             x = 1.0 - self.norm_offset + 0.1 * rand(v.shape)
         elif leaf == "o_norm":
             x = 1.0 + 0.1 * rand(v.shape)
@@ -356,7 +537,7 @@ class HybridConfig:
             x = -4.0 + rand(v.shape)                         # a between about 0.8 and 0.99
         elif leaf in ("x_b", "y_b", "conv_b", "gate_b", "sink", "loop_step", "q_b", "k_b", "v_b"):
             x = 0.2 * rand(v.shape)
-        elif leaf in ("up", "down"):                         # experts stacked along their inputs
+        elif leaf in ("up", "down") and self.layer_specs[int(name.split(".")[1])].moe:   # experts stacked along their inputs
             moe = self.layer_specs[int(name.split(".")[1])].moe
             n = v.shape[0] // moe.experts
             for e in range(moe.experts):
@@ -372,6 +553,12 @@ class HybridConfig:
             x = rand(v.shape) * v.shape[0] ** -0.5
         v.copy_(x.to(v.dtype))
 
+    def derive_(self, tensors) -> None:
+        """Fill the tensors that are other forms of stored ones (name -> tensor); every way of filling a segment ends here."""
+        for l, s in enumerate(self.layer_specs):
+            if hasattr(s.mixer, "derive_"):
+                s.mixer.derive_(lambda n, l=l: tensors[f"layers.{l}.{n}"])
+
     def zero_padding_(self, tensors) -> None:
         """Clear the padding columns and rows of a filled segment (name -> tensor)."""
         tensors["lm_head"][:, self.vocab:] = 0
@@ -385,13 +572,20 @@ class HybridConfig:
             o[s.mixer.out_width:s.mix_rows] = 0
             if s.ff:
                 o[s.mix_rows + s.ff:] = 0
+            if s.ff_after:
+                tensors[p + "down"][s.ff_after:] = 0
+            n, pad = (s.ff, s.ff_pad) if s.ff else (s.ff_after, s.ff_after_pad)
+            if n:
                 g = tensors[p + "gate_up"]
-                g[:, s.ff:s.ff_pad] = 0
-                g[:, s.ff_pad + s.ff:] = 0
+                g[:, n:pad] = 0
+                g[:, pad + n:] = 0
             if s.moe:
                 e = s.moe
-                tensors[p + "router"][:, e.experts + bool(e.shared_ff):] = 0
-                tensors[p + "up"][:, e.ff:] = 0
+                tensors[p + "router"][:, e.outputs + bool(e.shared_ff):] = 0
+                if not e.gated:
+                    tensors[p + "up"][:, e.ff:] = 0
+                elif e.ff % 32:
+                    e.gate_and_up(tensors[p + "up"])[:, -1, :, e.ff % 32:] = 0
                 tensors[p + "down"].view(e.experts, e.ff_pad, self.hidden)[:, e.ff:] = 0
                 if e.shared_ff:
                     tensors[p + "shared_up"][:, e.shared_ff:] = 0
@@ -412,6 +606,12 @@ def build_hybrid_layout(cfg: HybridConfig, tp: int = 1, elem_bytes: int = 2) -> 
         lay.tensors[name] = TensorSpec(name, tuple(shape), cur, n)
         cur = _align(cur + n)
 
+    def add_norm(name):
+        add(name, (cfg.hidden,))
+        if cfg.norm == "tanh":
+            add(name + "_b", (cfg.hidden,))
+            add(name + "_alpha", (1,))
+
     start = cur
     add("embed", (cfg.vocab, cfg.hidden))
     if cfg.loop is not None:
@@ -419,7 +619,7 @@ def build_hybrid_layout(cfg: HybridConfig, tp: int = 1, elem_bytes: int = 2) -> 
     lay.units.append(("embed", start, cur - start))
     for l, s in enumerate(cfg.layer_specs):
         start, p = cur, f"layers.{l}."
-        add(p + "norm1", (cfg.hidden,))
+        add_norm(p + "norm1")
         add(p + "in", (cfg.hidden, s.in_columns()[1]))
         for n, shape in s.mixer.tensors():
             add(p + n, shape)
@@ -428,16 +628,26 @@ def build_hybrid_layout(cfg: HybridConfig, tp: int = 1, elem_bytes: int = 2) -> 
             add(p + "gate_up", (cfg.hidden, 2 * s.ff_pad))
         if s.moe:
             e = s.moe
-            add(p + "norm2", (cfg.hidden,))
+            add_norm(p + "norm2")
             add(p + "router", (cfg.hidden, e.router_cols))
-            add(p + "up", (e.experts * cfg.hidden, e.ff_pad))
+            if e.correction:
+                add(p + "correction", (e.outputs,))
+            add(p + "up", (e.experts * cfg.hidden, e.up_cols))
             add(p + "down", (e.experts * e.ff_pad, cfg.hidden))
             if e.shared_ff:
                 add(p + "shared_up", (cfg.hidden, e.shared_pad))
                 add(p + "shared_down", (e.shared_pad, cfg.hidden))
+        if s.ff_after:
+            add_norm(p + "norm2")
+            add(p + "gate_up", (cfg.hidden, 2 * s.ff_after_pad))
+            add(p + "down", (s.ff_after_pad, cfg.hidden))
+        if cfg.streams:
+            for q in s.sublayers:
+                for n, shape in (("in", (cfg.streams,)), ("out", (cfg.streams,)), ("mix", (cfg.streams, cfg.streams))):
+                    add(f"{p}hc{q}_{n}", shape)
         lay.units.append((f"layer.{l}", start, cur - start))
     start = cur
-    add("final_norm", (cfg.hidden,))
+    add_norm("final_norm")
     add("lm_head", (cfg.hidden, cfg.vocab_pad))
     lay.units.append(("head", start, cur - start))
     lay.total_bytes = cur

@@ -89,6 +89,7 @@ class WeightSegment:
         if self.cfg.tied:
             self._views["lm_head"][:, :self.cfg.vocab].copy_(self._views["embed"].t())
         self.cfg.zero_padding_(self._views)
+        self.cfg.derive_(self._views)
         return self
 
     def save(self, directory) -> Path:

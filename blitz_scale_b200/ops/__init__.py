@@ -57,16 +57,31 @@ class KVPair(NamedTuple):
     v: torch.Tensor
 
 
-KVLayer = Union[torch.Tensor, KVPair]
+class LatentKV(NamedTuple):
+    """Paged cache of a latent attention layer: [pages, page, 1, rank + rotated dimensions].  A row is the key of every head,
+    its first ``rank`` columns the value of every head, before the heads' own projections."""
+    pool: torch.Tensor
+    rank: int
+
+
+KVLayer = Union[torch.Tensor, KVPair, LatentKV]
 
 
 def _kv(kv: KVLayer):
     """(key pool, value pool, rows per page in the pools, pages, value size)"""
+    if isinstance(kv, LatentKV):
+        assert kv.pool.is_contiguous()
+        return _p(kv.pool), _p(kv.pool), kv.pool.shape[1], kv.pool.shape[0], kv.rank
     if isinstance(kv, KVPair):
         assert kv.k.is_contiguous() and kv.v.is_contiguous() and kv.k.shape[:3] == kv.v.shape[:3]
         return _p(kv.k), _p(kv.v), kv.k.shape[1], kv.k.shape[0], kv.v.shape[3]
     assert kv.is_contiguous()
     return _p(kv), ctypes.c_void_p(kv.data_ptr() + kv.stride(1) * kv.element_size()), 2 * kv.shape[2], kv.shape[0], kv.shape[4]
+
+
+def _bias(bias: Optional[torch.Tensor], q_heads: int):
+    assert bias is None or (bias.is_contiguous() and bias.dim() == 2 and bias.shape[0] == q_heads)
+    return _p(bias), 0 if bias is None else bias.shape[1]
 
 
 def _gate(gate: Optional[torch.Tensor]):
@@ -145,7 +160,7 @@ def _tensor_core_operands(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, N
 
 
 def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *, residual=None,
-         epilogue: str = "store", alpha: float = 1.0, groups: int = 1, b_layout: str = "kn", bn: int = 0, split_k: int = 0, static_b: bool = False,
+         epilogue: str = "store", alpha: float = 1.0, groups: int = 1, a_step: int = 0, out_step: int = 0, b_layout: str = "kn", bn: int = 0, split_k: int = 0, static_b: bool = False,
          decode_path: Optional[bool] = None, decode_split: int = 0, pair_path: Optional[bool] = None,
          pair_bnf: int = 0, pair_upp: int = 0, pair_nacc: int = 0) -> torch.Tensor:
     """``out = a @ b`` on tcgen05 with a fused epilogue.
@@ -168,14 +183,17 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *
     ``out`` may be fp32 with 16-bit operands (the accumulator is stored unrounded); epilogue 'axpy' adds
     ``alpha * (a @ b)`` to an fp32 ``out`` (residual streams kept in 32 bits); 'softcap' stores
     ``alpha * tanh((a @ b) / alpha)`` in fp32 (logits).  ``groups`` > 1: block-diagonal product,
-    a [M, groups * K], b [groups * K, N] (the blocks stacked), out [M, groups * N].  fp32 operands, and 16-bit ones
+    a [M, groups * K], b [groups * K, N] (the blocks stacked), out [M, groups * N]; ``a_step`` / ``out_step``: columns from a
+    group to the next one in a and out, where the blocks' columns are parts of wider ones.  fp32 operands, and 16-bit ones
     whose sizes the tensor-core kernels do not take, run on the CUDA cores in fp32 arithmetic.
     """
     assert a.is_cuda and a.dim() == 2 and b.dim() == 2 and a.stride(1) == 1 and b.stride(1) == 1
     M, K = a.shape
-    if groups > 1:
-        assert K % groups == 0 and epilogue == "store" and b_layout == "kn" and b.shape[0] == K
-        K //= groups
+    if groups > 1 or a_step or out_step:
+        assert b.shape[0] % groups == 0 and epilogue == "store" and b_layout == "kn"
+        K = b.shape[0] // groups
+        a_step, out_step = a_step or K, out_step or b.shape[1]
+        assert a_step * (groups - 1) + K <= a.shape[1] and out_step >= b.shape[1]
     if b_layout == "kn":
         assert b.shape[0] == K * groups
         bcols = b.shape[1]
@@ -186,7 +204,8 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *
     N = bcols // 2 if epi == 2 else bcols
     if out is None:
         out = torch.empty((M, groups * N), dtype=a.dtype, device=a.device)
-    assert out.shape == (M, groups * N) and out.stride(1) == 1
+    assert out.stride(1) == 1 and out.shape[0] == M
+    assert out.shape[1] >= out_step * (groups - 1) + N if out_step else out.shape[1] == N
     if epi in (5, 6):
         assert out.dtype == torch.float32
     elif out.dtype != a.dtype:
@@ -194,12 +213,12 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *
         epi = _EPI_STORE_F32
     if M == 0:
         return out
-    if a.dtype == torch.float32 or (groups > 1 and K % 64) or not _tensor_core_operands(a, b, out, N, K):
+    if a.dtype == torch.float32 or (a_step | out_step) % 8 or not _tensor_core_operands(a, b, out, N, K):
         if epi == 1 or b_layout != "kn":
             raise TypeError("gemm: epilogue 'add' and 'nk' weights need the tensor-core kernels")
         assert b.dtype == a.dtype
         _check(lib().blitz_gemm_simt(_p(a), a.stride(0), _p(b), b.stride(0), _p(out), out.stride(0), M, N, K, epi,
-                                     N if epi == 2 else 0, alpha, groups, _dt3(a), _stream()), "blitz_gemm_simt")
+                                     N if epi == 2 else 0, alpha, groups, a_step, out_step, _dt3(a), _stream()), "blitz_gemm_simt")
         return out
     if epi == 1:
         assert residual is not None and residual.shape == (M, N) and residual.stride(0) == out.stride(0)
@@ -233,7 +252,7 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *
     rc = lib().blitz_gemm(_p(a), a.stride(0), _p(b), b.stride(0), _p(out), out.stride(0), _p(residual), M, N, K,
                           0 if b_layout == "kn" else 1, epi, N if epi == 2 else 0, _dt(a), bn, split_k,
                           _p(ws), ws.numel(), _p(tickets), tickets.numel(), _p(status_word(a.device)), alpha,
-                          groups, _stream())
+                          groups, a_step, out_step, _stream())
     _check(rc, "blitz_gemm")
     return out
 
@@ -335,11 +354,13 @@ def attn_decode(q: torch.Tensor, kv_layer: KVLayer, indices: torch.Tensor, indpt
                 last_page_len: torch.Tensor, *, q_heads: int, kv_heads: int, head_dim: int, page_size: int,
                 num_splits: int = 1, workspace: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
                 sm_scale: Optional[float] = None, window: int = 0, keep_first: int = 0, softcap: float = 0.0,
-                sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """q: [batch, >= q_heads*head_dim] (row pitch free, e.g. a view of the fused qkv buffer).  ``window`` > 0: only the
     last that many positions and the first ``keep_first`` are visible (and read); ``softcap`` > 0:
     scores are cap * tanh(score / cap); ``sink`` [q_heads]: a term e^sink in the softmax denominator; ``gate``
-    [batch, q_heads]: a head's output is multiplied by its sigmoid.  Values may have a size of their own (KVPair)."""
+    [batch, q_heads]: a head's output is multiplied by its sigmoid; ``bias`` [q_heads, n]: added to the scaled scores by the
+    key's distance, the last column for all longer ones.  Values may have a size of their own (KVPair)."""
     B = indptr.numel() - 1
     kp, vp, page_rows, pages, vdim = _kv(kv_layer)
     if out is None:
@@ -351,15 +372,19 @@ def attn_decode(q: torch.Tensor, kv_layer: KVLayer, indices: torch.Tensor, indpt
         sm_scale = head_dim ** -0.5
     _check(lib().blitz_attn_decode(_p(q), q.stride(0), kp, vp, _p(indices), _p(indptr), _p(last_page_len),
                                    _p(out), out.stride(0), _p(workspace), B, q_heads, kv_heads, head_dim, vdim, page_size,
-                                   page_rows, pages, num_splits, sm_scale, window, keep_first, softcap, _p(sink), *_gate(gate),
+                                   page_rows, pages, num_splits, sm_scale, window, keep_first, softcap, _p(sink), *_bias(bias, q_heads), *_gate(gate),
                                    _p(status_word(q.device)), _dt(q), _stream()), "blitz_attn_decode")
     return out
 
 
 def attn_tensor_core(q: torch.Tensor, q_heads: int, kv_heads: int, head_dim: int, page_size: int, value_dim: int = 0) -> bool:
     """Whether attn_decode and attn_prefill_paged take these head sizes (attn_ragged takes every one)."""
-    return (q.dtype in _DT and all(8 <= d <= 128 and d % 8 == 0 for d in (head_dim, value_dim or head_dim)) and page_size >= 8
-            and page_size & (page_size - 1) == 0 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0)
+    return (q.dtype in _DT and attn_head_sizes(head_dim, value_dim or head_dim, page_size) and q.stride(0) % 8 == 0
+            and q.data_ptr() % 16 == 0)
+
+
+def attn_head_sizes(head_dim: int, value_dim: int, page_size: int) -> bool:
+    return all(8 <= d <= 128 and d % 8 == 0 for d in (head_dim, value_dim)) and page_size >= 8 and page_size & (page_size - 1) == 0
 
 
 def prefill_work_list(q_lens, kv_lens, page_size: int, device, skip: int = 0) -> torch.Tensor:
@@ -385,11 +410,12 @@ def attn_prefill_paged(q: torch.Tensor, kv_layer: KVLayer, page_indices: torch.T
                        q_heads: int, kv_heads: int, head_dim: int, page_size: int, out: Optional[torch.Tensor] = None,
                        sm_scale: Optional[float] = None, poly_exp: bool = False, window: int = 0, keep_first: int = 0,
                        softcap: float = 0.0, sink: Optional[torch.Tensor] = None,
-                       gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                       gate: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of the pass's rows over the paged cache (which already holds the rows' own keys and values,
     after whatever earlier passes stored).  ``q``: rotated query columns, e.g. the fused qkv buffer (rope_kv_store);
     ``page_indices``: the sequences' page ids back to back, covering prefix + rows; ``work`` from `prefill_work_list`
-    for the same sequences.  ``window`` / ``keep_first`` / ``softcap`` / ``sink`` / ``gate`` as for `attn_decode`."""
+    for the same sequences.  ``window`` / ``keep_first`` / ``softcap`` / ``sink`` / ``gate`` / ``bias`` as for `attn_decode`
+    (no bias beside a window, cap or sink)."""
     T = q.shape[0]
     kp, vp, page_rows, pages, vdim = _kv(kv_layer)
     if out is None:
@@ -400,7 +426,7 @@ def attn_prefill_paged(q: torch.Tensor, kv_layer: KVLayer, page_indices: torch.T
     _check(lib().blitz_attn_prefill_paged(_p(q), q.stride(0), kp, vp, _p(out), out.stride(0), _p(page_indices),
                                           _p(work), work.shape[0], T, q_heads, kv_heads, head_dim, vdim, page_size, page_rows,
                                           pages, sm_scale, 1 if poly_exp else 0, window, keep_first, softcap, _p(sink),
-                                          *_gate(gate), _p(status_word(q.device)), _dt(q), _stream()), "blitz_attn_prefill_paged")
+                                          *_bias(bias, q_heads), *_gate(gate), _p(status_word(q.device)), _dt(q), _stream()), "blitz_attn_prefill_paged")
     return out
 
 
@@ -460,33 +486,123 @@ def rope_store(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Ten
 def attn_ragged(q: torch.Tensor, kv_layer: KVLayer, pos: torch.Tensor, tok_indptr: Optional[torch.Tensor],
                 page_indptr: torch.Tensor, page_indices: torch.Tensor, out: torch.Tensor, *, q_heads: int, kv_heads: int,
                 dim: int, page_size: int, scale: float, window: int = 0, keep_first: int = 0, softcap: float = 0.0,
-                sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """General paged attention (CUDA cores, any head sizes, any element type); see csrc/kernels/attn_ragged.cu.  ``gate``
-    [T, q_heads]: a head's output is multiplied by its sigmoid."""
+    [T, q_heads]: a head's output is multiplied by its sigmoid; ``bias`` as for `attn_decode`."""
     T = q.shape[0]
     rows = page_indptr.numel() - 1
     assert q.stride(1) == 1 and out.stride(1) == 1
     kp, vp, page_rows, pages, vdim = _kv(kv_layer)
     _check(lib().blitz_attn_ragged(_p(q), q.stride(0), kp, vp, _p(out), out.stride(0), _p(pos), _p(tok_indptr),
-                                   _p(page_indptr), _p(page_indices), _p(sink), *_gate(gate), T, rows, q_heads, kv_heads, dim, vdim,
+                                   _p(page_indptr), _p(page_indices), _p(sink), *_bias(bias, q_heads),
+                                   kv_layer.pool.shape[3] if isinstance(kv_layer, LatentKV) else vdim, *_gate(gate), T, rows,
+                                   q_heads, kv_heads, dim, vdim,
                                    page_size, page_rows, pages, window, keep_first, scale, softcap, _p(status_word(q.device)),
                                    _dt3(q), _stream()), "blitz_attn_ragged")
+    return out
+
+
+def stream_mix(x: torch.Tensor, *, n: Optional[int] = None, ids: Optional[torch.Tensor] = None, embed: Optional[torch.Tensor] = None,
+               pending: Optional["Pending"] = None, read: Optional[torch.Tensor] = None, norm: Optional[Sequence[torch.Tensor]] = None,
+               out: Optional[torch.Tensor] = None, total: Optional[torch.Tensor] = None, write: bool = False,
+               rows: Optional[torch.Tensor] = None, row_offset: int = 0) -> None:
+    """Between two sublayers of a model with several residual streams (``x`` [T, streams, hidden] fp32), in one kernel.
+
+    ``embed`` (with ``ids``): every stream is the token's embedding, x is not read.  ``pending``: the last sublayer's output,
+    which the streams take up first (``write``: and keep).  Then u = sum_s read[s] x_s (None: the plain sum); ``total``
+    receives u (fp32), ``out`` receives tanh(alpha u) w + b with ``norm`` = (w, alpha, b).  ``rows``: result t comes from
+    token rows[t] + row_offset."""
+    T, S, H = x.shape
+    n = n if n is not None else (rows.numel() if rows is not None else T)
+    assert x.dtype == torch.float32 and x.is_contiguous() and (out is None or (norm is not None and out.is_contiguous()))
+    assert total is None or (total.dtype == torch.float32 and total.is_contiguous())
+    w, alpha, b = norm if out is not None else (None, None, None)
+    ref = embed if embed is not None else out if out is not None else pending.y if pending is not None else read
+    if ref is None:
+        ref = torch.empty(0, dtype=torch.bfloat16)        # a plain sum of fp32 streams
+    pd = pending if pending is not None else Pending(None, None, None)
+    assert pd.y is None or (pd.y.stride(1) == 1 and pd.y.stride(0) == H)
+    _check(lib().blitz_stream_mix(_p(ids), _p(embed), embed.shape[0] if embed is not None else 0, int(embed is not None), _p(x), _p(pd.y),
+                                  _p(pd.place), pd.place.shape[1] if pd.place is not None else 0, _p(pd.ident), _p(pd.prev), _p(pd.mix),
+                                  _p(pd.out), _p(read), _p(alpha), _p(w), _p(b), _p(rows), row_offset, _p(out), _p(total), int(write),
+                                  n, H, S, _p(status_word(x.device)), _dt3(ref), _stream()), "blitz_stream_mix")
+
+
+class Pending(NamedTuple):
+    """Output of a sublayer that the streams have not taken up: ``y`` [T, hidden], or rows that ``place`` [T, n] names (-1: none),
+    with ``ident`` [T] times ``prev`` [T, hidden] on top; the coefficients ``mix`` [streams, streams] and ``out`` [streams]."""
+    y: Optional[torch.Tensor]
+    mix: Optional[torch.Tensor]
+    out: Optional[torch.Tensor]
+    place: Optional[torch.Tensor] = None
+    ident: Optional[torch.Tensor] = None
+    prev: Optional[torch.Tensor] = None
+
+
+def norm_store(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor, kv_layer: KVLayer,
+               q_w: torch.Tensor, k_w: torch.Tensor, *, q_heads: int, kv_heads: int, dim: int, page_size: int, eps: float,
+               temp_coef: float = 0.0, temp_every: int = 0) -> None:
+    """RMSNorm of every query head (in place, times a temperature that grows with the position) and key head; keys and values go
+    to the paged cache.  q, k, v: column ranges of one projection."""
+    T = q.shape[0]
+    assert all(x.stride(0) == q.stride(0) and x.stride(1) == 1 for x in (q, k, v))
+    kp, vp, page_rows, pages, vdim = _kv(kv_layer)
+    _check(lib().blitz_norm_store(_p(q), _p(k), _p(v), q.stride(0), _p(q_w), _p(k_w), eps, temp_coef, temp_every, _p(pos), _p(slot),
+                                  kp, vp, T, q_heads, kv_heads, dim, vdim, page_size, page_rows, pages, _p(status_word(q.device)),
+                                  _dt3(q), _stream()), "blitz_norm_store")
+
+
+# ---------------------------------------------------------------------------------------------- latent attention
+def latent_store(cq: Optional[torch.Tensor], ckv: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor, kv: LatentKV,
+                 cq_w: Optional[torch.Tensor], ckv_w: torch.Tensor, freqs: torch.Tensor, *, eps: float) -> None:
+    """RMSNorm of the queries' latent (in place) and of the keys' latent (to the cache), and the rotated key part (to the
+    cache).  cq, ckv: column ranges of one projection."""
+    T = ckv.shape[0]
+    pages, page, _, width = kv.pool.shape
+    assert ckv.shape[1] == width and ckv.stride(1) == 1 and (cq is None or (cq.stride(0) == ckv.stride(0) and cq.stride(1) == 1))
+    _check(lib().blitz_latent_store(_p(cq), _p(ckv), ckv.stride(0), _p(cq_w), _p(ckv_w), _p(pos), _p(slot), _p(kv.pool), _p(freqs), eps,
+                                    T, cq.shape[1] if cq is not None else 0, kv.rank, width - kv.rank, page, pages,
+                                    _p(status_word(ckv.device)), _dt3(ckv), _stream()), "blitz_latent_store")
+
+
+def latent_rotate(q: torch.Tensor, out: torch.Tensor, pos: torch.Tensor, freqs: torch.Tensor, *, heads: int, dim: int, rot: int,
+                  out_step: int) -> None:
+    """Rotate the last ``rot`` dimensions of every head of q [T, heads * (dim + rot)]; head h's go to columns h * out_step on of
+    ``out`` (which may be a view of q: in place)."""
+    assert q.stride(1) == 1 and out.stride(1) == 1 and q.shape[1] == heads * (dim + rot)
+    _check(lib().blitz_latent_rotate(_p(q), q.stride(0), _p(out), out.stride(0), out_step, _p(pos), _p(freqs), q.shape[0], heads, dim,
+                                     rot, _dt3(q), _stream()), "blitz_latent_rotate")
+
+
+def latent_gather(kv: LatentKV, pages: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """The rows of the named pages, back to back: out [pages * page, width]."""
+    n, page, width = pages.numel(), kv.pool.shape[1], kv.pool.shape[3]
+    assert out.is_contiguous() and out.shape == (n * page, width) and pages.dtype == torch.int32
+    _check(lib().blitz_latent_gather(_p(kv.pool), _p(pages), _p(out), n, page * width * out.element_size(), kv.pool.shape[0],
+                                     _p(status_word(out.device)), _stream()), "blitz_latent_gather")
     return out
 
 
 # ---------------------------------------------------------------------------------------------- mixture of experts
 class ExpertPlan:
     """Work list of the grouped products of a step, in buffers for up to ``max_tokens`` tokens (see csrc/kernels/moe_route.cu):
-    filled by `moe_route` on the device, read by `gemm_grouped` and by `stream_norm` (``place``)."""
+    filled by `moe_route` on the device, read by `gemm_grouped` and by `stream_norm` or `stream_mix` (``place``: -1 where a
+    token chose an identity expert, whose weights are summed in ``ident``)."""
 
-    def __init__(self, max_tokens: int, experts: int, top: int, shared: bool, device):
+    def __init__(self, max_tokens: int, experts: int, top: int, shared: bool, device, identity: int = 0):
         i32 = lambda *shape: torch.zeros(*shape, dtype=torch.int32, device=device)
         self.experts, self.top, self.shared, self.max_tokens = experts, top, int(shared), max_tokens
         rows = max_tokens * (top + self.shared)
         self.pairs, self.counters, self.num_tiles = i32(max_tokens * top, 2), i32(2 * experts + 1), i32(1)
         self.src, self.factors = i32(rows), torch.zeros(rows, 2, dtype=torch.float32, device=device)
         self._place, self._tiles = i32(rows), i32(self.tiles_at_most(max_tokens, 64), 4)
+        self.identity, self._ident = identity, torch.zeros(max_tokens, dtype=torch.float32, device=device) if identity else None
         self.tokens, self.tile_rows = 0, 128
+
+    @property
+    def ident(self) -> Optional[torch.Tensor]:
+        return None if self._ident is None else self._ident[:self.tokens]
 
     def tiles_at_most(self, tokens: int, tile_rows: int) -> int:
         pairs = tokens * self.top
@@ -502,26 +618,31 @@ class ExpertPlan:
 
     def tiles_usually(self):
         """(tiles, rows of one) of an even spread over the experts."""
-        pairs = self.tokens * self.top
+        pairs = self.tokens * self.top * self.experts // (self.experts + self.identity)
         used = max(1, round(self.experts * (1.0 - (1.0 - 1.0 / self.experts) ** pairs)))
-        return used + max(0, pairs - used * self.tile_rows // 2) // self.tile_rows, min(self.tile_rows, -(-pairs // used))
+        return used + max(0, pairs - used * self.tile_rows // 2) // self.tile_rows, min(self.tile_rows, max(1, -(-pairs // used)))
 
 
 def moe_route(logits: torch.Tensor, plan: ExpertPlan, *, weight_on_input: bool = True, renormalize: bool = False,
+              softmax: bool = False, correction: Optional[torch.Tensor] = None, groups: int = 0, keep: int = 0,
               tile_rows: int = 128) -> ExpertPlan:
-    """Choose experts from fp32 router logits [T, experts (+ 1: gate of the shared expert)] and sort the rows by expert."""
+    """Choose experts from fp32 router logits [T, experts (+ identity experts, or + 1: gate of the shared expert)] and sort the
+    rows by expert.  ``softmax``: scores are a softmax over all outputs (else sigmoids); ``correction``: added to the scores
+    the choice is made by; ``groups``: only experts of the best ``keep`` of so many equal groups can be chosen."""
     T = logits.shape[0]
-    assert logits.dtype == torch.float32 and logits.stride(1) == 1 and logits.shape[1] >= plan.experts + plan.shared
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1 and logits.shape[1] >= plan.experts + plan.identity + plan.shared
+    assert correction is None or (correction.is_contiguous() and correction.numel() == plan.experts + plan.identity)
     assert T <= plan.max_tokens and tile_rows >= 64
     plan.tokens, plan.tile_rows = T, tile_rows
     _check(lib().blitz_moe_route(_p(logits), logits.stride(0), T, plan.experts, plan.top, plan.shared, int(weight_on_input),
-                                 int(renormalize), tile_rows, plan.tiles_at_most(T, tile_rows), _p(plan.pairs), _p(plan.counters),
+                                 int(renormalize), plan.identity, int(softmax), groups, keep, _p(correction),
+                                 0 if correction is None else _dt3(correction), _p(plan._ident), tile_rows, plan.tiles_at_most(T, tile_rows), _p(plan.pairs), _p(plan.counters),
                                  _p(plan.src), _p(plan.factors), _p(plan._place), _p(plan._tiles), _p(plan.num_tiles),
                                  _p(status_word(logits.device)), _stream()), "blitz_moe_route")
     return plan
 
 
-_ACT = {"none": 0, "relu2": 1}
+_ACT = {"none": 0, "relu2": 1, "silu_gate": 2}
 
 
 def grouped_tensor_core(a: torch.Tensor, *matrices: Optional[torch.Tensor]) -> bool:
@@ -534,13 +655,15 @@ def gemm_grouped(a: torch.Tensor, b: torch.Tensor, plan: ExpertPlan, out: torch.
                  gather: bool = False, act: str = "none", factors: bool = False, bn: int = 0, fetch: int = 0) -> torch.Tensor:
     """out[r] = after_r * act(before_r * (a[row] @ b[expert of r])) for the plan's sorted rows r; ``b`` [experts, K, N];
     ``shared`` [K', N']: the shared expert's matrix for the rows behind (K' and N' columns of a and out).  ``gather``: row r
-    reads the activation of its token, else sorted row r.  ``factors``: apply the plan's factors (else both are 1).  ``bn``
+    reads the activation of its token, else sorted row r.  ``act`` "silu_gate": b has 32 gate columns, the 32 up columns they
+    gate, and so on (`interleave_gate`), out half as many.  ``factors``: apply the plan's factors (else both are 1).  ``bn``
     forces the tile width, ``fetch`` how rows are gathered (1 TMA, 2 copying warps)."""
     E, K, N = b.shape
     assert E == plan.experts and b.is_contiguous() and a.stride(1) == 1 and out.stride(1) == 1 and a.dtype == b.dtype == out.dtype
     assert (shared is not None) == bool(plan.shared) and out.shape[0] >= plan.rows
     Ks, Ns = (K, N) if shared is None else shared.shape
-    assert a.shape[1] >= max(K, Ks) and out.shape[1] >= max(N, Ns) and (shared is None or shared.is_contiguous())
+    assert act != "silu_gate" or (shared is None and N % 64 == 0)
+    assert a.shape[1] >= max(K, Ks) and out.shape[1] >= (N // 2 if act == "silu_gate" else max(N, Ns)) and (shared is None or shared.is_contiguous())
     src, fac = plan.src if gather else None, plan.factors if factors else None
     row0, shared_rows = plan.tokens * plan.top, plan.tokens * plan.shared
     most = plan.tiles_at_most(plan.tokens, plan.tile_rows)
@@ -555,6 +678,12 @@ def gemm_grouped(a: torch.Tensor, b: torch.Tensor, plan: ExpertPlan, out: torch.
                                     *plan.tiles_usually(), row0, shared_rows, plan.tokens, _ACT[act], bn, fetch,
                                     _p(status_word(a.device)), _dt(a), _stream()), "blitz_gemm_grouped")
     return out
+
+
+def interleave_gate(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+    """[K, n] gate and up matrices (n a multiple of 32) -> [K, 2 n], 32 columns of one and of the other in turn."""
+    K, n = gate.shape
+    return torch.stack([gate.reshape(K, n // 32, 32), up.reshape(K, n // 32, 32)], 2).reshape(K, 2 * n)
 
 
 def gla_recurrent(q, k, v, g, low, a2, a2_b, norm, state: torch.Tensor, out: torch.Tensor, pos, tok_indptr, seq_slot, *,

@@ -54,7 +54,7 @@ def _declare(L: ctypes.CDLL) -> None:
             fn.restype = res
 
     sig("blitz_gemm", [c_p, c_i64, c_p, c_i64, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_i64,
-                       c_p, c_i, c_p, c_f, c_i, c_p])
+                       c_p, c_i, c_p, c_f, c_i, c_i, c_i, c_p])
     sig("blitz_gemm_workspace_bytes", [c_i], c_i64)
     sig("blitz_gemm_decode", [c_p, c_i64, c_p, c_i64, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_f,
                               c_p])
@@ -87,18 +87,25 @@ def _declare(L: ctypes.CDLL) -> None:
     sig("blitz_rope_kv_store", [c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_p, c_i, c_p])
     sig("blitz_attn_decode_workspace_bytes", [c_i, c_i, c_i, c_i], c_i64)
     sig("blitz_attn_decode", [c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f,
-                              c_i, c_i, c_f, c_p, c_p, c_i64, c_p, c_i, c_p])
+                              c_i, c_i, c_f, c_p, c_p, c_i, c_p, c_i64, c_p, c_i, c_p])
     sig("blitz_attn_prefill_paged", [c_p, c_i64, c_p, c_p, c_p, c_i64, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f,
-                                     c_i, c_i, c_i, c_f, c_p, c_p, c_i64, c_p, c_i, c_p])
+                                     c_i, c_i, c_i, c_f, c_p, c_p, c_i, c_p, c_i64, c_p, c_i, c_p])
     # models with an fp32 residual stream and recurrent layers
-    sig("blitz_gemm_simt", [c_p, c_i64, c_p, c_i64, c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_p])
+    sig("blitz_gemm_simt", [c_p, c_i64, c_p, c_i64, c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_i, c_i, c_p])
     sig("blitz_stream_norm", [c_p, c_p, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_p, c_i,
                               c_p])
     sig("blitz_rope_store", [c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_f, c_i, c_i, c_i, c_i, c_i, c_i, c_i,
                              c_i, c_i, c_i, c_p, c_i, c_p])
-    sig("blitz_attn_ragged", [c_p, c_i64, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_i,
+    sig("blitz_stream_mix", [c_p, c_p, c_i, c_i, c_p, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_p, c_p, c_i,
+                             c_i, c_i, c_i, c_p, c_i, c_p])
+    sig("blitz_norm_store", [c_p, c_p, c_p, c_i64, c_p, c_p, c_f, c_f, c_i, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i,
+                             c_p, c_i, c_p])
+    sig("blitz_latent_store", [c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_f, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_i, c_p])
+    sig("blitz_latent_rotate", [c_p, c_i64, c_p, c_i64, c_i, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_p])
+    sig("blitz_latent_gather", [c_p, c_p, c_p, c_i, c_i64, c_i, c_p, c_p])
+    sig("blitz_attn_ragged", [c_p, c_i64, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_i,
                               c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_p, c_i, c_p])
-    sig("blitz_moe_route", [c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p])
+    sig("blitz_moe_route", [c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_i, c_p, c_i, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p])
     sig("blitz_gemm_grouped", [c_p, c_i64, c_i, c_p, c_p, c_i, c_i, c_i, c_p, c_i, c_i, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i, c_i,
                                c_i, c_i, c_i, c_i, c_i, c_p, c_i, c_p])
     sig("blitz_gemm_grouped_simt", [c_p, c_i64, c_p, c_p, c_i, c_i, c_p, c_i, c_i, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i,

@@ -5,7 +5,8 @@ of every recurrent run, so the host bookkeeping (native PagePool, SlotPool and B
 are or what shape each has.  A layer that runs several times in one forward pass has one entry per run; a layer that
 reads another layer's keys and values has that layer's pool as its entry.
 
-A pool is one tensor with a key and a value plane per page, or a pair of tensors where keys and values differ in size.
+A pool is one tensor with a key and a value plane per page, or a pair of tensors where keys and values differ in size, or one
+tensor of latent rows.
 
 Slots are not cleared when they change hands: the kernels start from zero at position 0.  KV pools are zero-filled once
 (the attention kernels require finite values in every slot of an allocated page)."""
@@ -17,12 +18,13 @@ from typing import List, Optional, Union
 import torch
 
 from ..models.hybrid_config import HybridConfig
-from ..ops import KVPair
+from ..ops import KVPair, LatentKV
 
 
 @dataclass
 class RunCache:
-    kv: Optional[Union[torch.Tensor, KVPair]] = None   # [pages, 2, page, kv_heads, dim], or two [pages, page, kv_heads, size]
+    # [pages, 2, page, kv_heads, dim], or two [pages, page, kv_heads, size], or latent rows [pages, page, 1, width]
+    kv: Optional[Union[torch.Tensor, KVPair, LatentKV]] = None
     state: Optional[torch.Tensor] = None   # fp32: [slots, heads, dim, vdim] or [slots, width]
     hist: Optional[torch.Tensor] = None    # last inputs of a short convolution: [slots, taps - 1, width]
 
@@ -35,6 +37,8 @@ class HybridCache:
         for r, (m, source) in enumerate(zip(cfg.run_mixers(), cfg.kv_runs())):
             if m.kind == "attention" and source != r:
                 self.runs.append(RunCache(kv=self.runs[source].kv))
+            elif m.kind == "latent":
+                self.runs.append(RunCache(kv=LatentKV(zeros(num_pages, page_size, 1, m.width), m.kv_rank)))
             elif m.kind == "attention" and m.vdim != m.dim:
                 self.runs.append(RunCache(kv=KVPair(*(zeros(num_pages, page_size, m.kv_heads, n) for n in (m.dim, m.vdim)))))
             elif m.kind == "attention":
@@ -48,7 +52,8 @@ class HybridCache:
     def bytes(self) -> int:
         held = {}
         for r in self.runs:
-            for t in (*(r.kv if isinstance(r.kv, KVPair) else (r.kv,)), r.state, r.hist):
+            pools = r.kv if isinstance(r.kv, KVPair) else (r.kv.pool,) if isinstance(r.kv, LatentKV) else (r.kv,)
+            for t in (*pools, r.state, r.hist):
                 if t is not None:
                     held[t.data_ptr()] = t.numel() * t.element_size()
         return sum(held.values())
