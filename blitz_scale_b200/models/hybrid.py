@@ -138,6 +138,7 @@ class HybridRunner:
         self._scratch: Dict[str, torch.Tensor] = {}
         if not ms:
             return
+        self._latent_ws = max((ops.attn_latent_workspace(m.heads, m.kv_rank, dev) for m in ms), key=torch.Tensor.numel)
         rows = lambda m: max_batch if self._expands(m, dt) else max_tokens
         self._q = torch.empty(max_tokens * max(m.heads * m.qdim for m in ms), dtype=dt, device=dev)
         self._q_latent = torch.empty(max(rows(m) * m.heads * m.width for m in ms), dtype=dt, device=dev)
@@ -299,9 +300,13 @@ class HybridRunner:
             ops.gemm(q[:n], self._w(l, "uk"), out=ql, groups=H, a_step=mx.qdim, out_step=W, static_b=True)
             ops.latent_rotate(q[:n], ql[:, R:], m.pos[:n], freqs, out_step=W, **rotate)
             single = not m.is_prefill or n == m.singles
-            ops.attn_ragged(ql, kv, m.pos, None if single else m.tok_indptr, m.page_indptr[:n + 1] if single else m.page_indptr,
-                            m.page_indices, ol, q_heads=H, kv_heads=1, dim=W, page_size=self.page_size, scale=mx.scale,
-                            gate=gate[:n] if gate is not None else None)
+            g = gate[:n] if gate is not None else None
+            if single and ops.attn_latent_supported(ql, n, H, kv):
+                ops.attn_latent(ql, kv, m.page_indices, m.page_indptr[:n + 1], m.last_page_len[:n], heads=H, scale=mx.scale,
+                                workspace=self._latent_ws, out=ol, gate=g)
+            else:
+                ops.attn_ragged(ql, kv, m.pos, None if single else m.tok_indptr, m.page_indptr[:n + 1] if single else m.page_indptr,
+                                m.page_indices, ol, q_heads=H, kv_heads=1, dim=W, page_size=self.page_size, scale=mx.scale, gate=g)
             ops.gemm(ol, self._w(l, "uv"), out=mid[:n, :H * mx.vdim], groups=H, a_step=R, out_step=mx.vdim, static_b=True)
         if n < T:
             self._latent_prompts(l, mx, q, gate, kv, mid, m, n, freqs, rotate)
@@ -422,7 +427,7 @@ class HybridRunner:
 
     def decode_launches(self) -> int:
         """Kernels of this library in one decode step."""
-        per = {"attention": 2, "latent": 6, "gla": 1, "rglru": 3}
+        per = {"attention": 2, "latent": 7, "gla": 1, "rglru": 3}
         specs = [self.cfg.layer_specs[r.layer] for r in self.runs]
         n = sum(3 + per[s.mixer.kind] + bool(s.ff) + 3 * bool(s.ff_after) + 5 * bool(s.moe) for s in specs)
         return n + 3      # final norm, head product, arg-max

@@ -584,6 +584,30 @@ def latent_gather(kv: LatentKV, pages: torch.Tensor, out: torch.Tensor) -> torch
     return out
 
 
+def attn_latent_supported(q: torch.Tensor, batch: int, heads: int, kv: LatentKV) -> bool:
+    """Whether attn_latent takes these sizes (attn_ragged takes every one)."""
+    _, page, _, width = kv.pool.shape
+    return q.dtype in _DT and bool(lib().blitz_attn_latent_supported(batch, heads, width, kv.rank, page))
+
+
+def attn_latent_workspace(heads: int, rank: int, device) -> torch.Tensor:
+    return torch.empty(int(lib().blitz_attn_latent_workspace_bytes(heads, rank)), dtype=torch.uint8, device=device)
+
+
+def attn_latent(q: torch.Tensor, kv: LatentKV, indices: torch.Tensor, indptr: torch.Tensor, last_page_len: torch.Tensor, *, heads: int,
+                scale: float, workspace: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Decode attention over latent rows: q [batch, heads * width] against every cached row as it is, out [batch, heads * rank] =
+    the weighted sums of the rows' first ``rank`` columns, times the sigmoid of ``gate`` [batch, heads]."""
+    B = indptr.numel() - 1
+    pages, page, _, width = kv.pool.shape
+    assert q.shape == (B, heads * width) and out.shape == (B, heads * kv.rank) and q.stride(1) == 1 and out.stride(1) == 1
+    assert workspace.numel() >= int(lib().blitz_attn_latent_workspace_bytes(heads, kv.rank))
+    _check(lib().blitz_attn_latent(_p(q), q.stride(0), _p(kv.pool), _p(indices), _p(indptr), _p(last_page_len), _p(out), out.stride(0),
+                                   _p(workspace), B, heads, width, kv.rank, page, pages, scale, *_gate(gate), _p(status_word(q.device)),
+                                   _dt(q), _stream()), "blitz_attn_latent")
+    return out
+
+
 # ---------------------------------------------------------------------------------------------- mixture of experts
 class ExpertPlan:
     """Work list of the grouped products of a step, in buffers for up to ``max_tokens`` tokens (see csrc/kernels/moe_route.cu):
