@@ -163,17 +163,19 @@ def main():
                     "equal size, and their kernels against the roofline (bench/hybrid_bench.py; one GPU)")
     ap.add_argument("--komulorn", action="store_true", help="instead: the same for the Komulorn design, attention with shared caches "
                     "and a mixture of experts (bench/komulorn_bench.py; one GPU)")
+    ap.add_argument("--vofidra", action="store_true", help="instead: the same for the Vofidra design, several residual streams, latent "
+                    "attention and experts with identity experts (bench/vofidra_bench.py; one GPU)")
     ap.add_argument("--hybrid-part", default="all", choices=["all", "models", "kernels"])
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm()
-    if args.hybrid or args.komulorn:
+    if args.hybrid or args.komulorn or args.vofidra:
         sys.path.insert(0, os.path.join(ROOT, "bench"))
-        import hybrid_bench
-        import komulorn_bench
+        import importlib
+        module = "vofidra_bench" if args.vofidra else "komulorn_bench" if args.komulorn else "hybrid_bench"
         sampler = ClockSampler(0)
         sampler.start()
-        result = (komulorn_bench if args.komulorn else hybrid_bench).run(args.hybrid_part)
+        result = importlib.import_module(module).run(args.hybrid_part)
         result["clocks"] = sampler.stop()
         print(json.dumps(result))
         return 0
