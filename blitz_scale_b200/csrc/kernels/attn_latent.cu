@@ -3,19 +3,23 @@
 //
 //   out[b][h] = sigmoid(gate[b][h]) * sum_j softmax_j(scale * q[b][h] . row_j) row_j[0 .. rank)
 //
-// All heads of a token read the same rows, so a block of keys is one operand for up to 128 query rows (heads):
+// All heads of a token read the same rows, so both products have the keys on one side and the heads on the other.  The keys
+// and the value columns take the 128 rows of an instruction, the heads its N columns, of which any 16, 32 or 64 cost about
+// the same:
 //
-//   S = Q K^T      tcgen05.mma, A = Q (heads x width, smem), B = K (keys x width, smem), S in TMEM, two buffers
-//   P = softmax    thread = head: one pass over its row of S, P written back over S's first columns (16 bit)
-//   O += P V       tcgen05.mma, A = P (TMEM), B = the first columns of the same K tile in smem, O in TMEM
+//   S = K Q^T       tcgen05.mma, A = K (keys x width, smem), B = Q (heads x width, smem), S in TMEM, two buffers
+//   P = softmax     thread = key: one score per head; P goes to shared memory as [key][head], 16 bit, two buffers
+//   O += V^T P      tcgen05.mma, A = the first columns of the same K tile, read transposed, B = P; O in TMEM, a row per value
+//                   column, a column per head, 128 value columns per instruction
 //
-// Rows beyond the heads hold whatever the shared memory behind Q holds; they are computed and never looked at, and warps
-// without a head do nothing.  Up to 256 value columns fit beside S in tensor memory; larger ranks run as two items that read
-// the same keys, as do heads beyond what shared memory holds queries for.
+// A head's probabilities refer to the score of the sequence's first key here, and to the maximum so far once some score has
+// exceeded that by more than 2^40 (in bf16 and fp32 a factor changes no digit; fp16: 2^8); one vote per block decides, and O and
+// the row sums are rescaled then.  Row sums stay in the threads until the end.
+// More than 64 heads run as groups that read the same keys.
 //
-// Load, MMA and softmax warps walk the blocks on their own; S of the next block is issued before P V of the current one if its
-// keys are there, also across sequences, and Q has two buffers, so that the tensor core works while the softmax does.  The row maximum a head's
-// probabilities refer to moves only when it has grown by more than 2^8; O is then rescaled in place.
+// A load warp, a warp for each product and the softmax warps walk the blocks on their own, also across sequences.  An MMA
+// warp stays converged and one elected lane issues, which keeps the operand descriptors in uniform registers: an instruction
+// then costs about what the tensor core needs, not what its issue takes.
 //
 // The key blocks of all sequences, laid end to end, are dealt to the CTAs in equal contiguous shares whatever the lengths
 // are: the work list follows from the page table on the device, so that the launch can be captured in a graph.  A CTA's
@@ -28,81 +32,116 @@
 
 namespace blitz {
 
-constexpr int kLaThreads = 192;       // softmax warps 0-3, MMA warp, load warp
-constexpr int kLaMaxHeads = 128;      // query rows of an item
-constexpr int kLaValueCols = 256;     // value columns of an item
-constexpr int kLaMaxStages = 6;
+constexpr int kLaThreads = 224;       // softmax warps 0-3, S warp, load warp, O warp
+constexpr int kLaMaxHeads = 64;       // heads of an item
+constexpr int kLaMaxRank = 512;
+constexpr int kLaMaxStages = 8;
 constexpr int kLaMaxBatch = 4096;
+constexpr int kLaMaxCtas = 160;
 constexpr int kLaSmem = 227 * 1024;
-constexpr float kLaRescaleAt = 8.f;   // log2 units
 
 struct LatentParams {
   const int32_t *indices, *indptr, *last_page_len;
   void* out;                    // [batch][out_stride], head h's rank columns from h * rank on
   const void* gate;             // [batch][gate_stride], or null
   int64_t out_stride, gate_stride;
-  float *part_o, *part_lse;     // [grid][2][group][value columns], [grid][2][group]
-  int batch, heads, group, subs, halves, rank, vcols, slabs, steps, stages, page_size, max_pages, box_tokens, oob_row;
+  float *part_o, *part_lse;     // [grid][2][group][rank], [grid][2][group]
+  int* blocks_before;           // [batch + 1], for the merge
+  int batch, heads, group, subs, rank, slabs, steps, stages, q_bufs, page_shift, max_pages, box_shift, oob_row, static_table;
   float scale_log2;
   int* status;
 };
 
-template <int KT>
-__device__ __forceinline__ int la_length(const LatentParams& p, int b) {
-  const int npages = p.indptr[b + 1] - p.indptr[b];
-  return npages > 0 ? (npages - 1) * p.page_size + p.last_page_len[b] : 0;
-}
-
-// A CTA's share of the blocks as pieces of sequences.  Blocks are numbered sequence by sequence, all blocks of one sub-item
-// (head group, value half) before the next one's; s_pref[b] counts the blocks of a sub-item before sequence b.
+// A CTA's share of the blocks as pieces of sequences.  Blocks are numbered sequence by sequence, all blocks of one head group
+// before the next one's; pref[b] counts the blocks of a head group before sequence b.
 struct LaPiece {
   int b, sub, beg, end, blocks;  // blocks [beg, end) of the sequence's `blocks`
 };
 struct LaWalk {
   const int* pref;
-  int batch, subs;
-  int64_t x, hi;
-  int b;
-  __device__ __forceinline__ LaWalk(const int* pref_, int batch_, int subs_, int cta, int ctas) : pref(pref_), batch(batch_), subs(subs_) {
-    const int64_t total = static_cast<int64_t>(pref[batch]) * subs;
-    x = total * cta / ctas;
-    hi = total * (cta + 1) / ctas;
-    int lo = 0, up = batch - 1;
-    while (lo < up) {
-      const int mid = (lo + up + 1) >> 1;
-      if (static_cast<int64_t>(pref[mid]) * subs <= x) lo = mid; else up = mid - 1;
-    }
-    b = lo;
-  }
+  int subs, x, hi, b;
+  // share: first block, end, sequence of the first block
+  __device__ __forceinline__ LaWalk(const int* pref_, int subs_, const int* share)
+      : pref(pref_), subs(subs_), x(share[0]), hi(share[1]), b(share[2]) {}
   __device__ __forceinline__ bool next(LaPiece& q) {
     if (x >= hi) return false;
-    while (static_cast<int64_t>(pref[b + 1]) * subs <= x) ++b;
-    const int n = pref[b + 1] - pref[b];
-    const int rem = static_cast<int>(x - static_cast<int64_t>(pref[b]) * subs);
+    while (pref[b + 1] * subs <= x) ++b;
+    const int n = pref[b + 1] - pref[b], rem = x - pref[b] * subs;
     q.b = b;
     q.blocks = n;
     q.sub = rem / n;
     q.beg = rem - q.sub * n;
-    q.end = static_cast<int>(min(static_cast<int64_t>(n), q.beg + (hi - x)));
+    q.end = min(n, q.beg + (hi - x));
     x += q.end - q.beg;
     return true;
   }
 };
 
-template <typename T, int KT>
+// Blocks of the next piece, 0 at the end; the same in every lane, and known to be so.
+__device__ __forceinline__ int la_next(LaWalk& w) {
+  LaPiece q;
+  const int n = w.next(q) ? q.end - q.beg : 0;
+  return __shfl_sync(0xffffffffu, n, 0);
+}
+
+__device__ __forceinline__ void la_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+// Whether the predicate holds for any of the 128 softmax threads (a barrier).
+__device__ __forceinline__ bool la_any(bool v) {
+  uint32_t r;
+  asm volatile(
+      "{\n\t"
+      ".reg .pred p, q;\n\t"
+      "setp.ne.u32 p, %1, 0;\n\t"
+      "barrier.cta.red.or.pred q, 1, 128, p;\n\t"
+      "selp.b32 %0, 1, 0, q;\n\t"
+      "}\n"
+      : "=r"(r)
+      : "r"(v ? 1u : 0u)
+      : "memory");
+  return r != 0;
+}
+// order-preserving map of a float to a signed integer, and back
+__device__ __forceinline__ int la_key(float x) {
+  const int i = __float_as_int(x);
+  return i ^ ((i >> 31) & 0x7fffffff);
+}
+__device__ __forceinline__ float la_unkey(int k) { return __int_as_float(k ^ ((k >> 31) & 0x7fffffff)); }
+
+// v[i] of every lane, i < 32: lane i receives the sum over the lanes.
+__device__ __forceinline__ float la_transpose_sum(float (&v)[32], int lane) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const bool up = lane & o;
+#pragma unroll
+    for (int i = 0; i < o; ++i) {
+      const float give = up ? v[i] : v[i + o], keep = up ? v[i + o] : v[i];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+    }
+  }
+  return v[0];
+}
+
+template <typename T, int KT, int NH>
 __global__ void __launch_bounds__(kLaThreads, 1)
 attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k, const LatentParams p) {
   constexpr uint32_t kFmt = std::is_same<T, __nv_bfloat16>::value ? 1u : 0u;
   constexpr int KB = KT * 128;  // bytes of a slab of 64 columns of a key block
+  constexpr int QB = NH * 128;  // the same of Q
+  constexpr int PB = KT * 128;  // bytes of P: a row of up to 64 heads per key
+  constexpr int kSoft = KT / 32;  // warps with keys
+  constexpr float kRescaleAt = std::is_same<T, __nv_bfloat16>::value ? 40.f : 8.f;  // log2 units
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw_addr = ptx::smem_u32(smem_raw);
   uint8_t* smem = smem_raw + (((raw_addr + 1023u) & ~1023u) - raw_addr);
-  const int QB = (p.group + 7) / 8 * 1024;  // bytes of a slab of Q
-  uint8_t* sQ = smem;                        // [2]
-  uint8_t* sK = sQ + 2 * p.slabs * QB;       // [stages]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sK + p.stages * p.slabs * KB);
-  uint64_t* q_full = bars;         // [2] per piece
-  uint64_t* q_empty = bars + 2;    // [2]
+  uint8_t* sQ = smem;                                    // [q_bufs]
+  uint8_t* sK = sQ + p.q_bufs * p.slabs * QB;            // [stages]; instructions read up to a slab behind a block's end
+  uint8_t* sP = sK + p.stages * p.slabs * KB;            // [2]
+  float* s_red = reinterpret_cast<float*>(sP + 2 * PB);  // [4][NH]
+  float* s_ref = s_red + 4 * NH;                         // [NH] the maximum probabilities refer to, log2 units
+  float* s_fac = s_ref + NH;                             // [NH] rescaling, or 1 / row sum
+  uint64_t* bars = reinterpret_cast<uint64_t*>(s_fac + NH);
+  uint64_t* q_full = bars;         // [q_bufs] per piece
+  uint64_t* q_empty = bars + 2;    // [q_bufs]
   uint64_t* s_full = bars + 4;     // [2] per block
   uint64_t* p_ready = bars + 6;    // [2]
   uint64_t* pv_done = bars + 8;    // [2]
@@ -112,20 +151,24 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   uint64_t* k_empty = k_full + kLaMaxStages;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(k_empty + kLaMaxStages);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  int* s_pref = reinterpret_cast<int*>(tmem_slot + 2);  // [batch + 1]
+  int* s_share = reinterpret_cast<int*>(tmem_slot + 2);  // [4] this CTA's first block, end, sequence of the first
+  int* s_sums = s_share + 4;                             // [128] blocks of 32 sequences
+  int* s_pref = s_sums + kLaMaxBatch / 32;               // [batch + 1] blocks before a sequence
+  int* s_page = s_pref + p.batch + 1;                   // [batch + 1] its first page entry
+  int* s_len = s_page + p.batch + 1;                    // [batch]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int active = (p.group + 31) / 32;  // softmax warps with a head
+  constexpr int kWarps = kLaThreads / 32;
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < 2; ++i) {
       ptx::mbar_init(&q_full[i], 1);
       ptx::mbar_init(&q_empty[i], 1);
       ptx::mbar_init(&s_full[i], 1);
-      ptx::mbar_init(&p_ready[i], 32 * active);
+      ptx::mbar_init(&p_ready[i], KT);
       ptx::mbar_init(&pv_done[i], 1);
     }
     ptx::mbar_init(o_full, 1);
-    ptx::mbar_init(o_free, 32 * active);
+    ptx::mbar_init(o_free, 128);
     for (int i = 0; i < p.stages; ++i) {
       ptx::mbar_init(&k_full[i], 1);
       ptx::mbar_init(&k_empty[i], 1);
@@ -135,73 +178,97 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     ptx::tma_prefetch_desc(&tmap_q);
     ptx::tma_prefetch_desc(&tmap_k);
   }
+  // query rows behind the last head stay zero: their scores are zero and ask for no rescaling
+  for (int i = threadIdx.x; i < p.q_bufs * p.slabs * QB / 16; i += kLaThreads) reinterpret_cast<uint4*>(sQ)[i] = make_uint4(0, 0, 0, 0);
+  ptx::fence_proxy_async_smem();
   if (warp == 4) {
     ptx::tmem_alloc(tmem_slot, 512);
     ptx::tmem_relinquish();
   }
-  __syncthreads();
-  ptx::griddep_launch_dependents();
-  ptx::griddep_wait();
-  for (int b = threadIdx.x; b < p.batch; b += kLaThreads) s_pref[b + 1] = (la_length<KT>(p, b) + KT - 1) / KT;
+  // the work list; with a page table that no running kernel writes, while the previous kernel still runs
+  if (!p.static_table) ptx::griddep_wait();
+  const int chunks32 = (p.batch + 31) / 32;
+  for (int i = warp; i < chunks32; i += kWarps) {  // sums over 32 sequences
+    const int b = i * 32 + lane;
+    int v = 0;
+    if (b < p.batch) {
+      const int first = p.indptr[b], npages = p.indptr[b + 1] - first;
+      const int len = npages > 0 ? ((npages - 1) << p.page_shift) + p.last_page_len[b] : 0;
+      s_page[b] = first;
+      if (b == p.batch - 1) s_page[b + 1] = first + npages;
+      s_len[b] = len;
+      v = (len + KT - 1) / KT;
+    }
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int u = __shfl_up_sync(0xffffffffu, v, o);
+      if (lane >= o) v += u;
+    }
+    if (b < p.batch) s_pref[b + 1] = v;
+    if (lane == 31) s_sums[i] = v;
+  }
   if (threadIdx.x == 0) s_pref[0] = 0;
   __syncthreads();
-  if (warp == 0) {
-    int carry = 0;
-    for (int b0 = 0; b0 < p.batch; b0 += 32) {
-      int v = b0 + lane < p.batch ? s_pref[b0 + lane + 1] : 0;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const int u = __shfl_up_sync(0xffffffffu, v, o);
-        if (lane >= o) v += u;
-      }
-      v += carry;
-      if (b0 + lane < p.batch) s_pref[b0 + lane + 1] = v;
-      carry = __shfl_sync(0xffffffffu, v, 31);
+  for (int i = warp; i < chunks32; i += kWarps) {
+    int before = 0;
+    for (int k = lane; k < i; k += 32) before += s_sums[k];
+    before = __reduce_add_sync(0xffffffffu, before);
+    if (i * 32 + lane < p.batch) s_pref[i * 32 + lane + 1] += before;
+  }
+  __syncthreads();
+  {
+    const int total = s_pref[p.batch] * p.subs, G = gridDim.x, cta = blockIdx.x;
+    const int x = total * cta / G, hi = total * (cta + 1) / G;
+    if (threadIdx.x == 0) {
+      s_share[0] = x;
+      s_share[1] = hi;
     }
+    for (int b = threadIdx.x; b < p.batch; b += kLaThreads)
+      if (s_pref[b] * p.subs <= x && x < s_pref[b + 1] * p.subs) s_share[2] = b;
   }
   ptx::tc_fence_before_sync();
   __syncthreads();
   ptx::tc_fence_after_sync();
-  const uint32_t tmem_base = *tmem_slot;
-  const uint32_t tmem_O = tmem_base + 256;  // S buffers at + 0 and + 128
+  ptx::griddep_launch_dependents();
+  if (warp != 5) ptx::griddep_wait();  // (the load warp looks its first rows up before)
+  if (blockIdx.x == 0 && warp < 4)
+    for (int b = threadIdx.x; b <= p.batch; b += 128) p.blocks_before[b] = s_pref[b];
+  const uint32_t tmem_base = __shfl_sync(0xffffffffu, *tmem_slot, 0);
+  const int chunks = (p.rank + 127) / 128;     // of value columns
+  const uint32_t tmem_O = tmem_base + 2 * NH;  // S buffers at + 0 and + NH; chunk c of O at tmem_O + c * NH
   auto wait = [&](uint64_t* bar, uint32_t parity) { return ptx::bounded_mbar_wait(bar, parity, abort_flag); };
+  auto all_wait = [&](uint64_t* bar, uint32_t parity) { return __all_sync(0xffffffffu, wait(bar, parity)) != 0; };
 
   if (warp == 5) {
     // ------------------------------------------------------------ load warp
-    const int bt = p.box_tokens;
-    const bool mine = lane < KT / bt;
+    const int bt = 1 << p.box_shift;
+    const bool mine = lane < (KT >> p.box_shift);
     auto warp_wait = [&](uint64_t* bar, uint32_t parity) {
       int ok = 1;
       if (lane == 0) ok = wait(bar, parity) ? 1 : 0;
       return __shfl_sync(0xffffffffu, ok, 0) != 0;
     };
     auto box_row = [&](const LaPiece& q, int blk) {  // this lane's first row of a block in the pool
-      const int tok = blk * KT + lane * bt, slot = tok / p.page_size;
-      const int pg0 = p.indptr[q.b], npages = p.indptr[q.b + 1] - pg0;
+      const int tok = blk * KT + lane * bt, slot = tok >> p.page_shift;
+      const int pg0 = s_page[q.b], npages = s_page[q.b + 1] - pg0;
       if (!mine || slot >= npages) return p.oob_row;  // past the pool: the box arrives as zeros
       int page = p.indices[pg0 + slot];
       if (page < 0 || page >= p.max_pages) {
         if (p.status) atomicCAS(p.status, 0, kStatusBadIndex);
         page = 0;
       }
-      return page * p.page_size + (tok & (p.page_size - 1));
+      return (page << p.page_shift) + (tok & ((1 << p.page_shift) - 1));
     };
-    LaWalk walk(s_pref, p.batch, p.subs, blockIdx.x, gridDim.x);
-    LaPiece q;
-    bool ok = true;
-    int stage = 0;
-    uint32_t phase = 1, n = 0;  // a stage's first round needs no wait (the other parity counts as passed)
-    for (; ok && walk.next(q); ++n) {
-      if (n >= 2) ok = warp_wait(&q_empty[n & 1], ((n >> 1) - 1) & 1);
-      if (!ok) break;
-      if (lane == 0) {
-        ptx::mbar_expect_tx(&q_full[n & 1], static_cast<uint32_t>(p.slabs * p.group) * 128u);
-        for (int s = 0; s < p.slabs; ++s)
-          ptx::tma_load_3d(sQ + ((n & 1) * p.slabs + s) * QB, &tmap_q, &q_full[n & 1], s * 64, q.sub / p.halves * p.group, q.b);
-      }
-      int row = box_row(q, q.beg);
-      for (int blk = q.beg; blk < q.end; ++blk) {
-        const int row_next = blk + 1 < q.end ? box_row(q, blk + 1) : p.oob_row;
+    LaWalk walk(s_pref, p.subs, s_share);
+    LaPiece q, qn;
+    bool ok = true, more = walk.next(q);
+    int stage = 0, qb = 0;
+    uint32_t phase = 1, q_phase = 1;  // a buffer's first round needs no wait (the other parity counts as passed)
+    int row = more ? box_row(q, q.beg) : 0;
+    ptx::griddep_wait();
+    while (ok && more) {
+      bool more_next = false;
+      for (int blk = q.beg; blk < q.end && ok; ++blk) {
         ok = warp_wait(&k_empty[stage], phase);
         if (!ok) break;
         if (lane == 0) ptx::mbar_expect_tx(&k_full[stage], static_cast<uint32_t>(p.slabs) * KB);
@@ -209,209 +276,287 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         if (mine)
           for (int s = 0; s < p.slabs; ++s)
             ptx::tma_load_2d(sK + (stage * p.slabs + s) * KB + lane * bt * 128, &tmap_k, &k_full[stage], s * 64, row);
-        row = row_next;
+        if (++stage == p.stages) {
+          stage = 0;
+          phase ^= 1u;
+        }
+        if (blk == q.beg) {
+          ok = warp_wait(&q_empty[qb], q_phase);
+          if (!ok) break;
+          if (lane == 0) {
+            ptx::mbar_expect_tx(&q_full[qb], static_cast<uint32_t>(p.slabs * p.group) * 128u);
+            for (int s = 0; s < p.slabs; ++s)
+              ptx::tma_load_3d(sQ + (qb * p.slabs + s) * QB, &tmap_q, &q_full[qb], s * 64, q.sub * p.group, q.b);
+          }
+          if (++qb == p.q_bufs) {
+            qb = 0;
+            q_phase ^= 1u;
+          }
+          more_next = walk.next(qn);
+        }
+        // the next block's rows are looked up a block ahead of their use
+        row = blk + 1 < q.end ? box_row(q, blk + 1) : more_next ? box_row(qn, qn.beg) : 0;
+      }
+      q = qn;
+      more = more_next;
+    }
+    if (!ok && lane == 0 && p.status) atomicCAS(p.status, 0, kStatusTimeoutProducer);
+  } else if (warp == 4) {
+    // ------------------------------------------------------------ S
+    const bool leader = ptx::elect_one();
+    constexpr uint32_t idesc = ptx::make_idesc_f16(kFmt, 0u, 0u, 128, NH);
+    LaWalk walk(s_pref, p.subs, s_share);
+    int stage = 0, qb = 0;
+    uint32_t phase = 0, q_phase = 0, g = 0;
+    bool ok = true;
+    for (int n = la_next(walk); n > 0 && ok; n = la_next(walk)) {
+      ok = all_wait(&q_full[qb], q_phase);
+      for (int i = 0; i < n && ok; ++i, ++g) {
+        ok = all_wait(&k_full[stage], phase);
+        if (ok && g >= 2) ok = all_wait(&p_ready[g & 1], ((g >> 1) - 1) & 1);  // the scores of two blocks ago have been read
+        if (!ok) break;
+        ptx::tc_fence_after_sync();
+        uint64_t a = ptx::make_smem_desc(ptx::smem_u32(sK + stage * p.slabs * KB), 16, 1024, ptx::kLayoutSw128);
+        uint64_t b = ptx::make_smem_desc(ptx::smem_u32(sQ + qb * p.slabs * QB), 16, 1024, ptx::kLayoutSw128);
+        const uint32_t d = tmem_base + (g & 1) * NH;
+        for (int s = 0; s < p.steps / 4; ++s) {
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            if (leader) ptx::umma_f16_ss(d, a + k * 2, b + k * 2, idesc, (s | k) != 0 ? 1u : 0u);
+          a += KB / 16;
+          b += QB / 16;
+        }
+        for (int s = p.steps & ~3; s < p.steps; ++s) {
+          if (leader) ptx::umma_f16_ss(d, a, b, idesc, s != 0 ? 1u : 0u);
+          a += 2;
+          b += 2;
+        }
+        if (leader) ptx::umma_commit(&s_full[g & 1]);
         if (++stage == p.stages) {
           stage = 0;
           phase ^= 1u;
         }
       }
+      if (leader) ptx::umma_commit(&q_empty[qb]);
+      if (++qb == p.q_bufs) {
+        qb = 0;
+        q_phase ^= 1u;
+      }
     }
-    if (!ok && lane == 0 && p.status) atomicCAS(p.status, 0, kStatusTimeoutProducer);
-  } else if (warp == 4) {
-    // ------------------------------------------------------------ MMA warp: one thread issues
-    if (lane == 0) {
-      const uint32_t idesc_s = ptx::make_idesc_f16(kFmt, 0u, 0u, 128, KT);
-      LaWalk ws(s_pref, p.batch, p.subs, blockIdx.x, gridDim.x), wo = ws;
-      LaPiece ps, po;
-      bool ok = true, more_s = ws.next(ps), more_o = wo.next(po);
-      uint32_t gs = 0, go = 0, ns = 0, no = 0;  // blocks and pieces whose S, and whose P V, has been issued
-      int blk_s = ps.beg, blk_o = po.beg, stage_s = 0, stage_o = 0;
-      uint32_t phase_s = 0;
-      auto ready_S = [&]() {
-        return ptx::mbar_test_wait(&k_full[stage_s], phase_s) && (blk_s != ps.beg || ptx::mbar_test_wait(&q_full[ns & 1], (ns >> 1) & 1));
-      };
-      auto issue_S = [&]() {
-        ptx::tc_fence_after_sync();
-        const uint32_t a = ptx::smem_u32(sQ + (ns & 1) * p.slabs * QB), bb = ptx::smem_u32(sK + stage_s * p.slabs * KB);
-        const uint32_t d = tmem_base + (gs & 1) * 128;
-        for (int k = 0; k < p.steps; ++k)
-          ptx::umma_f16_ss(d, ptx::make_smem_desc(a + (k >> 2) * QB + (k & 3) * 32, 16, 1024, ptx::kLayoutSw128),
-                           ptx::make_smem_desc(bb + (k >> 2) * KB + (k & 3) * 32, 16, 1024, ptx::kLayoutSw128), idesc_s, k != 0 ? 1u : 0u);
-        ptx::umma_commit(&s_full[gs & 1]);
-        ++gs;
-        if (++stage_s == p.stages) {
-          stage_s = 0;
-          phase_s ^= 1u;
-        }
-        if (++blk_s == ps.end) {
-          ptx::umma_commit(&q_empty[ns & 1]);
-          ++ns;
-          more_s = ws.next(ps);
-          blk_s = ps.beg;
-        }
-      };
-      uint32_t spins = 0;
-      uint64_t t0 = 0;
-      while (ok && more_o) {
-        // whichever can go first: the next S (at most one block ahead of P V), or P V of the oldest block
-        if (more_s && gs - go < 2 && ready_S()) {
-          issue_S();
-          spins = 0;
-          continue;
-        }
-        if (gs == go || !ptx::mbar_test_wait(&p_ready[go & 1], (go >> 1) & 1)) {
-          if ((++spins & 63u) == 0) {
-            const uint64_t now = ptx::globaltimer_ns();
-            if (spins == 64u) t0 = now;
-            if (*abort_flag || now - t0 > ptx::kDefaultWaitNs) {
-              *abort_flag = 1;
-              ok = false;
-            }
-          }
-          continue;
-        }
-        spins = 0;
-        if (blk_o == po.beg && no > 0) ok = wait(o_free, (no - 1) & 1);  // the last piece's O has been read
+    if (!ok && leader && p.status) atomicCAS(p.status, 0, kStatusTimeoutMma);
+  } else if (warp == 6) {
+    // ------------------------------------------------------------ O += V^T P
+    const bool leader = ptx::elect_one();
+    constexpr uint32_t idesc = ptx::make_idesc_f16(kFmt, 1u, 1u, 128, NH);
+    LaWalk walk(s_pref, p.subs, s_share);
+    int stage = 0;
+    uint32_t g = 0, o_phase = 1;  // (the first piece needs no wait)
+    bool ok = true;
+    for (int n = la_next(walk); n > 0 && ok; n = la_next(walk), o_phase ^= 1u) {
+      ok = all_wait(o_free, o_phase);  // the last piece's O has been read
+      for (int i = 0; i < n && ok; ++i, ++g) {
+        ok = all_wait(&p_ready[g & 1], (g >> 1) & 1);
         if (!ok) break;
         ptx::tc_fence_after_sync();
-        const int half = po.sub % p.halves;
-        const int cols = min(p.vcols, p.rank - half * kLaValueCols);
-        const uint32_t idesc_o = ptx::make_idesc_f16(kFmt, 0u, 1u, 128, (cols + 15) / 16 * 16);
-        const uint32_t bb = ptx::smem_u32(sK + stage_o * p.slabs * KB) + half * (kLaValueCols / 64) * KB;
+        for (int c = 0; c < chunks; ++c) {
+          // (value columns behind the last one are rows of O that nobody reads)
+          const uint64_t a = ptx::make_smem_desc(ptx::smem_u32(sK + (stage * p.slabs + c * 2) * KB), KB, 1024, ptx::kLayoutSw128);
+          const uint64_t b = ptx::make_smem_desc(ptx::smem_u32(sP + (g & 1) * PB), PB, 1024, ptx::kLayoutSw128);
 #pragma unroll
-        for (int k = 0; k < KT / 16; ++k)
-          ptx::umma_f16_ts(tmem_O, tmem_base + (go & 1) * 128 + k * 8, ptx::make_smem_desc(bb + k * 2048, KB, 1024, ptx::kLayoutSw128),
-                           idesc_o, (blk_o != po.beg || k != 0) ? 1u : 0u);
-        ptx::umma_commit(&k_empty[stage_o]);
-        ptx::umma_commit(&pv_done[go & 1]);
-        ++go;
-        if (++stage_o == p.stages) stage_o = 0;
-        if (++blk_o == po.end) {
-          ptx::umma_commit(o_full);
-          ++no;
-          more_o = wo.next(po);
-          blk_o = po.beg;
+          for (int k = 0; k < KT / 16; ++k)
+            if (leader) ptx::umma_f16_ss(tmem_O + c * NH, a + k * 128, b + k * 128, idesc, (i | k) != 0 ? 1u : 0u);
         }
+        if (leader) {
+          ptx::umma_commit(&k_empty[stage]);
+          ptx::umma_commit(&pv_done[g & 1]);
+          if (i == n - 1) ptx::umma_commit(o_full);
+        }
+        if (++stage == p.stages) stage = 0;
       }
-      if (!ok && p.status) atomicCAS(p.status, 0, kStatusTimeoutMma);
     }
-  } else if (warp < active) {
-    // ------------------------------------------------------------ softmax warps: thread = head
+    if (!ok && leader && p.status) atomicCAS(p.status, 0, kStatusTimeoutMma);
+  } else {
+    // ------------------------------------------------------------ softmax warps: thread = key, then thread = value column
     const int r = warp * 32 + lane;
     const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
-    const uint32_t tO = tmem_O + lane_addr;
-    LaWalk walk(s_pref, p.batch, p.subs, blockIdx.x, gridDim.x);
+    const bool soft = warp < kSoft;
+    LaWalk walk(s_pref, p.subs, s_share);
     LaPiece q;
-    bool ok = true;
+    bool ok = true;  // of this thread; the four warps keep meeting at the barriers
     uint32_t g = 0, n = 0;
-    for (; ok && walk.next(q); ++n) {
-      const int len = la_length<KT>(p, q.b), half = q.sub % p.halves, head = q.sub / p.halves * p.group + r;
-      const int cols = min(p.vcols, p.rank - half * kLaValueCols);
-      const bool mine = r < p.group;
-      float gate = 1.f;
-      if (p.gate != nullptr && mine) gate = sigmoid_f(to_f<T>(reinterpret_cast<const T*>(p.gate)[q.b * p.gate_stride + head]));
-      float m_ref = 0.f, l = 0.f;
-      for (int blk = q.beg; blk < q.end; ++blk, ++g) {
-        if (!wait(&s_full[g & 1], (g >> 1) & 1)) {
-          ok = false;
-          break;
-        }
-        ptx::tc_fence_after_sync();
-        const uint32_t tS = tmem_base + (g & 1) * 128 + lane_addr;
-        uint32_t v[KT / 32][32];
-#pragma unroll
-        for (int i = 0; i < KT / 32; ++i) ptx::tmem_ld_32x32(tS + i * 32, v[i]);
-        ptx::tmem_ld_wait();
-        auto score = [&](int i) -> uint32_t& { return v[i >> 5][i & 31]; };
-        const int valid = len - blk * KT;
-        if (valid < KT) {
-#pragma unroll
-          for (int i = 0; i < KT; ++i)
-            if (i >= valid) score(i) = 0xff800000u;  // -inf
-        }
-        float mxs[8];
-#pragma unroll
-        for (int i = 0; i < 8; ++i) mxs[i] = __uint_as_float(score(i));
-#pragma unroll
-        for (int i = 8; i < KT - 8; i += 16)
-#pragma unroll
-          for (int k = 0; k < 8; ++k) mxs[k] = ptx::fmax3(mxs[k], __uint_as_float(score(i + 2 * k)), __uint_as_float(score(i + 2 * k + 1)));
-#pragma unroll
-        for (int i = KT - 8; i < KT; ++i) mxs[i & 7] = fmaxf(mxs[i & 7], __uint_as_float(score(i)));
-        float mx = fmaxf(ptx::fmax3(mxs[0], mxs[1], mxs[2]), ptx::fmax3(mxs[3], mxs[4], mxs[5]));
-        mx = ptx::fmax3(mx, mxs[6], mxs[7]) * p.scale_log2;
-        if (blk == q.beg) {
-          m_ref = mx;
-        } else {
-          const bool grow = mx > m_ref + kLaRescaleAt;
-          if (__any_sync(0xffffffffu, grow && mine)) {
-            if (!wait(&pv_done[(g - 1) & 1], ((g - 1) >> 1) & 1)) {  // O is settled
-              ok = false;
-              break;
-            }
-            ptx::tc_fence_after_sync();
-            const float alpha = grow ? ptx::ex2_approx(m_ref - mx) : 1.f;
+    const uint32_t tO = tmem_O + lane_addr;
+    // a piece's output: to the result, or where the partial sums of incomplete pieces go
+    auto emit = [&](auto* row) {
+      using U = std::remove_pointer_t<decltype(row)>;
 #pragma unroll 1
-            for (int c = 0; c < cols; c += 32) {
-              uint32_t o[32];
-              ptx::tmem_ld_32x32(tO + c, o);
+      for (int c = 0; c < chunks; ++c) {
+        const int d = c * 128 + r;
+#pragma unroll 1
+        for (int h0 = 0; h0 < NH; h0 += 16) {
+          uint32_t o[16];
+          ptx::tmem_ld_32x16(tO + c * NH + h0, o);
+          ptx::tmem_ld_wait();
+          if (c == chunks - 1 && h0 == NH - 16) {  // the next piece may overwrite O
+            ptx::tc_fence_before_sync();
+            ptx::mbar_arrive(o_free);
+          }
+          if (d >= p.rank || h0 >= p.group) continue;
+          U* dst = row + h0 * p.rank + d;
+          const bool all = h0 + 16 <= p.group;
+#pragma unroll
+          for (int i = 0; i < 16; i += 4) {
+            const float4 f = *reinterpret_cast<const float4*>(s_fac + h0 + i);
+            const float y[4] = {__uint_as_float(o[i]) * f.x, __uint_as_float(o[i + 1]) * f.y, __uint_as_float(o[i + 2]) * f.z,
+                                __uint_as_float(o[i + 3]) * f.w};
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+              if (all || h0 + i + k < p.group) stf<U>(dst, y[k]);
+              dst += p.rank;
+            }
+          }
+        }
+      }
+    };
+    for (; walk.next(q); ++n) {
+      const int len = s_len[q.b], head0 = q.sub * p.group;
+      // of the thread's keys, per head: row sum, and the references (the same in all threads; for many heads in shared memory)
+      constexpr bool kRefRegs = NH <= 32;
+      float l[NH], ref[kRefRegs ? NH : 1] = {};
+#pragma unroll
+      for (int h = 0; h < NH; ++h) l[h] = 0.f;
+      auto reference = [&](int h) { return kRefRegs ? ref[kRefRegs ? h : 0] : s_ref[h]; };
+      for (int blk = q.beg; blk < q.end; ++blk, ++g) {
+        float x[NH];  // scores relative to the references, log2 units
+        const bool first = blk == q.beg;
+        bool grow = false;
+        if (soft) {
+          if (ok) ok = wait(&s_full[g & 1], (g >> 1) & 1);
+          ptx::tc_fence_after_sync();
+          const uint32_t tS = tmem_base + (g & 1) * NH + lane_addr;
+#pragma unroll
+          for (int i = 0; i < NH; i += 16) {
+            uint32_t v[16];
+            ptx::tmem_ld_32x16(tS + i, v);
+            ptx::tmem_ld_wait();
+#pragma unroll
+            for (int k = 0; k < 16; ++k) x[i + k] = fmaf(__uint_as_float(v[k]), p.scale_log2, first ? 0.f : -reference(i + k));
+          }
+          if (blk * KT + KT > len && blk * KT + r >= len) {
+#pragma unroll
+            for (int h = 0; h < NH; ++h) x[h] = -INFINITY;
+          }
+          if (first) {  // the first key's scores are the references
+            if (r == 0) {
+#pragma unroll
+              for (int h = 0; h < NH; ++h) s_ref[h] = x[h];
+            }
+            asm volatile("bar.sync 2, %0;" ::"n"(KT) : "memory");
+#pragma unroll
+            for (int h = 0; h < NH; ++h) {
+              if (kRefRegs) ref[kRefRegs ? h : 0] = s_ref[h];
+              x[h] -= s_ref[h];
+            }
+          }
+          float mx = -INFINITY;
+#pragma unroll
+          for (int h = 0; h < NH; h += 2) mx = ptx::fmax3(mx, x[h], x[h + 1]);
+          grow = mx > kRescaleAt;
+        }
+        if (la_any(grow)) {
+          // new references: the maximum over the block and over the old ones
+          if (soft) {
+            int mine = 0;
+#pragma unroll
+            for (int h = 0; h < NH; ++h) {
+              const int k = __reduce_max_sync(0xffffffffu, la_key(x[h]));
+              if ((h & 31) == lane) mine = k;
+              if ((h & 31) == 31 || h == NH - 1)
+                if (lane <= (h & 31)) s_red[warp * NH + (h & ~31) + lane] = la_unkey(mine);
+            }
+          }
+          la_sync();
+          if (r < NH) {
+            float m = 0.f;
+#pragma unroll
+            for (int w = 0; w < kSoft; ++w) m = fmaxf(m, s_red[w * NH + r]);
+            s_fac[r] = ptx::ex2_approx(-m);
+            s_ref[r] += m;
+            s_red[r] = m;  // (this thread has read the column)
+          }
+          la_sync();
+#pragma unroll
+          for (int h = 0; h < NH; ++h) {
+            x[h] -= s_red[h];
+            if (kRefRegs) ref[kRefRegs ? h : 0] = s_ref[h];
+          }
+          if (!first) {
+            if (ok) ok = wait(&pv_done[(g - 1) & 1], ((g - 1) >> 1) & 1);  // O is settled
+            ptx::tc_fence_after_sync();
+#pragma unroll
+            for (int h = 0; h < NH; ++h) l[h] *= s_fac[h];
+#pragma unroll 1
+            for (int c = 0; c < chunks * NH; c += 16) {
+              uint32_t o[16];
+              ptx::tmem_ld_32x16(tO + c, o);
               ptx::tmem_ld_wait();
 #pragma unroll
-              for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
-              ptx::tmem_st_32x32(tO + c, o);
+              for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_fac[(c + i) % NH]);
+              ptx::tmem_st_32x16(tO + c, o);
             }
             ptx::tmem_st_wait();
-            l *= alpha;
-            if (grow) m_ref = mx;
+            ptx::tc_fence_before_sync();
+            la_sync();
           }
         }
-        float rs[4] = {0.f, 0.f, 0.f, 0.f};
+        if (soft) {
+          if (g >= 2 && ok) ok = wait(&pv_done[g & 1], ((g >> 1) - 1) & 1);  // P of two blocks ago has been read
+          uint8_t* prow = sP + (g & 1) * PB + r * 128;
 #pragma unroll
-        for (int h = 0; h < KT / 64; ++h) {  // 64 scores -> 32 columns of pairs
-          uint32_t pk[32];
+          for (int h = 0; h < NH; h += 8) {
+            float e[8];
 #pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            const float e0 = ptx::ex2_approx(fmaf(__uint_as_float(score(h * 64 + 2 * i)), p.scale_log2, -m_ref));
-            const float e1 = ptx::ex2_approx(fmaf(__uint_as_float(score(h * 64 + 2 * i + 1)), p.scale_log2, -m_ref));
-            rs[i & 3] += e0 + e1;
-            pk[i] = pk2<T>(e0, e1);
-          }
-          ptx::tmem_st_32x32(tS + h * 32, pk);
-        }
-        ptx::tmem_st_wait();
-        l += (rs[0] + rs[1]) + (rs[2] + rs[3]);
-        ptx::tc_fence_before_sync();
-        ptx::mbar_arrive(&p_ready[g & 1]);
-      }
-      if (ok) ok = wait(o_full, n & 1);
-      if (!ok) break;
-      ptx::tc_fence_after_sync();
-      const bool whole = q.beg == 0 && q.end == q.blocks;
-      const float inv = l > 0.f ? (whole ? gate : 1.f) / l : 0.f;
-      T* dst = reinterpret_cast<T*>(p.out) + q.b * p.out_stride + static_cast<int64_t>(head) * p.rank + half * kLaValueCols;
-      const int64_t part = (static_cast<int64_t>(blockIdx.x) * 2 + (n > 0)) * p.group + r;
-      if (!whole && mine) p.part_lse[part] = m_ref + log2f(l);
-#pragma unroll 1
-      for (int c = 0; c < cols; c += 32) {
-        uint32_t o[32];
-        ptx::tmem_ld_32x32(tO + c, o);
-        ptx::tmem_ld_wait();
-        if (c + 32 >= cols) {  // the next piece may overwrite O
-          ptx::tc_fence_before_sync();
-          ptx::mbar_arrive(o_free);
-        }
-        if (mine) {
-#pragma unroll
-          for (int i = 0; i < 32; i += 8) {
-            if (c + i < cols) {
-              float x[8];
-#pragma unroll
-              for (int k = 0; k < 8; ++k) x[k] = __uint_as_float(o[i + k]) * inv;
-              if (whole) *reinterpret_cast<uint4*>(dst + c + i) = pack8<T>(x);
-              else stf8<float>(p.part_o + part * p.vcols + c + i, x);
+            for (int i = 0; i < 8; ++i) {
+              e[i] = ptx::ex2_approx(x[h + i]);
+              l[h + i] += e[i];
             }
+            *reinterpret_cast<uint4*>(prow + (((h >> 3) ^ (r & 7)) << 4)) = pack8<T>(e);
           }
+          ptx::fence_proxy_async_smem();
+          ptx::tc_fence_before_sync();
+          ptx::mbar_arrive(&p_ready[g & 1]);
         }
+      }
+      // row sums: over a warp's keys, then over the warps
+      if (soft) {
+#pragma unroll
+        for (int h0 = 0; h0 < NH; h0 += 32) {
+          float t[32];
+#pragma unroll
+          for (int i = 0; i < 32; ++i) t[i] = h0 + i < NH ? l[(h0 + i) % NH] : 0.f;
+          const float sum = la_transpose_sum(t, lane);
+          if (h0 + lane < NH) s_red[warp * NH + h0 + lane] = sum;
+        }
+      }
+      la_sync();
+      const bool whole = q.beg == 0 && q.end == q.blocks;
+      const int64_t part = (static_cast<int64_t>(blockIdx.x) * 2 + (n > 0)) * p.group;
+      if (r < p.group) {
+        float sum = 0.f;
+#pragma unroll
+        for (int w = 0; w < kSoft; ++w) sum += s_red[w * NH + r];
+        float f = sum > 0.f ? 1.f / sum : 0.f;
+        if (whole && p.gate != nullptr) f *= sigmoid_f(to_f<T>(reinterpret_cast<const T*>(p.gate)[q.b * p.gate_stride + head0 + r]));
+        s_fac[r] = f;
+        if (!whole) p.part_lse[part + r] = s_ref[r] + log2f(sum);
+      }
+      la_sync();
+      if (ok) ok = wait(o_full, n & 1);
+      ptx::tc_fence_after_sync();
+      if (whole) emit(reinterpret_cast<T*>(p.out) + q.b * p.out_stride + static_cast<int64_t>(head0) * p.rank);
+      else emit(p.part_o + part * p.rank);
+      if (la_any(!ok)) {  // (also: s_fac, s_red and s_ref have been read)
+        ok = false;
+        break;
       }
     }
     if (!ok && p.status && lane == 0) atomicCAS(p.status, 0, kStatusTimeoutEpilogue);
@@ -426,93 +571,117 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
 }
 
 // Rows whose blocks lie in more than one CTA's share: out = sum_c w_c o_c / sum_c w_c, w_c = 2^(lse_c - max lse).  Rows without
-// keys become zeros.  A warp per head.
-template <typename T, int KT>
-__global__ void __launch_bounds__(256) attn_latent_merge_kernel(const LatentParams p, int ctas) {
+// keys become zeros.  `per` warps per head (1, or all eight where there are few rows).
+template <typename T>
+__global__ void __launch_bounds__(256) attn_latent_merge_kernel(const LatentParams p, int ctas, int per) {
   ptx::griddep_launch_dependents();
   ptx::griddep_wait();
-  __shared__ int s_sum[2];
+  extern __shared__ float s_acc[];  // [8][rank], several warps per head only
   const int b = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  if (threadIdx.x < 2) s_sum[threadIdx.x] = 0;
-  __syncthreads();
-  int before = 0, all = 0;
-  for (int i = threadIdx.x; i < p.batch; i += blockDim.x) {
-    const int n = (la_length<KT>(p, i) + KT - 1) / KT;
-    all += n;
-    before += i < b ? n : 0;
+  const int head = blockIdx.y * (8 / per) + warp / per, share = warp % per;
+  if (head >= p.heads) return;  // (with several warps per head: all of a block or none)
+  const int before = p.blocks_before[b], blocks = p.blocks_before[b + 1] - before, total = p.blocks_before[p.batch] * p.subs;
+  T* dst = reinterpret_cast<T*>(p.out) + b * p.out_stride + static_cast<int64_t>(head) * p.rank;
+  if (blocks == 0) {
+    if (share == 0)
+      for (int c = lane; c < p.rank; c += 32) stf<T>(dst + c, 0.f);
+    return;
   }
-  before = __reduce_add_sync(0xffffffffu, before);
-  all = __reduce_add_sync(0xffffffffu, all);
-  if (lane == 0) {
-    atomicAdd(&s_sum[0], before);
-    atomicAdd(&s_sum[1], all);
+  const int beg = before * p.subs + head / p.group * blocks;
+  const int c0 = ((beg + 1) * ctas - 1) / total, c1 = ((beg + blocks) * ctas - 1) / total;
+  if (c0 == c1) return;  // one CTA has done all of it
+  constexpr int kRounds = kLaMaxCtas / 32;
+  float w[kRounds];
+  int at[kRounds];
+  float m = -INFINITY, sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < kRounds; ++i) {
+    w[i] = -INFINITY;
+    at[i] = -1;
+    if (c0 + i * 32 > c1) continue;
+    const int c = c0 + i * 32 + lane, lo = total * c / ctas;
+    // the piece is its CTA's first one unless the CTA's share begins before this sequence; with more CTAs than blocks some
+    // have none
+    if (c <= c1 && lo < total * (c + 1) / ctas) {
+      at[i] = (c * 2 + (lo < beg ? 1 : 0)) * p.group + head % p.group;
+      w[i] = p.part_lse[at[i]];
+    }
+    m = fmaxf(m, w[i]);
   }
-  __syncthreads();
-  const int head = blockIdx.y * 8 + warp;
-  if (head >= p.heads) return;
-  const int64_t total = static_cast<int64_t>(s_sum[1]) * p.subs;
-  const int blocks = (la_length<KT>(p, b) + KT - 1) / KT;
+  m = warp_max(m);
+#pragma unroll
+  for (int i = 0; i < kRounds; ++i) {
+    w[i] = exp2f(w[i] - m);
+    sum += w[i];
+  }
+  sum = warp_sum(sum);
   const float gate = p.gate ? sigmoid_f(to_f<T>(reinterpret_cast<const T*>(p.gate)[b * p.gate_stride + head])) : 1.f;
-  for (int half = 0; half < p.halves; ++half) {
-    const int cols = min(p.vcols, p.rank - half * kLaValueCols);
-    T* dst = reinterpret_cast<T*>(p.out) + b * p.out_stride + static_cast<int64_t>(head) * p.rank + half * kLaValueCols;
-    if (blocks == 0) {
-      for (int c = lane; c < cols; c += 32) stf<T>(dst + c, 0.f);
-      continue;
-    }
-    const int64_t beg = static_cast<int64_t>(s_sum[0]) * p.subs + static_cast<int64_t>(head / p.group * p.halves + half) * blocks;
-    const int c0 = static_cast<int>(((beg + 1) * ctas - 1) / total), c1 = static_cast<int>(((beg + blocks) * ctas - 1) / total);
-    if (c0 == c1) continue;  // one CTA has done all of it
-    // the piece is its CTA's first one unless the CTA's share begins before this sequence
-    auto part = [&](int c) { return (static_cast<int64_t>(c) * 2 + (total * c / ctas < beg ? 1 : 0)) * p.group + head % p.group; };
-    auto has = [&](int c) { return total * c / ctas < total * (c + 1) / ctas; };  // (more CTAs than blocks: some have none)
-    float m = -INFINITY;
-    for (int c = c0 + lane; c <= c1; c += 32)
-      if (has(c)) m = fmaxf(m, p.part_lse[part(c)]);
-    m = warp_max(m);
-    float acc[kLaValueCols / 32] = {}, sum = 0.f;
-    for (int c = c0; c <= c1; ++c) {
-      if (!has(c)) continue;
-      const int64_t at = part(c);
-      const float w = exp2f(p.part_lse[at] - m);
-      sum += w;
+  float acc[kLaMaxRank / 32] = {};
 #pragma unroll
-      for (int k = 0; k < kLaValueCols / 32; ++k)
-        if (k * 32 + lane < cols) acc[k] += w * p.part_o[at * p.vcols + k * 32 + lane];
-    }
-    const float f = gate / sum;
+  for (int i = 0; i < kRounds; ++i) {
+    const int cnt = min(32, c1 - (c0 + i * 32) + 1);
+#pragma unroll 2
+    for (int j = share; j < cnt; j += per) {
+      const int a = __shfl_sync(0xffffffffu, at[i], j);
+      const float wj = __shfl_sync(0xffffffffu, w[i], j);
+      if (a < 0) continue;
+      const float* src = p.part_o + static_cast<int64_t>(a) * p.rank;
 #pragma unroll
-    for (int k = 0; k < kLaValueCols / 32; ++k)
-      if (k * 32 + lane < cols) stf<T>(dst + k * 32 + lane, acc[k] * f);
+      for (int k = 0; k < kLaMaxRank / 32; ++k)
+        if (k * 32 + lane < p.rank) acc[k] += wj * src[k * 32 + lane];
+    }
+  }
+  const float f = gate / sum;
+  if (per == 1) {
+#pragma unroll
+    for (int k = 0; k < kLaMaxRank / 32; ++k)
+      if (k * 32 + lane < p.rank) stf<T>(dst + k * 32 + lane, acc[k] * f);
+    return;
+  }
+#pragma unroll
+  for (int k = 0; k < kLaMaxRank / 32; ++k)
+    if (k * 32 + lane < p.rank) s_acc[warp * p.rank + k * 32 + lane] = acc[k];
+  __syncthreads();
+  for (int c = threadIdx.x; c < p.rank; c += blockDim.x) {
+    float v = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v += s_acc[i * p.rank + c];
+    stf<T>(dst + c, v * f);
   }
 }
 
 struct LatentPlan {
-  int kt, group, halves, vcols, slabs, stages;
+  int kt, group, nh, slabs, stages, q_bufs;
   size_t smem;
 };
-// How the heads are grouped and how tall a key block is: blocks of 128 keys and as many heads as possible, at least two stages.
-static bool latent_plan(int batch, int heads, int width, int rank, int page_size, LatentPlan* out) {
-  if (batch < 1 || batch > kLaMaxBatch || heads < 1 || rank < 8 || rank > 2 * kLaValueCols || width < rank || ((width | rank) & 7)) return false;
+// How the heads are grouped and how tall a key block is: as many heads as possible; blocks of 128 keys if two stages of them fit,
+// else of 64 (with more than 32 heads 64 first: four small stages beat two tall ones there); queries double buffered if that
+// leaves room.
+static bool latent_plan(int batch, int heads, int width, int rank, int page_size, int kt_hint, LatentPlan* out) {
+  if (batch < 1 || batch > kLaMaxBatch || heads < 1 || rank < 8 || rank > kLaMaxRank || width < rank || ((width | rank) & 7)) return false;
   if (page_size < 8 || (page_size & (page_size - 1)) != 0) return false;
   LatentPlan pl;
   pl.slabs = (width + 63) / 64;
-  pl.halves = rank > kLaValueCols ? 2 : 1;
-  pl.vcols = rank > kLaValueCols ? kLaValueCols : rank;
-  const int fixed = 1024 + (12 + 2 * kLaMaxStages) * 8 + 8 + (batch + 1) * 4;
   for (int groups = 1; groups <= heads; ++groups) {
     if (heads % groups || heads / groups > kLaMaxHeads) continue;
     pl.group = heads / groups;
-    for (int kt = 128; kt >= 64; kt /= 2) {
-      const int room = kLaSmem - fixed - 2 * pl.slabs * ((pl.group + 7) / 8 * 1024);
-      int stages = room / (pl.slabs * kt * 128);
-      if (stages < 2) continue;
-      pl.kt = kt;
-      pl.stages = stages < kLaMaxStages ? stages : kLaMaxStages;
-      // (the 128-row view of the last slab of Q ends in the key stages behind it)
-      pl.smem = fixed + 2 * pl.slabs * ((pl.group + 7) / 8 * 1024) + (size_t)pl.stages * pl.slabs * kt * 128;
-      *out = pl;
-      return true;
+    pl.nh = pl.group <= 16 ? 16 : pl.group <= 32 ? 32 : 64;
+    const int fixed = 1024 + 6 * pl.nh * 4 + (12 + 2 * kLaMaxStages) * 8 + 8 + 16 + kLaMaxBatch / 32 * 4 + (batch + 1) * 12;
+    const int tall_first = pl.nh <= 32;
+    for (int i = 0; i < 2; ++i) {
+      const int kt = (i == 0) == (tall_first != 0) ? 128 : 64;
+      if (kt_hint && kt != kt_hint) continue;
+      for (int bufs = 2; bufs >= 1; --bufs) {
+        const int rest = fixed + 2 * kt * 128 + bufs * pl.slabs * pl.nh * 128, stage = pl.slabs * kt * 128;
+        const int stages = (kLaSmem - rest) / stage;
+        if (rest > kLaSmem || stages < (bufs == 2 && kt == 64 ? 3 : 2)) continue;
+        pl.kt = kt;
+        pl.q_bufs = bufs;
+        pl.stages = stages < kLaMaxStages ? stages : kLaMaxStages;
+        pl.smem = rest + (size_t)pl.stages * stage;
+        *out = pl;
+        return true;
+      }
     }
   }
   return false;
@@ -525,53 +694,64 @@ using namespace blitz;
 
 int blitz_attn_latent_supported(int batch, int heads, int width, int rank, int page_size) {
   LatentPlan pl;
-  return latent_plan(batch, heads, width, rank, page_size, &pl) ? 1 : 0;
+  return latent_plan(batch, heads, width, rank, page_size, 0, &pl) ? 1 : 0;
 }
 
 // Bytes of fp32 scratch for the partial sums, whatever the batch is.
 int64_t blitz_attn_latent_workspace_bytes(int heads, int rank) {
-  const int group = heads < kLaMaxHeads ? heads : kLaMaxHeads, cols = rank < kLaValueCols ? rank : kLaValueCols;
-  return (int64_t)device_sm_count() * 2 * group * (cols + 1) * (int64_t)sizeof(float);
+  const int group = heads < kLaMaxHeads ? heads : kLaMaxHeads;
+  return (int64_t)device_sm_count() * 2 * group * (rank + 1) * (int64_t)sizeof(float) + (kLaMaxBatch + 1) * (int64_t)sizeof(int);
 }
 
 // q [batch][q_stride]: heads of `width` columns; pool [max_pages][page_size][width], the first `rank` columns are the values;
 // out [batch][out_stride]: heads of `rank` columns.  width, rank: multiples of 8, rank up to 512; page_size: a power of two >= 8;
-// gate [batch][gate_stride] or null.  A row without pages gives zeros.
+// gate [batch][gate_stride] or null.  A row without pages gives zeros.  kt_hint: keys per block, 0 = choose, else 64 or 128.
+// static_table: no kernel still running in the stream writes indices, indptr or last_page_len.
 int blitz_attn_latent(const void* q, int64_t q_stride, const void* pool, const int32_t* indices, const int32_t* indptr,
                       const int32_t* last_page_len, void* out, int64_t out_stride, void* workspace, int batch, int heads, int width, int rank,
-                      int page_size, int max_pages, float sm_scale, const void* gate, int64_t gate_stride, int* status, int dtype,
+                      int page_size, int max_pages, float sm_scale, const void* gate, int64_t gate_stride, int kt_hint, int static_table, int* status, int dtype,
                       cudaStream_t stream) {
   if (batch <= 0) return 0;
   LatentPlan pl;
-  if (!latent_plan(batch, heads, width, rank, page_size, &pl) || workspace == nullptr || max_pages < 1) return -1;
-  if ((q_stride & 7) || (out_stride & 7) || (reinterpret_cast<uintptr_t>(out) & 15) || (reinterpret_cast<uintptr_t>(workspace) & 31)) return -1;
+  if (!latent_plan(batch, heads, width, rank, page_size, kt_hint, &pl) || workspace == nullptr || max_pages < 1) return -1;
+  if ((q_stride & 7) || (reinterpret_cast<uintptr_t>(workspace) & 15)) return -1;
+  const int sms = device_sm_count() < kLaMaxCtas ? device_sm_count() : kLaMaxCtas;
+  // block numbers times CTAs are 32-bit
+  if (((int64_t)max_pages * page_size / 64 + batch) * (heads / pl.group) * (sms + 1) >= ((int64_t)1 << 31)) return -1;
   const int bt = page_size < 64 ? page_size : 64;
   CUtensorMap tq, tk;
   if (!get_tmap_3d(&tq, q, (uint64_t)width, (uint64_t)heads, (uint64_t)batch, (uint64_t)width * 2, (uint64_t)q_stride * 2, 64,
                    (uint32_t)pl.group, 1))
     return -2;
   if (!get_tmap_2d(&tk, pool, (uint64_t)width, (uint64_t)max_pages * page_size, (uint64_t)width * 2, 64, (uint32_t)bt)) return -2;
-  const int sms = device_sm_count();
   LatentParams p;
   p.indices = indices; p.indptr = indptr; p.last_page_len = last_page_len; p.out = out; p.gate = gate;
   p.out_stride = out_stride; p.gate_stride = gate_stride;
-  p.batch = batch; p.heads = heads; p.group = pl.group; p.halves = pl.halves; p.subs = heads / pl.group * pl.halves; p.rank = rank;
-  p.vcols = pl.vcols; p.slabs = pl.slabs; p.steps = (width + 15) / 16; p.stages = pl.stages; p.page_size = page_size; p.max_pages = max_pages; p.box_tokens = bt;
-  p.oob_row = max_pages * page_size;
+  p.batch = batch; p.heads = heads; p.group = pl.group; p.subs = heads / pl.group; p.rank = rank;
+  p.slabs = pl.slabs; p.steps = (width + 15) / 16; p.stages = pl.stages; p.q_bufs = pl.q_bufs;
+  p.page_shift = __builtin_ctz(page_size); p.box_shift = __builtin_ctz(bt); p.static_table = static_table;
+  p.max_pages = max_pages; p.oob_row = max_pages * page_size;
   p.part_o = reinterpret_cast<float*>(workspace);
-  p.part_lse = p.part_o + (int64_t)sms * 2 * pl.group * pl.vcols;
+  p.part_lse = p.part_o + (int64_t)sms * 2 * pl.group * rank;
+  p.blocks_before = reinterpret_cast<int*>(p.part_lse + (int64_t)sms * 2 * pl.group);
+  const int per = (int64_t)batch * heads >= 8 * (int64_t)sms ? 1 : 8;  // warps per head in the merge
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status;
-  auto go = [&](auto type, auto keys) -> int {
+  auto go = [&](auto type, auto keys, auto cols) -> int {
     using T = decltype(type);
-    constexpr int KT = decltype(keys)::value;
+    constexpr int KT = decltype(keys)::value, NH = decltype(cols)::value;
     static PerDeviceOnce once;
-    cudaError_t e = once.run([] { return cudaFuncSetAttribute(attn_latent_kernel<T, KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kLaSmem); });
-    if (e == cudaSuccess) e = launch_pdl(attn_latent_kernel<T, KT>, dim3(sms), dim3(kLaThreads), pl.smem, stream, tq, tk, p);
-    if (e == cudaSuccess) e = launch_pdl(attn_latent_merge_kernel<T, KT>, dim3(batch, (heads + 7) / 8), dim3(256), 0, stream, p, sms);
+    cudaError_t e = once.run([] { return cudaFuncSetAttribute(attn_latent_kernel<T, KT, NH>, cudaFuncAttributeMaxDynamicSharedMemorySize, kLaSmem); });
+    if (e == cudaSuccess) e = launch_pdl(attn_latent_kernel<T, KT, NH>, dim3(sms), dim3(kLaThreads), pl.smem, stream, tq, tk, p);
+    if (e == cudaSuccess) e = launch_pdl(attn_latent_merge_kernel<T>, dim3(batch, (heads * per + 7) / 8), dim3(256),
+                                          per > 1 ? (size_t)8 * rank * sizeof(float) : 0, stream, p, sms, per);
     return (int)e;
   };
+  auto wide = [&](auto type, auto keys) {
+    return pl.nh == 16 ? go(type, keys, std::integral_constant<int, 16>{}) : pl.nh == 32 ? go(type, keys, std::integral_constant<int, 32>{})
+                                                                                           : go(type, keys, std::integral_constant<int, 64>{});
+  };
   auto tall = [&](auto type) {
-    return pl.kt == 128 ? go(type, std::integral_constant<int, 128>{}) : go(type, std::integral_constant<int, 64>{});
+    return pl.kt == 128 ? wide(type, std::integral_constant<int, 128>{}) : wide(type, std::integral_constant<int, 64>{});
   };
   return dtype == 1 ? tall(__nv_bfloat16{}) : tall(__half{});
 }

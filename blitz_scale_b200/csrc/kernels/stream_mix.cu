@@ -11,7 +11,7 @@
 // its identity experts times what the sublayer read.
 //
 // No reduction over the columns: a thread owns four columns and walks tokens, with the coefficients of its layer and its
-// columns' weights in registers.
+// columns' weights in registers.  The rows of the next token's experts are looked up a token ahead.
 #include "launch.cuh"
 #include "ptx.cuh"
 #include "scalar.cuh"
@@ -61,9 +61,15 @@ __device__ __forceinline__ void cols_store(T* p, const Cols<VEC>& c) {
   else stf<T>(p, c.v[0]);
 }
 
+// As they lie in memory.
+template <typename T, int VEC>
+struct alignas(VEC * sizeof(T)) RawCols {
+  T e[VEC];
+};
+
 enum SmPending : int { kSmNone = 0, kSmDense = 1, kSmRows = 2 };
 
-template <typename T, int VEC, int S, int PEND>
+template <typename T, int VEC, int S, int PEND, int AT_ONCE>
 __global__ void __launch_bounds__(256) stream_mix_kernel(const StreamMixParams p) {
   ptx::griddep_launch_dependents();
   const int64_t H = p.hidden;
@@ -89,8 +95,16 @@ __global__ void __launch_bounds__(256) stream_mix_kernel(const StreamMixParams p
   }
   ptx::griddep_wait();
   if (!on) return;
+  auto source = [&](int t) { return p.rows ? p.rows[t] + p.row_offset : t; };
+  int place[AT_ONCE];  // the first rows of a token
+  auto look_up = [&](int src) {
+    const int32_t* rows = p.add_row + static_cast<int64_t>(src) * p.n_add;
+#pragma unroll
+    for (int k = 0; k < AT_ONCE; ++k) place[k] = k < p.n_add ? rows[k] : -1;
+  };
+  if (PEND == kSmRows && static_cast<int>(blockIdx.x) < p.tokens) look_up(source(blockIdx.x));
   for (int t = blockIdx.x; t < p.tokens; t += gridDim.x) {
-    const int src = p.rows ? p.rows[t] + p.row_offset : t;
+    const int src = source(t);
     Cols<VEC> x[S];
     float* xr = p.x + static_cast<int64_t>(src) * S * H + c;
     if (p.from_embed) {
@@ -106,46 +120,52 @@ __global__ void __launch_bounds__(256) stream_mix_kernel(const StreamMixParams p
     }
     if (PEND != kSmNone) {
       Cols<VEC> y = {};
-      auto add = [&](float f, const Cols<VEC>& r) {
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) y.v[i] += f * r.v[i];
-      };
       const T* yp = reinterpret_cast<const T*>(p.y) + c;
       if (PEND == kSmDense) {
         y = cols_load<T, VEC>(yp + src * H);
       } else {
-        const int32_t* rows = p.add_row + static_cast<int64_t>(src) * p.n_add;
-        for (int k0 = 0; k0 < p.n_add; k0 += 4) {  // four rows requested at once
-          int r[4];
-          Cols<VEC> v[4];
+        using Raw = RawCols<T, VEC>;
+        auto get = [&](const T* q) { return *reinterpret_cast<const Raw*>(q); };
+        auto sum = [&](float f, const Raw& r) {
 #pragma unroll
-          for (int k = 0; k < 4; ++k) r[k] = k0 + k < p.n_add ? rows[k0 + k] : -1;
+          for (int i = 0; i < VEC; ++i) y.v[i] += f * ldf<T>(&r.e[i]);
+        };
+        Raw v[AT_ONCE], same;
+        float f = 0.f, use[AT_ONCE];
 #pragma unroll
-          for (int k = 0; k < 4; ++k)
-            if (r[k] >= 0) v[k] = cols_load<T, VEC>(yp + r[k] * H);
-#pragma unroll
-          for (int k = 0; k < 4; ++k)
-            if (r[k] >= 0) add(1.f, v[k]);
+        for (int k = 0; k < AT_ONCE; ++k) {  // all requested before the first is used
+          use[k] = place[k] >= 0 ? 1.f : 0.f;
+          v[k] = get(yp + max(place[k], 0) * H);
         }
         if (p.ident) {
-          const float f = p.ident[src];
-          if (f != 0.f) add(f, cols_load<T, VEC>(reinterpret_cast<const T*>(p.prev) + src * H + c));
+          f = p.ident[src];
+          same = get(reinterpret_cast<const T*>(p.prev) + src * H + c);
         }
+        if (t + static_cast<int>(gridDim.x) < p.tokens) look_up(source(t + gridDim.x));
+#pragma unroll
+        for (int k = 0; k < AT_ONCE; ++k)
+          if (use[k] != 0.f) sum(1.f, v[k]);
+        for (int k = AT_ONCE; k < p.n_add; ++k) {
+          const int r = p.add_row[static_cast<int64_t>(src) * p.n_add + k];
+          if (r >= 0) sum(1.f, get(yp + r * H));
+        }
+        if (f != 0.f) sum(f, same);
       }
-      Cols<VEC> n[S];
 #pragma unroll
-      for (int t2 = 0; t2 < S; ++t2)
+      for (int i = 0; i < VEC; ++i) {
+        float n[S];
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) {
-          float a = ow[t2] * y.v[i];
+        for (int t2 = 0; t2 < S; ++t2) {
+          n[t2] = ow[t2] * y.v[i];
 #pragma unroll
-          for (int s = 0; s < S; ++s) a = fmaf(mix[s][t2], x[s].v[i], a);
-          n[t2].v[i] = a;
+          for (int s = 0; s < S; ++s) n[t2] = fmaf(mix[s][t2], x[s].v[i], n[t2]);
         }
 #pragma unroll
-      for (int s = 0; s < S; ++s) {
-        x[s] = n[s];
-        if (p.write) cols_store<float, VEC>(xr + s * H, x[s]);
+        for (int s = 0; s < S; ++s) x[s].v[i] = n[s];
+      }
+      if (p.write) {
+#pragma unroll
+        for (int s = 0; s < S; ++s) cols_store<float, VEC>(xr + s * H, x[s]);
       }
     }
     if (p.h == nullptr && p.u == nullptr) continue;
@@ -175,9 +195,10 @@ static cudaError_t launch_stream_mix(const StreamMixParams& p, cudaStream_t stre
   // a block that walks several tokens reads the coefficients once
   const int most = (device_sm_count() * (2048 / threads) + chunks - 1) / chunks;
   const dim3 grid(p.tokens < most ? p.tokens : most, chunks), block(threads);
-  if (p.y == nullptr) return launch_pdl(stream_mix_kernel<T, VEC, S, kSmNone>, grid, block, 0, stream, p);
-  if (p.add_row == nullptr) return launch_pdl(stream_mix_kernel<T, VEC, S, kSmDense>, grid, block, 0, stream, p);
-  return launch_pdl(stream_mix_kernel<T, VEC, S, kSmRows>, grid, block, 0, stream, p);
+  if (p.y == nullptr) return launch_pdl(stream_mix_kernel<T, VEC, S, kSmNone, 1>, grid, block, 0, stream, p);
+  if (p.add_row == nullptr) return launch_pdl(stream_mix_kernel<T, VEC, S, kSmDense, 1>, grid, block, 0, stream, p);
+  if (p.n_add <= 4) return launch_pdl(stream_mix_kernel<T, VEC, S, kSmRows, 4>, grid, block, 0, stream, p);
+  return launch_pdl(stream_mix_kernel<T, VEC, S, kSmRows, 8>, grid, block, 0, stream, p);
 }
 
 }  // namespace blitz

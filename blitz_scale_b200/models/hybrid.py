@@ -303,7 +303,7 @@ class HybridRunner:
             g = gate[:n] if gate is not None else None
             if single and ops.attn_latent_supported(ql, n, H, kv):
                 ops.attn_latent(ql, kv, m.page_indices, m.page_indptr[:n + 1], m.last_page_len[:n], heads=H, scale=mx.scale,
-                                workspace=self._latent_ws, out=ol, gate=g)
+                                workspace=self._latent_ws, out=ol, gate=g, static_table=True)
             else:
                 ops.attn_ragged(ql, kv, m.pos, None if single else m.tok_indptr, m.page_indptr[:n + 1] if single else m.page_indptr,
                                 m.page_indices, ol, q_heads=H, kv_heads=1, dim=W, page_size=self.page_size, scale=mx.scale, gate=g)

@@ -595,15 +595,18 @@ def attn_latent_workspace(heads: int, rank: int, device) -> torch.Tensor:
 
 
 def attn_latent(q: torch.Tensor, kv: LatentKV, indices: torch.Tensor, indptr: torch.Tensor, last_page_len: torch.Tensor, *, heads: int,
-                scale: float, workspace: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                scale: float, workspace: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None,
+                keys: int = 0, static_table: bool = False) -> torch.Tensor:
     """Decode attention over latent rows: q [batch, heads * width] against every cached row as it is, out [batch, heads * rank] =
-    the weighted sums of the rows' first ``rank`` columns, times the sigmoid of ``gate`` [batch, heads]."""
+    the weighted sums of the rows' first ``rank`` columns, times the sigmoid of ``gate`` [batch, heads].  ``keys``: per block, 64 or 128 (0: chosen).
+    ``static_table`` promises that no kernel still running in this stream writes the page table (indices, indptr,
+    last_page_len), so that the work list can be made before the predecessor has finished."""
     B = indptr.numel() - 1
     pages, page, _, width = kv.pool.shape
     assert q.shape == (B, heads * width) and out.shape == (B, heads * kv.rank) and q.stride(1) == 1 and out.stride(1) == 1
     assert workspace.numel() >= int(lib().blitz_attn_latent_workspace_bytes(heads, kv.rank))
     _check(lib().blitz_attn_latent(_p(q), q.stride(0), _p(kv.pool), _p(indices), _p(indptr), _p(last_page_len), _p(out), out.stride(0),
-                                   _p(workspace), B, heads, width, kv.rank, page, pages, scale, *_gate(gate), _p(status_word(q.device)),
+                                   _p(workspace), B, heads, width, kv.rank, page, pages, scale, *_gate(gate), keys, int(static_table), _p(status_word(q.device)),
                                    _dt(q), _stream()), "blitz_attn_latent")
     return out
 
