@@ -83,10 +83,13 @@ def bench_models(out, sizes=("h4096", "h2048"), configs=configs):
                 if cfg.family == "hybrid":
                     for e in (s.moe for s in cfg.layer_specs if s.moe):
                         # experts that no token of the step chooses are not read (expected number, choices being random)
-                        weights -= e.experts * (1 - e.top / e.experts) ** B * 4 * cfg.hidden * e.ff_pad
+                        weights -= e.experts * (1 - e.top / e.outputs) ** B * 2 * cfg.hidden * (e.up_cols + e.ff_pad)
+                    for x in (s.mixer for s in cfg.layer_specs if s.mixer.kind == "latent"):
+                        weights -= 2 * x.heads * (x.width * x.qdim + x.kv_rank * x.vdim)      # of prompts only
                     # window and kept tokens of the attention layers; states are read and written
                     kv = sum(x.kv_heads * (x.dim + x.vdim) * 2 * (min(ctx, x.window + x.keep_first) if x.window else ctx)
                              for x in cfg.run_mixers() if x.kind == "attention")
+                    kv += sum(x.width * 2 * ctx for x in cfg.run_mixers() if x.kind == "latent")
                     data = B * (kv + 2 * cfg.state_bytes_per_sequence())
                 else:
                     data = B * ctx * cfg.kv_bytes_per_token()

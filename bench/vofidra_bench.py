@@ -92,7 +92,8 @@ def bench_kernels(out, size):
         h, W, R = la["heads"], la["kv_rank"] + la["rot_dim"], la["kv_rank"]
         pools = [ops.LatentKV(rnd(idx.numel(), 64, 1, W), R) for _ in range(min(40, n_copies(2 * B * ctx * W)))]
         q, o, gate, ws = rnd(B, h * W), torch.empty(B, h * R, dtype=bf, device=dev), rnd(B, h), ops.attn_latent_workspace(h, R, dev)
-        t = timeit(lambda i: ops.attn_latent(q, pools[i], idx, indptr, last, heads=h, scale=W ** -0.5, workspace=ws, out=o, gate=gate), copies=len(pools))
+        t = timeit(lambda i: ops.attn_latent(q, pools[i], idx, indptr, last, heads=h, scale=W ** -0.5, workspace=ws, out=o, gate=gate, static_table=True),
+                   copies=len(pools))
         rep("attn_latent", t, by=2.0 * B * ctx * W + 2.0 * B * h * (W + R), fl=2.0 * B * ctx * h * (W + R), batch=B, ctx=ctx)
         del pools
     # ---- what surrounds the latent: block-diagonal products, beside an ordinary product of the same size
@@ -148,13 +149,14 @@ def bench_kernels(out, size):
         x1 = [torch.randn(T, H, device=dev) for _ in range(min(40, n_copies(T * H * 4)))]
         per = top
         y, rows, ident = rnd(T * per, H), torch.randperm(T * per, device=dev).to(torch.int32).view(T, per), torch.rand(T, device=dev)
+        every = rows.clone()
         rows[torch.rand(T, per, device=dev) < I / (E + I)] = -1
         real = float((rows >= 0).sum()) / T
         mix, v = rnd(STREAMS, STREAMS), rnd(STREAMS)
         norm = (w, torch.full((1,), 0.5, dtype=bf, device=dev), w)
         t = timeit(lambda i: ops.stream_norm(x1[i], w, 1e-6, o), copies=len(x1))
         rep("stream_norm (Komulorn)", t, by=T * H * 6.0, tokens=T)
-        t = timeit(lambda i: ops.stream_norm(x1[i], w, 1e-6, o, add=y, add_rows=rows.clamp(min=0)), copies=len(x1))
+        t = timeit(lambda i: ops.stream_norm(x1[i], w, 1e-6, o, add=y, add_rows=every), copies=len(x1))
         rep("stream_norm with the experts' rows (Komulorn)", t, by=T * H * (10.0 + 2.0 * per), tokens=T)
         pd = ops.Pending(y[:T], mix, v)
         t = timeit(lambda i: ops.stream_mix(xf[i], pending=pd, read=v, norm=norm, out=o, write=True), copies=nc)

@@ -25,6 +25,9 @@
 // are: the work list follows from the page table on the device, so that the launch can be captured in a graph.  A CTA's
 // share begins and ends anywhere in a sequence; it leaves at most two incomplete pieces (fp32 partial sums), which a second
 // kernel merges.
+//
+// The tokens of prompts go through the same kernel, each as a row of its own that sees the keys up to its position (for models
+// whose expanded heads the prompt kernel does not take).
 #include "launch.cuh"
 #include "ptx.cuh"
 #include "scalar.cuh"
@@ -42,6 +45,8 @@ constexpr int kLaSmem = 227 * 1024;
 
 struct LatentParams {
   const int32_t *indices, *indptr, *last_page_len;
+  const int32_t *pos, *tok_indptr;  // rows are tokens of prompts: their positions, and the first tokens of `rows` sequences
+  int rows, first_token;            // (else null: a row per sequence)
   void* out;                    // [batch][out_stride], head h's rank columns from h * rank on
   const void* gate;             // [batch][gate_stride], or null
   int64_t out_stride, gate_stride;
@@ -154,8 +159,8 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   int* s_share = reinterpret_cast<int*>(tmem_slot + 2);  // [4] this CTA's first block, end, sequence of the first
   int* s_sums = s_share + 4;                             // [128] blocks of 32 sequences
   int* s_pref = s_sums + kLaMaxBatch / 32;               // [batch + 1] blocks before a sequence
-  int* s_page = s_pref + p.batch + 1;                   // [batch + 1] its first page entry
-  int* s_len = s_page + p.batch + 1;                    // [batch]
+  int* s_page = s_pref + p.batch + 1;                   // [batch] its first page entry
+  int* s_len = s_page + p.batch;                        // [batch]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   constexpr int kWarps = kLaThreads / 32;
 
@@ -192,10 +197,11 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     const int b = i * 32 + lane;
     int v = 0;
     if (b < p.batch) {
-      const int first = p.indptr[b], npages = p.indptr[b + 1] - first;
-      const int len = npages > 0 ? ((npages - 1) << p.page_shift) + p.last_page_len[b] : 0;
+      const int row = p.pos ? row_of_token(p.tok_indptr, p.rows, p.first_token + b) : b;
+      const int first = p.indptr[row], npages = p.indptr[row + 1] - first;
+      int len = 0;
+      if (npages > 0) len = p.pos ? min(p.pos[b] + 1, npages << p.page_shift) : ((npages - 1) << p.page_shift) + p.last_page_len[b];
       s_page[b] = first;
-      if (b == p.batch - 1) s_page[b + 1] = first + npages;
       s_len[b] = len;
       v = (len + KT - 1) / KT;
     }
@@ -217,8 +223,8 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   }
   __syncthreads();
   {
-    const int total = s_pref[p.batch] * p.subs, G = gridDim.x, cta = blockIdx.x;
-    const int x = total * cta / G, hi = total * (cta + 1) / G;
+    const int64_t total = s_pref[p.batch] * p.subs;
+    const int x = static_cast<int>(total * blockIdx.x / gridDim.x), hi = static_cast<int>(total * (blockIdx.x + 1) / gridDim.x);
     if (threadIdx.x == 0) {
       s_share[0] = x;
       s_share[1] = hi;
@@ -250,9 +256,8 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     };
     auto box_row = [&](const LaPiece& q, int blk) {  // this lane's first row of a block in the pool
       const int tok = blk * KT + lane * bt, slot = tok >> p.page_shift;
-      const int pg0 = s_page[q.b], npages = s_page[q.b + 1] - pg0;
-      if (!mine || slot >= npages) return p.oob_row;  // past the pool: the box arrives as zeros
-      int page = p.indices[pg0 + slot];
+      if (!mine || tok >= s_len[q.b]) return p.oob_row;  // past the pool: the box arrives as zeros
+      int page = p.indices[s_page[q.b] + slot];
       if (page < 0 || page >= p.max_pages) {
         if (p.status) atomicCAS(p.status, 0, kStatusBadIndex);
         page = 0;
@@ -580,7 +585,8 @@ __global__ void __launch_bounds__(256) attn_latent_merge_kernel(const LatentPara
   const int b = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head = blockIdx.y * (8 / per) + warp / per, share = warp % per;
   if (head >= p.heads) return;  // (with several warps per head: all of a block or none)
-  const int before = p.blocks_before[b], blocks = p.blocks_before[b + 1] - before, total = p.blocks_before[p.batch] * p.subs;
+  const int before = p.blocks_before[b], blocks = p.blocks_before[b + 1] - before, all = p.blocks_before[p.batch] * p.subs;
+  const int64_t total = all;
   T* dst = reinterpret_cast<T*>(p.out) + b * p.out_stride + static_cast<int64_t>(head) * p.rank;
   if (blocks == 0) {
     if (share == 0)
@@ -588,7 +594,8 @@ __global__ void __launch_bounds__(256) attn_latent_merge_kernel(const LatentPara
     return;
   }
   const int beg = before * p.subs + head / p.group * blocks;
-  const int c0 = ((beg + 1) * ctas - 1) / total, c1 = ((beg + blocks) * ctas - 1) / total;
+  auto cta_of = [&](int block) { return static_cast<int>(((block + 1) * static_cast<int64_t>(ctas) - 1) / total); };
+  const int c0 = cta_of(beg), c1 = cta_of(beg + blocks - 1);
   if (c0 == c1) return;  // one CTA has done all of it
   constexpr int kRounds = kLaMaxCtas / 32;
   float w[kRounds];
@@ -599,10 +606,10 @@ __global__ void __launch_bounds__(256) attn_latent_merge_kernel(const LatentPara
     w[i] = -INFINITY;
     at[i] = -1;
     if (c0 + i * 32 > c1) continue;
-    const int c = c0 + i * 32 + lane, lo = total * c / ctas;
+    const int c = c0 + i * 32 + lane, lo = static_cast<int>(total * c / ctas);
     // the piece is its CTA's first one unless the CTA's share begins before this sequence; with more CTAs than blocks some
     // have none
-    if (c <= c1 && lo < total * (c + 1) / ctas) {
+    if (c <= c1 && lo < static_cast<int>(total * (c + 1) / ctas)) {
       at[i] = (c * 2 + (lo < beg ? 1 : 0)) * p.group + head % p.group;
       w[i] = p.part_lse[at[i]];
     }
@@ -666,7 +673,7 @@ static bool latent_plan(int batch, int heads, int width, int rank, int page_size
     if (heads % groups || heads / groups > kLaMaxHeads) continue;
     pl.group = heads / groups;
     pl.nh = pl.group <= 16 ? 16 : pl.group <= 32 ? 32 : 64;
-    const int fixed = 1024 + 6 * pl.nh * 4 + (12 + 2 * kLaMaxStages) * 8 + 8 + 16 + kLaMaxBatch / 32 * 4 + (batch + 1) * 12;
+    const int fixed = 1024 + 6 * pl.nh * 4 + (12 + 2 * kLaMaxStages) * 8 + 8 + 16 + kLaMaxBatch / 32 * 4 + (3 * batch + 1) * 4;
     const int tall_first = pl.nh <= 32;
     for (int i = 0; i < 2; ++i) {
       const int kt = (i == 0) == (tall_first != 0) ? 128 : 64;
@@ -706,18 +713,19 @@ int64_t blitz_attn_latent_workspace_bytes(int heads, int rank) {
 // q [batch][q_stride]: heads of `width` columns; pool [max_pages][page_size][width], the first `rank` columns are the values;
 // out [batch][out_stride]: heads of `rank` columns.  width, rank: multiples of 8, rank up to 512; page_size: a power of two >= 8;
 // gate [batch][gate_stride] or null.  A row without pages gives zeros.  kt_hint: keys per block, 0 = choose, else 64 or 128.
-// static_table: no kernel still running in the stream writes indices, indptr or last_page_len.
+// static_table: no kernel still running in the stream writes indices, indptr, last_page_len, pos or tok_indptr.
+// pos [batch], tok_indptr [rows + 1] (both or none): the batch are tokens first_token .. of `rows` sequences, whose pages indptr
+// [rows + 1] names; each sees the keys up to its position.  last_page_len is not read then.
 int blitz_attn_latent(const void* q, int64_t q_stride, const void* pool, const int32_t* indices, const int32_t* indptr,
-                      const int32_t* last_page_len, void* out, int64_t out_stride, void* workspace, int batch, int heads, int width, int rank,
+                      const int32_t* last_page_len, const int32_t* pos, const int32_t* tok_indptr, int rows, int first_token, void* out, int64_t out_stride, void* workspace, int batch, int heads, int width, int rank,
                       int page_size, int max_pages, float sm_scale, const void* gate, int64_t gate_stride, int kt_hint, int static_table, int* status, int dtype,
                       cudaStream_t stream) {
   if (batch <= 0) return 0;
   LatentPlan pl;
   if (!latent_plan(batch, heads, width, rank, page_size, kt_hint, &pl) || workspace == nullptr || max_pages < 1) return -1;
+  if ((pos == nullptr) != (tok_indptr == nullptr) || (pos && rows < 1)) return -1;
   if ((q_stride & 7) || (reinterpret_cast<uintptr_t>(workspace) & 15)) return -1;
   const int sms = device_sm_count() < kLaMaxCtas ? device_sm_count() : kLaMaxCtas;
-  // block numbers times CTAs are 32-bit
-  if (((int64_t)max_pages * page_size / 64 + batch) * (heads / pl.group) * (sms + 1) >= ((int64_t)1 << 31)) return -1;
   const int bt = page_size < 64 ? page_size : 64;
   CUtensorMap tq, tk;
   if (!get_tmap_3d(&tq, q, (uint64_t)width, (uint64_t)heads, (uint64_t)batch, (uint64_t)width * 2, (uint64_t)q_stride * 2, 64,
@@ -725,7 +733,8 @@ int blitz_attn_latent(const void* q, int64_t q_stride, const void* pool, const i
     return -2;
   if (!get_tmap_2d(&tk, pool, (uint64_t)width, (uint64_t)max_pages * page_size, (uint64_t)width * 2, 64, (uint32_t)bt)) return -2;
   LatentParams p;
-  p.indices = indices; p.indptr = indptr; p.last_page_len = last_page_len; p.out = out; p.gate = gate;
+  p.indices = indices; p.indptr = indptr; p.last_page_len = last_page_len;
+  p.pos = pos; p.tok_indptr = tok_indptr; p.rows = rows; p.first_token = first_token; p.out = out; p.gate = gate;
   p.out_stride = out_stride; p.gate_stride = gate_stride;
   p.batch = batch; p.heads = heads; p.group = pl.group; p.subs = heads / pl.group; p.rank = rank;
   p.slabs = pl.slabs; p.steps = (width + 15) / 16; p.stages = pl.stages; p.q_bufs = pl.q_bufs;

@@ -26,6 +26,7 @@ sublayer before it, joins them and norms the result::
                single tokens: block-diagonal GEMM (queries into the latent space) -> rotation -> attention over the cached
                rows, one key and value for all heads -> block-diagonal GEMM (values out of the latent space);
                prompts: rotation -> gather of the cached rows -> GEMMs (keys, values of all heads) -> attention
+               (heads that the prompt kernel does not take: as single tokens)
     gla:       one kernel (decay projection, recurrence, output norm, gate), or the chunked kernels for prompts
     rglru:     conv_causal -> block-diagonal GEMM (gates, fp32 out) -> rglru_scan
 
@@ -301,9 +302,11 @@ class HybridRunner:
             ops.latent_rotate(q[:n], ql[:, R:], m.pos[:n], freqs, out_step=W, **rotate)
             single = not m.is_prefill or n == m.singles
             g = gate[:n] if gate is not None else None
-            if single and ops.attn_latent_supported(ql, n, H, kv):
-                ops.attn_latent(ql, kv, m.page_indices, m.page_indptr[:n + 1], m.last_page_len[:n], heads=H, scale=mx.scale,
-                                workspace=self._latent_ws, out=ol, gate=g, static_table=True)
+            if ops.attn_latent_supported(ql, n if single else min(n, ops.ATTN_LATENT_ROWS), H, kv):
+                rows = m.batch if not single else n
+                ops.attn_latent(ql, kv, m.page_indices, m.page_indptr[:rows + 1], m.last_page_len[:rows], heads=H, scale=mx.scale,
+                                workspace=self._latent_ws, out=ol, gate=g, static_table=True,
+                                **({} if single else dict(pos=m.pos[:n], tok_indptr=m.tok_indptr)))
             else:
                 ops.attn_ragged(ql, kv, m.pos, None if single else m.tok_indptr, m.page_indptr[:n + 1] if single else m.page_indptr,
                                 m.page_indices, ol, q_heads=H, kv_heads=1, dim=W, page_size=self.page_size, scale=mx.scale, gate=g)

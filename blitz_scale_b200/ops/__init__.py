@@ -594,21 +594,39 @@ def attn_latent_workspace(heads: int, rank: int, device) -> torch.Tensor:
     return torch.empty(int(lib().blitz_attn_latent_workspace_bytes(heads, rank)), dtype=torch.uint8, device=device)
 
 
+ATTN_LATENT_ROWS = 1024     # tokens of prompts in one launch
+
+
 def attn_latent(q: torch.Tensor, kv: LatentKV, indices: torch.Tensor, indptr: torch.Tensor, last_page_len: torch.Tensor, *, heads: int,
                 scale: float, workspace: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None,
-                keys: int = 0, static_table: bool = False) -> torch.Tensor:
+                keys: int = 0, static_table: bool = False, pos: Optional[torch.Tensor] = None,
+                tok_indptr: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Decode attention over latent rows: q [batch, heads * width] against every cached row as it is, out [batch, heads * rank] =
-    the weighted sums of the rows' first ``rank`` columns, times the sigmoid of ``gate`` [batch, heads].  ``keys``: per block, 64 or 128 (0: chosen).
+    the weighted sums of the rows' first ``rank`` columns, times the sigmoid of ``gate`` [batch, heads].  With ``pos`` and
+    ``tok_indptr`` the batch are the tokens of a ragged step (as for `attn_ragged`), each sees the keys up to its position.  ``keys``: per block, 64 or 128 (0: chosen).
     ``static_table`` promises that no kernel still running in this stream writes the page table (indices, indptr,
     last_page_len), so that the work list can be made before the predecessor has finished."""
-    B = indptr.numel() - 1
+    assert (pos is None) == (tok_indptr is None)
+    B = q.shape[0]
+    if pos is not None and B > ATTN_LATENT_ROWS:
+        for t in range(0, B, ATTN_LATENT_ROWS):
+            part = slice(t, min(B, t + ATTN_LATENT_ROWS))
+            _attn_latent(q[part], kv, indices, indptr, last_page_len, heads, scale, workspace, out[part], None if gate is None else gate[part],
+                         keys, static_table, pos[part], tok_indptr, t)
+        return out
+    _attn_latent(q, kv, indices, indptr, last_page_len, heads, scale, workspace, out, gate, keys, static_table, pos, tok_indptr, 0)
+    return out
+
+
+def _attn_latent(q, kv, indices, indptr, last_page_len, heads, scale, workspace, out, gate, keys, static_table, pos, tok_indptr, first) -> None:
+    rows = indptr.numel() - 1
+    B = rows if pos is None else q.shape[0]
     pages, page, _, width = kv.pool.shape
     assert q.shape == (B, heads * width) and out.shape == (B, heads * kv.rank) and q.stride(1) == 1 and out.stride(1) == 1
     assert workspace.numel() >= int(lib().blitz_attn_latent_workspace_bytes(heads, kv.rank))
-    _check(lib().blitz_attn_latent(_p(q), q.stride(0), _p(kv.pool), _p(indices), _p(indptr), _p(last_page_len), _p(out), out.stride(0),
-                                   _p(workspace), B, heads, width, kv.rank, page, pages, scale, *_gate(gate), keys, int(static_table), _p(status_word(q.device)),
+    _check(lib().blitz_attn_latent(_p(q), q.stride(0), _p(kv.pool), _p(indices), _p(indptr), _p(last_page_len), _p(pos),
+                                   _p(tok_indptr), rows, first, _p(out), out.stride(0), _p(workspace), B, heads, width, kv.rank, page, pages, scale, *_gate(gate), keys, int(static_table), _p(status_word(q.device)),
                                    _dt(q), _stream()), "blitz_attn_latent")
-    return out
 
 
 # ---------------------------------------------------------------------------------------------- mixture of experts

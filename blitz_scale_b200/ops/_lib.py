@@ -104,7 +104,7 @@ def _declare(L: ctypes.CDLL) -> None:
     sig("blitz_latent_rotate", [c_p, c_i64, c_p, c_i64, c_i, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_p])
     sig("blitz_attn_latent_supported", [c_i, c_i, c_i, c_i, c_i], c_i)
     sig("blitz_attn_latent_workspace_bytes", [c_i, c_i], c_i64)
-    sig("blitz_attn_latent", [c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_p, c_i64, c_i, c_i, c_p, c_i, c_p])
+    sig("blitz_attn_latent", [c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_p, c_i64, c_i, c_i, c_p, c_i, c_p])
     sig("blitz_latent_gather", [c_p, c_p, c_p, c_i, c_i64, c_i, c_p, c_p])
     sig("blitz_attn_ragged", [c_p, c_i64, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_i,
                               c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_p, c_i, c_p])

@@ -90,7 +90,7 @@ def test_token_by_token_from_the_first(folders, dtype):
 
 @pytest.mark.parametrize("graphs", [True, False])
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["regular", "odd", "values", "wide"])
+@pytest.mark.parametrize("name", ["regular", "odd", "values", "wide", "deep"])
 def test_mixed_batch_with_reused_pages(folders, name, dtype, graphs):
     """Unequal requests side by side: portions of some beside single tokens of others, one sitting out, and later ones on
     the pages of those that have ended; a pool that holds no more than the live ones need."""

@@ -299,6 +299,28 @@ def test_latent_decode_attention(ops, case, lens):
             check("tensor cores")
 
 
+@pytest.mark.parametrize("H,W,R,page", [(5, 136, 104, 16), (32, 544, 512, 64), (72, 80, 64, 32)])
+def test_latent_attention_of_prompt_tokens(ops, H, W, R, page):
+    """Tokens of a ragged step as rows of their own, behind any prefix, in several launches: against the general kernel."""
+    lens, q_lens = [900, 1, 65, 300, 1100], [900, 1, 2, 260, 130]
+    g = torch.Generator().manual_seed(H)
+    npages = [-(-n // page) for n in lens]
+    perm = torch.randperm(sum(npages), generator=g).tolist()
+    kv = ops.LatentKV(torch.randn(sum(npages), page, 1, W, generator=g).to(DEV, BF), R)
+    T = sum(q_lens)
+    q, gate = torch.randn(T, H * W, generator=g).to(DEV, BF), torch.randn(T, H, generator=g).to(DEV, BF)
+    pos = _i32([p for n, ql in zip(lens, q_lens) for p in range(n - ql, n)])
+    tokp, indptr = (_i32([sum(x[:i]) for i in range(len(lens) + 1)]) for x in (q_lens, npages))
+    want, got = torch.empty(T, H * R, dtype=BF, device=DEV), torch.full((T, H * R), math.nan, dtype=BF, device=DEV)
+    scale = 1.2 * W ** -0.5
+    ops.attn_ragged(q, kv, pos, tokp, indptr, _i32(perm), want, q_heads=H, kv_heads=1, dim=W, page_size=page, scale=scale, gate=gate)
+    ops.attn_latent(q, kv, _i32(perm), indptr, indptr, heads=H, scale=scale, workspace=ops.attn_latent_workspace(H, R, DEV), out=got, gate=gate,
+                    pos=pos, tok_indptr=tokp)
+    ops.check_status()
+    err = (got.float() - want.float()).norm(dim=1) / want.float().norm(dim=1)
+    assert float(err.max()) < 2e-2, int(err.argmax())
+
+
 @pytest.mark.parametrize("M", [1, 5, 130, 300])
 @pytest.mark.parametrize("G,K,N,a_step,out_step", [(5, 48, 104, 80, 136), (32, 64, 256, 96, 288), (3, 13, 21, 19, 27), (4, 256, 64, 256, 64), (2, 72, 40, 72, 40),
                                                    (1, 24, 16, 40, 24), (8, 200, 8, 208, 16)])

@@ -114,9 +114,12 @@ CASES = {
     # values of another size than keys, twelve query heads on a key head, one stream, no groups, no identity experts
     "values": config([attention(heads=12, kv_heads=1, dim=128, vdim=96, rows=32, bias_max=64, temp=(0.2, 7)), latent(heads=2, dim=96, rot_dim=32, vdim=128, q_rank=64, kv_rank=256)],
                      [moe(experts=5, identity=0, top=2, groups=None), dense(ff=64)], width=136, vocab=152, cap=5.0, streams=1),
-    # a latent of two value halves, queries in two head groups, many streams
+    # a latent of several chunks of value columns, many streams
     "wide": config([latent(heads=32, dim=16, rot_dim=64, vdim=16, q_rank=40, kv_rank=320, scale=0.05), attention(heads=4, kv_heads=4, dim=40, vdim=24, rows=11, bias_max=50)],
                    [moe(experts=20, identity=12, top=6, ff=32, groups=(8, 3)), moe(experts=2, identity=6, top=4, ff=24, groups=(2, 1))], width=96, vocab=128, streams=5),
+    # expanded heads larger than the prompt kernel takes: prompts stay in the latent space; more than 64 heads
+    "deep": config([latent(heads=3, dim=120, rot_dim=40, vdim=136, q_rank=72, kv_rank=72), latent(heads=72, dim=8, rot_dim=16, vdim=8, q_rank=64, kv_rank=136, scale=0.1)],
+                   [None, moe()], width=104, vocab=144, streams=4),
     # nothing a multiple of 8
     "odd": config([latent(heads=3, dim=13, rot_dim=6, vdim=11, q_rank=35, kv_rank=21), attention(heads=9, kv_heads=3, dim=22, vdim=13, rows=7, bias_max=12, temp=(1.5, 3))],
                   [dense(ff=51), moe(experts=4, identity=1, top=2, ff=33, groups=None)], width=121, vocab=157, streams=2),
