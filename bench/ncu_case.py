@@ -3,6 +3,7 @@
     python bench/ncu_case.py gemm M N K [epilogue]       # 3 launches of the tcgen05 GEMM
     python bench/ncu_case.py attn_decode B CTX            # 3 launches of the paged decode attention
     python bench/ncu_case.py experts T                    # 3 rounds of router, grouped up and grouped down product
+    python bench/ncu_case.py latent B CTX                 # 3 launches of latent decode attention, and of stream_mix over B * CTX / 32 tokens
     python bench/ncu_case.py attn_prefill_paged B N       # 3 launches of the paged prefill attention (64-token pages)
 """
 import os
@@ -57,6 +58,23 @@ def main():
             ops.moe_route(z, plan)
             ops.gemm_grouped(h, up, plan, act, shared=s_up, gather=True, act="relu2", factors=True)
             ops.gemm_grouped(act, down, plan, y, shared=s_down)
+    elif kind == "latent":
+        B, ctx = map(int, sys.argv[2:4])
+        h, W, R, page, H, S = 32, 288, 256, 64, 2048, 4
+        npg = (ctx + page - 1) // page
+        rnd = lambda *s: torch.randn(*s, device="cuda", dtype=torch.bfloat16)
+        kv = ops.LatentKV(rnd(B * npg, page, 1, W), R)
+        idx = torch.randperm(B * npg, device="cuda").to(torch.int32)
+        indptr = (torch.arange(B + 1, device="cuda") * npg).to(torch.int32)
+        last = torch.full((B,), ctx - (npg - 1) * page, device="cuda", dtype=torch.int32)
+        q, o, gate, ws = rnd(B, h * W), rnd(B, h * R), rnd(B, h), ops.attn_latent_workspace(h, R, "cuda")
+        T = B * ctx // 32
+        x, y, hh = torch.randn(T, S, H, device="cuda"), rnd(T, H), rnd(T, H)
+        pending, norm = ops.Pending(y, rnd(S, S), rnd(S)), (rnd(H), rnd(1), rnd(H))
+        torch.cuda.synchronize()
+        for _ in range(3):
+            ops.attn_latent(q, kv, idx, indptr, last, heads=h, scale=W ** -0.5, workspace=ws, out=o, gate=gate)
+            ops.stream_mix(x, pending=pending, read=norm[2][:S].contiguous(), norm=norm, out=hh, write=True)
     elif kind == "decode_step":
         # two eager decode steps of the full model (no CUDA graph), for a per-kernel launch list of one step:
         #   ncu --metrics gpu__time_duration.sum -k regex:"blitz|gemm|attn|rms|rope|argmax|embedding|sample" ...

@@ -104,7 +104,7 @@ def bench_kernels(out, size):
         t = timeit(lambda i: ops.gemm(q, uk[i], out=ql, groups=h, a_step=kd, out_step=W, static_b=True), copies=nc)
         rep("gemm into the latent space (block-diagonal)", t, by=2.0 * (h * dm * R + M * h * (dm + R)), fl=2.0 * M * h * dm * R, M=M)
         uv, ol, o = [rnd(h * R, vd) for _ in range(nc)], rnd(M, h * R), torch.empty(M, h * vd, dtype=bf, device=dev)
-        t = timeit(lambda i: ops.gemm(ol, uv[i], out=o, groups=h, a_step=R, out_step=vd, static_b=True), copies=nc)
+        t = timeit(lambda i: ops.gemm(ol, uv[i], out=o, groups=h, a_step=R, out_step=vd, static_b=True, bn=64, split_k=1), copies=nc)
         rep("gemm out of the latent space (block-diagonal)", t, by=2.0 * (h * R * vd + M * h * (vd + R)), fl=2.0 * M * h * vd * R, M=M)
         gates = [rnd(4096, 512) for _ in range(40)]
         g_in, g_out = rnd(M, 4096), torch.empty(M, 16 * 512, device=dev)

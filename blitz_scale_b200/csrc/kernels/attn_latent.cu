@@ -661,9 +661,8 @@ struct LatentPlan {
   int kt, group, nh, slabs, stages, q_bufs;
   size_t smem;
 };
-// How the heads are grouped and how tall a key block is: as many heads as possible; blocks of 128 keys if two stages of them fit,
-// else of 64 (with more than 32 heads 64 first: four small stages beat two tall ones there); queries double buffered if that
-// leaves room.
+// How the heads are grouped and how tall a key block is: as many heads as possible; blocks of 64 keys, whose stages are more, or,
+// with few rows and heads, blocks of 128, which are through sooner; queries double buffered if that leaves room.
 static bool latent_plan(int batch, int heads, int width, int rank, int page_size, int kt_hint, LatentPlan* out) {
   if (batch < 1 || batch > kLaMaxBatch || heads < 1 || rank < 8 || rank > kLaMaxRank || width < rank || ((width | rank) & 7)) return false;
   if (page_size < 8 || (page_size & (page_size - 1)) != 0) return false;
@@ -674,7 +673,7 @@ static bool latent_plan(int batch, int heads, int width, int rank, int page_size
     pl.group = heads / groups;
     pl.nh = pl.group <= 16 ? 16 : pl.group <= 32 ? 32 : 64;
     const int fixed = 1024 + 6 * pl.nh * 4 + (12 + 2 * kLaMaxStages) * 8 + 8 + 16 + kLaMaxBatch / 32 * 4 + (3 * batch + 1) * 4;
-    const int tall_first = pl.nh <= 32;
+    const int tall_first = pl.nh <= 32 && batch < 64;
     for (int i = 0; i < 2; ++i) {
       const int kt = (i == 0) == (tall_first != 0) ? 128 : 64;
       if (kt_hint && kt != kt_hint) continue;

@@ -310,7 +310,9 @@ class HybridRunner:
             else:
                 ops.attn_ragged(ql, kv, m.pos, None if single else m.tok_indptr, m.page_indptr[:n + 1] if single else m.page_indptr,
                                 m.page_indices, ol, q_heads=H, kv_heads=1, dim=W, page_size=self.page_size, scale=mx.scale, gate=g)
-            ops.gemm(ol, self._w(l, "uv"), out=mid[:n, :H * mx.vdim], groups=H, a_step=R, out_step=mx.vdim, static_b=True)
+            # few rows: a tile per head is enough, and an exchange of K splits would cost more than it saves
+            narrow = dict(bn=64, split_k=1) if n <= ops.PAIR_GEMM_MAX_M else {}
+            ops.gemm(ol, self._w(l, "uv"), out=mid[:n, :H * mx.vdim], groups=H, a_step=R, out_step=mx.vdim, static_b=True, **narrow)
         if n < T:
             self._latent_prompts(l, mx, q, gate, kv, mid, m, n, freqs, rotate)
 
