@@ -13,8 +13,8 @@
 //                   column, a column per head, 128 value columns per instruction
 //
 // A head's probabilities refer to the score of the sequence's first key here, and to the maximum so far once some score has
-// exceeded that by more than 2^40 (in bf16 and fp32 a factor changes no digit; fp16: 2^8); one vote per block decides, and O and
-// the row sums are rescaled then.  Row sums stay in the threads until the end.
+// exceeded that by more than 2^40 (bf16 probabilities and fp32 sums have the range; fp16: 2^8); one vote per block decides, and O
+// and the row sums are rescaled then.  Row sums stay in the threads until the end.
 // More than 64 heads run as groups that read the same keys.
 //
 // A load warp, a warp for each product and the softmax warps walk the blocks on their own, also across sequences.  An MMA
