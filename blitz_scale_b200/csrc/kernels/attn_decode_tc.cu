@@ -41,6 +41,10 @@
 // A bias by distance per head, bias[h][min(i - j, bias_len - 1)], is added to the scaled scores; only chunks with a distance
 // inside the table look it up (four entries a lane, requested before the wait for the chunk).
 //
+// The window may be a chunk counted from position 0 (`chunked`: the keys of the position's own chunk are visible), and weights may
+// be sigmoids of the scores instead of a softmax (`sigmoid`): then nothing refers to a maximum or is normalised, and warps and
+// splits just add up.
+//
 // Replaces src/kernel/attention_decode.cu:13-40 and the host-side plan of
 // src/kernel/flashinfer_types.cu:52-80.
 #include "launch.cuh"
@@ -74,6 +78,7 @@ struct DecodeTcParams {
   int64_t gate_stride;
   int tail_box_tokens;  // box height of the second tensor map, used for the last (partly filled) chunk of a sequence
   float scale_log2;
+  int chunked, sigmoid;         // see the top of the file
   int window, keep_first;       // 0: every key; else a token sees the last `window` positions and the first `keep_first`
   float cap_scale, cap_log2;    // soft cap (cap_log2 > 0): score in log2 units = cap_log2 * tanh(q.k * cap_scale)
   const void* sink;             // [q_heads] in the activation type, or null
@@ -118,7 +123,7 @@ __device__ __forceinline__ DecItem dec_item(const DecodeTcParams& p, int item) {
   it.pg_beg = p.indptr[it.b];
   const int npages = p.indptr[it.b + 1] - it.pg_beg;
   it.seq_len = npages > 0 ? (npages - 1) * p.page_size + p.last_page_len[it.b] : 0;
-  it.lo = p.window > 0 ? max(0, it.seq_len - p.window) : 0;
+  it.lo = p.window > 0 ? (p.chunked ? max(0, it.seq_len - 1) / p.window * p.window : max(0, it.seq_len - p.window)) : 0;
   it.first = min(p.keep_first, it.lo);
   it.n_first = (it.first + kTcChunk - 1) / kTcChunk;
   it.c_window = max(it.lo / kTcChunk, it.n_first);
@@ -351,19 +356,23 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
             s_lo[k] = score(s_lo[k]) + (PLAIN ? 0.f : bias[k]);
             s_hi[k] = score(s_hi[k]) + (PLAIN ? 0.f : bias[2 + k]);
           }
-          float mx = -INFINITY;
-          if (v0) mx = fmaxf(mx, s_lo[0]);
-          if (v1) mx = fmaxf(mx, s_lo[1]);
-          if (v2) mx = fmaxf(mx, s_hi[0]);
-          if (v3) mx = fmaxf(mx, s_hi[1]);
-          mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-          mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+          const bool plain_sum = !PLAIN && p.sigmoid;
+          float mx = plain_sum ? 0.f : -INFINITY;
+          if (!plain_sum) {
+            if (v0) mx = fmaxf(mx, s_lo[0]);
+            if (v1) mx = fmaxf(mx, s_lo[1]);
+            if (v2) mx = fmaxf(mx, s_hi[0]);
+            if (v3) mx = fmaxf(mx, s_hi[1]);
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+          }
           const float m_new = fmaxf(m, mx);
           const float alpha = exp2f(m - m_new);  // m = -inf -> 0
-          const float p0 = v0 ? exp2f(s_lo[0] - m_new) : 0.f;
-          const float p1 = v1 ? exp2f(s_lo[1] - m_new) : 0.f;
-          const float p2 = v2 ? exp2f(s_hi[0] - m_new) : 0.f;
-          const float p3 = v3 ? exp2f(s_hi[1] - m_new) : 0.f;
+          auto weight = [&](float x) { return plain_sum ? __fdividef(1.f, 1.f + exp2f(fminf(-x, 120.f))) : exp2f(x - m_new); };
+          const float p0 = v0 ? weight(s_lo[0]) : 0.f;
+          const float p1 = v1 ? weight(s_lo[1]) : 0.f;
+          const float p2 = v2 ? weight(s_hi[0]) : 0.f;
+          const float p3 = v3 ? weight(s_hi[1]) : 0.f;
           l = l * alpha + (p0 + p1 + p2 + p3);
           m = m_new;
           const uint32_t pa0 = pk2<T>(p0, p1), pa2 = pk2<T>(p2, p3);
@@ -426,6 +435,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
           }
         }
         if (with_sink) L += exp2f(sink - M);
+        if (!PLAIN && p.sigmoid) L = 1.f;
         float val = L > 0.f ? O / L : 0.f;
         if (p.num_splits == 1) {
           if (!PLAIN && p.gate != nullptr) val *= head_gate(reinterpret_cast<const T*>(p.gate) + it.b * p.gate_stride + head);
@@ -457,7 +467,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
 template <typename T>
 __global__ void attn_merge_tc_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
                                      T* __restrict__ out, int64_t out_stride, int q_heads, int hd, int num_splits,
-                                     const T* __restrict__ sink, const T* __restrict__ gate, int64_t gate_stride) {
+                                     const T* __restrict__ sink, const T* __restrict__ gate, int64_t gate_stride, int sum_only) {
   const int b = blockIdx.x, head = blockIdx.y;
   const int64_t base = (static_cast<int64_t>(b) * q_heads + head) * num_splits;
   float M = -INFINITY;
@@ -475,6 +485,7 @@ __global__ void attn_merge_tc_kernel(const float* __restrict__ part_o, const flo
       }
       if (sink) wsum += exp2f(snk - M);
     }
+    if (sum_only) wsum = 1.f;  // (every split's reference is zero: the weights are ones)
     const float val = wsum > 0.f ? acc / wsum * g : 0.f;
     T* op = out + static_cast<int64_t>(b) * out_stride + static_cast<int64_t>(head) * hd;
     if (std::is_same<T, __nv_bfloat16>::value)
@@ -499,7 +510,7 @@ static int launch_tc(const CUtensorMap (&tm)[4], const DecodeTcParams& p, int ba
 
 template <typename T>
 static int launch_tc(const CUtensorMap (&tm)[4], const DecodeTcParams& p, int batch, cudaStream_t stream) {
-  const bool plain = p.dim == p.vdim && (p.dim == 64 || p.dim == 128) && p.v_rows > 0 && p.gate == nullptr && p.bias == nullptr && p.kv_div == 1;
+  const bool plain = p.dim == p.vdim && (p.dim == 64 || p.dim == 128) && p.v_rows > 0 && p.gate == nullptr && p.bias == nullptr && p.kv_div == 1 && !p.sigmoid;
   if (plain) return p.dim == 64 ? launch_tc<T, 64, 64, true>(tm, p, batch, stream) : launch_tc<T, 128, 128, true>(tm, p, batch, stream);
   if (p.dim > 64)
     return p.vdim > 64 ? launch_tc<T, 128, 128, false>(tm, p, batch, stream) : launch_tc<T, 128, 64, false>(tm, p, batch, stream);
@@ -535,10 +546,11 @@ int64_t blitz_attn_decode_workspace_bytes(int batch, int q_heads, int head_dim, 
 int blitz_attn_decode(const void* q, int64_t q_stride, const void* k_pool, const void* v_pool, const int32_t* indices,
                       const int32_t* indptr, const int32_t* last_page_len, void* out, int64_t out_stride,
                       void* workspace, int batch, int q_heads, int kv_heads, int dim, int vdim, int page_size, int page_rows,
-                      int max_pages, int num_splits, float sm_scale, int window, int keep_first, float softcap,
+                      int max_pages, int num_splits, float sm_scale, int window, int keep_first, int chunked, int sigmoid, float softcap,
                       const void* sink, const void* bias, int bias_len, const void* gate, int64_t gate_stride, int* status, int dtype, cudaStream_t stream) {
   if (batch <= 0) return 0;
   if (window < 0 || keep_first < 0 || softcap < 0.f || (bias != nullptr && bias_len < 1)) return -1;
+  if ((chunked && (window < 1 || keep_first)) || (sigmoid && (sink || softcap > 0.f))) return -1;
   if (num_splits < 1 || kv_heads < 1 || (q_heads % kv_heads) != 0 || (q_stride & 1)) return -1;
   if (dim < 8 || dim > 128 || (dim & 7) || vdim < 8 || vdim > 128 || (vdim & 7)) return -1;
   if (page_size < 8 || (page_size & (page_size - 1)) != 0 || page_rows < page_size) return -1;
@@ -569,6 +581,7 @@ int blitz_attn_decode(const void* q, int64_t q_stride, const void* k_pool, const
   p.page_size = page_size; p.max_pages = max_pages; p.dim = dim; p.vdim = vdim; p.page_rows = page_rows; p.v_rows = one ? page_size : 0;
   p.num_splits = num_splits; p.box_tokens = bt; p.tail_box_tokens = bt_tail;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = g_tc_trace;
+  p.chunked = chunked; p.sigmoid = sigmoid;
   p.window = window; p.keep_first = keep_first; p.sink = sink; p.bias = bias; p.bias_len = bias_len; p.gate = gate; p.gate_stride = gate_stride;
   p.cap_scale = softcap > 0.f ? sm_scale / softcap : 0.f; p.cap_log2 = softcap * 1.4426950408889634f;
   int rc = dtype == 1 ? launch_tc<__nv_bfloat16>(tm, p, batch, stream) : launch_tc<__half>(tm, p, batch, stream);
@@ -577,7 +590,7 @@ int blitz_attn_decode(const void* q, int64_t q_stride, const void* k_pool, const
     auto merge = [&](auto type) {
       using T = decltype(type);
       attn_merge_tc_kernel<T><<<dim3(batch, q_heads), vdim > 64 ? 128 : 64, 0, stream>>>(
-          p.part_o, p.part_lse, (T*)out, out_stride, q_heads, vdim, num_splits, (const T*)sink, (const T*)gate, gate_stride);
+          p.part_o, p.part_lse, (T*)out, out_stride, q_heads, vdim, num_splits, (const T*)sink, (const T*)gate, gate_stride, sigmoid);
     };
     if (dtype == 1) merge(__nv_bfloat16{});
     else merge(__half{});
@@ -682,6 +695,7 @@ extern "C" int blitz_attn_decode_noalloc(const void* q, int64_t q_stride, const 
   p.max_pages = max_pages; p.num_splits = num_splits; p.box_tokens = bt; p.tail_box_tokens = bt_tail;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = nullptr;
   p.kv_div = 1; p.dim = p.vdim = head_dim; p.page_rows = 2 * page_size; p.v_rows = page_size; p.gate = nullptr; p.gate_stride = 0;
+  p.chunked = p.sigmoid = 0;
   p.window = 0; p.keep_first = 0; p.sink = nullptr; p.bias = nullptr; p.bias_len = 0; p.cap_scale = p.cap_log2 = 0.f;
   int sms = 0;
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
@@ -697,9 +711,9 @@ extern "C" int blitz_attn_decode_noalloc(const void* q, int64_t q_stride, const 
   dim3 grid(batch, q_heads);
   if (dtype == 1)
     attn_merge_tc_kernel<__nv_bfloat16><<<grid, head_dim, 0, stream>>>(p.part_o, p.part_lse, (__nv_bfloat16*)out, out_stride,
-                                                                       q_heads, head_dim, num_splits, nullptr, nullptr, 0);
+                                                                       q_heads, head_dim, num_splits, nullptr, nullptr, 0, 0);
   else
     attn_merge_tc_kernel<__half><<<grid, head_dim, 0, stream>>>(p.part_o, p.part_lse, (__half*)out, out_stride, q_heads,
-                                                                head_dim, num_splits, nullptr, nullptr, 0);
+                                                                head_dim, num_splits, nullptr, nullptr, 0, 0);
   return (int)cudaGetLastError();
 }

@@ -26,6 +26,9 @@
 // share begins and ends anywhere in a sequence; it leaves at most two incomplete pieces (fp32 partial sums), which a second
 // kernel merges.
 //
+// A sliding window leaves the blocks before it out (a sequence's blocks are counted from its first visible key's on); a sink is one
+// more term of the row sum, added where a row's sum is complete.
+//
 // The tokens of prompts go through the same kernel, each as a row of its own that sees the keys up to its position (for models
 // whose expanded heads the prompt kernel does not take).
 #include "launch.cuh"
@@ -49,6 +52,8 @@ struct LatentParams {
   int rows, first_token;            // (else null: a row per sequence)
   void* out;                    // [batch][out_stride], head h's rank columns from h * rank on
   const void* gate;             // [batch][gate_stride], or null
+  const void* sink;             // [heads] in the activation type, or null
+  int window;                   // a row sees the last `window` positions (0: all)
   int64_t out_stride, gate_stride;
   float *part_o, *part_lse;     // [grid][2][group][rank], [grid][2][group]
   int* blocks_before;           // [batch + 1], for the merge
@@ -192,6 +197,8 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   }
   // the work list; with a page table that no running kernel writes, while the previous kernel still runs
   if (!p.static_table) ptx::griddep_wait();
+  auto first_key = [&](int len) { return p.window > 0 ? max(0, len - p.window) : 0; };
+  auto first_block = [&](int len) { return first_key(len) / KT; };
   const int chunks32 = (p.batch + 31) / 32;
   for (int i = warp; i < chunks32; i += kWarps) {  // sums over 32 sequences
     const int b = i * 32 + lane;
@@ -203,7 +210,7 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       if (npages > 0) len = p.pos ? min(p.pos[b] + 1, npages << p.page_shift) : ((npages - 1) << p.page_shift) + p.last_page_len[b];
       s_page[b] = first;
       s_len[b] = len;
-      v = (len + KT - 1) / KT;
+      v = (len + KT - 1) / KT - first_block(len);
     }
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
@@ -255,7 +262,7 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       return __shfl_sync(0xffffffffu, ok, 0) != 0;
     };
     auto box_row = [&](const LaPiece& q, int blk) {  // this lane's first row of a block in the pool
-      const int tok = blk * KT + lane * bt, slot = tok >> p.page_shift;
+      const int tok = (first_block(s_len[q.b]) + blk) * KT + lane * bt, slot = tok >> p.page_shift;
       if (!mine || tok >= s_len[q.b]) return p.oob_row;  // past the pool: the box arrives as zeros
       int page = p.indices[s_page[q.b] + slot];
       if (page < 0 || page >= p.max_pages) {
@@ -424,6 +431,7 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     };
     for (; walk.next(q); ++n) {
       const int len = s_len[q.b], head0 = q.sub * p.group;
+      const int key0 = first_block(len) * KT, lo = first_key(len) - key0;  // position of block 0's first key; first visible key there
       // of the thread's keys, per head: row sum, and the references (the same in all threads; for many heads in shared memory)
       constexpr bool kRefRegs = NH <= 32;
       float l[NH], ref[kRefRegs ? NH : 1] = {};
@@ -446,12 +454,12 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
 #pragma unroll
             for (int k = 0; k < 16; ++k) x[i + k] = fmaf(__uint_as_float(v[k]), p.scale_log2, first ? 0.f : -reference(i + k));
           }
-          if (blk * KT + KT > len && blk * KT + r >= len) {
+          if ((key0 + blk * KT + KT > len && key0 + blk * KT + r >= len) || blk * KT + r < lo) {
 #pragma unroll
             for (int h = 0; h < NH; ++h) x[h] = -INFINITY;
           }
-          if (first) {  // the first key's scores are the references
-            if (r == 0) {
+          if (first) {  // the first visible key's scores are the references
+            if (r == (blk == 0 ? lo : 0)) {
 #pragma unroll
               for (int h = 0; h < NH; ++h) s_ref[h] = x[h];
             }
@@ -549,6 +557,8 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         float sum = 0.f;
 #pragma unroll
         for (int w = 0; w < kSoft; ++w) sum += s_red[w * NH + r];
+        if (whole && p.sink != nullptr)
+          sum += exp2f(fminf(to_f<T>(reinterpret_cast<const T*>(p.sink)[head0 + r]) * 1.4426950408889634f - s_ref[r], 120.f));
         float f = sum > 0.f ? 1.f / sum : 0.f;
         if (whole && p.gate != nullptr) f *= sigmoid_f(to_f<T>(reinterpret_cast<const T*>(p.gate)[q.b * p.gate_stride + head0 + r]));
         s_fac[r] = f;
@@ -616,12 +626,14 @@ __global__ void __launch_bounds__(256) attn_latent_merge_kernel(const LatentPara
     m = fmaxf(m, w[i]);
   }
   m = warp_max(m);
+  const float sink = p.sink ? to_f<T>(reinterpret_cast<const T*>(p.sink)[head]) * 1.4426950408889634f : -INFINITY;
+  m = fmaxf(m, sink);
 #pragma unroll
   for (int i = 0; i < kRounds; ++i) {
     w[i] = exp2f(w[i] - m);
     sum += w[i];
   }
-  sum = warp_sum(sum);
+  sum = warp_sum(sum) + exp2f(sink - m);
   const float gate = p.gate ? sigmoid_f(to_f<T>(reinterpret_cast<const T*>(p.gate)[b * p.gate_stride + head])) : 1.f;
   float acc[kLaMaxRank / 32] = {};
 #pragma unroll
@@ -711,17 +723,17 @@ int64_t blitz_attn_latent_workspace_bytes(int heads, int rank) {
 
 // q [batch][q_stride]: heads of `width` columns; pool [max_pages][page_size][width], the first `rank` columns are the values;
 // out [batch][out_stride]: heads of `rank` columns.  width, rank: multiples of 8, rank up to 512; page_size: a power of two >= 8;
-// gate [batch][gate_stride] or null.  A row without pages gives zeros.  kt_hint: keys per block, 0 = choose, else 64 or 128.
+// gate [batch][gate_stride] or null; window (0 = none) and sink ([heads] or null): see the top of the file.  A row without pages gives zeros.  kt_hint: keys per block, 0 = choose, else 64 or 128.
 // static_table: no kernel still running in the stream writes indices, indptr, last_page_len, pos or tok_indptr.
 // pos [batch], tok_indptr [rows + 1] (both or none): the batch are tokens first_token .. of `rows` sequences, whose pages indptr
 // [rows + 1] names; each sees the keys up to its position.  last_page_len is not read then.
 int blitz_attn_latent(const void* q, int64_t q_stride, const void* pool, const int32_t* indices, const int32_t* indptr,
                       const int32_t* last_page_len, const int32_t* pos, const int32_t* tok_indptr, int rows, int first_token, void* out, int64_t out_stride, void* workspace, int batch, int heads, int width, int rank,
-                      int page_size, int max_pages, float sm_scale, const void* gate, int64_t gate_stride, int kt_hint, int static_table, int* status, int dtype,
+                      int page_size, int max_pages, float sm_scale, int window, const void* sink, const void* gate, int64_t gate_stride, int kt_hint, int static_table, int* status, int dtype,
                       cudaStream_t stream) {
   if (batch <= 0) return 0;
   LatentPlan pl;
-  if (!latent_plan(batch, heads, width, rank, page_size, kt_hint, &pl) || workspace == nullptr || max_pages < 1) return -1;
+  if (!latent_plan(batch, heads, width, rank, page_size, kt_hint, &pl) || workspace == nullptr || max_pages < 1 || window < 0) return -1;
   if ((pos == nullptr) != (tok_indptr == nullptr) || (pos && rows < 1)) return -1;
   if ((q_stride & 7) || (reinterpret_cast<uintptr_t>(workspace) & 15)) return -1;
   const int sms = device_sm_count() < kLaMaxCtas ? device_sm_count() : kLaMaxCtas;
@@ -733,6 +745,7 @@ int blitz_attn_latent(const void* q, int64_t q_stride, const void* pool, const i
   if (!get_tmap_2d(&tk, pool, (uint64_t)width, (uint64_t)max_pages * page_size, (uint64_t)width * 2, 64, (uint32_t)bt)) return -2;
   LatentParams p;
   p.indices = indices; p.indptr = indptr; p.last_page_len = last_page_len;
+  p.window = window; p.sink = sink;
   p.pos = pos; p.tok_indptr = tok_indptr; p.rows = rows; p.first_token = first_token; p.out = out; p.gate = gate;
   p.out_stride = out_stride; p.gate_stride = gate_stride;
   p.batch = batch; p.heads = heads; p.group = pl.group; p.subs = heads / pl.group; p.rank = rank;

@@ -45,6 +45,10 @@
 // requested before it waits for the scores) into shared memory, where the lanes of a warp, rows that follow one another, read
 // neighbouring words.  Blocks whose every distance is beyond the table share its last entry, which moves the reference.
 //
+// The window may be a chunk counted from position 0 (`chunked`): a row sees the keys of its own chunk.  Weights may be sigmoids of
+// the scores (template parameter SIG; EXT with it): no maximum, no row sum, no rescaling.  sigmoid(x) = 1 / (1 + e^-x); two
+// neighbours share a reciprocal, 1 / a = b / (a b), with e^-x held below 2^60 (a weight below that is zero next to any other).
+//
 // Replaces FlashInfer's BatchPrefillWithRaggedKVCacheWrapper / paged wrapper calls and their host Plan()
 // (src/kernel/attention_prefill.cu:11-45, src/kernel/flashinfer_types.cu:24-49).
 #include "launch.cuh"
@@ -68,12 +72,13 @@ struct PagedPrefillParams {
   const int32_t* work;          // [entries][kPpWorkInts], heaviest first
   int entries, q_heads, kv_heads, vdim, page_size, page_rows, box_tokens, oob_row;  // page n's token `off`: pool row n * page_rows + off
   float scale_log2;
+  int chunked;                // EXT: the window is a chunk
   int window, keep_first;     // EXT: a row sees the last `window` positions (0: all) and the first `keep_first`
   float cap_scale, cap_log2;  // EXT: soft cap (cap_log2 > 0): score in log2 units = cap_log2 * tanh(q.k * cap_scale)
   float small_max;            // EXT: largest |q.k| the polynomial takes (0: never)
   float poly[4];              // EXT: score in log2 units = x (poly[0] + poly[1] x^2 + poly[2] x^4 + poly[3] x^6), x = q.k
   const void* sink;           // EXT: [q_heads] in the activation type, or null
-  const void* bias;           // BIAS: [q_heads][bias_len] in the activation type
+  const void* bias;           // BIAS: [q_heads][bias_len] in the activation type (SIG: [q_heads], or null)
   int bias_len;
   int* status;
   long long* trace;  // profiling aid (null in production): clock stamps of CTA 0's first item, see the set_trace call
@@ -122,7 +127,7 @@ __device__ __forceinline__ PpItem pp_item(const PagedPrefillParams& p, int idx) 
   }
   it.n_first = it.b_window = 0;
   if (EXT && p.window > 0) {
-    const int lo = max(0, it.prefix + it.q0 - p.window + 1);  // first key in the window of the item's first row
+    const int p0 = it.prefix + it.q0, lo = p.chunked ? p0 - p0 % p.window : max(0, p0 - p.window + 1);  // first key in the window of the item's first row
     it.n_first = (min(p.keep_first, lo) + kPpTile - 1) / kPpTile;
     it.b_window = max(lo / kPpTile, it.n_first);
 #pragma unroll
@@ -139,7 +144,7 @@ __device__ __forceinline__ int pp_index(int r, int total) {
   return idx < total ? idx : -1;
 }
 
-template <typename T, int HD, int VD, bool POLY, bool EXT, bool BIAS>
+template <typename T, int HD, int VD, bool POLY, bool EXT, bool BIAS, bool SIG>
 __global__ void __launch_bounds__(kPpThreads, 1)
 attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                           const __grid_constant__ CUtensorMap tmap_v, const PagedPrefillParams p) {
@@ -364,7 +369,9 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       first = false;
       const int q_idx = it.q0 + t * kPpTile + r_;  // row within the chunk
       const int limit = it.prefix + q_idx;         // last key position this row may see
+      const int chunk_from = EXT && p.chunked ? limit - limit % p.window : -1;  // first key of the row's chunk
       float m_ref = 0.f, l = 0.f;
+      const float sig_bias = SIG && p.bias ? -1.4426950408889634f * to_f<T>(reinterpret_cast<const T*>(p.bias)[it.head]) : 0.f;
       const T* bias_row = BIAS ? reinterpret_cast<const T*>(p.bias) + static_cast<int64_t>(it.head) * p.bias_len : nullptr;
       const float far_bias = BIAS ? to_f<T>(bias_row[p.bias_len - 1]) * 1.4426950408889634f : 0.f;
       for (int j = 0; j < my_blocks; ++j) {
@@ -397,11 +404,37 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         // does the block hold a key that some row of the tile may not see?
         bool masked = kv0 + kPpTile - 1 > row0;
         if (EXT && p.window > 0)
-          masked = masked || (kv0 <= row0 + kPpTile - 1 - p.window && kv0 + kPpTile > p.keep_first);
-        const int from = (EXT && p.window > 0) ? limit - p.window + 1 : 0;
+          masked = masked || (p.chunked ? kv0 < (row0 + kPpTile - 1) / p.window * p.window
+                                        : kv0 <= row0 + kPpTile - 1 - p.window && kv0 + kPpTile > p.keep_first);
+        const int from = (EXT && p.window > 0) ? chunk_from >= 0 ? chunk_from : limit - p.window + 1 : 0;
         auto visible = [&](int i) {  // key i of the block to this row
           return kv0 + i <= limit && (!EXT || kv0 + i >= from || kv0 + i < p.keep_first);
         };
+        if constexpr (SIG) {
+          const float neg_scale = -p.scale_log2;
+          auto weights = [&](auto&& hidden) {
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+              uint32_t pk[32];
+#pragma unroll
+              for (int i = 0; i < 32; ++i) {
+                const int c = h * 64 + 2 * i;
+                const float a = 1.f + ptx::ex2_approx(fminf(fmaf(__uint_as_float(score(c)), neg_scale, sig_bias), 60.f));
+                const float b = 1.f + ptx::ex2_approx(fminf(fmaf(__uint_as_float(score(c + 1)), neg_scale, sig_bias), 60.f));
+                const float r = __fdividef(1.f, a * b);
+                pk[i] = pk2<T>(hidden(c) ? 0.f : b * r, hidden(c + 1) ? 0.f : a * r);
+              }
+              ptx::tmem_st_32x32(tS + h * 32, pk);
+            }
+          };
+          if (masked) weights([&](int i) { return !visible(i); });
+          else weights([](int) { return false; });
+          ptx::tmem_st_wait();
+          ptx::tc_fence_before_sync();
+          ptx::mbar_arrive(&p_ready[t]);
+          l = 1.f;
+          continue;
+        }
         const bool capped = EXT && p.cap_log2 > 0.f;
         float bias = 0.f;  // of every score of the block, in log2 units
         if (near) {
@@ -574,15 +607,15 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   }
 }
 
-template <typename T, int HD, int VD, bool POLY, bool EXT, bool BIAS>
+template <typename T, int HD, int VD, bool POLY, bool EXT, bool BIAS, bool SIG>
 static int launch_paged_prefill(const CUtensorMap (&tm)[3], const PagedPrefillParams& p, int grid, cudaStream_t stream) {
   constexpr int kSmem = PpCfg<HD, VD>::kSmemBytes + (BIAS ? PpCfg<HD, VD>::kBiasFloats * 4 : 0);
   static PerDeviceOnce once;
   cudaError_t e = once.run([] {
-    return cudaFuncSetAttribute(attn_prefill_paged_kernel<T, HD, VD, POLY, EXT, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
+    return cudaFuncSetAttribute(attn_prefill_paged_kernel<T, HD, VD, POLY, EXT, BIAS, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
   });
   if (e != cudaSuccess) return (int)e;
-  attn_prefill_paged_kernel<T, HD, VD, POLY, EXT, BIAS><<<grid, kPpThreads, kSmem, stream>>>(tm[0], tm[1], tm[2], p);
+  attn_prefill_paged_kernel<T, HD, VD, POLY, EXT, BIAS, SIG><<<grid, kPpThreads, kSmem, stream>>>(tm[0], tm[1], tm[2], p);
   return (int)cudaGetLastError();
 }
 
@@ -606,17 +639,18 @@ void blitz_attn_prefill_paged_set_trace(long long* buf) { blitz::g_pp_trace = bu
 // index of its first page id, number of its pages, tokens cached for it (chunk included), which 256-row pair, 0, 0.
 // page_size: a power of two >= 8.  dim and vdim: multiples of 8 up to 128.  flags bit 0: compute a quarter of the
 // exponentials on the FMA pipe (not with a window, cap or sink).  window (0 = none) / keep_first, softcap (0 = none), sink
-// and gate (null = none): see the top of the file.  bias: [q_heads][bias_len] in the activation type, or null (not with a
-// window, cap or sink).
+// and gate (null = none), chunked and sigmoid: see the top of the file.  bias: [q_heads][bias_len] in the activation type, or null
+// (not with a window, cap or sink; with sigmoid weights only bias_len 1).
 int blitz_attn_prefill_paged(const void* q, int64_t q_stride, const void* k_pool, const void* v_pool, void* out, int64_t out_stride,
                              const int32_t* page_indices, const int32_t* work, int entries, int num_tokens,
                              int q_heads, int kv_heads, int dim, int vdim, int page_size, int page_rows, int max_pages,
-                             float sm_scale, int flags, int window, int keep_first, float softcap, const void* sink,
+                             float sm_scale, int flags, int window, int keep_first, int chunked, int sigmoid, float softcap, const void* sink,
                              const void* bias, int bias_len, const void* gate, int64_t gate_stride, int* status, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0 || entries <= 0) return 0;
   if (dim < 8 || dim > 128 || (dim & 7) || vdim < 8 || vdim > 128 || (vdim & 7)) return -1;
   if (kv_heads < 1 || (q_heads % kv_heads) != 0 || (out_stride & 7) || (q_stride & 7)) return -1;
   if (window < 0 || keep_first < 0 || softcap < 0.f) return -1;
+  if ((chunked && (window < 1 || keep_first)) || (sigmoid && (sink || softcap > 0.f || (bias && bias_len != 1)))) return -1;
   if (page_size < 8 || (page_size & (page_size - 1)) != 0 || page_rows < page_size || work == nullptr) return -1;
   if ((reinterpret_cast<uintptr_t>(work) & 15) != 0 || (reinterpret_cast<uintptr_t>(out) & 15) != 0) return -1;
   const int bt = page_size < 64 ? page_size : 64;
@@ -635,6 +669,7 @@ int blitz_attn_prefill_paged(const void* q, int64_t q_stride, const void* k_pool
   p.q_heads = q_heads; p.kv_heads = kv_heads; p.page_size = page_size; p.box_tokens = bt;
   p.oob_row = (int)rows;
   p.scale_log2 = sm_scale * 1.4426950408889634f; p.status = status; p.trace = g_pp_trace;
+  p.chunked = chunked;
   p.window = window; p.keep_first = keep_first; p.sink = sink; p.bias = bias; p.bias_len = bias_len;
   p.cap_scale = softcap > 0.f ? sm_scale / softcap : 0.f; p.cap_log2 = softcap * 1.4426950408889634f;
   // tanh(z) = z (k0 + k1 z^2 + k2 z^4 + k3 z^6) for |z| <= 0.5 (Chebyshev interpolation of tanh(z) / z in z^2, absolute
@@ -648,21 +683,24 @@ int blitz_attn_prefill_paged(const void* q, int64_t q_stride, const void* k_pool
   const int sms = device_sm_count();
   const int grid = (int)(total < sms ? total : sms);
   const bool poly = (flags & 1) != 0, ext = window > 0 || softcap > 0.f || sink != nullptr;
-  if (bias != nullptr && (ext || bias_len < 1)) return -1;
-  auto sized = [&](auto type, auto poly_, auto ext_, auto bias_) {
+  if (bias != nullptr && !sigmoid && (ext || bias_len < 1)) return -1;
+  auto sized = [&](auto type, auto poly_, auto ext_, auto bias_, auto sig_) {
     using T = decltype(type);
-    constexpr bool P = decltype(poly_)::value, X = decltype(ext_)::value, B = decltype(bias_)::value;
+    constexpr bool P = decltype(poly_)::value, X = decltype(ext_)::value, B = decltype(bias_)::value, G = decltype(sig_)::value;
     if (dim > 64)
-      return vdim > 64 ? launch_paged_prefill<T, 128, 128, P, X, B>(tm, p, grid, stream)
-                       : launch_paged_prefill<T, 128, 64, P, X, B>(tm, p, grid, stream);
-    return vdim > 64 ? launch_paged_prefill<T, 64, 128, P, X, B>(tm, p, grid, stream)
-                     : launch_paged_prefill<T, 64, 64, P, X, B>(tm, p, grid, stream);
+      return vdim > 64 ? launch_paged_prefill<T, 128, 128, P, X, B, G>(tm, p, grid, stream)
+                       : launch_paged_prefill<T, 128, 64, P, X, B, G>(tm, p, grid, stream);
+    return vdim > 64 ? launch_paged_prefill<T, 64, 128, P, X, B, G>(tm, p, grid, stream)
+                     : launch_paged_prefill<T, 64, 64, P, X, B, G>(tm, p, grid, stream);
   };
   auto launch = [&](auto type) {
-    if (bias != nullptr) return sized(type, std::false_type{}, std::false_type{}, std::true_type{});
-    if (ext) return sized(type, std::false_type{}, std::true_type{}, std::false_type{});
-    if (poly) return sized(type, std::true_type{}, std::false_type{}, std::false_type{});
-    return sized(type, std::false_type{}, std::false_type{}, std::false_type{});
+    const std::false_type no{};
+    const std::true_type yes{};
+    if (sigmoid) return sized(type, no, yes, no, yes);
+    if (bias != nullptr) return sized(type, no, no, yes, no);
+    if (ext) return sized(type, no, yes, no, no);
+    if (poly) return sized(type, yes, no, no, no);
+    return sized(type, no, no, no, no);
   };
   return dtype == 1 ? launch(__nv_bfloat16{}) : launch(__half{});
 }

@@ -7,6 +7,9 @@
 //   out           = sum_j e^score_j v_j / (e^sink + sum_j e^score_j)        no sink: the plain softmax
 //   out           = sigmoid(gate) * out                                     no gate: as it is
 //
+// `chunked`: the window is a chunk, visible(i, j) = j <= i and floor(i / window) = floor(j / window).  `sigmoid`: no softmax,
+// out = sum_j sigmoid(score_j) v_j.
+//
 // Keys and values may differ in size, and values may be the first columns of the keys' rows (v_row: their pitch).
 // It serves the 32-bit mode and head sizes that the tensor-core kernels do not take.  A warp owns one (token, query
 // head): keys go over the lanes 32 at a time for the scores, head dimensions go over the lanes for the weighted sum.
@@ -34,7 +37,7 @@ struct RaggedAttnParams {
   const void* sink;
   const void* bias;   // [q_heads][bias_len] by distance, the last entry for all longer ones; or null
   int bias_len, v_row;
-  int num_tokens, rows, q_heads, kv_heads, dim, vdim, page_size, page_rows, max_pages, window, keep_first;
+  int num_tokens, rows, q_heads, kv_heads, dim, vdim, page_size, page_rows, max_pages, window, keep_first, chunked, sigmoid;
   float scale, softcap;
   int* status;
 };
@@ -83,7 +86,7 @@ __global__ void __launch_bounds__(kRgWarps * 32) attn_ragged_kernel(const Ragged
     m = ldf<T>(reinterpret_cast<const T*>(p.sink) + h);
     l = 1.f;
   }
-  const int lo = p.window > 0 ? max(0, i - p.window + 1) : 0;  // first key of the window
+  const int lo = p.window > 0 ? (p.chunked ? i - i % p.window : max(0, i - p.window + 1)) : 0;  // first key of the window
   const int first = min(p.keep_first, lo);                     // kept keys in front of it
   const int nkeys = first + (i - lo + 1);                      // kept keys, then the window's
   for (int base = 0; base < nkeys; base += 32) {
@@ -97,14 +100,20 @@ __global__ void __launch_bounds__(kRgWarps * 32) attn_ragged_kernel(const Ragged
       if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
       if (bias) s += ldf<T>(bias + min(i - (n < first ? n : lo + n - first), p.bias_len - 1));
     }
-    const float mx = fmaxf(m, warp_max(s));
-    if (mx == -INFINITY) continue;
-    const float corr = expf(m - mx);
-    const float w = expf(s - mx);
-    l = l * corr + warp_sum(w);
-    m = mx;
+    float w;
+    if (p.sigmoid) {
+      w = row >= 0 ? sigmoid_f(s) : 0.f;
+      l = 1.f;
+    } else {
+      const float mx = fmaxf(m, warp_max(s));
+      if (mx == -INFINITY) continue;
+      const float corr = expf(m - mx);
+      w = expf(s - mx);
+      l = l * corr + warp_sum(w);
+      m = mx;
 #pragma unroll
-    for (int d = 0; d < kRgMaxDim / 32; ++d) acc[d] *= corr;
+      for (int d = 0; d < kRgMaxDim / 32; ++d) acc[d] *= corr;
+    }
     const int cnt = min(32, nkeys - base);
     for (int k = 0; k < cnt; ++k) {
       const float wk = __shfl_sync(0xffffffffu, w, k);
@@ -142,13 +151,13 @@ int blitz_attn_ragged(const void* q, int64_t q_stride, const void* k_pool, const
                       const int32_t* pos, const int32_t* tok_indptr, const int32_t* page_indptr,
                       const int32_t* page_indices, const void* sink, const void* bias, int bias_len, int v_row, const void* gate, int64_t gate_stride, int num_tokens,
                       int rows, int q_heads, int kv_heads, int dim, int vdim, int page_size, int page_rows, int max_pages,
-                      int window, int keep_first, float scale, float softcap, int* status, int dtype, cudaStream_t stream) {
+                      int window, int keep_first, int chunked, int sigmoid, float scale, float softcap, int* status, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0 || rows <= 0) return 0;
   if (dim <= 0 || vdim <= 0 || vdim > kRgMaxDim || dim > kRgMaxQueryDim || kv_heads <= 0 || q_heads % kv_heads != 0 || window < 0 ||
-      keep_first < 0 || v_row < vdim || (bias && bias_len < 1))
+      keep_first < 0 || v_row < vdim || (chunked && (window < 1 || keep_first)) || (sigmoid && sink) || (bias && bias_len < 1))
     return -1;
   RaggedAttnParams p{q, k_pool, v_pool, gate, out, q_stride, out_stride, gate_stride, pos, tok_indptr, page_indptr, page_indices,
-                     sink, bias, bias_len, v_row, num_tokens, rows, q_heads, kv_heads, dim, vdim, page_size, page_rows, max_pages, window, keep_first,
+                     sink, bias, bias_len, v_row, num_tokens, rows, q_heads, kv_heads, dim, vdim, page_size, page_rows, max_pages, window, keep_first, chunked, sigmoid,
                      scale, softcap, status};
   const int64_t items = static_cast<int64_t>(num_tokens) * q_heads;
   const dim3 grid((unsigned)((items + kRgWarps - 1) / kRgWarps));

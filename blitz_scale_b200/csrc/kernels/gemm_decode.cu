@@ -31,6 +31,7 @@
 #include "launch.cuh"
 #include "ptx.cuh"
 #include "tmap.cuh"
+#include "gemm_gate.cuh"
 #include <cstdlib>
 #include <type_traits>
 
@@ -55,7 +56,8 @@ struct DecGemmParams {
   int kb_per_split;  // K blocks per CTA of a cluster
   int slice;         // tokens each cluster rank reduces and stores (multiple of 32: TMEM is read 32 columns at a time)
   int static_w;      // weights do not depend on earlier kernels of the stream
-  float alpha;       // axpy; soft cap
+  float alpha;       // axpy; soft cap; limit of the clamped unit
+  float beta;        // clamped unit (R: its biases)
   int smem_bytes;    // dynamic shared memory of this launch (227 KB, or about half of it for two CTAs per SM)
   int* status;
 };
@@ -107,7 +109,7 @@ template <typename T, int EPI>
 __device__ __forceinline__ void dec_store32(const DecGemmParams& p, const float (&g)[32], const float (&u)[32], int n,
                                             int b0, int b_end) {
   if (n >= p.N) return;
-  if (EPI >= 4) {
+  if (epi_f32(EPI)) {
     float* cf = reinterpret_cast<float*>(p.C) + n;
     float old[32];
     const float inv = EPI == 6 ? 1.f / p.alpha : 0.f;
@@ -121,7 +123,11 @@ __device__ __forceinline__ void dec_store32(const DecGemmParams& p, const float 
     return;
   }
   T* c = reinterpret_cast<T*>(p.C) + n;
-  float res[32];
+  float res[32], bias_g = 0.f, bias_u = 0.f;
+  if (EPI == kEpiClampGlu) {
+    bias_g = ldf<T>(reinterpret_cast<const T*>(p.R) + n);
+    bias_u = ldf<T>(reinterpret_cast<const T*>(p.R) + p.up_col_off + n);
+  }
   if (EPI == 1) {
     // C may alias R (in-place residual update): read all residual values before the first store, otherwise
     // every load would have to wait for the store before it
@@ -135,6 +141,7 @@ __device__ __forceinline__ void dec_store32(const DecGemmParams& p, const float 
     if (b < b_end) {
       float v = g[i];
       if (EPI == 2) v = dec_silu(v) * u[i];
+      if (EPI == kEpiClampGlu) v = clamp_glu(v + bias_g, u[i] + bias_u, p.alpha, p.beta);
       if (EPI == 1) v += res[i];
       c[static_cast<int64_t>(b) * p.ldc] = dec_cvt<T>(v);
     }
@@ -146,7 +153,7 @@ __global__ void __launch_bounds__(kDecThreads, 1)
 gemm_decode_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
                    const DecGemmParams p) {
   using Cfg = DecCfg;
-  constexpr int kHalves = (EPI == 2) ? 2 : 1;
+  constexpr int kHalves = (epi_gated(EPI)) ? 2 : 1;
   constexpr int kWBytes = kHalves * kDecTile * kDecBK * 2;  // weight bytes per stage
   constexpr uint32_t kFmt = std::is_same<T, __nv_bfloat16>::value ? 1u : 0u;
   const int cols = kHalves * p.npad;  // TMEM columns per accumulator
@@ -207,7 +214,7 @@ gemm_decode_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_cons
         const int n0 = tile * kDecTile;
         ptx::tma_load_2d(sw, &tmap_w, &full_bar[stage], n0, kb * kDecBK);
         ptx::tma_load_2d(sw + 8192, &tmap_w, &full_bar[stage], n0 + 64, kb * kDecBK);
-        if (EPI == 2) {
+        if (epi_gated(EPI)) {
           ptx::tma_load_2d(sw + 16384, &tmap_w, &full_bar[stage], p.up_col_off + n0, kb * kDecBK);
           ptx::tma_load_2d(sw + 24576, &tmap_w, &full_bar[stage], p.up_col_off + n0 + 64, kb * kDecBK);
         }
@@ -295,7 +302,7 @@ gemm_decode_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_cons
             const uint64_t xdesc = ptx::make_smem_desc(x_base + k * 32, 16, 1024, ptx::kLayoutSw128);
             const uint32_t accum = (kb != kb_beg || k != 0) ? 1u : 0u;
             ptx::umma_f16_ss(d_tmem, wdesc, xdesc, idesc, accum);
-            if (EPI == 2) {
+            if (epi_gated(EPI)) {
               const uint64_t udesc = ptx::make_smem_desc(w_base + 16384 + k * 2048, 8192, 1024, ptx::kLayoutSw128);
               ptx::umma_f16_ss(d_tmem + static_cast<uint32_t>(p.npad), udesc, xdesc, idesc, accum);
             }
@@ -337,7 +344,7 @@ gemm_decode_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_cons
           uint32_t v[32];
           float g[32], up[32];
           ptx::tmem_ld_32x32(taddr + c, v);
-          if (EPI == 2) {
+          if (epi_gated(EPI)) {
             uint32_t t[32];
             ptx::tmem_ld_32x32(taddr + p.npad + c, t);
             ptx::tmem_ld_wait();
@@ -486,7 +493,7 @@ static cudaError_t launch_dec(const CUtensorMap& tx, const CUtensorMap& tw, DecG
     return cudaSuccess;
   });
   if (e0 != cudaSuccess) return e0;
-  const int halves = EPI == 2 ? 2 : 1;
+  const int halves = epi_gated(EPI) ? 2 : 1;
   const int stage_bytes = DecCfg::x_stage_bytes(p.npad) + halves * kDecTile * kDecBK * 2;
   // One CTA per SM.  BLITZ_DECODE_OCC=2 runs two CTAs per SM on half the shared memory each (so that one CTA's
   // set-up or reduction overlaps the other's weight stream); measured on B200 it changes nothing (15.2 vs 15.3 us
@@ -535,22 +542,23 @@ int blitz_get_pdl() { return blitz::pdl_flag(); }
 // Whether blitz_gemm_decode takes this problem (the general GEMM handles everything else).
 int blitz_gemm_decode_supported(int M, int N, int K, int b_layout, int epilogue) {
   return M >= 1 && M <= 256 && b_layout == 0 &&
-         ((epilogue >= 0 && epilogue <= 2) || (epilogue >= 4 && epilogue <= 6)) && (N & 7) == 0 && (K & 7) == 0;
+         ((epilogue >= 0 && epilogue <= 2) || (epilogue >= 4 && epilogue <= blitz::kEpiClampGlu)) && (N & 7) == 0 && (K & 7) == 0;
 }
 
 // C = X W (+R | silu-mul).  X [M, lda>=K], W [K, ldb>=columns] row-major, C/R [M, ldc>=N].  dtype 0 fp16, 1 bf16.
 // epilogue 0 store, 1 add R (C may be R), 2 silu(gate)*up with the up columns starting at up_col_off, 4 store with C in
-// fp32, 5 C += alpha * acc with C in fp32, 6 alpha * tanh(acc / alpha) with C in fp32.
+// fp32, 5 C += alpha * acc with C in fp32, 6 alpha * tanh(acc / alpha) with C in fp32, 7 clamped gated unit (gemm_gate.cuh; R:
+// its biases, alpha: its limit).
 // static_w != 0 promises that W was not written by kernels still running in this stream (weights), which lets
 // the kernel start streaming it before its predecessor has finished.  split_hint: 0 = choose, 1 = no K split,
 // n = at most n CTAs (a cluster) per 128-feature tile.
 // Returns a cudaError_t value, -1 for arguments it cannot take, -2 when the TMA encoder is missing.
 int blitz_gemm_decode(const void* X, int64_t lda, const void* W, int64_t ldb, void* C, int64_t ldc, const void* R,
                       int M, int N, int K, int epilogue, int up_col_off, int dtype, int static_w, int split_hint,
-                      int* status, float alpha, cudaStream_t stream) {
+                      int* status, float alpha, float beta, cudaStream_t stream) {
   using namespace blitz;
   if (!blitz_gemm_decode_supported(M, N, K, 0, epilogue)) return -1;
-  if ((lda & 7) || (ldb & 7) || (epilogue == 2 && (up_col_off & 7))) return -1;
+  if ((lda & 7) || (ldb & 7) || (epi_gated(epilogue) && (up_col_off & 7))) return -1;
   const int sms = device_sm_count();
   DecGemmParams p;
   p.C = C;
@@ -566,16 +574,18 @@ int blitz_gemm_decode(const void* X, int64_t lda, const void* W, int64_t ldb, vo
   p.tiles = (N + kDecTile - 1) / kDecTile;
   p.static_w = static_w;
   p.alpha = alpha;
+  p.beta = beta;
   p.status = status;
 
   CUtensorMap tx, tw;
   if (!get_tmap_2d(&tx, X, (uint64_t)K, (uint64_t)M, (uint64_t)lda * 2, kDecBK, (uint32_t)p.x_box_rows)) return -2;
-  const int w_cols = epilogue == 2 ? up_col_off + N : N;
+  const int w_cols = epi_gated(epilogue) ? up_col_off + N : N;
   if (!get_tmap_2d(&tw, W, (uint64_t)w_cols, (uint64_t)K, (uint64_t)ldb * 2, 64, kDecBK)) return -2;
 
   cudaError_t e;
   if (dtype == 1) {
     e = epilogue == 2   ? launch_dec<__nv_bfloat16, 2>(tx, tw, p, split_hint, sms, stream)
+        : epilogue == 7 ? launch_dec<__nv_bfloat16, 7>(tx, tw, p, split_hint, sms, stream)
         : epilogue == 4 ? launch_dec<__nv_bfloat16, 4>(tx, tw, p, split_hint, sms, stream)
         : epilogue == 6 ? launch_dec<__nv_bfloat16, 6>(tx, tw, p, split_hint, sms, stream)
         : epilogue == 5 ? launch_dec<__nv_bfloat16, 5>(tx, tw, p, split_hint, sms, stream)
@@ -583,6 +593,7 @@ int blitz_gemm_decode(const void* X, int64_t lda, const void* W, int64_t ldb, vo
                         : launch_dec<__nv_bfloat16, 0>(tx, tw, p, split_hint, sms, stream);
   } else {
     e = epilogue == 2   ? launch_dec<__half, 2>(tx, tw, p, split_hint, sms, stream)
+        : epilogue == 7 ? launch_dec<__half, 7>(tx, tw, p, split_hint, sms, stream)
         : epilogue == 4 ? launch_dec<__half, 4>(tx, tw, p, split_hint, sms, stream)
         : epilogue == 6 ? launch_dec<__half, 6>(tx, tw, p, split_hint, sms, stream)
         : epilogue == 5 ? launch_dec<__half, 5>(tx, tw, p, split_hint, sms, stream)

@@ -37,6 +37,7 @@
 #include "launch.cuh"
 #include "ptx.cuh"
 #include "tmap.cuh"
+#include "gemm_gate.cuh"
 #include <cstdlib>
 #include <type_traits>
 
@@ -55,7 +56,8 @@ constexpr int kPairFinalStagingBytes = kPairSlabsMax * 4 * 4096;  // a pair's la
 struct PairParams {
   void* C;         // fp32 outputs (the 16-bit ones are stored through tmap_c)
   const void* R;
-  float alpha;     // axpy; soft cap
+  float alpha;     // axpy; soft cap; limit of the clamped unit
+  float beta;      // clamped unit (R: its biases)
   int64_t ldc;
   int M, N, K;
   int bnf;         // UMMA N = accumulator columns of a tile (128 or 256)
@@ -227,7 +229,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
           const int nt = n_super * nacc + a;
           uint8_t* sb = smem + stage * stage_bytes + a_bytes + a * b_bytes;
           int col;
-          if (EPI == 2) col = (rank == 0 ? 0 : p.up_col_off) + nt * half;
+          if (epi_gated(EPI)) col = (rank == 0 ? 0 : p.up_col_off) + nt * half;
           else col = nt * bnf + static_cast<int>(rank) * half;
           for (int s = 0; s < half / 64; ++s)
             ptx::tma_load_2d_pair(sb + s * 8192, &tmap_b, full0 + 8u * stage, col + s * 64, kb * kPairBK);
@@ -525,7 +527,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                     for (int j = 0; j < n_contrib; ++j) {
                       const float* src = p.ws + ((static_cast<size_t>(pair + 1 + j) * 2 + rank) * nacc + a) * slot_floats;
                       uint8_t* dst = smem + static_cast<size_t>(j) * round_bytes;
-                      if (EPI == 2) {
+                      if (epi_gated(EPI)) {
                         // gate columns [r * w, (r + 1) * w) and up columns half + the same, w = out_cols / rounds
                         const uint32_t w = static_cast<uint32_t>(p.out_cols / rounds);
                         ptx::bulk_load_1d(dst, src + static_cast<size_t>(r * w) * kPairRows, w * kPairRows * 4, fix_bar);
@@ -562,7 +564,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                 uint32_t v[32];
                 float gt[32], up[32];
                 ptx::tmem_ld_32x32(taddr + c, v);
-                if (EPI == 2) {
+                if (epi_gated(EPI)) {
                   uint32_t t[32];
                   ptx::tmem_ld_32x32(taddr + half + c, t);
                   ptx::tmem_ld_wait();
@@ -586,7 +588,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                           *reinterpret_cast<const float4*>(base + static_cast<size_t>(c_in / 4 + jj) * (kPairRows * 16));
                       gt[4 * jj] += f.x; gt[4 * jj + 1] += f.y; gt[4 * jj + 2] += f.z; gt[4 * jj + 3] += f.w;
                     }
-                    if (EPI == 2) {
+                    if (epi_gated(EPI)) {
                       const uint8_t* ub = base + round_bytes / 2;
 #pragma unroll
                       for (int jj = 0; jj < 8; ++jj) {
@@ -597,7 +599,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                     }
                   }
                 }
-                if (EPI >= 4) {
+                if (epi_f32(EPI)) {
                   // fp32 output: a thread's 32 columns are a whole 128-byte line, stored directly
                   if (row_ok) {
                     float* dst = reinterpret_cast<float*>(p.C) + static_cast<int64_t>(row) * p.ldc + n0 + c;
@@ -625,7 +627,13 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                   continue;
                 }
                 uint4 o4[4];
-                pair_convert32<T, EPI>(gt, up, rpre[i], o4);
+                if (EPI == kEpiClampGlu) {
+                  float y[32];
+                  clamp_glu32<T>(reinterpret_cast<const T*>(p.R), p.up_col_off, n0 + c, p.N, p.alpha, p.beta, gt, up, y);
+                  pair_convert32<T, 0>(y, up, rpre[i], o4);
+                } else {
+                  pair_convert32<T, EPI>(gt, up, rpre[i], o4);
+                }
                 // 128-byte rows, 16-byte chunks XOR-swizzled by row: the layout the TMA store expects
                 uint8_t* rowp = boxes + ((i & (nbuf - 1)) * 4 + q) * 4096 + lane * 128;
 #pragma unroll
@@ -721,7 +729,7 @@ static int pair_launch(const CUtensorMap& ta, const CUtensorMap& tb, const CUten
   // partials and each finalises its share of the slabs.  upp_hint = -n asks for n parts.
   p.split = 0;
   int upp = 0;
-  if (EPI != 2 && p.nacc == 1 && upp_hint <= 0) {
+  if (!epi_gated(EPI) && p.nacc == 1 && upp_hint <= 0) {
     int parts = upp_hint < 0 ? -upp_hint : max_pairs / tiles;
     if (parts > nslab) parts = nslab;
     if (parts > 4) parts = 4;
@@ -779,12 +787,13 @@ void blitz_gemm_pair_set_trace(unsigned long long* buf) { blitz::g_pair_trace = 
 
 // Whether blitz_gemm_pair takes this problem.
 int blitz_gemm_pair_supported(int M, int N, int K, int b_layout, int epilogue) {
-  return M >= 1 && b_layout == 0 && ((epilogue >= 0 && epilogue <= 2) || (epilogue >= 4 && epilogue <= 6)) && (N & 7) == 0 && (K & 7) == 0 && N >= 64;
+  return M >= 1 && b_layout == 0 && ((epilogue >= 0 && epilogue <= 2) || (epilogue >= 4 && epilogue <= blitz::kEpiClampGlu)) && (N & 7) == 0 && (K & 7) == 0 && N >= 64;
 }
 
 // C = A W (+R | silu-mul).  A [M, lda>=K], W [K, ldb>=columns] row-major, C/R [M, ldc>=N].  dtype 0 fp16, 1 bf16.
 // epilogue 0 store, 1 add R (C may be R), 2 silu(gate)*up with the up columns starting at up_col_off, 4 store with C in
-// fp32, 5 C += alpha * acc with C in fp32, 6 alpha * tanh(acc / alpha) with C in fp32.
+// fp32, 5 C += alpha * acc with C in fp32, 6 alpha * tanh(acc / alpha) with C in fp32, 7 clamped gated unit (gemm_gate.cuh; R:
+// its biases, alpha: its limit).
 // bnf_hint: accumulator columns per tile (0 = choose, 128 or 256); nacc_hint: tiles per pair that share the
 // activation tiles (0 = choose, 1 or 2); upp_hint: units per CTA pair (0 = choose; -n = cut every tile into n
 // equal K parts, one pair each).
@@ -794,10 +803,10 @@ int blitz_gemm_pair_supported(int M, int N, int K, int b_layout, int epilogue) {
 int blitz_gemm_pair(const void* A, int64_t lda, const void* W, int64_t ldb, void* C, int64_t ldc, const void* R, int M,
                     int N, int K, int epilogue, int up_col_off, int dtype, int static_b, int bnf_hint, int nacc_hint,
                     int upp_hint, void* ws, int64_t ws_bytes, unsigned* flags, int num_flags, int* status,
-                    float alpha, cudaStream_t stream) {
+                    float alpha, float beta, cudaStream_t stream) {
   using namespace blitz;
   if (!blitz_gemm_pair_supported(M, N, K, 0, epilogue) || !ws || !flags) return -1;
-  if ((lda & 7) || (ldb & 7) || (ldc & 7) || (epilogue == 2 && (up_col_off & 7))) return -1;
+  if ((lda & 7) || (ldb & 7) || (ldc & 7) || (epi_gated(epilogue) && (up_col_off & 7))) return -1;
   if (bnf_hint != 0 && bnf_hint != 128 && bnf_hint != 256) return -1;
   if (nacc_hint < 0 || nacc_hint > 2) return -1;
   const int sms = device_sm_count();
@@ -805,6 +814,7 @@ int blitz_gemm_pair(const void* A, int64_t lda, const void* W, int64_t ldb, void
   p.R = R;
   p.C = C;
   p.alpha = alpha;
+  p.beta = beta;
   p.ldc = ldc;
   p.M = M;
   p.N = N;
@@ -817,13 +827,13 @@ int blitz_gemm_pair(const void* A, int64_t lda, const void* W, int64_t ldb, void
   // every cut through a tile costs a partial exchange.  256 columns once no tile is cut into more than about six
   // pieces; two accumulators once there are about one and a half tiles per pair (measured: the gate-up projection of
   // Llama-3-8B, 112 tiles, takes 59.5 us on 56 pairs with two accumulators against 62.5 us on 74 pairs with one).
-  const int oc256 = epilogue == 2 ? 128 : 256;
+  const int oc256 = epi_gated(epilogue) ? 128 : 256;
   const int tiles256 = p.tiles_m * ((N + oc256 - 1) / oc256);
   int bnf = bnf_hint ? bnf_hint : (tiles256 * 6 >= sms / 2 ? 256 : 128);
   int nacc = nacc_hint ? nacc_hint : ((bnf == 256 && tiles256 * 4 >= sms * 3) ? 2 : 1);
   p.bnf = bnf;
   p.nacc = nacc;
-  p.out_cols = epilogue == 2 ? bnf / 2 : bnf;
+  p.out_cols = epi_gated(epilogue) ? bnf / 2 : bnf;
   p.tiles_n = (N + p.out_cols - 1) / p.out_cols;
   p.supers_n = (p.tiles_n + nacc - 1) / nacc;
   p.static_b = static_b;
@@ -836,9 +846,9 @@ int blitz_gemm_pair(const void* A, int64_t lda, const void* W, int64_t ldb, void
 
   CUtensorMap ta, tb, tc;
   if (!get_tmap_2d(&ta, A, (uint64_t)K, (uint64_t)M, (uint64_t)lda * 2, kPairBK, kPairRows)) return -2;
-  const int w_cols = epilogue == 2 ? up_col_off + N : N;
+  const int w_cols = epi_gated(epilogue) ? up_col_off + N : N;
   if (!get_tmap_2d(&tb, W, (uint64_t)w_cols, (uint64_t)K, (uint64_t)ldb * 2, 64, kPairBK)) return -2;
-  if (epilogue >= 4) {
+  if (epi_f32(epilogue)) {
     tc = ta;  // fp32 outputs are stored without TMA; the map is not used
   } else if (!get_tmap_2d(&tc, C, (uint64_t)N, (uint64_t)M, (uint64_t)ldc * 2, 64, 32)) {
     return -2;
@@ -846,6 +856,7 @@ int blitz_gemm_pair(const void* A, int64_t lda, const void* W, int64_t ldb, void
 
   if (dtype == 1) {
     return epilogue == 2   ? pair_launch<__nv_bfloat16, 2>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
+           : epilogue == 7 ? pair_launch<__nv_bfloat16, 7>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
            : epilogue == 4 ? pair_launch<__nv_bfloat16, 4>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
            : epilogue == 6 ? pair_launch<__nv_bfloat16, 6>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
            : epilogue == 5 ? pair_launch<__nv_bfloat16, 5>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
@@ -853,6 +864,7 @@ int blitz_gemm_pair(const void* A, int64_t lda, const void* W, int64_t ldb, void
                            : pair_launch<__nv_bfloat16, 0>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream);
   }
   return epilogue == 2   ? pair_launch<__half, 2>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
+           : epilogue == 7 ? pair_launch<__half, 7>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
            : epilogue == 4 ? pair_launch<__half, 4>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
            : epilogue == 6 ? pair_launch<__half, 6>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)
            : epilogue == 5 ? pair_launch<__half, 5>(ta, tb, tc, p, upp_hint, ws_bytes, num_flags, stream)

@@ -12,6 +12,7 @@
 #include "ptx.cuh"
 #include "scalar.cuh"
 #include "grouped.cuh"
+#include "gemm_gate.cuh"
 
 namespace blitz {
 
@@ -23,16 +24,17 @@ struct SimtGemmParams {
   void* C;
   int64_t lda, ldb, ldc;
   int M, N, K, up_off, a_step, c_step;
-  float alpha;
+  float alpha, beta;
+  const void* bias;
 };
 
-enum SimtEpilogue : int { kSimtStore = 0, kSimtSiluMul = 2, kSimtStoreF32 = 4, kSimtAxpyF32 = 5, kSimtCapF32 = 6 };
+enum SimtEpilogue : int { kSimtStore = 0, kSimtSiluMul = 2, kSimtStoreF32 = 4, kSimtAxpyF32 = 5, kSimtCapF32 = 6, kSimtClampGlu = kEpiClampGlu };
 
 template <typename T, int EPI>
 __global__ void __launch_bounds__(kSgThreads) gemm_simt_kernel(const SimtGemmParams p) {
   ptx::griddep_launch_dependents();
   ptx::griddep_wait();
-  constexpr int H = EPI == kSimtSiluMul ? 2 : 1;
+  constexpr int H = epi_gated(EPI) ? 2 : 1;
   __shared__ float sA[kSgK][kSgT + 1];
   __shared__ float sB[H][kSgK][kSgT];
   const int m0 = blockIdx.y * kSgT, n0 = blockIdx.x * kSgT, g = blockIdx.z;
@@ -90,6 +92,11 @@ __global__ void __launch_bounds__(kSgThreads) gemm_simt_kernel(const SimtGemmPar
         reinterpret_cast<float*>(p.C)[at] = p.alpha * tanhf(acc[0][i][j] / p.alpha);
       } else if (EPI == kSimtStoreF32) {
         reinterpret_cast<float*>(p.C)[at] = acc[0][i][j];
+      } else if (EPI == kSimtClampGlu) {
+        const T* bias = reinterpret_cast<const T*>(p.bias) + n;
+        const float z = fminf(acc[0][i][j] + ldf<T>(bias), p.alpha);
+        const float u = fminf(fmaxf(acc[H - 1][i][j] + ldf<T>(bias + p.up_off), -p.alpha), p.alpha);
+        stf<T>(reinterpret_cast<T*>(p.C) + at, z * sigmoid_f(p.beta * z) * (u + 1.f));
       } else if (EPI == kSimtSiluMul) {
         stf<T>(reinterpret_cast<T*>(p.C) + at, silu_acc(acc[0][i][j]) * acc[H - 1][i][j]);
       } else {
@@ -104,6 +111,7 @@ static cudaError_t launch_simt(const SimtGemmParams& p, int epi, int groups, cud
   const dim3 grid((p.N + kSgT - 1) / kSgT, (p.M + kSgT - 1) / kSgT, groups), block(kSgThreads);
   switch (epi) {
     case kSimtSiluMul: return launch_pdl(gemm_simt_kernel<T, kSimtSiluMul>, grid, block, 0, stream, p);
+    case kSimtClampGlu: return launch_pdl(gemm_simt_kernel<T, kSimtClampGlu>, grid, block, 0, stream, p);
     case kSimtStoreF32: return launch_pdl(gemm_simt_kernel<T, kSimtStoreF32>, grid, block, 0, stream, p);
     case kSimtCapF32: return launch_pdl(gemm_simt_kernel<T, kSimtCapF32>, grid, block, 0, stream, p);
     case kSimtAxpyF32: return launch_pdl(gemm_simt_kernel<T, kSimtAxpyF32>, grid, block, 0, stream, p);
@@ -181,14 +189,16 @@ using namespace blitz;
 
 // C[M, N] = A[M, K] B[K, N] per group; dtype 0 fp16, 1 bf16, 2 fp32 (of A and B, and of C unless the epilogue says
 // fp32).  epilogue 0 store, 2 silu(gate) * up with the up columns of B from up_off on, 4 store as fp32,
-// 5 C += alpha * acc with C fp32, 6 alpha * tanh(acc / alpha) as fp32.  a_step, c_step: columns of A and C between two groups.
+// 5 C += alpha * acc with C fp32, 6 alpha * tanh(acc / alpha) as fp32, 7 clamped gated unit
+// (gemm_gate.cuh).  a_step, c_step: columns of A and C between two groups.
 int blitz_gemm_simt(const void* A, int64_t lda, const void* B, int64_t ldb, void* C, int64_t ldc, int M, int N, int K,
-                    int epilogue, int up_off, float alpha, int groups, int a_step, int c_step, int dtype, cudaStream_t stream) {
+                    int epilogue, int up_off, const void* bias, float alpha, float beta, int groups, int a_step, int c_step, int dtype, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0 || groups <= 0) return 0;
-  if (epilogue != 0 && epilogue != 2 && epilogue != 4 && epilogue != 5 && epilogue != 6) return -1;
+  if (epilogue != 0 && epilogue != 2 && epilogue != 4 && epilogue != 5 && epilogue != 6 && epilogue != kEpiClampGlu) return -1;
+  if (epilogue == kEpiClampGlu && bias == nullptr) return -1;
   if (epilogue == 6 && !(alpha > 0.f)) return -1;
   if ((M + kSgT - 1) / kSgT > 65535 || groups > 65535) return -1;
-  SimtGemmParams p{A, B, C, lda, ldb, ldc, M, N, K, up_off, a_step, c_step, alpha};
+  SimtGemmParams p{A, B, C, lda, ldb, ldc, M, N, K, up_off, a_step, c_step, alpha, beta, bias};
   cudaError_t e = cudaSuccess;
   BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_simt<T>(p, epilogue, groups, stream)));
   return (int)e;

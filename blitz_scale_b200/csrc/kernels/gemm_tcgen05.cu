@@ -13,6 +13,7 @@
 //   store f32  C = acc, C in fp32           (what a recurrence takes in 32 bits)
 //   axpy f32   C += alpha * acc, C in fp32  (output projections of models whose residual stream is fp32)
 //   cap f32    C = alpha * tanh(acc / alpha), C in fp32  (soft-capped logits)
+//   clamp_glu  a clamped gated unit with biases (gemm_gate.cuh)
 //
 // Block-diagonal products (groups > 1): B is `groups` blocks [K,N] stacked along K; group g takes the K columns of A
 // from g * a_step on and the N columns of C from g * c_step on (heads of a wider activation).  An N tile belongs to one group and simply starts its K walk there
@@ -35,6 +36,7 @@
 #include "launch.cuh"
 #include "ptx.cuh"
 #include "tmap.cuh"
+#include "gemm_gate.cuh"
 #include <type_traits>
 
 namespace blitz {
@@ -72,7 +74,8 @@ struct GemmParams {
   uint32_t wait_value;
   int n_fast;  // tensor-parallel fusion: N runs fastest over the tiles, M blocks start at m_rot (see gemm_tile_blocks)
   int m_rot;
-  float alpha;      // axpy; soft cap
+  float alpha;      // axpy; soft cap; limit of the clamped unit
+  float beta;       // clamped unit (R: its biases)
   int groups;       // diagonal blocks (1: an ordinary product); N and K are those of one block
   int group_tiles;  // N tiles per block
   int a_step, c_step;  // columns of A and C between two blocks
@@ -180,7 +183,12 @@ __device__ __forceinline__ void store_chunk(const GemmParams& p, const float (&a
     return;
   }
   uint32_t out[16];
-  if (EPI == kEpiSiluMul) {
+  if (EPI == kEpiClampGlu) {
+    float y[32];
+    clamp_glu32<T>(reinterpret_cast<const T*>(p.R), p.up_col_off, col0, p.N, p.alpha, p.beta, acc, up, y);
+#pragma unroll
+    for (int i = 0; i < 16; ++i) out[i] = pack2<T>(y[2 * i], y[2 * i + 1]);
+  } else if (epi_gated(EPI)) {
 #pragma unroll
     for (int i = 0; i < 16; ++i) out[i] = pack2<T>(silu_f(acc[2 * i]) * up[2 * i], silu_f(acc[2 * i + 1]) * up[2 * i + 1]);
   } else if (EPI == kEpiAdd) {
@@ -249,7 +257,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_b,
                     const GemmParams p) {
   using Cfg = GemmCfg<BN>;
-  constexpr int kOutCols = (EPI == kEpiSiluMul) ? BN / 2 : BN;  // output columns per tile
+  constexpr int kOutCols = (epi_gated(EPI)) ? BN / 2 : BN;  // output columns per tile
   constexpr uint32_t kFmt = std::is_same<T, __nv_bfloat16>::value ? 1u : 0u;
   constexpr uint32_t kIdesc = ptx::make_idesc_f16(kFmt, 0u, B_KMAJOR ? 0u : 1u, kBM, BN);
   const int S = Cfg::num_stages(p.a_box_rows);
@@ -350,7 +358,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
           uint8_t* sb = smem_b + stage * Cfg::kBBytes;
           if (B_KMAJOR) {
             // B is [N,K]: one box of BN rows x 64 K-elements per half (silu: gate rows then up rows).
-            if (EPI == kEpiSiluMul) {
+            if (epi_gated(EPI)) {
               ptx::tma_load_2d(sb, &tmap_b, &full_bar[stage], kb * kBK, n0);
               ptx::tma_load_2d(sb + (BN / 2) * 128, &tmap_b, &full_bar[stage], kb * kBK, p.up_col_off + n0);
             } else {
@@ -362,7 +370,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
 #pragma unroll
             for (int s = 0; s < kSlabs; ++s) {
               int col;
-              if (EPI == kEpiSiluMul) {
+              if (epi_gated(EPI)) {
                 constexpr int kHalfSlabs = kSlabs / 2;
                 col = (s < kHalfSlabs) ? (n0 + s * 64) : (p.up_col_off + n0 + (s - kHalfSlabs) * 64);
               } else {
@@ -462,7 +470,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
           uint32_t v[32];
           float a[32], u[32];
           ptx::tmem_ld_32x32(taddr + c, v);
-          if (EPI == kEpiSiluMul) {
+          if (epi_gated(EPI)) {
             uint32_t t[32];
             ptx::tmem_ld_32x32(taddr + BN / 2 + c, t);
             ptx::tmem_ld_wait();
@@ -524,7 +532,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
                 for (int j = 0; j < 8; ++j) {
                   a[4 * j] += f[j].x; a[4 * j + 1] += f[j].y; a[4 * j + 2] += f[j].z; a[4 * j + 3] += f[j].w;
                 }
-                if (EPI == kEpiSiluMul) {
+                if (epi_gated(EPI)) {
 #pragma unroll
                   for (int j = 0; j < 8; ++j)
                     f[j] = __ldcg(reinterpret_cast<const float4*>(ps + static_cast<size_t>((BN / 2 + c) / 4 + j) * (kBM * 4)));
@@ -573,8 +581,8 @@ static cudaError_t dispatch_bn(int bn, const CUtensorMap& ta, const CUtensorMap&
     case 256: return launch_gemm<T, 256, B_KMAJOR, EPI>(ta, tb, p, grid, stream);
     case 128: return launch_gemm<T, 128, B_KMAJOR, EPI>(ta, tb, p, grid, stream);
     default:
-      if (EPI == kEpiSiluMul) return launch_gemm<T, 128, B_KMAJOR, EPI>(ta, tb, p, grid, stream);
-      return launch_gemm<T, 64, B_KMAJOR, (EPI == kEpiSiluMul ? kEpiStore : EPI)>(ta, tb, p, grid, stream);
+      if (epi_gated(EPI)) return launch_gemm<T, 128, B_KMAJOR, EPI>(ta, tb, p, grid, stream);
+      return launch_gemm<T, 64, B_KMAJOR, (epi_gated(EPI) ? static_cast<int>(kEpiStore) : EPI)>(ta, tb, p, grid, stream);
   }
 }
 
@@ -584,6 +592,7 @@ static cudaError_t dispatch_epi(int epi, int bn, const CUtensorMap& ta, const CU
   switch (epi) {
     case kEpiAdd: return dispatch_bn<T, B_KMAJOR, kEpiAdd>(bn, ta, tb, p, grid, stream);
     case kEpiSiluMul: return dispatch_bn<T, B_KMAJOR, kEpiSiluMul>(bn, ta, tb, p, grid, stream);
+    case kEpiClampGlu: return dispatch_bn<T, B_KMAJOR, kEpiClampGlu>(bn, ta, tb, p, grid, stream);
     case kEpiStoreF32: return dispatch_bn<T, B_KMAJOR, kEpiStoreF32>(bn, ta, tb, p, grid, stream);
     case kEpiCapF32: return dispatch_bn<T, B_KMAJOR, kEpiCapF32>(bn, ta, tb, p, grid, stream);
     case kEpiAxpyF32: return dispatch_bn<T, B_KMAJOR, kEpiAxpyF32>(bn, ta, tb, p, grid, stream);
@@ -617,11 +626,11 @@ int blitz_gemm_tile_n(int M, int N, int epilogue, int bn_hint) {
   const int sms = device_sm_count();
   int bn = bn_hint;
   if (!bn) {
-    const int oc256 = epilogue == kEpiSiluMul ? 128 : 256;
+    const int oc256 = epi_gated(epilogue) ? 128 : 256;
     const int tiles256 = ((M + kBM - 1) / kBM) * ((N + oc256 - 1) / oc256);
     bn = tiles256 >= sms ? 256 : 128;
   }
-  if (epilogue == kEpiSiluMul && bn < 128) bn = 128;
+  if (epi_gated(epilogue) && bn < 128) bn = 128;
   return bn;
 }
 
@@ -637,20 +646,20 @@ struct BlitzGemmTp {
 static int gemm_impl(const void* A, int64_t lda, const void* B, int64_t ldb, void* C, int64_t ldc, const void* R, int M,
                      int N, int K, int b_layout, int epilogue, int up_col_off, int dtype, int bn_hint, int split_hint,
                      void* ws, int64_t ws_bytes, unsigned* tickets, int num_tickets, int* status,
-                     const BlitzGemmTp* tpa, float alpha, int groups, int a_step, int c_step, cudaStream_t stream) {
+                     const BlitzGemmTp* tpa, float alpha, float beta, int groups, int a_step, int c_step, cudaStream_t stream) {
   using namespace blitz;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if (groups < 1 || (groups > 1 && (((a_step | c_step) & 7) != 0 || a_step < 0 || c_step < N || b_layout != 0 || tpa != nullptr ||
                                     (epilogue != kEpiStore && epilogue != kEpiStoreF32))))
     return -1;
   if ((N & 7) || (K & 7) || (lda & 7) || (ldb & 7) || (ldc & 7)) return -1;
-  if (epilogue == kEpiSiluMul && (up_col_off & 7)) return -1;
+  if (epi_gated(epilogue) && (up_col_off & 7)) return -1;
   const int sms = device_sm_count();
   // 256-wide tiles are the most efficient per FLOP (a 128xNx16 instruction costs ~95 cycles at N = 64,
   // ~105 at N = 128, ~150 at N = 256); when they would leave SMs idle, 128-wide tiles plus split-K win.
   const int bn = blitz_gemm_tile_n(M, N * groups, epilogue, bn_hint);
-  const int out_cols = epilogue == kEpiSiluMul ? bn / 2 : bn;
-  const int b_cols_total = epilogue == kEpiSiluMul ? up_col_off + N : N;
+  const int out_cols = epi_gated(epilogue) ? bn / 2 : bn;
+  const int b_cols_total = epi_gated(epilogue) ? up_col_off + N : N;
 
   GemmParams p;
   p.C = C;
@@ -668,6 +677,7 @@ static int gemm_impl(const void* A, int64_t lda, const void* B, int64_t ldb, voi
   p.a_step = a_step;
   p.c_step = c_step;
   p.alpha = alpha;
+  p.beta = beta;
   p.status = status;
   p.tp = 1; p.tp_rank = 0; p.rows_per_rank = M; p.wait_flags = nullptr; p.n_wait = 0; p.wait_value = 0; p.m_rot = 0; p.n_fast = 0;
   for (int i = 0; i < 8; ++i) { p.push_base[i] = nullptr; p.push_flags[i] = nullptr; }
@@ -713,7 +723,7 @@ static int gemm_impl(const void* A, int64_t lda, const void* B, int64_t ldb, voi
   } else if (b_layout == 0) {
     okb = get_tmap_2d(&tb, B, (uint64_t)b_cols_total, (uint64_t)K, (uint64_t)ldb * 2, 64, kBK);
   } else {
-    const uint32_t box_rows = epilogue == kEpiSiluMul ? bn / 2 : bn;
+    const uint32_t box_rows = epi_gated(epilogue) ? bn / 2 : bn;
     okb = get_tmap_2d(&tb, B, (uint64_t)K, (uint64_t)b_cols_total, (uint64_t)ldb * 2, kBK, box_rows);
   }
   if (!okb) return -2;
@@ -733,11 +743,11 @@ static int gemm_impl(const void* A, int64_t lda, const void* B, int64_t ldb, voi
 
 int blitz_gemm(const void* A, int64_t lda, const void* B, int64_t ldb, void* C, int64_t ldc, const void* R, int M,
                int N, int K, int b_layout, int epilogue, int up_col_off, int dtype, int bn_hint, int split_hint,
-               void* ws, int64_t ws_bytes, unsigned* tickets, int num_tickets, int* status, float alpha, int groups,
+               void* ws, int64_t ws_bytes, unsigned* tickets, int num_tickets, int* status, float alpha, float beta, int groups,
                int a_step, int c_step, cudaStream_t stream) {
   if (epilogue == blitz::kEpiPushRS) return -1;
   return gemm_impl(A, lda, B, ldb, C, ldc, R, M, N, K, b_layout, epilogue, up_col_off, dtype, bn_hint, split_hint, ws,
-                   ws_bytes, tickets, num_tickets, status, nullptr, alpha, groups, a_step, c_step, stream);
+                   ws_bytes, tickets, num_tickets, status, nullptr, alpha, beta, groups, a_step, c_step, stream);
 }
 
 // Tensor-parallel variant: epilogue 3 pushes the partial result to the owner ranks' staging areas
@@ -748,7 +758,7 @@ int blitz_gemm_tp(const void* A, int64_t lda, const void* B, int64_t ldb, void* 
                   void* ws, int64_t ws_bytes, unsigned* tickets, int num_tickets, int* status, const BlitzGemmTp* tp,
                   cudaStream_t stream) {
   return gemm_impl(A, lda, B, ldb, C, ldc, R, M, N, K, b_layout, epilogue, up_col_off, dtype, bn_hint, split_hint, ws,
-                   ws_bytes, tickets, num_tickets, status, tp, 1.f, 1, 0, 0, stream);
+                   ws_bytes, tickets, num_tickets, status, tp, 1.f, 0.f, 1, 0, 0, stream);
 }
 
 }  // extern "C"

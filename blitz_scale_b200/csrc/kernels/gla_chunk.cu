@@ -22,6 +22,9 @@
 // products that involve them split their fp32 operands into two bf16 numbers (x = hi + lo, relative error 2^-17) and
 // drop only the lo * lo term.
 //
+// Second form (WKV, see gla.cu): o_t sees the decays up to the token before it, so q takes b_(t-1) where the first form takes b_t,
+// the scores are those of s < t, and the token's own score is sum_c q_tc u_c k_tc without any decay.
+//
 // A block of 16 warps owns (row, head, 64 or 128 value columns) and walks the row's chunks with the state in registers; everything
 // a chunk reads from global memory is requested one chunk (the gates: half a chunk) ahead.  The blocks of one head form a thread-block cluster, which exchanges the 64 partial sums of squares per chunk through
 // distributed shared memory, so that the output norm and the gate are applied here and nothing but the result is
@@ -44,7 +47,10 @@ constexpr float kGcMaxDecay = 80.f;
 struct GlaChunkParams {
   const __nv_bfloat16 *q, *k, *v, *g, *low;
   int64_t row;
-  const __nv_bfloat16 *a2, *a2_b, *norm;
+  const float* low32;    // WKV: [tokens][low_row], instead of low
+  int64_t low_row;
+  const __nv_bfloat16 *a2, *a2_b, *norm, *bonus;  // norm: head h's from h * norm_step on; bonus [heads * dim]: WKV
+  int norm_step;
   float* cum;      // [tokens][heads * dim]: running sums of the log decays within each chunk
   float* state;    // [slots][heads][dim][vdim]
   __nv_bfloat16* out;
@@ -62,8 +68,9 @@ __device__ __forceinline__ float log_sigmoid_ex2(float z) {
   return fminf(z, 0.f) - l;
 }
 
-// Running sum of log(sigmoid(low a2 + b)) / tau over a chunk; a thread per channel.
+// Running sum of log(sigmoid(low a2 + b)) / tau (WKV: -exp(tanh(low) a2 + b)) over a chunk; a thread per channel.
 constexpr int kGdThreads = 128;
+template <bool WKV>
 __global__ void __launch_bounds__(kGdThreads) gla_decay_kernel(const GlaChunkParams p) {
   ptx::griddep_launch_dependents();
   ptx::griddep_wait();
@@ -72,7 +79,8 @@ __global__ void __launch_bounds__(kGdThreads) gla_decay_kernel(const GlaChunkPar
   const int t0 = p.tok_indptr[r] + blockIdx.y * kGcC, n = min(kGcC, p.tok_indptr[r + 1] - t0);
   if (n <= 0) return;
   for (int i = threadIdx.x; i < n * p.rank; i += kGdThreads)
-    s_low[i] = ldf(p.low + static_cast<int64_t>(t0 + i / p.rank) * p.row + i % p.rank);
+    s_low[i] = WKV ? tanhf(p.low32[static_cast<int64_t>(t0 + i / p.rank) * p.low_row + i % p.rank])
+                   : ldf(p.low + static_cast<int64_t>(t0 + i / p.rank) * p.row + i % p.rank);
   __syncthreads();
   const int c = blockIdx.x * kGdThreads + threadIdx.x;
   if (c >= hk) return;
@@ -89,7 +97,8 @@ __global__ void __launch_bounds__(kGdThreads) gla_decay_kernel(const GlaChunkPar
     for (int i = 0; i < kKeep; ++i)
       if (i < p.rank) z += low[i] * w[i];
     for (int i = kKeep; i < p.rank; ++i) z += low[i] * ldf(p.a2 + static_cast<int64_t>(i) * hk + c);
-    sum += log_sigmoid_ex2(z) * p.inv_tau;
+    sum += WKV ? -fminf(__expf(z), 104.f)  // (e^-104 is zero in fp32; larger steps would only cost the sum its digits)
+               : log_sigmoid_ex2(z) * p.inv_tau;
     p.cum[static_cast<int64_t>(t0 + t) * hk + c] = sum;
   }
 }
@@ -117,6 +126,7 @@ struct GcSmem {
   float ss[2][kParts][kGcC];              // partial sums of squares of every cluster rank, by parity of the chunk
   float part[4][kGcC];
   float norm[VB];
+  float own[kGcC];                        // WKV: scores of the tokens with themselves
   int wide[4];                            // block whose decay the factored form cannot hold
   __nv_bfloat16 qh[kGcC * kQ], ql[kGcC * kQ];  // q'
   __nv_bfloat16 ih[kGcC * kQ], il[kGcC * kQ];  // q e^b
@@ -131,7 +141,7 @@ __device__ __forceinline__ void gc_tile(int tile, int& i, int& j) {
   j = tile >= 6 ? i : (tile >= 3 ? tile - 3 : tile >= 1 ? tile - 1 : 0);
 }
 
-template <int DK, int VB>
+template <int DK, int VB, bool WKV>
 __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunkParams p) {
   using bf = __nv_bfloat16;
   using SM = GcSmem<DK, VB>;
@@ -195,7 +205,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
   // blocks the registers do not hold b as well: it is read, from L2, when the chunk starts)
   constexpr bool kAheadB = VB == kGcV;
   uint4 rq[NV], rk[NV], rv[VB / 64];
-  float rb8[NV][8], rref[2];
+  float rb8[NV][8], rbq[WKV ? NV : 1][8], rref[2];  // rbq: b of the token before (what q takes)
   auto request_b = [&](int chunk) {
     const int base = chunk * kGcC, last = min(kGcC, len - base) - 1;
     const float* cum = p.cum + static_cast<int64_t>(t_beg + base) * hk + h * p.dim;
@@ -205,6 +215,11 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
 #pragma unroll
       for (int j = 0; j < 8; ++j) rb8[i][j] = 0.f;
       if (e < kVecs && c < p.dim) ldf8(cum + static_cast<int64_t>(min(t, last)) * hk + c, rb8[i]);  // no decay past the end
+      if (WKV) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) rbq[WKV ? i : 0][j] = 0.f;
+        if (e < kVecs && c < p.dim && t > 0) ldf8(cum + static_cast<int64_t>(min(t - 1, last)) * hk + c, rbq[WKV ? i : 0]);
+      }
     }
   };
   auto request = [&](int chunk) {
@@ -242,7 +257,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
   request(0);
   keep_borders(0);
   if (tid < 4) sm.wide[tid] = 0;
-  if (tid < nv) sm.norm[tid] = ldf(p.norm + v0 + tid);
+  if (tid < nv) sm.norm[tid] = ldf(p.norm + static_cast<int64_t>(h) * p.norm_step + v0 + tid);
   __syncthreads();
 
   for (int ch = 0; ch < nchunks; ++ch) {
@@ -259,11 +274,21 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
         unpack8<bf>(rk[i], k8);
         ldf8(ref + blk * DK + c, lo8);
         ldf8(ref + (blk + 1) * DK + c, hi8);
+        if (WKV) {  // the lanes of a token are neighbours
+          float u8[8] = {}, own = 0.f;
+          if (c < p.dim) ldf8(p.bonus + h * p.dim + c, u8);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) own += q8[j] * u8[j] * k8[j];
+#pragma unroll
+          for (int o = 1; o < DK / 8; o <<= 1) own += __shfl_xor_sync(0xffffffffu, own, o);
+          if (c == 0) sm.own[t] = own;
+        }
+        const float(&b8)[8] = WKV ? rbq[WKV ? i : 0] : rb8[i];
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
           q8[j] *= p.q_scale;
-          i8[j] = q8[j] * __expf(rb8[i][j]);
-          q8[j] *= __expf(rb8[i][j] - lo8[j]);
+          i8[j] = q8[j] * __expf(b8[j]);
+          q8[j] *= __expf(b8[j] - lo8[j]);
           k8[j] *= __expf(hi8[j] - rb8[i][j]);
         }
         auto put = [&](const float (&x)[8], bf* dh, bf* dl) {
@@ -310,10 +335,10 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
         for (int e = 0; e < 8; ++e) {
           const int t = i * kGcB + g + ((e >> 1) & 1) * 8, s = i * kGcB + (e >> 2) * 8 + 2 * t4 + (e & 1);
           float x = 0.f;
-          if (s <= t && t < n_tok) {
+          if ((WKV ? s < t : s <= t) && t < n_tok) {
             const bf* qr = p.q + static_cast<int64_t>(t_beg + base + t) * p.row + h * p.dim;
             const bf* kr = p.k + static_cast<int64_t>(t_beg + base + s) * p.row + h * p.dim;
-            const float *bt = cum + static_cast<int64_t>(t) * hk, *bs = cum + static_cast<int64_t>(s) * hk;
+            const float *bt = cum + static_cast<int64_t>(WKV ? t - 1 : t) * hk, *bs = cum + static_cast<int64_t>(s) * hk;
             for (int c = 0; c < p.dim; ++c) x += ldf(qr + c) * ldf(kr + c) * __expf(bt[c] - bs[c]);
             x *= p.q_scale;
           }
@@ -355,6 +380,8 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
           if (i == j) {  // above the diagonal (a factored score may be anything there)
             if (s > t) x = 0.f;
             if (s + 1 > t) y = 0.f;
+            if (WKV && s == t) x = sm.own[i * kGcB + t];
+            if (WKV && s + 1 == t) y = sm.own[i * kGcB + t];
           }
           uint32_t hi, lo;
           split2(x, y, hi, lo);
@@ -509,9 +536,9 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
     }
 }
 
-template <int DK, int VB>
+template <int DK, int VB, bool WKV>
 static cudaError_t launch_gla_chunk(const GlaChunkParams& p, int rows, cudaStream_t stream) {
-  auto kern = gla_chunk_kernel<DK, VB>;
+  auto kern = gla_chunk_kernel<DK, VB, WKV>;
   constexpr int smem = (int)sizeof(GcSmem<DK, VB>);
   static_assert(smem <= 227 * 1024, "shared memory");
   static PerDeviceOnce once;
@@ -523,10 +550,29 @@ static cudaError_t launch_gla_chunk(const GlaChunkParams& p, int rows, cudaStrea
 
 // 128 value columns per block halve the work that every block of a head repeats (scaled operands, scores); 64 give twice
 // as many blocks, which is worth more while they do not fill the GPU.
-template <int DK>
+template <int DK, bool WKV>
 static cudaError_t launch_gla_width(const GlaChunkParams& p, int rows, int sms, cudaStream_t stream) {
   const bool wide = p.vdim > kGcV && (int64_t)rows * p.heads * ((p.vdim + kGcV - 1) / kGcV) > sms;
-  return wide ? launch_gla_chunk<DK, 2 * kGcV>(p, rows, stream) : launch_gla_chunk<DK, kGcV>(p, rows, stream);
+  return wide ? launch_gla_chunk<DK, 2 * kGcV, WKV>(p, rows, stream) : launch_gla_chunk<DK, kGcV, WKV>(p, rows, stream);
+}
+
+template <bool WKV>
+static int gla_chunk_any(const GlaChunkParams& p, int rows, int max_len, cudaStream_t stream) {
+  if (p.heads > 65535 || rows > 65535 || (p.row & 7) || (p.out_stride & 1)) return -1;
+  for (const void* x : {p.q, p.k, p.v})
+    if (reinterpret_cast<uintptr_t>(x) & 15) return -1;
+  if (WKV && (reinterpret_cast<uintptr_t>(p.bonus) & 15)) return -1;
+  if ((reinterpret_cast<uintptr_t>(p.g) | reinterpret_cast<uintptr_t>(p.out)) & 3) return -1;
+  if (reinterpret_cast<uintptr_t>(p.cum) & 15) return -1;
+  const int hk = p.heads * p.dim;
+  cudaError_t e = launch_pdl(gla_decay_kernel<WKV>, dim3((hk + kGdThreads - 1) / kGdThreads, (max_len + kGcC - 1) / kGcC, rows),
+                             dim3(kGdThreads), (size_t)kGcC * p.rank * sizeof(float), stream, p);
+  if (e != cudaSuccess) return (int)e;
+  const int sms = device_sm_count();
+  e = p.dim <= 32   ? launch_gla_width<32, WKV>(p, rows, sms, stream)
+      : p.dim <= 64 ? launch_gla_width<64, WKV>(p, rows, sms, stream)
+                    : launch_gla_width<128, WKV>(p, rows, sms, stream);
+  return (int)e;
 }
 
 }  // namespace blitz
@@ -549,23 +595,25 @@ int blitz_gla_chunk(const void* q, const void* k, const void* v, const void* g, 
                     cudaStream_t stream) {
   using bf = __nv_bfloat16;
   if (rows <= 0 || max_len <= 0) return 0;
-  if (!blitz_gla_chunk_supported(dim, vdim, rank) || (row & 7) || (out_stride & 1) || !(tau > 0.f) || heads > 65535 || rows > 65535)
-    return -1;
-  for (const void* x : {q, k, v})
-    if (reinterpret_cast<uintptr_t>(x) & 15) return -1;
-  if ((reinterpret_cast<uintptr_t>(g) | reinterpret_cast<uintptr_t>(out)) & 3) return -1;
-  if (reinterpret_cast<uintptr_t>(cum) & 15) return -1;
-  GlaChunkParams p{(const bf*)q, (const bf*)k, (const bf*)v, (const bf*)g, (const bf*)low, row, (const bf*)a2, (const bf*)a2_b,
-                   (const bf*)norm, cum, state, (bf*)out, out_stride, pos, tok_indptr, seq_slot, heads, dim, vdim, rank,
-                   num_slots, q_scale, 1.f / tau, eps, status};
-  const int hk = heads * dim;
-  cudaError_t e = launch_pdl(gla_decay_kernel, dim3((hk + kGdThreads - 1) / kGdThreads, (max_len + kGcC - 1) / kGcC, rows),
-                             dim3(kGdThreads), (size_t)kGcC * rank * sizeof(float), stream, p);
-  if (e != cudaSuccess) return (int)e;
-  const int sms = device_sm_count();
-  e = dim <= 32 ? launch_gla_width<32>(p, rows, sms, stream) : dim <= 64 ? launch_gla_width<64>(p, rows, sms, stream)
-                                                                        : launch_gla_width<128>(p, rows, sms, stream);
-  return (int)e;
+  if (!blitz_gla_chunk_supported(dim, vdim, rank) || !(tau > 0.f)) return -1;
+  GlaChunkParams p{(const bf*)q, (const bf*)k, (const bf*)v, (const bf*)g, (const bf*)low, row, nullptr, 0, (const bf*)a2,
+                   (const bf*)a2_b, (const bf*)norm, nullptr, 0, cum, state, (bf*)out, out_stride, pos, tok_indptr, seq_slot,
+                   heads, dim, vdim, rank, num_slots, q_scale, 1.f / tau, eps, status};
+  return gla_chunk_any<false>(p, rows, max_len, stream);
+}
+
+// The second form (see blitz_wkv_recurrent for what differs); bonus 16-byte aligned, dim a multiple of 8.
+int blitz_wkv_chunk(const void* q, const void* k, const void* v, const void* g, int64_t row, const float* low, int64_t low_row,
+                    const void* a2, const void* a2_b, const void* bonus, const void* norm, float* cum, float* state, void* out,
+                    int64_t out_stride, const int32_t* pos, const int32_t* tok_indptr, const int32_t* seq_slot, int rows,
+                    int max_len, int heads, int dim, int vdim, int rank, int num_slots, float eps, int* status, cudaStream_t stream) {
+  using bf = __nv_bfloat16;
+  if (rows <= 0 || max_len <= 0) return 0;
+  if (!blitz_gla_chunk_supported(dim, vdim, rank) || low == nullptr || bonus == nullptr) return -1;
+  GlaChunkParams p{(const bf*)q, (const bf*)k, (const bf*)v, (const bf*)g, nullptr, row, low, low_row, (const bf*)a2,
+                   (const bf*)a2_b, (const bf*)norm, (const bf*)bonus, vdim, cum, state, (bf*)out, out_stride, pos, tok_indptr, seq_slot,
+                   heads, dim, vdim, rank, num_slots, 1.f, 1.f, eps, status};
+  return gla_chunk_any<true>(p, rows, max_len, stream);
 }
 
 }  // extern "C"

@@ -5,7 +5,7 @@
 //   latent_rotate   the last `rot` dimensions of every query head, in place or to where the absorbed queries are
 //   latent_gather   whole pages, back to back (prompts: the operand of the product that expands keys and values)
 //
-// Rotation pairs are (i, i + rot / 2); frequencies are unevaluated sums of two fp32 numbers as in rope_store.cu.
+// Rotation pairs are (i, i + rot / 2), or (2 i, 2 i + 1); frequencies are unevaluated sums of two fp32 numbers as in rope_store.cu.
 #include "launch.cuh"
 #include "ptx.cuh"
 #include "scalar.cuh"
@@ -30,7 +30,7 @@ struct LatentStoreParams {
   void* pool;       // [max_pages][page_size][rank + rot]
   const float2* freq;
   float eps;
-  int q_rank, rank, rot, page_size, max_pages;
+  int q_rank, rank, rot, interleaved, page_size, max_pages;
   int* status;
 };
 
@@ -89,9 +89,10 @@ __global__ void __launch_bounds__(256) latent_store_kernel(const LatentStorePara
   const float pos = static_cast<float>(p.pos[t]);
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     const float2 a = latent_angle(pos, p.freq[i]);
-    const float u = ldf<T>(ckv + p.rank + i), v = ldf<T>(ckv + p.rank + half + i);
-    stf<T>(dst + p.rank + i, u * a.x - v * a.y);
-    stf<T>(dst + p.rank + half + i, v * a.x + u * a.y);
+    const int iu = p.rank + (p.interleaved ? 2 * i : i), iv = p.interleaved ? iu + 1 : iu + half;
+    const float u = ldf<T>(ckv + iu), v = ldf<T>(ckv + iv);
+    stf<T>(dst + iu, u * a.x - v * a.y);
+    stf<T>(dst + iv, v * a.x + u * a.y);
   }
 }
 
@@ -104,7 +105,7 @@ struct LatentRotateParams {
   int heads, dim, rot, out_step;
 };
 
-template <typename T, int V>
+template <typename T, int V, bool PAIRS>
 __global__ void __launch_bounds__(256) latent_rotate_kernel(const LatentRotateParams p) {
   ptx::griddep_launch_dependents();
   ptx::griddep_wait();
@@ -119,8 +120,30 @@ __global__ void __launch_bounds__(256) latent_rotate_kernel(const LatentRotatePa
   __syncthreads();
   for (int it = threadIdx.x; it < p.heads * vec; it += blockDim.x) {
     const int h = it / vec, i = (it - h * vec) * V;
-    const T* src = reinterpret_cast<const T*>(p.q) + t * p.row + static_cast<int64_t>(h) * (p.dim + p.rot) + p.dim + i;
-    T* dst = reinterpret_cast<T*>(p.out) + t * p.out_row + static_cast<int64_t>(h) * p.out_step + i;
+    const T* src = reinterpret_cast<const T*>(p.q) + t * p.row + static_cast<int64_t>(h) * (p.dim + p.rot) + p.dim + (PAIRS ? 2 * i : i);
+    T* dst = reinterpret_cast<T*>(p.out) + t * p.out_row + static_cast<int64_t>(h) * p.out_step + (PAIRS ? 2 * i : i);
+    if constexpr (PAIRS) {
+      float x[2 * V];
+      if constexpr (V == 4) {
+        ldf8<T>(src, x);
+      } else {
+        x[0] = ldf<T>(src);
+        x[1] = ldf<T>(src + 1);
+      }
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        const float cs = s_ang[i + j], sn = s_ang[half + i + j], u = x[2 * j], v = x[2 * j + 1];
+        x[2 * j] = u * cs - v * sn;
+        x[2 * j + 1] = v * cs + u * sn;
+      }
+      if constexpr (V == 4) {
+        stf8<T>(dst, x);
+      } else {
+        stf<T>(dst, x[0]);
+        stf<T>(dst + 1, x[1]);
+      }
+      continue;
+    }
     float u[V], v[V];
     if constexpr (V == 8) {
       ldf8<T>(src, u);
@@ -166,12 +189,12 @@ using namespace blitz;
 
 // cq (q_rank columns, may be null) and ckv (rank + rot columns): column ranges of one projection with row pitch `row`.
 int blitz_latent_store(void* cq, const void* ckv, int64_t row, const void* cq_w, const void* ckv_w, const int32_t* pos, const int32_t* slot,
-                       void* pool, const void* freq, float eps, int num_tokens, int q_rank, int rank, int rot, int page_size,
+                       void* pool, const void* freq, float eps, int num_tokens, int q_rank, int rank, int rot, int interleaved, int page_size,
                        int max_pages, int* status, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (rank <= 0 || rot < 0 || (rot & 1) || (rot > 0 && freq == nullptr) || (cq && (q_rank <= 0 || cq_w == nullptr))) return -1;
   LatentStoreParams p{cq, ckv, row, cq_w, ckv_w, pos, slot, pool, reinterpret_cast<const float2*>(freq), eps,
-                      q_rank, rank, rot, page_size, max_pages, status};
+                      q_rank, rank, rot, interleaved, page_size, max_pages, status};
   const uintptr_t al = dtype == 2 ? 32 : 16;
   bool wide = ((q_rank | rank | rot | row) & 7) == 0;
   for (const void* x : {(const void*)cq, ckv, cq_w, ckv_w, (const void*)pool}) wide = wide && (reinterpret_cast<uintptr_t>(x) % al) == 0;
@@ -189,20 +212,23 @@ int blitz_latent_store(void* cq, const void* ckv, int64_t row, const void* cq_w,
 
 // q: heads of dim + rot columns; head h's rotated part goes to out + h * out_step (its first rotated column).
 int blitz_latent_rotate(const void* q, int64_t row, void* out, int64_t out_row, int out_step, const int32_t* pos, const void* freq,
-                        int num_tokens, int heads, int dim, int rot, int dtype, cudaStream_t stream) {
+                        int num_tokens, int heads, int dim, int rot, int interleaved, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0 || rot == 0) return 0;
   if (heads <= 0 || dim < 0 || rot < 0 || (rot & 1) || rot > 4096 || freq == nullptr) return -1;
   LatentRotateParams p{q, out, row, out_row, pos, reinterpret_cast<const float2*>(freq), heads, dim, rot, out_step};
   const uintptr_t al = dtype == 2 ? 32 : 16;
-  const bool wide = (rot & 15) == 0 && ((dim | row | out_row | out_step) & 7) == 0 && reinterpret_cast<uintptr_t>(q) % al == 0 &&
+  const bool wide = (rot & (interleaved ? 7 : 15)) == 0 && ((dim | row | out_row | out_step) & 7) == 0 && reinterpret_cast<uintptr_t>(q) % al == 0 &&
                     reinterpret_cast<uintptr_t>(out) % al == 0;
-  const int items = heads * (rot / 2) / (wide ? 8 : 1);
+  const int items = heads * (rot / 2) / (wide ? (interleaved ? 4 : 8) : 1);
   const dim3 grid(num_tokens), block(items <= 64 ? 64 : items <= 128 ? 128 : 256);
   const size_t smem = (size_t)rot * sizeof(float);
   auto go = [&](auto type) {
     using T = decltype(type);
-    return wide ? launch_pdl(latent_rotate_kernel<T, 8>, grid, block, smem, stream, p)
-                : launch_pdl(latent_rotate_kernel<T, 1>, grid, block, smem, stream, p);
+    if (interleaved)
+      return wide ? launch_pdl(latent_rotate_kernel<T, 4, true>, grid, block, smem, stream, p)
+                  : launch_pdl(latent_rotate_kernel<T, 1, true>, grid, block, smem, stream, p);
+    return wide ? launch_pdl(latent_rotate_kernel<T, 8, false>, grid, block, smem, stream, p)
+                : launch_pdl(latent_rotate_kernel<T, 1, false>, grid, block, smem, stream, p);
   };
   cudaError_t e = cudaSuccess;
   BLITZ_DISPATCH_DTYPE3(dtype, (e = go(T{})));

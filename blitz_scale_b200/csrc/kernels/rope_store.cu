@@ -3,7 +3,8 @@
 // values of another size than the keys, fp32 or 16-bit activations, and a choice of what the value plane of the cache
 // receives: the value columns of the projection, or the keys as projected, before rotation (models without a value
 // projection).  Biases of the projections are added here, in fp32, before the rotation; `gain` multiplies the rotated
-// dimensions (scaled rotations).  Layers that read another layer's cache pass no keys: only q is rotated.
+// dimensions (scaled rotations).  Layers that read another layer's cache pass no keys: only q is rotated.  NORM: before the
+// rotation the whole row of queries, and that of keys, is divided by its root mean square and multiplied by a weight per column.
 //
 // (elementwise.cu's rope_kv_store is the special case of a fully rotated half-split head with a value projection.)
 //
@@ -27,13 +28,15 @@ struct RopeStoreParams {
   void *k_pool, *v_pool;  // row of token `off` of page n: n * page_rows + off
   const float2* freq;  // [rot_dims / 2] (high, low)
   float gain;
+  const void *q_w, *k_w;  // NORM: [q_heads * dim], [kv_heads * dim]
+  float eps;
   int q_heads, kv_heads, dim, vdim, rot_dims, interleaved, page_size, page_rows, max_pages;
   int* status;
 };
 
 enum RopeMode : int { kRopeAny = 0, kRopeWidePairs = 1, kRopeWideHalves = 2 };  // wide: eight elements per access
 
-template <typename T, int MODE>
+template <typename T, int MODE, bool NORM>
 __global__ void __launch_bounds__(256, MODE == kRopeAny ? 5 : 4) rope_store_kernel(const RopeStoreParams p) {
   ptx::griddep_launch_dependents();
   ptx::griddep_wait();
@@ -54,6 +57,32 @@ __global__ void __launch_bounds__(256, MODE == kRopeAny ? 5 : 4) rope_store_kern
   const T* k = reinterpret_cast<const T*>(p.k) + t * p.row;
   const T *q_b = reinterpret_cast<const T*>(p.q_b), *k_b = reinterpret_cast<const T*>(p.k_b), *v_b = reinterpret_cast<const T*>(p.v_b);
   const int heads = p.q_heads + (s >= 0 ? p.kv_heads : 0);
+  const T *q_w = reinterpret_cast<const T*>(p.q_w), *k_w = reinterpret_cast<const T*>(p.k_w);
+  float q_f = 1.f, k_f = 1.f;
+  if (NORM) {
+    __shared__ float red[2][33];
+    auto squares = [&](const T* x, int n) {
+      float ss = 0.f;
+      if (MODE != kRopeAny) {
+        for (int i = threadIdx.x * 8; i < n; i += blockDim.x * 8) {
+          float v[8];
+          ldf8<T>(x + i, v);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) ss += v[j] * v[j];
+        }
+      } else {
+        for (int i = threadIdx.x; i < n; i += blockDim.x) {
+          const float v = ldf<T>(x + i);
+          ss += v * v;
+        }
+      }
+      return ss;
+    };
+    const int nq = p.q_heads * p.dim, nk = p.k ? p.kv_heads * p.dim : 0;
+    const float sq = squares(q, nq), sk = squares(k, nk);
+    q_f = rsqrtf(block_sum(sq, red[0]) / static_cast<float>(nq) + p.eps);
+    if (p.k) k_f = rsqrtf(block_sum(sk, red[1]) / static_cast<float>(nk) + p.eps);
+  }
   auto angles = [&]() {
     const float pos = static_cast<float>(p.pos[t]);
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
@@ -78,6 +107,14 @@ __global__ void __launch_bounds__(256, MODE == kRopeAny ? 5 : 4) rope_store_kern
 #pragma unroll
         for (int j = 0; j < 8; ++j) x[j] += b[j];
       }
+      if (NORM && src != p.v) {
+        const bool is_q = src == q;
+        float w[8];
+        ldf8<T>((is_q ? q_w : k_w) + at, w);
+        const float f = is_q ? q_f : k_f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[j] *= f * w[j];
+      }
     };
     if (MODE == kRopeWidePairs) {
       // eight elements (four pairs) per access; dimensions that pass unchanged ride along
@@ -85,7 +122,7 @@ __global__ void __launch_bounds__(256, MODE == kRopeAny ? 5 : 4) rope_store_kern
       for (int it = threadIdx.x; it < heads * vec; it += blockDim.x) {
         const int head = it / vec, d0 = (it - head * vec) * 8;
         const bool is_q = head < p.q_heads;
-        if (is_q && d0 >= p.rot_dims && !q_b) continue;
+        if (is_q && d0 >= p.rot_dims && !q_b && !NORM) continue;
         const int64_t at = static_cast<int64_t>(is_q ? head : head - p.q_heads) * p.dim + d0;
         float x[8], y[8];
         load8(is_q ? q : k, is_q ? q_b : k_b, at, x);
@@ -116,7 +153,7 @@ __global__ void __launch_bounds__(256, MODE == kRopeAny ? 5 : 4) rope_store_kern
         m.c = it - head * vec;
         m.is_q = head < p.q_heads;
         m.base = static_cast<int64_t>(m.is_q ? head : head - p.q_heads) * p.dim;
-        m.on = it < items && !(m.is_q && m.c >= turns && !q_b);
+        m.on = it < items && !(m.is_q && m.c >= turns && !q_b && !NORM);
         return m;
       };
       auto first = [&](const Item& m) { return m.base + (m.c < turns ? m.c * 8 : p.rot_dims + (m.c - turns) * 8); };
@@ -156,7 +193,13 @@ __global__ void __launch_bounds__(256, MODE == kRopeAny ? 5 : 4) rope_store_kern
       const T* v = reinterpret_cast<const T*>(p.v) + t * p.row;
       for (int i = threadIdx.x * 8; i < vrow; i += blockDim.x * 8) {
         float x[8];
-        load8(v, v_b, i, x);
+        ldf8<T>(v + i, x);
+        if (v_b) {
+          float b[8];
+          ldf8<T>(v_b + i, b);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) x[j] += b[j];
+        }
         stf8<T>(vdst + i, x);
       }
     }
@@ -184,6 +227,12 @@ __global__ void __launch_bounds__(256, MODE == kRopeAny ? 5 : 4) rope_store_kern
       u += ldf<T>(bias + base + iu);
       v += ldf<T>(bias + base + iv);
     }
+    if (NORM) {
+      const T* w = (is_q ? q_w : k_w) + base;
+      const float f = is_q ? q_f : k_f;
+      u *= f * ldf<T>(w + iu);
+      v *= f * ldf<T>(w + iv);
+    }
     const float ru = u * cs - v * sn, rv = v * cs + u * sn;
     if (vec) {
       stf2<T>(dst + iu, ru, rv);
@@ -204,10 +253,11 @@ __global__ void __launch_bounds__(256, MODE == kRopeAny ? 5 : 4) rope_store_kern
   for (int it = threadIdx.x; it < heads * rest; it += blockDim.x) {
     const int head = it / rest;
     const bool is_q = head < p.q_heads;
-    if (is_q && !q_b) continue;
+    if (is_q && !q_b && !NORM) continue;
     const int64_t at = static_cast<int64_t>(is_q ? head : head - p.q_heads) * p.dim + p.rot_dims + it % rest;
     const T* bias = is_q ? q_b : k_b;
-    const float x = ldf<T>((is_q ? q : k) + at) + (bias ? ldf<T>(bias + at) : 0.f);
+    float x = ldf<T>((is_q ? q : k) + at) + (bias ? ldf<T>(bias + at) : 0.f);
+    if (NORM) x *= (is_q ? q_f : k_f) * ldf<T>((is_q ? q_w : k_w) + at);
     stf<T>((is_q ? q : kdst) + at, x);
     if (!is_q && p.v == nullptr) stf<T>(vdst + at, x);
   }
@@ -223,30 +273,33 @@ extern "C" {
 using namespace blitz;
 
 // Pools: [max_pages][page_rows][heads][size]; a page's `page_size` token rows are its first ones (with one tensor for keys
-// and values page_rows is 2 page_size and v_pool points at the first value plane).
+// and values page_rows is 2 page_size and v_pool points at the first value plane).  q_w, k_w: weights of the norms over whole rows, or null.
 int blitz_rope_store(void* q, const void* k, const void* v, const void* q_b, const void* k_b, const void* v_b, int64_t row,
+                     const void* q_w, const void* k_w, float eps,
                      const int32_t* pos, const int32_t* slot, void* k_pool, void* v_pool, const void* freq, float gain,
                      int num_tokens, int q_heads, int kv_heads, int dim, int vdim, int rot_dims, int interleaved, int page_size,
                      int page_rows, int max_pages, int* status, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (rot_dims < 0 || (rot_dims & 1) || rot_dims > dim || rot_dims > 4096 || (rot_dims > 0 && freq == nullptr)) return -1;
   if (k != nullptr && v == nullptr && vdim != dim) return -1;
-  RopeStoreParams p{q, k, v, q_b, k_b, v_b, row, pos, slot, k_pool, v_pool, reinterpret_cast<const float2*>(freq), gain, q_heads,
+  if (q_w != nullptr && (q_b || k_b || (k && (k_w == nullptr || v == nullptr)))) return -1;
+  RopeStoreParams p{q, k, v, q_b, k_b, v_b, row, pos, slot, k_pool, v_pool, reinterpret_cast<const float2*>(freq), gain, q_w, k_w, eps, q_heads,
                     kv_heads, dim, vdim, rot_dims, interleaved, page_size, page_rows, max_pages, status};
   const uintptr_t al = dtype == 2 ? 32 : 16;
   bool wide = ((dim | vdim | row) & 7) == 0 && (interleaved || (rot_dims & 15) == 0);
-  for (const void* x : {(const void*)q, k, v, q_b, k_b, v_b, (const void*)k_pool, (const void*)v_pool})
+  for (const void* x : {(const void*)q, k, v, q_b, k_b, v_b, q_w, k_w, (const void*)k_pool, (const void*)v_pool})
     wide = wide && (reinterpret_cast<uintptr_t>(x) % al) == 0;
   const dim3 grid(num_tokens), block(wide && (q_heads + kv_heads) * dim <= 2048 ? 128 : 256);
   const size_t smem = (size_t)rot_dims * sizeof(float);
-  auto go = [&](auto type) {
+  auto go = [&](auto type, auto norm) {
     using T = decltype(type);
-    if (!wide) return launch_pdl(rope_store_kernel<T, kRopeAny>, grid, block, smem, stream, p);
-    return interleaved ? launch_pdl(rope_store_kernel<T, kRopeWidePairs>, grid, block, smem, stream, p)
-                       : launch_pdl(rope_store_kernel<T, kRopeWideHalves>, grid, block, smem, stream, p);
+    constexpr bool N = decltype(norm)::value;
+    if (!wide) return launch_pdl(rope_store_kernel<T, kRopeAny, N>, grid, block, smem, stream, p);
+    return interleaved ? launch_pdl(rope_store_kernel<T, kRopeWidePairs, N>, grid, block, smem, stream, p)
+                       : launch_pdl(rope_store_kernel<T, kRopeWideHalves, N>, grid, block, smem, stream, p);
   };
   cudaError_t e = cudaSuccess;
-  BLITZ_DISPATCH_DTYPE3(dtype, (e = go(T{})));
+  BLITZ_DISPATCH_DTYPE3(dtype, (e = q_w ? go(T{}, std::true_type{}) : go(T{}, std::false_type{})));
   return (int)e;
 }
 

@@ -85,7 +85,7 @@ REGISTRY: Dict[str, ModelConfig] = {c.name: c for c in [
 
 def hybrid_registry():
     """Shapes of the models whose layers differ (a separate table: the native twin of the registry holds the uniform ones)."""
-    from . import komulorn, vofidra
+    from . import komulorn, norusun, vofidra
     from .fafudra import shape_config
     mixed = ("gla", "attention", "rglru", "gla")
     return {c.name: c for c in [
@@ -114,11 +114,24 @@ def hybrid_registry():
         vofidra.shape_config("vofidra_13b", 128256, 2048, 28, heads=16, kv_heads=4, dim=128, latent=dict(heads=32, dim=64, rot_dim=32,
                              vdim=64, q_rank=768, kv_rank=256), experts=48, identity=16, top=6, groups=8, keep=4, ff=1536,
                              dense_ff=8192, streams=4, gb=26),
+        # several residual streams with scalar norms and convolved mixer inputs; linear attention with a token shift, latent
+        # attention in a window, attention without softmax beside a state space: likewise, the last one of 8 B parameters
+        norusun.shape_config("norusun_tiny", 2048, 320, ("wkv", "latent_attention", "parallel", "wkv"), 512, wkv=(5, 64, 24),
+                             latent=dict(heads=4, dim=64, rot_dim=32, vdim=64, q_rank=192, kv_rank=128, window=70), heads=8, kv_heads=2,
+                             dim=64, chunk=96, ssd=dict(heads=6, vdim=64, state=64, groups=2, taps=4, norm_groups=3), streams=2, taps=4),
+        norusun.shape_config("norusun_odd", 1003, 122, ("parallel", "wkv", "latent_attention"), 77, wkv=(3, 13, 5),
+                             latent=dict(heads=3, dim=13, rot_dim=6, vdim=11, q_rank=35, kv_rank=21, window=19), heads=6, kv_heads=3,
+                             dim=22, vdim=17, rot_dims=10, chunk=23, ssd=dict(heads=5, vdim=7, state=9, groups=1, taps=3, norm_groups=5),
+                             streams=3, taps=2),
+        norusun.shape_config("norusun_8b", 128256, 4096, ("wkv", "latent_attention", "parallel", "latent_attention") * 8, 14336, wkv=(32, 128, 64),
+                             latent=dict(heads=32, dim=96, rot_dim=32, vdim=128, q_rank=1024, kv_rank=512, window=2048), heads=32,
+                             kv_heads=8, dim=128, chunk=2048,
+                             ssd=dict(heads=64, vdim=64, state=128, groups=8, taps=4, norm_groups=8), streams=2, taps=4, gb=16),
     ]}
 
 
 # designs described by data: "architecture" of config.json -> module of this package with parse_config and to_segment
-DESIGNS = {"Fafudra": "fafudra", "Komulorn": "komulorn", "Vofidra": "vofidra"}
+DESIGNS = {"Fafudra": "fafudra", "Komulorn": "komulorn", "Vofidra": "vofidra", "Norusun": "norusun"}
 
 
 def design_module(name: str):

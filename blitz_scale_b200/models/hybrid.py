@@ -20,6 +20,9 @@ sublayer before it, joins them and norms the result::
     stream_mix -> GEMM (in) -> mixer -> GEMM (out)
     -> stream_mix -> GEMM (gate||up, SiLU*mul) -> GEMM (down)     or router, moe_route and the grouped products as above
 
+With RMS norms that kernel is stream_rms.  Mixers may read their input plus a causal convolution of it (and the mixes of a token
+shift): stream_rms does that too where every row is one token, token_conv behind it where there are longer rows.
+
     attention: rope_store (biases, rotation, paged write) or norm_store (norm of every head, paged write)
                -> attention over the pages (window, cap, sink, gate per head, bias by distance)
     latent:    latent_store (norms, shared rotated key, paged write) -> GEMM (queries), then
@@ -29,6 +32,11 @@ sublayer before it, joins them and norms the result::
                (heads that the prompt kernel does not take: as single tokens)
     gla:       one kernel (decay projection, recurrence, output norm, gate), or the chunked kernels for prompts
     rglru:     conv_causal -> block-diagonal GEMM (gates, fp32 out) -> rglru_scan
+    wkv:       one block-diagonal GEMM over the mixes (receptance, keys, values, gates), GEMM (decay, fp32 out) -> recurrence with
+               output norm and gate, or the chunked kernels for prompts
+    parallel:  attention as above (norm over whole rows with the rotation; chunks, sigmoid weights), and
+               token_conv (SiLU) -> state-space recurrence with gate, or the chunked kernel for prompts -> norm in parts;
+               an output product each, side by side: the next stream_rms norms and adds them
 
 A step may hold rows of any length (StepMeta.singles of one token first): single tokens go to the decode kernels, the
 others to the prefill kernels, everything else runs over all tokens at once.
@@ -41,7 +49,8 @@ import torch
 
 from .. import ops
 from ..runtime.hybrid_cache import HybridCache
-from .hybrid_config import AttentionMixer, ExpertsSpec, GLAMixer, HybridConfig, LatentAttentionMixer, LayerSpec, RGLRUMixer
+from .hybrid_config import (AttentionMixer, ExpertsSpec, GLAMixer, HybridConfig, LatentAttentionMixer, LayerSpec, ParallelMixer, RGLRUMixer,
+                            SSDMixer, WKVMixer)
 from .llama import StepMeta
 from .weights import WeightSegment
 
@@ -67,19 +76,21 @@ class HybridRunner:
             if key not in self._mid:
                 self._mid[key] = torch.zeros(max_tokens, s.out_rows, dtype=dt, device=dev)
         rw = max((m.width for m in cfg.run_mixers() if m.kind == "rglru"), default=0)
-        self._conv = torch.empty(max_tokens * rw, dtype=dt, device=dev) if rw else None
+        cw = max([rw] + [m.channels for m in cfg.run_parts() if m.kind == "ssd"])
+        self._conv = torch.empty(max_tokens * cw, dtype=dt, device=dev) if cw else None
         self._gates = torch.empty(max_tokens * 2 * rw, dtype=torch.float32, device=dev) if rw else None
-        ck = max((m.heads * m.dim for m in cfg.run_mixers() if m.kind == "gla"), default=0)
+        ck = max((m.heads * m.dim for m in cfg.run_mixers() if m.kind in ("gla", "wkv")), default=0)
         self._cum = torch.empty(max_tokens * ck, dtype=torch.float32, device=dev) if ck and dt == torch.bfloat16 else None
         self._init_experts(max_tokens, dev, dt)
         self._init_streams(max_tokens, max_batch, dev, dt)
         self._init_latent(max_tokens, max_batch, dev, dt)
+        self._init_shift(max_tokens, max_batch, dev, dt)
         self.last = torch.empty(max_batch, H, dtype=torch.float32, device=dev)
         self._logits_pad = torch.zeros(max_batch, cfg.vocab_pad, dtype=torch.float32, device=dev)
         self.logits = self._logits_pad[:, :cfg.vocab]
         self.tokens = torch.empty(max_batch, dtype=torch.int32, device=dev)
         self._freqs = {}
-        for m in cfg.run_mixers():
+        for m in cfg.run_parts():
             if m.kind == "attention" and self._rot_key(m) not in self._freqs:
                 stretch = m.yarn.stretch(m.rot_dims, m.rot_base) if m.yarn else None
                 self._freqs[self._rot_key(m)] = ops.rope_freqs(m.rot_dims, m.rot_base, dev, stretch)
@@ -127,7 +138,8 @@ class HybridRunner:
         self._ids: Optional[torch.Tensor] = None
         if not c.streams:
             return
-        self._y = torch.empty(max_tokens, c.hidden, dtype=dt, device=dev)
+        pair = any(m.kind == "parallel" for m in c.run_mixers())
+        self._y = torch.empty(max_tokens * (2 if pair else 1), c.hidden, dtype=dt, device=dev)
         self._head_in = torch.empty(max_batch, c.hidden, dtype=dt, device=dev)
         ff = max(s.ff_after_pad for s in c.layer_specs)
         self._ff = torch.empty(max_tokens * ff, dtype=dt, device=dev) if ff else None
@@ -144,6 +156,20 @@ class HybridRunner:
         self._q = torch.empty(max_tokens * max(m.heads * m.qdim for m in ms), dtype=dt, device=dev)
         self._q_latent = torch.empty(max(rows(m) * m.heads * m.width for m in ms), dtype=dt, device=dev)
         self._o_latent = torch.empty(max(rows(m) * m.heads * m.kv_rank for m in ms), dtype=dt, device=dev)
+
+    def _init_shift(self, max_tokens: int, max_batch: int, dev, dt) -> None:
+        """Buffers of convolved mixer inputs, token shifts and mixers side by side."""
+        c = self.cfg
+        wkv = [m for m in c.run_mixers() if m.kind == "wkv"]
+        mixes = max([1 if c.mix_taps else 0] + [len(m.MIXES) for m in wkv])
+        self._mixed = torch.empty(max_tokens * mixes * c.hidden, dtype=dt, device=dev) if mixes else None
+        if wkv:
+            self._last_h = torch.empty(max_batch, c.hidden, dtype=dt, device=dev)
+            self._rkvg = torch.empty(max_tokens * 4 * max(m.out_width for m in wkv), dtype=dt, device=dev)
+            self._low = torch.empty(max_tokens * max(m.rank + 7 for m in wkv), dtype=torch.float32, device=dev)
+        # (padding columns stay zero because nothing ever writes them)
+        self._mid_right = {m.right.out_width: torch.zeros(max_tokens, m.right_rows, dtype=dt, device=dev)
+                           for m in c.run_mixers() if m.kind == "parallel"}
 
     def _expands(self, m: LatentAttentionMixer, dt) -> bool:
         """Whether prompts run over expanded keys and values on the tensor cores (else over the latent rows)."""
@@ -182,16 +208,35 @@ class HybridRunner:
             out, plan = self._experts(l, spec.moe, h)
             self._pending = (out, plan.place)
 
-    def _norm(self, name: str) -> tuple:
-        return self.seg[name], self.seg[name + "_alpha"], self.seg[name + "_b"]
+    def _streams(self, norm: Optional[str] = None, **what) -> None:
+        """The streams take up what is pending (``write``: and keep it) and are joined; ``norm``: name of the norm of ``out``."""
+        what.update(self._embeddings(), pending=self._pending)
+        if self.cfg.norm == "tanh":
+            weights = dict(norm=(self.seg[norm], self.seg[norm + "_alpha"], self.seg[norm + "_b"])) if norm else {}
+            ops.stream_mix(self.res, **what, **weights)
+        else:
+            ops.stream_rms(self.res, eps=self.cfg.rms_eps, w=self.seg[norm] if norm else None, w_offset=self.cfg.norm_offset, **what)
 
-    def _join(self, l: int, q: int, T: int) -> torch.Tensor:
+    def _join(self, l: int, q: int, T: int, **more) -> torch.Tensor:
         """Input of sublayer q of layer l; the streams take up what is pending."""
-        take, h = self._pending is not None, self.normed[:T]
-        ops.stream_mix(self.res[:T], **self._embeddings(), pending=self._pending, read=self._w(l, f"hc{q}_in"),
-                       norm=self._norm(f"layers.{l}.norm{q}"), out=h, write=take)
+        take, h = self._pending is not None, more.pop("out", self.normed[:T])
+        self._streams(f"layers.{l}.norm{q}", n=T, read=self._w(l, f"hc{q}_in"), out=h, write=take, **more)
         self._fresh = self._fresh and not take
         return h
+
+    def _join_convolved(self, r: int, l: int, mx, m: StepMeta) -> torch.Tensor:
+        """Input of the mixer of layer l: the norm's output plus its causal convolution, or with a token shift its mixes [T, mixes *
+        hidden]."""
+        T, H, rc = m.num_tokens, self.cfg.hidden, self.cache.runs[r]
+        mu = self._w(l, "mu") if mx.kind == "wkv" else None
+        width = H * (mu.shape[0] if mu is not None else 1)
+        out = self._mixed[:T * width].view(T, width)
+        conv = self._w(l, "mix_conv")
+        if not m.is_prefill:
+            return self._join(l, 1, T, out=out, tokens=ops.TokenState(conv, rc.mix_hist, mu, rc.shift), pos=m.pos, seq_slot=m.seq_slot)
+        h = self._join(l, 1, T)
+        shift = dict(mu=mu, shift=rc.shift, last=self._last_h) if mu is not None else {}
+        return ops.token_conv(h, conv, rc.mix_hist, out, m.pos, m.tok_indptr, m.seq_slot, residual=True, **shift)
 
     def _embeddings(self) -> dict:
         return dict(ids=self._ids, embed=self.seg["embed"]) if self._fresh else {}
@@ -200,23 +245,34 @@ class HybridRunner:
         self._pending = ops.Pending(y, self._w(l, f"hc{q}_mix"), self._w(l, f"hc{q}_out"), **rows)
 
     def _run_layer_streams(self, r: int, l: int, spec: LayerSpec, m: StepMeta) -> None:
-        T = m.num_tokens
+        T, c = m.num_tokens, self.cfg
         if r == 0:
             self._pending, self._fresh, self._ids = None, True, m.ids
-        h, y = self._join(l, 1, T), self._y[:T]
+        h, y = self._join_convolved(r, l, spec.mixer, m) if c.mix_taps else self._join(l, 1, T), self._y[:T]
         cols, width = spec.in_columns()
-        proj = self._proj[:T * width].view(T, width)
-        ops.gemm(h, self._w(l, "in"), out=proj, static_b=True)
         mid = self._mid[self._mid_key(spec)][:T]
-        getattr(self, "_" + spec.mixer.kind)(r, l, spec.mixer, {n: proj[:, at:at + w] for n, (at, w) in cols.items()}, mid, m)
-        ops.gemm(mid, self._w(l, "out"), out=y, static_b=True)
-        self._leave(l, 1, y)
+        if spec.mixer.kind == "wkv":                 # its projections have an input each
+            self._wkv(r, l, spec.mixer, h, mid, m)
+        else:
+            proj = self._proj[:T * width].view(T, width)
+            ops.gemm(h, self._w(l, "in"), out=proj, static_b=True)
+            getattr(self, "_" + spec.mixer.kind)(r, l, spec.mixer, {n: proj[:, at:at + w] for n, (at, w) in cols.items()}, mid, m)
+        if spec.mixer.kind == "parallel":
+            both, H = self._y[:2 * T].view(T, 2 * c.hidden), c.hidden
+            ops.gemm(mid, self._w(l, "out"), out=both[:, :H], static_b=True)
+            ops.gemm(self._mid_right[spec.mixer.right.out_width][:T], self._w(l, "r_out"), out=both[:, H:], static_b=True)
+            self._leave(l, 1, both, norms=(self._w(l, "l_out_norm"), self._w(l, "r_out_norm")))
+        else:
+            ops.gemm(mid, self._w(l, "out"), out=y, static_b=True)
+            self._leave(l, 1, y)
         if spec.ff_after:
             h = self._join(l, 2, T)
             act = self._ff[:T * spec.ff_after_pad].view(T, spec.ff_after_pad)
-            ops.gemm(h, self._w(l, "gate_up"), out=act, epilogue="silu_mul", static_b=True)
+            unit = (dict(epilogue="clamp_glu", alpha=spec.unit.limit, beta=spec.unit.beta, bias=self._w(l, "gate_up_b")) if spec.unit
+                    else dict(epilogue="silu_mul"))
+            ops.gemm(h, self._w(l, "gate_up"), out=act, static_b=True, **unit)
             ops.gemm(act, self._w(l, "down"), out=y, static_b=True)
-            self._leave(l, 2, y)
+            self._leave(l, 2, y, **(dict(bias=self._w(l, "down_b")) if spec.unit else {}))
         elif spec.moe:
             h = self._join(l, 2, T)
             out, plan = self._experts(l, spec.moe, h)
@@ -251,19 +307,23 @@ class HybridRunner:
         ops.gemm_grouped(act, down, plan, out, shared=s_down)
         return out, plan
 
-    def _attention(self, r: int, l: int, mx: AttentionMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta) -> None:
+    def _attention(self, r: int, l: int, mx: AttentionMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta,
+                   prefix: str = "") -> None:
         T, kv = m.num_tokens, self.cache.runs[r].kv
+        w = lambda n: self._w(l, prefix + n)
         if mx.qk_norm:
             temp = dict(temp_coef=mx.q_temp.coef, temp_every=mx.q_temp.every) if mx.q_temp else {}
-            ops.norm_store(p["q"], p["k"], p["v"], m.pos, m.slot, kv, self._w(l, "q_norm"), self._w(l, "k_norm"), q_heads=mx.heads,
+            ops.norm_store(p["q"], p["k"], p["v"], m.pos, m.slot, kv, w("q_norm"), w("k_norm"), q_heads=mx.heads,
                            kv_heads=mx.kv_heads, dim=mx.dim, page_size=self.page_size, eps=self.cfg.rms_eps, **temp)
         else:
-            biases = {n + "_b": self._w(l, n + "_b") for n in ("q", "k", "v") if mx.bias and n in p}
+            biases = {n + "_b": w(n + "_b") for n in ("q", "k", "v") if mx.bias and n in p}
+            if mx.whole_norm:
+                biases = dict(q_w=w("q_norm"), k_w=w("k_norm"), eps=self.cfg.rms_eps)
             ops.rope_store(p["q"], p.get("k"), p.get("v"), m.pos, m.slot, kv, self._freqs[self._rot_key(mx)], q_heads=mx.heads,
                            kv_heads=mx.kv_heads, dim=mx.dim, rot_dims=mx.rot_dims, page_size=self.page_size,
                            interleaved=mx.interleaved, gain=mx.yarn.gain if mx.yarn else 1.0, **biases)
-        extra = dict(window=mx.window, keep_first=mx.keep_first, softcap=mx.softcap, sink=self._w(l, "sink") if mx.sink else None,
-                     bias=self._w(l, "rel_by_distance") if mx.rel else None)
+        extra = dict(window=mx.window, keep_first=mx.keep_first, softcap=mx.softcap, sink=w("sink") if mx.sink else None,
+                     bias=w("rel_by_distance") if mx.rel else w("weight_b") if mx.sigmoid else None, chunked=mx.chunked, sigmoid=mx.sigmoid)
         gate = p.get("g")
         if not ops.attn_tensor_core(p["q"], mx.heads, mx.kv_heads, mx.dim, self.page_size, mx.vdim):
             ops.attn_ragged(p["q"], kv, m.pos, m.tok_indptr if m.is_prefill else None, m.page_indptr, m.page_indices, mid,
@@ -291,10 +351,12 @@ class HybridRunner:
     def _latent(self, r: int, l: int, mx: LatentAttentionMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta) -> None:
         T, H, R, W, kv = m.num_tokens, mx.heads, mx.kv_rank, mx.width, self.cache.runs[r].kv
         freqs, gate = self._freqs[(mx.rot_dim, mx.rot_base, None)], p.get("g")
-        ops.latent_store(p["dq"], p["dkv"], m.pos, m.slot, kv, self._w(l, "dq_norm"), self._w(l, "dkv_norm"), freqs, eps=self.cfg.rms_eps)
+        ops.latent_store(p["dq"], p["dkv"], m.pos, m.slot, kv, self._w(l, "dq_norm"), self._w(l, "dkv_norm"), freqs, eps=self.cfg.rms_eps,
+                         interleaved=mx.interleaved)
         q = self._q[:T * H * mx.qdim].view(T, H * mx.qdim)
         ops.gemm(p["dq"], self._w(l, "uq"), out=q, static_b=True)
-        rotate = dict(heads=H, dim=mx.dim, rot=mx.rot_dim)
+        rotate = dict(heads=H, dim=mx.dim, rot=mx.rot_dim, interleaved=mx.interleaved)
+        extra = dict(window=mx.window, sink=self._w(l, "sink") if mx.sink else None)
         n = m.batch if not m.is_prefill else m.singles if self._expands(mx, q.dtype) else T    # rows that go through the latent space
         if n:
             ql, ol = self._q_latent[:n * H * W].view(n, H * W), self._o_latent[:n * H * R].view(n, H * R)
@@ -305,28 +367,24 @@ class HybridRunner:
             if ops.attn_latent_supported(ql, n if single else min(n, ops.ATTN_LATENT_ROWS), H, kv):
                 rows = m.batch if not single else n
                 ops.attn_latent(ql, kv, m.page_indices, m.page_indptr[:rows + 1], m.last_page_len[:rows], heads=H, scale=mx.scale,
-                                workspace=self._latent_ws, out=ol, gate=g, static_table=True,
+                                workspace=self._latent_ws, out=ol, gate=g, static_table=True, **extra,
                                 **({} if single else dict(pos=m.pos[:n], tok_indptr=m.tok_indptr)))
             else:
                 ops.attn_ragged(ql, kv, m.pos, None if single else m.tok_indptr, m.page_indptr[:n + 1] if single else m.page_indptr,
-                                m.page_indices, ol, q_heads=H, kv_heads=1, dim=W, page_size=self.page_size, scale=mx.scale, gate=g)
+                                m.page_indices, ol, q_heads=H, kv_heads=1, dim=W, page_size=self.page_size, scale=mx.scale, gate=g, **extra)
             # few rows: a tile per head is enough, and an exchange of K splits would cost more than it saves
             narrow = dict(bn=64, split_k=1) if n <= ops.PAIR_GEMM_MAX_M else {}
             ops.gemm(ol, self._w(l, "uv"), out=mid[:n, :H * mx.vdim], groups=H, a_step=R, out_step=mx.vdim, static_b=True, **narrow)
         if n < T:
-            self._latent_prompts(l, mx, q, gate, kv, mid, m, n, freqs, rotate)
+            self._latent_prompts(l, mx, q, gate, kv, mid, m, n, freqs, rotate, extra)
 
-    def _latent_prompts(self, l: int, mx: LatentAttentionMixer, q, gate, kv: ops.LatentKV, mid, m: StepMeta, n: int, freqs, rotate) -> None:
+    def _latent_prompts(self, l: int, mx: LatentAttentionMixer, q, gate, kv: ops.LatentKV, mid, m: StepMeta, n: int, freqs, rotate, extra) -> None:
         """Rows from n on: keys and values of all their sequences' cached rows are expanded into a pool of their own, some heads
-        at a time where that would be large."""
+        at a time where that would be large.  With a window only the pages that one of a sequence's rows sees."""
         ops.latent_rotate(q[n:], q[n:, mx.dim:], m.pos[n:], freqs, out_step=mx.qdim, **rotate)
         ps = self.page_size
-        pages = [-(-kv_len // ps) for kv_len in m.kv_lens_host]
-        first, total = sum(pages[:n]), sum(pages)
-        np_ = total - first
-        # page i of the expanded pool is the i-th page of these sequences
-        index = torch.arange(-first, np_, dtype=torch.int32, device=q.device)
-        rows = ops.latent_gather(kv, m.page_indices[first:total], self._room("rows", (np_ * ps, mx.width), q.dtype))
+        index, pages, np_ = self._expanded_pages(m, n, mx.window, q.device)
+        rows = ops.latent_gather(kv, pages, self._room("rows", (np_ * ps, mx.width), q.dtype))
         H = mx.heads
         heads = max(1, min(H, self.EXPANDED_BYTES // (np_ * ps * (mx.qdim + mx.vdim) * 2)))
         for h0 in range(0, H, heads):
@@ -337,8 +395,32 @@ class HybridRunner:
             ops.gemm(rows[:, :mx.kv_rank], self._w(l, "v_up")[:, h0 * mx.vdim:(h0 + hn) * mx.vdim], out=v.view(np_ * ps, -1), static_b=True)
             ops.attn_prefill_paged(q[:, h0 * mx.qdim:(h0 + hn) * mx.qdim], ops.KVPair(k, v), index, m.prefill_work, q_heads=hn, kv_heads=hn,
                                    head_dim=mx.qdim, page_size=ps, sm_scale=mx.scale, out=mid[:, h0 * mx.vdim:(h0 + hn) * mx.vdim],
-                                   gate=gate[:, h0:h0 + hn] if gate is not None else None)
+                                   gate=gate[:, h0:h0 + hn] if gate is not None else None, window=extra["window"],
+                                   sink=extra["sink"][h0:h0 + hn] if extra["sink"] is not None else None)
 
+    def _expanded_pages(self, m: StepMeta, n: int, window: int, dev) -> tuple:
+        """For the sequences from n on: where their page entries are in the expanded pool, the pages it holds, and how many."""
+        ps = self.page_size
+        pages = [-(-kv_len // ps) for kv_len in m.kv_lens_host]
+        first, total = sum(pages[:n]), sum(pages)
+        if not window:       # page i of the expanded pool is the i-th page of these sequences
+            return torch.arange(-first, total - first, dtype=torch.int32, device=dev), m.page_indices[first:total], total - first
+        key = (n, window)
+        if self._expanded is None or self._expanded[0] is not m or key not in self._expanded[1]:
+            index, need, at = [0] * first, [], first
+            for s in range(n, len(pages)):
+                # (the attention kernel walks whole blocks of keys)
+                lo = max(0, m.kv_lens_host[s] - m.seq_lens_host[s] - window + 1) // ops.PREFILL_KEY_BLOCK * ops.PREFILL_KEY_BLOCK // ps
+                index += [0] * lo + list(range(len(need), len(need) + pages[s] - lo))
+                need += range(at + lo, at + pages[s])
+                at += pages[s]
+            both = torch.tensor(index + need, dtype=torch.int32).to(dev, non_blocking=True)
+            if self._expanded is None or self._expanded[0] is not m:
+                self._expanded = (m, {})
+            self._expanded[1][key] = (both[:len(index)], m.page_indices.index_select(0, both[len(index):]), len(need))
+        return self._expanded[1][key]
+
+    _expanded: Optional[tuple] = None       # (step, tables) of the last prefill pass
     EXPANDED_BYTES = 1 << 30      # of expanded keys and values at a time
 
     def _room(self, name: str, shape: tuple, dt) -> torch.Tensor:
@@ -373,6 +455,51 @@ class HybridRunner:
         ops.rglru_scan(u, gates, self._w(l, "gate_b"), self._w(l, "lam"), p["y"], p["x"], self._w(l, "y_b"), rc.state, rc.hist,
                        mid, m.pos, indptr, m.seq_slot, block=mx.block)
 
+    def _wkv(self, r: int, l: int, mx: WKVMixer, h: torch.Tensor, mid: torch.Tensor, m: StepMeta) -> None:
+        """h: the mixes, [T, 5 * hidden]."""
+        T, H, N, rc = m.num_tokens, self.cfg.hidden, mx.out_width, self.cache.runs[r]
+        out = self._rkvg[:T * 4 * N].view(T, 4 * N)
+        w = self._w(l, "rkvg")
+        if T <= ops.PAIR_GEMM_MAX_M and N % 8 == 0 and H * N >= self.SEPARATE_WEIGHTS:
+            for i in range(4):                       # large weights, few rows: the weight-streaming products
+                ops.gemm(h[:, i * H:(i + 1) * H], w[i * H:(i + 1) * H], out=out[:, i * N:(i + 1) * N], static_b=True)
+        else:
+            ops.gemm(h[:, :4 * H], w, out=out, groups=4, static_b=True)
+        w1 = self._w(l, "w1")
+        low = self._low[:T * w1.shape[1]].view(T, w1.shape[1])
+        narrow = dict(bn=64, split_k=4 if T <= 2048 else 1) if T > ops.DECODE_GEMM_MAX_M else {}     # as for a router's columns
+        ops.gemm(h[:, 4 * H:], w1, out=low, static_b=True, **narrow)
+        parts = [out[:, i * N:(i + 1) * N] for i in range(4)]
+        weights = [self._w(l, n) for n in ("w2", "w0", "bonus", "o_norm")]
+        args = dict(rank=mx.rank, eps=self.cfg.rms_eps)
+        ns = m.batch if not m.is_prefill else m.singles
+        if ns:
+            ops.wkv(*parts, low, *weights, rc.state, mid, m.pos, None, m.seq_slot[:ns], **args)
+        if m.batch > ns:
+            ops.wkv(*parts, low, *weights, rc.state, mid, m.pos, m.tok_indptr[ns:], m.seq_slot[ns:], row_lens=m.seq_lens_host[ns:],
+                    cum=self._cum, **args)
+
+    SEPARATE_WEIGHTS = 1 << 21    # elements of one of the four matrices
+
+    def _parallel(self, r: int, l: int, mx: ParallelMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta) -> None:
+        left = {n[2:]: v for n, v in p.items() if n.startswith("l_")}
+        self._attention(r, l, mx.left, left, mid, m, prefix="l_")
+        self._ssd(r, l, mx.right, p["r_z"], p["r_xbc"], p["r_dt"], self._mid_right[mx.right.out_width][:m.num_tokens], m, "r_")
+
+    def _ssd(self, r: int, l: int, mx: SSDMixer, z, xbc, dt, mid: torch.Tensor, m: StepMeta, prefix: str) -> None:
+        T, rc = m.num_tokens, self.cache.runs[r]
+        w = lambda n: self._w(l, prefix + n)
+        u = self._conv[:T * mx.channels].view(T, mx.channels)
+        ops.token_conv(xbc, w("conv"), rc.hist, u, m.pos, m.tok_indptr if m.is_prefill else None, m.seq_slot, bias=w("conv_b"), silu=True)
+        n = mx.groups * mx.state
+        parts = [u[:, :mx.out_width], u[:, mx.out_width:mx.out_width + n], u[:, mx.out_width + n:], z, dt, w("dt_bias"), w("A_log"), w("D")]
+        ns = m.batch if not m.is_prefill else m.singles
+        if ns:
+            ops.ssd(*parts, rc.state, mid, m.pos, None, m.seq_slot[:ns], groups=mx.groups)
+        if m.batch > ns:
+            ops.ssd(*parts, rc.state, mid, m.pos, m.tok_indptr[ns:], m.seq_slot[ns:], groups=mx.groups, row_lens=m.seq_lens_host[ns:])
+        ops.part_norm(mid[:, :mx.out_width], w("o_norm"), mx.norm_groups, self.cfg.rms_eps)
+
     # ------------------------------------------------------------------ head
     def logits_of(self, n: int, rows: Optional[torch.Tensor] = None, row_offset: int = 0) -> torch.Tensor:
         """fp32 logits of `n` rows of the stream: rows 0 .. n - 1, or `rows` (+ row_offset)."""
@@ -380,8 +507,7 @@ class HybridRunner:
         cap = dict(epilogue="softcap", alpha=c.logit_softcap) if c.logit_softcap else {}
         if c.streams:
             h = self._head_in[:n]
-            ops.stream_mix(self.res, n=n, **self._embeddings(), pending=self._pending, norm=self._norm("final_norm"), out=h, rows=rows,
-                           row_offset=row_offset)
+            self._streams("final_norm", n=n, out=h, rows=rows, row_offset=row_offset)
             ops.gemm(h, self.seg["lm_head"], out=self._logits_pad[:n], static_b=True, **cap)
             return self.logits[:n]
         add = {} if rows is not None else self._take_pending()
@@ -403,7 +529,7 @@ class HybridRunner:
         """[batch, hidden]: the stream (or the sum of the streams) at the last row of every sequence of a prefill pass."""
         if self.cfg.streams:
             last = self.last[:m.batch]
-            ops.stream_mix(self.res, n=m.batch, **self._embeddings(), pending=self._pending, total=last, rows=m.tok_indptr[1:], row_offset=-1)
+            self._streams(n=m.batch, total=last, rows=m.tok_indptr[1:], row_offset=-1)
             return last
         return torch.index_select(self.res, 0, m.tok_indptr[1:] - 1, out=self.last[:m.batch])
 
@@ -432,7 +558,8 @@ class HybridRunner:
 
     def decode_launches(self) -> int:
         """Kernels of this library in one decode step."""
-        per = {"attention": 2, "latent": 7, "gla": 1, "rglru": 3}
+        per = {"attention": 2, "latent": 7, "gla": 1, "rglru": 3, "parallel": 6}
+        per["wkv"] = 5 if any(m.kind == "wkv" and m.out_width * m.hidden >= self.SEPARATE_WEIGHTS for m in self.cfg.run_mixers()) else 2
         specs = [self.cfg.layer_specs[r.layer] for r in self.runs]
         n = sum(3 + per[s.mixer.kind] + bool(s.ff) + 3 * bool(s.ff_after) + 5 * bool(s.moe) for s in specs)
         return n + 3      # final norm, head product, arg-max

@@ -1,10 +1,10 @@
 """Shapes and constants of models whose layers differ: a list of layers over an fp32 residual stream, or several of them,
-each with a mixer (attention, latent attention, gated linear attention, gated linear recurrence) and an optional
-feed-forward, with an optional block of layers that runs several times.  The feed-forward is a gated one beside the mixer
+each with a mixer (attention, latent attention, gated linear attention, gated linear recurrence, linear attention with a token
+shift and a bonus, state space, or two of them side by side) and an optional feed-forward, with an optional block of layers that runs several times.  The feed-forward is a gated one beside the mixer
 (both read one norm), or a gated one or a mixture of experts behind it (with a norm of its own).
 
-Everything a kernel needs is a field here, so a design is described by data: `models/fafudra.py`, `models/komulorn.py` and
-`models/vofidra.py` fill these records from a checkpoint's config.json, the registry from shapes.  `ModelConfig` (config.py) stays the record of
+Everything a kernel needs is a field here, so a design is described by data: `models/fafudra.py`, `models/komulorn.py`,
+`models/vofidra.py` and `models/norusun.py` fill these records from a checkpoint's config.json, the registry from shapes.  `ModelConfig` (config.py) stays the record of
 the uniform Llama-type models; both offer what the engine, the worker and the router read (name, vocab, hidden,
 layers, eos_token, param_gb, kv_bytes_per_token).
 
@@ -16,9 +16,9 @@ Weight segment of such a model (one allocation, matrices ``[in, out]``, every te
           | shared_up [hidden, shared ff] | shared_down [shared ff, hidden] }
     final_norm [hidden] | lm_head [hidden, vocab]
 
-Every norm of a model with the dynamic-tanh norm has two more tensors (``norm1_b`` and ``norm1_alpha``), a sublayer of a
+A norm's weight is one number where `norm_scalar` says so.  Every norm of a model with the dynamic-tanh norm has two more tensors (``norm1_b`` and ``norm1_alpha``), a sublayer of a
 model with several streams its coefficients (``hc1_in``, ``hc1_out``, ``hc1_mix``), a gated feed-forward behind the mixer
-``gate_up`` and ``down``.  Some tensors are derived from others when a segment is filled (`derive_`): forms of one matrix that
+``gate_up`` and ``down`` (with a clamped unit also their biases), a layer whose mixer reads a convolution of its input ``mix_conv``.  Some tensors are derived from others when a segment is filled (`derive_`): forms of one matrix that
 different kernels read.
 
 A layer has two wide projections per side: ``in`` holds every projection of the mixer next to each other and ``out``
@@ -131,6 +131,9 @@ class AttentionMixer:
     qk_norm: bool = False         # RMSNorm of every query and key head (no rotation, no biases)
     q_temp: Optional["QueryTemperature"] = None   # with qk_norm: queries grow with the position
     rel: Optional["DistanceBias"] = None          # learned bias by distance and head, added to the scaled scores
+    whole_norm: bool = False      # RMSNorm over all query heads together, and over all key heads, before the rotation
+    chunked: bool = False         # the window is a chunk counted from position 0: a position sees its own chunk's keys
+    sigmoid: bool = False         # weights are sigmoids of score + a learned number per head, not normalised
     kind = "attention"
 
     def __post_init__(self):
@@ -142,6 +145,12 @@ class AttentionMixer:
             raise ValueError("attention mixer: normed queries and keys come without rotation, biases or shared caches")
         if self.q_temp and not self.qk_norm:
             raise ValueError("attention mixer: a query temperature goes with normed queries")
+        if self.whole_norm and (self.qk_norm or self.bias or self.value_is_key or self.kv_from is not None):
+            raise ValueError("attention mixer: a norm over all heads comes without other norms, biases or shared caches")
+        if self.chunked and (not self.window or self.keep_first):
+            raise ValueError("attention mixer: chunks have a size and no kept tokens")
+        if self.sigmoid and (self.rel or self.softcap or self.sink):
+            raise ValueError("attention mixer: sigmoid weights do not go with a bias by distance, a cap or a sink")
         if self.rel and (self.window or self.softcap or self.sink):
             raise ValueError("attention mixer: a bias by distance does not go with a window, a cap or a sink")
 
@@ -168,6 +177,10 @@ class AttentionMixer:
         out = ([("sink", (self.heads,))] if self.sink else []) + ([(n + "_b", (w,)) for n, w in self._qkv()] if self.bias else [])
         if self.qk_norm:
             out += [("q_norm", (self.dim,)), ("k_norm", (self.dim,))]
+        if self.whole_norm:
+            out += [("q_norm", (self.heads * self.dim,)), ("k_norm", (self.kv_heads * self.dim,))]
+        if self.sigmoid:
+            out.append(("weight_b", (self.heads, 1)))
         if self.rel:
             out += [("rel", (self.rel.rows, self.heads)), ("rel_by_distance", (self.heads, len(self.rel.rows_by_distance())))]
         return out
@@ -181,7 +194,7 @@ class AttentionMixer:
 class LatentAttentionMixer:
     """Attention whose keys and values come from one latent vector per token, which is cached together with a rotated key part
     that all heads share; queries come from a latent of their own.  Per head: `dim` unrotated and `rot_dim` rotated query and
-    key dimensions (half-split pairs), values of `vdim`."""
+    key dimensions, values of `vdim`."""
     heads: int
     dim: int
     rot_dim: int
@@ -191,6 +204,9 @@ class LatentAttentionMixer:
     scale: float
     rot_base: float
     gate: bool = True             # as in AttentionMixer
+    interleaved: bool = False     # rotation pairs, as in AttentionMixer
+    window: int = 0               # likewise
+    sink: bool = False            # likewise
     kind = "latent"
     kv_heads = 1                  # as the cache sees it: one key, its first kv_rank columns the value
 
@@ -220,7 +236,7 @@ class LatentAttentionMixer:
         H = self.heads
         return [("dq_norm", (self.q_rank,)), ("dkv_norm", (self.kv_rank,)), ("uq", (self.q_rank, H * self.qdim)),
                 ("uk", (H * self.dim, self.kv_rank)), ("uv", (H * self.kv_rank, self.vdim)),
-                ("k_up", (self.width, H * self.qdim)), ("v_up", (self.kv_rank, H * self.vdim))]
+                ("k_up", (self.width, H * self.qdim)), ("v_up", (self.kv_rank, H * self.vdim))] + ([("sink", (H,))] if self.sink else [])
 
     def derive_(self, t) -> None:
         H, R = self.heads, self.kv_rank
@@ -284,8 +300,119 @@ class RGLRUMixer:
                 ("gate_b", (2 * w,)), ("lam", (w,))]
 
 
-Mixer = Union[AttentionMixer, LatentAttentionMixer, GLAMixer, RGLRUMixer]
+@dataclass(frozen=True)
+class WKVMixer:
+    """Linear attention with a decay per key channel that depends on the token, a bonus for the current token and a token shift:
+    each of its five projections reads a mix of the token's row and the one before it."""
+    hidden: int
+    heads: int
+    dim: int
+    rank: int                     # of the decay projection
+    kind = "wkv"
+    MIXES = ("r", "k", "v", "g", "w")
+
+    @property
+    def vdim(self) -> int:
+        return self.dim
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.dim
+
+    def projections(self) -> List[Tuple[str, int]]:
+        return []                 # (each has an input of its own)
+
+    def tensors(self) -> List[Tuple[str, Tuple[int, ...]]]:
+        # rkvg: the four projections stacked along their inputs, as the blocks of a block-diagonal product
+        H, n = self.hidden, self.out_width
+        return [("mu", (len(self.MIXES), H)), ("rkvg", (4 * H, n)), ("w1", (H, pad8(self.rank))), ("w2", (self.rank, n)), ("w0", (n,)),
+                ("bonus", (n,)), ("o_norm", (n,))]
+
+    def state_floats(self) -> int:
+        return self.heads * self.dim * self.dim
+
+    def zero_padding_(self, t) -> None:
+        t("w1")[:, self.rank:] = 0
+
+
+@dataclass(frozen=True)
+class SSDMixer:
+    """State-space recurrence with a decay per head behind a short convolution, gated and normed in `norm_groups` parts."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int                   # of heads that share their input and output vectors
+    taps: int
+    norm_groups: int
+    kind = "ssd"
+
+    def __post_init__(self):
+        if self.heads % self.groups or self.out_width % self.norm_groups or self.taps < 1:
+            raise ValueError(f"state-space mixer: {self.heads} heads in {self.groups} groups, {self.norm_groups} norm groups, {self.taps} taps")
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:
+        """Of the convolution: x, B and C."""
+        return self.out_width + 2 * self.groups * self.state
+
+    def projections(self) -> List[Tuple[str, int]]:
+        return [("z", self.out_width), ("xbc", self.channels), ("dt", self.heads)]
+
+    def tensors(self) -> List[Tuple[str, Tuple[int, ...]]]:
+        h = (self.heads,)
+        return [("conv", (self.taps, self.channels)), ("conv_b", (self.channels,)), ("dt_bias", h), ("A_log", h), ("D", h),
+                ("o_norm", (self.out_width,))]
+
+    def state_floats(self) -> int:
+        return self.heads * self.state * self.vdim
+
+
+@dataclass(frozen=True)
+class ParallelMixer:
+    """Two mixers side by side on one input; half the sum of their outputs, each RMS-normed over the model's width.  The names of
+    the left one's projections and tensors start with l_, the right one's with r_ (``out`` is the left one's output projection)."""
+    hidden: int
+    left: AttentionMixer
+    right: SSDMixer
+    kind = "parallel"
+
+    def parts(self):
+        return (("l_", self.left), ("r_", self.right))
+
+    @property
+    def out_width(self) -> int:
+        return self.left.out_width
+
+    @property
+    def right_rows(self) -> int:
+        return pad8(self.right.out_width)
+
+    def projections(self) -> List[Tuple[str, int]]:
+        return [(p + n, w) for p, m in self.parts() for n, w in m.projections()]
+
+    def tensors(self) -> List[Tuple[str, Tuple[int, ...]]]:
+        return [(p + n, shape) for p, m in self.parts() for n, shape in m.tensors()] + [
+            ("r_out", (self.right_rows, self.hidden)), ("l_out_norm", (self.hidden,)), ("r_out_norm", (self.hidden,))]
+
+    def derive_(self, t) -> None:
+        for p, m in self.parts():
+            if hasattr(m, "derive_"):
+                m.derive_(lambda n, p=p: t(p + n))
+
+    def zero_padding_(self, t) -> None:
+        t("r_out")[self.right.out_width:] = 0
+
+
+Mixer = Union[AttentionMixer, LatentAttentionMixer, GLAMixer, RGLRUMixer, WKVMixer, SSDMixer, ParallelMixer]
 PAGED = ("attention", "latent")   # mixers with a paged cache; the others keep a state per sequence
+
+
+def mixer_parts(m: Mixer) -> Tuple[Mixer, ...]:
+    return (m.left, m.right) if m.kind == "parallel" else (m,)
 
 
 @dataclass(frozen=True)
@@ -355,15 +482,29 @@ class ExpertsSpec:
 
 
 @dataclass(frozen=True)
+class ClampedUnit:
+    """A feed-forward's gated unit with biases: g = min(gate, limit), u = up within +- limit, g sigmoid(beta g) (u + 1)."""
+    limit: float
+    beta: float = 1.702
+
+    def __post_init__(self):
+        if not self.limit > 0:
+            raise ValueError(f"clamped unit: the limit must be positive, not {self.limit}")
+
+
+@dataclass(frozen=True)
 class LayerSpec:
     mixer: Mixer
     ff: int = 0                   # width of the gated feed-forward beside the mixer; 0: none
     moe: Optional[ExpertsSpec] = None   # experts behind the mixer, with a norm of their own
     ff_after: int = 0             # width of a gated feed-forward behind the mixer, with a norm of its own; 0: none
+    unit: Optional[ClampedUnit] = None  # its unit (None: silu(gate) * up, no biases)
 
     def __post_init__(self):
         if bool(self.ff) + bool(self.moe) + bool(self.ff_after) > 1:
             raise ValueError("a layer has a feed-forward beside its mixer, one behind it, or experts behind it")
+        if self.unit and not self.ff_after:
+            raise ValueError("a clamped unit belongs to a feed-forward behind the mixer")
 
     @property
     def sublayers(self) -> Tuple[int, ...]:
@@ -422,6 +563,8 @@ class HybridConfig:
     logit_softcap: float = 0.0    # logits become cap * tanh(logits / cap); 0: none
     tied: bool = True             # the head is the embedding table
     norm: str = "rms"             # "tanh": the dynamic-tanh norm, tanh(alpha x) w + b
+    norm_scalar: bool = False     # a norm's weight is one number
+    mix_taps: int = 0             # mixers read their input plus a causal convolution of it with this many taps; 0: none
     streams: int = 0              # residual streams joined by learned coefficients; 0: one, with plain sums
     design: str = "fafudra"       # module of this package that maps checkpoint names (weights of a folder)
     family = "hybrid"
@@ -438,8 +581,20 @@ class HybridConfig:
             if any(getattr(src, n) != getattr(s.mixer, n) for n in same):
                 raise ValueError(f"{self.name}: layers {j} and {i} share keys and values but differ in {', '.join(same)}")
         lp = self.loop
-        if self.norm not in ("rms", "tanh") or (self.norm == "tanh") != (self.streams > 0):
-            raise ValueError(f"{self.name}: the dynamic-tanh norm and several streams come together")
+        if self.norm not in ("rms", "tanh") or (self.norm == "tanh" and not self.streams):
+            raise ValueError(f"{self.name}: the dynamic-tanh norm comes with several streams")
+        plain = self.norm == "tanh" or not self.streams
+        if plain and (self.norm_scalar or self.mix_taps or any(s.mixer.kind in ("wkv", "parallel") or s.unit for s in self.layer_specs)):
+            raise ValueError(f"{self.name}: scalar norms, convolved inputs, token shifts, mixers side by side and clamped units go with "
+                             "several streams and RMS norms")
+        if not plain and any(s.moe for s in self.layer_specs):
+            raise ValueError(f"{self.name}: experts do not go with several streams and RMS norms")
+        if any(s.mixer.kind == "ssd" for s in self.layer_specs):
+            raise ValueError(f"{self.name}: a state-space mixer comes beside another mixer")
+        if not 0 <= self.mix_taps <= 16 or any(getattr(p, "taps", 1) > 16 for s in self.layer_specs for p in mixer_parts(s.mixer)):
+            raise ValueError(f"{self.name}: convolutions have up to 16 taps")
+        if any(getattr(p, "hidden", self.hidden) != self.hidden for s in self.layer_specs for p in (s.mixer,)):
+            raise ValueError(f"{self.name}: a mixer is built for another width")
         if not 0 <= self.streams <= 8:
             raise ValueError(f"{self.name}: at most 8 streams")
         if self.streams and (lp is not None or any(s.ff or (s.moe and s.moe.shared_ff) for s in self.layer_specs)):
@@ -468,6 +623,10 @@ class HybridConfig:
     def run_mixers(self) -> List[Mixer]:
         return [self.layer_specs[r.layer].mixer for r in self.runs()]
 
+    def run_parts(self) -> List[Mixer]:
+        """The same with mixers side by side one by one."""
+        return [p for m in self.run_mixers() for p in mixer_parts(m)]
+
     def kv_runs(self) -> List[int]:
         """For every layer run the run whose keys and values it reads (its own, but for layers that share another's)."""
         latest: Dict[int, int] = {}
@@ -480,13 +639,17 @@ class HybridConfig:
 
     def kv_bytes_per_token(self, tp: int = 1, elem: int = 2) -> int:
         per = lambda m: m.width if m.kind == "latent" else m.kv_heads * (m.dim + m.vdim) if m.kv_from is None else 0
-        return sum(per(m) * elem for m in self.run_mixers() if m.kind in PAGED)
+        return sum(per(m) * elem for m in self.run_parts() if m.kind in PAGED)
 
     def state_bytes_per_sequence(self, elem: int = 2) -> int:
-        n = 0
-        for m in self.run_mixers():
+        n = elem * max(0, self.mix_taps - 1) * self.hidden * len(self.runs())
+        for m in self.run_parts():
             if m.kind == "gla":
                 n += 4 * m.state_floats()
+            elif m.kind == "wkv":
+                n += 4 * m.state_floats() + elem * m.hidden
+            elif m.kind == "ssd":
+                n += 4 * m.state_floats() + elem * (m.taps - 1) * m.channels
             elif m.kind == "rglru":
                 n += 4 * m.width + elem * (m.taps - 1) * m.width
         return n
@@ -494,15 +657,15 @@ class HybridConfig:
     def attention_work(self, length: int) -> Tuple[int, int]:
         """(KV heads, positions) of the attention run with the fewest heads and of the one that looks furthest back, for a
         sequence of `length` tokens: what the number of key splits is chosen from.  (0, 0) without attention."""
-        a = [m for m in self.run_mixers() if m.kind in PAGED]
+        a = [m for m in self.run_parts() if m.kind in PAGED]
         if not a:
             return 0, 0
-        span = max(min(length, m.window + m.keep_first) if getattr(m, "window", 0) else length for m in a)
+        span = max(min(length, m.window + getattr(m, "keep_first", 0)) if getattr(m, "window", 0) else length for m in a)
         return min(m.kv_heads for m in a), span
 
     @property
     def recurrent(self) -> bool:
-        return any(m.kind not in PAGED for m in self.run_mixers())
+        return self.mix_taps > 1 or any(m.kind not in PAGED for m in self.run_parts())
 
     @property
     def vocab_pad(self) -> int:
@@ -511,6 +674,8 @@ class HybridConfig:
     def init_(self, name: str, v: torch.Tensor, rand) -> None:
         """Random weights with activations of order one; `rand(shape)` gives normal numbers on v's device."""
         leaf = name.rsplit(".", 1)[-1]
+        if leaf.startswith(("l_", "r_")):                    # one of two mixers side by side
+            leaf = leaf[2:]
         if leaf.endswith("norm_alpha") or leaf in ("norm1_alpha", "norm2_alpha"):
             x = 0.7 + 0.1 * rand(v.shape)
         elif leaf in ("norm1_b", "norm2_b", "final_norm_b", "rel", "correction"):
@@ -521,7 +686,17 @@ class HybridConfig:
             x = 1.0 + 0.2 * rand(v.shape)
         elif leaf in ("hc1_mix", "hc2_mix"):
             x = torch.eye(v.shape[0], device=v.device) + 0.1 * rand(v.shape)
-        elif leaf in ("q_norm", "k_norm", "dq_norm", "dkv_norm"):
+        elif leaf == "mu":
+            x = 0.5 + 0.2 * rand(v.shape)
+        elif leaf == "rkvg":                                 # four matrices stacked along their inputs
+            x = rand(v.shape) * (v.shape[0] // 4) ** -0.5
+        elif leaf in ("w0", "dt_bias", "weight_b"):
+            x = -2.0 + 0.5 * rand(v.shape)
+        elif leaf in ("bonus", "A_log"):
+            x = 0.5 * rand(v.shape)
+        elif leaf in ("gate_up_b", "down_b"):
+            x = 0.1 * rand(v.shape)
+        elif leaf in ("q_norm", "k_norm", "dq_norm", "dkv_norm", "D", "out_norm"):
             x = 1.0 + 0.1 * rand(v.shape)
         elif leaf == "uk":                                   # stacked by head: [heads * dim, rank], the rank is the input
             x = rand(v.shape) * v.shape[1] ** -0.5
@@ -543,7 +718,7 @@ class HybridConfig:
             for e in range(moe.experts):
                 v[e * n:(e + 1) * n].copy_((rand((n, v.shape[1])) * n ** -0.5).to(v.dtype))
             return
-        elif leaf == "conv":
+        elif leaf in ("conv", "mix_conv"):
             x = rand(v.shape) * v.shape[0] ** -0.5
         elif leaf == "embed":
             x = rand(v.shape)
@@ -574,6 +749,12 @@ class HybridConfig:
                 o[s.mix_rows + s.ff:] = 0
             if s.ff_after:
                 tensors[p + "down"][s.ff_after:] = 0
+            if s.unit:
+                b = tensors[p + "gate_up_b"]
+                b[s.ff_after:s.ff_after_pad] = 0
+                b[s.ff_after_pad + s.ff_after:] = 0
+            if hasattr(s.mixer, "zero_padding_"):
+                s.mixer.zero_padding_(lambda n, p=p: tensors[p + n])
             n, pad = (s.ff, s.ff_pad) if s.ff else (s.ff_after, s.ff_after_pad)
             if n:
                 g = tensors[p + "gate_up"]
@@ -607,7 +788,7 @@ def build_hybrid_layout(cfg: HybridConfig, tp: int = 1, elem_bytes: int = 2) -> 
         cur = _align(cur + n)
 
     def add_norm(name):
-        add(name, (cfg.hidden,))
+        add(name, (1,) if cfg.norm_scalar else (cfg.hidden,))
         if cfg.norm == "tanh":
             add(name + "_b", (cfg.hidden,))
             add(name + "_alpha", (1,))
@@ -620,6 +801,8 @@ def build_hybrid_layout(cfg: HybridConfig, tp: int = 1, elem_bytes: int = 2) -> 
     for l, s in enumerate(cfg.layer_specs):
         start, p = cur, f"layers.{l}."
         add_norm(p + "norm1")
+        if cfg.mix_taps:
+            add(p + "mix_conv", (cfg.mix_taps, cfg.hidden))
         add(p + "in", (cfg.hidden, s.in_columns()[1]))
         for n, shape in s.mixer.tensors():
             add(p + n, shape)
@@ -641,6 +824,9 @@ def build_hybrid_layout(cfg: HybridConfig, tp: int = 1, elem_bytes: int = 2) -> 
             add_norm(p + "norm2")
             add(p + "gate_up", (cfg.hidden, 2 * s.ff_after_pad))
             add(p + "down", (s.ff_after_pad, cfg.hidden))
+        if s.unit:
+            add(p + "gate_up_b", (2 * s.ff_after_pad,))
+            add(p + "down_b", (cfg.hidden,))
         if cfg.streams:
             for q in s.sublayers:
                 for n, shape in (("in", (cfg.streams,)), ("out", (cfg.streams,)), ("mix", (cfg.streams, cfg.streams))):

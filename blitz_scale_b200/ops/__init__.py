@@ -116,7 +116,7 @@ def check_status(device=None, reset: bool = True) -> int:
 
 
 # ---------------------------------------------------------------------------------------------- GEMM
-_EPI = {"store": 0, "add": 1, "silu_mul": 2, "axpy": 5, "softcap": 6}
+_EPI = {"store": 0, "add": 1, "silu_mul": 2, "axpy": 5, "softcap": 6, "clamp_glu": 7}
 _EPI_STORE_F32 = 4
 
 
@@ -160,7 +160,7 @@ def _tensor_core_operands(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, N
 
 
 def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *, residual=None,
-         epilogue: str = "store", alpha: float = 1.0, groups: int = 1, a_step: int = 0, out_step: int = 0, b_layout: str = "kn", bn: int = 0, split_k: int = 0, static_b: bool = False,
+         epilogue: str = "store", alpha: float = 1.0, beta: float = 1.0, bias: Optional[torch.Tensor] = None, groups: int = 1, a_step: int = 0, out_step: int = 0, b_layout: str = "kn", bn: int = 0, split_k: int = 0, static_b: bool = False,
          decode_path: Optional[bool] = None, decode_split: int = 0, pair_path: Optional[bool] = None,
          pair_bnf: int = 0, pair_upp: int = 0, pair_nacc: int = 0) -> torch.Tensor:
     """``out = a @ b`` on tcgen05 with a fused epilogue.
@@ -182,7 +182,8 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *
 
     ``out`` may be fp32 with 16-bit operands (the accumulator is stored unrounded); epilogue 'axpy' adds
     ``alpha * (a @ b)`` to an fp32 ``out`` (residual streams kept in 32 bits); 'softcap' stores
-    ``alpha * tanh((a @ b) / alpha)`` in fp32 (logits).  ``groups`` > 1: block-diagonal product,
+    ``alpha * tanh((a @ b) / alpha)`` in fp32 (logits); 'clamp_glu' is a clamped gated unit over [gate | up] columns with
+    ``bias`` (as many as b's columns): g = min(gate, alpha), u = up within +- alpha, g * sigmoid(beta g) * (u + 1).  ``groups`` > 1: block-diagonal product,
     a [M, groups * K], b [groups * K, N] (the blocks stacked), out [M, groups * N]; ``a_step`` / ``out_step``: columns from a
     group to the next one in a and out, where the blocks' columns are parts of wider ones.  fp32 operands, and 16-bit ones
     whose sizes the tensor-core kernels do not take, run on the CUDA cores in fp32 arithmetic.
@@ -201,7 +202,10 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *
         assert b.shape[1] == K
         bcols = b.shape[0]
     epi = _EPI[epilogue]
-    N = bcols // 2 if epi == 2 else bcols
+    gated = epi in (2, 7)
+    N = bcols // 2 if gated else bcols
+    if epi == 7:
+        assert bias is not None and bias.is_contiguous() and bias.numel() == bcols and bias.dtype == a.dtype and alpha > 0
     if out is None:
         out = torch.empty((M, groups * N), dtype=a.dtype, device=a.device)
     assert out.stride(1) == 1 and out.shape[0] == M
@@ -218,10 +222,11 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *
             raise TypeError("gemm: epilogue 'add' and 'nk' weights need the tensor-core kernels")
         assert b.dtype == a.dtype
         _check(lib().blitz_gemm_simt(_p(a), a.stride(0), _p(b), b.stride(0), _p(out), out.stride(0), M, N, K, epi,
-                                     N if epi == 2 else 0, alpha, groups, a_step, out_step, _dt3(a), _stream()), "blitz_gemm_simt")
+                                     N if gated else 0, _p(bias), alpha, beta, groups, a_step, out_step, _dt3(a), _stream()), "blitz_gemm_simt")
         return out
     if epi == 1:
         assert residual is not None and residual.shape == (M, N) and residual.stride(0) == out.stride(0)
+    extra = bias if epi == 7 else residual
     ws, tickets = gemm_workspace(a.device)
     # the decode kernel re-reads the activation tile with every weight tile, which the SM's load path cannot keep up
     # with beyond ~128 rows; from there on the tiled kernel is faster
@@ -237,21 +242,21 @@ def gemm(a: torch.Tensor, b: torch.Tensor, out: Optional[torch.Tensor] = None, *
         use_pair = pair_path
     if use_pair:
         pws, pflags = pair_gemm_workspace(a.device)
-        rc = lib().blitz_gemm_pair(_p(a), a.stride(0), _p(b), b.stride(0), _p(out), out.stride(0), _p(residual), M, N,
-                                   K, epi, N if epi == 2 else 0, _dt(a), int(static_b), pair_bnf, pair_nacc, pair_upp,
+        rc = lib().blitz_gemm_pair(_p(a), a.stride(0), _p(b), b.stride(0), _p(out), out.stride(0), _p(extra), M, N,
+                                   K, epi, N if gated else 0, _dt(a), int(static_b), pair_bnf, pair_nacc, pair_upp,
                                    _p(pws), pws.numel(), _p(pflags), pflags.numel(), _p(status_word(a.device)),
-                                   alpha, _stream())
+                                   alpha, beta, _stream())
         _check(rc, "blitz_gemm_pair")
         return out
     if use_dec:
-        rc = lib().blitz_gemm_decode(_p(a), a.stride(0), _p(b), b.stride(0), _p(out), out.stride(0), _p(residual), M, N,
-                                     K, epi, N if epi == 2 else 0, _dt(a), int(static_b), decode_split,
-                                     _p(status_word(a.device)), alpha, _stream())
+        rc = lib().blitz_gemm_decode(_p(a), a.stride(0), _p(b), b.stride(0), _p(out), out.stride(0), _p(extra), M, N,
+                                     K, epi, N if gated else 0, _dt(a), int(static_b), decode_split,
+                                     _p(status_word(a.device)), alpha, beta, _stream())
         _check(rc, "blitz_gemm_decode")
         return out
-    rc = lib().blitz_gemm(_p(a), a.stride(0), _p(b), b.stride(0), _p(out), out.stride(0), _p(residual), M, N, K,
-                          0 if b_layout == "kn" else 1, epi, N if epi == 2 else 0, _dt(a), bn, split_k,
-                          _p(ws), ws.numel(), _p(tickets), tickets.numel(), _p(status_word(a.device)), alpha,
+    rc = lib().blitz_gemm(_p(a), a.stride(0), _p(b), b.stride(0), _p(out), out.stride(0), _p(extra), M, N, K,
+                          0 if b_layout == "kn" else 1, epi, N if gated else 0, _dt(a), bn, split_k,
+                          _p(ws), ws.numel(), _p(tickets), tickets.numel(), _p(status_word(a.device)), alpha, beta,
                           groups, a_step, out_step, _stream())
     _check(rc, "blitz_gemm")
     return out
@@ -355,12 +360,13 @@ def attn_decode(q: torch.Tensor, kv_layer: KVLayer, indices: torch.Tensor, indpt
                 num_splits: int = 1, workspace: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
                 sm_scale: Optional[float] = None, window: int = 0, keep_first: int = 0, softcap: float = 0.0,
                 sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                bias: Optional[torch.Tensor] = None, chunked: bool = False, sigmoid: bool = False) -> torch.Tensor:
     """q: [batch, >= q_heads*head_dim] (row pitch free, e.g. a view of the fused qkv buffer).  ``window`` > 0: only the
     last that many positions and the first ``keep_first`` are visible (and read); ``softcap`` > 0:
     scores are cap * tanh(score / cap); ``sink`` [q_heads]: a term e^sink in the softmax denominator; ``gate``
     [batch, q_heads]: a head's output is multiplied by its sigmoid; ``bias`` [q_heads, n]: added to the scaled scores by the
-    key's distance, the last column for all longer ones.  Values may have a size of their own (KVPair)."""
+    key's distance, the last column for all longer ones.  ``chunked``: the window is a chunk counted from position 0, of which
+    the keys up to the position are visible; ``sigmoid``: the weights are sigmoids of the scores, not normalised.  Values may have a size of their own (KVPair)."""
     B = indptr.numel() - 1
     kp, vp, page_rows, pages, vdim = _kv(kv_layer)
     if out is None:
@@ -372,7 +378,7 @@ def attn_decode(q: torch.Tensor, kv_layer: KVLayer, indices: torch.Tensor, indpt
         sm_scale = head_dim ** -0.5
     _check(lib().blitz_attn_decode(_p(q), q.stride(0), kp, vp, _p(indices), _p(indptr), _p(last_page_len),
                                    _p(out), out.stride(0), _p(workspace), B, q_heads, kv_heads, head_dim, vdim, page_size,
-                                   page_rows, pages, num_splits, sm_scale, window, keep_first, softcap, _p(sink), *_bias(bias, q_heads), *_gate(gate),
+                                   page_rows, pages, num_splits, sm_scale, window, keep_first, int(chunked), int(sigmoid), softcap, _p(sink), *_bias(bias, q_heads), *_gate(gate),
                                    _p(status_word(q.device)), _dt(q), _stream()), "blitz_attn_decode")
     return out
 
@@ -406,16 +412,20 @@ def prefill_work_list(q_lens, kv_lens, page_size: int, device, skip: int = 0) ->
     return torch.tensor(rec, dtype=torch.int32).reshape(-1, 8).to(device, non_blocking=True)
 
 
+PREFILL_KEY_BLOCK = 128     # keys that attn_prefill_paged walks at a time
+
+
 def attn_prefill_paged(q: torch.Tensor, kv_layer: KVLayer, page_indices: torch.Tensor, work: torch.Tensor, *,
                        q_heads: int, kv_heads: int, head_dim: int, page_size: int, out: Optional[torch.Tensor] = None,
                        sm_scale: Optional[float] = None, poly_exp: bool = False, window: int = 0, keep_first: int = 0,
                        softcap: float = 0.0, sink: Optional[torch.Tensor] = None,
-                       gate: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                       gate: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None, chunked: bool = False,
+                       sigmoid: bool = False) -> torch.Tensor:
     """Causal attention of the pass's rows over the paged cache (which already holds the rows' own keys and values,
     after whatever earlier passes stored).  ``q``: rotated query columns, e.g. the fused qkv buffer (rope_kv_store);
     ``page_indices``: the sequences' page ids back to back, covering prefix + rows; ``work`` from `prefill_work_list`
-    for the same sequences.  ``window`` / ``keep_first`` / ``softcap`` / ``sink`` / ``gate`` / ``bias`` as for `attn_decode`
-    (no bias beside a window, cap or sink)."""
+    for the same sequences.  ``window`` / ``keep_first`` / ``softcap`` / ``sink`` / ``gate`` / ``bias`` / ``chunked`` / ``sigmoid``
+    as for `attn_decode` (no bias beside a window, cap or sink; with sigmoid weights a bias of one column)."""
     T = q.shape[0]
     kp, vp, page_rows, pages, vdim = _kv(kv_layer)
     if out is None:
@@ -425,7 +435,7 @@ def attn_prefill_paged(q: torch.Tensor, kv_layer: KVLayer, page_indices: torch.T
     assert work.dtype == torch.int32 and work.dim() == 2 and work.shape[1] == 8 and work.is_contiguous()
     _check(lib().blitz_attn_prefill_paged(_p(q), q.stride(0), kp, vp, _p(out), out.stride(0), _p(page_indices),
                                           _p(work), work.shape[0], T, q_heads, kv_heads, head_dim, vdim, page_size, page_rows,
-                                          pages, sm_scale, 1 if poly_exp else 0, window, keep_first, softcap, _p(sink),
+                                          pages, sm_scale, 1 if poly_exp else 0, window, keep_first, int(chunked), int(sigmoid), softcap, _p(sink),
                                           *_bias(bias, q_heads), *_gate(gate), _p(status_word(q.device)), _dt(q), _stream()), "blitz_attn_prefill_paged")
     return out
 
@@ -471,14 +481,17 @@ def rope_freqs(dims: int, base: float, device, stretch: Optional[Sequence[float]
 def rope_store(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tensor], pos: torch.Tensor, slot: torch.Tensor,
                kv_layer: KVLayer, freqs: torch.Tensor, *, q_heads: int, kv_heads: int, dim: int, rot_dims: int,
                page_size: int, interleaved: bool, gain: float = 1.0, q_b: Optional[torch.Tensor] = None,
-               k_b: Optional[torch.Tensor] = None, v_b: Optional[torch.Tensor] = None) -> None:
+               k_b: Optional[torch.Tensor] = None, v_b: Optional[torch.Tensor] = None, q_w: Optional[torch.Tensor] = None,
+               k_w: Optional[torch.Tensor] = None, eps: float = 0.0) -> None:
     """Rotate q in place and write rotated keys and the values to the paged cache.  q, k, v: column ranges of one
     projection ([T, ...] views with a common row pitch); ``v`` None: the values are the keys before rotation; ``k`` None:
-    nothing is written.  ``q_b``, ``k_b``, ``v_b``: biases, added first.  ``gain`` multiplies the rotated dimensions."""
+    nothing is written.  ``q_b``, ``k_b``, ``v_b``: biases, added first.  ``gain`` multiplies the rotated dimensions.  ``q_w``,
+    ``k_w``: before the rotation the rows of queries and keys get an RMS norm over all heads together, with these weights."""
+    assert (q_w is None or q_w.numel() == q_heads * dim) and (k_w is None or k_w.numel() == kv_heads * dim)
     T = q.shape[0]
     assert q.stride(1) == 1 and all(x is None or (x.stride(0) == q.stride(0) and x.stride(1) == 1) for x in (k, v))
     kp, vp, page_rows, pages, vdim = _kv(kv_layer)
-    _check(lib().blitz_rope_store(_p(q), _p(k), _p(v), _p(q_b), _p(k_b), _p(v_b), q.stride(0), _p(pos), _p(slot), kp, vp, _p(freqs),
+    _check(lib().blitz_rope_store(_p(q), _p(k), _p(v), _p(q_b), _p(k_b), _p(v_b), q.stride(0), _p(q_w), _p(k_w), eps, _p(pos), _p(slot), kp, vp, _p(freqs),
                                   gain, T, q_heads, kv_heads, dim, vdim, rot_dims, int(interleaved), page_size, page_rows, pages,
                                   _p(status_word(q.device)), _dt3(q), _stream()), "blitz_rope_store")
 
@@ -487,9 +500,9 @@ def attn_ragged(q: torch.Tensor, kv_layer: KVLayer, pos: torch.Tensor, tok_indpt
                 page_indptr: torch.Tensor, page_indices: torch.Tensor, out: torch.Tensor, *, q_heads: int, kv_heads: int,
                 dim: int, page_size: int, scale: float, window: int = 0, keep_first: int = 0, softcap: float = 0.0,
                 sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                bias: Optional[torch.Tensor] = None, chunked: bool = False, sigmoid: bool = False) -> torch.Tensor:
     """General paged attention (CUDA cores, any head sizes, any element type); see csrc/kernels/attn_ragged.cu.  ``gate``
-    [T, q_heads]: a head's output is multiplied by its sigmoid; ``bias`` as for `attn_decode`."""
+    [T, q_heads]: a head's output is multiplied by its sigmoid; ``bias``, ``chunked`` and ``sigmoid`` as for `attn_decode`."""
     T = q.shape[0]
     rows = page_indptr.numel() - 1
     assert q.stride(1) == 1 and out.stride(1) == 1
@@ -498,7 +511,7 @@ def attn_ragged(q: torch.Tensor, kv_layer: KVLayer, pos: torch.Tensor, tok_indpt
                                    _p(page_indptr), _p(page_indices), _p(sink), *_bias(bias, q_heads),
                                    kv_layer.pool.shape[3] if isinstance(kv_layer, LatentKV) else vdim, *_gate(gate), T, rows,
                                    q_heads, kv_heads, dim, vdim,
-                                   page_size, page_rows, pages, window, keep_first, scale, softcap, _p(status_word(q.device)),
+                                   page_size, page_rows, pages, window, keep_first, int(chunked), int(sigmoid), scale, softcap, _p(status_word(q.device)),
                                    _dt3(q), _stream()), "blitz_attn_ragged")
     return out
 
@@ -531,13 +544,73 @@ def stream_mix(x: torch.Tensor, *, n: Optional[int] = None, ids: Optional[torch.
 
 class Pending(NamedTuple):
     """Output of a sublayer that the streams have not taken up: ``y`` [T, hidden], or rows that ``place`` [T, n] names (-1: none),
-    with ``ident`` [T] times ``prev`` [T, hidden] on top; the coefficients ``mix`` [streams, streams] and ``out`` [streams]."""
+    with ``ident`` [T] times ``prev`` [T, hidden] on top; the coefficients ``mix`` [streams, streams] and ``out`` [streams].  For
+    `stream_rms` also: ``bias`` [hidden] on top of y, or ``norms`` = (w0, w1): y has two outputs side by side, [T, 2 hidden], of which
+    half the sum of the RMS-normed ones counts."""
     y: Optional[torch.Tensor]
     mix: Optional[torch.Tensor]
     out: Optional[torch.Tensor]
     place: Optional[torch.Tensor] = None
     ident: Optional[torch.Tensor] = None
     prev: Optional[torch.Tensor] = None
+    bias: Optional[torch.Tensor] = None
+    norms: Optional[tuple] = None
+
+
+class TokenState(NamedTuple):
+    """What a causal convolution of a token's row reads beside it: ``conv`` [taps, width], the last inputs by slot ``hist`` [slots,
+    taps - 1, width], and for mixes with the row before it ``mu`` [mixes, width] and that row by slot, ``shift`` [slots, width]."""
+    conv: torch.Tensor
+    hist: torch.Tensor
+    mu: Optional[torch.Tensor] = None
+    shift: Optional[torch.Tensor] = None
+
+
+def stream_rms(x: torch.Tensor, *, eps: float, n: Optional[int] = None, ids: Optional[torch.Tensor] = None,
+               embed: Optional[torch.Tensor] = None, pending: Optional[Pending] = None, read: Optional[torch.Tensor] = None,
+               w: Optional[torch.Tensor] = None, w_offset: float = 0.0, out: Optional[torch.Tensor] = None, total: Optional[torch.Tensor] = None,
+               write: bool = False, rows: Optional[torch.Tensor] = None, row_offset: int = 0, tokens: Optional[TokenState] = None,
+               pos: Optional[torch.Tensor] = None, seq_slot: Optional[torch.Tensor] = None) -> None:
+    """`stream_mix` with an RMS norm: ``out`` receives u / sqrt(mean(u^2) + eps) * (w_offset + w), w one number or one per column.
+    ``tokens`` (decode: a token per row, ``pos`` and ``seq_slot`` say which): out is that plus its causal convolution, or with mixes
+    [n, mixes * hidden]; see `token_conv`, which does the same for rows of any length."""
+    T, S, H = x.shape
+    n = n if n is not None else (rows.numel() if rows is not None else T)
+    assert x.dtype == torch.float32 and x.is_contiguous() and (out is None or (w is not None and out.is_contiguous()))
+    assert total is None or (total.dtype == torch.float32 and total.is_contiguous())
+    ref = embed if embed is not None else out if out is not None else pending.y if pending is not None else read
+    if ref is None:
+        ref = torch.empty(0, dtype=torch.bfloat16)        # a plain sum of fp32 streams
+    pd = pending if pending is not None else Pending(None, None, None)
+    assert pd.y is None or (pd.y.stride(1) == 1 and pd.place is None)
+    w0, w1 = pd.norms or (None, None)
+    y1 = ctypes.c_void_p(pd.y.data_ptr() + H * pd.y.element_size()) if pd.norms else None
+    ts = tokens if tokens is not None else TokenState(None, None)
+    taps, mixes = (0 if ts.conv is None else ts.conv.shape[0]), (0 if ts.mu is None else ts.mu.shape[0])
+    assert tokens is None or (n == seq_slot.numel() and out is not None and out.numel() == n * max(1, mixes) * H)
+    _check(lib().blitz_stream_rms(_p(ids), _p(embed), embed.shape[0] if embed is not None else 0, int(embed is not None), _p(x), _p(pd.y), y1,
+                                  pd.y.stride(0) if pd.y is not None else H, _p(pd.bias), _p(w0), _p(w1), _p(pd.mix), _p(pd.out), _p(read),
+                                  _p(w), int(w is not None and w.numel() > 1), w_offset, eps, _p(rows), row_offset, _p(out), _p(total),
+                                  int(write), _p(ts.conv), taps, _p(ts.hist), _p(ts.mu), mixes, _p(ts.shift), _p(pos), _p(seq_slot),
+                                  0 if ts.hist is None else ts.hist.shape[0], n, H, S, _p(status_word(x.device)), _dt3(ref), _stream()),
+           "blitz_stream_rms")
+
+
+def token_conv(x: torch.Tensor, conv: torch.Tensor, hist: torch.Tensor, out: torch.Tensor, pos, tok_indptr, seq_slot, *,
+               bias: Optional[torch.Tensor] = None, silu: bool = False, residual: bool = False, mu: Optional[torch.Tensor] = None,
+               shift: Optional[torch.Tensor] = None, last: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal convolution of every column of ``x`` [T, width] over the rows of a step, with the history [slots, taps - 1, width] it
+    reads and brings up to date: silu of it, or x plus it (``residual``).  ``mu`` [mixes, width]: out [T, mixes * width] are the
+    mixes with the token before, which ``shift`` [slots, width] holds between steps (``last`` [rows, width]: scratch).
+    ``tok_indptr`` None: one token per row."""
+    slots, keep, width = hist.shape
+    mixes = 0 if mu is None else mu.shape[0]
+    assert x.stride(1) == 1 and out.stride(1) == 1 and x.shape[1] == width and conv.shape == (keep + 1, width)
+    assert conv.is_contiguous() and hist.is_contiguous() and out.shape[1] >= max(1, mixes) * width
+    _check(lib().blitz_token_conv(_p(x), x.stride(0), _p(conv), _p(bias), _p(hist), _p(out), out.stride(0), int(silu), int(residual), _p(mu),
+                                  mixes, _p(shift), _p(last), _p(pos), _p(tok_indptr), _p(seq_slot), x.shape[0], seq_slot.numel(), width,
+                                  keep + 1, slots, _p(status_word(x.device)), _dt3(x), _stream()), "blitz_token_conv")
+    return out
 
 
 def norm_store(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor, kv_layer: KVLayer,
@@ -555,24 +628,24 @@ def norm_store(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, pos: torch.Ten
 
 # ---------------------------------------------------------------------------------------------- latent attention
 def latent_store(cq: Optional[torch.Tensor], ckv: torch.Tensor, pos: torch.Tensor, slot: torch.Tensor, kv: LatentKV,
-                 cq_w: Optional[torch.Tensor], ckv_w: torch.Tensor, freqs: torch.Tensor, *, eps: float) -> None:
+                 cq_w: Optional[torch.Tensor], ckv_w: torch.Tensor, freqs: torch.Tensor, *, eps: float, interleaved: bool = False) -> None:
     """RMSNorm of the queries' latent (in place) and of the keys' latent (to the cache), and the rotated key part (to the
     cache).  cq, ckv: column ranges of one projection."""
     T = ckv.shape[0]
     pages, page, _, width = kv.pool.shape
     assert ckv.shape[1] == width and ckv.stride(1) == 1 and (cq is None or (cq.stride(0) == ckv.stride(0) and cq.stride(1) == 1))
     _check(lib().blitz_latent_store(_p(cq), _p(ckv), ckv.stride(0), _p(cq_w), _p(ckv_w), _p(pos), _p(slot), _p(kv.pool), _p(freqs), eps,
-                                    T, cq.shape[1] if cq is not None else 0, kv.rank, width - kv.rank, page, pages,
+                                    T, cq.shape[1] if cq is not None else 0, kv.rank, width - kv.rank, int(interleaved), page, pages,
                                     _p(status_word(ckv.device)), _dt3(ckv), _stream()), "blitz_latent_store")
 
 
 def latent_rotate(q: torch.Tensor, out: torch.Tensor, pos: torch.Tensor, freqs: torch.Tensor, *, heads: int, dim: int, rot: int,
-                  out_step: int) -> None:
+                  out_step: int, interleaved: bool = False) -> None:
     """Rotate the last ``rot`` dimensions of every head of q [T, heads * (dim + rot)]; head h's go to columns h * out_step on of
     ``out`` (which may be a view of q: in place)."""
     assert q.stride(1) == 1 and out.stride(1) == 1 and q.shape[1] == heads * (dim + rot)
     _check(lib().blitz_latent_rotate(_p(q), q.stride(0), _p(out), out.stride(0), out_step, _p(pos), _p(freqs), q.shape[0], heads, dim,
-                                     rot, _dt3(q), _stream()), "blitz_latent_rotate")
+                                     rot, int(interleaved), _dt3(q), _stream()), "blitz_latent_rotate")
 
 
 def latent_gather(kv: LatentKV, pages: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
@@ -600,10 +673,11 @@ ATTN_LATENT_ROWS = 1024     # tokens of prompts in one launch
 def attn_latent(q: torch.Tensor, kv: LatentKV, indices: torch.Tensor, indptr: torch.Tensor, last_page_len: torch.Tensor, *, heads: int,
                 scale: float, workspace: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None,
                 keys: int = 0, static_table: bool = False, pos: Optional[torch.Tensor] = None,
-                tok_indptr: Optional[torch.Tensor] = None) -> torch.Tensor:
+                tok_indptr: Optional[torch.Tensor] = None, window: int = 0, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Decode attention over latent rows: q [batch, heads * width] against every cached row as it is, out [batch, heads * rank] =
     the weighted sums of the rows' first ``rank`` columns, times the sigmoid of ``gate`` [batch, heads].  With ``pos`` and
-    ``tok_indptr`` the batch are the tokens of a ragged step (as for `attn_ragged`), each sees the keys up to its position.  ``keys``: per block, 64 or 128 (0: chosen).
+    ``tok_indptr`` the batch are the tokens of a ragged step (as for `attn_ragged`), each sees the keys up to its position.  ``window`` > 0: only the
+    last that many positions; ``sink`` [heads]: a term e^sink in the softmax denominator.  ``keys``: per block, 64 or 128 (0: chosen).
     ``static_table`` promises that no kernel still running in this stream writes the page table (indices, indptr,
     last_page_len), so that the work list can be made before the predecessor has finished."""
     assert (pos is None) == (tok_indptr is None)
@@ -612,20 +686,20 @@ def attn_latent(q: torch.Tensor, kv: LatentKV, indices: torch.Tensor, indptr: to
         for t in range(0, B, ATTN_LATENT_ROWS):
             part = slice(t, min(B, t + ATTN_LATENT_ROWS))
             _attn_latent(q[part], kv, indices, indptr, last_page_len, heads, scale, workspace, out[part], None if gate is None else gate[part],
-                         keys, static_table, pos[part], tok_indptr, t)
+                         keys, static_table, pos[part], tok_indptr, t, window, sink)
         return out
-    _attn_latent(q, kv, indices, indptr, last_page_len, heads, scale, workspace, out, gate, keys, static_table, pos, tok_indptr, 0)
+    _attn_latent(q, kv, indices, indptr, last_page_len, heads, scale, workspace, out, gate, keys, static_table, pos, tok_indptr, 0, window, sink)
     return out
 
 
-def _attn_latent(q, kv, indices, indptr, last_page_len, heads, scale, workspace, out, gate, keys, static_table, pos, tok_indptr, first) -> None:
+def _attn_latent(q, kv, indices, indptr, last_page_len, heads, scale, workspace, out, gate, keys, static_table, pos, tok_indptr, first, window, sink) -> None:
     rows = indptr.numel() - 1
     B = rows if pos is None else q.shape[0]
     pages, page, _, width = kv.pool.shape
     assert q.shape == (B, heads * width) and out.shape == (B, heads * kv.rank) and q.stride(1) == 1 and out.stride(1) == 1
     assert workspace.numel() >= int(lib().blitz_attn_latent_workspace_bytes(heads, kv.rank))
     _check(lib().blitz_attn_latent(_p(q), q.stride(0), _p(kv.pool), _p(indices), _p(indptr), _p(last_page_len), _p(pos),
-                                   _p(tok_indptr), rows, first, _p(out), out.stride(0), _p(workspace), B, heads, width, kv.rank, page, pages, scale, *_gate(gate), keys, int(static_table), _p(status_word(q.device)),
+                                   _p(tok_indptr), rows, first, _p(out), out.stride(0), _p(workspace), B, heads, width, kv.rank, page, pages, scale, window, _p(sink), *_gate(gate), keys, int(static_table), _p(status_word(q.device)),
                                    _dt(q), _stream()), "blitz_attn_latent")
 
 
@@ -790,3 +864,59 @@ def gla(q, k, v, g, low, a2, a2_b, norm, state: torch.Tensor, out: torch.Tensor,
                                  longest, heads, dim, vdim, rank, slots, dim ** -0.5, tau, eps, _p(status_word(q.device)),
                                  _stream()), "blitz_gla_chunk")
     return out
+
+
+def wkv(r, k, v, g, low: torch.Tensor, a2, a2_b, bonus, norm, state: torch.Tensor, out: torch.Tensor, pos, tok_indptr, seq_slot, *,
+        rank: int, eps: float, row_lens=None, cum: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Linear attention that sees the state before the token plus the token itself with a bonus, with decays exp(-exp(tanh(low) a2 +
+    a2_b)) from ``low`` [T, >= rank] fp32; then the norm of every head (``norm`` [heads * vdim]) and silu(g).  Otherwise as `gla`."""
+    slots, heads, dim, vdim = state.shape
+    assert low.dtype == torch.float32 and low.stride(1) == 1 and state.dtype == torch.float32 and state.is_contiguous() and out.stride(1) == 1
+    assert all(t.stride(0) == r.stride(0) and t.stride(1) == 1 for t in (k, v, g))
+    longest = 1 if tok_indptr is None else max(row_lens)
+    aligned = all(t.data_ptr() % 16 == 0 for t in (r, k, v, bonus)) and r.stride(0) % 8 == 0 and g.data_ptr() % 4 == 0
+    args = [_p(r), _p(k), _p(v), _p(g), r.stride(0), _p(low), low.stride(0), _p(a2), _p(a2_b), _p(bonus), _p(norm)]
+    if (longest < GLA_CHUNK_MIN_LEN or r.dtype != torch.bfloat16 or not aligned or out.stride(0) % 2 or out.data_ptr() % 4
+            or not lib().blitz_gla_chunk_supported(dim, vdim, rank)):
+        _check(lib().blitz_wkv_recurrent(*args, _p(state), _p(out), out.stride(0), _p(pos), _p(tok_indptr), _p(seq_slot), seq_slot.numel(),
+                                         heads, dim, vdim, rank, slots, eps, int(tok_indptr is not None), _p(status_word(r.device)),
+                                         _dt3(r), _stream()), "blitz_wkv_recurrent")
+        return out
+    n = r.shape[0] * heads * dim
+    if cum is None:
+        cum = torch.empty(n, dtype=torch.float32, device=r.device)
+    assert cum.dtype == torch.float32 and cum.numel() >= n
+    _check(lib().blitz_wkv_chunk(*args, _p(cum), _p(state), _p(out), out.stride(0), _p(pos), _p(tok_indptr), _p(seq_slot), seq_slot.numel(),
+                                 longest, heads, dim, vdim, rank, slots, eps, _p(status_word(r.device)), _stream()), "blitz_wkv_chunk")
+    return out
+
+
+SSD_CHUNK_MIN_LEN = 16
+
+
+def ssd(x, B, C, z, dt, dt_bias, A_log, D, state: torch.Tensor, out: torch.Tensor, pos, tok_indptr, seq_slot, *, groups: int,
+        row_lens=None) -> torch.Tensor:
+    """State-space recurrence with a decay per head over the rows of a step, gated by silu(z); ``state`` [slots, heads, state, vdim]
+    fp32.  x, B, C: column ranges of one buffer; z, dt: of another.  Prompts in bf16 go through the chunked tensor-core kernel."""
+    slots, heads, dim, vdim = state.shape
+    assert state.dtype == torch.float32 and state.is_contiguous() and out.stride(1) == 1
+    assert B.stride(0) == x.stride(0) == C.stride(0) and z.stride(0) == dt.stride(0)
+    args = [_p(x), _p(B), _p(C), x.stride(0), _p(z), _p(dt), z.stride(0), _p(dt_bias), _p(A_log), _p(D), _p(state), _p(out), out.stride(0),
+            _p(pos), _p(tok_indptr), _p(seq_slot), seq_slot.numel(), heads, groups, dim, vdim, slots, _p(status_word(x.device))]
+    longest = 1 if tok_indptr is None else max(row_lens)
+    aligned = all(t.data_ptr() % 16 == 0 for t in (x, B, C)) and x.stride(0) % 8 == 0 and all(t.data_ptr() % 4 == 0 and t.stride(0) % 2 == 0 for t in (z, out))
+    if longest < SSD_CHUNK_MIN_LEN or x.dtype != torch.bfloat16 or not aligned or not lib().blitz_ssd_chunk_supported(dim, vdim):
+        _check(lib().blitz_ssd_recurrent(*args, _dt3(x), _stream()), "blitz_ssd_recurrent")
+    else:
+        _check(lib().blitz_ssd_chunk(*args, _stream()), "blitz_ssd_chunk")
+    return out
+
+
+def part_norm(x: torch.Tensor, w: torch.Tensor, parts: int, eps: float) -> torch.Tensor:
+    """RMS norm of the rows of ``x`` [T, width] in equal parts, each by its own root mean square, in place, times ``w`` [width]."""
+    T, width = x.shape
+    assert x.stride(1) == 1 and w.numel() == width and width % parts == 0
+    for t in range(0, T, 65535):
+        rows = x[t:t + 65535]
+        _check(lib().blitz_part_norm(_p(rows), x.stride(0), _p(w), eps, rows.shape[0], parts, width // parts, _dt3(x), _stream()), "blitz_part_norm")
+    return x

@@ -54,13 +54,13 @@ def _declare(L: ctypes.CDLL) -> None:
             fn.restype = res
 
     sig("blitz_gemm", [c_p, c_i64, c_p, c_i64, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_i64,
-                       c_p, c_i, c_p, c_f, c_i, c_i, c_i, c_p])
+                       c_p, c_i, c_p, c_f, c_f, c_i, c_i, c_i, c_p])
     sig("blitz_gemm_workspace_bytes", [c_i], c_i64)
-    sig("blitz_gemm_decode", [c_p, c_i64, c_p, c_i64, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_f,
+    sig("blitz_gemm_decode", [c_p, c_i64, c_p, c_i64, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_f, c_f,
                               c_p])
     sig("blitz_gemm_decode_supported", [c_i, c_i, c_i, c_i, c_i], c_i)
     sig("blitz_gemm_pair", [c_p, c_i64, c_p, c_i64, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p,
-                            c_i64, c_p, c_i, c_p, c_f, c_p])
+                            c_i64, c_p, c_i, c_p, c_f, c_f, c_p])
     sig("blitz_gemm_pair_supported", [c_i, c_i, c_i, c_i, c_i], c_i)
     sig("blitz_gemm_pair_workspace_bytes", [c_i], c_i64)
     sig("blitz_set_pdl", [c_i], None)
@@ -87,27 +87,27 @@ def _declare(L: ctypes.CDLL) -> None:
     sig("blitz_rope_kv_store", [c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_p, c_i, c_p])
     sig("blitz_attn_decode_workspace_bytes", [c_i, c_i, c_i, c_i], c_i64)
     sig("blitz_attn_decode", [c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f,
-                              c_i, c_i, c_f, c_p, c_p, c_i, c_p, c_i64, c_p, c_i, c_p])
+                              c_i, c_i, c_i, c_i, c_f, c_p, c_p, c_i, c_p, c_i64, c_p, c_i, c_p])
     sig("blitz_attn_prefill_paged", [c_p, c_i64, c_p, c_p, c_p, c_i64, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f,
-                                     c_i, c_i, c_i, c_f, c_p, c_p, c_i, c_p, c_i64, c_p, c_i, c_p])
+                                     c_i, c_i, c_i, c_i, c_i, c_f, c_p, c_p, c_i, c_p, c_i64, c_p, c_i, c_p])
     # models with an fp32 residual stream and recurrent layers
-    sig("blitz_gemm_simt", [c_p, c_i64, c_p, c_i64, c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_i, c_i, c_p])
+    sig("blitz_gemm_simt", [c_p, c_i64, c_p, c_i64, c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_p, c_f, c_f, c_i, c_i, c_i, c_i, c_p])
     sig("blitz_stream_norm", [c_p, c_p, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_p, c_i,
                               c_p])
-    sig("blitz_rope_store", [c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_f, c_i, c_i, c_i, c_i, c_i, c_i, c_i,
+    sig("blitz_rope_store", [c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_f, c_p, c_p, c_p, c_p, c_p, c_f, c_i, c_i, c_i, c_i, c_i, c_i, c_i,
                              c_i, c_i, c_i, c_p, c_i, c_p])
     sig("blitz_stream_mix", [c_p, c_p, c_i, c_i, c_p, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_p, c_p, c_i,
                              c_i, c_i, c_i, c_p, c_i, c_p])
     sig("blitz_norm_store", [c_p, c_p, c_p, c_i64, c_p, c_p, c_f, c_f, c_i, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i,
                              c_p, c_i, c_p])
-    sig("blitz_latent_store", [c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_f, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_i, c_p])
-    sig("blitz_latent_rotate", [c_p, c_i64, c_p, c_i64, c_i, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_p])
+    sig("blitz_latent_store", [c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_f, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_i, c_p])
+    sig("blitz_latent_rotate", [c_p, c_i64, c_p, c_i64, c_i, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
     sig("blitz_attn_latent_supported", [c_i, c_i, c_i, c_i, c_i], c_i)
     sig("blitz_attn_latent_workspace_bytes", [c_i, c_i], c_i64)
-    sig("blitz_attn_latent", [c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_p, c_i64, c_i, c_i, c_p, c_i, c_p])
+    sig("blitz_attn_latent", [c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_p, c_i64, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p, c_p, c_i64, c_i, c_i, c_p, c_i, c_p])
     sig("blitz_latent_gather", [c_p, c_p, c_p, c_i, c_i64, c_i, c_p, c_p])
     sig("blitz_attn_ragged", [c_p, c_i64, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_i,
-                              c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_p, c_i, c_p])
+                              c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_p, c_i, c_p])
     sig("blitz_moe_route", [c_p, c_i64, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_i, c_p, c_i, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p])
     sig("blitz_gemm_grouped", [c_p, c_i64, c_i, c_p, c_p, c_i, c_i, c_i, c_p, c_i, c_i, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i, c_i,
                                c_i, c_i, c_i, c_i, c_i, c_p, c_i, c_p])
@@ -122,6 +122,19 @@ def _declare(L: ctypes.CDLL) -> None:
                               c_p])
     sig("blitz_rglru_scan", [c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_i, c_i,
                              c_i, c_i, c_i, c_i, c_p, c_i, c_p])
+    sig("blitz_stream_rms", [c_p, c_p, c_i, c_i, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_f, c_f, c_p, c_i, c_p,
+                             c_p, c_i, c_p, c_i, c_p, c_p, c_i, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_p, c_i, c_p])
+    sig("blitz_token_conv", [c_p, c_i64, c_p, c_p, c_p, c_p, c_i64, c_i, c_i, c_p, c_i, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i,
+                             c_p, c_i, c_p])
+    sig("blitz_wkv_recurrent", [c_p, c_p, c_p, c_p, c_i64, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i,
+                                c_i, c_i, c_i, c_f, c_i, c_p, c_i, c_p])
+    sig("blitz_wkv_chunk", [c_p, c_p, c_p, c_p, c_i64, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i,
+                            c_i, c_i, c_i, c_i, c_f, c_p, c_p])
+    ssd = [c_p, c_p, c_p, c_i64, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_p]
+    sig("blitz_ssd_recurrent", ssd + [c_i, c_p])
+    sig("blitz_ssd_chunk", ssd + [c_p])
+    sig("blitz_ssd_chunk_supported", [c_i, c_i], c_i)
+    sig("blitz_part_norm", [c_p, c_i64, c_p, c_f, c_i, c_i, c_i, c_i, c_p])
     # comm kernels
     pp = ctypes.POINTER(c_p)
     pi64 = ctypes.POINTER(c_i64)

@@ -5,6 +5,8 @@ of every recurrent run, so the host bookkeeping (native PagePool, SlotPool and B
 are or what shape each has.  A layer that runs several times in one forward pass has one entry per run; a layer that
 reads another layer's keys and values has that layer's pool as its entry.
 
+A mixer that consists of two has the pool of one and the state of the other in its entry.
+
 A pool is one tensor with a key and a value plane per page, or a pair of tensors where keys and values differ in size, or one
 tensor of latent rows.
 
@@ -17,7 +19,7 @@ from typing import List, Optional, Union
 
 import torch
 
-from ..models.hybrid_config import HybridConfig
+from ..models.hybrid_config import HybridConfig, mixer_parts
 from ..ops import KVPair, LatentKV
 
 
@@ -25,8 +27,10 @@ from ..ops import KVPair, LatentKV
 class RunCache:
     # [pages, 2, page, kv_heads, dim], or two [pages, page, kv_heads, size], or latent rows [pages, page, 1, width]
     kv: Optional[Union[torch.Tensor, KVPair, LatentKV]] = None
-    state: Optional[torch.Tensor] = None   # fp32: [slots, heads, dim, vdim] or [slots, width]
+    state: Optional[torch.Tensor] = None   # fp32: [slots, heads, dim, vdim] (keys or state by values) or [slots, width]
     hist: Optional[torch.Tensor] = None    # last inputs of a short convolution: [slots, taps - 1, width]
+    mix_hist: Optional[torch.Tensor] = None  # the same of the convolution of a mixer's input
+    shift: Optional[torch.Tensor] = None   # a mixer's last input: [slots, width]
 
 
 class HybridCache:
@@ -35,25 +39,35 @@ class HybridCache:
         self.runs: List[RunCache] = []
         zeros = lambda *shape: torch.zeros(*shape, dtype=dtype, device=device)
         for r, (m, source) in enumerate(zip(cfg.run_mixers(), cfg.kv_runs())):
-            if m.kind == "attention" and source != r:
-                self.runs.append(RunCache(kv=self.runs[source].kv))
-            elif m.kind == "latent":
-                self.runs.append(RunCache(kv=LatentKV(zeros(num_pages, page_size, 1, m.width), m.kv_rank)))
-            elif m.kind == "attention" and m.vdim != m.dim:
-                self.runs.append(RunCache(kv=KVPair(*(zeros(num_pages, page_size, m.kv_heads, n) for n in (m.dim, m.vdim)))))
-            elif m.kind == "attention":
-                self.runs.append(RunCache(kv=zeros(num_pages, 2, page_size, m.kv_heads, m.dim)))
-            elif m.kind == "gla":
-                self.runs.append(RunCache(state=torch.zeros(num_slots, m.heads, m.dim, m.vdim, device=device)))
-            else:
-                self.runs.append(RunCache(state=torch.zeros(num_slots, m.width, device=device),
-                                          hist=torch.zeros(num_slots, m.taps - 1, m.width, dtype=dtype, device=device)))
+            rc = RunCache()
+            self.runs.append(rc)
+            if cfg.mix_taps:
+                rc.mix_hist = zeros(num_slots, cfg.mix_taps - 1, cfg.hidden)
+            for m in mixer_parts(m):
+                if m.kind == "attention" and source != r:
+                    rc.kv = self.runs[source].kv
+                elif m.kind == "latent":
+                    rc.kv = LatentKV(zeros(num_pages, page_size, 1, m.width), m.kv_rank)
+                elif m.kind == "attention" and m.vdim != m.dim:
+                    rc.kv = KVPair(*(zeros(num_pages, page_size, m.kv_heads, n) for n in (m.dim, m.vdim)))
+                elif m.kind == "attention":
+                    rc.kv = zeros(num_pages, 2, page_size, m.kv_heads, m.dim)
+                elif m.kind in ("gla", "wkv"):
+                    rc.state = torch.zeros(num_slots, m.heads, m.dim, m.vdim, device=device)
+                    if m.kind == "wkv":
+                        rc.shift = zeros(num_slots, m.hidden)
+                elif m.kind == "ssd":
+                    rc.state = torch.zeros(num_slots, m.heads, m.state, m.vdim, device=device)
+                    rc.hist = zeros(num_slots, m.taps - 1, m.channels)
+                else:
+                    rc.state = torch.zeros(num_slots, m.width, device=device)
+                    rc.hist = zeros(num_slots, m.taps - 1, m.width)
 
     def bytes(self) -> int:
         held = {}
         for r in self.runs:
             pools = r.kv if isinstance(r.kv, KVPair) else (r.kv.pool,) if isinstance(r.kv, LatentKV) else (r.kv,)
-            for t in (*pools, r.state, r.hist):
+            for t in (*pools, r.state, r.hist, r.mix_hist, r.shift):
                 if t is not None:
                     held[t.data_ptr()] = t.numel() * t.element_size()
         return sum(held.values())
