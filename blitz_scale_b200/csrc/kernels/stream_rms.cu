@@ -20,7 +20,8 @@
 namespace blitz {
 
 constexpr int kSrMaxStreams = 8;
-constexpr int kSrKeep = 4;  // groups of columns of a thread
+constexpr int kSrKeep = 4;  // groups of columns of u that a thread keeps in registers; further ones are kept in shared memory
+constexpr int kSrThreads = 512;
 
 struct StreamRmsParams {
   const int32_t* ids;       // from_embed
@@ -72,10 +73,11 @@ struct SrCols {
 };
 
 template <typename T, int VEC, int S, bool CONV>
-__global__ void stream_rms_kernel(const StreamRmsParams p) {
+__global__ void __launch_bounds__(kSrThreads) stream_rms_kernel(const StreamRmsParams p) {
   using C = SrCols<T, VEC>;
   using F = SrCols<float, VEC>;
   __shared__ float s_mix[S * S], s_out[S], s_in[S], red[33], red2[33];
+  extern __shared__ __align__(16) float s_keep[];
   ptx::griddep_launch_dependents();
   const T *w = reinterpret_cast<const T*>(p.w), *bias = reinterpret_cast<const T*>(p.bias);
   for (int i = threadIdx.x; i < S * S; i += blockDim.x) {  // weights are not written by kernels still running
@@ -116,10 +118,7 @@ __global__ void stream_rms_kernel(const StreamRmsParams p) {
   }
   F keep[kSrKeep];
   float ss = 0.f;
-#pragma unroll
-  for (int g = 0; g < kSrKeep; ++g) {
-    const int i = threadIdx.x + g * blockDim.x;
-    if (i >= n) continue;
+  auto collect = [&](int i) {
     const int c = i * VEC;
     F x[S];
     if (p.from_embed) {
@@ -173,8 +172,15 @@ __global__ void stream_rms_kernel(const StreamRmsParams p) {
 #pragma unroll
     for (int k = 0; k < VEC; ++k) ss += u.v[k] * u.v[k];
     if (p.u) u.store(p.u + static_cast<int64_t>(t) * p.hidden + c);
-    keep[g] = u;
+    return u;
+  };
+  const int behind = kSrKeep * blockDim.x;
+#pragma unroll
+  for (int g = 0; g < kSrKeep; ++g) {
+    const int i = threadIdx.x + g * blockDim.x;
+    if (i < n) keep[g] = collect(i);
   }
+  for (int i = threadIdx.x + behind; i < n; i += blockDim.x) collect(i).store(s_keep + (i - behind) * VEC);
   if (p.h == nullptr) return;
   const float scale = rsqrtf(block_sum(ss, red) / static_cast<float>(p.hidden) + p.eps);
   const float gain = p.w_step ? 0.f : p.w_offset + ldf<T>(w);
@@ -189,20 +195,17 @@ __global__ void stream_rms_kernel(const StreamRmsParams p) {
       slot = -1;
     }
   }
-#pragma unroll
-  for (int g = 0; g < kSrKeep; ++g) {
-    const int i = threadIdx.x + g * blockDim.x;
-    if (i >= n) continue;
+  auto finish = [&](int i, const F& u) {
     const int c = i * VEC;
     C h;
     if (p.w_step) {
       C a;
       a.load(w + c);
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) h.v[k] = keep[g].v[k] * scale * (p.w_offset + a.v[k]);
+      for (int k = 0; k < VEC; ++k) h.v[k] = u.v[k] * scale * (p.w_offset + a.v[k]);
     } else {
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) h.v[k] = keep[g].v[k] * scale * gain;
+      for (int k = 0; k < VEC; ++k) h.v[k] = u.v[k] * scale * gain;
     }
     if (CONV) {
       h.round();
@@ -240,10 +243,20 @@ __global__ void stream_rms_kernel(const StreamRmsParams p) {
           for (int k = 0; k < VEC; ++k) b.v[k] = h.v[k] + (prev.v[k] - h.v[k]) * b.v[k];
           b.store(out + static_cast<int64_t>(m) * p.hidden + c);
         }
-        continue;
+        return;
       }
     }
     h.store(out + c);
+  };
+#pragma unroll
+  for (int g = 0; g < kSrKeep; ++g) {
+    const int i = threadIdx.x + g * blockDim.x;
+    if (i < n) finish(i, keep[g]);
+  }
+  for (int i = threadIdx.x + behind; i < n; i += blockDim.x) {
+    F u;
+    u.load(s_keep + (i - behind) * VEC);
+    finish(i, u);
   }
 }
 
@@ -274,13 +287,14 @@ int blitz_stream_rms(const int32_t* ids, const void* embed, int vocab, int from_
   const int vec = (hidden & 3) || (y_row & 3) ? 1 : 4, n = hidden / vec;
   int threads = 32;
   while (threads < n && threads < 256) threads <<= 1;
-  while (threads * kSrKeep < n && threads < 1024) threads <<= 1;
-  if (threads * kSrKeep < n) return -1;
+  while (threads * kSrKeep < n && threads < kSrThreads) threads <<= 1;
+  const size_t smem = threads * kSrKeep < n ? (size_t)(n - threads * kSrKeep) * vec * sizeof(float) : 0;
+  if (smem > 40 * 1024) return -1;
   auto go = [&](auto type, auto v, auto s) -> cudaError_t {
     using T = decltype(type);
     constexpr int V = decltype(v)::value, S = decltype(s)::value;
-    return conv ? launch_pdl(stream_rms_kernel<T, V, S, true>, dim3(tokens), dim3(threads), 0, stream, p)
-                : launch_pdl(stream_rms_kernel<T, V, S, false>, dim3(tokens), dim3(threads), 0, stream, p);
+    return conv ? launch_pdl(stream_rms_kernel<T, V, S, true>, dim3(tokens), dim3(threads), smem, stream, p)
+                : launch_pdl(stream_rms_kernel<T, V, S, false>, dim3(tokens), dim3(threads), smem, stream, p);
   };
   auto wide = [&](auto type, auto s) -> cudaError_t {
     return vec == 4 ? go(type, std::integral_constant<int, 4>{}, s) : go(type, std::integral_constant<int, 1>{}, s);

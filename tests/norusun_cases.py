@@ -37,7 +37,7 @@ def dense(ff=136, limit=1.5):
     return {"kind": "dense", "ff": ff, "limit": limit}
 
 
-def config(mixers, mlps, width=200, vocab=211, eps=0.02, streams=3, taps=4) -> dict:
+def config(mixers, mlps, width=200, vocab=211, eps=0.06, streams=3, taps=4) -> dict:
     out = {"architecture": "Norusun", "canon": {"taps": taps}, "norm": {"eps": eps}, "vocab": vocab, "width": width, "streams": streams,
            "layers": [{"type": kind, "mixer": m, "mlp": f} for (kind, m, _), f in zip(mixers, mlps)]}
     out = json.loads(json.dumps(out))
@@ -60,18 +60,18 @@ def weights(c: dict, seed: int = 11, dtype=torch.bfloat16) -> Dict[str, torch.Te
         p, m, f, q = f"l{i}.mix.", L["mixer"], L["mlp"], f"l{i}.mlp."
         for k in (1, 2) if f else (1,):
             w[f"l{i}.norm{k}"] = one()
-            w[f"l{i}.hc{k}.in"] = 1.0 / S + 0.4 * r(S)
-            w[f"l{i}.hc{k}.out"] = 0.8 + 0.5 * r(S)
-            w[f"l{i}.hc{k}.mix"] = 0.7 * torch.eye(S) + 0.35 * r(S, S)
-        w[f"l{i}.canon1"] = 0.45 * r(H, taps)
+            w[f"l{i}.hc{k}.in"] = 1.0 / S + 0.25 * r(S)
+            w[f"l{i}.hc{k}.out"] = 0.8 + 0.3 * r(S)
+            w[f"l{i}.hc{k}.mix"] = 0.8 * torch.eye(S) + 0.25 * r(S, S)
+        w[f"l{i}.canon1"] = 0.3 * r(H, taps)
         if L["type"] == "wkv":
             n = m["heads"] * m["dim"]
             for s in "rkvgw":
                 w[p + "mu." + s] = 0.5 + 0.4 * r(H)
             for s in "rkvg":
-                w[p + s] = 1.3 * lin(n, H)
+                w[p + s] = lin(n, H)
             w[p + "w1"], w[p + "w2"], w[p + "w0"] = 1.5 * lin(rank, H), 1.5 * lin(n, rank), -1.5 + 0.8 * r(n)
-            w[p + "u"], w[p + "norm"], w[p + "o"] = 0.5 + 1.2 * r(m["heads"], m["dim"]), 1.0 + 0.3 * r(n), 1.5 * lin(H, n)
+            w[p + "u"], w[p + "norm"], w[p + "o"] = 0.5 + 1.2 * r(m["heads"], m["dim"]), 1.0 + 0.3 * r(n), lin(H, n)
         elif L["type"] == "latent_attention":
             h, d, rd = m["heads"], m["dim"], m["rot_dim"]
             w[p + "dq"], w[p + "dkv"] = lin(m["q_rank"], H), 1.5 * lin(m["kv_rank"] + rd, H)

@@ -276,14 +276,18 @@ MIXERS = {"wkv": wkv, "latent_attention": latent_attention, "parallel": side_by_
 
 
 class Plain:
-    def __init__(self, config: dict, weights: Dict[str, torch.Tensor], dtype=torch.float64, flaws=()):
-        self.c, self.dtype, self.flaws = config, dtype, tuple(flaws)
+    """`rounded`: a shorter type that what enters and leaves every sublayer is rounded to, for an idea of how much rounding alone
+    changes a position's logits."""
+
+    def __init__(self, config: dict, weights: Dict[str, torch.Tensor], dtype=torch.float64, flaws=(), rounded=None):
+        self.c, self.dtype, self.flaws, self.rounded = config, dtype, tuple(flaws), rounded
         assert all(f in FLAWS for f in self.flaws)
         self.w = {n: t.to(dtype) for n, t in weights.items()}
 
     def run(self, tokens: List[int], keep: Optional[list] = None) -> torch.Tensor:
         """Logits at every position; `keep` collects the sum of the streams after every layer."""
         c, eps, fl = self.c, self.c["norm"]["eps"], self.flaws
+        short = lambda t: t if self.rounded is None else t.to(self.rounded).to(t.dtype)
         x = self.w["embed"][torch.tensor(tokens)]
         xs = torch.stack([x] * c["streams"])
         for i, L in enumerate(c["layers"]):
@@ -293,14 +297,14 @@ class Plain:
                 if q == 2 and not L.get("mlp"):
                     continue
                 hc = {n: self.w[f"l{i}.hc{q}.{n}"] for n in ("in", "out", "mix")}
-                h = scalar_norm(streams_in(xs, hc["in"], fl), self.w[f"l{i}.norm{q}"], eps, fl)
+                h = short(scalar_norm(streams_in(xs, hc["in"], fl), self.w[f"l{i}.norm{q}"], eps, fl))
                 if q == 2:
                     y = clamped_ff(h, mlp, L["mlp"]["limit"], fl)
                 else:
                     conv = causal_conv(h, self.w[f"l{i}.canon1"], fl)
-                    h = conv if "conv_no_residual" in fl else h + conv
+                    h = short(conv if "conv_no_residual" in fl else h + conv)
                     y = MIXERS[L["type"]](h, mix, L["mixer"], eps, fl)
-                xs = streams_out(xs, hc["mix"], hc["out"], y, fl)
+                xs = streams_out(xs, hc["mix"], hc["out"], short(y), fl)
             if keep is not None:
                 keep.append(xs.sum(0))
         x = xs[-1] if "last_stream_only" in fl else xs.sum(0)
