@@ -165,14 +165,16 @@ def main():
                     "and a mixture of experts (bench/komulorn_bench.py; one GPU)")
     ap.add_argument("--vofidra", action="store_true", help="instead: the same for the Vofidra design, several residual streams, latent "
                     "attention and experts with identity experts (bench/vofidra_bench.py; one GPU)")
+    ap.add_argument("--norusun", action="store_true", help="instead: the same for the Norusun design, linear attention, latent attention in "
+                    "a window, sigmoid attention in chunks beside a state space (bench/norusun_bench.py; one GPU)")
     ap.add_argument("--hybrid-part", default="all", choices=["all", "models", "kernels"])
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm()
-    if args.hybrid or args.komulorn or args.vofidra:
+    if args.hybrid or args.komulorn or args.vofidra or args.norusun:
         sys.path.insert(0, os.path.join(ROOT, "bench"))
         import importlib
-        module = "vofidra_bench" if args.vofidra else "komulorn_bench" if args.komulorn else "hybrid_bench"
+        module = next((n + "_bench" for n in ("norusun", "vofidra", "komulorn") if getattr(args, n)), "hybrid_bench")
         sampler = ClockSampler(0)
         sampler.start()
         result = importlib.import_module(module).run(args.hybrid_part)

@@ -87,9 +87,9 @@ def bench_models(out, sizes=("h4096", "h2048"), configs=configs):
                     for x in (s.mixer for s in cfg.layer_specs if s.mixer.kind == "latent"):
                         weights -= 2 * x.heads * (x.width * x.qdim + x.kv_rank * x.vdim)      # of prompts only
                     # window and kept tokens of the attention layers; states are read and written
-                    kv = sum(x.kv_heads * (x.dim + x.vdim) * 2 * (min(ctx, x.window + x.keep_first) if x.window else ctx)
-                             for x in cfg.run_mixers() if x.kind == "attention")
-                    kv += sum(x.width * 2 * ctx for x in cfg.run_mixers() if x.kind == "latent")
+                    seen = lambda x: ctx if not x.window else ctx % x.window + 1 if x.chunked else min(ctx, x.window + x.keep_first)
+                    kv = sum(x.kv_heads * (x.dim + x.vdim) * 2 * seen(x) for x in cfg.run_parts() if x.kind == "attention")
+                    kv += sum(x.width * 2 * min(ctx, x.window or ctx) for x in cfg.run_mixers() if x.kind == "latent")
                     data = B * (kv + 2 * cfg.state_bytes_per_sequence())
                 else:
                     data = B * ctx * cfg.kv_bytes_per_token()

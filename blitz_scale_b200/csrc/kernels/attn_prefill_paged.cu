@@ -46,8 +46,9 @@
 // neighbouring words.  Blocks whose every distance is beyond the table share its last entry, which moves the reference.
 //
 // The window may be a chunk counted from position 0 (`chunked`): a row sees the keys of its own chunk.  Weights may be sigmoids of
-// the scores (template parameter SIG; EXT with it): no maximum, no row sum, no rescaling.  sigmoid(x) = 1 / (1 + e^-x); two
-// neighbours share a reciprocal, 1 / a = b / (a b), with e^-x held below 2^60 (a weight below that is zero next to any other).
+// the scores (template parameter SIG; EXT with it): no maximum, no row sum, no rescaling.  sigmoid(x) = 1 / (1 + e^-x); four
+// neighbours share a reciprocal, 1 / a = b (c d) / (a b c d), unless a product of some four leaves the range of fp32 (one vote per
+// half a block).
 //
 // Replaces FlashInfer's BatchPrefillWithRaggedKVCacheWrapper / paged wrapper calls and their host Plan()
 // (src/kernel/attention_prefill.cu:11-45, src/kernel/flashinfer_types.cu:24-49).
@@ -391,6 +392,63 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         }
         pp_trace(p, tracer, t, j, 1);
         ptx::tc_fence_after_sync();
+        if constexpr (SIG) {
+          const int kv0 = it.block(j) * kPpTile, row0 = it.prefix + it.q0 + t * kPpTile;
+          // the block's visible keys, of this row and of all rows of the tile
+          const int from = p.window > 0 ? chunk_from >= 0 ? chunk_from : limit - p.window + 1 : 0;
+          const int lo = from - kv0, hi = limit - kv0, last = row0 + kPpTile - 1;
+          const bool early = p.window > 0 && kv0 < (p.chunked ? last / p.window * p.window : last - p.window + 1);  // keys before some row's first
+          const bool masked = kv0 + kPpTile - 1 > row0 || early;
+          const uint64_t scale2 = ptx::f32x2(-p.scale_log2, -p.scale_log2), bias2 = ptx::f32x2(sig_bias, sig_bias),
+                         one2 = ptx::f32x2(1.f, 1.f);
+          auto weights = [&](auto&& hidden) {
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {  // 64 scores -> 32 columns of pairs
+              uint32_t v[2][32], pk[32];
+              ptx::tmem_ld_32x32(tS + h * 64, v[0]);
+              ptx::tmem_ld_32x32(tS + h * 64 + 32, v[1]);
+              ptx::tmem_ld_wait();
+              // 1 + e^-x of scores c and c + 1
+              auto denominators = [&](int c) {
+                const int k = c - h * 64;
+                const float2 x = ptx::f32x2_get(
+                    ptx::fma_f32x2(ptx::f32x2(__uint_as_float(v[k >> 5][k & 31]), __uint_as_float(v[k >> 5][(k & 31) + 1])), scale2, bias2));
+                return ptx::fma_f32x2(ptx::f32x2(ptx::ex2_approx(x.x), ptx::ex2_approx(x.y)), one2, one2);
+              };
+              float smallest = 1.f;
+#pragma unroll
+              for (int i = 0; i < 32; i += 2) {
+                const int c = h * 64 + 2 * i;
+                const uint64_t ab = denominators(c), cd = denominators(c + 2);
+                const float2 f = ptx::f32x2_get(ab), g = ptx::f32x2_get(cd);
+                const float fp = f.x * f.y, gp = g.x * g.y, r = ptx::rcp_approx(fp * gp);
+                smallest = fminf(smallest, r);
+                const float rf = r * gp, rg = r * fp;
+                const float2 w = ptx::f32x2_get(ptx::mul_f32x2(ptx::f32x2(f.y, f.x), ptx::f32x2(rf, rf)));
+                const float2 z = ptx::f32x2_get(ptx::mul_f32x2(ptx::f32x2(g.y, g.x), ptx::f32x2(rg, rg)));
+                pk[i] = pk2<T>(hidden(c) ? 0.f : w.x, hidden(c + 1) ? 0.f : w.y);
+                pk[i + 1] = pk2<T>(hidden(c + 2) ? 0.f : z.x, hidden(c + 3) ? 0.f : z.y);
+              }
+              if (__any_sync(0xffffffffu, !(smallest > 1e-36f))) {  // a product left the range: one reciprocal each
+#pragma unroll
+                for (int i = 0; i < 32; ++i) {
+                  const int c = h * 64 + 2 * i;
+                  const float2 d = ptx::f32x2_get(denominators(c));
+                  pk[i] = pk2<T>(hidden(c) ? 0.f : ptx::rcp_approx(d.x), hidden(c + 1) ? 0.f : ptx::rcp_approx(d.y));
+                }
+              }
+              ptx::tmem_st_32x32(tS + h * 32, pk);
+            }
+          };
+          if (!masked) weights([](int) { return false; });
+          else if (!early) weights([&](int i) { return i > hi; });
+          else weights([&](int i) { return i > hi || i < lo; });
+          ptx::tmem_st_wait();
+          ptx::tc_fence_before_sync();
+          ptx::mbar_arrive(&p_ready[t]);
+          l = 1.f;
+          continue;
+        }
         uint32_t v0[32], v1[32], v2[32], v3[32];  // the row's 128 scores (fp32 bits)
         ptx::tmem_ld_32x32(tS, v0);
         ptx::tmem_ld_32x32(tS + 32, v1);
@@ -410,31 +468,6 @@ attn_prefill_paged_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         auto visible = [&](int i) {  // key i of the block to this row
           return kv0 + i <= limit && (!EXT || kv0 + i >= from || kv0 + i < p.keep_first);
         };
-        if constexpr (SIG) {
-          const float neg_scale = -p.scale_log2;
-          auto weights = [&](auto&& hidden) {
-#pragma unroll
-            for (int h = 0; h < 2; ++h) {
-              uint32_t pk[32];
-#pragma unroll
-              for (int i = 0; i < 32; ++i) {
-                const int c = h * 64 + 2 * i;
-                const float a = 1.f + ptx::ex2_approx(fminf(fmaf(__uint_as_float(score(c)), neg_scale, sig_bias), 60.f));
-                const float b = 1.f + ptx::ex2_approx(fminf(fmaf(__uint_as_float(score(c + 1)), neg_scale, sig_bias), 60.f));
-                const float r = __fdividef(1.f, a * b);
-                pk[i] = pk2<T>(hidden(c) ? 0.f : b * r, hidden(c + 1) ? 0.f : a * r);
-              }
-              ptx::tmem_st_32x32(tS + h * 32, pk);
-            }
-          };
-          if (masked) weights([&](int i) { return !visible(i); });
-          else weights([](int) { return false; });
-          ptx::tmem_st_wait();
-          ptx::tc_fence_before_sync();
-          ptx::mbar_arrive(&p_ready[t]);
-          l = 1.f;
-          continue;
-        }
         const bool capped = EXT && p.cap_log2 > 0.f;
         float bias = 0.f;  // of every score of the block, in log2 units
         if (near) {
@@ -650,7 +683,7 @@ int blitz_attn_prefill_paged(const void* q, int64_t q_stride, const void* k_pool
   if (dim < 8 || dim > 128 || (dim & 7) || vdim < 8 || vdim > 128 || (vdim & 7)) return -1;
   if (kv_heads < 1 || (q_heads % kv_heads) != 0 || (out_stride & 7) || (q_stride & 7)) return -1;
   if (window < 0 || keep_first < 0 || softcap < 0.f) return -1;
-  if ((chunked && (window < 1 || keep_first)) || (sigmoid && (sink || softcap > 0.f || (bias && bias_len != 1)))) return -1;
+  if ((chunked && (window < 1 || keep_first)) || (sigmoid && (sink || softcap > 0.f || keep_first || (bias && bias_len != 1)))) return -1;
   if (page_size < 8 || (page_size & (page_size - 1)) != 0 || page_rows < page_size || work == nullptr) return -1;
   if ((reinterpret_cast<uintptr_t>(work) & 15) != 0 || (reinterpret_cast<uintptr_t>(out) & 15) != 0) return -1;
   const int bt = page_size < 64 ? page_size : 64;

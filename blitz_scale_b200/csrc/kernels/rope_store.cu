@@ -37,7 +37,7 @@ struct RopeStoreParams {
 enum RopeMode : int { kRopeAny = 0, kRopeWidePairs = 1, kRopeWideHalves = 2 };  // wide: eight elements per access
 
 template <typename T, int MODE, bool NORM>
-__global__ void __launch_bounds__(256, MODE == kRopeAny ? 5 : 4) rope_store_kernel(const RopeStoreParams p) {
+__global__ void __launch_bounds__(NORM && MODE == kRopeWideHalves ? 1024 : 256, NORM && MODE == kRopeWideHalves ? 1 : MODE == kRopeAny ? 5 : 4) rope_store_kernel(const RopeStoreParams p) {
   ptx::griddep_launch_dependents();
   ptx::griddep_wait();
   extern __shared__ float s_ang[];  // [rot_dims / 2] cos, [rot_dims / 2] sin
@@ -59,8 +59,8 @@ __global__ void __launch_bounds__(256, MODE == kRopeAny ? 5 : 4) rope_store_kern
   const int heads = p.q_heads + (s >= 0 ? p.kv_heads : 0);
   const T *q_w = reinterpret_cast<const T*>(p.q_w), *k_w = reinterpret_cast<const T*>(p.k_w);
   float q_f = 1.f, k_f = 1.f;
-  if (NORM) {
-    __shared__ float red[2][33];
+  __shared__ float red[2][33];
+  if (NORM && MODE != kRopeWideHalves) {
     auto squares = [&](const T* x, int n) {
       float ss = 0.f;
       if (MODE != kRopeAny) {
@@ -107,7 +107,7 @@ __global__ void __launch_bounds__(256, MODE == kRopeAny ? 5 : 4) rope_store_kern
 #pragma unroll
         for (int j = 0; j < 8; ++j) x[j] += b[j];
       }
-      if (NORM && src != p.v) {
+      if (NORM && MODE != kRopeWideHalves) {
         const bool is_q = src == q;
         float w[8];
         ldf8<T>((is_q ? q_w : k_w) + at, w);
@@ -165,6 +165,28 @@ __global__ void __launch_bounds__(256, MODE == kRopeAny ? 5 : 4) rope_store_kern
         if (m.c < turns) load8(m.is_q ? q : k, m.is_q ? q_b : k_b, first(m) + half, v);
       };
       request();
+      if (NORM) {  // every thread has one item at most (see the launch): its values are what the norms are taken over
+        float ss = 0.f;
+        if (m.on) {
+#pragma unroll
+          for (int j = 0; j < 8; ++j) ss += u[j] * u[j] + (m.c < turns ? v[j] * v[j] : 0.f);
+        }
+        q_f = rsqrtf(block_sum(m.is_q ? ss : 0.f, red[0]) / static_cast<float>(p.q_heads * p.dim) + p.eps);
+        if (p.k) k_f = rsqrtf(block_sum(m.is_q ? 0.f : ss, red[1]) / static_cast<float>(p.kv_heads * p.dim) + p.eps);
+        if (m.on) {
+          const float f = m.is_q ? q_f : k_f;
+          const T* w = (m.is_q ? q_w : k_w) + first(m);
+          float a[8];
+          ldf8<T>(w, a);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) u[j] *= f * a[j];
+          if (m.c < turns) {
+            ldf8<T>(w + half, a);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] *= f * a[j];
+          }
+        }
+      }
       angles();
       for (int it = threadIdx.x; it < items; it += blockDim.x) {
         if (it != static_cast<int>(threadIdx.x)) {
@@ -289,7 +311,10 @@ int blitz_rope_store(void* q, const void* k, const void* v, const void* q_b, con
   bool wide = ((dim | vdim | row) & 7) == 0 && (interleaved || (rot_dims & 15) == 0);
   for (const void* x : {(const void*)q, k, v, q_b, k_b, v_b, q_w, k_w, (const void*)k_pool, (const void*)v_pool})
     wide = wide && (reinterpret_cast<uintptr_t>(x) % al) == 0;
-  const dim3 grid(num_tokens), block(wide && (q_heads + kv_heads) * dim <= 2048 ? 128 : 256);
+  const int items = (q_heads + (k ? kv_heads : 0)) * (rot_dims / 16 + (dim - rot_dims) / 8);  // of the wide half-split form
+  if (q_w && !interleaved && items > 1024) wide = false;
+  const int one_each = q_w && wide && !interleaved ? (items + 31) / 32 * 32 : 0;
+  const dim3 grid(num_tokens), block(one_each ? one_each : wide && (q_heads + kv_heads) * dim <= 2048 ? 128 : 256);
   const size_t smem = (size_t)rot_dims * sizeof(float);
   auto go = [&](auto type, auto norm) {
     using T = decltype(type);

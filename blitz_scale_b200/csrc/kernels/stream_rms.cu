@@ -16,6 +16,7 @@
 #include "launch.cuh"
 #include "ptx.cuh"
 #include "scalar.cuh"
+#include "tmap.cuh"
 
 namespace blitz {
 
@@ -72,14 +73,46 @@ struct SrCols {
   }
 };
 
+// Columns as they lie in memory.
+template <typename T, int VEC>
+struct alignas(VEC * sizeof(T)) SrRaw {
+  T e[VEC];
+};
+
+// What the convolution reads beside the token's row, requested before the norm is known: up to kSrTaps taps and kSrMixes mixes.
+constexpr int kSrTaps = 4, kSrMixes = 5;
+template <typename T, int VEC>
+struct SrEarly {
+  SrRaw<T, VEC> conv[kSrTaps], hist[kSrTaps - 1], mu[kSrMixes], prev;  // taps and history end at the last place
+};
+
 template <typename T, int VEC, int S, bool CONV>
-__global__ void __launch_bounds__(kSrThreads) stream_rms_kernel(const StreamRmsParams p) {
+__global__ void __launch_bounds__(kSrThreads, 1) stream_rms_kernel(const StreamRmsParams p) {
   using C = SrCols<T, VEC>;
   using F = SrCols<float, VEC>;
   __shared__ float s_mix[S * S], s_out[S], s_in[S], red[33], red2[33];
   extern __shared__ __align__(16) float s_keep[];
   ptx::griddep_launch_dependents();
   const T *w = reinterpret_cast<const T*>(p.w), *bias = reinterpret_cast<const T*>(p.bias);
+  constexpr int kKeep = CONV ? 2 : kSrKeep;
+  const bool ahead = CONV && p.taps <= kSrTaps && p.mixes <= kSrMixes;
+  using Raw = SrRaw<T, VEC>;
+  SrEarly<T, VEC> early[CONV ? kKeep : 1];
+  auto raw = [](const void* base, int64_t at) { return *reinterpret_cast<const Raw*>(reinterpret_cast<const T*>(base) + at); };
+  if (CONV && ahead) {
+#pragma unroll
+    for (int g = 0; g < kKeep; ++g) {
+      const int c = (threadIdx.x + g * blockDim.x) * VEC;
+      SrEarly<T, VEC>& e = early[CONV ? g : 0];
+      if (c >= p.hidden) continue;
+#pragma unroll
+      for (int j = 0; j < kSrTaps; ++j)
+        if (j >= kSrTaps - p.taps) e.conv[j] = raw(p.conv, static_cast<int64_t>(j - (kSrTaps - p.taps)) * p.hidden + c);
+#pragma unroll
+      for (int m = 0; m < kSrMixes; ++m)
+        if (m < p.mixes) e.mu[m] = raw(p.mu, static_cast<int64_t>(m) * p.hidden + c);
+    }
+  }
   for (int i = threadIdx.x; i < S * S; i += blockDim.x) {  // weights are not written by kernels still running
     if (p.mix) s_mix[i] = ldf<T>(reinterpret_cast<const T*>(p.mix) + i);
     if (i < S) {
@@ -97,6 +130,28 @@ __global__ void __launch_bounds__(kSrThreads) stream_rms_kernel(const StreamRmsP
     const int id = p.ids[src];
     if (id >= 0 && id < p.vocab) er = reinterpret_cast<const T*>(p.embed) + static_cast<int64_t>(id) * p.hidden;
     else if (p.status && threadIdx.x == 0) atomicCAS(p.status, 0, kStatusBadIndex);
+  }
+  int slot = -1, at = 0;
+  if (CONV) {
+    slot = p.seq_slot[t];
+    at = p.pos[t];
+    if (slot >= p.num_slots) {
+      if (p.status && threadIdx.x == 0) atomicCAS(p.status, 0, kStatusBadIndex);
+      slot = -1;
+    }
+  }
+  if (CONV && ahead && slot >= 0) {
+#pragma unroll
+    for (int g = 0; g < kKeep; ++g) {
+      const int c = (threadIdx.x + g * blockDim.x) * VEC;
+      SrEarly<T, VEC>& e = early[CONV ? g : 0];
+      if (c >= p.hidden) continue;
+#pragma unroll
+      for (int j = 0; j + 1 < kSrTaps; ++j)
+        if (j >= kSrTaps - p.taps)
+          e.hist[j] = raw(p.hist, (static_cast<int64_t>(slot) * (p.taps - 1) + j - (kSrTaps - p.taps)) * p.hidden + c);
+      if (p.mixes > 0 && at > 0) e.prev = raw(p.shift, static_cast<int64_t>(slot) * p.hidden + c);
+    }
   }
   const T* y0 = p.y ? reinterpret_cast<const T*>(p.y) + src * p.y_row : nullptr;
   const T* y1 = p.y1 ? reinterpret_cast<const T*>(p.y1) + src * p.y_row : nullptr;
@@ -116,7 +171,7 @@ __global__ void __launch_bounds__(kSrThreads) stream_rms_kernel(const StreamRmsP
     f0 = 0.5f * rsqrtf(block_sum(a, red) / static_cast<float>(p.hidden) + p.eps);
     f1 = 0.5f * rsqrtf(block_sum(b, red2) / static_cast<float>(p.hidden) + p.eps);
   }
-  F keep[kSrKeep];
+  F keep[kKeep];
   float ss = 0.f;
   auto collect = [&](int i) {
     const int c = i * VEC;
@@ -174,9 +229,9 @@ __global__ void __launch_bounds__(kSrThreads) stream_rms_kernel(const StreamRmsP
     if (p.u) u.store(p.u + static_cast<int64_t>(t) * p.hidden + c);
     return u;
   };
-  const int behind = kSrKeep * blockDim.x;
+  const int behind = kKeep * blockDim.x;
 #pragma unroll
-  for (int g = 0; g < kSrKeep; ++g) {
+  for (int g = 0; g < kKeep; ++g) {
     const int i = threadIdx.x + g * blockDim.x;
     if (i < n) keep[g] = collect(i);
   }
@@ -186,17 +241,45 @@ __global__ void __launch_bounds__(kSrThreads) stream_rms_kernel(const StreamRmsP
   const float gain = p.w_step ? 0.f : p.w_offset + ldf<T>(w);
   const int per = CONV && p.mixes > 0 ? p.mixes : 1;
   T* out = reinterpret_cast<T*>(p.h) + static_cast<int64_t>(t) * per * p.hidden;
-  int slot = -1, at = 0;
-  if (CONV) {
-    slot = p.seq_slot[t];
-    at = p.pos[t];
-    if (slot >= p.num_slots) {
-      if (p.status && threadIdx.x == 0) atomicCAS(p.status, 0, kStatusBadIndex);
-      slot = -1;
+  auto convolved = [&](int c, C h, const SrEarly<T, VEC>& e) {
+    h.round();
+    const C now = h;
+    auto add = [&](const Raw& a, const Raw& b) {
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) h.v[k] += ldf<T>(&a.e[k]) * ldf<T>(&b.e[k]);
+    };
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) h.v[k] += ldf<T>(&e.conv[kSrTaps - 1].e[k]) * now.v[k];
+    if (slot >= 0) {
+      T* hist = reinterpret_cast<T*>(p.hist) + static_cast<int64_t>(slot) * (p.taps - 1) * p.hidden + c;
+#pragma unroll
+      for (int j = 0; j + 1 < kSrTaps; ++j) {
+        const int first = kSrTaps - p.taps;
+        if (j < first) continue;
+        if (kSrTaps - 1 - j <= at) add(e.conv[j], e.hist[j]);
+        if (j > first) *reinterpret_cast<Raw*>(hist + static_cast<int64_t>(j - first - 1) * p.hidden) = e.hist[j];
+      }
+      if (p.taps > 1) now.store(hist + static_cast<int64_t>(p.taps - 2) * p.hidden);
     }
-  }
-  auto finish = [&](int i, const F& u) {
-    const int c = i * VEC;
+    if (p.mixes == 0) {
+      h.store(out + c);
+      return;
+    }
+    h.round();
+    float d[VEC];
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) d[k] = (slot >= 0 && at > 0 ? ldf<T>(&e.prev.e[k]) : 0.f) - h.v[k];
+    if (slot >= 0) h.store(reinterpret_cast<T*>(p.shift) + static_cast<int64_t>(slot) * p.hidden + c);
+#pragma unroll
+    for (int m = 0; m < kSrMixes; ++m) {
+      if (m >= p.mixes) continue;
+      C b;
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) b.v[k] = h.v[k] + d[k] * ldf<T>(&e.mu[m].e[k]);
+      b.store(out + static_cast<int64_t>(m) * p.hidden + c);
+    }
+  };
+  auto normed = [&](int c, const F& u) {
     C h;
     if (p.w_step) {
       C a;
@@ -207,6 +290,9 @@ __global__ void __launch_bounds__(kSrThreads) stream_rms_kernel(const StreamRmsP
 #pragma unroll
       for (int k = 0; k < VEC; ++k) h.v[k] = u.v[k] * scale * gain;
     }
+    return h;
+  };
+  auto finish = [&](int c, C h) {
     if (CONV) {
       h.round();
       const T* conv = reinterpret_cast<const T*>(p.conv) + c;
@@ -249,14 +335,17 @@ __global__ void __launch_bounds__(kSrThreads) stream_rms_kernel(const StreamRmsP
     h.store(out + c);
   };
 #pragma unroll
-  for (int g = 0; g < kSrKeep; ++g) {
+  for (int g = 0; g < kKeep; ++g) {
     const int i = threadIdx.x + g * blockDim.x;
-    if (i < n) finish(i, keep[g]);
+    if (i >= n) continue;
+    const C h = normed(i * VEC, keep[g]);
+    if (CONV && ahead) convolved(i * VEC, h, early[CONV ? g : 0]);
+    else finish(i * VEC, h);
   }
   for (int i = threadIdx.x + behind; i < n; i += blockDim.x) {
     F u;
     u.load(s_keep + (i - behind) * VEC);
-    finish(i, u);
+    finish(i * VEC, normed(i * VEC, u));
   }
 }
 
@@ -286,9 +375,11 @@ int blitz_stream_rms(const int32_t* ids, const void* embed, int vocab, int from_
                     eps, w_offset, hidden, vocab, row_offset, from_embed, write, w_step, taps, mixes, num_slots, status};
   const int vec = (hidden & 3) || (y_row & 3) ? 1 : 4, n = hidden / vec;
   int threads = 32;
-  while (threads < n && threads < 256) threads <<= 1;
-  while (threads * kSrKeep < n && threads < kSrThreads) threads <<= 1;
-  const size_t smem = threads * kSrKeep < n ? (size_t)(n - threads * kSrKeep) * vec * sizeof(float) : 0;
+  // few tokens: as many threads as there are groups
+  while (threads < n && threads < (tokens <= 2 * device_sm_count() ? kSrThreads : 256)) threads <<= 1;
+  const int keep = conv ? 2 : kSrKeep;
+  while (threads * keep < n && threads < kSrThreads) threads <<= 1;
+  const size_t smem = threads * keep < n ? (size_t)(n - threads * keep) * vec * sizeof(float) : 0;
   if (smem > 40 * 1024) return -1;
   auto go = [&](auto type, auto v, auto s) -> cudaError_t {
     using T = decltype(type);
