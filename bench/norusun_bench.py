@@ -180,11 +180,6 @@ def bench_kernels(out, size):
         by, fl = 2.0 * (4 * M * H + 4 * H * n + 4 * M * n), 8.0 * M * H * n
         t = timeit(lambda i: ops.gemm(a5[:, :4 * H], ws[i], out=o4, groups=4, static_b=True), copies=nc)
         rep("gemm of four mixes (block-diagonal)", t, by=by, fl=fl, M=M)
-        if M <= ops.PAIR_GEMM_MAX_M:
-            def four(i):
-                for k in range(4):
-                    ops.gemm(a5[:, k * H:(k + 1) * H], ws[i][k * H:(k + 1) * H], out=o4[:, k * n:(k + 1) * n], static_b=True)
-            rep("gemm of four mixes (one by one)", timeit(four, copies=nc), by=by, fl=fl, M=M)
         wide = [w_.view(H, 4 * n) for w_ in ws]
         t = timeit(lambda i: ops.gemm(a, wide[i], out=o4, static_b=True), copies=nc)
         rep("gemm store, as many columns (uniform model)", t, by=2.0 * (M * H + 4 * H * n + 4 * M * n), fl=fl, M=M)
@@ -198,7 +193,8 @@ def bench_kernels(out, size):
     a2, a2b, gn = rnd(gr, gh * gd) * gr ** -0.5, 2 + rnd(gh * gd), rnd(gv)
     gw = 2 * gh * gd + 2 * gh * gv + gr
     gcut = lambda x: x.split([gh * gd, gh * gd, gh * gv, gh * gv, gr], 1)
-    w2, w0, bonus, on = rnd(rank, n) * rank ** -0.5, -2 + rnd(n), rnd(n), rnd(n)
+    w2, w0, bonus, on = rnd(rank, n) * rank ** -0.5, -2.5 + 0.5 * rnd(n), rnd(n), rnd(n)
+    w3 = w0 + 3
     for lens in ([8192], [2048] * 4, [256] * 32):
         T, B = sum(lens), len(lens)
         pos, indptr, slots = i32([p for k in lens for p in range(k)]), i32([sum(lens[:i]) for i in range(B + 1)]), torch.arange(B, dtype=torch.int32, device=dev)
@@ -208,6 +204,8 @@ def bench_kernels(out, size):
         rep("gla prompts (Fafudra)", t, by=T * 2.0 * (gw + gh * gv) + B * gh * gd * gv * 8.0, fl=T * gh * (4.0 * gd * gv + 64.0 * (gd + gv)), sequences=B, length=lens[0])
         x, low, o, st = rnd(T, 4 * n), torch.randn(T, rank, device=dev), torch.empty(T, n, dtype=bf, device=dev), torch.zeros(B, wh, wd, wd, device=dev)
         t = timeit(lambda i: ops.wkv(*x.split(n, 1), low, w2, w0, bonus, on, st, o, pos, indptr, slots, rank=rank, eps=1e-5, row_lens=lens, cum=cum))
+        t2 = timeit(lambda i: ops.wkv(*x.split(n, 1), low, w2, w3, bonus, on, st, o, pos, indptr, slots, rank=rank, eps=1e-5, row_lens=lens, cum=cum))
+        rep("wkv prompts, very fast decays", t2, by=T * (10.0 * n + 4.0 * rank) + B * wh * wd * wd * 8.0, fl=T * wh * (4.0 * wd * wd + 128.0 * wd), sequences=B, length=lens[0])
         rep("wkv prompts", t, by=T * (10.0 * n + 4.0 * rank) + B * wh * wd * wd * 8.0, fl=T * wh * (4.0 * wd * wd + 128.0 * wd), sequences=B, length=lens[0])
         S, P, N, G = sp["heads"], sp["vdim"], sp["state"], sp["groups"]
         u, z, o, st = rnd(T, C), rnd(T, S * P + S), torch.empty(T, S * P, dtype=bf, device=dev), torch.zeros(B, S, N, P, device=dev)

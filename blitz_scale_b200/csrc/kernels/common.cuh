@@ -90,6 +90,20 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   __syncthreads();
   return red[32];
 }
+// The same for two numbers with a single barrier; `red` must not be in use by anything before that barrier.
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2 (&red)[32]) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+  a = warp_sum(a);
+  b = warp_sum(b);
+  if (lane == 0) red[warp] = make_float2(a, b);
+  __syncthreads();
+  float2 s = red[0];
+  for (int w = 1; w < nw; ++w) {
+    s.x += red[w].x;
+    s.y += red[w].y;
+  }
+  return s;
+}
 __device__ __forceinline__ float block_max(float v, float* red) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
   v = warp_max(v);

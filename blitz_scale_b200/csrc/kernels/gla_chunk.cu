@@ -16,7 +16,7 @@
 // and every product takes the factor between two block borders from a table: block (i, j < i) scales k~ by
 // e^(r_i - r_(j+1)) <= 1, the state term scales q' by e^(r_i), the state update scales k~ by e^(b_end - r_(j+1)).  Only
 // within one block is the factor e^(r_i - r_(i+1)) >= 1; when a channel decays by more than e^-80 within 16 tokens, which
-// that form cannot hold, the block's 136 scores are computed one by one from the unscaled inputs.
+// that form cannot hold, the block's 136 scores are computed one by one from the unscaled inputs, a warp per row.
 //
 // 32-bit arithmetic where the design asks for it: decays, their sums and exponentials and the state are fp32, and the
 // products that involve them split their fp32 operands into two bf16 numbers (x = hi + lo, relative error 2^-17) and
@@ -69,37 +69,50 @@ __device__ __forceinline__ float log_sigmoid_ex2(float z) {
 }
 
 // Running sum of log(sigmoid(low a2 + b)) / tau (WKV: -exp(tanh(low) a2 + b)) over a chunk; a thread per channel.
-constexpr int kGdThreads = 128;
+constexpr int kGdThreads = 128, kGdPitch = kGcC + 4, kGdMaxRank = 128;
 template <bool WKV>
 __global__ void __launch_bounds__(kGdThreads) gla_decay_kernel(const GlaChunkParams p) {
   ptx::griddep_launch_dependents();
   ptx::griddep_wait();
-  extern __shared__ float s_low[];  // [64][rank]
+  extern __shared__ __align__(16) float s_low[];  // [rank][kGdPitch] by token, and behind it the channels' coefficients [rank][kGdThreads]
+  float* s_w = s_low + p.rank * kGdPitch;
   const int r = blockIdx.z, hk = p.heads * p.dim;
   const int t0 = p.tok_indptr[r] + blockIdx.y * kGcC, n = min(kGcC, p.tok_indptr[r + 1] - t0);
   if (n <= 0) return;
+  const int c = blockIdx.x * kGdThreads + threadIdx.x;
+  for (int i = 0; i < p.rank; ++i) s_w[i * kGdThreads + threadIdx.x] = c < hk ? ldf(p.a2 + static_cast<int64_t>(i) * hk + c) : 0.f;
   for (int i = threadIdx.x; i < n * p.rank; i += kGdThreads)
-    s_low[i] = WKV ? tanhf(p.low32[static_cast<int64_t>(t0 + i / p.rank) * p.low_row + i % p.rank])
+    s_low[i % p.rank * kGdPitch + i / p.rank] = WKV ? tanhf(p.low32[static_cast<int64_t>(t0 + i / p.rank) * p.low_row + i % p.rank])
                    : ldf(p.low + static_cast<int64_t>(t0 + i / p.rank) * p.row + i % p.rank);
   __syncthreads();
-  const int c = blockIdx.x * kGdThreads + threadIdx.x;
   if (c >= hk) return;
-  constexpr int kKeep = 16;  // coefficients kept in registers
-  float w[kKeep];
-#pragma unroll
-  for (int i = 0; i < kKeep; ++i) w[i] = i < p.rank ? ldf(p.a2 + static_cast<int64_t>(i) * hk + c) : 0.f;
   const float bias = ldf(p.a2_b + c);
   float sum = 0.f;
-  for (int t = 0; t < n; ++t) {
-    const float* low = s_low + t * p.rank;
-    float z = bias;
+  constexpr int kAtOnce = 16;  // tokens whose sums a thread forms together
+  for (int first = 0; first < n; first += kAtOnce) {
+    float zs[kAtOnce];
 #pragma unroll
-    for (int i = 0; i < kKeep; ++i)
-      if (i < p.rank) z += low[i] * w[i];
-    for (int i = kKeep; i < p.rank; ++i) z += low[i] * ldf(p.a2 + static_cast<int64_t>(i) * hk + c);
-    sum += WKV ? -fminf(__expf(z), 104.f)  // (e^-104 is zero in fp32; larger steps would only cost the sum its digits)
-               : log_sigmoid_ex2(z) * p.inv_tau;
-    p.cum[static_cast<int64_t>(t0 + t) * hk + c] = sum;
+    for (int k = 0; k < kAtOnce; ++k) zs[k] = bias;
+    for (int i = 0; i < p.rank; ++i) {
+      const float w = s_w[i * kGdThreads + threadIdx.x];
+#pragma unroll
+      for (int k = 0; k < kAtOnce; k += 4) {  // (what lies behind the last token is not used)
+        const float4 a = *reinterpret_cast<const float4*>(s_low + i * kGdPitch + first + k);
+        zs[k] = fmaf(a.x, w, zs[k]);
+        zs[k + 1] = fmaf(a.y, w, zs[k + 1]);
+        zs[k + 2] = fmaf(a.z, w, zs[k + 2]);
+        zs[k + 3] = fmaf(a.w, w, zs[k + 3]);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < kAtOnce; ++k) {
+      const int t = first + k;
+      if (t >= n) break;
+      const float z = zs[k];
+      // (e^-104 is zero in fp32; larger steps would only cost the sum its digits)
+      sum += WKV ? -fminf(__expf(z), 104.f) : log_sigmoid_ex2(z) * p.inv_tau;
+      p.cum[static_cast<int64_t>(t0 + t) * hk + c] = sum;
+    }
   }
 }
 
@@ -134,6 +147,20 @@ struct GcSmem {
   __nv_bfloat16 ah[kGcC * kA], al[kGcC * kA];
   __nv_bfloat16 sh[DK * kV], sl[DK * kV];
 };
+
+// N neighbouring elements (the address is a multiple of N elements).
+template <int N, typename T>
+__device__ __forceinline__ void ldn(const T* p, float (&v)[N]) {
+  if constexpr (N == 4) {
+    const float4 f = ldf4(p);
+    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+  } else if constexpr (N == 2) {
+    const float2 f = ldf2(p);
+    v[0] = f.x; v[1] = f.y;
+  } else {
+    v[0] = ldf(p);
+  }
+}
 
 // Tiles 0 .. 5: (1,0) (2,0) (2,1) (3,0) (3,1) (3,2); 6 .. 9: the diagonal.
 __device__ __forceinline__ void gc_tile(int tile, int& i, int& j) {
@@ -328,27 +355,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
-      if (i == j && sm.wide[i]) {
-        const float* cum = p.cum + static_cast<int64_t>(t_beg + base) * hk + h * p.dim;
-        // one score at a time: entry e of the fragment
-#pragma unroll 1
-        for (int e = 0; e < 8; ++e) {
-          const int t = i * kGcB + g + ((e >> 1) & 1) * 8, s = i * kGcB + (e >> 2) * 8 + 2 * t4 + (e & 1);
-          float x = 0.f;
-          if ((WKV ? s < t : s <= t) && t < n_tok) {
-            const bf* qr = p.q + static_cast<int64_t>(t_beg + base + t) * p.row + h * p.dim;
-            const bf* kr = p.k + static_cast<int64_t>(t_beg + base + s) * p.row + h * p.dim;
-            const float *bt = cum + static_cast<int64_t>(WKV ? t - 1 : t) * hk, *bs = cum + static_cast<int64_t>(s) * hk;
-            for (int c = 0; c < p.dim; ++c) x += ldf(qr + c) * ldf(kr + c) * __expf(bt[c] - bs[c]);
-            x *= p.q_scale;
-          }
-#pragma unroll
-          for (int n = 0; n < 2; ++n)
-#pragma unroll
-            for (int f = 0; f < 4; ++f)
-              if (n * 4 + f == e) acc[n][f] = x;
-        }
-      } else {
+      if (!(i == j && sm.wide[i])) {
         const float* fs = sm.fs + warp * DK + 2 * t4;
 #pragma unroll
         for (int kk = 0; kk < DK / 16; ++kk) {
@@ -376,6 +383,7 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
           const int t = g + half * 8, s = n * 8 + 2 * t4;
+          if (i == j && sm.wide[i]) continue;
           float x = acc[n][2 * half], y = acc[n][2 * half + 1];
           if (i == j) {  // above the diagonal (a factored score may be anything there)
             if (s > t) x = 0.f;
@@ -389,6 +397,51 @@ __global__ void __launch_bounds__(kGcThreads, 1) gla_chunk_kernel(const GlaChunk
           *reinterpret_cast<uint32_t*>(sm.ah + at) = hi;
           *reinterpret_cast<uint32_t*>(sm.al + at) = lo;
         }
+    }
+    // blocks that the factored form cannot hold: a warp per row, the scores one by one from the unscaled inputs
+    for (int i = 0; i < 4; ++i) {
+      if (!sm.wide[i]) continue;
+      constexpr int CH = DK / 32;  // channels of a lane
+      const int t = warp, c = lane * CH;
+      const bool on = i * kGcB + t < n_tok && c < p.dim;
+      const int64_t tok = t_beg + base + i * kGcB;
+      float q[CH], bt[CH], x[kGcB];
+#pragma unroll
+      for (int e = 0; e < CH; ++e) q[e] = bt[e] = 0.f;
+      if (on) {
+        ldn<CH>(p.q + (tok + t) * p.row + h * p.dim + c, q);
+        if (!WKV || i * kGcB + t > 0) ldn<CH>(p.cum + (tok + t - (WKV ? 1 : 0)) * hk + h * p.dim + c, bt);
+      }
+#pragma unroll
+      for (int s = 0; s < kGcB; ++s) {
+        x[s] = 0.f;
+        if (on && (WKV ? s < t : s <= t)) {
+          float k[CH], bs[CH];
+          ldn<CH>(p.k + (tok + s) * p.row + h * p.dim + c, k);
+          ldn<CH>(p.cum + (tok + s) * hk + h * p.dim + c, bs);
+#pragma unroll
+          for (int e = 0; e < CH; ++e) x[s] += q[e] * k[e] * __expf(bt[e] - bs[e]);
+          x[s] *= p.q_scale;
+        }
+      }
+      // lane s receives the sum of x[s] over the lanes (both halves of the warp the same)
+#pragma unroll
+      for (int o = 8; o > 0; o >>= 1) {
+        const bool up = lane & o;
+#pragma unroll
+        for (int s = 0; s < o; ++s) {
+          const float give = up ? x[s] : x[s + o], keep = up ? x[s + o] : x[s];
+          x[s] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+        }
+      }
+      x[0] += __shfl_xor_sync(0xffffffffu, x[0], 16);
+      if (lane < kGcB) {
+        const float y = WKV && lane == t ? sm.own[i * kGcB + t] : x[0];
+        const bf hi = __float2bfloat16_rn(y);
+        const int at = (i * kGcB + t) * SM::kA + i * kGcB + lane;
+        sm.ah[at] = hi;
+        sm.al[at] = __float2bfloat16_rn(y - __bfloat162float(hi));
+      }
     }
     __syncthreads();
 
@@ -565,8 +618,15 @@ static int gla_chunk_any(const GlaChunkParams& p, int rows, int max_len, cudaStr
   if ((reinterpret_cast<uintptr_t>(p.g) | reinterpret_cast<uintptr_t>(p.out)) & 3) return -1;
   if (reinterpret_cast<uintptr_t>(p.cum) & 15) return -1;
   const int hk = p.heads * p.dim;
-  cudaError_t e = launch_pdl(gla_decay_kernel<WKV>, dim3((hk + kGdThreads - 1) / kGdThreads, (max_len + kGcC - 1) / kGcC, rows),
-                             dim3(kGdThreads), (size_t)kGcC * p.rank * sizeof(float), stream, p);
+  const size_t smem = (size_t)p.rank * (kGdPitch + kGdThreads) * sizeof(float);
+  static PerDeviceOnce once;
+  cudaError_t e = once.run([] {
+    return cudaFuncSetAttribute(gla_decay_kernel<WKV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                kGdMaxRank * (kGdPitch + kGdThreads) * (int)sizeof(float));
+  });
+  if (e != cudaSuccess) return (int)e;
+  e = launch_pdl(gla_decay_kernel<WKV>, dim3((hk + kGdThreads - 1) / kGdThreads, (max_len + kGcC - 1) / kGcC, rows),
+                             dim3(kGdThreads), smem, stream, p);
   if (e != cudaSuccess) return (int)e;
   const int sms = device_sm_count();
   e = p.dim <= 32   ? launch_gla_width<32, WKV>(p, rows, sms, stream)
@@ -583,7 +643,7 @@ using namespace blitz;
 // Whether the chunked kernel takes these sizes (bf16 only; vectors of 8 elements).
 int blitz_gla_chunk_supported(int dim, int vdim, int rank) {
   return dim > 0 && dim <= 128 && (dim & 7) == 0 && vdim > 0 && (vdim & 7) == 0 && vdim <= kGcV * kGcMaxCluster && rank > 0 &&
-         rank <= 128;
+         rank <= kGdMaxRank;
 }
 
 // Rows of at least one token each: tokens tok_indptr[r] .. tok_indptr[r + 1]; max_len: the longest row.  cum: fp32 scratch

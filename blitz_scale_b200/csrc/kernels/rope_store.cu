@@ -59,7 +59,7 @@ __global__ void __launch_bounds__(NORM && MODE == kRopeWideHalves ? 1024 : 256, 
   const int heads = p.q_heads + (s >= 0 ? p.kv_heads : 0);
   const T *q_w = reinterpret_cast<const T*>(p.q_w), *k_w = reinterpret_cast<const T*>(p.k_w);
   float q_f = 1.f, k_f = 1.f;
-  __shared__ float red[2][33];
+  __shared__ float2 red[32];
   if (NORM && MODE != kRopeWideHalves) {
     auto squares = [&](const T* x, int n) {
       float ss = 0.f;
@@ -79,9 +79,9 @@ __global__ void __launch_bounds__(NORM && MODE == kRopeWideHalves ? 1024 : 256, 
       return ss;
     };
     const int nq = p.q_heads * p.dim, nk = p.k ? p.kv_heads * p.dim : 0;
-    const float sq = squares(q, nq), sk = squares(k, nk);
-    q_f = rsqrtf(block_sum(sq, red[0]) / static_cast<float>(nq) + p.eps);
-    if (p.k) k_f = rsqrtf(block_sum(sk, red[1]) / static_cast<float>(nk) + p.eps);
+    const float2 ss = block_sum2(squares(q, nq), squares(k, nk), red);
+    q_f = rsqrtf(ss.x / static_cast<float>(nq) + p.eps);
+    if (p.k) k_f = rsqrtf(ss.y / static_cast<float>(nk) + p.eps);
   }
   auto angles = [&]() {
     const float pos = static_cast<float>(p.pos[t]);
@@ -165,29 +165,50 @@ __global__ void __launch_bounds__(NORM && MODE == kRopeWideHalves ? 1024 : 256, 
         if (m.c < turns) load8(m.is_q ? q : k, m.is_q ? q_b : k_b, first(m) + half, v);
       };
       request();
+      auto copy_values = [&]() {
+        if (p.v == nullptr || s < 0) return;
+        const T* v = reinterpret_cast<const T*>(p.v) + t * p.row;
+        for (int i = threadIdx.x * 8; i < vrow; i += blockDim.x * 8) {
+          float x[8];
+          ldf8<T>(v + i, x);
+          if (v_b) {
+            float b[8];
+            ldf8<T>(v_b + i, b);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x[j] += b[j];
+          }
+          stf8<T>(vdst + i, x);
+        }
+      };
+      float wu[8], wv[8];
+      if (NORM) {  // while the values are on their way
+        if (m.on) {
+          const T* w = (m.is_q ? q_w : k_w) + first(m);
+          ldf8<T>(w, wu);
+          if (m.c < turns) ldf8<T>(w + half, wv);
+        }
+        copy_values();
+        angles();
+      }
       if (NORM) {  // every thread has one item at most (see the launch): its values are what the norms are taken over
         float ss = 0.f;
         if (m.on) {
 #pragma unroll
           for (int j = 0; j < 8; ++j) ss += u[j] * u[j] + (m.c < turns ? v[j] * v[j] : 0.f);
         }
-        q_f = rsqrtf(block_sum(m.is_q ? ss : 0.f, red[0]) / static_cast<float>(p.q_heads * p.dim) + p.eps);
-        if (p.k) k_f = rsqrtf(block_sum(m.is_q ? 0.f : ss, red[1]) / static_cast<float>(p.kv_heads * p.dim) + p.eps);
+        const float2 sum = block_sum2(m.is_q ? ss : 0.f, m.is_q ? 0.f : ss, red);
+        q_f = rsqrtf(sum.x / static_cast<float>(p.q_heads * p.dim) + p.eps);
+        if (p.k) k_f = rsqrtf(sum.y / static_cast<float>(p.kv_heads * p.dim) + p.eps);
         if (m.on) {
           const float f = m.is_q ? q_f : k_f;
-          const T* w = (m.is_q ? q_w : k_w) + first(m);
-          float a[8];
-          ldf8<T>(w, a);
 #pragma unroll
-          for (int j = 0; j < 8; ++j) u[j] *= f * a[j];
-          if (m.c < turns) {
-            ldf8<T>(w + half, a);
-#pragma unroll
-            for (int j = 0; j < 8; ++j) v[j] *= f * a[j];
+          for (int j = 0; j < 8; ++j) {
+            u[j] *= f * wu[j];
+            if (m.c < turns) v[j] *= f * wv[j];
           }
         }
       }
-      angles();
+      if (!NORM) angles();
       for (int it = threadIdx.x; it < items; it += blockDim.x) {
         if (it != static_cast<int>(threadIdx.x)) {
           m = item(it);
@@ -210,6 +231,7 @@ __global__ void __launch_bounds__(NORM && MODE == kRopeWideHalves ? 1024 : 256, 
         }
         stf8<T>(dst + at, u);
       }
+      if (NORM) return;
     }
     if (p.v != nullptr && s >= 0) {
       const T* v = reinterpret_cast<const T*>(p.v) + t * p.row;

@@ -504,6 +504,38 @@ __global__ void __launch_bounds__(256) part_norm_kernel(T* x, int64_t row, const
   }
 }
 
+// The same with a warp per part, for parts that a warp holds in registers: `kPartVecs` groups of eight per lane.
+constexpr int kPartVecs = 4;
+template <typename T>
+__global__ void __launch_bounds__(256) part_norm_warp_kernel(T* x, int64_t row, const T* w, float eps, int parts, int part, int64_t items) {
+  ptx::griddep_launch_dependents();
+  ptx::griddep_wait();
+  const int64_t item = static_cast<int64_t>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  if (item >= items) return;
+  const int lane = threadIdx.x & 31, n = part / 8, which = static_cast<int>(item % parts);
+  T* xr = x + item / parts * row + static_cast<int64_t>(which) * part;
+  const T* wr = w + static_cast<int64_t>(which) * part;
+  float v[kPartVecs][8], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < kPartVecs; ++k)
+    if (lane + k * 32 < n) ldf8<T>(xr + (lane + k * 32) * 8, v[k]);
+#pragma unroll
+  for (int k = 0; k < kPartVecs; ++k)
+    if (lane + k * 32 < n)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss += v[k][j] * v[k][j];
+  const float f = rsqrtf(warp_sum(ss) / static_cast<float>(part) + eps);
+#pragma unroll
+  for (int k = 0; k < kPartVecs; ++k)
+    if (lane + k * 32 < n) {
+      float g[8];
+      ldf8<T>(wr + (lane + k * 32) * 8, g);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[k][j] *= f * g[j];
+      stf8<T>(xr + (lane + k * 32) * 8, v[k]);
+    }
+}
+
 }  // namespace blitz
 
 extern "C" {
@@ -560,6 +592,9 @@ int blitz_part_norm(void* x, int64_t row, const void* w, float eps, int tokens, 
   const dim3 grid(parts, tokens), block(n <= 64 ? 64 : n <= 256 ? 128 : 256);
   auto go = [&](auto type) {
     using T = decltype(type);
+    const int64_t items = (int64_t)tokens * parts;
+    if (wide && part <= 256 * kPartVecs && items / 8 >= device_sm_count())
+      return launch_pdl(part_norm_warp_kernel<T>, dim3((unsigned)((items + 7) / 8)), dim3(256), 0, stream, (T*)x, row, (const T*)w, eps, parts, part, items);
     return wide ? launch_pdl(part_norm_kernel<T, 8>, grid, block, 0, stream, (T*)x, row, (const T*)w, eps, part)
                 : launch_pdl(part_norm_kernel<T, 1>, grid, block, 0, stream, (T*)x, row, (const T*)w, eps, part);
   };

@@ -87,10 +87,11 @@ struct SrEarly {
 };
 
 template <typename T, int VEC, int S, bool CONV>
-__global__ void __launch_bounds__(kSrThreads, 1) stream_rms_kernel(const StreamRmsParams p) {
+__global__ void __launch_bounds__(kSrThreads, CONV ? 1 : 2) stream_rms_kernel(const StreamRmsParams p) {
   using C = SrCols<T, VEC>;
   using F = SrCols<float, VEC>;
-  __shared__ float s_mix[S * S], s_out[S], s_in[S], red[33], red2[33];
+  __shared__ float s_mix[S * S], s_out[S], s_in[S];
+  __shared__ float2 red[32], red2[32];
   extern __shared__ __align__(16) float s_keep[];
   ptx::griddep_launch_dependents();
   const T *w = reinterpret_cast<const T*>(p.w), *bias = reinterpret_cast<const T*>(p.bias);
@@ -168,8 +169,9 @@ __global__ void __launch_bounds__(kSrThreads, 1) stream_rms_kernel(const StreamR
         b += d.v[k] * d.v[k];
       }
     }
-    f0 = 0.5f * rsqrtf(block_sum(a, red) / static_cast<float>(p.hidden) + p.eps);
-    f1 = 0.5f * rsqrtf(block_sum(b, red2) / static_cast<float>(p.hidden) + p.eps);
+    const float2 sum = block_sum2(a, b, red2);
+    f0 = 0.5f * rsqrtf(sum.x / static_cast<float>(p.hidden) + p.eps);
+    f1 = 0.5f * rsqrtf(sum.y / static_cast<float>(p.hidden) + p.eps);
   }
   F keep[kKeep];
   float ss = 0.f;
@@ -237,7 +239,7 @@ __global__ void __launch_bounds__(kSrThreads, 1) stream_rms_kernel(const StreamR
   }
   for (int i = threadIdx.x + behind; i < n; i += blockDim.x) collect(i).store(s_keep + (i - behind) * VEC);
   if (p.h == nullptr) return;
-  const float scale = rsqrtf(block_sum(ss, red) / static_cast<float>(p.hidden) + p.eps);
+  const float scale = rsqrtf(block_sum2(ss, 0.f, red).x / static_cast<float>(p.hidden) + p.eps);
   const float gain = p.w_step ? 0.f : p.w_offset + ldf<T>(w);
   const int per = CONV && p.mixes > 0 ? p.mixes : 1;
   T* out = reinterpret_cast<T*>(p.h) + static_cast<int64_t>(t) * per * p.hidden;
@@ -376,7 +378,7 @@ int blitz_stream_rms(const int32_t* ids, const void* embed, int vocab, int from_
   const int vec = (hidden & 3) || (y_row & 3) ? 1 : 4, n = hidden / vec;
   int threads = 32;
   // few tokens: as many threads as there are groups
-  while (threads < n && threads < (tokens <= 2 * device_sm_count() ? kSrThreads : 256)) threads <<= 1;
+  while (threads < n && threads < (tokens <= device_sm_count() ? kSrThreads : 256)) threads <<= 1;
   const int keep = conv ? 2 : kSrKeep;
   while (threads * keep < n && threads < kSrThreads) threads <<= 1;
   const size_t smem = threads * keep < n ? (size_t)(n - threads * keep) * vec * sizeof(float) : 0;

@@ -459,12 +459,7 @@ class HybridRunner:
         """h: the mixes, [T, 5 * hidden]."""
         T, H, N, rc = m.num_tokens, self.cfg.hidden, mx.out_width, self.cache.runs[r]
         out = self._rkvg[:T * 4 * N].view(T, 4 * N)
-        w = self._w(l, "rkvg")
-        if T <= ops.PAIR_GEMM_MAX_M and N % 8 == 0 and H * N >= self.SEPARATE_WEIGHTS:
-            for i in range(4):                       # large weights, few rows: the weight-streaming products
-                ops.gemm(h[:, i * H:(i + 1) * H], w[i * H:(i + 1) * H], out=out[:, i * N:(i + 1) * N], static_b=True)
-        else:
-            ops.gemm(h[:, :4 * H], w, out=out, groups=4, static_b=True)
+        ops.gemm(h[:, :4 * H], self._w(l, "rkvg"), out=out, groups=4, static_b=True)
         w1 = self._w(l, "w1")
         low = self._low[:T * w1.shape[1]].view(T, w1.shape[1])
         narrow = dict(bn=64, split_k=4 if T <= 2048 else 1) if T > ops.DECODE_GEMM_MAX_M else {}     # as for a router's columns
@@ -478,8 +473,6 @@ class HybridRunner:
         if m.batch > ns:
             ops.wkv(*parts, low, *weights, rc.state, mid, m.pos, m.tok_indptr[ns:], m.seq_slot[ns:], row_lens=m.seq_lens_host[ns:],
                     cum=self._cum, **args)
-
-    SEPARATE_WEIGHTS = 1 << 21    # elements of one of the four matrices
 
     def _parallel(self, r: int, l: int, mx: ParallelMixer, p: Dict[str, torch.Tensor], mid: torch.Tensor, m: StepMeta) -> None:
         left = {n[2:]: v for n, v in p.items() if n.startswith("l_")}
@@ -558,8 +551,7 @@ class HybridRunner:
 
     def decode_launches(self) -> int:
         """Kernels of this library in one decode step."""
-        per = {"attention": 2, "latent": 7, "gla": 1, "rglru": 3, "parallel": 6}
-        per["wkv"] = 5 if any(m.kind == "wkv" and m.out_width * m.hidden >= self.SEPARATE_WEIGHTS for m in self.cfg.run_mixers()) else 2
+        per = {"attention": 2, "latent": 7, "gla": 1, "rglru": 3, "wkv": 2, "parallel": 6}
         specs = [self.cfg.layer_specs[r.layer] for r in self.runs]
         n = sum(3 + per[s.mixer.kind] + bool(s.ff) + 3 * bool(s.ff_after) + 5 * bool(s.moe) for s in specs)
         return n + 3      # final norm, head product, arg-max
