@@ -131,16 +131,19 @@ def bench_kernels(out, size):
         rep("stream_rms", t, by=by, tokens=T)
         two = ops.Pending(y, mix, v, norms=(w, w))
         t = timeit(lambda i: ops.stream_rms(xf[i], pending=two, out=o, **args), copies=len(xf))
+        o32 = torch.empty(T, H, device=dev)
+        t2 = timeit(lambda i: ops.stream_rms(xf[i], pending=pd, out=o32, **args), copies=len(xf))
+        rep("stream_rms, fp32 output", t2, by=by + 2.0 * T * H, tokens=T)
         rep("stream_rms, two normed outputs", t, by=by + 2.0 * T * H, tokens=T)
         pos, slots = torch.full((T,), 9, dtype=torch.int32, device=dev), torch.arange(T, dtype=torch.int32, device=dev)
-        hist, shift = torch.zeros(T, TAPS - 1, H, dtype=bf, device=dev), torch.zeros(T, H, dtype=bf, device=dev)
+        hist, shift = torch.zeros(T, TAPS - 1, H, device=dev), torch.zeros(T, H, device=dev)
         if T <= 256:
             st = ops.TokenState(conv, hist)
             t = timeit(lambda i: ops.stream_rms(xf[i], pending=pd, out=o, tokens=st, pos=pos, seq_slot=slots, **args), copies=len(xf))
-            rep("stream_rms with the convolution (decode)", t, by=by + 4.0 * T * H * (TAPS - 1), tokens=T)
+            rep("stream_rms with the convolution (decode)", t, by=by + 8.0 * T * H * (TAPS - 1), tokens=T)
             st = ops.TokenState(conv, hist, mu, shift)
             t = timeit(lambda i: ops.stream_rms(xf[i], pending=pd, out=o5, tokens=st, pos=pos, seq_slot=slots, **args), copies=len(xf))
-            rep("stream_rms with convolution and mixes (decode)", t, by=by + 4.0 * T * H * (TAPS - 1) + 12.0 * T * H, tokens=T)
+            rep("stream_rms with convolution and mixes (decode)", t, by=by + 8.0 * T * H * (TAPS - 1) + 16.0 * T * H, tokens=T)
         del xf
     C = sp["heads"] * sp["vdim"] + 2 * sp["groups"] * sp["state"]
     cb, zero, sc = rnd(C), torch.zeros(max(C, H), dtype=bf, device=dev), rnd(TAPS, C)
@@ -159,11 +162,12 @@ def bench_kernels(out, size):
         rep("token_conv, silu", t, by=T * C * 4.0, sequences=B, length=lens[0])
         if lens[0] == 1:
             continue
-        t = timeit(lambda i: ops.token_conv(cut(xs[i], H), conv, hh, cut(us[i], H), pos, indptr, slots, residual=True), copies=nc)
-        rep("token_conv, input and its convolution", t, by=T * H * 4.0, sequences=B, length=lens[0])
-        o5, shift, lasth = [torch.empty(T, 5 * H, dtype=bf, device=dev) for _ in range(2)], torch.zeros(B, H, dtype=bf, device=dev), torch.empty(B, H, dtype=bf, device=dev)
-        t = timeit(lambda i: ops.token_conv(cut(xs[i % nc], H), conv, hh, o5[i % 2], pos, indptr, slots, residual=True, mu=mu, shift=shift, last=lasth), copies=2)
-        rep("token_conv with mixes", t, by=T * H * 12.0, sequences=B, length=lens[0])
+        x32, h32 = [torch.randn(T, H, device=dev) for _ in range(2)], torch.zeros(B, TAPS - 1, H, device=dev)
+        t = timeit(lambda i: ops.token_conv(x32[i], conv, h32, cut(us[i], H), pos, indptr, slots, residual=True), copies=2)
+        rep("token_conv, fp32 input and its convolution", t, by=T * H * 6.0, sequences=B, length=lens[0])
+        o5, shift, lasth = [torch.empty(T, 5 * H, dtype=bf, device=dev) for _ in range(2)], torch.zeros(B, H, device=dev), torch.empty(B, H, device=dev)
+        t = timeit(lambda i: ops.token_conv(x32[i % 2], conv, h32, o5[i % 2], pos, indptr, slots, residual=True, mu=mu, shift=shift, last=lasth), copies=2)
+        rep("token_conv with mixes", t, by=T * H * 14.0, sequences=B, length=lens[0])
     # ---- products
     n = wh * wd
     for M in (8192, 256, 64, 1):

@@ -11,7 +11,8 @@
 //   m_i  = h + (h_previous - h) mu_i                                  CONV with mixes: one row per mix
 //
 // A block per token.  A thread keeps its columns of u in registers between the two passes; every other value of a column is
-// only used by the thread that owns the column, the histories (by slot) included.  At the start every stream is the token's
+// only used by the thread that owns the column, the histories (by slot, fp32) included: what the norm gives is not rounded before
+// the convolution and the mixes are done.  At the start every stream is the token's
 // embedding; the first kernels read the embedding table instead of the streams.
 #include "launch.cuh"
 #include "ptx.cuh"
@@ -37,11 +38,12 @@ struct StreamRmsParams {
   const void* w;            // [1] or [hidden]
   const int32_t* rows;      // result t comes from token rows[t] + row_offset (null: t)
   void* h;                  // [tokens][hidden] (mixes: [tokens][mixes][hidden]), or null
+  int h32;                  // h is fp32 (no convolution)
   float* u;                 // [tokens][hidden], or null
   const void* conv;         // [taps][hidden], or null
-  void* hist;               // [slots][taps - 1][hidden]
+  float* hist;              // [slots][taps - 1][hidden]
   const void* mu;           // [mixes][hidden]
-  void* shift;              // [slots][hidden]
+  float* shift;             // [slots][hidden]
   const int32_t *pos, *seq_slot;
   float eps, w_offset;
   int hidden, vocab, row_offset, from_embed, write, w_step, taps, mixes, num_slots;
@@ -63,14 +65,6 @@ struct SrCols {
     if constexpr (VEC == 4) stf4<T>(p, make_float4(v[0], v[1], v[2], v[3]));
     else stf<T>(p, v[0]);
   }
-  __device__ __forceinline__ void round() {  // to what a store and a load would give
-#pragma unroll
-    for (int i = 0; i < VEC; ++i) {
-      T e;
-      stf<T>(&e, v[i]);
-      v[i] = ldf<T>(&e);
-    }
-  }
 };
 
 // Columns as they lie in memory.
@@ -83,11 +77,12 @@ struct alignas(VEC * sizeof(T)) SrRaw {
 constexpr int kSrTaps = 4, kSrMixes = 5;
 template <typename T, int VEC>
 struct SrEarly {
-  SrRaw<T, VEC> conv[kSrTaps], hist[kSrTaps - 1], mu[kSrMixes], prev;  // taps and history end at the last place
+  SrRaw<T, VEC> conv[kSrTaps], mu[kSrMixes];
+  SrCols<float, VEC> hist[kSrTaps - 1], prev;  // taps and history end at the last place
 };
 
 template <typename T, int VEC, int S, bool CONV>
-__global__ void __launch_bounds__(kSrThreads, CONV ? 1 : 2) stream_rms_kernel(const StreamRmsParams p) {
+__global__ void __launch_bounds__(kSrThreads, CONV || S > 4 ? 1 : 2) stream_rms_kernel(const StreamRmsParams p) {
   using C = SrCols<T, VEC>;
   using F = SrCols<float, VEC>;
   __shared__ float s_mix[S * S], s_out[S], s_in[S];
@@ -150,8 +145,8 @@ __global__ void __launch_bounds__(kSrThreads, CONV ? 1 : 2) stream_rms_kernel(co
 #pragma unroll
       for (int j = 0; j + 1 < kSrTaps; ++j)
         if (j >= kSrTaps - p.taps)
-          e.hist[j] = raw(p.hist, (static_cast<int64_t>(slot) * (p.taps - 1) + j - (kSrTaps - p.taps)) * p.hidden + c);
-      if (p.mixes > 0 && at > 0) e.prev = raw(p.shift, static_cast<int64_t>(slot) * p.hidden + c);
+          e.hist[j].load(p.hist + (static_cast<int64_t>(slot) * (p.taps - 1) + j - (kSrTaps - p.taps)) * p.hidden + c);
+      if (p.mixes > 0 && at > 0) e.prev.load(p.shift + static_cast<int64_t>(slot) * p.hidden + c);
     }
   }
   const T* y0 = p.y ? reinterpret_cast<const T*>(p.y) + src * p.y_row : nullptr;
@@ -244,22 +239,23 @@ __global__ void __launch_bounds__(kSrThreads, CONV ? 1 : 2) stream_rms_kernel(co
   const int per = CONV && p.mixes > 0 ? p.mixes : 1;
   T* out = reinterpret_cast<T*>(p.h) + static_cast<int64_t>(t) * per * p.hidden;
   auto convolved = [&](int c, C h, const SrEarly<T, VEC>& e) {
-    h.round();
-    const C now = h;
-    auto add = [&](const Raw& a, const Raw& b) {
+    F now;
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) h.v[k] += ldf<T>(&a.e[k]) * ldf<T>(&b.e[k]);
+    for (int k = 0; k < VEC; ++k) now.v[k] = h.v[k];
+    auto add = [&](const Raw& a, const F& b) {
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) h.v[k] += ldf<T>(&a.e[k]) * b.v[k];
     };
 #pragma unroll
     for (int k = 0; k < VEC; ++k) h.v[k] += ldf<T>(&e.conv[kSrTaps - 1].e[k]) * now.v[k];
     if (slot >= 0) {
-      T* hist = reinterpret_cast<T*>(p.hist) + static_cast<int64_t>(slot) * (p.taps - 1) * p.hidden + c;
+      float* hist = p.hist + static_cast<int64_t>(slot) * (p.taps - 1) * p.hidden + c;
 #pragma unroll
       for (int j = 0; j + 1 < kSrTaps; ++j) {
         const int first = kSrTaps - p.taps;
         if (j < first) continue;
         if (kSrTaps - 1 - j <= at) add(e.conv[j], e.hist[j]);
-        if (j > first) *reinterpret_cast<Raw*>(hist + static_cast<int64_t>(j - first - 1) * p.hidden) = e.hist[j];
+        if (j > first) e.hist[j].store(hist + static_cast<int64_t>(j - first - 1) * p.hidden);
       }
       if (p.taps > 1) now.store(hist + static_cast<int64_t>(p.taps - 2) * p.hidden);
     }
@@ -267,11 +263,13 @@ __global__ void __launch_bounds__(kSrThreads, CONV ? 1 : 2) stream_rms_kernel(co
       h.store(out + c);
       return;
     }
-    h.round();
     float d[VEC];
 #pragma unroll
-    for (int k = 0; k < VEC; ++k) d[k] = (slot >= 0 && at > 0 ? ldf<T>(&e.prev.e[k]) : 0.f) - h.v[k];
-    if (slot >= 0) h.store(reinterpret_cast<T*>(p.shift) + static_cast<int64_t>(slot) * p.hidden + c);
+    for (int k = 0; k < VEC; ++k) {
+      d[k] = (slot >= 0 && at > 0 ? e.prev.v[k] : 0.f) - h.v[k];
+      now.v[k] = h.v[k];
+    }
+    if (slot >= 0) now.store(p.shift + static_cast<int64_t>(slot) * p.hidden + c);
 #pragma unroll
     for (int m = 0; m < kSrMixes; ++m) {
       if (m >= p.mixes) continue;
@@ -296,16 +294,18 @@ __global__ void __launch_bounds__(kSrThreads, CONV ? 1 : 2) stream_rms_kernel(co
   };
   auto finish = [&](int c, C h) {
     if (CONV) {
-      h.round();
       const T* conv = reinterpret_cast<const T*>(p.conv) + c;
-      T* hist = reinterpret_cast<T*>(p.hist) + static_cast<int64_t>(slot < 0 ? 0 : slot) * (p.taps - 1) * p.hidden + c;
-      C a, now = h;
+      float* hist = p.hist + static_cast<int64_t>(slot < 0 ? 0 : slot) * (p.taps - 1) * p.hidden + c;
+      C a;
+      F now;
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) now.v[k] = h.v[k];
       a.load(conv + static_cast<int64_t>(p.taps - 1) * p.hidden);
 #pragma unroll
       for (int k = 0; k < VEC; ++k) h.v[k] += a.v[k] * now.v[k];
       if (slot >= 0) {
         for (int j = 0; j + 1 < p.taps; ++j) {  // the oldest first; what a place holds moves to the one before it
-          C b;
+          F b;
           b.load(hist + static_cast<int64_t>(j) * p.hidden);
           if (j > 0) b.store(hist + static_cast<int64_t>(j - 1) * p.hidden);
           if (p.taps - 1 - j <= at) {
@@ -317,12 +317,13 @@ __global__ void __launch_bounds__(kSrThreads, CONV ? 1 : 2) stream_rms_kernel(co
         if (p.taps > 1) now.store(hist + static_cast<int64_t>(p.taps - 2) * p.hidden);
       }
       if (p.mixes > 0) {
-        h.round();
-        C prev = {};
+        F prev = {};
         if (slot >= 0) {
-          T* shift = reinterpret_cast<T*>(p.shift) + static_cast<int64_t>(slot) * p.hidden + c;
+          float* shift = p.shift + static_cast<int64_t>(slot) * p.hidden + c;
           if (at > 0) prev.load(shift);
-          h.store(shift);
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) now.v[k] = h.v[k];
+          now.store(shift);
         }
         for (int m = 0; m < p.mixes; ++m) {
           C b;
@@ -333,6 +334,13 @@ __global__ void __launch_bounds__(kSrThreads, CONV ? 1 : 2) stream_rms_kernel(co
         }
         return;
       }
+    }
+    if (!CONV && p.h32) {
+      F wide;
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) wide.v[k] = h.v[k];
+      wide.store(reinterpret_cast<float*>(p.h) + static_cast<int64_t>(t) * p.hidden + c);
+      return;
     }
     h.store(out + c);
   };
@@ -356,13 +364,13 @@ __global__ void __launch_bounds__(kSrThreads, CONV ? 1 : 2) stream_rms_kernel(co
 extern "C" {
 using namespace blitz;
 
-// See the top of the file.  x fp32 [tokens][streams][hidden]; embed, y, y1, h, histories and all weights in the activation type
-// (dtype 0 fp16, 1 bf16, 2 fp32).  y null: the streams stay as they are (`write` must be 0 then).  w_step: 0 one norm weight, 1 a
+// See the top of the file.  x fp32 [tokens][streams][hidden]; embed, y, y1, h and all weights in the activation type (dtype 0 fp16,
+// 1 bf16, 2 fp32); h32: h is fp32.  y null: the streams stay as they are (`write` must be 0 then).  w_step: 0 one norm weight, 1 a
 // weight per column.  conv null: no convolution; else every row is one token of a sequence with a state slot (negative: none).
 int blitz_stream_rms(const int32_t* ids, const void* embed, int vocab, int from_embed, float* x, const void* y, const void* y1,
                      int64_t y_row, const void* bias, const void* w0, const void* w1, const void* mix, const void* out_w,
                      const void* in_w, const void* w, int w_step, float w_offset, float eps, const int32_t* rows, int row_offset, void* h,
-                     float* u, int write, const void* conv, int taps, void* hist, const void* mu, int mixes, void* shift,
+                     int h32, float* u, int write, const void* conv, int taps, float* hist, const void* mu, int mixes, float* shift,
                      const int32_t* pos, const int32_t* seq_slot, int num_slots, int tokens, int hidden, int streams, int* status,
                      int dtype, cudaStream_t stream) {
   if (tokens <= 0) return 0;
@@ -371,9 +379,9 @@ int blitz_stream_rms(const int32_t* ids, const void* embed, int vocab, int from_
   if (y == nullptr ? (write != 0 || y1 != nullptr) : (mix == nullptr || out_w == nullptr)) return -1;
   if (y1 && (w0 == nullptr || w1 == nullptr || bias != nullptr)) return -1;
   if (h && w == nullptr) return -1;
-  if (rows && write) return -1;
+  if ((rows && write) || (h32 && conv)) return -1;
   if (conv && (rows || !h || taps < 1 || !pos || !seq_slot || (taps > 1 && !hist) || (mixes > 0 && (!mu || !shift)))) return -1;
-  StreamRmsParams p{ids, embed, x, y, y1, y_row, bias, w0, w1, mix, out_w, in_w, w, rows, h, u, conv, hist, mu, shift, pos, seq_slot,
+  StreamRmsParams p{ids, embed, x, y, y1, y_row, bias, w0, w1, mix, out_w, in_w, w, rows, h, h32, u, conv, hist, mu, shift, pos, seq_slot,
                     eps, w_offset, hidden, vocab, row_offset, from_embed, write, w_step, taps, mixes, num_slots, status};
   const int vec = (hidden & 3) || (y_row & 3) ? 1 : 4, n = hidden / vec;
   int threads = 32;

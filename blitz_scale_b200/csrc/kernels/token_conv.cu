@@ -11,6 +11,9 @@
 // through `last`).  With one token per row the convolution writes its history itself.  A row whose first token has position 0
 // starts from nothing and reads neither.
 //
+// Inputs and histories may be fp32 where outputs and weights are shorter (template parameter X): what a norm gives is then rounded
+// once, behind the convolution and the mixes.
+//
 // A thread walks `span` tokens of VEC channels with the last taps - 1 inputs in registers.
 #include "launch.cuh"
 #include "ptx.cuh"
@@ -58,9 +61,10 @@ struct TcvCols {
   }
 };
 
-template <typename T, int VEC, int TAPS>
+template <typename T, typename X, int VEC, int TAPS>
 __global__ void __launch_bounds__(kTcvThreads) token_conv_kernel(const TokenConvParams p) {
   using C = TcvCols<T, VEC>;
+  using I = TcvCols<X, VEC>;
   ptx::griddep_launch_dependents();
   const int c = (blockIdx.x * kTcvThreads + threadIdx.x) * VEC;
   const int64_t W = p.width;
@@ -76,12 +80,12 @@ __global__ void __launch_bounds__(kTcvThreads) token_conv_kernel(const TokenConv
   }
   ptx::griddep_wait();
   if (!on) return;
-  const T* x = reinterpret_cast<const T*>(p.x) + c;
-  T* hist = reinterpret_cast<T*>(p.hist) + c;
+  const X* x = reinterpret_cast<const X*>(p.x) + c;
+  X* hist = reinterpret_cast<X*>(p.hist) + c;
   T* out = reinterpret_cast<T*>(p.out) + c;
   const bool single = p.tok_indptr == nullptr;
   const int t0 = single ? blockIdx.y : blockIdx.y * p.span, t1 = single ? t0 + 1 : min(p.num_tokens, t0 + p.span);
-  C in[TAPS];  // inputs, oldest first; in[TAPS - 1] is the current token's
+  I in[TAPS];  // inputs, oldest first; in[TAPS - 1] is the current token's
   auto slot_of = [&](int b) {
     const int slot = p.seq_slot[b];
     if (slot >= p.num_slots) {
@@ -102,7 +106,7 @@ __global__ void __launch_bounds__(kTcvThreads) token_conv_kernel(const TokenConv
       }
     }
   };
-  auto convolve = [&](const C& raw) {
+  auto convolve = [&](const I& raw) {
 #pragma unroll
     for (int j = 0; j + 1 < TAPS; ++j) in[j] = in[j + 1];
     in[TAPS - 1] = raw;
@@ -120,7 +124,7 @@ __global__ void __launch_bounds__(kTcvThreads) token_conv_kernel(const TokenConv
     return a;
   };
   if (single) {
-    C raw;
+    I raw;
     raw.load(x + t0 * p.row);
     fill(t0, t0, t0);
     const int slot = slot_of(t0);
@@ -131,36 +135,33 @@ __global__ void __launch_bounds__(kTcvThreads) token_conv_kernel(const TokenConv
         if (j >= TAPS - p.taps + 1) in[j].store(hist + (static_cast<int64_t>(slot) * (p.taps - 1) + j - (TAPS - p.taps + 1)) * W);
     return;
   }
-  auto rounded = [](C a) {
+  auto as_input = [](const C& a) {
+    I b;
 #pragma unroll
-    for (int k = 0; k < VEC; ++k) {
-      T e;
-      stf<T>(&e, a.v[k]);
-      a.v[k] = ldf<T>(&e);
-    }
-    return a;
+    for (int k = 0; k < VEC; ++k) b.v[k] = a.v[k];
+    return b;
   };
-  C prev = {};
+  I prev = {};
   int b = row_of_token(p.tok_indptr, p.rows, t0);
   int first = p.tok_indptr[b], end = p.tok_indptr[b + 1];
   auto begin = [&](int t) {  // token t is the first one here of row b
     if (p.mixes > 0) {
       prev = {};
       if (t > first) {
-        C raw;
+        I raw;
         raw.load(x + (t - 1) * p.row);
         fill(b, t - 1, first);
-        prev = rounded(convolve(raw));
+        prev = as_input(convolve(raw));
         return;  // (its inputs are the ones before token t)
       }
       const int slot = slot_of(b);
-      if (slot >= 0 && p.pos[first] > 0) prev.load(reinterpret_cast<const T*>(p.shift) + slot * W + c);
+      if (slot >= 0 && p.pos[first] > 0) prev.load(reinterpret_cast<const X*>(p.shift) + slot * W + c);
     }
     fill(b, t, first);
   };
   begin(t0);
   for (int base = t0; base < t1; base += kTcvAhead) {
-    C raw[kTcvAhead];
+    I raw[kTcvAhead];
 #pragma unroll
     for (int k = 0; k < kTcvAhead; ++k) {
       raw[k] = {};
@@ -183,7 +184,7 @@ __global__ void __launch_bounds__(kTcvThreads) token_conv_kernel(const TokenConv
         a.store(out + t * p.out_row);
         continue;
       }
-      const C h = rounded(a);
+      const I h = as_input(a);
       for (int m = 0; m < p.mixes; ++m) {
         C mu;
         mu.load(reinterpret_cast<const T*>(p.mu) + m * W + c);
@@ -191,7 +192,7 @@ __global__ void __launch_bounds__(kTcvThreads) token_conv_kernel(const TokenConv
         for (int i = 0; i < VEC; ++i) mu.v[i] = fmaf(prev.v[i] - h.v[i], mu.v[i], h.v[i]);
         mu.store(out + t * p.out_row + m * W);
       }
-      if (t + 1 == end) h.store(reinterpret_cast<T*>(p.last) + b * W + c);
+      if (t + 1 == end) h.store(reinterpret_cast<X*>(p.last) + b * W + c);
       prev = h;
     }
   }
@@ -217,13 +218,13 @@ __global__ void __launch_bounds__(256) conv_keep_kernel(const TokenConvParams p)
   if (p.mixes > 0) const_cast<T*>(reinterpret_cast<const T*>(p.shift))[slot * W + c] = reinterpret_cast<const T*>(p.last)[r * W + c];
 }
 
-template <typename T, int VEC>
+template <typename T, typename X, int VEC>
 static cudaError_t launch_token_conv(const TokenConvParams& p, cudaStream_t stream) {
   const int units = (p.width + VEC - 1) / VEC;
   const int spans = p.tok_indptr ? (p.num_tokens + p.span - 1) / p.span : p.num_tokens;
   const dim3 grid((units + kTcvThreads - 1) / kTcvThreads, spans), block(kTcvThreads);
-  return p.taps <= 4 ? launch_pdl(token_conv_kernel<T, VEC, 4>, grid, block, 0, stream, p)
-                     : launch_pdl(token_conv_kernel<T, (VEC > 4 ? 4 : VEC), kTcvMaxTaps>, dim3((p.width / (VEC > 4 ? 4 : VEC) + kTcvThreads) / kTcvThreads, spans),
+  return p.taps <= 4 ? launch_pdl(token_conv_kernel<T, X, VEC, 4>, grid, block, 0, stream, p)
+                     : launch_pdl(token_conv_kernel<T, X, (VEC > 4 ? 4 : VEC), kTcvMaxTaps>, dim3((p.width / (VEC > 4 ? 4 : VEC) + kTcvThreads) / kTcvThreads, spans),
                                   block, 0, stream, p);
 }
 
@@ -232,10 +233,11 @@ static cudaError_t launch_token_conv(const TokenConvParams& p, cudaStream_t stre
 extern "C" {
 using namespace blitz;
 
-// See the top of the file; everything in the activation type (dtype 0 fp16, 1 bf16, 2 fp32).  tok_indptr null: one token per row
+// See the top of the file; everything in the activation type (dtype 0 fp16, 1 bf16, 2 fp32), but with x32 x, hist, shift and last in
+// fp32.  tok_indptr null: one token per row
 // (no mixes then).  With tok_indptr the histories are brought up to date by a second launch.
 int blitz_token_conv(const void* x, int64_t row, const void* conv, const void* conv_b, void* hist, void* out, int64_t out_row,
-                     int silu, int residual, const void* mu, int mixes, void* shift, void* last, const int32_t* pos,
+                     int silu, int residual, int x32, const void* mu, int mixes, void* shift, void* last, const int32_t* pos,
                      const int32_t* tok_indptr, const int32_t* seq_slot, int num_tokens, int rows, int width, int taps, int num_slots,
                      int* status, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0 || rows <= 0) return 0;
@@ -244,26 +246,24 @@ int blitz_token_conv(const void* x, int64_t row, const void* conv, const void* c
   TokenConvParams p{x, row, conv, conv_b, hist, out, out_row, mu, shift, last, pos, tok_indptr, seq_slot,
                     num_tokens, rows, width, taps, num_slots, num_tokens >= 2048 ? 32 : 8, silu, residual, mixes, status};
   if ((tok_indptr ? num_tokens / p.span : num_tokens) >= 65535 || rows > 65535) return -1;
-  const int es = dtype == 2 ? 4 : 2;
+  const int es = dtype == 2 ? 4 : 2, xs = x32 ? 4 : es;
   auto all = [&](int v) {
     bool ok = ((width | row | out_row) & (v - 1)) == 0;
-    const uintptr_t al = (uintptr_t)(v * es);
-    for (const void* q : {x, conv, conv_b, (const void*)hist, (const void*)out, mu, (const void*)shift, (const void*)last})
-      ok = ok && (reinterpret_cast<uintptr_t>(q) % al) == 0;
+    for (const void* q : {conv, conv_b, (const void*)out, mu}) ok = ok && (reinterpret_cast<uintptr_t>(q) % (v * es)) == 0;
+    for (const void* q : {x, (const void*)hist, (const void*)shift, (const void*)last}) ok = ok && (reinterpret_cast<uintptr_t>(q) % (v * xs)) == 0;
     return ok;
   };
   const int vec = all(8) && (int64_t)num_tokens * width >= (1 << 20) ? 8 : all(4) ? 4 : 1;
   cudaError_t e = cudaSuccess;
-  if (vec == 8) {
-    BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_token_conv<T, 8>(p, stream)));
-  } else if (vec == 4) {
-    BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_token_conv<T, 4>(p, stream)));
-  } else {
-    BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_token_conv<T, 1>(p, stream)));
-  }
+  auto go = [&](auto type, auto input) -> cudaError_t {
+    using T = decltype(type);
+    using X = decltype(input);
+    return vec == 8 ? launch_token_conv<T, X, 8>(p, stream) : vec == 4 ? launch_token_conv<T, X, 4>(p, stream) : launch_token_conv<T, X, 1>(p, stream);
+  };
+  BLITZ_DISPATCH_DTYPE3(dtype, (e = x32 ? go(T{}, float{}) : go(T{}, T{})));
   if (e != cudaSuccess || tok_indptr == nullptr || (taps < 2 && mixes == 0)) return (int)e;
   const dim3 grid((width + 255) / 256, rows);
-  BLITZ_DISPATCH_DTYPE3(dtype, (e = launch_pdl(conv_keep_kernel<T>, grid, dim3(256), 0, stream, p)));
+  BLITZ_DISPATCH_DTYPE3(x32 ? 2 : dtype, (e = launch_pdl(conv_keep_kernel<T>, grid, dim3(256), 0, stream, p)));
   return (int)e;
 }
 

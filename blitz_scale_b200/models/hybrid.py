@@ -163,8 +163,10 @@ class HybridRunner:
         wkv = [m for m in c.run_mixers() if m.kind == "wkv"]
         mixes = max([1 if c.mix_taps else 0] + [len(m.MIXES) for m in wkv])
         self._mixed = torch.empty(max_tokens * mixes * c.hidden, dtype=dt, device=dev) if mixes else None
+        # what the convolution reads is not rounded
+        self._unmixed = torch.empty(max_tokens, c.hidden, dtype=torch.float32, device=dev) if mixes else None
         if wkv:
-            self._last_h = torch.empty(max_batch, c.hidden, dtype=dt, device=dev)
+            self._last_h = torch.empty(max_batch, c.hidden, dtype=torch.float32, device=dev)
             self._rkvg = torch.empty(max_tokens * 4 * max(m.out_width for m in wkv), dtype=dt, device=dev)
             self._low = torch.empty(max_tokens * max(m.rank + 7 for m in wkv), dtype=torch.float32, device=dev)
         # (padding columns stay zero because nothing ever writes them)
@@ -234,7 +236,7 @@ class HybridRunner:
         conv = self._w(l, "mix_conv")
         if not m.is_prefill:
             return self._join(l, 1, T, out=out, tokens=ops.TokenState(conv, rc.mix_hist, mu, rc.shift), pos=m.pos, seq_slot=m.seq_slot)
-        h = self._join(l, 1, T)
+        h = self._join(l, 1, T, out=self._unmixed[:T])
         shift = dict(mu=mu, shift=rc.shift, last=self._last_h) if mu is not None else {}
         return ops.token_conv(h, conv, rc.mix_hist, out, m.pos, m.tok_indptr, m.seq_slot, residual=True, **shift)
 

@@ -642,12 +642,12 @@ class HybridConfig:
         return sum(per(m) * elem for m in self.run_parts() if m.kind in PAGED)
 
     def state_bytes_per_sequence(self, elem: int = 2) -> int:
-        n = elem * max(0, self.mix_taps - 1) * self.hidden * len(self.runs())
+        n = 4 * max(0, self.mix_taps - 1) * self.hidden * len(self.runs())
         for m in self.run_parts():
             if m.kind == "gla":
                 n += 4 * m.state_floats()
             elif m.kind == "wkv":
-                n += 4 * m.state_floats() + elem * m.hidden
+                n += 4 * (m.state_floats() + m.hidden)
             elif m.kind == "ssd":
                 n += 4 * m.state_floats() + elem * (m.taps - 1) * m.channels
             elif m.kind == "rglru":

@@ -559,7 +559,8 @@ class Pending(NamedTuple):
 
 class TokenState(NamedTuple):
     """What a causal convolution of a token's row reads beside it: ``conv`` [taps, width], the last inputs by slot ``hist`` [slots,
-    taps - 1, width], and for mixes with the row before it ``mu`` [mixes, width] and that row by slot, ``shift`` [slots, width]."""
+    taps - 1, width], and for mixes with the row before it ``mu`` [mixes, width] and that row by slot, ``shift`` [slots, width].  Both
+    histories are fp32."""
     conv: torch.Tensor
     hist: torch.Tensor
     mu: Optional[torch.Tensor] = None
@@ -571,26 +572,30 @@ def stream_rms(x: torch.Tensor, *, eps: float, n: Optional[int] = None, ids: Opt
                w: Optional[torch.Tensor] = None, w_offset: float = 0.0, out: Optional[torch.Tensor] = None, total: Optional[torch.Tensor] = None,
                write: bool = False, rows: Optional[torch.Tensor] = None, row_offset: int = 0, tokens: Optional[TokenState] = None,
                pos: Optional[torch.Tensor] = None, seq_slot: Optional[torch.Tensor] = None) -> None:
-    """`stream_mix` with an RMS norm: ``out`` receives u / sqrt(mean(u^2) + eps) * (w_offset + w), w one number or one per column.
+    """`stream_mix` with an RMS norm: ``out`` receives u / sqrt(mean(u^2) + eps) * (w_offset + w), w one number or one per column
+    (``out`` may be fp32 beside shorter weights).
     ``tokens`` (decode: a token per row, ``pos`` and ``seq_slot`` say which): out is that plus its causal convolution, or with mixes
     [n, mixes * hidden]; see `token_conv`, which does the same for rows of any length."""
     T, S, H = x.shape
     n = n if n is not None else (rows.numel() if rows is not None else T)
     assert x.dtype == torch.float32 and x.is_contiguous() and (out is None or (w is not None and out.is_contiguous()))
     assert total is None or (total.dtype == torch.float32 and total.is_contiguous())
-    ref = embed if embed is not None else out if out is not None else pending.y if pending is not None else read
+    ref = embed if embed is not None else w if w is not None else pending.y if pending is not None else read
     if ref is None:
         ref = torch.empty(0, dtype=torch.bfloat16)        # a plain sum of fp32 streams
+    h32 = out is not None and out.dtype != ref.dtype
     pd = pending if pending is not None else Pending(None, None, None)
     assert pd.y is None or (pd.y.stride(1) == 1 and pd.place is None)
+    assert not h32 or (out.dtype == torch.float32 and tokens is None)
     w0, w1 = pd.norms or (None, None)
     y1 = ctypes.c_void_p(pd.y.data_ptr() + H * pd.y.element_size()) if pd.norms else None
     ts = tokens if tokens is not None else TokenState(None, None)
     taps, mixes = (0 if ts.conv is None else ts.conv.shape[0]), (0 if ts.mu is None else ts.mu.shape[0])
+    assert all(t is None or (t.dtype == torch.float32 and t.is_contiguous()) for t in (ts.hist, ts.shift))
     assert tokens is None or (n == seq_slot.numel() and out is not None and out.numel() == n * max(1, mixes) * H)
     _check(lib().blitz_stream_rms(_p(ids), _p(embed), embed.shape[0] if embed is not None else 0, int(embed is not None), _p(x), _p(pd.y), y1,
                                   pd.y.stride(0) if pd.y is not None else H, _p(pd.bias), _p(w0), _p(w1), _p(pd.mix), _p(pd.out), _p(read),
-                                  _p(w), int(w is not None and w.numel() > 1), w_offset, eps, _p(rows), row_offset, _p(out), _p(total),
+                                  _p(w), int(w is not None and w.numel() > 1), w_offset, eps, _p(rows), row_offset, _p(out), int(h32), _p(total),
                                   int(write), _p(ts.conv), taps, _p(ts.hist), _p(ts.mu), mixes, _p(ts.shift), _p(pos), _p(seq_slot),
                                   0 if ts.hist is None else ts.hist.shape[0], n, H, S, _p(status_word(x.device)), _dt3(ref), _stream()),
            "blitz_stream_rms")
@@ -602,14 +607,15 @@ def token_conv(x: torch.Tensor, conv: torch.Tensor, hist: torch.Tensor, out: tor
     """Causal convolution of every column of ``x`` [T, width] over the rows of a step, with the history [slots, taps - 1, width] it
     reads and brings up to date: silu of it, or x plus it (``residual``).  ``mu`` [mixes, width]: out [T, mixes * width] are the
     mixes with the token before, which ``shift`` [slots, width] holds between steps (``last`` [rows, width]: scratch).
-    ``tok_indptr`` None: one token per row."""
+    ``tok_indptr`` None: one token per row.  x, hist, shift and last may be fp32 beside shorter weights and outputs."""
     slots, keep, width = hist.shape
+    assert all(t is None or t.dtype == x.dtype for t in (hist, shift, last)) and (x.dtype == out.dtype or x.dtype == torch.float32)
     mixes = 0 if mu is None else mu.shape[0]
     assert x.stride(1) == 1 and out.stride(1) == 1 and x.shape[1] == width and conv.shape == (keep + 1, width)
     assert conv.is_contiguous() and hist.is_contiguous() and out.shape[1] >= max(1, mixes) * width
-    _check(lib().blitz_token_conv(_p(x), x.stride(0), _p(conv), _p(bias), _p(hist), _p(out), out.stride(0), int(silu), int(residual), _p(mu),
+    _check(lib().blitz_token_conv(_p(x), x.stride(0), _p(conv), _p(bias), _p(hist), _p(out), out.stride(0), int(silu), int(residual), int(x.dtype != out.dtype), _p(mu),
                                   mixes, _p(shift), _p(last), _p(pos), _p(tok_indptr), _p(seq_slot), x.shape[0], seq_slot.numel(), width,
-                                  keep + 1, slots, _p(status_word(x.device)), _dt3(x), _stream()), "blitz_token_conv")
+                                  keep + 1, slots, _p(status_word(x.device)), _dt3(out), _stream()), "blitz_token_conv")
     return out
 
 

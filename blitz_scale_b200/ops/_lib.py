@@ -122,9 +122,9 @@ def _declare(L: ctypes.CDLL) -> None:
                               c_p])
     sig("blitz_rglru_scan", [c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_i, c_i,
                              c_i, c_i, c_i, c_i, c_p, c_i, c_p])
-    sig("blitz_stream_rms", [c_p, c_p, c_i, c_i, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_f, c_f, c_p, c_i, c_p,
+    sig("blitz_stream_rms", [c_p, c_p, c_i, c_i, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_f, c_f, c_p, c_i, c_p, c_i,
                              c_p, c_i, c_p, c_i, c_p, c_p, c_i, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_p, c_i, c_p])
-    sig("blitz_token_conv", [c_p, c_i64, c_p, c_p, c_p, c_p, c_i64, c_i, c_i, c_p, c_i, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i,
+    sig("blitz_token_conv", [c_p, c_i64, c_p, c_p, c_p, c_p, c_i64, c_i, c_i, c_i, c_p, c_i, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i,
                              c_p, c_i, c_p])
     sig("blitz_wkv_recurrent", [c_p, c_p, c_p, c_p, c_i64, c_p, c_i64, c_p, c_p, c_p, c_p, c_p, c_p, c_i64, c_p, c_p, c_p, c_i, c_i, c_i,
                                 c_i, c_i, c_i, c_f, c_i, c_p, c_i, c_p])

@@ -29,8 +29,8 @@ class RunCache:
     kv: Optional[Union[torch.Tensor, KVPair, LatentKV]] = None
     state: Optional[torch.Tensor] = None   # fp32: [slots, heads, dim, vdim] (keys or state by values) or [slots, width]
     hist: Optional[torch.Tensor] = None    # last inputs of a short convolution: [slots, taps - 1, width]
-    mix_hist: Optional[torch.Tensor] = None  # the same of the convolution of a mixer's input
-    shift: Optional[torch.Tensor] = None   # a mixer's last input: [slots, width]
+    mix_hist: Optional[torch.Tensor] = None  # the same of the convolution of a mixer's input, fp32
+    shift: Optional[torch.Tensor] = None   # a mixer's last input: [slots, width], fp32
 
 
 class HybridCache:
@@ -42,7 +42,7 @@ class HybridCache:
             rc = RunCache()
             self.runs.append(rc)
             if cfg.mix_taps:
-                rc.mix_hist = zeros(num_slots, cfg.mix_taps - 1, cfg.hidden)
+                rc.mix_hist = torch.zeros(num_slots, cfg.mix_taps - 1, cfg.hidden, device=device)
             for m in mixer_parts(m):
                 if m.kind == "attention" and source != r:
                     rc.kv = self.runs[source].kv
@@ -55,7 +55,7 @@ class HybridCache:
                 elif m.kind in ("gla", "wkv"):
                     rc.state = torch.zeros(num_slots, m.heads, m.dim, m.vdim, device=device)
                     if m.kind == "wkv":
-                        rc.shift = zeros(num_slots, m.hidden)
+                        rc.shift = torch.zeros(num_slots, m.hidden, device=device)
                 elif m.kind == "ssd":
                     rc.state = torch.zeros(num_slots, m.heads, m.state, m.vdim, device=device)
                     rc.hist = zeros(num_slots, m.taps - 1, m.channels)

@@ -72,6 +72,9 @@ def test_streams(ops, S, H, dt):
                 ops.stream_rms(xd, **kw, pending=pending, read=dev(in_w), w=dev(weight), w_offset=off, out=h, write=pending is not None)
                 assert _rel(h, norm(plain.streams_in(xs, d(in_w)))) < tol, (name, fresh)
                 assert _rel(xd.transpose(0, 1), xs if pending is not None else d(x).transpose(0, 1)) < 1e-6
+                h32 = torch.empty(T, H, device=DEV)
+                ops.stream_rms(x.to(DEV), **kw, pending=pending, read=dev(in_w), w=dev(weight), w_offset=off, out=h32)
+                assert _rel(h32, norm(plain.streams_in(xs, d(in_w)))) < 3e-6
                 # some rows only, nothing kept, the plain sum
                 at = torch.tensor([5, 2, 9, 2])
                 xd, h, tot = x.to(DEV), torch.empty(4, H, dtype=dt, device=DEV), torch.empty(4, H, device=DEV)
@@ -100,15 +103,14 @@ def test_convolved_input_of_decoded_tokens(ops, taps, mixes, H, dt):
     n, slots, lens = 3, 5, (20, 9, 14)
     conv, mu, w = (0.6 * r(taps, H)).to(dt), (0.5 + 0.4 * r(mixes, H)).to(dt) if mixes else None, r(1).to(dt)
     one = torch.ones(1, dtype=dt, device=DEV)
-    state = ops.TokenState(dev(conv), torch.full((slots, taps - 1, H), 50.0, dtype=dt, device=DEV), dev(mu) if mixes else None,
-                           torch.full((slots, H), 50.0, dtype=dt, device=DEV) if mixes else None)
+    state = ops.TokenState(dev(conv), torch.full((slots, taps - 1, H), 50.0, device=DEV), dev(mu) if mixes else None,
+                           torch.full((slots, H), 50.0, device=DEV) if mixes else None)
     x = [r(k, 1, H) for k in lens]
-    rounded = lambda t: t.to(dt).double()
     want = []
     for s in x:
-        h = rounded(plain.rms(d(s[:, 0]), 0.01) * d(w))
+        h = plain.rms(d(s[:, 0]), 0.01) * d(w)
         c = h + plain.causal_conv(h, d(conv).T)
-        want.append(_mixes(rounded(c), d(mu)) if mixes else c)
+        want.append(_mixes(c, d(mu)) if mixes else c)
     slot_of, at, got = (3, 0, 4), [0] * n, [[] for _ in lens]
     k = 0
     while any(a < m for a, m in zip(at, lens)):
@@ -123,7 +125,7 @@ def test_convolved_input_of_decoded_tokens(ops, taps, mixes, H, dt):
         k += 1
     ops.check_status()
     for a, b in zip(got, want):
-        assert _worst(torch.stack(a), b) < (3e-6 if dt == F32 else 8e-3)
+        assert _worst(torch.stack(a), b) < (3e-6 if dt == F32 else 5e-3)
     if taps > 1:
         assert bool((state.hist[[1, 2]] == 50.0).all())
 
@@ -131,34 +133,34 @@ def test_convolved_input_of_decoded_tokens(ops, taps, mixes, H, dt):
 # ------------------------------------------------------------------------------------------------ short convolutions
 @pytest.mark.parametrize("W", [5, 64, 1036, 8200])
 @pytest.mark.parametrize("taps,mixes", [(1, 0), (3, 0), (4, 0), (4, 5), (6, 2), (1, 5), (2, 1)])
-@pytest.mark.parametrize("dt", [BF, F32])
-def test_token_convolution(ops, W, taps, mixes, dt):
+@pytest.mark.parametrize("dt,xt", [(BF, BF), (BF, F32), (F32, F32)])
+def test_token_convolution(ops, W, taps, mixes, dt, xt):
     """Portions of many sizes of several sequences side by side, on slots that hold other sequences' remains."""
     g = torch.Generator().manual_seed(W + taps)
     r = lambda *s: torch.randn(*s, generator=g)
     conv, bias = (r(taps, W) * taps ** -0.5).to(dt), (0.3 * r(W)).to(dt)
     mu = (0.5 + 0.4 * r(mixes, W)).to(dt) if mixes else None
     cuts = {0: [1, 2, 40, 1, 3, 53], 1: [2, 2, 1, 1, 2, 1], 2: [70, 1, 0, 1, 1, 30]}
-    x = {i: r(sum(c), W).to(dt) for i, c in cuts.items()}
+    x = {i: r(sum(c), W).to(xt) for i, c in cuts.items()}
     kind = dict(residual=True) if mixes else dict(bias=dev(bias), silu=True) if taps % 2 == 0 else dict(bias=dev(bias))
 
     def expect(s):
         c = plain.causal_conv(d(s), d(conv).T)
         if mixes:
-            return _mixes((d(s) + c).to(dt).double(), d(mu))
+            return _mixes(d(s) + c, d(mu))
         c = c + d(bias)
         return F.silu(c) if taps % 2 == 0 else c
-    hist = torch.full((5, taps - 1, W), 30.0, dtype=dt, device=DEV)
-    shift = torch.full((5, W), 30.0, dtype=dt, device=DEV) if mixes else None
+    hist = torch.full((5, taps - 1, W), 30.0, dtype=xt, device=DEV)
+    shift = torch.full((5, W), 30.0, dtype=xt, device=DEV) if mixes else None
     got, at, slot = {i: [] for i in cuts}, {i: 0 for i in cuts}, {0: 4, 1: 2, 2: 0}
     for k in range(6):
         live = [i for i in cuts if cuts[i][k]]
         n = [cuts[i][k] for i in live]
-        buf = torch.zeros(sum(n), W + 8, dtype=dt, device=DEV)       # a column range of a wider buffer
+        buf = torch.zeros(sum(n), W + 8, dtype=xt, device=DEV)       # a column range of a wider buffer
         rows = buf[:, :W]
         rows.copy_(torch.cat([x[i][at[i]:at[i] + c] for i, c in zip(live, n)]))
         out = torch.full((sum(n), max(1, mixes) * W), 9.0, dtype=dt, device=DEV)
-        more = dict(mu=dev(mu), shift=shift, last=torch.empty(len(n), W, dtype=dt, device=DEV)) if mixes else {}
+        more = dict(mu=dev(mu), shift=shift, last=torch.empty(len(n), W, dtype=xt, device=DEV)) if mixes else {}
         pos = _i32([at[i] + t for i, c in zip(live, n) for t in range(c)])
         single = not mixes and all(c == 1 for c in n)
         ops.token_conv(rows, dev(conv), hist, out, pos, None if single else _i32([sum(n[:j]) for j in range(len(n) + 1)]),
